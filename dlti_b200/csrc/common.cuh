@@ -152,7 +152,7 @@ __device__ __forceinline__ void mbar_wait(uint32_t bar, uint32_t parity) {
 }
 
 // ---------------------------------------------------------------------------
-// TMA (cp.async.bulk.tensor) — SASS: UTMALDG / UTMASTG
+// TMA (cp.async.bulk.tensor)
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ void tma_prefetch_desc(const CUtensorMap* m) {
   asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(m)) : "memory");
@@ -191,7 +191,7 @@ __device__ __forceinline__ void tma_store_wait_read() {
 __device__ __forceinline__ void fence_proxy_async_smem() {
   asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
 }
-// 1D bulk copy global -> shared (SASS: UBLKCP). bytes % 16 == 0.
+// 1D bulk copy global -> shared. bytes % 16 == 0.
 __device__ __forceinline__ void bulk_load_1d(uint32_t dst_smem, const void* src, uint32_t bytes,
                                              uint32_t bar) {
   asm volatile(
@@ -209,7 +209,7 @@ __device__ __forceinline__ void bulk_store_1d(void* dst, uint32_t src_smem, uint
 }
 
 // ---------------------------------------------------------------------------
-// tcgen05 / TMEM — SASS: UTCHMMA, LDTM, STTM, UTCBAR
+// tcgen05 / TMEM
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ void tmem_alloc(uint32_t dst_smem_addr, uint32_t ncols) {
   asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(
@@ -321,8 +321,8 @@ __device__ __forceinline__ uint64_t umma_smem_desc(uint32_t smem_addr, uint32_t 
 // preparing each one. Descriptors are split into a precomputed (lo, hi) pair and the per-MMA work is one
 // 32-bit add of a compile-time offset. Equally important: run the issue loop WARP-UNIFORMLY (whole warp,
 // uniform operands, warp index / TMEM base made uniform with __shfl_sync) and predicate only the
-// tcgen05 instructions on elect_one_sync(): issuing from inside `if (lane == 0)` makes the compiler wrap
-// every UTCHMMA in an ELECT / R2UR / BRA.U.ANY waterfall (traced: ~60 clk per MMA).
+// tcgen05 instructions on elect_one_sync(): issuing from inside `if (lane == 0)` costs ~60 clk per MMA
+// (clock64 timeline of the issuing warp).
 struct DescLoHi {
   uint32_t lo, hi;
   __device__ __forceinline__ uint64_t at(uint32_t byte_off) const {

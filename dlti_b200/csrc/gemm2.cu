@@ -320,8 +320,8 @@ gemm2_kernel(const Gemm2Params p, const GatherJob gj, const WaitSpec ws_, const 
 
   if (warp == 0) {
     // ===================== A producer (both CTAs): this CTA's 128 rows of A =====================
-    // One elected thread; the loop body is kept minimal — a k-block lasts ~512 clk on the tensor cores and every
-    // UTMALDG costs the issuing thread on the order of 100 clk, which is why A and B have separate producer
+    // One elected thread; the loop body is kept minimal — a k-block lasts ~512 clk on the tensor cores and
+    // every TMA tensor load costs the issuing thread on the order of 100 clk, which is why A and B have separate producer
     // threads (with one thread the input-gradient form, two B boxes per stage, was issue-bound: 1,180 vs cuBLAS
     // 1,296 TFLOP/s sustained).
     bool a_ready = true;          // K11: every unit of A has already landed
