@@ -135,15 +135,20 @@ _ALIASES = {
 }
 
 
-def resolve_config(name_or_path: str) -> LlamaConfig:
-    """Preset name, HF hub id of a known Llama-2 size, or a directory with config.json."""
+def resolve_config(name_or_path: str):
+    """Preset name, HF hub id of a known Llama-2 size, or a directory with config.json (the model family is chosen by
+    its architecture key, models/registry.py)."""
     import copy
 
-    if name_or_path in PRESETS:
-        return copy.deepcopy(PRESETS[name_or_path])
+    from . import registry
+
     if name_or_path in _ALIASES:
         return copy.deepcopy(PRESETS[_ALIASES[name_or_path]])
+    cfg = registry.preset(name_or_path)
+    if cfg is not None:
+        return cfg
     p = Path(name_or_path)
     if (p / "config.json").exists():
-        return LlamaConfig.load(p)
-    raise ValueError(f"unknown model config '{name_or_path}' (presets: {sorted(PRESETS)})")
+        return registry.config_from_dir(p)
+    known = sorted(n for f in registry.FAMILIES.values() for n in f.presets)
+    raise ValueError(f"unknown model config '{name_or_path}' (presets: {known})")

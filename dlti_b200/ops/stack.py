@@ -1,0 +1,341 @@
+"""Ops of the layer-stack models (models/stack.py): kernels in csrc/stack.cu, recurrent.cu, attention_paged.cu and
+gemm_f32.cu; PyTorch restatements for CPU tensors, as in the other op modules.
+
+Activations are [rows, n] views whose row pitch is a multiple of 8 elements (`act`). The residual stream is fp32.
+Ops with `acc=True` consume the fp32 accumulator of gemm_skinny_acc and leave it zero."""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass
+
+import torch
+
+from ..models.stack import round8
+from . import _debug, _lib
+from .gemm import gemm, gemm_skinny
+
+_V, _I, _L, _F = C.c_void_p, C.c_int, C.c_longlong, C.c_float
+_p = _lib.ptr
+
+
+def act(rows: int, n: int, dtype, device) -> torch.Tensor:
+    return torch.empty((rows, round8(n)), dtype=dtype, device=device)[:, :n]
+
+
+def linear(a: torch.Tensor, w: torch.Tensor, out_dtype=None) -> torch.Tensor:
+    """a [T, K] · w [N, K]^T -> [T, N]; N is a multiple of 8 (stack weights are padded)."""
+    if not _lib.use_native(a):
+        return (a.float() @ w.float().t()).to(out_dtype or a.dtype)
+    if a.dtype == torch.float32:
+        M, K = a.shape
+        N = w.shape[0]
+        out = torch.empty((M, N), dtype=torch.float32, device=a.device)
+        f = _lib.fn("dlti_gemm_f32", [_V, _V, _V, _I, _I, _I, _L, _L, _L, _V])
+        _lib.check(f(_p(a), _p(w), _p(out), M, N, K, a.stride(0), w.stride(0), out.stride(0), _lib.stream_ptr()), "gemm_f32")
+        return out
+    if a.shape[0] <= 256 and out_dtype in (None, a.dtype):
+        return gemm_skinny(a, w)
+    return gemm(a, w, out_dtype=out_dtype)
+
+
+# ---- rows --------------------------------------------------------------------------------------------------
+def embed_rows(ids, table):
+    """Token rows as the fp32 residual stream [T, d] and as the first GEMM's input (the same tensor in fp32)."""
+    _debug.check_range("embed_rows", "ids", ids, 0, table.shape[0])
+    T, d = ids.numel(), table.shape[1]
+    if not _lib.use_native(table):
+        x = table[ids].float()
+        return x, (x if table.dtype == torch.float32 else table[ids])
+    x = torch.empty((T, d), dtype=torch.float32, device=table.device)
+    xa = None if table.dtype == torch.float32 else act(T, d, table.dtype, table.device)
+    f = _lib.fn("dlti_embed_rows", [_V, _V, _V, _V, _L, _L, _I, _L, _I, _V])
+    _lib.check(f(_p(ids), _p(table), _p(x), _p(xa), 0 if xa is None else xa.stride(0), T, d, table.shape[0],
+                 _lib.dtype_code(table.dtype), _lib.stream_ptr()), "embed_rows")
+    return x, (x if xa is None else xa)
+
+
+def _rms(x, eps):
+    return x / torch.sqrt(x.square().mean(-1, keepdim=True) + eps)
+
+
+def post_norm_add_(y, x, w, eps, one_plus, dtype, acc=False, want=True):
+    """x += norm(y) * w (1 + w with one_plus), in place on the fp32 residual [T, d]; y has at least d columns. Returns
+    the new residual as the next GEMM's input (x itself in fp32; None unless want)."""
+    T, d = x.shape
+    if not _lib.use_native(x):
+        x += _rms(y[:, :d].float(), eps) * (w + 1 if one_plus else w)
+        return x if dtype == torch.float32 else x.to(dtype)
+    xa = None if dtype == torch.float32 or not want else act(T, d, dtype, x.device)
+    f = _lib.fn("dlti_post_norm_add", [_V, _L, _V, _V, _V, _L, _L, _I, _F, _I, _I, _I, _V])
+    _lib.check(f(_p(y), y.stride(0), _p(x), _p(w), _p(xa), 0 if xa is None else xa.stride(0), T, d, float(eps), int(one_plus),
+                 int(acc), _lib.dtype_code(dtype), _lib.stream_ptr()), "post_norm_add")
+    return x if dtype == torch.float32 else xa
+
+
+def rms_rows(x, idx, w, eps, one_plus, dtype):
+    """norm(x[idx]) * w in the compute dtype; idx None = all rows."""
+    if not _lib.use_native(x):
+        xs = x if idx is None else x[idx]
+        return (_rms(xs, eps) * (w + 1 if one_plus else w)).to(dtype)
+    rows = x.shape[0] if idx is None else idx.numel()
+    out = act(rows, x.shape[1], dtype, x.device)
+    f = _lib.fn("dlti_rms_rows", [_V, _V, _V, _V, _L, _L, _I, _F, _I, _I, _V])
+    _lib.check(f(_p(x), _p(idx), _p(w), _p(out), out.stride(0), rows, x.shape[1], float(eps), int(one_plus),
+                 _lib.dtype_code(dtype), _lib.stream_ptr()), "rms_rows")
+    return out
+
+
+def relu2(u, ff, dtype, acc=False):
+    """Square of relu of the first ff columns."""
+    if not _lib.use_native(u):
+        return torch.relu(u[:, :ff].float()).square().to(dtype)
+    T = u.shape[0]
+    h = act(T, ff, dtype, u.device)
+    f = _lib.fn("dlti_relu2", [_V, _L, _V, _L, _L, _I, _I, _I, _V])
+    _lib.check(f(_p(u), u.stride(0), _p(h), h.stride(0), T, ff, int(acc), _lib.dtype_code(dtype), _lib.stream_ptr()), "relu2")
+    return h
+
+
+def gated_norm(y, gate, w, eps, groups, gate_first, acc=False):
+    """gate_first: norm(y * silu(gate)) * w; else norm(y) * w * sigmoid(gate). The norm runs over `groups` equal parts of
+    the row. gate: [T, >= n] view (a section of a projection; of its accumulator with acc)."""
+    T, n = y.shape
+    if not _lib.use_native(y):
+        g = gate[:, :n].float()
+        v = y.float() * torch.nn.functional.silu(g) if gate_first else y.float()
+        v = _rms(v.reshape(T, groups, -1), eps).reshape(T, n) * w
+        return (v if gate_first else v * torch.sigmoid(g)).to(y.dtype)
+    out = act(T, n, y.dtype, y.device)
+    f = _lib.fn("dlti_gated_norm", [_V, _L, _V, _L, _V, _V, _L, _L, _I, _I, _F, _I, _I, _I, _V])
+    _lib.check(f(_p(y), y.stride(0), _p(gate), gate.stride(0), _p(w), _p(out), out.stride(0), T, n, groups, float(eps),
+                 int(gate_first), int(acc), _lib.dtype_code(y.dtype), _lib.stream_ptr()), "gated_norm")
+    return out
+
+
+# ---- attention ---------------------------------------------------------------------------------------------
+_tables: dict = {}
+
+
+def rope_tables(max_pos: int, dims: int, base: float, device):
+    """fp32 cos / sin [max_pos, dims/2] of position * base^(-2i/dims), the angle taken in double precision."""
+    key = (max_pos, dims, base, str(device))
+    t = _tables.get(key)
+    if t is None:
+        f = base ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
+        a = torch.arange(max_pos, dtype=torch.float64)[:, None] * f[None, :]
+        t = _tables[key] = (a.cos().float().to(device), a.sin().float().to(device))
+    return t
+
+
+@dataclass
+class Rows:
+    """Where a step's token rows belong: nd decode rows (sequence s = row s), then prompt rows; sequence nd + i owns rows
+    nd + cu[i] ... nd + cu[i + 1]. ctx[s] = tokens of sequence s after the step, pos[t] / seq[t] = position and sequence
+    of row t, slots[t] = its cache slot (-1: none), state[s] = recurrent-state slot (-1: none)."""
+    pos: torch.Tensor
+    seq: torch.Tensor
+    slots: torch.Tensor
+    ctx: torch.Tensor
+    cu: torch.Tensor | None
+    tables: torch.Tensor
+    state: torch.Tensor
+    nd: int
+    max_seqlen: int
+    max_ctx: int
+
+    @property
+    def nseq(self) -> int:
+        return self.nd + (0 if self.cu is None else self.cu.numel() - 1)
+
+    def bounds(self, s: int) -> tuple[int, int, int]:
+        """(first row, rows, first position) of sequence s (host side; CPU restatements only)."""
+        if s < self.nd:
+            r0, n = s, 1
+        else:
+            r0 = self.nd + int(self.cu[s - self.nd])
+            n = int(self.cu[s - self.nd + 1]) - int(self.cu[s - self.nd])
+        return r0, n, int(self.ctx[s]) - n
+
+
+def qk_norm_rope_cache(proj, sec, m, q_norm, k_norm, eps, rows: Rows, tabs, kc, vc, dtype, packed=False, acc=False):
+    """Merged projection rows -> rotated queries (each head normalised first when norms are given), keys and values in
+    the paged cache at rows.slots, and the sigmoid of the head gates [T, H] (None without gates).
+    packed: also return [q heads | k heads | v heads] rows, the layout of the varlen prefill kernel; keys and values of a
+    layer without own ones are then copied from the cache."""
+    T, H, G = proj.shape[0], m.heads, m.kv_heads
+    own = "k" in sec
+    rot = m.rope.dims if m.rope is not None else 0
+    _debug.check_range("qk_norm_rope_cache", "slots", rows.slots, 0, kc.shape[0] * kc.shape[1], allow=-1)
+    if not _lib.use_native(proj):
+        ok = rows.slots >= 0
+        kf, vf = kc.view(-1, G, kc.shape[3]), vc.view(-1, G, vc.shape[3])
+
+        def prep(name, heads, nw):
+            x = proj[:, sec[name]:sec[name] + heads * m.dim].float().reshape(T, heads, m.dim)
+            if nw is not None:
+                x = _rms(x, eps) * nw
+            if rot:
+                c, s = (t[rows.pos.long()][:, None, :] for t in tabs)
+                h = rot // 2
+                a, b = (x[..., 0:rot:2], x[..., 1:rot:2]) if m.rope.interleaved else (x[..., :h], x[..., h:rot])
+                u, v = a * c - b * s, b * c + a * s
+                r = torch.stack([u, v], -1).flatten(-2) if m.rope.interleaved else torch.cat([u, v], -1)
+                x = torch.cat([r, x[..., rot:]], -1)
+            return x.to(dtype)
+
+        q = prep("q", H, q_norm)
+        if own:
+            k = prep("k", G, k_norm)
+            v = proj[:, sec["v"]:sec["v"] + G * m.vdim].reshape(T, G, m.vdim).to(dtype)
+            kf[rows.slots[ok], :, :m.dim] = k[ok]
+            vf[rows.slots[ok], :, :m.vdim] = v[ok]
+        gate = torch.sigmoid(proj[:, sec["g"]:sec["g"] + H].float()) if "g" in sec else None
+        if packed:
+            k, v = kf[rows.slots.clamp_min(0)][..., :m.dim], vf[rows.slots.clamp_min(0)][..., :m.vdim]
+            return torch.cat([q.reshape(T, -1), k.reshape(T, -1), v.reshape(T, -1)], 1), gate
+        return q.reshape(T, -1), gate
+    dev = proj.device
+    gate = torch.empty((T, H), dtype=torch.float32, device=dev) if "g" in sec else None
+    if packed:
+        assert m.dim == m.vdim
+        q = torch.empty((T, (H + 2 * G) * m.dim), dtype=dtype, device=dev)
+        hd, es = m.dim, q.element_size()
+        kp, vp = q.data_ptr() + H * hd * es, q.data_ptr() + (H + G) * hd * es
+    else:
+        hd = round8(m.dim)
+        q = torch.empty((T, H * hd), dtype=dtype, device=dev)
+        kp = vp = 0
+    f = _lib.fn("dlti_qk_norm_rope_cache", [_V, _L, _I, _I, _I, _I, _V, _V, _F, _V, _V, _V, _I, _I, _V, _V, _V, _I, _I, _V, _L, _I, _V,
+                                            _V, _V, _L, _I, _I, _I, _I, _I, _I, _V])
+    _lib.check(f(_p(proj), proj.stride(0), sec["q"], sec["k"] if own else -1, sec["v"] if own else -1, sec["g"] if "g" in sec else -1,
+                 _p(q_norm), _p(k_norm), float(eps), _p(rows.pos), _p(tabs[0]) if rot else None, _p(tabs[1]) if rot else None, rot,
+                 int(m.rope.interleaved) if rot else 1, _p(rows.slots), _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(q), q.stride(0), hd,
+                 kp, vp, _p(gate), T, H, G, m.dim, m.vdim, int(acc), _lib.dtype_code(dtype), _lib.stream_ptr()), "qk_norm_rope_cache")
+    return q, gate
+
+
+def paged_attention_ref(q, m, rows: Rows, kc, vc, gate):
+    """Every row against the cached keys of its sequence that it may see."""
+    T, H, G = q.shape[0], m.heads, m.kv_heads
+    bs, hd = kc.shape[1], q.shape[1] // H
+    kf, vf = kc.view(-1, G, kc.shape[3]).float(), vc.view(-1, G, vc.shape[3]).float()
+    out = torch.zeros(T, H, m.vdim)
+    for t in range(T):
+        s, p = int(rows.seq[t]), int(rows.pos[t])
+        j = torch.arange(p // m.chunk * m.chunk if m.chunk else 0, min(p + 1, int(rows.ctx[s])))
+        if not len(j):
+            continue
+        sl = rows.tables[s, j // bs].long() * bs + j % bs
+        k = kf[sl][..., :m.dim].repeat_interleave(H // G, 1)
+        v = vf[sl][..., :m.vdim].repeat_interleave(H // G, 1)
+        qq = q[t].float().view(H, hd)[:, :m.dim]
+        w = torch.softmax(torch.einsum("hd,jhd->hj", qq, k) * m.scale, -1)
+        out[t] = torch.einsum("hj,jhd->hd", w, v)
+    if gate is not None:
+        out *= gate[:, :, None]
+    return out.reshape(T, -1).to(q.dtype)
+
+
+def attn_rows(q, m, rows: Rows, kc, vc, gate, out):
+    """fp32-arithmetic attention of the rows of q, one warp per (row, head)."""
+    hd = q.shape[1] // m.heads
+    f = _lib.fn("dlti_attn_rows", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _V, _I, _I, _I, _I, _I, _F, _V, _V, _L, _L, _I, _V])
+    _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], kc.shape[1],
+                 _p(rows.ctx), _p(rows.seq), _p(rows.pos), m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.scale, _p(gate), _p(out),
+                 out.stride(0), q.shape[0], _lib.dtype_code(q.dtype), _lib.stream_ptr()), "attn_rows")
+    return out
+
+
+def paged_attention(q, m, rows: Rows, kc, vc, gate):
+    """Attention of every row of a step over the paged cache -> [T, heads * vdim], head outputs times `gate` [T, H]."""
+    if not _lib.use_native(q):
+        return paged_attention_ref(q, m, rows, kc, vc, gate)
+    _debug.check_paged("paged_attention", rows.tables, rows.ctx, kc.shape[0], kc.shape[1])
+    out = act(q.shape[0], m.heads * m.vdim, q.dtype, q.device)
+    return attn_rows(q, m, rows, kc, vc, gate, out)
+
+
+# ---- recurrences -------------------------------------------------------------------------------------------
+def short_conv(proj, col, C_, w, b, state, rows: Rows, dtype, acc=False, width=0):
+    """silu of the causal convolution of channels [col, col + C_) of the projection rows; w [taps, >= C_] tap-major,
+    state [slots, taps - 1, C_] = inputs of earlier steps (read only; linear_scan's tail job renews it). Returns (out
+    [T, C_], proj): with acc (decode rows only) proj is the projection rounded to the compute dtype, else as given."""
+    T, taps = proj.shape[0], w.shape[0]
+    if not _lib.use_native(proj):
+        out = torch.zeros(T, C_)
+        for s in range(rows.nseq):
+            r0, n, start = rows.bounds(s)
+            x = proj[r0:r0 + n, col:col + C_].float()
+            slot = int(rows.state[s])
+            h = state[slot].float() if start > 0 and slot >= 0 else torch.zeros(taps - 1, C_)
+            x = torch.cat([h, x])
+            out[r0:r0 + n] = b[:C_] + sum(w[k, :C_] * x[k:k + n] for k in range(taps))
+        return torch.nn.functional.silu(out).to(dtype), proj
+    out = act(T, C_, dtype, proj.device)
+    raw = act(T, width, dtype, proj.device) if acc else None
+    f = _lib.fn("dlti_short_conv", [_V, _L, _I, _I, _I, _V, _V, _I, _V, _V, _V, _V, _V, _I, _V, _L, _V, _L, _I, _L, _I, _I, _V])
+    _lib.check(f(_p(proj), proj.stride(0), col, C_, taps, _p(w), _p(b), w.stride(0), _p(state), _p(rows.state), _p(rows.seq),
+                 _p(rows.ctx), _p(rows.cu), rows.nd, _p(out), out.stride(0), _p(raw), 0 if raw is None else raw.stride(0), width, T,
+                 int(acc), _lib.dtype_code(dtype), _lib.stream_ptr()), "short_conv")
+    return out, (raw if acc else proj)
+
+
+@dataclass
+class Decay:
+    """Decay and step size of a recurrence: a constant factor per head (const), or per token from raw step sizes dt
+    (softplus(dt + bias), decay exp(-exp(A_log) * step))."""
+    const: torch.Tensor | None = None
+    dt: torch.Tensor | None = None
+    dt_bias: torch.Tensor | None = None
+    A_log: torch.Tensor | None = None
+    D: torch.Tensor | None = None
+
+
+def linear_scan_ref(q, k, v, decay: Decay, state, rows: Rows, heads, groups, N, P, silu, conv_src, conv_col, conv_state):
+    T, dtype = q.shape[0], v.dtype
+    f = (lambda x: torch.nn.functional.silu(x.float()).to(dtype).float()) if silu else (lambda x: x.float())
+    rep = heads // groups
+    qf, kf = (f(x).reshape(T, groups, N).repeat_interleave(rep, 1) for x in (q, k))
+    vf = f(v).reshape(T, heads, P)
+    if decay.const is not None:
+        st, a = torch.ones(T, heads), decay.const.expand(T, heads)
+    else:
+        st = torch.nn.functional.softplus(decay.dt.float() + decay.dt_bias, threshold=1e9)
+        a = torch.exp(-torch.exp(decay.A_log) * st)
+    out = torch.zeros(T, heads, P)
+    for s in range(rows.nseq):
+        r0, n, start = rows.bounds(s)
+        slot = int(rows.state[s])
+        S = state[slot].clone() if start > 0 and slot >= 0 else torch.zeros(heads, N, P)
+        for t in range(r0, r0 + n):
+            S = a[t][:, None, None] * S + kf[t][:, :, None] * (st[t][:, None] * vf[t])[:, None, :]
+            out[t] = (qf[t][:, :, None] * S).sum(1)
+        if slot >= 0:
+            state[slot] = S
+            if conv_state is not None:
+                rest = conv_state.shape[1]
+                h = conv_state[slot] if start > 0 else torch.zeros_like(conv_state[slot])
+                x = torch.cat([h, conv_src[r0:r0 + n, conv_col:conv_col + conv_state.shape[2]].to(h.dtype)])
+                conv_state[slot] = x[x.shape[0] - rest:].clone()
+    if decay.D is not None:
+        out += decay.D[:, None] * vf
+    return out.reshape(T, -1).to(dtype)
+
+
+def linear_scan(q, k, v, decay: Decay, state, rows: Rows, heads, groups, N, P, silu=False, conv_src=None, conv_col=0, conv_state=None):
+    """S <- a S + k (step v)^T, o = S^T q (+ D v) over the rows of every sequence; q, k [T, groups * N] views, v [T,
+    heads * P], state [slots, heads, N, P] fp32 updated in place. silu: applied to q, k, v on load. conv_state: renewed
+    from the rows of conv_src (see short_conv)."""
+    if not _lib.use_native(q):
+        return linear_scan_ref(q, k, v, decay, state, rows, heads, groups, N, P, silu, conv_src, conv_col, conv_state)
+    out = act(q.shape[0], heads * P, v.dtype, q.device)
+    f = _lib.fn("dlti_linear_scan", [_V, _L, _V, _L, _V, _L, _I, _I, _V, _V, _L, _V, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _V,
+                                     _L, _V, _L, _I, _I, _I, _V, _I, _V])
+    dt = decay.dt
+    _lib.check(f(_p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), heads // groups, int(silu), _p(decay.const), _p(dt),
+                 0 if dt is None else dt.stride(0), _p(decay.dt_bias), _p(decay.A_log), _p(decay.D), _p(state), _p(rows.state),
+                 _p(rows.ctx), _p(rows.cu), rows.nd, 0, rows.nseq, heads, N, P, _p(out), out.stride(0), _p(conv_src),
+                 0 if conv_src is None else conv_src.stride(0), conv_col, 0 if conv_state is None else conv_state.shape[1],
+                 0 if conv_state is None else conv_state.shape[2], _p(conv_state), _lib.dtype_code(v.dtype), _lib.stream_ptr()),
+               "linear_scan")
+    return out

@@ -20,8 +20,9 @@ import torch
 
 from ..models.config import LlamaConfig
 from ..ops import serving as S
-from .kv_cache import BlockManager, KVCache
-from .model_runner import ModelRunner, TPContext, TPWeights
+from ..models.registry import family_of
+from .kv_cache import BlockManager, KVCache, SlotManager, StateCache
+from .model_runner import TPContext, TPWeights
 from .params import Request, SamplingParams, StepOutput
 from .scheduler import Batch, Scheduler
 from .tokenizer import IncrementalDetokenizer
@@ -35,21 +36,29 @@ class StepLayout:
     packed prompts; B = nd + npf rows are sampled; block tables are [nd, mb]; src[t] >= 0 means "the input
     token of row t is the token sampled at row src[t] of the previous step" (it is still on the device).
     64-bit sections first, then the 32-bit ones (each padded to a whole word); the tables come last so that
-    a prefix copy carries everything but unused table rows."""
-    _I64 = ("ids", "slots", "last", "seeds", "pslots", "pdst", "csrc")
-    _I32 = ("pos", "src", "ctx", "cu", "ecu", "topk", "temp", "topp", "tables")
+    a prefix copy carries everything but unused table rows.
 
-    def __init__(self, T: int, nd: int, npf: int, mb: int, ns: int | None = None, P: int = 0):
+    `full` (runners with per_sequence = True): ctx, tables and the recurrent-state slots sslot cover the prompts
+    too, rseq[T] names each row's sequence, and segs holds the boundaries of the prompt rows cut at the attention
+    chunk edges (one list after the other, nsg entries in all)."""
+    _I64 = ("ids", "slots", "last", "seeds", "pslots", "pdst", "csrc")
+    _I32 = ("pos", "src", "ctx", "cu", "ecu", "sslot", "rseq", "segs", "topk", "temp", "topp", "tables")
+
+    def __init__(self, T: int, nd: int, npf: int, mb: int, ns: int | None = None, P: int = 0, full: bool = False,
+                 nsg: int = 0, nl: int | None = None):
         """ns: prompts that are sampled in this step (default: all npf; fewer under chunked prefill, where a
         prompt's earlier chunks only fill the cache). P > 0: some prompt rows continue a prompt whose first P
         tokens (over all such prompts) are already in the paged cache: pslots[P] = their cache slots,
         pdst[P] / csrc[T - nd] = where prefix tokens / this step's prompt rows sit in the extended
-        [prefix | chunk] attention layout, ecu[npf + 1] = its sequence boundaries."""
+        [prefix | chunk] attention layout, ecu[npf + 1] = its sequence boundaries. nl: rows whose logits are wanted
+        when that is not one per sampled sequence."""
         ns = npf if ns is None else ns
         self.T, self.nd, self.npf, self.mb, self.ns, self.P = T, nd, npf, mb, ns, P
         B = nd + ns
-        self.n = dict(ids=T, slots=T, last=B, seeds=B, pslots=P, pdst=P, csrc=(T - nd) if P else 0, pos=T, src=T, ctx=nd,
-                      cu=npf + 1 if npf else 0, ecu=npf + 1 if P else 0, topk=B, temp=B, topp=B, tables=nd * mb)
+        nt = self.nt = nd + (npf if full else 0)             # sequences with a context length and a block table
+        self.n = dict(ids=T, slots=T, last=B if nl is None else nl, seeds=B, pslots=P, pdst=P, csrc=(T - nd) if P else 0,
+                      pos=T, src=T, ctx=nt, cu=npf + 1 if npf else 0, ecu=npf + 1 if P else 0, sslot=nt if full else 0,
+                      rseq=T if full else 0, segs=nsg, topk=B, temp=B, topp=B, tables=nt * mb)
         o = 0
         self.off = {}
         for k in self._I64:
@@ -70,15 +79,32 @@ class StepLayout:
         for k in self._I32:
             n = self.n[k]
             out[k] = buf[self.off[k]:self.off[k] + (n + 1) // 2].view(f32 if k in ("temp", "topp") else i32)[:n]
-        out["tables"] = out["tables"].reshape(self.nd, self.mb) if self.nd * self.mb else out["tables"]
+        out["tables"] = out["tables"].reshape(self.nt, self.mb) if self.nt * self.mb else out["tables"]
         return out
 
 
-class PackedStep:
-    __slots__ = ("layout", "slot", "max_seqlen", "want_lp", "max_ext")
+def _chunk_segments(cu, starts, chunk: int) -> tuple[list[int], int]:
+    """Boundaries of the prompt rows (relative to the first prompt row) as independent causal sequences: a prompt is
+    cut wherever its position reaches a multiple of `chunk` (0: not at all). Returns (boundaries, longest piece); no
+    boundaries when some prompt continues in the middle of a chunk, whose earlier keys are only in the cache."""
+    out, longest = [0], 0
+    for i, a in enumerate(starts):
+        n = cu[i + 1] - cu[i]
+        if (a % chunk) if chunk else a:
+            return [], 0
+        for s in range(0, n, chunk or n):
+            e = min(n, s + (chunk or n))
+            out.append(cu[i] + e)
+            longest = max(longest, e - s)
+    return out, longest
 
-    def __init__(self, layout: StepLayout, slot, max_seqlen: int, max_ext: int = 0):
+
+class PackedStep:
+    __slots__ = ("layout", "slot", "max_seqlen", "want_lp", "max_ext", "segs")
+
+    def __init__(self, layout: StepLayout, slot, max_seqlen: int, max_ext: int = 0, segs: dict | None = None):
         self.layout, self.slot, self.max_seqlen, self.want_lp, self.max_ext = layout, slot, max_seqlen, False, max_ext
+        self.segs = segs or {}       # attention chunk size -> (offset, count, longest) inside the layout's segs section
 
 
 class LLMEngine:
@@ -98,11 +124,27 @@ class LLMEngine:
             # as long as max_model_len
             raise ValueError(f"max_model_len ({self.max_model_len}) exceeds max_num_batched_tokens "
                              f"({max_num_batched_tokens}): raise the latter or enable chunked prefill")
+        runner_cls = family_of(cfg).runner()
+        self.per_sequence = runner_cls.per_sequence
+        if self.per_sequence and self.world > 1:
+            raise ValueError(f"{cfg.name}: tensor parallelism is not available for this model family")
+        kv_specs, state_specs = runner_cls.cache_specs(cfg, weights)
+        self.slots = None
+        if any(s is not None for s in state_specs):
+            if enable_prefix_caching:
+                raise ValueError(f"{cfg.name}: prefix caching shares pages of keys and values, but this model also carries "
+                                 "recurrent state from token to token")
+            self.slots = SlotManager(max_num_seqs)
+            self.states = StateCache(state_specs, max_num_seqs, self.dtype, self.device)
+        else:
+            self.states = None
         if num_blocks is None:
-            per_block = KVCache.bytes_per_block(cfg.num_hidden_layers, block_size, weights.KV, cfg.head_dim, self.dtype)
+            per_block = max(1, KVCache.bytes_per_block_specs(kv_specs, block_size, self.dtype))
             if self.device.type == "cuda":
                 free, total = torch.cuda.mem_get_info(self.device)
                 budget = max(0, free - (1 - gpu_memory_utilization) * total - (2 << 30))
+                if self.per_sequence:                    # never more pages than max_num_seqs full sequences can hold
+                    budget = min(budget, max_num_seqs * -(-self.max_model_len // block_size) * per_block)
                 num_blocks = max(64, int(budget // per_block))
                 if self.world > 1:                       # every rank must agree
                     import torch.distributed as dist
@@ -111,11 +153,14 @@ class LLMEngine:
                     num_blocks = int(t.item())
             else:
                 num_blocks = 256
-        self.kv = KVCache(cfg.num_hidden_layers, num_blocks, block_size, weights.KV, cfg.head_dim, self.dtype, self.device)
+        self.kv = KVCache.from_specs(kv_specs, num_blocks, block_size, self.dtype, self.device)
         self.blocks = BlockManager(num_blocks, block_size, enable_prefix_caching)
         self.sched = Scheduler(self.blocks, max_num_seqs, max_num_batched_tokens, self.max_model_len,
-                               mixed=mixed_batches, prefill_chunk=prefill_chunk)
-        self.runner = ModelRunner(cfg, weights, self.kv, tp)
+                               mixed=mixed_batches, prefill_chunk=prefill_chunk, slots=self.slots)
+        if self.per_sequence:
+            self.runner = runner_cls(cfg, weights, self.kv, self.states, self.max_model_len)
+        else:
+            self.runner = runner_cls(cfg, weights, self.kv, tp)
         self.max_blocks_per_seq = -(-self.max_model_len // block_size)
         self.requests: dict[str, Request] = {}
         self.detok: dict[str, IncrementalDetokenizer] = {}
@@ -197,17 +242,29 @@ class LLMEngine:
         return dst
 
     def pack_step(self, nd: int, ids, pos, slots, ctx, tables, cu, max_seqlen: int, sampling=None,
-                  src=None, sampled_prompts: int | None = None, prefix=None) -> "PackedStep":
+                  src=None, sampled_prompts: int | None = None, prefix=None, sslots=None, starts=None,
+                  want=None) -> "PackedStep":
         """Lay one step's metadata out in a pinned host buffer (see StepLayout). ids/pos/slots cover all T
         rows (decode rows first); ctx/tables the nd decode rows; cu the packed prompts (relative to row nd);
         sampling = (temperature, top_k, top_p, seeds) per sampled row or None. sampled_prompts: how many of the
         prompts (the first ones) end in this step; prefix = (pslots, pdst, csrc, ecu, max_ext) when prompt rows
-        continue prompts whose earlier tokens are in the cache."""
+        continue prompts whose earlier tokens are in the cache.
+        For a runner with per_sequence = True, ctx / tables / sslots (state slots) cover the prompts too and starts[i]
+        is the number of prompt i's tokens that earlier steps ran. want: the rows whose logits the step returns
+        instead of the last row of every sampled sequence."""
         T, npf = len(ids), max(0, len(cu) - 1)
+        full = self.per_sequence
+        segs, seg_at = [], {}
+        if full and npf:
+            for c in self.cfg.chunks:
+                s, longest = _chunk_segments(cu, starts, c)
+                seg_at[c] = (len(segs), len(s), longest)
+                segs += s
         ns = npf if sampled_prompts is None else sampled_prompts
         mb = max((len(t) for t in tables), default=0)
         mb = (mb + 7) & ~7
-        lay = StepLayout(T, nd, npf, mb, ns, len(prefix[0]) if prefix is not None else 0)
+        lay = StepLayout(T, nd, npf, mb, ns, len(prefix[0]) if prefix is not None else 0, full, len(segs),
+                         None if want is None else len(want))
         slot = self._host_buffer("step", lay.words)
         v = lay.views(slot[0].numpy(), np)
         v["ids"][:] = ids
@@ -216,23 +273,33 @@ class LLMEngine:
         v["src"][:] = -1
         if src is not None and nd:
             v["src"][:nd] = src
-        if nd:
+        if full:
+            v["sslot"][:] = sslots if sslots is not None else -1
+            v["rseq"][:nd] = np.arange(nd)
+            if npf:
+                v["rseq"][nd:] = np.repeat(np.arange(nd, nd + npf), np.diff(cu))
+                v["segs"][:] = segs
+        if lay.nt:
             v["ctx"][:] = ctx
             tab = v["tables"]
             for i, t in enumerate(tables):
                 tab[i, :len(t)] = t
         if npf:
             v["cu"][:] = cu
-            v["last"][nd:] = np.asarray(cu[1:ns + 1], dtype=np.int64) + (nd - 1)
-        if nd:
-            v["last"][:nd] = np.arange(nd)
+        if want is not None:
+            v["last"][:] = want
+        else:
+            if npf:
+                v["last"][nd:] = np.asarray(cu[1:ns + 1], dtype=np.int64) + (nd - 1)
+            if nd:
+                v["last"][:nd] = np.arange(nd)
         if prefix is not None:
             v["pslots"][:], v["pdst"][:], v["csrc"][:], v["ecu"][:] = prefix[:4]
         if sampling is not None:
             v["temp"][:], v["topk"][:], v["topp"][:], v["seeds"][:] = sampling
-        return PackedStep(lay, slot, int(max_seqlen), int(prefix[4]) if prefix is not None else 0)
+        return PackedStep(lay, slot, int(max_seqlen), int(prefix[4]) if prefix is not None else 0, seg_at)
 
-    def _pack_batch(self, batch: Batch) -> "PackedStep":
+    def _pack_batch(self, batch: Batch, want=None) -> "PackedStep":
         bs = self.blocks.block_size
         nd = batch.num_decode
         reqs = batch.requests
@@ -251,6 +318,8 @@ class LLMEngine:
             tables.append(r.blocks)
         max_seqlen = 0
         prefix = None
+        starts = []
+        sslots = [r.slot for r in reqs] if self.per_sequence else None
         if len(reqs) > nd:
             cu = [0]
             ar = self._arange
@@ -267,6 +336,11 @@ class LLMEngine:
                 sl.append(allslots[a:a + n])
                 cu.append(cu[-1] + n)
                 max_seqlen = max(max_seqlen, n)
+                if self.per_sequence:                        # its kernels read the earlier tokens from the cache itself
+                    starts.append(a)
+                    ctx.append(a + n)
+                    tables.append(r.blocks)
+                    continue
                 # extended [prefix | chunk] layout for the attention of prompts that are under way
                 pslots.append(allslots[:a])
                 pdst.append(ecu[-1] + ar[:a])
@@ -283,7 +357,8 @@ class LLMEngine:
                     # same text, whatever else the engine is doing
                     [(r.seed * 1000003 + len(r.output_ids) + r.pending) & 0x7FFFFFFFFFFFFFFF for r in reqs])
         return self.pack_step(nd, ids, pos, slots, ctx, tables, cu, max_seqlen, sampling, src,
-                              sampled_prompts=batch.num_sampled - nd, prefix=prefix)
+                              sampled_prompts=batch.num_sampled - nd, prefix=prefix, sslots=sslots, starts=starts,
+                              want=want)
 
     def _ring(self):
         """Shared-memory control ring between the driver and the workers (one node): created lazily by rank 0,
@@ -368,6 +443,13 @@ class LLMEngine:
         if lay.npf == 0 and self.use_graphs:
             return self._decode_graph(step)
         v = lay.views(self._to_device(step.slot, lay.words), torch)
+        if self.per_sequence:
+            segs = {c: (v["segs"][o:o + n], longest) for c, (o, n, longest) in step.segs.items()}
+            logits = self.runner.forward(self._feed(v["ids"], v["src"]), v["pos"], v["slots"], num_decode=lay.nd,
+                                         block_tables=v["tables"], ctx_lens=v["ctx"], cu_seqlens=v["cu"] if lay.npf else None,
+                                         max_seqlen=step.max_seqlen, last_idx=v["last"] if lay.npf else None,
+                                         max_ctx=self.max_model_len, state_slots=v["sslot"], row_seq=v["rseq"], segs=segs)
+            return logits, v
         logits = self.runner.forward(self._feed(v["ids"], v["src"]), v["pos"], v["slots"], num_decode=lay.nd,
                                      block_tables=v["tables"] if lay.nd else None, ctx_lens=v["ctx"] if lay.nd else None,
                                      cu_seqlens=v["cu"] if lay.npf else None, max_seqlen=step.max_seqlen,
@@ -398,13 +480,18 @@ class LLMEngine:
         dev, mbs = self.device, self.max_blocks_per_seq
         g = self.graphs.get(bucket)
         if g is None:
-            glay = StepLayout(bucket, bucket, 0, mbs)
+            glay = StepLayout(bucket, bucket, 0, mbs, full=self.per_sequence)
             buf = torch.zeros(glay.words, dtype=torch.int64, device=dev)
             st = glay.views(buf, torch)
             st["slots"].fill_(-1)
             st["src"].fill_(-1)
+            kw = {}
+            if self.per_sequence:
+                st["sslot"].fill_(-1)
+                st["rseq"].copy_(torch.arange(bucket, device=dev))
+                kw = dict(state_slots=st["sslot"], row_seq=st["rseq"])
             run = lambda: self.runner.forward(self._feed(st["ids"], st["src"]), st["pos"], st["slots"], num_decode=bucket,
-                                              block_tables=st["tables"], ctx_lens=st["ctx"], max_ctx=self.max_model_len)
+                                              block_tables=st["tables"], ctx_lens=st["ctx"], max_ctx=self.max_model_len, **kw)
             side = torch.cuda.Stream(device=dev)
             side.wait_stream(torch.cuda.current_stream())
             with torch.cuda.stream(side):                 # warm-up outside capture (workspaces, TMA maps)
@@ -430,6 +517,10 @@ class LLMEngine:
         dst["slots"][B:] = -1
         dst["ctx"][:B] = src["ctx"]
         dst["ctx"][B:] = 0
+        if self.per_sequence:
+            dst["sslot"][:B] = src["sslot"]
+            dst["sslot"][B:] = -1
+            dst["rseq"][:] = np.arange(bucket)
         w = min(lay.mb, mbs)
         dst["tables"][:B, :w] = src["tables"][:, :w]
         self._to_device(slot, glay.tables + (B * mbs + 1) // 2, buf)
@@ -544,6 +635,45 @@ class LLMEngine:
         if self.device.type == "cuda":
             torch.cuda.synchronize(self.device)
         return n
+
+    # ---- replay: given tokens instead of sampled ones -----------------------------------------------
+    def replay_step(self, entries: list[tuple["Request", list[int], list[int]]]) -> torch.Tensor | None:
+        """One engine step over tokens that are given: entries = (request, its next tokens, the places among them whose
+        logits are wanted). The same packing, cache bookkeeping and forward pass as step() (a request that has tokens in
+        the cache and brings one is a decode row, everything else prompt rows); nothing is sampled. Returns the wanted
+        logits [n, vocab] on the host, in the order of the entries, or None."""
+        decode = [e for e in entries if len(e[1]) == 1 and e[0].num_computed > 0]
+        rest = [e for e in entries if not (len(e[1]) == 1 and e[0].num_computed > 0)]
+        order = decode + rest
+        for r, toks, _ in order:
+            if any(not 0 <= t < self.cfg.vocab_size for t in toks):
+                raise ValueError(f"request {r.request_id}: token outside the vocabulary of {self.cfg.vocab_size}")
+            if r.num_computed + len(toks) > self.max_model_len:
+                raise ValueError(f"request {r.request_id}: longer than {self.max_model_len} tokens")
+            if not self.sched._acquire(r, r.num_computed + len(toks)):
+                raise RuntimeError(f"request {r.request_id}: out of cache pages or state slots")
+            r.prompt_ids.extend(toks)
+            r.chunk = len(toks)
+            r.status = "running"
+        row, rows = 0, {}
+        for r, toks, want in order:
+            rows[r.request_id] = [row + w for w in want]
+            row += len(toks)
+        want = [x for r, _, _ in entries for x in rows[r.request_id]]
+        batch = Batch("mixed", [e[0] for e in order], len(decode))
+        packed = self._pack_batch(batch, want=want if rest else None)
+        self._broadcast(packed)
+        logits, _ = self._forward_step(packed)
+        for r, toks, _ in order:
+            r.num_computed += len(toks)
+        if not want:
+            return None
+        return (logits if rest else logits[want]).float().cpu()
+
+    def replay_end(self, request: "Request") -> None:
+        """The request is over: its pages and its state slot go back."""
+        request.status = "finished"
+        self.sched.release(request)
 
     def shutdown_workers(self) -> None:
         if self.world > 1 and self.rank == 0:

@@ -1,9 +1,11 @@
 """Paged KV cache: fixed-size blocks + per-sequence block tables (vLLM's
 PagedAttention memory model, restated). Tensors: k_cache, v_cache = [L][num_blocks, block_size,
-KV_heads_local, head_dim] in the compute dtype; the block manager is pure host-side bookkeeping."""
+KV_heads_local, head_dim] in the compute dtype; the block manager is pure host-side bookkeeping.
+Layers with recurrent state keep it in a StateCache: one slot per sequence, handed out by a SlotManager."""
 from __future__ import annotations
 
 from collections import OrderedDict
+from dataclasses import dataclass
 
 import torch
 
@@ -118,13 +120,92 @@ class BlockManager:
         return 1.0 - len(self.free) / max(1, self.num_blocks)
 
 
+@dataclass(frozen=True)
+class KVSpec:
+    """One layer's cache row: kv_heads keys of `dim` and values of `vdim` elements per token. `source`: the layer
+    whose pages this layer reads instead of having its own."""
+    kv_heads: int
+    dim: int
+    vdim: int
+    source: int | None = None
+
+
+@dataclass(frozen=True)
+class StateSpec:
+    """One layer's recurrent state of a sequence: `heads` fp32 matrices [rows, cols] and, for layers with a short
+    convolution, its last `conv_rows` inputs of `conv_channels` channels."""
+    heads: int
+    rows: int
+    cols: int
+    conv_rows: int = 0
+    conv_channels: int = 0
+
+
+class SlotManager:
+    """Free list of recurrent-state slots; a sequence holds one from its admission until it ends or is preempted. A
+    slot is handed out as it is: the kernels start from zero at position 0 instead of reading it."""
+
+    def __init__(self, num_slots: int):
+        self.num_slots = num_slots
+        self.free = list(range(num_slots - 1, -1, -1))
+
+    def take(self) -> int:
+        return self.free.pop() if self.free else -1
+
+    def release(self, slot: int) -> None:
+        if slot >= 0:
+            self.free.append(slot)
+
+
+class StateCache:
+    """Recurrent states of all slots: per layer `ssm` [slots, heads, rows, cols] fp32 and `conv`
+    [slots, conv_rows, channels] in the compute dtype (None where a layer has none)."""
+
+    def __init__(self, specs: list, num_slots: int, dtype: torch.dtype, device):
+        self.num_slots = num_slots
+        self.ssm = [None if s is None else torch.zeros((num_slots, s.heads, s.rows, s.cols), dtype=torch.float32, device=device)
+                    for s in specs]
+        self.conv = [None if s is None or not s.conv_channels else
+                     torch.zeros((num_slots, s.conv_rows, s.conv_channels), dtype=dtype, device=device) for s in specs]
+
+    @staticmethod
+    def bytes_per_slot(specs: list, dtype: torch.dtype) -> int:
+        es = torch.empty(0, dtype=dtype).element_size()
+        return sum(4 * s.heads * s.rows * s.cols + es * s.conv_rows * s.conv_channels for s in specs if s is not None)
+
+
 class KVCache:
+    """Pages of every layer. Either uniform (num_layers x kv_heads x head_dim) or, with from_specs, shaped layer by
+    layer; a layer with a source aliases that layer's pages, a layer without keys (None) has none."""
+
     def __init__(self, num_layers: int, num_blocks: int, block_size: int, kv_heads: int, head_dim: int,
                  dtype: torch.dtype, device):
-        shape = (num_blocks, block_size, kv_heads, head_dim)
-        self.k = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
-        self.v = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
+        self._fill([KVSpec(kv_heads, head_dim, head_dim)] * num_layers, num_blocks, block_size, dtype, device)
+
+    @classmethod
+    def from_specs(cls, specs: list, num_blocks: int, block_size: int, dtype: torch.dtype, device) -> "KVCache":
+        kv = cls.__new__(cls)
+        kv._fill(specs, num_blocks, block_size, dtype, device)
+        return kv
+
+    def _fill(self, specs, num_blocks, block_size, dtype, device):
+        self.k, self.v = [], []
+        for s in specs:
+            if s is None:
+                self.k.append(None)
+                self.v.append(None)
+            elif s.source is not None:
+                self.k.append(self.k[s.source])
+                self.v.append(self.v[s.source])
+            else:
+                for out, d in ((self.k, s.dim), (self.v, s.vdim)):
+                    out.append(torch.zeros((num_blocks, block_size, s.kv_heads, d), dtype=dtype, device=device))
         self.num_blocks, self.block_size = num_blocks, block_size
+
+    @staticmethod
+    def bytes_per_block_specs(specs: list, block_size: int, dtype: torch.dtype) -> int:
+        es = torch.empty(0, dtype=dtype).element_size()
+        return sum(block_size * s.kv_heads * (s.dim + s.vdim) * es for s in specs if s is not None and s.source is None)
 
     @staticmethod
     def bytes_per_block(num_layers, block_size, kv_heads, head_dim, dtype) -> int:

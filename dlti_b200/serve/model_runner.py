@@ -26,7 +26,7 @@ from ..ops import attention as A
 from ..ops import elementwise as E
 from ..ops import serving as S
 from ..ops.gemm import gemm, gemm_skinny, gemm_skinny_acc, gemm_swiglu
-from .kv_cache import KVCache
+from .kv_cache import KVCache, KVSpec
 
 
 _FUSE_ACC = os.environ.get("DLTI_DECODE_FUSE_ACC", "1") == "1"    # A/B switch: consume the fp32 accumulators directly
@@ -330,6 +330,13 @@ class TPWeights:
 
 
 class ModelRunner:
+    per_sequence = False             # step metadata: decode rows and packed prompts (see engine.StepLayout)
+
+    @staticmethod
+    def cache_specs(cfg: LlamaConfig, weights: TPWeights):
+        """(key/value page specs, recurrent-state specs), one entry per layer."""
+        return [KVSpec(weights.KV, cfg.head_dim, cfg.head_dim)] * cfg.num_hidden_layers, [None] * cfg.num_hidden_layers
+
     def __init__(self, cfg: LlamaConfig, weights: TPWeights, kv: KVCache, tp: TPContext):
         self.cfg, self.w, self.kv, self.tp = cfg, weights, kv, tp
         self.scale = 1.0 / math.sqrt(cfg.head_dim)

@@ -44,6 +44,7 @@ class Request:
     output_ids: list[int] = field(default_factory=list)
     logprobs: list[float] = field(default_factory=list)
     blocks: list[int] = field(default_factory=list)
+    slot: int = -1                   # recurrent-state slot (models that have such state)
     status: str = "waiting"          # waiting | running | finished
     finish_reason: str | None = None
     first_token_time: float | None = None

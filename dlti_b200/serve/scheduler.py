@@ -11,7 +11,7 @@ from __future__ import annotations
 from collections import deque
 from dataclasses import dataclass
 
-from .kv_cache import BlockManager
+from .kv_cache import BlockManager, SlotManager
 from .params import Request
 
 
@@ -29,8 +29,10 @@ class Batch:
 
 class Scheduler:
     def __init__(self, blocks: BlockManager, max_num_seqs: int = 256, max_num_batched_tokens: int = 8192,
-                 max_model_len: int = 4096, mixed: bool = True, prefill_chunk: int = 0):
+                 max_model_len: int = 4096, mixed: bool = True, prefill_chunk: int = 0,
+                 slots: SlotManager | None = None):
         self.blocks = blocks
+        self.slots = slots           # recurrent-state slots, for models that carry state from token to token
         self.mixed = mixed           # False = prefill-first steps (no decode rows in a prefill pass)
         # > 0: a prompt contributes at most this many tokens to one step (chunked prefill): bounds how long a
         # step with prompt rows can stall the decode rows, and lets prompts longer than the token budget run.
@@ -52,10 +54,27 @@ class Scheduler:
             for r in list(q):
                 if r.request_id == request_id:
                     q.remove(r)
-                    self.blocks.release(r.blocks)
+                    self.release(r)
                     r.status, r.finish_reason = "finished", "abort"
                     return True
         return False
+
+    def _acquire(self, r: Request, num_tokens: int) -> bool:
+        """Cache space for num_tokens and, at its first step, a state slot. False: nothing was taken."""
+        if self.slots is not None and r.slot < 0 and not self.slots.free:
+            return False
+        if not self.blocks.ensure(r.blocks, num_tokens):
+            return False
+        if self.slots is not None and r.slot < 0:
+            r.slot = self.slots.take()
+        return True
+
+    def release(self, r: Request) -> None:
+        """Give back everything the request holds in the cache."""
+        self.blocks.release(r.blocks)
+        if self.slots is not None:
+            self.slots.release(r.slot)
+            r.slot = -1
 
     def _take_cached_prefix(self, r: Request) -> int:
         """Prefix caching: start a waiting request's block list with the cached blocks that already hold the
@@ -91,7 +110,7 @@ class Scheduler:
             if ok:
                 break
             victim = self.running.pop()           # preempt the youngest
-            self.blocks.release(victim.blocks)
+            self.release(victim)
             victim.status = "waiting"
             self.waiting.appendleft(victim)
             self.num_preemptions += 1
@@ -106,8 +125,8 @@ class Scheduler:
                 break
             n = r.num_tokens                      # prompt (+ already generated tokens if it was preempted)
             have = self._take_cached_prefix(r)    # tokens already in the cache (prefix caching), else 0
-            if (n - have > budget and (admitted or decode)) or not self.blocks.ensure(r.blocks, n + 1):
-                self.blocks.release(r.blocks)
+            if (n - have > budget and (admitted or decode)) or not self._acquire(r, n + 1):
+                self.release(r)
                 break
             self.waiting.popleft()
             r.status = "running"
@@ -153,7 +172,7 @@ class Scheduler:
             if c <= 0:
                 return False
             last = c == remaining
-            if not self.blocks.ensure(r.blocks, r.num_computed + c + (1 if last else 0)):
+            if not self._acquire(r, r.num_computed + c + (1 if last else 0)):
                 return False
             r.chunk = c
             budget -= c
@@ -172,7 +191,7 @@ class Scheduler:
                 break
             r.num_computed, r.prefill_done = self._take_cached_prefix(r), False
             if not take(r):
-                self.blocks.release(r.blocks)
+                self.release(r)
                 r.num_computed = 0
                 break
             self.waiting.popleft()
@@ -191,7 +210,7 @@ class Scheduler:
         return Batch(kind, decode + prompts, len(decode), len(decode) + len(complete))
 
     def _unschedule(self, victim: Request) -> None:
-        self.blocks.release(victim.blocks)
+        self.release(victim)
         victim.status = "waiting"
         victim.num_computed, victim.chunk, victim.prefill_done = 0, 0, False
         self.waiting.appendleft(victim)
@@ -203,4 +222,4 @@ class Scheduler:
             self.running.remove(req)
         elif req in self.waiting:                 # preempted while its last token was still in flight
             self.waiting.remove(req)
-        self.blocks.release(req.blocks)
+        self.release(req)
