@@ -22,6 +22,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
       sB[lk][r] = (n0 + r < N && k < K) ? B[(long long)(n0 + r) * ldb + k] : 0.f;
     }
     __syncthreads();
+    float part[4][4] = {};                 // 16 products at a time: two short sums lose less than one long one
 #pragma unroll
     for (int k = 0; k < TK; ++k) {
       float a[4], b[4];
@@ -30,8 +31,12 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        for (int j = 0; j < 4; ++j) part[i][j] = fmaf(a[i], b[j], part[i][j]);
     }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] += part[i][j];
     __syncthreads();
   }
 #pragma unroll

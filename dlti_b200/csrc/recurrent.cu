@@ -5,6 +5,7 @@
 // States live in slots [slots, heads, N, P] and are carried from step to step; a sequence whose step starts at position
 // 0 starts from zero whatever its slot holds.
 #include "common.cuh"
+#include "mma_sync.cuh"
 
 namespace {
 
@@ -27,6 +28,9 @@ struct ScanParams {
 
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+// exp(x) of a decay. Near 1 the rounding of exp itself repeats at every token and adds up over a long memory; 1 + expm1
+// rounds once.
+__device__ __forceinline__ float decay_of(float x) { return x > -0.5f ? 1.f + expm1f(x) : expf(x); }
 
 __device__ __forceinline__ void seq_rows(const ScanParams& p, int s, long long& row0, int& n, int& start) {
   if (s < p.nd) {
@@ -73,7 +77,7 @@ __global__ void __launch_bounds__(256) scan_kernel(const ScanParams p, int slice
     if (blockIdx.y == 0) conv_tail<T>(p, s, blockIdx.x - slices, conv_parts);
     return;
   }
-  __shared__ float sk[TT][8 * NR], sq[TT][8 * NR], sv[TT][32], part[TT][8][32], sa[TT];
+  __shared__ float sk[TT][8 * NR], sq[TT][8 * NR], sv[TT][32], part[TT][8][32], sstep[TT], sdecay[TT];
   long long row0;
   int n, start;
   seq_rows(p, s, row0, n, start);
@@ -115,18 +119,19 @@ __global__ void __launch_bounds__(256) scan_kernel(const ScanParams p, int slice
       sv[warp][lane] = x;
       if (lane == 0) {
         if (p.decay) {
-          sa[warp] = 1.f;
+          sstep[warp] = 1.f;
+          sdecay[warp] = cdec;
         } else {
-          sa[warp] = softplus_f(Cvt<T>::to_f(reinterpret_cast<const T*>(p.dt)[row * p.dt_ld + h]) + p.dt_bias[h]);
+          const float step = softplus_f(Cvt<T>::to_f(reinterpret_cast<const T*>(p.dt)[row * p.dt_ld + h]) + p.dt_bias[h]);
+          sstep[warp] = step;
+          sdecay[warp] = decay_of(-expf(p.A_log[h]) * step);
         }
       }
     }
     __syncthreads();
-    const float eA = p.decay ? 0.f : expf(p.A_log[h]);
     for (int t = 0; t < nt; ++t) {
-      const float sc = sa[t];
-      const float a = p.decay ? cdec : expf(-eA * sc);
-      const float vv = sv[t][lane] * sc;
+      const float a = sdecay[t];
+      const float vv = sv[t][lane] * sstep[t];
       float acc = 0.f;
 #pragma unroll
       for (int i = 0; i < NR; ++i) {
@@ -171,6 +176,307 @@ int launch_scan(const ScanParams& p, int nseq, cudaStream_t st) {
   return DLTI_ERR_TOO_LARGE;
 }
 
+// Chunked form for prompts, bf16: CTA = (32 columns of P, head, sequence), 4 warps, 64 tokens a chunk. With L_t the
+// running sum of log a within the chunk and d_s = step size,
+//     o_t   = exp(L_t) S^T q_t + sum_(s <= t) [exp(L_t - L_s) d_s (k_s . q_t)] v_s
+//     S'    = exp(L_63) S + sum_s k_s [exp(L_63 - L_s) d_s v_s]^T
+// q, k, v are exact bf16 operands; the three fp32 operands (S, the bracketed weights, the bracketed values) enter the
+// tensor-core products as hi + lo bf16 pairs, so the recurrence keeps 16+ mantissa bits everywhere. S lives in fp32
+// accumulator registers (warp w owns rows [w NT/4, (w+1) NT/4)) and, split, in shared memory as the next operand.
+constexpr int CQ = 64, CP = 32, CPP = CP + 8;
+template <int NT>
+struct ChunkSmem {
+  static constexpr int NP = NT + 8;
+  static constexpr int QK = CQ * NP * 2, V = CQ * CPP * 2, STAGE = 2 * QK + V;          // bytes
+  static constexpr int W = 2 * STAGE, S = W + 2 * V, VEC = S + 2 * NT * CPP * 2, BYTES = VEC + 3 * CQ * 4 + 16;
+};
+template <int NT>
+__global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int slices, int conv_parts) {
+  using L = ChunkSmem<NT>;
+  using bf16 = __nv_bfloat16;
+  const int s = p.seq0 + blockIdx.z;
+  if ((int)blockIdx.x >= slices) {
+    if (blockIdx.y == 0) conv_tail<bf16>(p, s, blockIdx.x - slices, conv_parts);
+    return;
+  }
+  extern __shared__ __align__(128) uint8_t smem[];
+  const uint32_t sb = smem_u32(smem);
+  float* sL = reinterpret_cast<float*>(smem + L::VEC);          // running log decay
+  float* sStep = sL + CQ;
+  float* sE = sStep + CQ;                                       // exp(L_63 - L_s) * step
+  long long row0;
+  int n, start;
+  seq_rows(p, s, row0, n, start);
+  const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c0 = blockIdx.x * CP, ncol = min(CP, p.P - c0), grp = h / p.rep;
+  const int slot = p.sslot[s];
+  const bf16* q = reinterpret_cast<const bf16*>(p.q) + row0 * p.q_ld + (long long)grp * p.N;
+  const bf16* k = reinterpret_cast<const bf16*>(p.k) + row0 * p.k_ld + (long long)grp * p.N;
+  const bf16* v = reinterpret_cast<const bf16*>(p.v) + row0 * p.v_ld + (long long)h * p.P + c0;
+  const float eA = p.decay ? 0.f : expf(p.A_log[h]);
+  const float la_c = p.decay ? fmaxf(logf(p.decay[h]), -80.f) : 0.f;
+  const float bias = p.decay ? 0.f : p.dt_bias[h];
+  const float Dh = p.D ? p.D[h] : 0.f;
+
+  auto load = [&](int stage, int t0) {
+    const uint32_t base = sb + stage * L::STAGE;
+    const int nc = p.N >> 3, vc = ncol >> 3;
+    for (int i = threadIdx.x; i < CQ * (NT / 8); i += 128) {
+      const int r = i / (NT / 8), c = i % (NT / 8);
+      const bool ok = t0 + r < n && c < nc;
+      const long long row = ok ? t0 + r : 0;
+      const int cc = ok ? c * 8 : 0;
+      cp_async16(base + (r * L::NP + c * 8) * 2, q + row * p.q_ld + cc, ok);
+      cp_async16(base + L::QK + (r * L::NP + c * 8) * 2, k + row * p.k_ld + cc, ok);
+    }
+    for (int i = threadIdx.x; i < CQ * (CP / 8); i += 128) {
+      const int r = i / (CP / 8), c = i % (CP / 8);
+      const bool ok = t0 + r < n && c < vc;
+      cp_async16(base + 2 * L::QK + (r * CPP + c * 8) * 2, v + (ok ? t0 + r : 0) * p.v_ld + (ok ? c * 8 : 0), ok);
+    }
+    cp_async_commit();
+  };
+  auto raw_dt = [&](int t0) {
+    const int t = t0 + threadIdx.x;
+    if (p.decay || threadIdx.x >= CQ || t >= n) return 0.f;
+    return __bfloat162float(reinterpret_cast<const bf16*>(p.dt)[(row0 + t) * p.dt_ld + h]) + bias;
+  };
+
+  constexpr int MT = NT / 64;                                    // 16-row state tiles of a warp
+  float S[MT][CP / 8][4];
+  float* st = p.state + (((long long)(slot < 0 ? 0 : slot) * p.heads + h) * p.N) * p.P + c0;
+  const int srow = warp * (NT / 4) + (lane >> 2), scol = (lane & 3) * 2;
+  const bool have = slot >= 0 && start > 0;
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        const int r = srow + i * 16 + 8 * y, c = j * 8 + scol;
+        const bool ok = have && r < p.N && c < ncol;             // ncol is a multiple of 8
+        S[i][j][2 * y] = ok ? st[(long long)r * p.P + c] : 0.f;
+        S[i][j][2 * y + 1] = ok ? st[(long long)r * p.P + c + 1] : 0.f;
+      }
+  auto publish = [&]() {                                         // S as hi / lo operands
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+        for (int y = 0; y < 2; ++y) {
+          uint32_t hi, lo;
+          split_pair(S[i][j][2 * y], S[i][j][2 * y + 1], hi, lo);
+          const int off = ((srow + i * 16 + 8 * y) * CPP + j * 8 + scol) * 2;
+          *reinterpret_cast<uint32_t*>(smem + L::S + off) = hi;
+          *reinterpret_cast<uint32_t*>(smem + L::S + NT * CPP * 2 + off) = lo;
+        }
+  };
+  load(0, 0);
+  float dt_next = raw_dt(0);
+  publish();
+  int it = 0;
+  for (int t0 = 0; t0 < n; t0 += CQ, ++it) {
+    const uint32_t base = sb + (it & 1) * L::STAGE;
+    if (threadIdx.x < CQ) {
+      const bool ok = t0 + (int)threadIdx.x < n;
+      const float step = !ok ? 0.f : (p.decay ? 1.f : softplus_f(dt_next));
+      float x = !ok ? 0.f : (p.decay ? la_c : -eA * step);
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float y = __shfl_up_sync(0xffffffffu, x, o);
+        if (lane >= o) x += y;
+      }
+      sStep[threadIdx.x] = step;
+      sL[threadIdx.x] = x;                                       // sums inside each half of the chunk
+    }
+    dt_next = raw_dt(t0 + CQ);
+    __syncthreads();                                             // stage (it + 1) & 1 free; half sums, S operands visible
+    if (t0 + CQ < n) {
+      load((it + 1) & 1, t0 + CQ);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    const float half = sL[31];
+    const float total = sL[CQ - 1] + half;
+    if (threadIdx.x < CQ) {
+      const float l = sL[threadIdx.x] + (threadIdx.x >= 32 ? half : 0.f);
+      sE[threadIdx.x] = expf(total - l) * sStep[threadIdx.x];
+    }
+    __syncthreads();                                             // tile landed, sE written
+    const bf16* sv = reinterpret_cast<const bf16*>(smem + (it & 1) * L::STAGE + 2 * L::QK);
+    for (int i = threadIdx.x; i < CQ * CP / 2; i += 128) {       // scaled values as hi / lo operands
+      const int r = i / (CP / 2), c = 2 * (i % (CP / 2));
+      const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + r * CPP + c));
+      uint32_t hi, lo;
+      split_pair(x.x * sE[r], x.y * sE[r], hi, lo);
+      *reinterpret_cast<uint32_t*>(smem + L::W + (r * CPP + c) * 2) = hi;
+      *reinterpret_cast<uint32_t*>(smem + L::W + L::V + (r * CPP + c) * 2) = lo;
+    }
+    // ---- outputs of this warp's 16 tokens ----
+    uint32_t qf[NT / 16][4];
+    {
+      const uint32_t qa = base + ((warp * 16 + (lane & 15)) * L::NP + (lane >> 4) * 8) * 2;
+#pragma unroll
+      for (int kk = 0; kk < NT / 16; ++kk) ldsm4(qf[kk], qa + kk * 32);
+    }
+    float o[CP / 8][4];
+#pragma unroll
+    for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) o[j][x] = 0.f;
+    {
+      const uint32_t sa = sb + L::S + ((lane & 15) * CPP + (lane >> 4) * 8) * 2;
+#pragma unroll
+      for (int kk = 0; kk < NT / 16; ++kk)
+#pragma unroll
+        for (int x = 0; x < 2; ++x)                              // hi, lo
+#pragma unroll
+          for (int j = 0; j < CP / 16; ++j) {
+            uint32_t b[4];
+            ldsm4_t(b, sa + x * (NT * CPP * 2) + (kk * 16 * CPP + j * 16) * 2);
+            mma_bf16(o[2 * j], qf[kk], b[0], b[1]);
+            mma_bf16(o[2 * j + 1], qf[kk], b[2], b[3]);
+          }
+    }
+    const int tr = warp * 16 + (lane >> 2);
+    float lt[2], el[2];
+#pragma unroll
+    for (int y = 0; y < 2; ++y) {
+      lt[y] = sL[tr + 8 * y] + (tr + 8 * y >= 32 ? half : 0.f);
+      el[y] = expf(lt[y]);
+    }
+#pragma unroll
+    for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) o[j][x] *= el[x >> 1];
+    for (int kb = 0; kb <= warp; ++kb) {                         // 16 keys at a time up to the diagonal
+      float g0[4] = {}, g1[4] = {};
+      const uint32_t ka = base + L::QK + ((kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * L::NP + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll
+      for (int kk = 0; kk < NT / 16; ++kk) {
+        uint32_t b[4];
+        ldsm4(b, ka + kk * 32);
+        mma_bf16(g0, qf[kk], b[0], b[1]);
+        mma_bf16(g1, qf[kk], b[2], b[3]);
+      }
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int t = tr + 8 * (x >> 1);
+        const int u0 = kb * 16 + scol + (x & 1), u1 = u0 + 8;
+        const float l0 = sL[u0] + (u0 >= 32 ? half : 0.f), l1 = sL[u1] + (u1 >= 32 ? half : 0.f);
+        g0[x] = u0 <= t ? g0[x] * sStep[u0] * expf(lt[x >> 1] - l0) : 0.f;
+        g1[x] = u1 <= t ? g1[x] * sStep[u1] * expf(lt[x >> 1] - l1) : 0.f;
+      }
+      uint32_t hi[4], lo[4];
+      split_pair(g0[0], g0[1], hi[0], lo[0]);
+      split_pair(g0[2], g0[3], hi[1], lo[1]);
+      split_pair(g1[0], g1[1], hi[2], lo[2]);
+      split_pair(g1[2], g1[3], hi[3], lo[3]);
+      const uint32_t va = base + 2 * L::QK + ((kb * 16 + (lane & 15)) * CPP + (lane >> 4) * 8) * 2;
+#pragma unroll
+      for (int j = 0; j < CP / 16; ++j) {
+        uint32_t b[4];
+        ldsm4_t(b, va + j * 32);
+        mma_bf16(o[2 * j], hi, b[0], b[1]);
+        mma_bf16(o[2 * j], lo, b[0], b[1]);
+        mma_bf16(o[2 * j + 1], hi, b[2], b[3]);
+        mma_bf16(o[2 * j + 1], lo, b[2], b[3]);
+      }
+    }
+#pragma unroll
+    for (int y = 0; y < 2; ++y) {
+      const int t = tr + 8 * y;
+      if (t0 + t < n) {
+        bf16* orow = reinterpret_cast<bf16*>(p.out) + (row0 + t0 + t) * p.o_ld + (long long)h * p.P + c0;
+#pragma unroll
+        for (int j = 0; j < CP / 8; ++j) {
+          const int c = j * 8 + scol;
+          if (c >= ncol) continue;
+          const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + t * CPP + c));
+          *reinterpret_cast<__nv_bfloat162*>(orow + c) = __floats2bfloat162_rn(o[j][2 * y] + Dh * x.x, o[j][2 * y + 1] + Dh * x.y);
+        }
+      }
+    }
+    __syncthreads();                                             // scaled values written; old S operands no longer read
+    // ---- state ----
+    const float keep = expf(total);
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) S[i][j][x] *= keep;
+#pragma unroll
+    for (int kb = 0; kb < CQ / 16; ++kb) {
+      uint32_t w[2][CP / 16][4];
+      const uint32_t wa = sb + L::W + ((kb * 16 + (lane & 15)) * CPP + (lane >> 4) * 8) * 2;
+#pragma unroll
+      for (int x = 0; x < 2; ++x)
+#pragma unroll
+        for (int j = 0; j < CP / 16; ++j) ldsm4_t(w[x][j], wa + x * L::V + j * 32);
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        // A = K^T: rows n, columns s, read transposed from K [s][n]
+        uint32_t a[4];
+        ldsm4_t(a, base + L::QK + ((kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * L::NP + warp * (NT / 4) + i * 16 + ((lane >> 3) & 1) * 8) * 2);
+#pragma unroll
+        for (int x = 0; x < 2; ++x)
+#pragma unroll
+          for (int j = 0; j < CP / 16; ++j) {
+            mma_bf16(S[i][2 * j], a, w[x][j][0], w[x][j][1]);
+            mma_bf16(S[i][2 * j + 1], a, w[x][j][2], w[x][j][3]);
+          }
+      }
+    }
+    publish();
+  }
+  if (slot >= 0) {
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+        for (int y = 0; y < 2; ++y) {
+          const int r = srow + i * 16 + 8 * y, c = j * 8 + scol;
+          if (r < p.N && c < ncol) {
+            st[(long long)r * p.P + c] = S[i][j][2 * y];
+            st[(long long)r * p.P + c + 1] = S[i][j][2 * y + 1];
+          }
+        }
+  }
+}
+
+template <int NT>
+int launch_chunk(const ScanParams& p, int nseq, cudaStream_t st) {
+  static bool done[64] = {};
+  int dev = 0;
+  DLTI_CUDA_CHECK(cudaGetDevice(&dev));
+  if (!done[dev & 63]) {
+    DLTI_CUDA_CHECK(cudaFuncSetAttribute(scan_chunk_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, ChunkSmem<NT>::BYTES));
+    done[dev & 63] = true;
+  }
+  const int slices = (p.P + CP - 1) / CP;
+  const int conv_parts = p.conv_state ? (p.conv_C + 1023) / 1024 : 0;
+  scan_chunk_kernel<NT><<<dim3(slices + conv_parts, p.heads, nseq), 128, ChunkSmem<NT>::BYTES, st>>>(p, slices, conv_parts);
+  dlti_count_launch();
+  return (int)cudaGetLastError();
+}
+
+// x = silu(x) in place, rounded to T
+template <typename T>
+__global__ void silu_rows_kernel(T* __restrict__ x, long long ld, long long rows, int n) {
+  const int pairs = n >> 1;
+  const long long total = rows * pairs;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / pairs;
+    uint32_t* p = reinterpret_cast<uint32_t*>(x + t * ld) + (int)(i - t * pairs);
+    const float2 f = Cvt<T>::unpack2(*p);
+    *p = Cvt<T>::pack2(silu_f(f.x), silu_f(f.y));
+  }
+}
+
 }  // namespace
 
 // Sequences [seq0, seq0 + nseq) of the step (the first nd sequences are single rows, sequence nd + i has the rows
@@ -189,4 +495,38 @@ DLTI_API int dlti_linear_scan(const void* q, long long q_ld, const void* k, long
   if (dtype == DLTI_BF16) return launch_scan<__nv_bfloat16>(p, nseq, st);
   if (dtype == DLTI_FP32) return launch_scan<float>(p, nseq, st);
   return DLTI_ERR_UNSUPPORTED;
+}
+
+// The chunked tensor-core form of the same for prompt sequences: bf16, N and P multiples of 8, N <= 256, q / k / v rows
+// 16-byte aligned, no silu (see dlti_silu_rows).
+DLTI_API int dlti_linear_scan_chunked(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long v_ld, int rep,
+                                      const float* decay, const void* dt, long long dt_ld, const float* dt_bias, const float* A_log,
+                                      const float* D, float* state, const int* sslot, const int* ctx, const int* cu, int nd, int seq0,
+                                      int nseq, int heads, int N, int P, void* out, long long o_ld, const void* conv_src,
+                                      long long conv_ld, int conv_col, int conv_rows, int conv_C, void* conv_state, cudaStream_t st) {
+  if (nseq <= 0) return 0;
+  if (heads < 1 || rep < 1 || nseq > 65535 || (!decay && (!dt || !dt_bias || !A_log))) return DLTI_ERR_BAD_ARG;
+  if (N % 8 || P % 8 || q_ld % 8 || k_ld % 8 || v_ld % 8 || o_ld % 2 ||
+      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15)) {
+    dlti_set_error("linear_scan_chunked: 16-byte aligned rows, N and P multiples of 8");
+    return DLTI_ERR_BAD_ARG;
+  }
+  if (conv_rows <= 0) conv_state = nullptr;
+  ScanParams p{q, k, v, q_ld, k_ld, v_ld, rep, 0, decay, dt, dt_ld, dt_bias, A_log, D, state, sslot, ctx, cu,
+               nd, seq0, heads, N, P, out, o_ld, conv_src, conv_ld, conv_col, conv_rows, conv_C, conv_state};
+  if (N <= 64) return launch_chunk<64>(p, nseq, st);
+  if (N <= 128) return launch_chunk<128>(p, nseq, st);
+  if (N <= 256) return launch_chunk<256>(p, nseq, st);
+  dlti_set_error("linear_scan_chunked: states of up to 256 rows");
+  return DLTI_ERR_TOO_LARGE;
+}
+
+DLTI_API int dlti_silu_rows(void* x, long long ld, long long rows, int n, int dtype, cudaStream_t st) {
+  if (rows <= 0 || n <= 0) return 0;
+  if (dtype != DLTI_BF16) return DLTI_ERR_UNSUPPORTED;
+  if (n % 2 || ld % 2) return DLTI_ERR_BAD_ARG;
+  const long long g = (rows * (n / 2) + 255) / 256, cap = (long long)dlti_num_sms() * 16;
+  silu_rows_kernel<__nv_bfloat16><<<(unsigned)(g < cap ? g : cap), 256, 0, st>>>((__nv_bfloat16*)x, ld, rows, n);
+  dlti_count_launch();
+  return (int)cudaGetLastError();
 }

@@ -23,7 +23,7 @@ import torch
 from ..config.args import TrainingArgs
 from ..data.collate import CausalLMCollator
 from ..data.synthetic import SyntheticInstructionDataset
-from ..models.config import resolve_config
+from ..models.config import LlamaConfig, resolve_config
 from ..models.lora import LoraConfig, print_trainable_parameters
 from ..parallel import comm
 from ..utils.metrics import (RULE, create_experiment_name, get_zero_stage_from_config,
@@ -149,6 +149,8 @@ def run_training(kind: str, argv: list[str] | None = None) -> dict | None:
     tokenizer = None
     model_dir = args.model_name if os.path.isdir(args.model_name) else None
     cfg = resolve_config(args.model_config or args.model_name)
+    if not isinstance(cfg, LlamaConfig):
+        raise SystemExit(f"{cfg.name}: training covers the Llama family; this model family is served only")
     pad_id = cfg.pad_token_id if cfg.pad_token_id is not None else cfg.eos_token_id   # pad = eos
     if not args.synthetic:
         from ..data.text import load_tokenizer

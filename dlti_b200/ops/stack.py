@@ -246,13 +246,58 @@ def attn_rows(q, m, rows: Rows, kc, vc, gate, out):
     return out
 
 
+_ws: dict = {}
+_ws_retired: list = []
+
+
+def _workspace(device, floats: int) -> torch.Tensor:
+    ws = _ws.get(str(device))
+    if ws is None or ws.numel() < floats:
+        if ws is not None:
+            _ws_retired.append(ws)             # captured CUDA graphs may still point at it
+        ws = _ws[str(device)] = torch.empty(max(floats, 1 << 20), dtype=torch.float32, device=device)
+    return ws
+
+
+def attn_paged_decode(q, m, rows: Rows, kc, vc, gate, out, splits: int | None = None):
+    """Decode rows (bf16): row b of q against the visible keys of sequence b, split over CTAs."""
+    B, hd, bs = q.shape[0], q.shape[1] // m.heads, kc.shape[1]
+    if splits is None:
+        reach = min(rows.max_ctx or 1 << 30, m.chunk or 1 << 30, rows.tables.shape[1] * bs)
+        ctas = B * m.kv_heads * -(-(m.heads // m.kv_heads) // 16)
+        splits = max(1, min(32, -(-3 * 148 // ctas), -(-reach // 128)))
+    ws = _workspace(q.device, B * m.heads * splits * (m.vdim + 2)) if splits > 1 else None
+    f = _lib.fn("dlti_attn_paged_decode", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _I, _I, _I, _I, _I, _I, _F, _V, _I, _V, _V, _L, _V])
+    _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], bs,
+                 _p(rows.ctx), B, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.scale, _p(gate), splits, _p(ws), _p(out),
+                 out.stride(0), _lib.stream_ptr()), "attn_paged_decode")
+    return out
+
+
+def attn_paged_prefill(q, m, rows: Rows, kc, vc, gate, out):
+    """Prompt rows (bf16): q, gate and out cover all rows of the step."""
+    hd = q.shape[1] // m.heads
+    f = _lib.fn("dlti_attn_paged_prefill", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _F, _V, _V,
+                                            _L, _V])
+    _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], kc.shape[1],
+                 _p(rows.ctx), _p(rows.cu), rows.nd, rows.nseq - rows.nd, rows.max_seqlen, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk,
+                 m.scale, _p(gate), _p(out), out.stride(0), _lib.stream_ptr()), "attn_paged_prefill")
+    return out
+
+
 def paged_attention(q, m, rows: Rows, kc, vc, gate):
     """Attention of every row of a step over the paged cache -> [T, heads * vdim], head outputs times `gate` [T, H]."""
     if not _lib.use_native(q):
         return paged_attention_ref(q, m, rows, kc, vc, gate)
     _debug.check_paged("paged_attention", rows.tables, rows.ctx, kc.shape[0], kc.shape[1])
     out = act(q.shape[0], m.heads * m.vdim, q.dtype, q.device)
-    return attn_rows(q, m, rows, kc, vc, gate, out)
+    if q.dtype == torch.float32 or max(kc.shape[3], vc.shape[3]) > 256:
+        return attn_rows(q, m, rows, kc, vc, gate, out)
+    if rows.nd:
+        attn_paged_decode(q[:rows.nd], m, rows, kc, vc, gate, out)
+    if rows.nseq > rows.nd:
+        attn_paged_prefill(q, m, rows, kc, vc, gate, out)
+    return out
 
 
 # ---- recurrences -------------------------------------------------------------------------------------------
@@ -324,18 +369,55 @@ def linear_scan_ref(q, k, v, decay: Decay, state, rows: Rows, heads, groups, N, 
 
 def linear_scan(q, k, v, decay: Decay, state, rows: Rows, heads, groups, N, P, silu=False, conv_src=None, conv_col=0, conv_state=None):
     """S <- a S + k (step v)^T, o = S^T q (+ D v) over the rows of every sequence; q, k [T, groups * N] views, v [T,
-    heads * P], state [slots, heads, N, P] fp32 updated in place. silu: applied to q, k, v on load. conv_state: renewed
+    heads * P], state [slots, heads, N, P] fp32 updated in place. silu: applied to q, k, v first (prompt rows of the views
+    may be overwritten with it). conv_state: renewed
     from the rows of conv_src (see short_conv)."""
     if not _lib.use_native(q):
         return linear_scan_ref(q, k, v, decay, state, rows, heads, groups, N, P, silu, conv_src, conv_col, conv_state)
     out = act(q.shape[0], heads * P, v.dtype, q.device)
+    nd, nseq = rows.nd, rows.nseq
+    conv = (conv_src, conv_col, conv_state)
+    if nseq > nd and q.dtype == torch.bfloat16 and N % 8 == 0 and P % 8 == 0 and N <= 256 and rows.max_seqlen >= _CHUNKED_FROM:
+        if nd:
+            _scan_tokens(q, k, v, decay, state, rows, 0, nd, heads, groups, N, P, silu, conv, out)
+        if silu:
+            for x in (q, k, v):
+                silu_rows_(x[nd:])
+        _scan_chunked(q, k, v, decay, state, rows, nd, nseq - nd, heads, groups, N, P, conv, out)
+    else:
+        _scan_tokens(q, k, v, decay, state, rows, 0, nseq, heads, groups, N, P, silu, conv, out)
+    return out
+
+
+_CHUNKED_FROM = 16           # longest portion of a step from which the chunked kernel takes its prompts
+
+
+def silu_rows_(x):
+    """In place on a [rows, n] bf16 section of a projection."""
+    f = _lib.fn("dlti_silu_rows", [_V, _L, _L, _I, _I, _V])
+    _lib.check(f(_p(x), x.stride(0), x.shape[0], x.shape[1], _lib.dtype_code(x.dtype), _lib.stream_ptr()), "silu_rows")
+
+
+def _conv_args(conv):
+    src, col, st = conv
+    return (_p(src), 0 if src is None else src.stride(0), col, 0 if st is None else st.shape[1], 0 if st is None else st.shape[2], _p(st))
+
+
+def _scan_tokens(q, k, v, decay, state, rows, seq0, nseq, heads, groups, N, P, silu, conv, out):
     f = _lib.fn("dlti_linear_scan", [_V, _L, _V, _L, _V, _L, _I, _I, _V, _V, _L, _V, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _V,
                                      _L, _V, _L, _I, _I, _I, _V, _I, _V])
     dt = decay.dt
     _lib.check(f(_p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), heads // groups, int(silu), _p(decay.const), _p(dt),
                  0 if dt is None else dt.stride(0), _p(decay.dt_bias), _p(decay.A_log), _p(decay.D), _p(state), _p(rows.state),
-                 _p(rows.ctx), _p(rows.cu), rows.nd, 0, rows.nseq, heads, N, P, _p(out), out.stride(0), _p(conv_src),
-                 0 if conv_src is None else conv_src.stride(0), conv_col, 0 if conv_state is None else conv_state.shape[1],
-                 0 if conv_state is None else conv_state.shape[2], _p(conv_state), _lib.dtype_code(v.dtype), _lib.stream_ptr()),
-               "linear_scan")
-    return out
+                 _p(rows.ctx), _p(rows.cu), rows.nd, seq0, nseq, heads, N, P, _p(out), out.stride(0), *_conv_args(conv),
+                 _lib.dtype_code(v.dtype), _lib.stream_ptr()), "linear_scan")
+
+
+def _scan_chunked(q, k, v, decay, state, rows, seq0, nseq, heads, groups, N, P, conv, out):
+    f = _lib.fn("dlti_linear_scan_chunked", [_V, _L, _V, _L, _V, _L, _I, _V, _V, _L, _V, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I,
+                                             _V, _L, _V, _L, _I, _I, _I, _V, _V])
+    dt = decay.dt
+    _lib.check(f(_p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), heads // groups, _p(decay.const), _p(dt),
+                 0 if dt is None else dt.stride(0), _p(decay.dt_bias), _p(decay.A_log), _p(decay.D), _p(state), _p(rows.state),
+                 _p(rows.ctx), _p(rows.cu), rows.nd, seq0, nseq, heads, N, P, _p(out), out.stride(0), *_conv_args(conv),
+                 _lib.stream_ptr()), "linear_scan_chunked")

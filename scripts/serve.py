@@ -18,9 +18,9 @@ sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 def build_engine(a):
     import torch
 
-    from dlti_b200.models.config import resolve_config
+    from dlti_b200.models.config import LlamaConfig, resolve_config
+    from dlti_b200.models.registry import family_of
     from dlti_b200.parallel import comm
-    from dlti_b200.serve.engine import LLMEngine
     from dlti_b200.serve.model_runner import TPContext, TPWeights
     from dlti_b200.serve.tokenizer import load_tokenizer
 
@@ -28,6 +28,17 @@ def build_engine(a):
     dtype = {"bf16": torch.bfloat16, "fp16": torch.float16, "fp32": torch.float32}[a.dtype]
     model_dir = a.model if a.model and os.path.isdir(a.model) else None
     cfg = resolve_config(a.model_config or a.model)
+    if not isinstance(cfg, LlamaConfig):                 # layer-stack families: one GPU, no adapters
+        fam = family_of(cfg)
+        if a.adapter:
+            raise SystemExit(f"{fam.name}: LoRA adapters are available for the Llama family only")
+        if info.world_size > 1:
+            raise SystemExit(f"{fam.name}: tensor parallelism is available for the Llama family only")
+        if info.device.type == "cuda" and dtype not in fam.dtypes:
+            raise SystemExit(f"{fam.name} has no {a.dtype} kernels")
+        w = (fam.load_weights(cfg, model_dir, info.device, dtype) if model_dir and not a.synthetic
+             else fam.random_weights(cfg, info.device, dtype, a.seed))
+        return info, cfg, make_engine(a, info, cfg, w, TPContext(), load_tokenizer(model_dir, cfg.vocab_size))
     fused = None
     if info.distributed and a.backend == "fused" and info.device.type == "cuda":
         from dlti_b200.parallel.fused import FusedComm
@@ -48,7 +59,11 @@ def build_engine(a):
             w.attach_adapter(load_adapter_state(a.adapter), load_adapter_config(a.adapter))
     else:
         w.init_random(a.seed)
-    tok = load_tokenizer(model_dir, cfg.vocab_size)
+    return info, cfg, make_engine(a, info, cfg, w, tp, load_tokenizer(model_dir, cfg.vocab_size))
+
+
+def make_engine(a, info, cfg, w, tp, tok):
+    from dlti_b200.serve.engine import LLMEngine
     eng = LLMEngine(cfg, w, tp, tok, info=info, block_size=a.block_size, num_blocks=a.num_blocks,
                     gpu_memory_utilization=a.gpu_memory_utilization, max_num_seqs=a.max_num_seqs,
                     max_num_batched_tokens=a.max_num_batched_tokens, max_model_len=a.max_model_len,
@@ -57,12 +72,12 @@ def build_engine(a):
                     enable_prefix_caching=a.enable_prefix_caching)
     if info.rank == 0 and not a.no_warmup:
         eng.warmup()                      # workers follow from worker_loop()
-    return info, cfg, eng
+    return eng
 
 
 def add_args(ap):
-    ap.add_argument("--model", type=str, default=None, help="HF checkpoint directory (or preset name)")
-    ap.add_argument("--model_config", type=str, default=None, help="tiny | llama2-7b | llama2-70b")
+    ap.add_argument("--model", type=str, default=None, help="checkpoint directory (Hugging Face Llama, or another family of models/registry.py) or preset name")
+    ap.add_argument("--model_config", type=str, default=None, help="preset: tiny | llama2-7b | llama2-70b | sigosun-1b | ...")
     ap.add_argument("--adapter", type=str, default=None, help="PEFT LoRA adapter directory served on top of the base")
     ap.add_argument("--merge_adapter", action="store_true",
                     help="fold the adapter into the base weights at load time (W' = W + alpha/r B A) instead of "

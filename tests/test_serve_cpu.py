@@ -318,9 +318,9 @@ def test_step_layout_roundtrip():
     import numpy as np
     from dlti_b200.serve.engine import StepLayout
     for kw, want in [(dict(), dict(ids=11, slots=11, last=5, seeds=5, pslots=0, pdst=0, csrc=0, pos=11, src=11, ctx=3,
-                                   cu=3, ecu=0, topk=5, temp=5, topp=5)),
+                                   cu=3, ecu=0, sslot=0, rseq=0, segs=0, topk=5, temp=5, topp=5)),
                      (dict(ns=1, P=6), dict(ids=11, slots=11, last=4, seeds=4, pslots=6, pdst=6, csrc=8, pos=11, src=11,
-                                            ctx=3, cu=3, ecu=3, topk=4, temp=4, topp=4))]:
+                                            ctx=3, cu=3, ecu=3, sslot=0, rseq=0, segs=0, topk=4, temp=4, topp=4))]:
         lay = StepLayout(T=11, nd=3, npf=2, mb=8, **kw)
         buf = np.zeros(lay.words, dtype=np.int64)
         v = lay.views(buf, np)
