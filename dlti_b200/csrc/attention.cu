@@ -55,6 +55,7 @@ struct AttnParams {
   long long T_total;
   float scale;           // 1/sqrt(hd)
   int dtype;
+  const float* gate;     // fwd, optional: [T_total, H] factors on the head outputs
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
@@ -749,7 +750,10 @@ __device__ __forceinline__ void mbar_wait_b(uint32_t bar, uint32_t parity) {
   }
 }
 
-template <typename T>
+// SPLIT: the softmax weights are written as two 16-bit terms (hi over columns 0-63 of the S buffer, what its rounding
+// left over columns 64-127) and both enter the PV product, so the weights keep fp32-like precision (16 mantissa bits)
+// for 1.5x the MMA work.
+template <typename T, bool SPLIT>
 __global__ void __launch_bounds__(F2_THREADS, 1)
 attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) {
   const int b = blockIdx.z, h = blockIdx.y;
@@ -847,6 +851,10 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk)
           umma_f16_ts(tO, tP + kk * 8, v.at(kk * 2048), idesc_pv, kk > 0 ? 1u : acc_on);
+        if constexpr (SPLIT) {
+#pragma unroll
+          for (int kk = 0; kk < 8; ++kk) umma_f16_ts(tO, tP + 64 + kk * 8, v.at(kk * 2048), idesc_pv, 1u);
+        }
         umma_commit(pv_done + 8 * X);
       };
       mbar_wait_b(q_full, 0);
@@ -939,15 +947,20 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
         const float neg_m = -m_ref;
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          uint32_t pk[16];
+          uint32_t pk[16], pl[16];
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
             const float p0 = ex2_approx(fmaf(__uint_as_float(v[32 * c + 2 * i]), sl2, neg_m));
             const float p1 = ex2_approx(fmaf(__uint_as_float(v[32 * c + 2 * i + 1]), sl2, neg_m));
             l += p0 + p1;
             pk[i] = Cvt<T>::pack2(p0, p1);
+            if constexpr (SPLIT) {
+              const float2 hi = Cvt<T>::unpack2(pk[i]);
+              pl[i] = Cvt<T>::pack2(p0 - hi.x, p1 - hi.y);
+            }
           }
           tmem_st_32x32b_x16(tS + c * 16, pk);
+          if constexpr (SPLIT) tmem_st_32x32b_x16(tS + 64 + c * 16, pl);
         }
         tmem_wait_st();
         tc_fence_before();
@@ -956,8 +969,9 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
       }
       mbar_wait_b(pv_done + 8 * X, (nX - 1) & 1);
       tc_fence_after();
-      const float inv = 1.f / l;
       const int qi = qbX * 128 + r;
+      float inv = 1.f / l;
+      if (p.gate && qi < seqlen) inv *= p.gate[(long long)(row0 + qi) * p.H + h];
       T* orow = reinterpret_cast<T*>(p.O) + (long long)(row0 + qi) * p.ldo + h * HD;
 #pragma unroll 1
       for (int c = 0; c < 4; ++c) {
@@ -1023,11 +1037,11 @@ DLTI_API int dlti_attn_fwd(const void* qkv, void* out, float* lse, const int* cu
     dim3 grid2(((max_seqlen + 127) / 128 + 1) / 2, H, batch);
     static bool cfg2[2] = {false, false};
     if (dtype == DLTI_BF16) {
-      if (!cfg2[0]) { DLTI_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd2_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, F2_SMEM)); cfg2[0] = true; }
-      attn_fwd2_kernel<__nv_bfloat16><<<grid2, F2_THREADS, F2_SMEM, st>>>(p, tm);
+      if (!cfg2[0]) { DLTI_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd2_kernel<__nv_bfloat16, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, F2_SMEM)); cfg2[0] = true; }
+      attn_fwd2_kernel<__nv_bfloat16, false><<<grid2, F2_THREADS, F2_SMEM, st>>>(p, tm);
     } else if (dtype == DLTI_FP16) {
-      if (!cfg2[1]) { DLTI_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd2_kernel<__half>, cudaFuncAttributeMaxDynamicSharedMemorySize, F2_SMEM)); cfg2[1] = true; }
-      attn_fwd2_kernel<__half><<<grid2, F2_THREADS, F2_SMEM, st>>>(p, tm);
+      if (!cfg2[1]) { DLTI_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd2_kernel<__half, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, F2_SMEM)); cfg2[1] = true; }
+      attn_fwd2_kernel<__half, false><<<grid2, F2_THREADS, F2_SMEM, st>>>(p, tm);
     } else {
       return DLTI_ERR_UNSUPPORTED;
     }
@@ -1050,6 +1064,31 @@ DLTI_API int dlti_attn_fwd(const void* qkv, void* out, float* lse, const int* cu
 }
 
 // dqkv [T, (H+2KV)*128] receives dq | dk | dv. D_scratch: [H, T] fp32 workspace.
+// Inference form with split softmax weights (see attn_fwd2_kernel), bf16, an optional gate [T, H] on the head outputs and
+// an output row pitch ldo (a multiple of 8).
+DLTI_API int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const int* cu_seqlens, int batch,
+                                 int max_seqlen, long long T_total, int H, int KV, int hd, float scale, cudaStream_t st) {
+  if (hd != HD) { dlti_set_error("attention: head_dim must be 128"); return DLTI_ERR_UNSUPPORTED; }
+  if (H % KV || ldo % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return DLTI_ERR_BAD_ARG;
+  if (batch <= 0 || T_total <= 0) return 0;
+  AttnParams p{};
+  p.cu_seqlens = cu_seqlens; p.H = H; p.KV = KV; p.W = (H + 2 * KV) * HD;
+  p.O = out; p.ldo = ldo; p.T_total = T_total; p.scale = scale; p.dtype = DLTI_BF16; p.gate = gate;
+  CUtensorMap tm;
+  const int rc = make_map(&tm, qkv, T_total, p.W, 128);
+  if (rc) return rc;
+  static bool cfg[64] = {};
+  int dev = 0;
+  DLTI_CUDA_CHECK(cudaGetDevice(&dev));
+  if (!cfg[dev & 63]) {
+    DLTI_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd2_kernel<__nv_bfloat16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, F2_SMEM));
+    cfg[dev & 63] = true;
+  }
+  attn_fwd2_kernel<__nv_bfloat16, true><<<dim3(((max_seqlen + 127) / 128 + 1) / 2, H, batch), F2_THREADS, F2_SMEM, st>>>(p, tm);
+  dlti_count_launch();
+  return (int)cudaGetLastError();
+}
+
 DLTI_API int dlti_attn_bwd(const void* dout, const void* qkv, const void* out, const float* lse,
                            float* D_scratch, void* dqkv, const int* cu_seqlens, int batch,
                            int max_seqlen, long long T_total, int H, int KV, int hd, float scale,

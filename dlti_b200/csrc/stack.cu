@@ -72,6 +72,16 @@ __global__ void embed_rows_kernel(const long long* __restrict__ ids, const T* __
   }
 }
 
+// out = acc (fp32), acc = 0
+__global__ void take_rows_kernel(float* __restrict__ acc, float* __restrict__ out, long long vec) {
+  griddep_wait();
+  griddep_launch();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < vec; i += (long long)gridDim.x * blockDim.x) {
+    reinterpret_cast<float4*>(out)[i] = reinterpret_cast<float4*>(acc)[i];
+    reinterpret_cast<float4*>(acc)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+}
+
 // x += norm(y) * w (or * (1 + w)); xa = T(x). One CTA per row; the row of y stays in registers.
 constexpr int PN_THREADS = 256;
 template <typename T, bool ACC, int PAIRS>
@@ -462,6 +472,16 @@ DLTI_API int dlti_embed_rows(const long long* ids, const void* table, float* x, 
   const int g = grid_for(tokens * d, 256);
   DISPATCH_T(dtype, DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, embed_rows_kernel<T>, dim3(g), dim3(256), 0, st, ids, (const T*)table, x,
                                                     (T*)xa, xa_ld, tokens, d, vocab)));
+  dlti_count_launch();
+  return 0;
+}
+
+// the decode GEMM's accumulator [rows, cols] as an fp32 result (cols a multiple of 4); zero on return
+DLTI_API int dlti_take_rows(float* acc, float* out, long long rows, int cols, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (cols % 4) return DLTI_ERR_BAD_ARG;
+  const long long vec = rows * (cols / 4);
+  DLTI_CUDA_CHECK(dlti_launch_pdl(rows, take_rows_kernel, dim3(grid_for(vec, 256)), dim3(256), 0, st, acc, out, vec));
   dlti_count_launch();
   return 0;
 }

@@ -12,7 +12,7 @@ import torch
 
 from ..models.stack import round8
 from . import _debug, _lib
-from .gemm import gemm, gemm_skinny
+from .gemm import gemm, gemm_skinny, gemm_skinny_acc
 
 _V, _I, _L, _F = C.c_void_p, C.c_int, C.c_longlong, C.c_float
 _p = _lib.ptr
@@ -36,6 +36,17 @@ def linear(a: torch.Tensor, w: torch.Tensor, out_dtype=None) -> torch.Tensor:
     if a.shape[0] <= 256 and out_dtype in (None, a.dtype):
         return gemm_skinny(a, w)
     return gemm(a, w, out_dtype=out_dtype)
+
+
+def linear_f32(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """linear with an fp32 result (logits)."""
+    if not _lib.use_native(a) or a.dtype == torch.float32 or a.shape[0] > 256:
+        return linear(a, w, out_dtype=torch.float32)
+    acc = gemm_skinny_acc(a, w)
+    out = torch.empty_like(acc)
+    f = _lib.fn("dlti_take_rows", [_V, _V, _L, _I, _V])
+    _lib.check(f(_p(acc), _p(out), acc.shape[0], acc.shape[1], _lib.stream_ptr()), "take_rows")
+    return out
 
 
 # ---- rows --------------------------------------------------------------------------------------------------
@@ -264,7 +275,7 @@ def attn_paged_decode(q, m, rows: Rows, kc, vc, gate, out, splits: int | None = 
     B, hd, bs = q.shape[0], q.shape[1] // m.heads, kc.shape[1]
     if splits is None:
         reach = min(rows.max_ctx or 1 << 30, m.chunk or 1 << 30, rows.tables.shape[1] * bs)
-        ctas = B * m.kv_heads * -(-(m.heads // m.kv_heads) // 16)
+        ctas = max(1, B) * m.kv_heads * -(-(m.heads // m.kv_heads) // 16)
         splits = max(1, min(32, -(-3 * 148 // ctas), -(-reach // 128)))
     ws = _workspace(q.device, B * m.heads * splits * (m.vdim + 2)) if splits > 1 else None
     f = _lib.fn("dlti_attn_paged_decode", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _I, _I, _I, _I, _I, _I, _F, _V, _I, _V, _V, _L, _V])
@@ -282,6 +293,22 @@ def attn_paged_prefill(q, m, rows: Rows, kc, vc, gate, out):
     _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], kc.shape[1],
                  _p(rows.ctx), _p(rows.cu), rows.nd, rows.nseq - rows.nd, rows.max_seqlen, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk,
                  m.scale, _p(gate), _p(out), out.stride(0), _lib.stream_ptr()), "attn_paged_prefill")
+    return out
+
+
+def packed_attention(qkv, m, rows: Rows, seg, kc, vc, gate):
+    """Attention of a step from packed [q | k | v] rows (qk_norm_rope_cache(packed=True)): decode rows through the pages,
+    prompt rows as independent causal pieces (seg = (boundaries, longest)) through the varlen tcgen05 kernel. Needs heads
+    of 128 and prompts whose visible keys all belong to this step."""
+    T, H = qkv.shape[0], m.heads
+    out = act(T, H * m.vdim, qkv.dtype, qkv.device)
+    nd = rows.nd
+    if nd:
+        attn_paged_decode(qkv[:nd, :H * m.dim], m, rows, kc, vc, gate, out)
+    q, o, g = qkv[nd:], out[nd:], None if gate is None else gate[nd:]
+    f = _lib.fn("dlti_attn_fwd_split", [_V, _V, _L, _V, _V, _I, _I, _L, _I, _I, _I, _F, _V])
+    _lib.check(f(_p(q), _p(o), o.stride(0), _p(g), _p(seg[0]), seg[0].numel() - 1, seg[1], T - nd, H, m.kv_heads, m.dim, m.scale,
+                 _lib.stream_ptr()), "attn_fwd_split")
     return out
 
 

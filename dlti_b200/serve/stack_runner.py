@@ -6,12 +6,19 @@ outputs only, so every sublayer reads the residual itself: the fp32 stream and, 
 the norm-and-add kernel writes next to it."""
 from __future__ import annotations
 
+import os
+
 import torch
 
 from ..models.stack import AttentionMixer, LightningMixer, Mamba2Mixer, StackConfig, StackWeights, mixer_sections, round8
 from ..ops import _lib
 from ..ops import stack as K
+from ..ops.gemm import gemm_skinny_acc
 from .kv_cache import KVCache, KVSpec, StateCache, StateSpec
+
+
+_FUSE_ACC = os.environ.get("DLTI_DECODE_FUSE_ACC", "1") == "1"    # A/B switch: consume the fp32 accumulators directly
+_PACKED_FROM = 64            # longest piece of a step from which the packed prefill kernel pays
 
 
 class StackRunner:
@@ -38,6 +45,9 @@ class StackRunner:
         self.sections = [mixer_sections(l.mixer) for l in cfg.layers]
         self.ropes = [K.rope_tables(max_len, l.mixer.rope.dims, l.mixer.rope.base, self.device)
                       if isinstance(l.mixer, AttentionMixer) and l.mixer.rope is not None else None for l in cfg.layers]
+        if self.device.type == "cuda" and "DLTI_PDL" not in os.environ:
+            # serving weights are static: the decode GEMMs may fetch weight tiles while the previous kernel drains
+            _lib.gpu_lib().dlti_set_pdl(2)
         self.trace = None            # set to a list: receives the residual stream after every layer (debugging)
 
     @torch.no_grad()
@@ -49,6 +59,9 @@ class StackRunner:
         rows = K.Rows(positions, row_seq, slots, ctx_lens, cu_seqlens, block_tables, state_slots, int(num_decode), max_seqlen,
                       max_ctx)
         x, xa = K.embed_rows(input_ids.view(-1), w.embed)
+        # decode-sized steps stream the weights through the stream-K GEMM; the next op consumes its fp32 accumulator
+        self.acc = acc = _FUSE_ACC and x.is_cuda and self.dtype == torch.bfloat16 and x.shape[0] <= 256
+        mm = gemm_skinny_acc if acc else K.linear
         for i, (l, lw) in enumerate(zip(cfg.layers, w.layers)):
             m = l.mixer
             if isinstance(m, AttentionMixer):
@@ -57,31 +70,41 @@ class StackRunner:
                 y = self._mamba2(i, m, lw, xa, rows)
             else:
                 y = self._lightning(i, m, lw, xa, rows)
-            xa = self._close(K.linear(y, lw["w_out"]), x, lw["norm1"])
+            xa = self._close(mm(y, lw["w_out"]), x, lw["norm1"])
             if l.mlp is not None:
-                h = K.relu2(K.linear(xa, lw["w_up"]), l.mlp.ff, self.dtype)
-                xa = self._close(K.linear(h, lw["w_down"]), x, lw["norm2"])
+                h = K.relu2(mm(xa, lw["w_up"]), l.mlp.ff, self.dtype, acc=acc)
+                xa = self._close(mm(h, lw["w_down"]), x, lw["norm2"])
             if self.trace is not None:
                 self.trace.append(x.clone())
         if last_idx is not None and last_idx.numel() == 0:
             return torch.empty((0, cfg.vocab_size), dtype=torch.float32, device=self.device)
         xn = K.rms_rows(x, last_idx, w.final_norm, cfg.norm_eps, cfg.norm_one_plus, self.dtype)
-        return K.linear(xn, w.lm_head, out_dtype=torch.float32)[:, :cfg.vocab_size]
+        return K.linear_f32(xn, w.lm_head)[:, :cfg.vocab_size]
 
     def _close(self, y, x, norm):
         """End of a sublayer: x += norm(y); returns the next sublayer's input."""
-        return K.post_norm_add_(y, x, norm, self.cfg.norm_eps, self.cfg.norm_one_plus, self.dtype)
+        return K.post_norm_add_(y, x, norm, self.cfg.norm_eps, self.cfg.norm_one_plus, self.dtype, acc=self.acc)
 
     def _attention(self, i, m: AttentionMixer, lw, xa, rows: K.Rows, segs):
-        q, gate = K.qk_norm_rope_cache(K.linear(xa, lw["w_in"]), self.sections[i], m, lw.get("q_norm"), lw.get("k_norm"),
-                                       self.cfg.norm_eps, rows, self.ropes[i], self.kv.k[i], self.kv.v[i], self.dtype)
+        seg = (segs or {}).get(m.chunk)
+        # whole prompts with heads of 128: the varlen tcgen05 kernel on rows cut at the chunk edges; everything else
+        # (portions that continue a chunk, other head sizes, fp32) reads the pages
+        packed = (seg is not None and seg[0].numel() > 1 and m.dim == m.vdim == 128 and self.dtype == torch.bfloat16
+                  and seg[1] >= _PACKED_FROM and xa.is_cuda)
+        proj = gemm_skinny_acc(xa, lw["w_in"]) if self.acc else K.linear(xa, lw["w_in"])
+        q, gate = K.qk_norm_rope_cache(proj, self.sections[i], m, lw.get("q_norm"), lw.get("k_norm"), self.cfg.norm_eps, rows,
+                                       self.ropes[i], self.kv.k[i], self.kv.v[i], self.dtype, packed=packed, acc=self.acc)
+        if packed:
+            return K.packed_attention(q, m, rows, seg, self.kv.k[i], self.kv.v[i], gate)
         return K.paged_attention(q, m, rows, self.kv.k[i], self.kv.v[i], gate)
 
     def _mamba2(self, i, m: Mamba2Mixer, lw, xa, rows: K.Rows):
         s, st = self.sections[i], self.states
         inner, gn = m.inner, m.groups * m.state
-        proj = K.linear(xa, lw["w_in"])
-        xbc, proj = K.short_conv(proj, s["xbc"], m.conv_channels, lw["conv"], lw["conv_b"], st.conv[i], rows, self.dtype)
+        acc = self.acc and rows.nd == xa.shape[0]                 # the convolution of prompt rows reads its neighbours' inputs
+        proj = gemm_skinny_acc(xa, lw["w_in"]) if acc else K.linear(xa, lw["w_in"])
+        xbc, proj = K.short_conv(proj, s["xbc"], m.conv_channels, lw["conv"], lw["conv_b"], st.conv[i], rows, self.dtype, acc=acc,
+                                 width=proj.shape[1])
         decay = K.Decay(dt=proj[:, s["dt"]:s["dt"] + m.heads], dt_bias=lw["dt_bias"], A_log=lw["A_log"], D=lw["D"])
         y = K.linear_scan(xbc[:, inner + gn:], xbc[:, inner:inner + gn], xbc[:, :inner], decay, st.ssm[i], rows, m.heads, m.groups,
                           m.state, m.vdim, conv_src=proj, conv_col=s["xbc"], conv_state=st.conv[i])
