@@ -21,7 +21,7 @@ magnitude, so no explicit L2 flush is needed between iterations ("inputs larger 
 
 `--impl reference` must run the unmodified reference; it is not installable here (no setup.py /
 pyproject; it needs deepspeed + peft + accelerate, absent from the image and from /opt/wheelhouse),
-so that arm prints {"impl": "reference", "unavailable": ...} and exits 0 (DESIGN.md §Reference arm).
+so that arm prints {"impl": "reference", "unavailable": ...} and exits 0.
 `--impl standin` runs the stock-PyTorch (cuBLAS + SDPA + NCCL) restatement under baseline/.
 """
 from __future__ import annotations
@@ -55,11 +55,15 @@ def parse():
     ap.add_argument("--offload", action="store_true",
                     help="run the ds_config as shipped (ZeRO-Offload of optimizer state and parameters to pinned host "
                          "memory) instead of the HBM-resident default; a secondary measurement, not the headline (689 ms vs 631 ms per step on one B200)")
+    ap.add_argument("--workload", default="train", choices=["train", "sigosun"],
+                    help="train: the headline benchmark (default). sigosun: prefill and decode throughput of the Sigosun family "
+                         "beside Llama models of equal size, with every kernel's fraction of its roofline (1 GPU)")
+    ap.add_argument("--sizes", default="2048x4,4096x2", help="--workload sigosun: width x groups of four layers, comma-separated")
     return ap.parse_args()
 
 
 class ClockSampler:
-    """nvidia-smi clocks / throttle reasons sampled DURING the timed region (B200_PROFILING.md)."""
+    """nvidia-smi clocks / throttle reasons sampled DURING the timed region."""
     Q = ("index,clocks.sm,clocks.max.sm,power.draw,clocks_event_reasons.active,"
          "clocks_event_reasons.hw_slowdown,clocks_event_reasons.hw_thermal_slowdown,"
          "clocks_event_reasons.sw_thermal_slowdown,clocks_event_reasons.sw_power_cap")
@@ -121,6 +125,14 @@ def main() -> None:
     a = parse()
     if a.impl == "reference":
         reference_arm(a)
+        return
+    if a.workload == "sigosun":
+        from dlti_b200.serve import layer_bench
+        try:
+            peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
+        except OSError:
+            peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+        layer_bench.run_cli(a.steps, a.warmup, a.sizes, peaks, ClockSampler(0))
         return
     if a.impl == "standin":
         sys.path.insert(0, os.path.join(ROOT, "baseline"))

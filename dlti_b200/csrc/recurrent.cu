@@ -170,9 +170,9 @@ int launch_scan(const ScanParams& p, int nseq, cudaStream_t st) {
     dlti_count_launch();                                                                                                      \
     return 0;                                                                                                                 \
   }
-  SCAN_CASE(4) SCAN_CASE(8) SCAN_CASE(16) SCAN_CASE(32)
+  SCAN_CASE(4) SCAN_CASE(8) SCAN_CASE(16) SCAN_CASE(32) SCAN_CASE(64)
 #undef SCAN_CASE
-  dlti_set_error("linear_scan: states of up to 256 rows");
+  dlti_set_error("linear_scan: states of up to 512 rows");
   return DLTI_ERR_TOO_LARGE;
 }
 

@@ -1,0 +1,329 @@
+"""Serving throughput of the Sigosun family beside Llama models of equal size, and the time of each kernel of the two
+against its roofline (`bench.py --workload sigosun`). Random weights; layer sizes of real models.
+
+Steps go through LLMEngine.pack_step / _run_step (packing, host-to-device copy, forward, sampling; decode steps replay
+CUDA graphs), timed with CUDA events. Kernels are timed one call at a time with the L2 overwritten before each."""
+from __future__ import annotations
+
+import json
+import statistics
+from dataclasses import replace
+
+import torch
+
+from ..models.config import LlamaConfig
+from ..models.registry import family_of
+from ..models.sigosun import SigosunConfig
+from ..models.stack import AttentionMixer, DenseMlp, Layer, LightningMixer, Mamba2Mixer, Rope, mixer_sections
+from ..ops import _lib
+from ..ops import attention as A
+from ..ops import elementwise as E
+from ..ops import serving as S
+from ..ops import stack as K
+from ..ops.gemm import gemm, gemm_skinny, gemm_skinny_acc
+from .engine import LLMEngine
+from .model_runner import TPContext
+from .tokenizer import ByteTokenizer
+
+
+def _sigosun(width: int, blocks: int) -> SigosunConfig:
+    heads = width // 128
+    att = AttentionMixer(heads=heads, kv_heads=max(1, heads // 4), dim=128, vdim=128, scale=128 ** -0.5, rope=Rope(128, 5e5), chunk=2048)
+    mam = Mamba2Mixer(heads=width // 32, vdim=64, state=128, groups=1, conv=4, norm_groups=1)
+    lig = LightningMixer(heads=heads, dim=128, vdim=128, decay=tuple(1 - 2.0 ** (-4 - h * 5 / heads) for h in range(heads)))
+    ff = DenseMlp(4 * width)
+    layers = []
+    for b in range(blocks):
+        layers += [Layer(att, ff), Layer(replace(att, kv_from=4 * b), ff), Layer(mam, None), Layer(lig, None)]
+    return SigosunConfig(hidden_size=width, vocab_size=32000, norm_eps=1e-6, layers=layers, name=f"sigosun-{width}x{4 * blocks}")
+
+
+def _llama(width: int, params: int) -> LlamaConfig:
+    """The Llama of the same width whose layers hold about `params` parameters (same key/value head ratio)."""
+    heads = width // 128
+    c = LlamaConfig(hidden_size=width, intermediate_size=round(width * 2.6875 / 256) * 256, num_attention_heads=heads,
+                    num_key_value_heads=max(1, heads // 4), num_hidden_layers=1, max_position_embeddings=16384)
+    n = max(1, round(params / c.params_per_layer()))
+    return replace(c, num_hidden_layers=n, name=f"llama-{width}x{n}")
+
+
+def _engine(cfg, max_len: int, seqs: int):
+    w = family_of(cfg).random_weights(cfg, "cuda", torch.bfloat16, 0)
+    return LLMEngine(cfg, w, TPContext(), ByteTokenizer(cfg.vocab_size), num_blocks=seqs * (max_len // 16) + 64, max_num_seqs=seqs,
+                     max_num_batched_tokens=16384, max_model_len=max_len)
+
+
+def _time(fn, warmup: int, iters: int) -> float:
+    for _ in range(warmup):
+        fn()
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    for _ in range(iters):
+        fn()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) / iters
+
+
+def _greedy(n: int):
+    return ([0.0] * n, [0] * n, [1.0] * n, [0] * n)
+
+
+def prefill_ms(eng: LLMEngine, nseq: int, length: int, warmup: int, iters: int) -> float:
+    bs = eng.blocks.block_size
+    per = -(-length // bs)
+    T = nseq * length
+    ids = torch.randint(3, eng.cfg.vocab_size, (T,)).tolist()
+    pos = list(range(length)) * nseq
+    slots = [(i * per) * bs + p for i in range(nseq) for p in range(length)]
+    tabs = [list(range(i * per, (i + 1) * per)) for i in range(nseq)]
+    cu = [i * length for i in range(nseq + 1)]
+    full = eng.per_sequence
+    step = lambda: eng.pack_step(0, ids, pos, slots, [length] * nseq if full else [], tabs if full else [], cu, length, _greedy(nseq),
+                                 sslots=list(range(nseq)), starts=[0] * nseq)
+    return _time(lambda: eng._run_step(step()), warmup, iters)
+
+
+def decode_ms(eng: LLMEngine, batch: int, ctx: int, warmup: int, iters: int) -> float:
+    bs = eng.blocks.block_size
+    per = -(-(ctx + 1) // bs)
+    tabs = [list(range(i * per, (i + 1) * per)) for i in range(batch)]
+    slots = [t[ctx // bs] * bs + ctx % bs for t in tabs]
+    step = lambda: eng.pack_step(batch, [5] * batch, [ctx] * batch, slots, [ctx + 1] * batch, tabs, [], 0, _greedy(batch),
+                                 sslots=list(range(batch)))
+    return _time(lambda: eng._run_step(step()), warmup, iters)
+
+
+def step_bytes(eng: LLMEngine, batch: int, ctx: int) -> int:
+    """What a decode step must move: every matrix once, the visible keys and values, recurrent states read and written."""
+    cfg, w = eng.cfg, eng.w
+    size = lambda t: t.numel() * t.element_size()
+    n = sum(size(t) for l in w.layers for t in l.values()) + size(w.lm_head)
+    if not eng.per_sequence:
+        return n + 2 * 2 * cfg.num_hidden_layers * batch * (ctx + 1) * w.KV * cfg.head_dim
+    for i, l in enumerate(cfg.layers):
+        m = l.mixer
+        if isinstance(m, AttentionMixer):
+            seen = ctx + 1 - (ctx // m.chunk * m.chunk if m.chunk else 0)
+            n += 2 * batch * seen * m.kv_heads * (m.dim + m.vdim)
+        else:
+            n += 2 * batch * 4 * eng.states.ssm[i][0].numel()
+    return n
+
+
+# ---- kernels -----------------------------------------------------------------------------------------------
+class _Kernels:
+    def __init__(self, peaks: dict, iters: int):
+        self.hbm, self.flops, self.iters = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12, iters
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+        self.rows: list[dict] = []
+
+    def run(self, model: str, phase: str, name: str, fn, nbytes: float, flops: float = 0.0):
+        for _ in range(3):
+            fn()
+        ts = []
+        for _ in range(self.iters):
+            self.flush.fill_(1)
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1) * 1e3)
+        us = statistics.median(ts)
+        roof = max(nbytes / self.hbm, flops / self.flops) * 1e6
+        self.rows.append({"model": model, "phase": phase, "kernel": name, "us": round(us, 2), "roof_us": round(roof, 2),
+                          "frac_of_roof": round(roof / us, 3), "bound": "flops" if flops / self.flops > nbytes / self.hbm else "bytes"})
+
+
+def _rows(lens, nd, tables, slots, max_ctx):
+    i32 = dict(dtype=torch.int32, device="cuda")
+    cu = [0]
+    for s, n in lens[nd:]:
+        cu.append(cu[-1] + n)
+    return K.Rows(torch.cat([torch.arange(s, s + n) for s, n in lens]).to(**i32),
+                  torch.cat([torch.full((n,), i) for i, (s, n) in enumerate(lens)]).to(**i32), slots,
+                  torch.tensor([s + n for s, n in lens], **i32), torch.tensor(cu, **i32) if len(cu) > 1 else None, tables,
+                  torch.arange(len(lens), **i32), nd, max([n for _, n in lens[nd:]], default=0), max_ctx)
+
+
+def kernels(width: int, peaks: dict, nseq: int, length: int, batch: int, ctx: int, iters: int) -> list[dict]:
+    """Each kernel of a prefill step of nseq prompts of `length` and of a decode step of `batch` rows at context ctx."""
+    k = _Kernels(peaks, iters)
+    cfg = _sigosun(width, 1)
+    att, mam, lig = cfg.layers[0].mixer, cfg.layers[2].mixer, cfg.layers[3].mixer
+    ll = _llama(width, 1)
+    dev, bf = "cuda", torch.bfloat16
+    H, G, hd, d = att.heads, att.kv_heads, 128, width
+    rnd = lambda *s: torch.randn(*s, device=dev, dtype=bf)
+    T, bs = nseq * length, 16
+    per = -(-max(length, ctx + 1) // bs)
+    n_all = max(nseq, batch)
+    tabs = torch.arange(n_all * per, dtype=torch.int32, device=dev).view(n_all, per)
+    kc, vc = rnd(n_all * per, bs, G, hd), rnd(n_all * per, bs, G, hd)
+    fa, qn = torch.ones(hd, device=dev), torch.ones(d, device=dev)
+    tab_r = K.rope_tables(max(length, ctx + 1), hd, 5e5, dev)
+    cos, sin = E.rope_tables(max(length, ctx + 1), hd, 5e5, dev)
+    sec = mixer_sections(att)
+    pslots = torch.cat([torch.arange(length) + i * per * bs for i in range(nseq)]).to(dev)
+    dslots = torch.tensor([i * per * bs + ctx for i in range(batch)], device=dev)
+    pr = _rows([(0, length)] * nseq, 0, tabs[:nseq].contiguous(), pslots, length)
+    dr = _rows([(ctx, 1)] * batch, batch, tabs[:batch].contiguous(), dslots, ctx + 1)
+    seen = ctx + 1 - ctx // att.chunk * att.chunk
+
+    def pairs(n, c):                                        # visible (query, key) pairs of one prompt
+        c = min(c or n, n)
+        full, rest = divmod(n, c)
+        return full * c * (c + 1) // 2 + rest * (rest + 1) // 2
+
+    # attention, whole prompts: the same number of visible pairs for both (Llama sees pieces of `chunk` as prompts)
+    cut = [i * length + s for i in range(nseq) for s in range(0, length, att.chunk)] + [T]
+    seg = (torch.tensor(cut, dtype=torch.int32, device=dev), min(length, att.chunk))
+    qkv, gate = rnd(T, (H + 2 * G) * hd), torch.rand(T, H, device=dev)
+    fl = 4.0 * nseq * pairs(length, att.chunk) * H * hd
+    io = T * (2 * H + 2 * G) * hd * 2
+    k.run("sigosun", "prefill", "attention (packed)", lambda: K.packed_attention(qkv, att, pr, seg, kc, vc, gate), io, fl)
+    k.run("llama", "prefill", "attention", lambda: A.attention_fwd(qkv, seg[0], seg[1], H, G, hd, want_lse=False), io, fl)
+    q = rnd(T, H * hd)
+    out = K.act(T, H * hd, bf, dev)
+    k.run("sigosun", "prefill", "attention (portions, paged)", lambda: K.attn_paged_prefill(q, att, pr, kc, vc, gate, out), io, fl)
+    # attention, decode
+    qd, gd, od = rnd(batch, H * hd), torch.rand(batch, H, device=dev), K.act(batch, H * hd, bf, dev)
+    k.run("sigosun", "decode", "attention", lambda: K.attn_paged_decode(qd, att, dr, kc, vc, gd, od), batch * seen * G * hd * 4)
+    lens = torch.full((batch,), seen, dtype=torch.int32, device=dev)
+    k.run("llama", "decode", "attention", lambda: S.paged_decode(qd, kc, vc, dr.tables, lens, H, G, hd, max_ctx=seen), batch * seen * G * hd * 4)
+    # projection rows -> rotated q, cache
+    for phase, r, n in (("prefill", pr, T), ("decode", dr, batch)):
+        acc = phase == "decode"
+        proj = torch.zeros(n, sec.total, device=dev) if acc else rnd(n, sec.total)
+        k.run("sigosun", phase, "q/k norm + rope + cache", lambda: K.qk_norm_rope_cache(
+            proj, sec, att, fa, fa, 1e-6, r, tab_r, kc, vc, bf, packed=not acc, acc=acc),
+            n * (sec.total * (8 if acc else 2) + (H + (0 if acc else 2 * G)) * hd * 2 + 2 * G * hd * 2 + 4 * H))
+        W = (H + 2 * G) * hd
+        if acc:
+            accb = torch.zeros(n, W, device=dev)
+            k.run("llama", phase, "rope + cache", lambda: S.acc_rope_cache(accb, bf, r.pos, cos, sin, r.slots, kc, vc, H, G, hd),
+                  n * (W * 10 + 2 * G * hd * 2))
+        else:
+            k.run("llama", phase, "rope + cache", lambda: S.rope_cache_(qkv, r.pos, cos, sin, r.slots, kc, vc, H, G, hd),
+                  n * ((H + G) * hd * 4 + G * hd * 2 + 2 * G * hd * 2))
+        # residual + norm
+        x, w16 = torch.randn(n, d, device=dev), torch.ones(d, device=dev, dtype=bf)
+        y = torch.zeros(n, d, device=dev) if acc else rnd(n, d)
+        k.run("sigosun", phase, "norm + residual", lambda: K.post_norm_add_(y, x, qn, 1e-6, True, bf, acc=acc),
+              n * d * ((8 if acc else 2) + 8 + 2))
+        res = rnd(n, d)
+        if acc:
+            k.run("llama", phase, "residual + norm", lambda: E.acc_add_rmsnorm(y, res, w16, 1e-6), n * d * (8 + 4 + 2))
+        else:
+            k.run("llama", phase, "residual + norm", lambda: E.rmsnorm_fwd(y, w16, 1e-6, residual=res), n * d * (2 + 4 + 2))
+        # activation
+        ff, lf = cfg.layers[0].mlp.ff, ll.intermediate_size
+        u = torch.zeros(n, ff, device=dev) if acc else rnd(n, ff)
+        k.run("sigosun", phase, "relu^2", lambda: K.relu2(u, ff, bf, acc=acc), n * ff * ((8 if acc else 2) + 2))
+        gu = torch.zeros(n, 2 * lf, device=dev) if acc else rnd(n, 2 * lf)
+        if acc:
+            k.run("llama", phase, "swiglu", lambda: E.acc_swiglu(gu, bf), n * lf * 18)
+        else:
+            k.run("llama", phase, "swiglu", lambda: E.swiglu_fwd(gu), n * lf * 6)
+    del qkv, q, out, u, gu
+    # GEMMs (the same kernels in both models)
+    for phase, n in (("prefill", T), ("decode", batch)):
+        mm = gemm if phase == "prefill" else gemm_skinny_acc
+        for model, name, N_, K_ in (("sigosun", "GEMM attention in", sec.total, d), ("llama", "GEMM qkv", (H + 2 * G) * hd, d),
+                                    ("sigosun", "GEMM mamba2 in", mixer_sections(mam).total, d),
+                                    ("sigosun", "GEMM lightning in", mixer_sections(lig).total, d),
+                                    ("sigosun", "GEMM up", 4 * d, d), ("llama", "GEMM gate_up", 2 * ll.intermediate_size, d),
+                                    ("sigosun", "GEMM down", d, 4 * d), ("llama", "GEMM down", d, ll.intermediate_size)):
+            a, b = rnd(n, K_), rnd(N_, K_)
+            k.run(model, phase, name, lambda: mm(a, b), 2 * (n * K_ + N_ * K_) + n * N_ * (2 if phase == "prefill" else 4), 2.0 * n * N_ * K_)
+            if phase == "decode":
+                gemm_skinny(a, b)                         # leaves the shared accumulator zero
+    # recurrent layers
+    sm, sl = mixer_sections(mam), mixer_sections(lig)
+    inner, gn, C = mam.inner, mam.groups * mam.state, mam.conv_channels
+    cw, cb = torch.rand(mam.conv, C, device=dev), torch.zeros(C, device=dev)
+    for phase, r, n, ns in (("prefill", pr, T, nseq), ("decode", dr, batch, batch)):
+        conv = torch.zeros(ns, mam.conv - 1, C, device=dev, dtype=bf)
+        ssm = torch.zeros(ns, mam.heads, mam.state, mam.vdim, device=dev)
+        acc = phase == "decode"
+        proj = torch.zeros(n, sm.total, device=dev) if acc else rnd(n, sm.total)
+        k.run("sigosun", phase, "short conv", lambda: K.short_conv(proj, sm["xbc"], C, cw, cb, conv, r, bf, acc=acc, width=sm.total),
+              n * (sm.total * 10 + C * 2 + (mam.conv - 1) * C * 2) if acc else n * C * 4)
+        p16, xbc = rnd(n, sm.total), rnd(n, C)
+        dec = K.Decay(dt=p16[:, sm["dt"]:sm["dt"] + mam.heads], dt_bias=torch.full((mam.heads,), -4.0, device=dev),
+                      A_log=torch.zeros(mam.heads, device=dev), D=torch.ones(mam.heads, device=dev))
+        q64 = 64
+        work = lambda h, N_, P_: 2.0 * n * h * (q64 * (N_ + P_) / 2 + 2 * N_ * P_) if phase == "prefill" else 4.0 * n * h * N_ * P_
+        k.run("sigosun", phase, "mamba2 scan", lambda: K.linear_scan(
+            xbc[:, inner + gn:], xbc[:, inner:inner + gn], xbc[:, :inner], dec, ssm, r, mam.heads, mam.groups, mam.state, mam.vdim,
+            conv_src=p16, conv_col=sm["xbc"], conv_state=conv),
+            n * (C + inner + mam.heads) * 2 + ns * 8 * ssm[0].numel(), work(mam.heads, mam.state, mam.vdim))
+        yb = rnd(n, inner)
+        k.run("sigosun", phase, "gated norm (mamba2)", lambda: K.gated_norm(yb, p16[:, :inner], torch.ones(inner, device=dev), 1e-6, 1, True),
+              n * inner * 6)
+        pl = rnd(n, sl.total)
+        st = torch.zeros(ns, lig.heads, lig.dim, lig.vdim, device=dev)
+        qk, vv = lig.heads * lig.dim, lig.heads * lig.vdim
+        dl = K.Decay(const=torch.tensor(lig.decay, device=dev))
+        k.run("sigosun", phase, "lightning silu + scan", lambda: K.linear_scan(
+            pl[:, :qk], pl[:, sl["k"]:sl["k"] + qk], pl[:, sl["v"]:sl["v"] + vv], dl, st, r, lig.heads, lig.heads, lig.dim, lig.vdim,
+            silu=True), n * (2 * qk + 2 * vv) * 2 + ns * 8 * st[0].numel(), work(lig.heads, lig.dim, lig.vdim))
+        k.run("sigosun", phase, "gated norm (lightning)", lambda: K.gated_norm(pl[:, :vv], pl[:, sl["g"]:sl["g"] + vv],
+                                                                              torch.ones(vv, device=dev), 1e-6, 1, False), n * vv * 6)
+    return k.rows
+
+
+def main(steps: int, warmup: int, sizes: str, peaks: dict, sampler) -> dict:
+    iters, warmup = max(3, steps), max(3, warmup)
+    out = {"metric": "Sigosun serving tok/s beside Llama of equal size", "impl": "dlti_b200", "dtype": "bf16",
+           "data": "synthetic (random token ids; random-init weights)", "steps": iters, "warmup": warmup, "sizes": [], "kernels": {}}
+    _lib.reset_launch_count()
+    for spec in sizes.split(","):
+        width, blocks = (int(x) for x in spec.split("x"))
+        sig = _sigosun(width, blocks)
+        lla = _llama(width, sig.num_params() - 2 * sig.vocab_size * width)
+        row = {"width": width, "rows": []}
+        for cfg in (sig, lla):
+            eng = _engine(cfg, 8704, 64)
+            e = {"model": cfg.name, "layers": cfg.num_hidden_layers, "params_m": round(cfg.num_params() / 1e6)}
+            for nseq, length in ((1, 8192), (4, 2048), (16, 512)):
+                ms = prefill_ms(eng, nseq, length, warmup, iters)
+                e[f"prefill {nseq}x{length}"] = {"ms": round(ms, 3), "tok_s": round(nseq * length / ms * 1e3)}
+            for batch, ctx in ((1, 1000), (16, 1000), (64, 1000), (64, 8000)):
+                ms = decode_ms(eng, batch, ctx, warmup + 2, 4 * iters)
+                floor = step_bytes(eng, batch, ctx) / peaks["hbm_gbs"] / 1e6
+                e[f"decode {batch}@{ctx}"] = {"ms": round(ms, 3), "tok_s": round(batch / ms * 1e3), "frac_of_byte_floor": round(floor / ms, 3)}
+            row["rows"].append(e)
+            del eng
+            torch.cuda.empty_cache()
+        out["sizes"].append(row)
+        out["kernels"][str(width)] = kernels(width, peaks, 4, 2048, 64, 1000, iters)
+        torch.cuda.empty_cache()
+    out["gpu_launches"] = _lib.launch_count()
+    out["clocks"] = sampler.stop()
+    out["config"] = {"sizes": sizes, "l2": "steps: weights larger than L2 or streamed once per step; kernels: L2 overwritten before every call",
+                     "peaks": {k: peaks[k] for k in ("hbm_gbs", "bf16_tflops")}}
+    return out
+
+
+def print_tables(out: dict, emit=print) -> None:
+    for s in out["sizes"]:
+        a, b = s["rows"]
+        emit(f"# {a['model']} ({a['params_m']} M) | {b['model']} ({b['params_m']} M)")
+        for key in a:
+            if isinstance(a[key], dict):
+                emit(f"{key:20s} {a[key]['ms']:9.3f} ms {a[key]['tok_s']:9d} tok/s | {b[key]['ms']:9.3f} ms {b[key]['tok_s']:9d} tok/s | "
+                     f"{a[key].get('frac_of_byte_floor', '')} {b[key].get('frac_of_byte_floor', '')}")
+    for w, rows in out["kernels"].items():
+        emit(f"# kernels, width {w}")
+        for r in rows:
+            emit(f"{r['model']:8s} {r['phase']:8s} {r['kernel']:30s} {r['us']:9.2f} us, roof {r['roof_us']:8.2f} us = {r['frac_of_roof']:.3f} ({r['bound']})")
+
+
+def run_cli(steps: int, warmup: int, sizes: str, peaks: dict, sampler) -> None:
+    out = main(steps, warmup, sizes, peaks, sampler)
+    import sys
+    print_tables(out, lambda s: print(s, file=sys.stderr))
+    print(json.dumps(out))
