@@ -188,7 +188,7 @@ template <int NT>
 struct ChunkSmem {
   static constexpr int NP = NT + 8;
   static constexpr int QK = CQ * NP * 2, V = CQ * CPP * 2, STAGE = 2 * QK + V;          // bytes
-  static constexpr int W = 2 * STAGE, S = W + 2 * V, VEC = S + 2 * NT * CPP * 2, BYTES = VEC + 3 * CQ * 4 + 16;
+  static constexpr int W = 2 * STAGE, S = W + 2 * V, VEC = S + 2 * NT * CPP * 2, BYTES = VEC + 5 * CQ * 4;
 };
 template <int NT>
 __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int slices, int conv_parts) {
@@ -201,9 +201,11 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
   }
   extern __shared__ __align__(128) uint8_t smem[];
   const uint32_t sb = smem_u32(smem);
-  float* sL = reinterpret_cast<float*>(smem + L::VEC);          // running log decay
+  float* sHalf = reinterpret_cast<float*>(smem + L::VEC);       // running log2 decay inside each half of the chunk
+  float* sL = sHalf + CQ;                                       // ... of the whole chunk
   float* sStep = sL + CQ;
-  float* sE = sStep + CQ;                                       // exp(L_63 - L_s) * step
+  float* sE = sStep + CQ;                                       // 2^(L_63 - L_s) * step
+  float* sF = sE + CQ;                                          // 2^(L_e - L_s) * step, e = last token of s's 16-block
   long long row0;
   int n, start;
   seq_rows(p, s, row0, n, start);
@@ -213,26 +215,35 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
   const bf16* q = reinterpret_cast<const bf16*>(p.q) + row0 * p.q_ld + (long long)grp * p.N;
   const bf16* k = reinterpret_cast<const bf16*>(p.k) + row0 * p.k_ld + (long long)grp * p.N;
   const bf16* v = reinterpret_cast<const bf16*>(p.v) + row0 * p.v_ld + (long long)h * p.P + c0;
-  const float eA = p.decay ? 0.f : expf(p.A_log[h]);
-  const float la_c = p.decay ? fmaxf(logf(p.decay[h]), -80.f) : 0.f;
+  constexpr float LOG2E = 1.4426950408889634f;
+  const float eA = p.decay ? 0.f : expf(p.A_log[h]) * LOG2E;
+  const float la_c = p.decay ? fmaxf(logf(p.decay[h]), -80.f) * LOG2E : 0.f;
   const float bias = p.decay ? 0.f : p.dt_bias[h];
   const float Dh = p.D ? p.D[h] : 0.f;
 
   auto load = [&](int stage, int t0) {
+    constexpr int STEP = 128 / (NT / 8);                         // rows per pass
     const uint32_t base = sb + stage * L::STAGE;
-    const int nc = p.N >> 3, vc = ncol >> 3;
-    for (int i = threadIdx.x; i < CQ * (NT / 8); i += 128) {
-      const int r = i / (NT / 8), c = i % (NT / 8);
-      const bool ok = t0 + r < n && c < nc;
-      const long long row = ok ? t0 + r : 0;
-      const int cc = ok ? c * 8 : 0;
-      cp_async16(base + (r * L::NP + c * 8) * 2, q + row * p.q_ld + cc, ok);
-      cp_async16(base + L::QK + (r * L::NP + c * 8) * 2, k + row * p.k_ld + cc, ok);
+    const int r0 = threadIdx.x / (NT / 8), c = threadIdx.x % (NT / 8);
+    {
+      const bool cok = c * 8 < p.N;
+      const bf16* qp = q + (t0 + r0) * p.q_ld + c * 8;           // never dereferenced where a row or column is out of range
+      const bf16* kp = k + (t0 + r0) * p.k_ld + c * 8;
+      const uint32_t dst = base + (r0 * L::NP + c * 8) * 2;
+#pragma unroll
+      for (int i = 0; i < CQ / STEP; ++i) {
+        const bool ok = cok && t0 + r0 + i * STEP < n;
+        cp_async16(dst + i * STEP * L::NP * 2, ok ? qp : q, ok);
+        cp_async16(dst + i * STEP * L::NP * 2 + L::QK, ok ? kp : k, ok);
+        qp += STEP * p.q_ld;
+        kp += STEP * p.k_ld;
+      }
     }
-    for (int i = threadIdx.x; i < CQ * (CP / 8); i += 128) {
-      const int r = i / (CP / 8), c = i % (CP / 8);
-      const bool ok = t0 + r < n && c < vc;
-      cp_async16(base + 2 * L::QK + (r * CPP + c * 8) * 2, v + (ok ? t0 + r : 0) * p.v_ld + (ok ? c * 8 : 0), ok);
+#pragma unroll
+    for (int i = 0; i < CQ * (CP / 8) / 128; ++i) {
+      const int r = threadIdx.x / (CP / 8) + i * (128 / (CP / 8)), cv = threadIdx.x % (CP / 8);
+      const bool ok = t0 + r < n && cv * 8 < ncol;
+      cp_async16(base + 2 * L::QK + (r * CPP + cv * 8) * 2, ok ? v + (t0 + r) * p.v_ld + cv * 8 : v, ok);
     }
     cp_async_commit();
   };
@@ -288,7 +299,7 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
         if (lane >= o) x += y;
       }
       sStep[threadIdx.x] = step;
-      sL[threadIdx.x] = x;                                       // sums inside each half of the chunk
+      sHalf[threadIdx.x] = x;
     }
     dt_next = raw_dt(t0 + CQ);
     __syncthreads();                                             // stage (it + 1) & 1 free; half sums, S operands visible
@@ -298,11 +309,13 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
     } else {
       cp_async_wait<0>();
     }
-    const float half = sL[31];
-    const float total = sL[CQ - 1] + half;
+    const float half = sHalf[31];
+    const float total = sHalf[CQ - 1] + half;
     if (threadIdx.x < CQ) {
-      const float l = sL[threadIdx.x] + (threadIdx.x >= 32 ? half : 0.f);
-      sE[threadIdx.x] = expf(total - l) * sStep[threadIdx.x];
+      const float l = sHalf[threadIdx.x], le = sHalf[threadIdx.x | 15], step = sStep[threadIdx.x];
+      sL[threadIdx.x] = l + (threadIdx.x >= 32 ? half : 0.f);
+      sE[threadIdx.x] = ex2(total - (l + (threadIdx.x >= 32 ? half : 0.f))) * step;
+      sF[threadIdx.x] = ex2(le - l) * step;
     }
     __syncthreads();                                             // tile landed, sE written
     const bf16* sv = reinterpret_cast<const bf16*>(smem + (it & 1) * L::STAGE + 2 * L::QK);
@@ -344,8 +357,8 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
     float lt[2], el[2];
 #pragma unroll
     for (int y = 0; y < 2; ++y) {
-      lt[y] = sL[tr + 8 * y] + (tr + 8 * y >= 32 ? half : 0.f);
-      el[y] = expf(lt[y]);
+      lt[y] = sL[tr + 8 * y];
+      el[y] = ex2(lt[y]);
     }
 #pragma unroll
     for (int j = 0; j < CP / 8; ++j)
@@ -361,13 +374,20 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
         mma_bf16(g0, qf[kk], b[0], b[1]);
         mma_bf16(g1, qf[kk], b[2], b[3]);
       }
+      if (kb < warp) {                                           // all keys precede all tokens: factored through the block's end
+        const float le = sL[kb * 16 + 15];
+        const float f0 = ex2(lt[0] - le), f1 = ex2(lt[1] - le);
+        const float2 a = *reinterpret_cast<const float2*>(sF + kb * 16 + scol), b = *reinterpret_cast<const float2*>(sF + kb * 16 + 8 + scol);
+        g0[0] *= a.x * f0; g0[1] *= a.y * f0; g0[2] *= a.x * f1; g0[3] *= a.y * f1;
+        g1[0] *= b.x * f0; g1[1] *= b.y * f0; g1[2] *= b.x * f1; g1[3] *= b.y * f1;
+      } else {
 #pragma unroll
-      for (int x = 0; x < 4; ++x) {
-        const int t = tr + 8 * (x >> 1);
-        const int u0 = kb * 16 + scol + (x & 1), u1 = u0 + 8;
-        const float l0 = sL[u0] + (u0 >= 32 ? half : 0.f), l1 = sL[u1] + (u1 >= 32 ? half : 0.f);
-        g0[x] = u0 <= t ? g0[x] * sStep[u0] * expf(lt[x >> 1] - l0) : 0.f;
-        g1[x] = u1 <= t ? g1[x] * sStep[u1] * expf(lt[x >> 1] - l1) : 0.f;
+        for (int x = 0; x < 4; ++x) {
+          const int t = tr + 8 * (x >> 1);
+          const int u0 = kb * 16 + scol + (x & 1), u1 = u0 + 8;
+          g0[x] = u0 <= t ? g0[x] * sStep[u0] * ex2(lt[x >> 1] - sL[u0]) : 0.f;
+          g1[x] = u1 <= t ? g1[x] * sStep[u1] * ex2(lt[x >> 1] - sL[u1]) : 0.f;
+        }
       }
       uint32_t hi[4], lo[4];
       split_pair(g0[0], g0[1], hi[0], lo[0]);
@@ -401,7 +421,7 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
     }
     __syncthreads();                                             // scaled values written; old S operands no longer read
     // ---- state ----
-    const float keep = expf(total);
+    const float keep = ex2(total);
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
@@ -467,13 +487,19 @@ int launch_chunk(const ScanParams& p, int nseq, cudaStream_t st) {
 // x = silu(x) in place, rounded to T
 template <typename T>
 __global__ void silu_rows_kernel(T* __restrict__ x, long long ld, long long rows, int n) {
-  const int pairs = n >> 1;
-  const long long total = rows * pairs;
+  const int vec = n >> 3;
+  const long long total = rows * vec;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
-    const long long t = i / pairs;
-    uint32_t* p = reinterpret_cast<uint32_t*>(x + t * ld) + (int)(i - t * pairs);
-    const float2 f = Cvt<T>::unpack2(*p);
-    *p = Cvt<T>::pack2(silu_f(f.x), silu_f(f.y));
+    const long long t = i / vec;
+    int4* p = reinterpret_cast<int4*>(x + t * ld) + (int)(i - t * vec);
+    int4 v = *p;
+    uint32_t* u = reinterpret_cast<uint32_t*>(&v);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = Cvt<T>::unpack2(u[j]);
+      u[j] = Cvt<T>::pack2(f.x / (1.f + __expf(-f.x)), f.y / (1.f + __expf(-f.y)));
+    }
+    *p = v;
   }
 }
 
@@ -524,8 +550,8 @@ DLTI_API int dlti_linear_scan_chunked(const void* q, long long q_ld, const void*
 DLTI_API int dlti_silu_rows(void* x, long long ld, long long rows, int n, int dtype, cudaStream_t st) {
   if (rows <= 0 || n <= 0) return 0;
   if (dtype != DLTI_BF16) return DLTI_ERR_UNSUPPORTED;
-  if (n % 2 || ld % 2) return DLTI_ERR_BAD_ARG;
-  const long long g = (rows * (n / 2) + 255) / 256, cap = (long long)dlti_num_sms() * 16;
+  if (n % 8 || ld % 8 || (reinterpret_cast<uintptr_t>(x) & 15)) return DLTI_ERR_BAD_ARG;
+  const long long g = (rows * (n / 8) + 255) / 256, cap = (long long)dlti_num_sms() * 16;
   silu_rows_kernel<__nv_bfloat16><<<(unsigned)(g < cap ? g : cap), 256, 0, st>>>((__nv_bfloat16*)x, ld, rows, n);
   dlti_count_launch();
   return (int)cudaGetLastError();

@@ -44,6 +44,62 @@ __device__ __forceinline__ void put2(T* row, long long i, float a, float b) {
   else *reinterpret_cast<float2*>(row + i) = make_float2(a, b);
 }
 
+// N (2, 4 or 8) consecutive elements at an offset that is a multiple of N
+template <typename T, bool ACC, int N>
+__device__ __forceinline__ void take_n(const void* row, long long i, float (&f)[N]) {
+  if constexpr (ACC) {
+    float* p = const_cast<float*>(reinterpret_cast<const float*>(row)) + i;
+    if constexpr (N == 2) {
+      const float2 v = *reinterpret_cast<float2*>(p);
+      *reinterpret_cast<float2*>(p) = make_float2(0.f, 0.f);
+      f[0] = round_to<T>(v.x); f[1] = round_to<T>(v.y);
+    } else {
+#pragma unroll
+      for (int j = 0; j < N / 4; ++j) {
+        const float4 v = reinterpret_cast<float4*>(p)[j];
+        reinterpret_cast<float4*>(p)[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        f[4 * j] = round_to<T>(v.x); f[4 * j + 1] = round_to<T>(v.y); f[4 * j + 2] = round_to<T>(v.z); f[4 * j + 3] = round_to<T>(v.w);
+      }
+    }
+  } else if constexpr (sizeof(T) == 2) {
+    const T* p = reinterpret_cast<const T*>(row) + i;
+    uint32_t u[N / 2];
+    if constexpr (N == 2) u[0] = *reinterpret_cast<const uint32_t*>(p);
+    else if constexpr (N == 4) *reinterpret_cast<uint2*>(u) = *reinterpret_cast<const uint2*>(p);
+    else *reinterpret_cast<uint4*>(u) = *reinterpret_cast<const uint4*>(p);
+#pragma unroll
+    for (int j = 0; j < N / 2; ++j) {
+      const float2 v = Cvt<T>::unpack2(u[j]);
+      f[2 * j] = v.x; f[2 * j + 1] = v.y;
+    }
+  } else {
+#pragma unroll
+    for (int j = 0; j < N; ++j) f[j] = reinterpret_cast<const float*>(row)[i + j];
+  }
+}
+template <typename T, int N>
+__device__ __forceinline__ void put_n(T* p, const float (&f)[N]) {
+  if constexpr (sizeof(T) == 2) {
+    uint32_t u[N / 2];
+#pragma unroll
+    for (int j = 0; j < N / 2; ++j) u[j] = Cvt<T>::pack2(f[2 * j], f[2 * j + 1]);
+    if constexpr (N == 2) *reinterpret_cast<uint32_t*>(p) = u[0];
+    else if constexpr (N == 4) *reinterpret_cast<uint2*>(p) = *reinterpret_cast<uint2*>(u);
+    else *reinterpret_cast<uint4*>(p) = *reinterpret_cast<uint4*>(u);
+  } else {
+#pragma unroll
+    for (int j = 0; j < N; ++j) p[j] = Cvt<T>::from_f(f[j]);
+  }
+}
+__device__ __forceinline__ void ld8(const float* p, float (&f)[8]) {
+  *reinterpret_cast<float4*>(f) = reinterpret_cast<const float4*>(p)[0];
+  *reinterpret_cast<float4*>(f + 4) = reinterpret_cast<const float4*>(p)[1];
+}
+__device__ __forceinline__ void st8(float* p, const float (&f)[8]) {
+  reinterpret_cast<float4*>(p)[0] = *reinterpret_cast<const float4*>(f);
+  reinterpret_cast<float4*>(p)[1] = *reinterpret_cast<const float4*>(f + 4);
+}
+
 __device__ __forceinline__ float block_sum(float v, float* red) {
   v = warp_sum(v);
   const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = blockDim.x >> 5;
@@ -122,6 +178,53 @@ __global__ void __launch_bounds__(PN_THREADS) post_norm_add_kernel(const void* _
   }
 }
 
+// the same in 16-byte pieces, every load issued before the reduction: 16-bit T, d and pitches multiples of 8
+template <typename T, bool ACC, int VPT>
+__global__ void __launch_bounds__(128) post_norm_add_vec_kernel(const void* __restrict__ y, long long y_ld, float* __restrict__ x,
+                                                               const float* __restrict__ w, T* __restrict__ xa, long long xa_ld,
+                                                               int d, float eps, float one) {
+  __shared__ float red[32];
+  const int vec = d >> 3;
+  float wv[VPT][8];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {                   // weights never change: they may come before the wait
+    const int v = threadIdx.x + i * 128;
+    if (v < vec) ld8(w + v * 8, wv[i]);
+  }
+  griddep_wait();
+  griddep_launch();
+  const long long row = blockIdx.x;
+  const void* yr = reinterpret_cast<const uint8_t*>(y) + row * y_ld * (ACC ? 4 : sizeof(T));
+  float* xr = x + row * d;
+  float yv[VPT][8], xv[VPT][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int v = threadIdx.x + i * 128;
+    if (v < vec) {
+      take_n<T, ACC, 8>(yr, v * 8, yv[i]);
+      ld8(xr + v * 8, xv[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i)
+    if (threadIdx.x + i * 128 < vec)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss += yv[i][j] * yv[i][j];
+  ss = block_sum(ss, red);
+  const float r = 1.f / sqrtf(ss / (float)d + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int v = threadIdx.x + i * 128;
+    if (v < vec) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) xv[i][j] += yv[i][j] * r * (one + wv[i][j]);
+      st8(xr + v * 8, xv[i]);
+      if (xa) put_n(xa + row * xa_ld + v * 8, xv[i]);
+    }
+  }
+}
+
 // out[i] = norm(x[idx[i]]) * w (or * (1 + w))
 template <typename T>
 __global__ void __launch_bounds__(PN_THREADS) rms_rows_kernel(const float* __restrict__ x, const long long* __restrict__ idx,
@@ -163,23 +266,23 @@ __global__ void relu2_kernel(const void* __restrict__ u, long long u_ld, T* __re
   }
 }
 // the same, 8 columns per thread (16-bit, both pitches and ff multiples of 8)
-template <typename T>
-__global__ void relu2_vec_kernel(const T* __restrict__ u, long long u_ld, T* __restrict__ h, long long h_ld, long long rows, int ff) {
+template <typename T, bool ACC>
+__global__ void relu2_vec_kernel(const void* __restrict__ u, long long u_ld, T* __restrict__ h, long long h_ld, long long rows, int ff) {
+  griddep_wait();
+  griddep_launch();
   const int vec = ff >> 3;
   const long long total = rows * vec;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
     const long long t = i / vec;
     const int c = 8 * (int)(i - t * vec);
-    int4 v = *reinterpret_cast<const int4*>(u + t * u_ld + c);
-    uint32_t* p = reinterpret_cast<uint32_t*>(&v);
+    float f[8];
+    take_n<T, ACC, 8>(reinterpret_cast<const uint8_t*>(u) + t * u_ld * (ACC ? 4 : sizeof(T)), c, f);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      float2 f = Cvt<T>::unpack2(p[j]);
-      f.x = fmaxf(f.x, 0.f);
-      f.y = fmaxf(f.y, 0.f);
-      p[j] = Cvt<T>::pack2(f.x * f.x, f.y * f.y);
+    for (int j = 0; j < 8; ++j) {
+      f[j] = fmaxf(f[j], 0.f);
+      f[j] *= f[j];
     }
-    *reinterpret_cast<int4*>(h + t * h_ld + c) = v;
+    put_n(h + t * h_ld + c, f);
   }
 }
 
@@ -228,6 +331,53 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const T* __restrict__ y
     for (int c = g * gs + (threadIdx.x & 31); c < (g + 1) * gs; c += 32) {
       const float v = (GATE_FIRST ? row_s[c] : Cvt<T>::to_f(yr[c]) * row_s[c]) * r * w[c];
       out[t * o_ld + c] = Cvt<T>::from_f(v);
+    }
+  }
+}
+
+// the same in 16-byte pieces for 16-bit T and groups of whole pieces: one CTA per (row, group), everything in registers
+template <typename T, bool GATE_FIRST, bool ACC, int VPT>
+__global__ void __launch_bounds__(256) gated_norm_vec_kernel(const T* __restrict__ y, long long y_ld, const void* __restrict__ gate,
+                                                             long long g_ld, const float* __restrict__ w, T* __restrict__ out,
+                                                             long long o_ld, int gs, float eps) {
+  __shared__ float red[32];
+  griddep_wait();
+  griddep_launch();
+  const long long t = blockIdx.x;
+  const int c0 = blockIdx.y * gs, vec = gs >> 3;
+  const T* yr = y + t * y_ld;
+  const void* gr = reinterpret_cast<const uint8_t*>(gate) + t * g_ld * (ACC ? 4 : sizeof(T));
+  float v[VPT][8], g[VPT][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int p = threadIdx.x + i * blockDim.x;
+    if (p < vec) {
+      take_n<T, false, 8>(yr, c0 + p * 8, v[i]);
+      take_n<T, ACC, 8>(gr, c0 + p * 8, g[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i)
+    if (threadIdx.x + i * blockDim.x < vec)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float e = 1.f / (1.f + __expf(-g[i][j]));
+        if (GATE_FIRST) v[i][j] *= g[i][j] * e;
+        else g[i][j] = e;
+        ss += v[i][j] * v[i][j];
+      }
+  ss = block_sum(ss, red);
+  const float r = 1.f / sqrtf(ss / (float)gs + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int p = threadIdx.x + i * blockDim.x;
+    if (p < vec) {
+      float wv[8];
+      ld8(w + c0 + p * 8, wv);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] *= r * wv[j] * (GATE_FIRST ? 1.f : g[i][j]);
+      put_n(out + t * o_ld + c0 + p * 8, v[i]);
     }
   }
 }
@@ -340,6 +490,84 @@ __global__ void __launch_bounds__(256) qk_norm_rope_cache_kernel(const QkvParams
   }
 }
 
+// The same for heads of 32 * VE (64, 128, 256) elements, interleaved pairs and 16-byte aligned sections: a lane owns VE
+// consecutive elements, so its rotation factors are the same for every head; a warp takes up to JPW jobs of one token and
+// issues their loads together.
+template <typename T, bool ACC, int VE, int JPW>
+__global__ void __launch_bounds__(256) qk_norm_rope_cache_vec_kernel(const QkvParams p, int jobs, int kvjobs) {
+  griddep_wait();
+  griddep_launch();
+  const int lane = threadIdx.x & 31;
+  const long long t = blockIdx.x;
+  const int job0 = (blockIdx.y * 8 + (threadIdx.x >> 5)) * JPW;
+  if (job0 >= jobs) return;
+  const uint8_t* row = reinterpret_cast<const uint8_t*>(p.proj) + t * p.ld * (ACC ? 4 : sizeof(T));
+  const long long slot = p.slots[t];
+  const bool own = p.ok >= 0;
+  const int e0 = lane * VE, half = p.rot >> 1;
+  float v[JPW][VE];
+#pragma unroll
+  for (int i = 0; i < JPW; ++i) {
+    const int job = job0 + i;
+    if (job < p.H) {
+      take_n<T, ACC, VE>(row, p.oq + job * (32 * VE) + e0, v[i]);
+    } else if (job < p.H + kvjobs) {
+      const int kh = job - p.H;                              // G keys, then G values
+      const bool is_k = kh < p.G;
+      const int g = is_k ? kh : kh - p.G;
+      if (own) take_n<T, ACC, VE>(row, (is_k ? p.ok : p.ov) + g * (32 * VE) + e0, v[i]);
+      else if (slot >= 0)
+        take_n<T, false, VE>(reinterpret_cast<const T*>(is_k ? p.kc : p.vc) + (slot * p.G + g) * (is_k ? p.kd : p.vd), e0, v[i]);
+      else
+#pragma unroll
+        for (int j = 0; j < VE; ++j) v[i][j] = 0.f;
+    }
+  }
+  float cs[VE / 2], sn[VE / 2];
+  const int ps = p.pos[t];
+#pragma unroll
+  for (int j = 0; j < VE / 2; ++j) {
+    const int pr = e0 / 2 + j;
+    cs[j] = pr < half ? p.cos_t[(long long)ps * half + pr] : 1.f;
+    sn[j] = pr < half ? p.sin_t[(long long)ps * half + pr] : 0.f;
+  }
+#pragma unroll
+  for (int i = 0; i < JPW; ++i) {
+    const int job = job0 + i;
+    if (job >= jobs) break;
+    if (job >= p.H + kvjobs) {
+      for (int h = lane; h < p.H; h += 32) p.gate[t * p.H + h] = sigmoid_f(take<T, ACC>(row, p.og + h));
+      break;
+    }
+    const bool is_q = job < p.H, is_v = job >= p.H + p.G;
+    const int g = is_q ? job : (is_v ? job - p.H - p.G : job - p.H);
+    if (is_q || (own && !is_v)) {
+      const float* nw = is_q ? p.qn : p.kn;
+      if (nw) {
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < VE; ++j) ss += v[i][j] * v[i][j];
+        const float r = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+#pragma unroll
+        for (int j = 0; j < VE; ++j) v[i][j] *= r * nw[e0 + j];
+      }
+#pragma unroll
+      for (int j = 0; j < VE / 2; ++j) {
+        const float a = v[i][2 * j], b = v[i][2 * j + 1];
+        v[i][2 * j] = a * cs[j] - b * sn[j];
+        v[i][2 * j + 1] = b * cs[j] + a * sn[j];
+      }
+    }
+    if (is_q) {
+      put_n(reinterpret_cast<T*>(p.q) + t * p.q_ld + (long long)g * p.q_hd + e0, v[i]);
+    } else {
+      void* pk = is_v ? p.vp : p.kp;
+      if (pk) put_n(reinterpret_cast<T*>(pk) + t * p.q_ld + (long long)g * p.q_hd + e0, v[i]);
+      if (own && slot >= 0) put_n(reinterpret_cast<T*>(is_v ? p.vc : p.kc) + (slot * p.G + g) * (is_v ? p.vd : p.kd) + e0, v[i]);
+    }
+  }
+}
+
 // Causal convolution of `taps` per channel + silu over the rows of every sequence of a step. src = projection rows
 // (channel 0 at column `col`); inputs from before the step come from conv_state [slots, taps - 1, C] (zero at position
 // 0). ACC additionally leaves the rounded projection row in `raw` (columns raw0 .. raw0 + raw_n): the gate, the step
@@ -401,6 +629,75 @@ __global__ void __launch_bounds__(256) short_conv_kernel(const ConvParams p) {
     if (two) o[1] = Cvt<T>::from_f(silu_f(a1));
   }
 }
+// The same, 8 channels x CONV_ROWS rows per thread with the window in registers (16-bit T, C and pitches multiples of 8,
+// TAPS fixed). Row blocks that touch the start of a sequence read rows or state tap by tap.
+constexpr int CONV_ROWS = 8;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) short_conv_vec_kernel(const ConvParams p) {
+  griddep_wait();
+  griddep_launch();
+  const int vec = p.C >> 3, cv = blockIdx.y * 128 + threadIdx.x;
+  if (cv >= vec) return;
+  const int c = cv * 8;
+  const long long t0 = (long long)blockIdx.x * CONV_ROWS;
+  const int nr = (int)min((long long)CONV_ROWS, p.rows - t0);
+  const T* src = reinterpret_cast<const T*>(p.src) + p.col + c;
+  const T* state = reinterpret_cast<const T*>(p.state) + c;
+  float w[TAPS][8], b[8];
+#pragma unroll
+  for (int k = 0; k < TAPS; ++k) ld8(p.w + (long long)k * p.w_ld + c, w[k]);
+  ld8(p.b + c, b);
+  T* out = reinterpret_cast<T*>(p.out) + c;
+  const int s0 = p.rseq[t0];
+  long long row0;
+  int n, start;
+  seq_rows(p.cu, p.ctx, p.nd, s0, row0, n, start);
+  auto emit = [&](long long t, const float (&a)[8]) {
+    float f[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) f[j] = a[j] / (1.f + __expf(-a[j]));
+    put_n(out + t * p.o_ld, f);
+  };
+  if (t0 - row0 >= TAPS - 1 && t0 + nr <= row0 + n) {            // all inputs are rows of this step
+    float x[TAPS - 1 + CONV_ROWS][8];
+#pragma unroll
+    for (int i = 0; i < TAPS - 1 + CONV_ROWS; ++i)
+      if (i < TAPS - 1 + nr) take_n<T, false, 8>(src + (t0 - (TAPS - 1) + i) * p.ld, 0, x[i]);
+#pragma unroll
+    for (int r = 0; r < CONV_ROWS; ++r)
+      if (r < nr) {
+        float a[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          a[j] = b[j];
+#pragma unroll
+          for (int k = 0; k < TAPS; ++k) a[j] += w[k][j] * x[r + k][j];
+        }
+        emit(t0 + r, a);
+      }
+    return;
+  }
+  for (int r = 0; r < nr; ++r) {
+    const long long t = t0 + r;
+    const int s = p.rseq[t];
+    seq_rows(p.cu, p.ctx, p.nd, s, row0, n, start);
+    const int local = (int)(t - row0), slot = p.sslot[s];
+    float a[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) a[j] = b[j];
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) {
+      const int q = local - (TAPS - 1) + k;
+      float x[8];
+      if (q >= 0) take_n<T, false, 8>(src + (row0 + q) * p.ld, 0, x);
+      else if (start > 0 && slot >= 0) take_n<T, false, 8>(state + ((long long)slot * (TAPS - 1) + q + TAPS - 1) * p.C, 0, x);
+      else continue;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[j] += w[k][j] * x[j];
+    }
+    emit(t, a);
+  }
+}
 // decode rows only: the projection comes as the decode GEMM's accumulator
 template <typename T>
 __global__ void __launch_bounds__(256) short_conv_acc_kernel(const ConvParams p) {
@@ -434,6 +731,41 @@ __global__ void __launch_bounds__(256) short_conv_acc_kernel(const ConvParams p)
   }
 }
 
+// the same, 8 columns per thread (C, col and every pitch multiples of 8)
+template <typename T>
+__global__ void __launch_bounds__(128) short_conv_acc_vec_kernel(const ConvParams p) {
+  griddep_wait();
+  griddep_launch();
+  const int col = (blockIdx.y * 128 + threadIdx.x) * 8;
+  if (col >= p.raw_n) return;
+  const long long t = blockIdx.x;
+  float v[8];
+  take_n<T, true, 8>(reinterpret_cast<const uint8_t*>(p.src) + t * p.ld * 4, col, v);
+  put_n(reinterpret_cast<T*>(p.raw) + t * p.raw_ld + col, v);
+  const int c = col - p.col;
+  if (c < 0 || c >= p.C) return;
+  const int slot = p.sslot[t];
+  float a[8], w[8];
+  ld8(p.b + c, a);
+  ld8(p.w + (long long)(p.taps - 1) * p.w_ld + c, w);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) a[j] += w[j] * v[j];
+  if (slot >= 0 && p.ctx[t] > 1) {
+    const T* st = reinterpret_cast<const T*>(p.state) + (long long)slot * (p.taps - 1) * p.C + c;
+#pragma unroll 3
+    for (int k = 0; k < p.taps - 1; ++k) {
+      float x[8];
+      take_n<T, false, 8>(st + (long long)k * p.C, 0, x);
+      ld8(p.w + (long long)k * p.w_ld + c, w);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[j] += w[j] * x[j];
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < 8; ++j) a[j] = a[j] / (1.f + __expf(-a[j]));
+  put_n(reinterpret_cast<T*>(p.out) + t * p.o_ld + c, a);
+}
+
 inline int grid_for(long long total, int block) {
   long long g = (total + block - 1) / block;
   const long long cap = (long long)dlti_num_sms() * 16;
@@ -443,6 +775,18 @@ inline int grid_for(long long total, int block) {
 template <typename T, bool ACC>
 int post_norm_add_t(const void* y, long long y_ld, float* x, const float* w, void* xa, long long xa_ld, long long rows, int d,
                     float eps, int one, cudaStream_t st) {
+  if constexpr (sizeof(T) == 2) {
+    if (d % 8 == 0 && d <= 8192 && y_ld % 8 == 0 && (!xa || xa_ld % 8 == 0) &&
+        ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(xa)) & 15) == 0) {
+      const int vpt = (d / 8 + 127) / 128;
+      auto kern = vpt <= 1 ? post_norm_add_vec_kernel<T, ACC, 1> : vpt <= 2 ? post_norm_add_vec_kernel<T, ACC, 2>
+                  : vpt <= 4 ? post_norm_add_vec_kernel<T, ACC, 4> : post_norm_add_vec_kernel<T, ACC, 8>;
+      DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)rows), dim3(128), 0, st, y, y_ld, x, w, (T*)xa, xa_ld, d, eps,
+                                      one ? 1.f : 0.f));
+      dlti_count_launch();
+      return 0;
+    }
+  }
   const int pairs = (d + 2 * PN_THREADS - 1) / (2 * PN_THREADS);
 #define PN_CASE(P)                                                                                                      \
   if (pairs <= P) {                                                                                                     \
@@ -508,12 +852,13 @@ DLTI_API int dlti_relu2(const void* u, long long u_ld, void* h, long long h_ld, 
                         cudaStream_t st) {
   if (rows <= 0) return 0;
   if (u_ld % 2 || h_ld % 2) return DLTI_ERR_BAD_ARG;
-  if (!acc && dtype == DLTI_BF16 && ff % 8 == 0 && u_ld % 8 == 0 && h_ld % 8 == 0 &&
+  if (dtype == DLTI_BF16 && ff % 8 == 0 && u_ld % 8 == 0 && h_ld % 8 == 0 &&
       ((reinterpret_cast<uintptr_t>(u) | reinterpret_cast<uintptr_t>(h)) & 15) == 0) {
-    relu2_vec_kernel<__nv_bfloat16><<<grid_for(rows * (ff / 8), 256), 256, 0, st>>>((const __nv_bfloat16*)u, u_ld, (__nv_bfloat16*)h,
-                                                                                    h_ld, rows, ff);
+    const dim3 g(grid_for(rows * (ff / 8), 256));
+    auto kern = acc ? relu2_vec_kernel<__nv_bfloat16, true> : relu2_vec_kernel<__nv_bfloat16, false>;
+    DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, g, dim3(256), 0, st, u, u_ld, (__nv_bfloat16*)h, h_ld, rows, ff));
     dlti_count_launch();
-    return (int)cudaGetLastError();
+    return 0;
   }
   const int g = grid_for(rows * ((ff + 1) / 2), 256);
   if (acc)
@@ -528,6 +873,20 @@ DLTI_API int dlti_gated_norm(const void* y, long long y_ld, const void* gate, lo
                              long long rows, int n, int groups, float eps, int gate_first, int acc, int dtype, cudaStream_t st) {
   if (rows <= 0) return 0;
   if (groups < 1 || n % groups) return DLTI_ERR_BAD_ARG;
+  const int gs = n / groups;
+  if (dtype == DLTI_BF16 && gs % 8 == 0 && gs <= 8 * 256 * 8 && y_ld % 8 == 0 && g_ld % 8 == 0 && o_ld % 8 == 0 && groups <= 65535 &&
+      ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+    using B = __nv_bfloat16;
+    const int vec = gs / 8, threads = vec <= 64 ? 64 : (vec <= 128 ? 128 : 256), vpt = (vec + threads - 1) / threads;
+#define GNV(GF, AC) (vpt <= 1 ? gated_norm_vec_kernel<B, GF, AC, 1> : vpt <= 2 ? gated_norm_vec_kernel<B, GF, AC, 2> \
+                     : vpt <= 4 ? gated_norm_vec_kernel<B, GF, AC, 4> : gated_norm_vec_kernel<B, GF, AC, 8>)
+    auto kern = gate_first ? (acc ? GNV(true, true) : GNV(true, false)) : (acc ? GNV(false, true) : GNV(false, false));
+#undef GNV
+    DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)rows, groups), dim3(threads), 0, st, (const B*)y, y_ld, gate, g_ld, w, (B*)out,
+                                    o_ld, gs, eps));
+    dlti_count_launch();
+    return 0;
+  }
   const size_t smem = (size_t)n * 4;
   if (smem > 48 * 1024) { dlti_set_error("gated_norm: rows of up to 12288 elements"); return DLTI_ERR_TOO_LARGE; }
 #define GN_CASE(GF, AC)                                                                                                          \
@@ -552,7 +911,25 @@ DLTI_API int dlti_qk_norm_rope_cache(const void* proj, long long ld, int oq, int
   if (rot / 2 + (dim - rot + 1) / 2 > 32 * QKV_MAXP) { dlti_set_error("qk_norm_rope_cache: heads of up to 512 dimensions"); return DLTI_ERR_TOO_LARGE; }
   QkvParams p{proj, ld, oq, ok, ov, og, qn, kn, eps, pos, cos_t, sin_t, rot, interleaved, slots, kc, vc, kd, vd,
               q, q_ld, q_hd, kp, vp, gate, tokens, H, G, dim, vdim};
-  const int jobs = H + ((ok >= 0 || kp) ? 2 * G : 0) + (og >= 0 ? 1 : 0);
+  const int kvjobs = (ok >= 0 || kp) ? 2 * G : 0, jobs = H + kvjobs + (og >= 0 ? 1 : 0);
+  const bool vec = dtype == DLTI_BF16 && (dim == 64 || dim == 128 || dim == 256) && vdim == dim && (interleaved || rot == 0) && ld % 8 == 0 &&
+                   q_ld % 8 == 0 && q_hd % 8 == 0 && kd % 8 == 0 && vd % 8 == 0 && oq % 8 == 0 && (ok < 0 || (ok % 8 == 0 && ov % 8 == 0)) &&
+                   tokens < (1ll << 31) &&
+                   ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kc) |
+                     reinterpret_cast<uintptr_t>(vc) | reinterpret_cast<uintptr_t>(kp) | reinterpret_cast<uintptr_t>(vp)) & 15) == 0;
+  if (vec) {
+    using B = __nv_bfloat16;
+#define QKV_CASE(VE)                                                                                                             \
+  if (dim == 32 * VE) {                                                                                                          \
+    const int jpw = acc ? 1 : 4;                                                                                                 \
+    auto kern = acc ? qk_norm_rope_cache_vec_kernel<B, true, VE, 1> : qk_norm_rope_cache_vec_kernel<B, false, VE, 4>;              \
+    DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, kern, dim3((unsigned)tokens, (jobs + 8 * jpw - 1) / (8 * jpw)), dim3(256), 0, st, p, jobs, kvjobs)); \
+  }
+    QKV_CASE(2) QKV_CASE(4) QKV_CASE(8)
+#undef QKV_CASE
+    dlti_count_launch();
+    return 0;
+  }
   const int g = grid_for(tokens * jobs * 32, 256);
   if (acc) DISPATCH_T(dtype, DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, qk_norm_rope_cache_kernel<T, true>, dim3(g), dim3(256), 0, st, p)));
   else DISPATCH_T(dtype, DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, qk_norm_rope_cache_kernel<T, false>, dim3(g), dim3(256), 0, st, p)));
@@ -569,8 +946,22 @@ DLTI_API int dlti_short_conv(const void* src, long long ld, int col, int C, int 
   ConvParams p{src, ld, col, C, taps, w, b, w_ld, state, sslot, rseq, ctx, cu, nd, out, o_ld, raw, raw_ld, raw_n, rows};
   if (acc) {
     if (nd != rows || !raw || raw_n % 2) return DLTI_ERR_BAD_ARG;
+    if (dtype == DLTI_BF16 && C % 8 == 0 && ld % 8 == 0 && col % 8 == 0 && raw_n % 8 == 0 && raw_ld % 8 == 0 && o_ld % 8 == 0 && w_ld % 4 == 0 &&
+        ((reinterpret_cast<uintptr_t>(src) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(raw) | reinterpret_cast<uintptr_t>(w) |
+          reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(state)) & 15) == 0) {
+      DLTI_CUDA_CHECK(dlti_launch_pdl(rows, short_conv_acc_vec_kernel<__nv_bfloat16>, dim3((unsigned)rows, (raw_n / 8 + 127) / 128), dim3(128), 0,
+                                      st, p));
+      dlti_count_launch();
+      return 0;
+    }
     const int g = grid_for(rows * (raw_n / 2), 256);
     DISPATCH_T(dtype, DLTI_CUDA_CHECK(dlti_launch_pdl(rows, short_conv_acc_kernel<T>, dim3(g), dim3(256), 0, st, p)));
+  } else if (dtype == DLTI_BF16 && taps >= 2 && taps <= 4 && C % 8 == 0 && ld % 8 == 0 && col % 8 == 0 && o_ld % 8 == 0 && w_ld % 4 == 0 &&
+             ((reinterpret_cast<uintptr_t>(src) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(w) |
+               reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(state)) & 15) == 0) {
+    using B = __nv_bfloat16;
+    auto kern = taps == 2 ? short_conv_vec_kernel<B, 2> : taps == 3 ? short_conv_vec_kernel<B, 3> : short_conv_vec_kernel<B, 4>;
+    DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)((rows + CONV_ROWS - 1) / CONV_ROWS), (C / 8 + 127) / 128), dim3(128), 0, st, p));
   } else {
     const int g = grid_for(rows * ((C + 1) / 2), 256);
     DISPATCH_T(dtype, DLTI_CUDA_CHECK(dlti_launch_pdl(rows, short_conv_kernel<T>, dim3(g), dim3(256), 0, st, p)));

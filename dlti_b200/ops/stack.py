@@ -408,7 +408,7 @@ def linear_scan(q, k, v, decay: Decay, state, rows: Rows, heads, groups, N, P, s
         if nd:
             _scan_tokens(q, k, v, decay, state, rows, 0, nd, heads, groups, N, P, silu, conv, out)
         if silu:
-            for x in (q, k, v):
+            for x in _merge_sections(q, k, v):
                 silu_rows_(x[nd:])
         _scan_chunked(q, k, v, decay, state, rows, nd, nseq - nd, heads, groups, N, P, conv, out)
     else:
@@ -419,8 +419,22 @@ def linear_scan(q, k, v, decay: Decay, state, rows: Rows, heads, groups, N, P, s
 _CHUNKED_FROM = 16           # longest portion of a step from which the chunked kernel takes its prompts
 
 
+def _merge_sections(*xs):
+    """Neighbouring sections of one projection as a single view where only alignment padding (< 8 columns) lies between
+    them, rounded up to whole 8-column pieces (padding columns are zero)."""
+    out = []
+    for x in xs:
+        n = round8(x.shape[1])
+        if out and x.stride(0) == out[-1].stride(0) and x.data_ptr() == out[-1].data_ptr() + out[-1].shape[1] * x.element_size():
+            n += out.pop().shape[1]
+            x = xs_base
+        xs_base = x
+        out.append(x.as_strided((x.shape[0], n), x.stride()))
+    return out
+
+
 def silu_rows_(x):
-    """In place on a [rows, n] bf16 section of a projection."""
+    """In place on a [rows, n] bf16 section of a projection, n a multiple of 8."""
     f = _lib.fn("dlti_silu_rows", [_V, _L, _L, _I, _I, _V])
     _lib.check(f(_p(x), x.stride(0), x.shape[0], x.shape[1], _lib.dtype_code(x.dtype), _lib.stream_ptr()), "silu_rows")
 
