@@ -176,22 +176,27 @@ int launch_scan(const ScanParams& p, int nseq, cudaStream_t st) {
   return DLTI_ERR_TOO_LARGE;
 }
 
-// Chunked form for prompts, bf16: CTA = (32 columns of P, head, sequence), 4 warps, 64 tokens a chunk. With L_t the
-// running sum of log a within the chunk and d_s = step size,
-//     o_t   = exp(L_t) S^T q_t + sum_(s <= t) [exp(L_t - L_s) d_s (k_s . q_t)] v_s
-//     S'    = exp(L_63) S + sum_s k_s [exp(L_63 - L_s) d_s v_s]^T
+// Chunked form for prompts, bf16: CTA = (32 columns of P, head, sequence), 64 tokens a chunk. With L_t the running sum of
+// log2 a within the chunk and d_s = step size,
+//     o_t   = 2^(L_t) S^T q_t + sum_(s <= t) [2^(L_t - L_s) d_s (k_s . q_t)] v_s
+//     S'    = 2^(L_63) S + sum_s k_s [2^(L_63 - L_s) d_s v_s]^T
 // q, k, v are exact bf16 operands; the three fp32 operands (S, the bracketed weights, the bracketed values) enter the
-// tensor-core products as hi + lo bf16 pairs, so the recurrence keeps 16+ mantissa bits everywhere. S lives in fp32
-// accumulator registers (warp w owns rows [w NT/4, (w+1) NT/4)) and, split, in shared memory as the next operand.
+// tensor-core products as hi + lo bf16 pairs, so the recurrence keeps 16+ mantissa bits everywhere.
+// Warps 0-3 compute the outputs (16 tokens each) from the S operand in shared memory; warps 4-7 meanwhile advance S, which
+// lives in their fp32 accumulators (NT / 4 rows each), and publish it as the next operand once warps 0-3 have read the old
+// one. Warp 4 also prepares the next chunk's decay vectors. One CTA-wide barrier per chunk.
 constexpr int CQ = 64, CP = 32, CPP = CP + 8;
 template <int NT>
 struct ChunkSmem {
   static constexpr int NP = NT + 8;
   static constexpr int QK = CQ * NP * 2, V = CQ * CPP * 2, STAGE = 2 * QK + V;          // bytes
-  static constexpr int W = 2 * STAGE, S = W + 2 * V, VEC = S + 2 * NT * CPP * 2, BYTES = VEC + 5 * CQ * 4;
+  static constexpr int W = 2 * STAGE, S = W + 2 * V, VEC = S + 2 * NT * CPP * 2, BYTES = VEC + 2 * 4 * CQ * 4;
+};
+struct ChunkVec {                                                // one chunk's vectors, 64 each
+  float *L, *step, *E, *F;                                       // L; d; 2^(L_63 - L_s) d; 2^(L_e - L_s) d, e = end of s's 16-block
 };
 template <int NT>
-__global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int slices, int conv_parts) {
+__global__ void __launch_bounds__(256, NT <= 128 ? 2 : 1) scan_chunk_kernel(const ScanParams p, int slices, int conv_parts) {
   using L = ChunkSmem<NT>;
   using bf16 = __nv_bfloat16;
   const int s = p.seq0 + blockIdx.z;
@@ -201,11 +206,6 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
   }
   extern __shared__ __align__(128) uint8_t smem[];
   const uint32_t sb = smem_u32(smem);
-  float* sHalf = reinterpret_cast<float*>(smem + L::VEC);       // running log2 decay inside each half of the chunk
-  float* sL = sHalf + CQ;                                       // ... of the whole chunk
-  float* sStep = sL + CQ;
-  float* sE = sStep + CQ;                                       // 2^(L_63 - L_s) * step
-  float* sF = sE + CQ;                                          // 2^(L_e - L_s) * step, e = last token of s's 16-block
   long long row0;
   int n, start;
   seq_rows(p, s, row0, n, start);
@@ -215,60 +215,180 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
   const bf16* q = reinterpret_cast<const bf16*>(p.q) + row0 * p.q_ld + (long long)grp * p.N;
   const bf16* k = reinterpret_cast<const bf16*>(p.k) + row0 * p.k_ld + (long long)grp * p.N;
   const bf16* v = reinterpret_cast<const bf16*>(p.v) + row0 * p.v_ld + (long long)h * p.P + c0;
+  const float Dh = p.D ? p.D[h] : 0.f;
+  auto vec = [&](int i) {
+    float* f = reinterpret_cast<float*>(smem + L::VEC) + (i & 1) * 4 * CQ;
+    return ChunkVec{f, f + CQ, f + 2 * CQ, f + 3 * CQ};
+  };
+  auto load = [&](int stage, int t0) {
+    constexpr int STEP = 256 / (NT / 8);                         // rows per pass
+    const uint32_t base = sb + stage * L::STAGE;
+    const int r0 = threadIdx.x / (NT / 8), c = threadIdx.x % (NT / 8);
+    const bool cok = c * 8 < p.N;
+    const bf16* qp = q + (t0 + r0) * p.q_ld + c * 8;             // never dereferenced where a row or column is out of range
+    const bf16* kp = k + (t0 + r0) * p.k_ld + c * 8;
+    const uint32_t dst = base + (r0 * L::NP + c * 8) * 2;
+#pragma unroll
+    for (int i = 0; i < CQ / STEP; ++i) {
+      const bool ok = cok && t0 + r0 + i * STEP < n;
+      cp_async16(dst + i * STEP * L::NP * 2, ok ? qp : q, ok);
+      cp_async16(dst + i * STEP * L::NP * 2 + L::QK, ok ? kp : k, ok);
+      qp += STEP * p.q_ld;
+      kp += STEP * p.k_ld;
+    }
+    const int r = threadIdx.x / (CP / 8), cv = threadIdx.x % (CP / 8);     // 64 rows x 4 pieces
+    const bool ok = t0 + r < n && cv * 8 < ncol;
+    cp_async16(base + 2 * L::QK + (r * CPP + cv * 8) * 2, ok ? v + (t0 + r) * p.v_ld + cv * 8 : v, ok);
+    cp_async_commit();
+  };
+  load(0, 0);
+
+  if (warp < 4) {
+    // ---- outputs of 16 tokens per chunk ----
+    const int scol = (lane & 3) * 2, tr = warp * 16 + (lane >> 2);
+    int it = 0;
+    for (int t0 = 0; t0 < n; t0 += CQ, ++it) {
+      cp_async_wait<0>();
+      __syncthreads();                                           // tile, vectors and S operand of this chunk are there
+      if (t0 + CQ < n) load((it + 1) & 1, t0 + CQ);
+      const uint32_t base = sb + (it & 1) * L::STAGE;
+      const ChunkVec cv = vec(it);
+      uint32_t qf[NT / 16][4];
+      {
+        const uint32_t qa = base + ((warp * 16 + (lane & 15)) * L::NP + (lane >> 4) * 8) * 2;
+#pragma unroll
+        for (int kk = 0; kk < NT / 16; ++kk) ldsm4(qf[kk], qa + kk * 32);
+      }
+      float o[CP / 8][4];
+#pragma unroll
+      for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) o[j][x] = 0.f;
+      {
+        const uint32_t sa = sb + L::S + ((lane & 15) * CPP + (lane >> 4) * 8) * 2;
+#pragma unroll
+        for (int kk = 0; kk < NT / 16; ++kk)
+#pragma unroll
+          for (int x = 0; x < 2; ++x)                            // hi, lo
+#pragma unroll
+            for (int j = 0; j < CP / 16; ++j) {
+              uint32_t b[4];
+              ldsm4_t(b, sa + x * (NT * CPP * 2) + (kk * 16 * CPP + j * 16) * 2);
+              mma_bf16(o[2 * j], qf[kk], b[0], b[1]);
+              mma_bf16(o[2 * j + 1], qf[kk], b[2], b[3]);
+            }
+      }
+      asm volatile("bar.arrive 2, 256;" ::: "memory");           // the old S operand has been read
+      const float lt[2] = {cv.L[tr], cv.L[tr + 8]};
+      const float el[2] = {ex2(lt[0]), ex2(lt[1])};
+#pragma unroll
+      for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) o[j][x] *= el[x >> 1];
+      for (int kb = 0; kb <= warp; ++kb) {                       // 16 keys at a time up to the diagonal
+        float g0[4] = {}, g1[4] = {};
+        const uint32_t ka = base + L::QK + ((kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * L::NP + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll
+        for (int kk = 0; kk < NT / 16; ++kk) {
+          uint32_t b[4];
+          ldsm4(b, ka + kk * 32);
+          mma_bf16(g0, qf[kk], b[0], b[1]);
+          mma_bf16(g1, qf[kk], b[2], b[3]);
+        }
+        if (kb < warp) {                                         // all keys precede all tokens: factored through the block's end
+          const float le = cv.L[kb * 16 + 15];
+          const float f0 = ex2(lt[0] - le), f1 = ex2(lt[1] - le);
+          const float2 a = *reinterpret_cast<const float2*>(cv.F + kb * 16 + scol), b = *reinterpret_cast<const float2*>(cv.F + kb * 16 + 8 + scol);
+          g0[0] *= a.x * f0; g0[1] *= a.y * f0; g0[2] *= a.x * f1; g0[3] *= a.y * f1;
+          g1[0] *= b.x * f0; g1[1] *= b.y * f0; g1[2] *= b.x * f1; g1[3] *= b.y * f1;
+        } else {
+#pragma unroll
+          for (int x = 0; x < 4; ++x) {
+            const int t = tr + 8 * (x >> 1);
+            const int u0 = kb * 16 + scol + (x & 1), u1 = u0 + 8;
+            g0[x] = u0 <= t ? g0[x] * cv.step[u0] * ex2(lt[x >> 1] - cv.L[u0]) : 0.f;
+            g1[x] = u1 <= t ? g1[x] * cv.step[u1] * ex2(lt[x >> 1] - cv.L[u1]) : 0.f;
+          }
+        }
+        uint32_t hi[4], lo[4];
+        split_pair(g0[0], g0[1], hi[0], lo[0]);
+        split_pair(g0[2], g0[3], hi[1], lo[1]);
+        split_pair(g1[0], g1[1], hi[2], lo[2]);
+        split_pair(g1[2], g1[3], hi[3], lo[3]);
+        const uint32_t va = base + 2 * L::QK + ((kb * 16 + (lane & 15)) * CPP + (lane >> 4) * 8) * 2;
+#pragma unroll
+        for (int j = 0; j < CP / 16; ++j) {
+          uint32_t b[4];
+          ldsm4_t(b, va + j * 32);
+          mma_bf16(o[2 * j], hi, b[0], b[1]);
+          mma_bf16(o[2 * j + 1], hi, b[2], b[3]);
+          mma_bf16(o[2 * j], lo, b[0], b[1]);
+          mma_bf16(o[2 * j + 1], lo, b[2], b[3]);
+        }
+      }
+      const bf16* sv = reinterpret_cast<const bf16*>(smem + (it & 1) * L::STAGE + 2 * L::QK);
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        const int t = tr + 8 * y;
+        if (t0 + t < n) {
+          bf16* orow = reinterpret_cast<bf16*>(p.out) + (row0 + t0 + t) * p.o_ld + (long long)h * p.P + c0;
+#pragma unroll
+          for (int j = 0; j < CP / 8; ++j) {
+            const int c = j * 8 + scol;
+            if (c >= ncol) continue;
+            const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + t * CPP + c));
+            *reinterpret_cast<__nv_bfloat162*>(orow + c) = __floats2bfloat162_rn(o[j][2 * y] + Dh * x.x, o[j][2 * y + 1] + Dh * x.y);
+          }
+        }
+      }
+    }
+    return;
+  }
+
+  // ---- state ----
+  const int sw = warp - 4;
   constexpr float LOG2E = 1.4426950408889634f;
   const float eA = p.decay ? 0.f : expf(p.A_log[h]) * LOG2E;
   const float la_c = p.decay ? fmaxf(logf(p.decay[h]), -80.f) * LOG2E : 0.f;
   const float bias = p.decay ? 0.f : p.dt_bias[h];
-  const float Dh = p.D ? p.D[h] : 0.f;
-
-  auto load = [&](int stage, int t0) {
-    constexpr int STEP = 128 / (NT / 8);                         // rows per pass
-    const uint32_t base = sb + stage * L::STAGE;
-    const int r0 = threadIdx.x / (NT / 8), c = threadIdx.x % (NT / 8);
-    {
-      const bool cok = c * 8 < p.N;
-      const bf16* qp = q + (t0 + r0) * p.q_ld + c * 8;           // never dereferenced where a row or column is out of range
-      const bf16* kp = k + (t0 + r0) * p.k_ld + c * 8;
-      const uint32_t dst = base + (r0 * L::NP + c * 8) * 2;
+  // warp 4: step sizes and decays of the chunk at t0, two consecutive tokens a lane
+  auto raw_dt = [&](int t0, float (&d)[2]) {
 #pragma unroll
-      for (int i = 0; i < CQ / STEP; ++i) {
-        const bool ok = cok && t0 + r0 + i * STEP < n;
-        cp_async16(dst + i * STEP * L::NP * 2, ok ? qp : q, ok);
-        cp_async16(dst + i * STEP * L::NP * 2 + L::QK, ok ? kp : k, ok);
-        qp += STEP * p.q_ld;
-        kp += STEP * p.k_ld;
-      }
+    for (int y = 0; y < 2; ++y) {
+      const int t = t0 + 2 * lane + y;
+      d[y] = (!p.decay && t < n) ? __bfloat162float(reinterpret_cast<const bf16*>(p.dt)[(row0 + t) * p.dt_ld + h]) + bias : 0.f;
     }
+  };
+  auto prepare = [&](int i, int t0, const float (&d)[2]) {
+    float step[2], l[2];
 #pragma unroll
-    for (int i = 0; i < CQ * (CP / 8) / 128; ++i) {
-      const int r = threadIdx.x / (CP / 8) + i * (128 / (CP / 8)), cv = threadIdx.x % (CP / 8);
-      const bool ok = t0 + r < n && cv * 8 < ncol;
-      cp_async16(base + 2 * L::QK + (r * CPP + cv * 8) * 2, ok ? v + (t0 + r) * p.v_ld + cv * 8 : v, ok);
+    for (int y = 0; y < 2; ++y) {
+      const bool ok = t0 + 2 * lane + y < n;
+      step[y] = !ok ? 0.f : (p.decay ? 1.f : softplus_f(d[y]));
+      l[y] = !ok ? 0.f : (p.decay ? la_c : -eA * step[y]);
     }
-    cp_async_commit();
+    l[1] += l[0];
+    float x = l[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float y = __shfl_up_sync(0xffffffffu, x, o);
+      if (lane >= o) x += y;
+    }
+    const float before = x - l[1];
+    const float total = __shfl_sync(0xffffffffu, x, 31);
+    const float le = __shfl_sync(0xffffffffu, x, lane | 7);      // end of this 16-token block
+    const float l0 = before + l[0], l1 = x;
+    const ChunkVec cv = vec(i);
+    *reinterpret_cast<float2*>(cv.L + 2 * lane) = make_float2(l0, l1);
+    *reinterpret_cast<float2*>(cv.step + 2 * lane) = make_float2(step[0], step[1]);
+    *reinterpret_cast<float2*>(cv.E + 2 * lane) = make_float2(ex2(total - l0) * step[0], ex2(total - l1) * step[1]);
+    *reinterpret_cast<float2*>(cv.F + 2 * lane) = make_float2(ex2(le - l0) * step[0], ex2(le - l1) * step[1]);
   };
-  auto raw_dt = [&](int t0) {
-    const int t = t0 + threadIdx.x;
-    if (p.decay || threadIdx.x >= CQ || t >= n) return 0.f;
-    return __bfloat162float(reinterpret_cast<const bf16*>(p.dt)[(row0 + t) * p.dt_ld + h]) + bias;
-  };
-
   constexpr int MT = NT / 64;                                    // 16-row state tiles of a warp
   float S[MT][CP / 8][4];
   float* st = p.state + (((long long)(slot < 0 ? 0 : slot) * p.heads + h) * p.N) * p.P + c0;
-  const int srow = warp * (NT / 4) + (lane >> 2), scol = (lane & 3) * 2;
+  const int srow = sw * (NT / 4) + (lane >> 2), scol = (lane & 3) * 2;
   const bool have = slot >= 0 && start > 0;
-#pragma unroll
-  for (int i = 0; i < MT; ++i)
-#pragma unroll
-    for (int j = 0; j < CP / 8; ++j)
-#pragma unroll
-      for (int y = 0; y < 2; ++y) {
-        const int r = srow + i * 16 + 8 * y, c = j * 8 + scol;
-        const bool ok = have && r < p.N && c < ncol;             // ncol is a multiple of 8
-        S[i][j][2 * y] = ok ? st[(long long)r * p.P + c] : 0.f;
-        S[i][j][2 * y + 1] = ok ? st[(long long)r * p.P + c + 1] : 0.f;
-      }
   auto publish = [&]() {                                         // S as hi / lo operands
 #pragma unroll
     for (int i = 0; i < MT; ++i)
@@ -283,151 +403,50 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
           *reinterpret_cast<uint32_t*>(smem + L::S + NT * CPP * 2 + off) = lo;
         }
   };
-  load(0, 0);
-  float dt_next = raw_dt(0);
+  float d[2] = {0.f, 0.f};
+  if (sw == 0) {
+    raw_dt(0, d);
+    prepare(0, 0, d);
+    raw_dt(CQ, d);
+  }
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        const int r = srow + i * 16 + 8 * y, c = j * 8 + scol;
+        const bool ok = have && r < p.N && c < ncol;             // ncol is a multiple of 8
+        S[i][j][2 * y] = ok ? st[(long long)r * p.P + c] : 0.f;
+        S[i][j][2 * y + 1] = ok ? st[(long long)r * p.P + c + 1] : 0.f;
+      }
   publish();
   int it = 0;
   for (int t0 = 0; t0 < n; t0 += CQ, ++it) {
+    cp_async_wait<0>();
+    __syncthreads();
+    if (t0 + CQ < n) load((it + 1) & 1, t0 + CQ);
     const uint32_t base = sb + (it & 1) * L::STAGE;
-    if (threadIdx.x < CQ) {
-      const bool ok = t0 + (int)threadIdx.x < n;
-      const float step = !ok ? 0.f : (p.decay ? 1.f : softplus_f(dt_next));
-      float x = !ok ? 0.f : (p.decay ? la_c : -eA * step);
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float y = __shfl_up_sync(0xffffffffu, x, o);
-        if (lane >= o) x += y;
-      }
-      sStep[threadIdx.x] = step;
-      sHalf[threadIdx.x] = x;
-    }
-    dt_next = raw_dt(t0 + CQ);
-    __syncthreads();                                             // stage (it + 1) & 1 free; half sums, S operands visible
-    if (t0 + CQ < n) {
-      load((it + 1) & 1, t0 + CQ);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    const float half = sHalf[31];
-    const float total = sHalf[CQ - 1] + half;
-    if (threadIdx.x < CQ) {
-      const float l = sHalf[threadIdx.x], le = sHalf[threadIdx.x | 15], step = sStep[threadIdx.x];
-      sL[threadIdx.x] = l + (threadIdx.x >= 32 ? half : 0.f);
-      sE[threadIdx.x] = ex2(total - (l + (threadIdx.x >= 32 ? half : 0.f))) * step;
-      sF[threadIdx.x] = ex2(le - l) * step;
-    }
-    __syncthreads();                                             // tile landed, sE written
+    const ChunkVec cv = vec(it);
     const bf16* sv = reinterpret_cast<const bf16*>(smem + (it & 1) * L::STAGE + 2 * L::QK);
-    for (int i = threadIdx.x; i < CQ * CP / 2; i += 128) {       // scaled values as hi / lo operands
-      const int r = i / (CP / 2), c = 2 * (i % (CP / 2));
+#pragma unroll
+    for (int i = 0; i < CQ * CP / 2 / 128; ++i) {                // scaled values as hi / lo operands
+      const int r = (threadIdx.x - 128) / (CP / 2) + i * (128 / (CP / 2)), c = 2 * (threadIdx.x % (CP / 2));
       const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + r * CPP + c));
+      const float e = cv.E[r];
       uint32_t hi, lo;
-      split_pair(x.x * sE[r], x.y * sE[r], hi, lo);
+      split_pair(x.x * e, x.y * e, hi, lo);
       *reinterpret_cast<uint32_t*>(smem + L::W + (r * CPP + c) * 2) = hi;
       *reinterpret_cast<uint32_t*>(smem + L::W + L::V + (r * CPP + c) * 2) = lo;
     }
-    // ---- outputs of this warp's 16 tokens ----
-    uint32_t qf[NT / 16][4];
-    {
-      const uint32_t qa = base + ((warp * 16 + (lane & 15)) * L::NP + (lane >> 4) * 8) * 2;
-#pragma unroll
-      for (int kk = 0; kk < NT / 16; ++kk) ldsm4(qf[kk], qa + kk * 32);
-    }
-    float o[CP / 8][4];
-#pragma unroll
-    for (int j = 0; j < CP / 8; ++j)
-#pragma unroll
-      for (int x = 0; x < 4; ++x) o[j][x] = 0.f;
-    {
-      const uint32_t sa = sb + L::S + ((lane & 15) * CPP + (lane >> 4) * 8) * 2;
-#pragma unroll
-      for (int kk = 0; kk < NT / 16; ++kk)
-#pragma unroll
-        for (int x = 0; x < 2; ++x)                              // hi, lo
-#pragma unroll
-          for (int j = 0; j < CP / 16; ++j) {
-            uint32_t b[4];
-            ldsm4_t(b, sa + x * (NT * CPP * 2) + (kk * 16 * CPP + j * 16) * 2);
-            mma_bf16(o[2 * j], qf[kk], b[0], b[1]);
-            mma_bf16(o[2 * j + 1], qf[kk], b[2], b[3]);
-          }
-    }
-    const int tr = warp * 16 + (lane >> 2);
-    float lt[2], el[2];
-#pragma unroll
-    for (int y = 0; y < 2; ++y) {
-      lt[y] = sL[tr + 8 * y];
-      el[y] = ex2(lt[y]);
-    }
-#pragma unroll
-    for (int j = 0; j < CP / 8; ++j)
-#pragma unroll
-      for (int x = 0; x < 4; ++x) o[j][x] *= el[x >> 1];
-    for (int kb = 0; kb <= warp; ++kb) {                         // 16 keys at a time up to the diagonal
-      float g0[4] = {}, g1[4] = {};
-      const uint32_t ka = base + L::QK + ((kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * L::NP + ((lane >> 3) & 1) * 8) * 2;
-#pragma unroll
-      for (int kk = 0; kk < NT / 16; ++kk) {
-        uint32_t b[4];
-        ldsm4(b, ka + kk * 32);
-        mma_bf16(g0, qf[kk], b[0], b[1]);
-        mma_bf16(g1, qf[kk], b[2], b[3]);
-      }
-      if (kb < warp) {                                           // all keys precede all tokens: factored through the block's end
-        const float le = sL[kb * 16 + 15];
-        const float f0 = ex2(lt[0] - le), f1 = ex2(lt[1] - le);
-        const float2 a = *reinterpret_cast<const float2*>(sF + kb * 16 + scol), b = *reinterpret_cast<const float2*>(sF + kb * 16 + 8 + scol);
-        g0[0] *= a.x * f0; g0[1] *= a.y * f0; g0[2] *= a.x * f1; g0[3] *= a.y * f1;
-        g1[0] *= b.x * f0; g1[1] *= b.y * f0; g1[2] *= b.x * f1; g1[3] *= b.y * f1;
-      } else {
-#pragma unroll
-        for (int x = 0; x < 4; ++x) {
-          const int t = tr + 8 * (x >> 1);
-          const int u0 = kb * 16 + scol + (x & 1), u1 = u0 + 8;
-          g0[x] = u0 <= t ? g0[x] * sStep[u0] * ex2(lt[x >> 1] - sL[u0]) : 0.f;
-          g1[x] = u1 <= t ? g1[x] * sStep[u1] * ex2(lt[x >> 1] - sL[u1]) : 0.f;
-        }
-      }
-      uint32_t hi[4], lo[4];
-      split_pair(g0[0], g0[1], hi[0], lo[0]);
-      split_pair(g0[2], g0[3], hi[1], lo[1]);
-      split_pair(g1[0], g1[1], hi[2], lo[2]);
-      split_pair(g1[2], g1[3], hi[3], lo[3]);
-      const uint32_t va = base + 2 * L::QK + ((kb * 16 + (lane & 15)) * CPP + (lane >> 4) * 8) * 2;
-#pragma unroll
-      for (int j = 0; j < CP / 16; ++j) {
-        uint32_t b[4];
-        ldsm4_t(b, va + j * 32);
-        mma_bf16(o[2 * j], hi, b[0], b[1]);
-        mma_bf16(o[2 * j], lo, b[0], b[1]);
-        mma_bf16(o[2 * j + 1], hi, b[2], b[3]);
-        mma_bf16(o[2 * j + 1], lo, b[2], b[3]);
-      }
-    }
-#pragma unroll
-    for (int y = 0; y < 2; ++y) {
-      const int t = tr + 8 * y;
-      if (t0 + t < n) {
-        bf16* orow = reinterpret_cast<bf16*>(p.out) + (row0 + t0 + t) * p.o_ld + (long long)h * p.P + c0;
-#pragma unroll
-        for (int j = 0; j < CP / 8; ++j) {
-          const int c = j * 8 + scol;
-          if (c >= ncol) continue;
-          const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + t * CPP + c));
-          *reinterpret_cast<__nv_bfloat162*>(orow + c) = __floats2bfloat162_rn(o[j][2 * y] + Dh * x.x, o[j][2 * y + 1] + Dh * x.y);
-        }
-      }
-    }
-    __syncthreads();                                             // scaled values written; old S operands no longer read
-    // ---- state ----
-    const float keep = ex2(total);
+    const float keep = ex2(cv.L[CQ - 1]);
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
       for (int j = 0; j < CP / 8; ++j)
 #pragma unroll
         for (int x = 0; x < 4; ++x) S[i][j][x] *= keep;
+    asm volatile("bar.sync 1, 128;" ::: "memory");               // scaled values written (warps 4-7)
 #pragma unroll
     for (int kb = 0; kb < CQ / 16; ++kb) {
       uint32_t w[2][CP / 16][4];
@@ -440,7 +459,7 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
       for (int i = 0; i < MT; ++i) {
         // A = K^T: rows n, columns s, read transposed from K [s][n]
         uint32_t a[4];
-        ldsm4_t(a, base + L::QK + ((kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * L::NP + warp * (NT / 4) + i * 16 + ((lane >> 3) & 1) * 8) * 2);
+        ldsm4_t(a, base + L::QK + ((kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * L::NP + sw * (NT / 4) + i * 16 + ((lane >> 3) & 1) * 8) * 2);
 #pragma unroll
         for (int x = 0; x < 2; ++x)
 #pragma unroll
@@ -450,6 +469,11 @@ __global__ void __launch_bounds__(128) scan_chunk_kernel(const ScanParams p, int
           }
       }
     }
+    if (sw == 0 && t0 + CQ < n) {
+      prepare(it + 1, t0 + CQ, d);
+      raw_dt(t0 + 2 * CQ, d);
+    }
+    asm volatile("bar.sync 2, 256;" ::: "memory");               // warps 0-3 have read the old operand
     publish();
   }
   if (slot >= 0) {
@@ -478,8 +502,8 @@ int launch_chunk(const ScanParams& p, int nseq, cudaStream_t st) {
     done[dev & 63] = true;
   }
   const int slices = (p.P + CP - 1) / CP;
-  const int conv_parts = p.conv_state ? (p.conv_C + 1023) / 1024 : 0;
-  scan_chunk_kernel<NT><<<dim3(slices + conv_parts, p.heads, nseq), 128, ChunkSmem<NT>::BYTES, st>>>(p, slices, conv_parts);
+  const int conv_parts = p.conv_state ? (p.conv_C + 2047) / 2048 : 0;
+  scan_chunk_kernel<NT><<<dim3(slices + conv_parts, p.heads, nseq), 256, ChunkSmem<NT>::BYTES, st>>>(p, slices, conv_parts);
   dlti_count_launch();
   return (int)cudaGetLastError();
 }

@@ -108,6 +108,7 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   __syncthreads();
   return warp_sum(l < nw ? red[l] : 0.f);
 }
+__device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }    // 16-bit outputs
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 
@@ -337,7 +338,7 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const T* __restrict__ y
 
 // the same in 16-byte pieces for 16-bit T and groups of whole pieces: one CTA per (row, group), everything in registers
 template <typename T, bool GATE_FIRST, bool ACC, int VPT>
-__global__ void __launch_bounds__(256) gated_norm_vec_kernel(const T* __restrict__ y, long long y_ld, const void* __restrict__ gate,
+__global__ void __launch_bounds__(512) gated_norm_vec_kernel(const T* __restrict__ y, long long y_ld, const void* __restrict__ gate,
                                                              long long g_ld, const float* __restrict__ w, T* __restrict__ out,
                                                              long long o_ld, int gs, float eps) {
   __shared__ float red[32];
@@ -362,7 +363,7 @@ __global__ void __launch_bounds__(256) gated_norm_vec_kernel(const T* __restrict
     if (threadIdx.x + i * blockDim.x < vec)
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        const float e = 1.f / (1.f + __expf(-g[i][j]));
+        const float e = fast_sigmoid(g[i][j]);
         if (GATE_FIRST) v[i][j] *= g[i][j] * e;
         else g[i][j] = e;
         ss += v[i][j] * v[i][j];
@@ -523,8 +524,16 @@ __global__ void __launch_bounds__(256) qk_norm_rope_cache_vec_kernel(const QkvPa
         for (int j = 0; j < VE; ++j) v[i][j] = 0.f;
     }
   }
-  float cs[VE / 2], sn[VE / 2];
+  float cs[VE / 2], sn[VE / 2], wq[VE], wk[VE];
   const int ps = p.pos[t];
+#pragma unroll
+  for (int j = 0; j < VE; j += 2) {
+    const float2 one = make_float2(1.f, 1.f);
+    const float2 a = p.qn ? *reinterpret_cast<const float2*>(p.qn + e0 + j) : one;
+    const float2 b = p.kn ? *reinterpret_cast<const float2*>(p.kn + e0 + j) : one;
+    wq[j] = a.x; wq[j + 1] = a.y;
+    wk[j] = b.x; wk[j + 1] = b.y;
+  }
 #pragma unroll
   for (int j = 0; j < VE / 2; ++j) {
     const int pr = e0 / 2 + j;
@@ -542,14 +551,13 @@ __global__ void __launch_bounds__(256) qk_norm_rope_cache_vec_kernel(const QkvPa
     const bool is_q = job < p.H, is_v = job >= p.H + p.G;
     const int g = is_q ? job : (is_v ? job - p.H - p.G : job - p.H);
     if (is_q || (own && !is_v)) {
-      const float* nw = is_q ? p.qn : p.kn;
-      if (nw) {
+      if (is_q ? p.qn : p.kn) {
         float ss = 0.f;
 #pragma unroll
         for (int j = 0; j < VE; ++j) ss += v[i][j] * v[i][j];
-        const float r = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+        const float r = rsqrtf(warp_sum(ss) * (1.f / (32 * VE)) + p.eps);
 #pragma unroll
-        for (int j = 0; j < VE; ++j) v[i][j] *= r * nw[e0 + j];
+        for (int j = 0; j < VE; ++j) v[i][j] *= r * (is_q ? wq[j] : wk[j]);
       }
 #pragma unroll
       for (int j = 0; j < VE / 2; ++j) {
@@ -655,23 +663,30 @@ __global__ void __launch_bounds__(128) short_conv_vec_kernel(const ConvParams p)
   auto emit = [&](long long t, const float (&a)[8]) {
     float f[8];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) f[j] = a[j] / (1.f + __expf(-a[j]));
+    for (int j = 0; j < 8; ++j) f[j] = a[j] * fast_sigmoid(a[j]);
     put_n(out + t * p.o_ld, f);
   };
   if (t0 - row0 >= TAPS - 1 && t0 + nr <= row0 + n) {            // all inputs are rows of this step
-    float x[TAPS - 1 + CONV_ROWS][8];
+    uint4 x[TAPS - 1 + CONV_ROWS];                               // still packed: all loads in flight at half the registers
+    const T* sp = src + (t0 - (TAPS - 1)) * p.ld;
 #pragma unroll
     for (int i = 0; i < TAPS - 1 + CONV_ROWS; ++i)
-      if (i < TAPS - 1 + nr) take_n<T, false, 8>(src + (t0 - (TAPS - 1) + i) * p.ld, 0, x[i]);
+      if (i < TAPS - 1 + nr) x[i] = *reinterpret_cast<const uint4*>(sp + i * p.ld);
 #pragma unroll
     for (int r = 0; r < CONV_ROWS; ++r)
       if (r < nr) {
         float a[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          a[j] = b[j];
+        for (int j = 0; j < 8; ++j) a[j] = b[j];
 #pragma unroll
-          for (int k = 0; k < TAPS; ++k) a[j] += w[k][j] * x[r + k][j];
+        for (int k = 0; k < TAPS; ++k) {
+          const uint32_t u[4] = {x[r + k].x, x[r + k].y, x[r + k].z, x[r + k].w};
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const float2 f = Cvt<T>::unpack2(u[j]);
+            a[2 * j] += w[k][2 * j] * f.x;
+            a[2 * j + 1] += w[k][2 * j + 1] * f.y;
+          }
         }
         emit(t0 + r, a);
       }
@@ -762,7 +777,7 @@ __global__ void __launch_bounds__(128) short_conv_acc_vec_kernel(const ConvParam
     }
   }
 #pragma unroll
-  for (int j = 0; j < 8; ++j) a[j] = a[j] / (1.f + __expf(-a[j]));
+  for (int j = 0; j < 8; ++j) a[j] *= fast_sigmoid(a[j]);
   put_n(reinterpret_cast<T*>(p.out) + t * p.o_ld + c, a);
 }
 
@@ -874,12 +889,12 @@ DLTI_API int dlti_gated_norm(const void* y, long long y_ld, const void* gate, lo
   if (rows <= 0) return 0;
   if (groups < 1 || n % groups) return DLTI_ERR_BAD_ARG;
   const int gs = n / groups;
-  if (dtype == DLTI_BF16 && gs % 8 == 0 && gs <= 8 * 256 * 8 && y_ld % 8 == 0 && g_ld % 8 == 0 && o_ld % 8 == 0 && groups <= 65535 &&
+  if (dtype == DLTI_BF16 && gs % 8 == 0 && gs <= 8 * 512 * 4 && y_ld % 8 == 0 && g_ld % 8 == 0 && o_ld % 8 == 0 && groups <= 65535 &&
       ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
     using B = __nv_bfloat16;
-    const int vec = gs / 8, threads = vec <= 64 ? 64 : (vec <= 128 ? 128 : 256), vpt = (vec + threads - 1) / threads;
+    const int vec = gs / 8, threads = vec <= 64 ? 64 : (vec <= 128 ? 128 : (vec <= 512 ? 256 : 512)), vpt = (vec + threads - 1) / threads;
 #define GNV(GF, AC) (vpt <= 1 ? gated_norm_vec_kernel<B, GF, AC, 1> : vpt <= 2 ? gated_norm_vec_kernel<B, GF, AC, 2> \
-                     : vpt <= 4 ? gated_norm_vec_kernel<B, GF, AC, 4> : gated_norm_vec_kernel<B, GF, AC, 8>)
+                     : gated_norm_vec_kernel<B, GF, AC, 4>)
     auto kern = gate_first ? (acc ? GNV(true, true) : GNV(true, false)) : (acc ? GNV(false, true) : GNV(false, false));
 #undef GNV
     DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)rows, groups), dim3(threads), 0, st, (const B*)y, y_ld, gate, g_ld, w, (B*)out,
