@@ -55,7 +55,11 @@ struct AttnParams {
   long long T_total;
   float scale;           // 1/sqrt(hd)
   int dtype;
-  const float* gate;     // fwd, optional: [T_total, H] factors on the head outputs
+  // split forward only. Rows [0, seq_q0[b]) of sequence b carry keys and values but no query; the output of its first
+  // query row goes to row seq_out0[b] of O (and of the gates). Null: every row is a query, in place.
+  const int *seq_q0, *seq_out0;
+  const float* gate;     // optional [output rows, H] factors on the head outputs
+  int vdim;              // value columns of a head that are written, head h at column h * vdim of O (0: 128)
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
@@ -764,6 +768,8 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
   const int pr = npair - 1 - (int)blockIdx.x;   // heavy (late) pairs first
   if (pr < 0) return;
   const int qbA = 2 * pr, qbB = 2 * pr + 1;
+  const int q0 = (SPLIT && p.seq_q0) ? p.seq_q0[b] : 0;
+  if (SPLIT && (qbB + 1) * 128 <= q0) return;   // both tiles hold no query
   const int nA = qbA + 1, nB = (qbB < nqb) ? qbB + 1 : 0;   // KV blocks each tile attends to
   const int nblk = nB > nA ? nB : nA;
   const bool hasB = nB > 0;
@@ -970,17 +976,21 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
       mbar_wait_b(pv_done + 8 * X, (nX - 1) & 1);
       tc_fence_after();
       const int qi = qbX * 128 + r;
+      const bool write = qi < seqlen && qi >= q0;
+      const long long orow_i = (SPLIT && p.seq_out0) ? p.seq_out0[b] + qi - q0 : row0 + qi;
+      const int vdim = (SPLIT && p.vdim) ? p.vdim : HD;
       float inv = 1.f / l;
-      if (p.gate && qi < seqlen) inv *= p.gate[(long long)(row0 + qi) * p.H + h];
-      T* orow = reinterpret_cast<T*>(p.O) + (long long)(row0 + qi) * p.ldo + h * HD;
+      if (SPLIT && p.gate && write) inv *= p.gate[orow_i * p.H + h];
+      T* orow = reinterpret_cast<T*>(p.O) + orow_i * p.ldo + h * vdim;
 #pragma unroll 1
       for (int c = 0; c < 4; ++c) {
         uint32_t o[32];
         tmem_ld_32x32b_x32(tO + c * 32, o);
         tmem_wait_ld();
-        if (qi < seqlen) {
+        if (write) {
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
+            if (SPLIT && c * 32 + 8 * k >= vdim) break;
             int4 ov;
             uint32_t* ou = reinterpret_cast<uint32_t*>(&ov);
 #pragma unroll
@@ -1064,16 +1074,18 @@ DLTI_API int dlti_attn_fwd(const void* qkv, void* out, float* lse, const int* cu
 }
 
 // dqkv [T, (H+2KV)*128] receives dq | dk | dv. D_scratch: [H, T] fp32 workspace.
-// Inference form with split softmax weights (see attn_fwd2_kernel), bf16, an optional gate [T, H] on the head outputs and
-// an output row pitch ldo (a multiple of 8).
-DLTI_API int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const int* cu_seqlens, int batch,
-                                 int max_seqlen, long long T_total, int H, int KV, int hd, float scale, cudaStream_t st) {
-  if (hd != HD) { dlti_set_error("attention: head_dim must be 128"); return DLTI_ERR_UNSUPPORTED; }
-  if (H % KV || ldo % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return DLTI_ERR_BAD_ARG;
+// Inference form with split softmax weights (see attn_fwd2_kernel), bf16: heads padded to 128 columns in qkv, vdim (a
+// multiple of 8) of them written; optional gate [output rows, H]; output row pitch ldo (a multiple of 8); optional
+// seq_q0 / seq_out0 (see AttnParams) for portions whose earlier keys and values lie in front of their rows.
+DLTI_API int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const int* cu_seqlens, const int* seq_q0,
+                                 const int* seq_out0, int batch, int max_seqlen, long long T_total, int H, int KV, int vdim, float scale,
+                                 cudaStream_t st) {
+  if (H % KV || ldo % 8 || vdim % 8 || vdim < 8 || vdim > HD || (seq_q0 == nullptr) != (seq_out0 == nullptr) || (reinterpret_cast<uintptr_t>(out) & 15)) return DLTI_ERR_BAD_ARG;
   if (batch <= 0 || T_total <= 0) return 0;
   AttnParams p{};
   p.cu_seqlens = cu_seqlens; p.H = H; p.KV = KV; p.W = (H + 2 * KV) * HD;
   p.O = out; p.ldo = ldo; p.T_total = T_total; p.scale = scale; p.dtype = DLTI_BF16; p.gate = gate;
+  p.seq_q0 = seq_q0; p.seq_out0 = seq_out0; p.vdim = vdim;
   CUtensorMap tm;
   const int rc = make_map(&tm, qkv, T_total, p.W, 128);
   if (rc) return rc;

@@ -394,9 +394,13 @@ struct QkvParams {
   const long long* slots; void *kc, *vc; int kd, vd;       // cache row pitches of a head
   void* q; long long q_ld; int q_hd;                       // rotated queries: row pitch, head pitch
   void *kp, *vp;                                           // packed keys / values (row pitch q_ld, head pitch q_hd) or null
+  const int* dst; int nd;                                  // packed: row of token t >= nd is nd + dst[t - nd] (null: t)
   float* gate;                                             // [tokens, H]
   long long tokens; int H, G, dim, vdim;
 };
+__device__ __forceinline__ long long q_row(const QkvParams& p, long long t) {
+  return (p.dst && t >= p.nd) ? p.nd + (long long)p.dst[t - p.nd] : t;
+}
 constexpr int QKV_MAXP = 8;               // pairs per lane: heads of up to 512
 template <typename T, bool ACC>
 __global__ void __launch_bounds__(256) qk_norm_rope_cache_kernel(const QkvParams p) {
@@ -420,7 +424,7 @@ __global__ void __launch_bounds__(256) qk_norm_rope_cache_kernel(const QkvParams
     if (job >= p.H + p.G) {                                          // a value head
       const int g = job - p.H - p.G;
       T* src = reinterpret_cast<T*>(p.vc) + (slot * p.G + g) * p.vd;
-      T* pk = p.vp ? reinterpret_cast<T*>(p.vp) + t * p.q_ld + (long long)g * p.q_hd : nullptr;
+      T* pk = p.vp ? reinterpret_cast<T*>(p.vp) + q_row(p, t) * p.q_ld + (long long)g * p.q_hd : nullptr;
       for (int c = lane; c < p.vdim; c += 32) {
         const T v = own ? Cvt<T>::from_f(take<T, ACC>(row, p.ov + g * p.vdim + c)) : (slot >= 0 ? src[c] : Cvt<T>::from_f(0.f));
         if (own && slot >= 0) src[c] = v;
@@ -431,8 +435,8 @@ __global__ void __launch_bounds__(256) qk_norm_rope_cache_kernel(const QkvParams
     const bool is_q = job < p.H;
     const int head = is_q ? job : job - p.H;
     T* cache = reinterpret_cast<T*>(p.kc) + (slot * p.G + head) * p.kd;
-    T* out = is_q ? reinterpret_cast<T*>(p.q) + t * p.q_ld + (long long)head * p.q_hd
-                  : (p.kp ? reinterpret_cast<T*>(p.kp) + t * p.q_ld + (long long)head * p.q_hd : nullptr);
+    T* out = is_q ? reinterpret_cast<T*>(p.q) + q_row(p, t) * p.q_ld + (long long)head * p.q_hd
+                  : (p.kp ? reinterpret_cast<T*>(p.kp) + q_row(p, t) * p.q_ld + (long long)head * p.q_hd : nullptr);
     if (!is_q && !own) {
       for (int c = lane; c < p.dim; c += 32) out[c] = slot >= 0 ? cache[c] : Cvt<T>::from_f(0.f);
       continue;
@@ -491,86 +495,79 @@ __global__ void __launch_bounds__(256) qk_norm_rope_cache_kernel(const QkvParams
   }
 }
 
-// The same for heads of 32 * VE (64, 128, 256) elements, interleaved pairs and 16-byte aligned sections: a lane owns VE
-// consecutive elements, so its rotation factors are the same for every head; a warp takes up to JPW jobs of one token and
-// issues their loads together.
-template <typename T, bool ACC, int VE, int JPW>
-__global__ void __launch_bounds__(256) qk_norm_rope_cache_vec_kernel(const QkvParams p, int jobs, int kvjobs) {
+// The same for heads of 8 * LPH (64, 128, 256) elements, interleaved pairs and 16-byte aligned sections: LPH lanes share a
+// head (8 consecutive elements each, so a lane's rotation factors are the same for every head), a warp takes 32 / LPH heads
+// of one token at a time and JPW such groups with all their loads in flight.
+template <typename T, bool ACC, int LPH, int JPW>
+__global__ void __launch_bounds__(128) qk_norm_rope_cache_vec_kernel(const QkvParams p, int jobs, int kvjobs) {
+  constexpr int HPW = 32 / LPH, HD = 8 * LPH;
   griddep_wait();
   griddep_launch();
-  const int lane = threadIdx.x & 31;
+  const int lane = threadIdx.x & 31, sub = lane % LPH, e0 = sub * 8, half = p.rot >> 1;
   const long long t = blockIdx.x;
-  const int job0 = (blockIdx.y * 8 + (threadIdx.x >> 5)) * JPW;
+  const int job0 = (blockIdx.y * 4 + (threadIdx.x >> 5)) * (HPW * JPW);
   if (job0 >= jobs) return;
   const uint8_t* row = reinterpret_cast<const uint8_t*>(p.proj) + t * p.ld * (ACC ? 4 : sizeof(T));
   const long long slot = p.slots[t];
+  const int ps = p.pos[t];
+  const long long to = q_row(p, t);
   const bool own = p.ok >= 0;
-  const int e0 = lane * VE, half = p.rot >> 1;
-  float v[JPW][VE];
+  float v[JPW][8];
 #pragma unroll
   for (int i = 0; i < JPW; ++i) {
-    const int job = job0 + i;
-    if (job < p.H) {
-      take_n<T, ACC, VE>(row, p.oq + job * (32 * VE) + e0, v[i]);
-    } else if (job < p.H + kvjobs) {
-      const int kh = job - p.H;                              // G keys, then G values
-      const bool is_k = kh < p.G;
-      const int g = is_k ? kh : kh - p.G;
-      if (own) take_n<T, ACC, VE>(row, (is_k ? p.ok : p.ov) + g * (32 * VE) + e0, v[i]);
-      else if (slot >= 0)
-        take_n<T, false, VE>(reinterpret_cast<const T*>(is_k ? p.kc : p.vc) + (slot * p.G + g) * (is_k ? p.kd : p.vd), e0, v[i]);
-      else
+    const int job = job0 + i * HPW + lane / LPH;
 #pragma unroll
-        for (int j = 0; j < VE; ++j) v[i][j] = 0.f;
+    for (int j = 0; j < 8; ++j) v[i][j] = 0.f;
+    if (job < p.H) {
+      take_n<T, ACC, 8>(row, p.oq + job * HD + e0, v[i]);
+    } else if (job < p.H + kvjobs) {
+      const bool is_k = job < p.H + p.G;
+      const int g = is_k ? job - p.H : job - p.H - p.G;      // G keys, then G values
+      if (own) take_n<T, ACC, 8>(row, (is_k ? p.ok : p.ov) + g * HD + e0, v[i]);
+      else if (slot >= 0)
+        take_n<T, false, 8>(reinterpret_cast<const T*>(is_k ? p.kc : p.vc) + (slot * p.G + g) * (is_k ? p.kd : p.vd), e0, v[i]);
     }
   }
-  float cs[VE / 2], sn[VE / 2], wq[VE], wk[VE];
-  const int ps = p.pos[t];
+  float cs[4], sn[4], wq[8], wk[8];
 #pragma unroll
-  for (int j = 0; j < VE; j += 2) {
-    const float2 one = make_float2(1.f, 1.f);
-    const float2 a = p.qn ? *reinterpret_cast<const float2*>(p.qn + e0 + j) : one;
-    const float2 b = p.kn ? *reinterpret_cast<const float2*>(p.kn + e0 + j) : one;
-    wq[j] = a.x; wq[j + 1] = a.y;
-    wk[j] = b.x; wk[j + 1] = b.y;
-  }
+  for (int j = 0; j < 8; ++j) wq[j] = wk[j] = 1.f;
+  if (p.qn) ld8(p.qn + e0, wq);
+  if (p.kn) ld8(p.kn + e0, wk);
 #pragma unroll
-  for (int j = 0; j < VE / 2; ++j) {
+  for (int j = 0; j < 4; ++j) {
     const int pr = e0 / 2 + j;
     cs[j] = pr < half ? p.cos_t[(long long)ps * half + pr] : 1.f;
     sn[j] = pr < half ? p.sin_t[(long long)ps * half + pr] : 0.f;
   }
 #pragma unroll
   for (int i = 0; i < JPW; ++i) {
-    const int job = job0 + i;
-    if (job >= jobs) break;
-    if (job >= p.H + kvjobs) {
-      for (int h = lane; h < p.H; h += 32) p.gate[t * p.H + h] = sigmoid_f(take<T, ACC>(row, p.og + h));
-      break;
-    }
+    const int job = job0 + i * HPW + lane / LPH;
     const bool is_q = job < p.H, is_v = job >= p.H + p.G;
-    const int g = is_q ? job : (is_v ? job - p.H - p.G : job - p.H);
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss += v[i][j] * v[i][j];
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);     // whole warp, also past the last job
+    if (job >= jobs) continue;
+    if (job >= p.H + kvjobs) {
+      for (int h = sub; h < p.H; h += LPH) p.gate[t * p.H + h] = sigmoid_f(take<T, ACC>(row, p.og + h));
+      continue;
+    }
     if (is_q || (own && !is_v)) {
-      if (is_q ? p.qn : p.kn) {
-        float ss = 0.f;
+      const float r = (is_q ? p.qn : p.kn) ? rsqrtf(ss * (1.f / HD) + p.eps) : 1.f;
 #pragma unroll
-        for (int j = 0; j < VE; ++j) ss += v[i][j] * v[i][j];
-        const float r = rsqrtf(warp_sum(ss) * (1.f / (32 * VE)) + p.eps);
-#pragma unroll
-        for (int j = 0; j < VE; ++j) v[i][j] *= r * (is_q ? wq[j] : wk[j]);
-      }
-#pragma unroll
-      for (int j = 0; j < VE / 2; ++j) {
-        const float a = v[i][2 * j], b = v[i][2 * j + 1];
+      for (int j = 0; j < 4; ++j) {
+        const float a = v[i][2 * j] * r * (is_q ? wq[2 * j] : wk[2 * j]), b = v[i][2 * j + 1] * r * (is_q ? wq[2 * j + 1] : wk[2 * j + 1]);
         v[i][2 * j] = a * cs[j] - b * sn[j];
         v[i][2 * j + 1] = b * cs[j] + a * sn[j];
       }
     }
     if (is_q) {
-      put_n(reinterpret_cast<T*>(p.q) + t * p.q_ld + (long long)g * p.q_hd + e0, v[i]);
+      put_n(reinterpret_cast<T*>(p.q) + to * p.q_ld + job * p.q_hd + e0, v[i]);
     } else {
+      const int g = is_v ? job - p.H - p.G : job - p.H;
       void* pk = is_v ? p.vp : p.kp;
-      if (pk) put_n(reinterpret_cast<T*>(pk) + t * p.q_ld + (long long)g * p.q_hd + e0, v[i]);
+      if (pk) put_n(reinterpret_cast<T*>(pk) + to * p.q_ld + g * p.q_hd + e0, v[i]);
       if (own && slot >= 0) put_n(reinterpret_cast<T*>(is_v ? p.vc : p.kc) + (slot * p.G + g) * (is_v ? p.vd : p.kd) + e0, v[i]);
     }
   }
@@ -781,6 +778,25 @@ __global__ void __launch_bounds__(128) short_conv_acc_vec_kernel(const ConvParam
   put_n(reinterpret_cast<T*>(p.out) + t * p.o_ld + c, a);
 }
 
+// Cached keys and values in front of a portion's rows: packed row rows[i] <- zero queries, keys and values of slot slots[i].
+// 16-byte pieces; heads are `hd` columns apart in the packed rows and kd / vd in the cache.
+__global__ void prefix_rows_kernel(__nv_bfloat16* __restrict__ packed, long long ld, int hd, const int* __restrict__ rows,
+                                   const int* __restrict__ slots, const __nv_bfloat16* __restrict__ kc,
+                                   const __nv_bfloat16* __restrict__ vc, int kd, int vd, int H, int G, long long total) {
+  const int pieces = (H + 2 * G) * (hd / 8);
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / pieces;
+    const int x = (int)(i - r * pieces), head = x / (hd / 8), c = x % (hd / 8) * 8;
+    int4 v = make_int4(0, 0, 0, 0);
+    if (head >= H) {
+      const bool is_k = head < H + G;
+      const int g = is_k ? head - H : head - H - G, w = is_k ? kd : vd;
+      if (c < w) v = *reinterpret_cast<const int4*>((is_k ? kc : vc) + ((long long)slots[r] * G + g) * w + c);
+    }
+    *reinterpret_cast<int4*>(packed + (long long)rows[r] * ld + head * hd + c) = v;
+  }
+}
+
 inline int grid_for(long long total, int block) {
   long long g = (total + block - 1) / block;
   const long long cap = (long long)dlti_num_sms() * 16;
@@ -919,28 +935,29 @@ DLTI_API int dlti_gated_norm(const void* y, long long y_ld, const void* gate, lo
 DLTI_API int dlti_qk_norm_rope_cache(const void* proj, long long ld, int oq, int ok, int ov, int og, const float* qn, const float* kn,
                                      float eps, const int* pos, const float* cos_t, const float* sin_t, int rot, int interleaved,
                                      const long long* slots, void* kc, void* vc, int kd, int vd, void* q, long long q_ld, int q_hd,
-                                     void* kp, void* vp, float* gate, long long tokens, int H, int G, int dim, int vdim, int acc,
+                                     void* kp, void* vp, const int* dst, int nd, float* gate, long long tokens, int H, int G, int dim, int vdim, int acc,
                                      int dtype, cudaStream_t st) {
   if (tokens <= 0) return 0;
   if (rot % 2 || rot > dim || ld % 2) return DLTI_ERR_BAD_ARG;
   if (rot / 2 + (dim - rot + 1) / 2 > 32 * QKV_MAXP) { dlti_set_error("qk_norm_rope_cache: heads of up to 512 dimensions"); return DLTI_ERR_TOO_LARGE; }
   QkvParams p{proj, ld, oq, ok, ov, og, qn, kn, eps, pos, cos_t, sin_t, rot, interleaved, slots, kc, vc, kd, vd,
-              q, q_ld, q_hd, kp, vp, gate, tokens, H, G, dim, vdim};
+              q, q_ld, q_hd, kp, vp, dst, nd, gate, tokens, H, G, dim, vdim};
   const int kvjobs = (ok >= 0 || kp) ? 2 * G : 0, jobs = H + kvjobs + (og >= 0 ? 1 : 0);
   const bool vec = dtype == DLTI_BF16 && (dim == 64 || dim == 128 || dim == 256) && vdim == dim && (interleaved || rot == 0) && ld % 8 == 0 &&
                    q_ld % 8 == 0 && q_hd % 8 == 0 && kd % 8 == 0 && vd % 8 == 0 && oq % 8 == 0 && (ok < 0 || (ok % 8 == 0 && ov % 8 == 0)) &&
                    tokens < (1ll << 31) &&
                    ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kc) |
-                     reinterpret_cast<uintptr_t>(vc) | reinterpret_cast<uintptr_t>(kp) | reinterpret_cast<uintptr_t>(vp)) & 15) == 0;
+                     reinterpret_cast<uintptr_t>(vc) | reinterpret_cast<uintptr_t>(kp) | reinterpret_cast<uintptr_t>(vp) | reinterpret_cast<uintptr_t>(qn) |
+                     reinterpret_cast<uintptr_t>(kn)) & 15) == 0;
   if (vec) {
     using B = __nv_bfloat16;
-#define QKV_CASE(VE)                                                                                                             \
-  if (dim == 32 * VE) {                                                                                                          \
-    const int jpw = acc ? 1 : 4;                                                                                                 \
-    auto kern = acc ? qk_norm_rope_cache_vec_kernel<B, true, VE, 1> : qk_norm_rope_cache_vec_kernel<B, false, VE, 4>;              \
-    DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, kern, dim3((unsigned)tokens, (jobs + 8 * jpw - 1) / (8 * jpw)), dim3(256), 0, st, p, jobs, kvjobs)); \
+#define QKV_CASE(LPH)                                                                                                            \
+  if (dim == 8 * LPH) {                                                                                                          \
+    const int per = 4 * (32 / LPH) * (acc ? 1 : 4);                                                                              \
+    auto kern = acc ? qk_norm_rope_cache_vec_kernel<B, true, LPH, 1> : qk_norm_rope_cache_vec_kernel<B, false, LPH, 4>;            \
+    DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, kern, dim3((unsigned)tokens, (jobs + per - 1) / per), dim3(128), 0, st, p, jobs, kvjobs)); \
   }
-    QKV_CASE(2) QKV_CASE(4) QKV_CASE(8)
+    QKV_CASE(8) QKV_CASE(16) QKV_CASE(32)
 #undef QKV_CASE
     dlti_count_launch();
     return 0;
@@ -950,6 +967,17 @@ DLTI_API int dlti_qk_norm_rope_cache(const void* proj, long long ld, int oq, int
   else DISPATCH_T(dtype, DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, qk_norm_rope_cache_kernel<T, false>, dim3(g), dim3(256), 0, st, p)));
   dlti_count_launch();
   return 0;
+}
+
+DLTI_API int dlti_prefix_rows(void* packed, long long ld, int hd, const int* rows, const int* slots, const void* kc, const void* vc,
+                              int kd, int vd, int H, int G, long long n, cudaStream_t st) {
+  if (n <= 0) return 0;
+  if (ld % 8 || hd % 8 || kd % 8 || vd % 8) return DLTI_ERR_BAD_ARG;
+  const long long total = n * (H + 2 * G) * (hd / 8);
+  prefix_rows_kernel<<<grid_for(total, 256), 256, 0, st>>>((__nv_bfloat16*)packed, ld, hd, rows, slots, (const __nv_bfloat16*)kc,
+                                                           (const __nv_bfloat16*)vc, kd, vd, H, G, total);
+  dlti_count_launch();
+  return (int)cudaGetLastError();
 }
 
 DLTI_API int dlti_short_conv(const void* src, long long ld, int col, int C, int taps, const float* w, const float* b, int w_ld,

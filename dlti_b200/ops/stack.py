@@ -168,11 +168,32 @@ class Rows:
         return r0, n, int(self.ctx[s]) - n
 
 
-def qk_norm_rope_cache(proj, sec, m, q_norm, k_norm, eps, rows: Rows, tabs, kc, vc, dtype, packed=False, acc=False):
+@dataclass
+class Pieces:
+    """The prompt rows of a step as independent causal sequences for one attention chunk size: a prompt is cut at every
+    chunk edge, and a portion that continues a chunk has the chunk's cached keys and values laid out in front of its own
+    rows. cu [n + 1]: boundaries in that extended layout; longest: its longest piece. With cached rows (prefix > 0): q0 [n]
+    = cached rows of a piece, out0 [n] = prompt row of its first own row, dst [prompt rows] = extended row of each prompt
+    row, prow / pslot [prefix] = extended row and cache slot of each cached token."""
+    cu: torch.Tensor
+    longest: int
+    rows: int
+    prefix: int = 0
+    q0: torch.Tensor | None = None
+    out0: torch.Tensor | None = None
+    dst: torch.Tensor | None = None
+    prow: torch.Tensor | None = None
+    pslot: torch.Tensor | None = None
+
+
+PACKED_HD = 128              # head columns of the packed layout
+
+
+def qk_norm_rope_cache(proj, sec, m, q_norm, k_norm, eps, rows: Rows, tabs, kc, vc, dtype, packed: Pieces | None = None, acc=False):
     """Merged projection rows -> rotated queries (each head normalised first when norms are given), keys and values in
     the paged cache at rows.slots, and the sigmoid of the head gates [T, H] (None without gates).
-    packed: also return [q heads | k heads | v heads] rows, the layout of the varlen prefill kernel; keys and values of a
-    layer without own ones are then copied from the cache."""
+    packed: return [q heads | k heads | v heads] rows instead, heads padded to 128 columns, the prompt rows in the extended
+    layout of `packed`; keys and values of a layer without own ones, and of cached rows, are copied from the cache."""
     T, H, G = proj.shape[0], m.heads, m.kv_heads
     own = "k" in sec
     rot = m.rope.dims if m.rope is not None else 0
@@ -201,27 +222,29 @@ def qk_norm_rope_cache(proj, sec, m, q_norm, k_norm, eps, rows: Rows, tabs, kc, 
             kf[rows.slots[ok], :, :m.dim] = k[ok]
             vf[rows.slots[ok], :, :m.vdim] = v[ok]
         gate = torch.sigmoid(proj[:, sec["g"]:sec["g"] + H].float()) if "g" in sec else None
-        if packed:
-            k, v = kf[rows.slots.clamp_min(0)][..., :m.dim], vf[rows.slots.clamp_min(0)][..., :m.vdim]
-            return torch.cat([q.reshape(T, -1), k.reshape(T, -1), v.reshape(T, -1)], 1), gate
         return q.reshape(T, -1), gate
     dev = proj.device
     gate = torch.empty((T, H), dtype=torch.float32, device=dev) if "g" in sec else None
-    if packed:
-        assert m.dim == m.vdim
-        q = torch.empty((T, (H + 2 * G) * m.dim), dtype=dtype, device=dev)
-        hd, es = m.dim, q.element_size()
-        kp, vp = q.data_ptr() + H * hd * es, q.data_ptr() + (H + G) * hd * es
+    kp = vp = dst = None
+    if packed is not None:
+        hd = PACKED_HD
+        n = rows.nd + packed.rows
+        q = (torch.empty if m.dim == m.vdim == hd else torch.zeros)((n, (H + 2 * G) * hd), dtype=dtype, device=dev)
+        kp, vp, dst = q[:, H * hd:], q[:, (H + G) * hd:], packed.dst
     else:
         hd = round8(m.dim)
         q = torch.empty((T, H * hd), dtype=dtype, device=dev)
-        kp = vp = 0
     f = _lib.fn("dlti_qk_norm_rope_cache", [_V, _L, _I, _I, _I, _I, _V, _V, _F, _V, _V, _V, _I, _I, _V, _V, _V, _I, _I, _V, _L, _I, _V,
-                                            _V, _V, _L, _I, _I, _I, _I, _I, _I, _V])
+                                            _V, _V, _I, _V, _L, _I, _I, _I, _I, _I, _I, _V])
     _lib.check(f(_p(proj), proj.stride(0), sec["q"], sec["k"] if own else -1, sec["v"] if own else -1, sec["g"] if "g" in sec else -1,
                  _p(q_norm), _p(k_norm), float(eps), _p(rows.pos), _p(tabs[0]) if rot else None, _p(tabs[1]) if rot else None, rot,
                  int(m.rope.interleaved) if rot else 1, _p(rows.slots), _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(q), q.stride(0), hd,
-                 kp, vp, _p(gate), T, H, G, m.dim, m.vdim, int(acc), _lib.dtype_code(dtype), _lib.stream_ptr()), "qk_norm_rope_cache")
+                 _p(kp), _p(vp), _p(dst), rows.nd, _p(gate), T, H, G, m.dim, m.vdim, int(acc), _lib.dtype_code(dtype),
+                 _lib.stream_ptr()), "qk_norm_rope_cache")
+    if packed is not None and packed.prefix:
+        f = _lib.fn("dlti_prefix_rows", [_V, _L, _I, _V, _V, _V, _V, _I, _I, _I, _I, _L, _V])
+        _lib.check(f(_p(q[rows.nd:]), q.stride(0), hd, _p(packed.prow), _p(packed.pslot), _p(kc), _p(vc), kc.shape[3], vc.shape[3], H, G,
+                     packed.prefix, _lib.stream_ptr()), "prefix_rows")
     return q, gate
 
 
@@ -296,19 +319,17 @@ def attn_paged_prefill(q, m, rows: Rows, kc, vc, gate, out):
     return out
 
 
-def packed_attention(qkv, m, rows: Rows, seg, kc, vc, gate):
-    """Attention of a step from packed [q | k | v] rows (qk_norm_rope_cache(packed=True)): decode rows through the pages,
-    prompt rows as independent causal pieces (seg = (boundaries, longest)) through the varlen tcgen05 kernel. Needs heads
-    of 128 and prompts whose visible keys all belong to this step."""
-    T, H = qkv.shape[0], m.heads
+def packed_attention(qkv, m, rows: Rows, pieces: Pieces, kc, vc, gate):
+    """Attention of a step from the packed rows of qk_norm_rope_cache: decode rows through the pages, prompt rows through the
+    varlen tcgen05 kernel. Needs heads of up to 128 dimensions, values in multiples of 8."""
+    T, H, nd = rows.pos.numel(), m.heads, rows.nd
     out = act(T, H * m.vdim, qkv.dtype, qkv.device)
-    nd = rows.nd
     if nd:
-        attn_paged_decode(qkv[:nd, :H * m.dim], m, rows, kc, vc, gate, out)
+        attn_paged_decode(qkv[:nd, :H * PACKED_HD], m, rows, kc, vc, gate, out)
     q, o, g = qkv[nd:], out[nd:], None if gate is None else gate[nd:]
-    f = _lib.fn("dlti_attn_fwd_split", [_V, _V, _L, _V, _V, _I, _I, _L, _I, _I, _I, _F, _V])
-    _lib.check(f(_p(q), _p(o), o.stride(0), _p(g), _p(seg[0]), seg[0].numel() - 1, seg[1], T - nd, H, m.kv_heads, m.dim, m.scale,
-                 _lib.stream_ptr()), "attn_fwd_split")
+    f = _lib.fn("dlti_attn_fwd_split", [_V, _V, _L, _V, _V, _V, _V, _I, _I, _L, _I, _I, _I, _F, _V])
+    _lib.check(f(_p(q), _p(o), o.stride(0), _p(g), _p(pieces.cu), _p(pieces.q0), _p(pieces.out0), pieces.cu.numel() - 1, pieces.longest,
+                 q.shape[0], H, m.kv_heads, m.vdim, m.scale, _lib.stream_ptr()), "attn_fwd_split")
     return out
 
 

@@ -39,8 +39,7 @@ class StepLayout:
     a prefix copy carries everything but unused table rows.
 
     `full` (runners with per_sequence = True): ctx, tables and the recurrent-state slots sslot cover the prompts
-    too, rseq[T] names each row's sequence, and segs holds the boundaries of the prompt rows cut at the attention
-    chunk edges (one list after the other, nsg entries in all)."""
+    too, rseq[T] names each row's sequence, and segs holds chunk_pieces of every attention chunk size (nsg entries)."""
     _I64 = ("ids", "slots", "last", "seeds", "pslots", "pdst", "csrc")
     _I32 = ("pos", "src", "ctx", "cu", "ecu", "sslot", "rseq", "segs", "topk", "temp", "topp", "tables")
 
@@ -83,20 +82,37 @@ class StepLayout:
         return out
 
 
-def _chunk_segments(cu, starts, chunk: int) -> tuple[list[int], int]:
-    """Boundaries of the prompt rows (relative to the first prompt row) as independent causal sequences: a prompt is
-    cut wherever its position reaches a multiple of `chunk` (0: not at all). Returns (boundaries, longest piece); no
-    boundaries when some prompt continues in the middle of a chunk, whose earlier keys are only in the cache."""
-    out, longest = [0], 0
+PACK_FROM = 64               # longest piece of a step's prompts from which they are laid out for the varlen prefill kernel
+PACK_PREFIX = 4              # ... and the most cached rows in front of them, per prompt row
+
+
+def chunk_pieces(cu, starts, tables, bs: int, chunk: int):
+    """The prompt rows of a step cut where their positions reach a multiple of `chunk` (0: not at all), for
+    ops.stack.Pieces. Returns (int32 array [cu | q0 | out0 | dst | prow | pslot] (only cu without cached rows), pieces,
+    longest piece, extended rows, cached rows), or None when the pieces are too short or the cached part too long."""
+    cue, q0, out0, dst, prow, pslot, longest, own = [0], [], [], [], [], [], 0, 0
     for i, a in enumerate(starts):
         n = cu[i + 1] - cu[i]
-        if (a % chunk) if chunk else a:
-            return [], 0
-        for s in range(0, n, chunk or n):
-            e = min(n, s + (chunk or n))
-            out.append(cu[i] + e)
-            longest = max(longest, e - s)
-    return out, longest
+        lo = a // chunk * chunk if chunk else 0              # first position the first piece sees
+        p, end = a, a + n
+        while p < end:
+            e = min(end, lo + chunk) if chunk else end
+            base, c = cue[-1], p - lo                        # c cached tokens, then rows p .. e
+            if c:
+                j = np.arange(lo, p)
+                prow.append(np.arange(base, base + c))
+                pslot.append(np.asarray(tables[i], dtype=np.int64)[j // bs] * bs + j % bs)
+            q0.append(c)
+            out0.append(cu[i] + p - a)
+            dst.append(np.arange(base + c, base + e - lo))
+            cue.append(base + e - lo)
+            longest, own = max(longest, e - lo), max(own, e - p)
+            p = lo = e
+    prefix = sum(map(len, prow))
+    if own < PACK_FROM or prefix > PACK_PREFIX * cu[-1]:
+        return None
+    arrays = [cue] + ([q0, out0, *dst, *prow, *pslot] if prefix else [])
+    return np.concatenate([np.asarray(x, dtype=np.int32) for x in arrays]), len(q0), longest, cue[-1], prefix
 
 
 class PackedStep:
@@ -104,7 +120,15 @@ class PackedStep:
 
     def __init__(self, layout: StepLayout, slot, max_seqlen: int, max_ext: int = 0, segs: dict | None = None):
         self.layout, self.slot, self.max_seqlen, self.want_lp, self.max_ext = layout, slot, max_seqlen, False, max_ext
-        self.segs = segs or {}       # attention chunk size -> (offset, count, longest) inside the layout's segs section
+        self.segs = segs or {}       # attention chunk size -> (offset in the segs section, then as chunk_pieces)
+
+
+def _pieces(s, n_rows: int, n: int, longest: int, rows: int, prefix: int):
+    from ..ops.stack import Pieces
+    if not prefix:
+        return Pieces(s[:n + 1], longest, rows)
+    o = [n + 1, 2 * n + 1, 3 * n + 1, 3 * n + 1 + n_rows, 3 * n + 1 + n_rows + prefix, 3 * n + 1 + n_rows + 2 * prefix]
+    return Pieces(s[:o[0]], longest, rows, prefix, s[o[0]:o[1]], s[o[1]:o[2]], s[o[2]:o[3]], s[o[3]:o[4]], s[o[4]:o[5]])
 
 
 class LLMEngine:
@@ -254,16 +278,18 @@ class LLMEngine:
         instead of the last row of every sampled sequence."""
         T, npf = len(ids), max(0, len(cu) - 1)
         full = self.per_sequence
-        segs, seg_at = [], {}
+        segs, seg_at, nsg = [], {}, 0
         if full and npf:
             for c in self.cfg.chunks:
-                s, longest = _chunk_segments(cu, starts, c)
-                seg_at[c] = (len(segs), len(s), longest)
-                segs += s
+                pc = chunk_pieces(cu, starts, tables[nd:], self.blocks.block_size, c)
+                if pc is not None:
+                    seg_at[c] = (nsg, *pc[1:])
+                    segs.append(pc[0])
+                    nsg += len(pc[0])
         ns = npf if sampled_prompts is None else sampled_prompts
         mb = max((len(t) for t in tables), default=0)
         mb = (mb + 7) & ~7
-        lay = StepLayout(T, nd, npf, mb, ns, len(prefix[0]) if prefix is not None else 0, full, len(segs),
+        lay = StepLayout(T, nd, npf, mb, ns, len(prefix[0]) if prefix is not None else 0, full, nsg,
                          None if want is None else len(want))
         slot = self._host_buffer("step", lay.words)
         v = lay.views(slot[0].numpy(), np)
@@ -278,7 +304,8 @@ class LLMEngine:
             v["rseq"][:nd] = np.arange(nd)
             if npf:
                 v["rseq"][nd:] = np.repeat(np.arange(nd, nd + npf), np.diff(cu))
-                v["segs"][:] = segs
+                if nsg:
+                    v["segs"][:] = np.concatenate(segs)
         if lay.nt:
             v["ctx"][:] = ctx
             tab = v["tables"]
@@ -444,7 +471,7 @@ class LLMEngine:
             return self._decode_graph(step)
         v = lay.views(self._to_device(step.slot, lay.words), torch)
         if self.per_sequence:
-            segs = {c: (v["segs"][o:o + n], longest) for c, (o, n, longest) in step.segs.items()}
+            segs = {c: _pieces(v["segs"][a[0]:], lay.T - lay.nd, *a[1:]) for c, a in step.segs.items()}
             logits = self.runner.forward(self._feed(v["ids"], v["src"]), v["pos"], v["slots"], num_decode=lay.nd,
                                          block_tables=v["tables"], ctx_lens=v["ctx"], cu_seqlens=v["cu"] if lay.npf else None,
                                          max_seqlen=step.max_seqlen, last_idx=v["last"] if lay.npf else None,

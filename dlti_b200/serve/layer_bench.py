@@ -180,10 +180,11 @@ def kernels(width: int, peaks: dict, nseq: int, length: int, batch: int, ctx: in
     # attention, whole prompts: the same number of visible pairs for both (Llama sees pieces of `chunk` as prompts)
     cut = [i * length + s for i in range(nseq) for s in range(0, length, att.chunk)] + [T]
     seg = (torch.tensor(cut, dtype=torch.int32, device=dev), min(length, att.chunk))
+    pieces = K.Pieces(seg[0], seg[1], T)
     qkv, gate = rnd(T, (H + 2 * G) * hd), torch.rand(T, H, device=dev)
     fl = 4.0 * nseq * pairs(length, att.chunk) * H * hd
     io = T * (2 * H + 2 * G) * hd * 2
-    k.run("sigosun", "prefill", "attention (packed)", lambda: K.packed_attention(qkv, att, pr, seg, kc, vc, gate), io, fl)
+    k.run("sigosun", "prefill", "attention (packed)", lambda: K.packed_attention(qkv, att, pr, pieces, kc, vc, gate), io, fl)
     k.run("llama", "prefill", "attention", lambda: A.attention_fwd(qkv, seg[0], seg[1], H, G, hd, want_lse=False), io, fl)
     q = rnd(T, H * hd)
     out = K.act(T, H * hd, bf, dev)
@@ -198,7 +199,7 @@ def kernels(width: int, peaks: dict, nseq: int, length: int, batch: int, ctx: in
         acc = phase == "decode"
         proj = torch.zeros(n, sec.total, device=dev) if acc else rnd(n, sec.total)
         k.run("sigosun", phase, "q/k norm + rope + cache", lambda: K.qk_norm_rope_cache(
-            proj, sec, att, fa, fa, 1e-6, r, tab_r, kc, vc, bf, packed=not acc, acc=acc),
+            proj, sec, att, fa, fa, 1e-6, r, tab_r, kc, vc, bf, packed=None if acc else pieces, acc=acc),
             n * (sec.total * (8 if acc else 2) + (H + (0 if acc else 2 * G)) * hd * 2 + 2 * G * hd * 2 + 4 * H))
         W = (H + 2 * G) * hd
         if acc:

@@ -18,7 +18,6 @@ from .kv_cache import KVCache, KVSpec, StateCache, StateSpec
 
 
 _FUSE_ACC = os.environ.get("DLTI_DECODE_FUSE_ACC", "1") == "1"    # A/B switch: consume the fp32 accumulators directly
-_PACKED_FROM = 64            # longest piece of a step from which the packed prefill kernel pays
 
 
 class StackRunner:
@@ -48,13 +47,14 @@ class StackRunner:
         if self.device.type == "cuda" and "DLTI_PDL" not in os.environ:
             # serving weights are static: the decode GEMMs may fetch weight tiles while the previous kernel drains
             _lib.gpu_lib().dlti_set_pdl(2)
+        self.pack_prompts = True     # False: all prompt attention reads the pages
         self.trace = None            # set to a list: receives the residual stream after every layer (debugging)
 
     @torch.no_grad()
     def forward(self, input_ids, positions, slots, *, num_decode: int = 0, block_tables=None, ctx_lens=None, cu_seqlens=None,
                 max_seqlen: int = 0, last_idx=None, max_ctx: int = 0, state_slots=None, row_seq=None, segs=None) -> torch.Tensor:
-        """One pass over T token rows (see ops.stack.Rows for the arguments). segs: attention chunk size -> (boundaries of
-        the prompt rows as independent causal pieces, longest piece). Returns fp32 logits of the rows `last_idx`."""
+        """One pass over T token rows (see ops.stack.Rows for the arguments). segs: attention chunk size ->
+        ops.stack.Pieces of the prompt rows (none: prompt attention reads the pages). Returns fp32 logits of the rows `last_idx`."""
         cfg, w = self.cfg, self.w
         rows = K.Rows(positions, row_seq, slots, ctx_lens, cu_seqlens, block_tables, state_slots, int(num_decode), max_seqlen,
                       max_ctx)
@@ -86,16 +86,17 @@ class StackRunner:
         return K.post_norm_add_(y, x, norm, self.cfg.norm_eps, self.cfg.norm_one_plus, self.dtype, acc=self.acc)
 
     def _attention(self, i, m: AttentionMixer, lw, xa, rows: K.Rows, segs):
-        seg = (segs or {}).get(m.chunk)
-        # whole prompts with heads of 128: the varlen tcgen05 kernel on rows cut at the chunk edges; everything else
-        # (portions that continue a chunk, other head sizes, fp32) reads the pages
-        packed = (seg is not None and seg[0].numel() > 1 and m.dim == m.vdim == 128 and self.dtype == torch.bfloat16
-                  and seg[1] >= _PACKED_FROM and xa.is_cuda)
+        # prompts with heads of up to 128: the varlen tcgen05 kernel on rows cut at the chunk edges; everything else
+        # (short portions, larger heads, fp32) reads the pages
+        packed = None
+        if (xa.is_cuda and self.dtype == torch.bfloat16 and 32 < max(m.dim, m.vdim) <= K.PACKED_HD and m.vdim % 8 == 0
+                and self.pack_prompts):
+            packed = (segs or {}).get(m.chunk)
         proj = gemm_skinny_acc(xa, lw["w_in"]) if self.acc else K.linear(xa, lw["w_in"])
         q, gate = K.qk_norm_rope_cache(proj, self.sections[i], m, lw.get("q_norm"), lw.get("k_norm"), self.cfg.norm_eps, rows,
                                        self.ropes[i], self.kv.k[i], self.kv.v[i], self.dtype, packed=packed, acc=self.acc)
-        if packed:
-            return K.packed_attention(q, m, rows, seg, self.kv.k[i], self.kv.v[i], gate)
+        if packed is not None:
+            return K.packed_attention(q, m, rows, packed, self.kv.k[i], self.kv.v[i], gate)
         return K.paged_attention(q, m, rows, self.kv.k[i], self.kv.v[i], gate)
 
     def _mamba2(self, i, m: Mamba2Mixer, lw, xa, rows: K.Rows):
