@@ -360,7 +360,7 @@ def short_conv(proj, col, C_, w, b, state, rows: Rows, dtype, acc=False, width=0
             r0, n, start = rows.bounds(s)
             x = proj[r0:r0 + n, col:col + C_].float()
             slot = int(rows.state[s])
-            h = state[slot].float() if start > 0 and slot >= 0 else torch.zeros(taps - 1, C_)
+            h = state[slot].float() if state is not None and start > 0 and slot >= 0 else torch.zeros(taps - 1, C_)
             x = torch.cat([h, x])
             out[r0:r0 + n] = b[:C_] + sum(w[k, :C_] * x[k:k + n] for k in range(taps))
         return torch.nn.functional.silu(out).to(dtype), proj
