@@ -348,6 +348,78 @@ int dlti_sample(const void* logits, long long ld, int batch, int V, const float*
                 unsigned long long step, long long* out, float* out_logprob, int dtype,
                 dlti_stream_t stream);
 
+/* ---- Layer-stack models (models/stack.py): csrc/stack.cu, recurrent.cu, attention_paged.cu, gemm_f32.cu. Row pitches (*_ld) in
+ * elements. Sequences of a step: the first nd are single rows, sequence nd + i has rows nd + cu[i] ... nd + cu[i+1]; ctx[s] = tokens
+ * of sequence s after the step, rseq[t] = sequence of row t, sslot[s] = its state slot (-1 = none). */
+/* C[M,N] = A[M,K] * B[N,K]^T in true fp32 (no TF32) */
+int dlti_gemm_f32(const float* A, const float* B, float* C, int M, int N, int K, long long lda, long long ldb, long
+    long ldc, dlti_stream_t stream);
+/* x[t] = table[ids[t]] as fp32; xa (16-bit, may be NULL) = the same rows */
+int dlti_embed_rows(const long long* ids, const void* table, float* x, void* xa, long long xa_ld, long long tokens, int
+    d, long long vocab, int dtype, dlti_stream_t stream);
+/* out = acc, acc = 0 (fp32 logits of the decode GEMM) */
+int dlti_take_rows(float* acc, float* out, long long rows, int cols, dlti_stream_t stream);
+/* x += RMSnorm(y) * w (1 + w with one_plus), fp32 residual x [rows,d]; xa (may be NULL) = x in dtype.
+ * acc: y is the fp32 accumulator of dlti_gemm_skinny, zero on return (also below) */
+int dlti_post_norm_add(const void* y, long long y_ld, float* x, const float* w, void* xa, long long xa_ld, long long
+    rows, int d, float eps, int one_plus, int acc, int dtype, dlti_stream_t stream);
+/* out[i] = RMSnorm(x[idx[i]]) * w; idx NULL = all rows */
+int dlti_rms_rows(const float* x, const long long* idx, const float* w, void* out, long long out_ld, long long rows,
+    int d, float eps, int one_plus, int dtype, dlti_stream_t stream);
+/* h = relu(u)^2 over the first ff columns */
+int dlti_relu2(const void* u, long long u_ld, void* h, long long h_ld, long long rows, int ff, int acc, int dtype,
+    dlti_stream_t stream);
+/* norm over `groups` parts of a row: gate_first ? norm(y * silu(gate)) * w : norm(y) * w * sigmoid(gate) */
+int dlti_gated_norm(const void* y, long long y_ld, const void* gate, long long g_ld, const float* w, void* out, long
+    long o_ld, long long rows, int n, int groups, float eps, int gate_first, int acc, int dtype, dlti_stream_t stream);
+/* projection rows (sections at columns oq/ok/ov/og; ok, og < 0 = absent) -> normed and rotated q, k and v into the paged
+ * cache at slots[t] (-1 = skip), sigmoid of the head gates. kp/vp: also packed k, v rows; dst: packed row of row t >= nd */
+int dlti_qk_norm_rope_cache(const void* proj, long long ld, int oq, int ok, int ov, int og, const float* qn, const
+    float* kn, float eps, const int* pos, const float* cos_t, const float* sin_t, int rot, int interleaved, const long
+    long* slots, void* kc, void* vc, int kd, int vd, void* q, long long q_ld, int q_hd, void* kp, void* vp, const int*
+    dst, int nd, float* gate, long long tokens, int H, int G, int dim, int vdim, int acc, int dtype, dlti_stream_t
+    stream);
+/* packed rows[i] <- zero queries, cached keys and values of slots[i] (portions that continue a chunk) */
+int dlti_prefix_rows(void* packed, long long ld, int hd, const int* rows, const int* slots, const void* kc, const void*
+    vc, int kd, int vd, int H, int G, long long n, dlti_stream_t stream);
+/* silu(causal convolution) of channels [col, col+C) of the rows of every sequence; inputs before the step come from state */
+int dlti_short_conv(const void* src, long long ld, int col, int C, int taps, const float* w, const float* b, int w_ld,
+    const void* state, const int* sslot, const int* rseq, const int* ctx, const int* cu, int nd, void* out, long long
+    o_ld, void* raw, long long raw_ld, int raw_n, long long rows, int acc, int dtype, dlti_stream_t stream);
+/* S <- a S + k (s v)^T, o = S^T q + D v token by token over sequences [seq0, seq0+nseq); a constant (decay) or from raw step
+ * sizes (dt, dt_bias, A_log); state [slots, heads, N, P] fp32; tail job: new convolution state from conv_src */
+int dlti_linear_scan(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long v_ld, int
+    rep, int silu, const float* decay, const void* dt, long long dt_ld, const float* dt_bias, const float* A_log, const
+    float* D, float* state, const int* sslot, const int* ctx, const int* cu, int nd, int seq0, int nseq, int heads, int
+    N, int P, void* out, long long o_ld, const void* conv_src, long long conv_ld, int conv_col, int conv_rows, int
+    conv_C, void* conv_state, int dtype, dlti_stream_t stream);
+/* the same for prompt sequences, 64 tokens at a time on the tensor cores (bf16) */
+int dlti_linear_scan_chunked(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long
+    v_ld, int rep, const float* decay, const void* dt, long long dt_ld, const float* dt_bias, const float* A_log, const
+    float* D, float* state, const int* sslot, const int* ctx, const int* cu, int nd, int seq0, int nseq, int heads, int
+    N, int P, void* out, long long o_ld, const void* conv_src, long long conv_ld, int conv_col, int conv_rows, int
+    conv_C, void* conv_state, dlti_stream_t stream);
+/* x = silu(x) in place */
+int dlti_silu_rows(void* x, long long ld, long long rows, int n, int dtype, dlti_stream_t stream);
+/* paged attention, one warp per (row, head), fp32 arithmetic; chunk > 0: a position sees its own chunk only */
+int dlti_attn_rows(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd, const int*
+    tables, int max_blocks, int bs, const int* ctx, const int* rseq, const int* pos, int H, int G, int dim, int vdim,
+    int chunk, float scale, const float* gate, void* out, long long o_ld, long long rows, int dtype, dlti_stream_t
+    stream);
+/* paged attention of prompt portions (bf16, heads <= 256) */
+int dlti_attn_paged_prefill(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
+    const int* tables, int max_blocks, int bs, const int* ctx, const int* cu, int nd, int nseq, int max_rows, int H,
+    int G, int dim, int vdim, int chunk, float scale, const float* gate, void* out, long long o_ld, dlti_stream_t
+    stream);
+/* paged attention of decode rows (bf16, grouped heads, split over CTAs); ws: batch * H * splits * (vdim + 2) floats */
+int dlti_attn_paged_decode(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
+    const int* tables, int max_blocks, int bs, const int* ctx, int batch, int H, int G, int dim, int vdim, int chunk,
+    float scale, const float* gate, int splits, float* ws, void* out, long long o_ld, dlti_stream_t stream);
+/* varlen causal attention with the softmax weights as two bf16 terms; see attention.cu */
+int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const int* cu_seqlens, const int*
+    seq_q0, const int* seq_out0, int batch, int max_seqlen, long long T_total, int H, int KV, int vdim, float scale,
+    dlti_stream_t stream);
+
 #ifdef DLTI_ATTN_TRACE
 /* Developer builds only (-DDLTI_ATTN_TRACE): clock64() timeline of CTA (0,0,0) of the last backward
  * kernels, [dQ | dK/dV][role: softmax, mma, producer][iteration < 64][event < 4]. */
