@@ -116,30 +116,47 @@ __device__ __forceinline__ void zero_pads(uint8_t* smem, int kd, int vd) {
   for (int st = 0; st < 2; ++st) {
     bf16* k = reinterpret_cast<bf16*>(smem + st * L::BYTES);
     bf16* v = reinterpret_cast<bf16*>(smem + st * L::BYTES + L::K_BYTES);
-    for (int i = threadIdx.x; i < KT * (DK - kd); i += blockDim.x) k[(i / (DK - kd)) * L::KP + kd + i % (DK - kd)] = __float2bfloat16(0.f);
-    for (int i = threadIdx.x; i < KT * (DV - vd); i += blockDim.x) v[(i / (DV - vd)) * L::VP + vd + i % (DV - vd)] = __float2bfloat16(0.f);
+    if (kd < DK)
+      for (int i = threadIdx.x; i < KT * (DK - kd); i += blockDim.x) k[(i / (DK - kd)) * L::KP + kd + i % (DK - kd)] = __float2bfloat16(0.f);
+    if (vd < DV)
+      for (int i = threadIdx.x; i < KT * (DV - vd); i += blockDim.x) v[(i / (DV - vd)) * L::VP + vd + i % (DV - vd)] = __float2bfloat16(0.f);
   }
 }
+// A thread's first 16-byte piece of a tile's keys / values and its step to the next one: no divisions in the loops
+struct Walk {
+  int kn, kr, kc, kdr, kdc, vn, vr, vc, vdr, vdc;
+  __device__ __forceinline__ explicit Walk(const PagedParams& p) {
+    const int t = threadIdx.x, n = blockDim.x;
+    kn = p.kd >> 3; kr = t / kn; kc = t % kn; kdr = n / kn; kdc = n % kn;
+    vn = p.vd >> 3; vr = t / vn; vc = t % vn; vdr = n / vn; vdc = n % vn;
+  }
+};
 // cp.async of keys and values [j0, j0 + 64) of one head of the sequence; rows at or past jend become zeros
 template <int DK, int DV>
-__device__ __forceinline__ void load_tile(uint32_t stage, const PagedParams& p, const int* slots, int g, int j0, int jend) {
+__device__ __forceinline__ void load_tile(uint32_t stage, const PagedParams& p, const Walk& w, const int* slots, int g, int j0, int jend) {
   using L = Tile<DK, DV>;
-  const int kc = p.kd >> 3, vc = p.vd >> 3, per = kc + vc;
-  const bf16* K = reinterpret_cast<const bf16*>(p.kc);
-  const bf16* V = reinterpret_cast<const bf16*>(p.vc);
-  for (int i = threadIdx.x; i < KT * per; i += blockDim.x) {
-    const int r = i / per, c = i - r * per;
-    const bool ok = j0 + r < jend;
-    const long long row = (long long)slots[r] * p.G + g;
-    if (c < kc) cp_async16(stage + (r * L::KP + c * 8) * 2, K + row * p.kd + c * 8, ok);
-    else cp_async16(stage + L::K_BYTES + (r * L::VP + (c - kc) * 8) * 2, V + row * p.vd + (c - kc) * 8, ok);
+  const bf16* K = reinterpret_cast<const bf16*>(p.kc) + g * p.kd;
+  const bf16* V = reinterpret_cast<const bf16*>(p.vc) + g * p.vd;
+  const int ks = p.G * p.kd, vs = p.G * p.vd;
+  for (int r = w.kr, c = w.kc; r < KT;) {
+    cp_async16(stage + (r * L::KP + c * 8) * 2, K + (long long)slots[r] * ks + c * 8, j0 + r < jend);
+    r += w.kdr;
+    c += w.kdc;
+    if (c >= w.kn) { c -= w.kn; ++r; }
+  }
+  for (int r = w.vr, c = w.vc; r < KT;) {
+    cp_async16(stage + L::K_BYTES + (r * L::VP + c * 8) * 2, V + (long long)slots[r] * vs + c * 8, j0 + r < jend);
+    r += w.vdr;
+    c += w.vdc;
+    if (c >= w.vn) { c -= w.vn; ++r; }
   }
   cp_async_commit();
 }
 __device__ __forceinline__ void tile_slots(int* slots, const PagedParams& p, const int* tab, int j0, int jend) {
   if (threadIdx.x < KT) {
     const int j = min(j0 + (int)threadIdx.x, jend - 1);
-    slots[threadIdx.x] = tab[j / p.bs] * p.bs + j % p.bs;
+    const int b = (p.bs & (p.bs - 1)) ? j / p.bs : j >> (31 - __clz(p.bs));
+    slots[threadIdx.x] = tab[b] * p.bs + j - b * p.bs;
   }
 }
 // this thread's elements of query rows as A fragments; q0 / q1: rows lane / 4 and lane / 4 + 8 (null: zeros)
@@ -239,17 +256,18 @@ __global__ void __launch_bounds__(256) attn_prefill_kernel(const PagedParams p) 
     for (int x = 0; x < 4; ++x) o[i][x] = 0.f;
   const float sl2 = p.scale * LOG2E_F;
   const uint32_t sbase = smem_u32(smem);
+  const Walk walk(p);
   zero_pads<DK, DV>(smem, p.kd, p.vd);
   tile_slots(s_slots[0], p, tab, jbeg, jend);
   __syncthreads();
-  load_tile<DK, DV>(sbase, p, s_slots[0], g, jbeg, jend);
+  load_tile<DK, DV>(sbase, p, walk, s_slots[0], g, jbeg, jend);
   int it = 0;
   for (int j0 = jbeg; j0 < jend; j0 += KT, ++it) {
     const bool more = j0 + KT < jend;
     if (more) tile_slots(s_slots[(it + 1) & 1], p, tab, j0 + KT, jend);
     __syncthreads();                               // the other stage is free, its slots are written
     if (more) {
-      load_tile<DK, DV>(sbase + ((it + 1) & 1) * L::BYTES, p, s_slots[(it + 1) & 1], g, j0 + KT, jend);
+      load_tile<DK, DV>(sbase + ((it + 1) & 1) * L::BYTES, p, walk, s_slots[(it + 1) & 1], g, j0 + KT, jend);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
@@ -346,10 +364,11 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const PagedParams p, i
     for (int x = 0; x < 4; ++x) o[i][x] = 0.f;
   const uint32_t sbase = smem_u32(smem);
   if (jbeg < jend) {
+    const Walk walk(p);
     zero_pads<DK, DV>(smem, p.kd, p.vd);
     tile_slots(s_slots[0], p, tab, jbeg, jend);
     __syncthreads();
-    load_tile<DK, DV>(sbase, p, s_slots[0], g, jbeg, jend);
+    load_tile<DK, DV>(sbase, p, walk, s_slots[0], g, jbeg, jend);
     uint32_t qf[DK / 16][4];
     const bf16* q = reinterpret_cast<const bf16*>(p.q) + (long long)b * p.q_ld + (long long)(g * rep + h0) * p.q_hd;
     const int r0 = lane >> 2, r1 = r0 + 8;
@@ -361,7 +380,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const PagedParams p, i
       if (more) tile_slots(s_slots[(it + 1) & 1], p, tab, j0 + KT, jend);
       __syncthreads();
       if (more) {
-        load_tile<DK, DV>(sbase + ((it + 1) & 1) * L::BYTES, p, s_slots[(it + 1) & 1], g, j0 + KT, jend);
+        load_tile<DK, DV>(sbase + ((it + 1) & 1) * L::BYTES, p, walk, s_slots[(it + 1) & 1], g, j0 + KT, jend);
         cp_async_wait<1>();
       } else {
         cp_async_wait<0>();

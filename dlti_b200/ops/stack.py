@@ -299,7 +299,7 @@ def attn_paged_decode(q, m, rows: Rows, kc, vc, gate, out, splits: int | None = 
     if splits is None:
         reach = min(rows.max_ctx or 1 << 30, m.chunk or 1 << 30, rows.tables.shape[1] * bs)
         ctas = max(1, B) * m.kv_heads * -(-(m.heads // m.kv_heads) // 16)
-        splits = max(1, min(32, -(-3 * 148 // ctas), -(-reach // 128)))
+        splits = max(1, min(32, 3 * 148 // ctas, -(-reach // 64)))     # one wave of three CTAs per SM
     ws = _workspace(q.device, B * m.heads * splits * (m.vdim + 2)) if splits > 1 else None
     f = _lib.fn("dlti_attn_paged_decode", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _I, _I, _I, _I, _I, _I, _F, _V, _I, _V, _V, _L, _V])
     _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], bs,
