@@ -21,7 +21,7 @@ from ..ops import elementwise as E
 from ..ops import serving as S
 from ..ops import stack as K
 from ..ops.gemm import gemm, gemm_skinny, gemm_skinny_acc
-from .engine import LLMEngine
+from .engine import LLMEngine, _pieces, chunk_pieces
 from .model_runner import TPContext
 from .tokenizer import ByteTokenizer
 
@@ -188,7 +188,16 @@ def kernels(width: int, peaks: dict, nseq: int, length: int, batch: int, ctx: in
     k.run("llama", "prefill", "attention", lambda: A.attention_fwd(qkv, seg[0], seg[1], H, G, hd, want_lse=False), io, fl)
     q = rnd(T, H * hd)
     out = K.act(T, H * hd, bf, dev)
-    k.run("sigosun", "prefill", "attention (portions, paged)", lambda: K.attn_paged_prefill(q, att, pr, kc, vc, gate, out), io, fl)
+    k.run("sigosun", "prefill", "attention (paged, heads > 128)", lambda: K.attn_paged_prefill(q, att, pr, kc, vc, gate, out), io, fl)
+    # the second half of every prompt, its first half cached
+    h = length // 2
+    own = _rows([(h, length - h)] * nseq, 0, tabs[:nseq].contiguous(), pslots.view(nseq, -1)[:, h:].reshape(-1), length)
+    arr, n_p, longest, ext, prefix = chunk_pieces([i * (length - h) for i in range(nseq + 1)], [h] * nseq, tabs[:nseq].tolist(), bs, att.chunk)
+    half = _pieces(torch.from_numpy(arr).to(dev), nseq * (length - h), n_p, longest, ext, prefix)
+    packed2 = rnd(ext, (H + 2 * G) * hd)
+    k.run("sigosun", "prefill", "attention (packed, half cached)", lambda: K.packed_attention(packed2, att, own, half, kc, vc, gate),
+          nseq * ((length - h) * 2 * H + length * 2 * G) * hd * 2, fl - 4.0 * nseq * pairs(h, att.chunk) * H * hd)
+    del packed2
     # attention, decode
     qd, gd, od = rnd(batch, H * hd), torch.rand(batch, H, device=dev), K.act(batch, H * hd, bf, dev)
     k.run("sigosun", "decode", "attention", lambda: K.attn_paged_decode(qd, att, dr, kc, vc, gd, od), batch * seen * G * hd * 4)
