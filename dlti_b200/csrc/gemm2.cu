@@ -45,6 +45,7 @@ struct Gemm2Params {
   int out_dtype, in_dtype;
   int accumulate;
   int vec_ok;
+  int relu2;        // 16-bit outputs become the square of their relu
   float alpha;
   uint32_t idesc;
   // Ragged last wave: when the tiles left for the last wave fill at most half of the clusters, each of them
@@ -805,6 +806,13 @@ gemm2_kernel(const Gemm2Params p, const GatherJob gj, const WaitSpec ws_, const 
             const uint16_t* rrow =
                 p.R ? reinterpret_cast<const uint16_t*>(p.R) + (long long)row * p.ldr + col0 : nullptr;
             const bool bf = p.out_dtype == DLTI_BF16;
+            if (p.relu2) {                 // same rounding points as the GEMM followed by the relu^2 kernel
+#pragma unroll
+              for (int i = 0; i < 32; ++i) {
+                const float x = fmaxf(bf ? __bfloat162float(__float2bfloat16_rn(f[i])) : __half2float(__float2half_rn(f[i])), 0.f);
+                f[i] = x * x;
+              }
+            }
             if (full) {
               if (rrow) {
 #pragma unroll
@@ -1091,11 +1099,11 @@ DLTI_API int dlti_gather_job_run(int ctas, cudaStream_t stream) {
 // configurations it does not cover (the caller then uses the 1-CTA kernel). stream_k: -1 = automatic
 // (ragged last wave only, and only when DLTI_GEMM_STREAMK=1), 0 = never, 1 = whenever the tile count is
 // not a multiple of the cluster count.
-DLTI_API int dlti_gemm_2cta(const void* A, const void* B, void* C, const void* R, int M, int N, int K,
-                            long long lda, long long ldb, long long ldc, long long ldr, int b_mn,
-                            const void* A2, const void* B2, int K2, long long lda2, long long ldb2,
-                            int in_dtype, int out_dtype, float alpha, int accumulate, int stream_k,
-                            cudaStream_t stream) {
+static int gemm_2cta_impl(const void* A, const void* B, void* C, const void* R, int M, int N, int K,
+                          long long lda, long long ldb, long long ldc, long long ldr, int b_mn,
+                          const void* A2, const void* B2, int K2, long long lda2, long long ldb2,
+                          int in_dtype, int out_dtype, float alpha, int accumulate, int stream_k, int relu2,
+                          cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return DLTI_ERR_BAD_ARG;
   if (in_dtype != DLTI_BF16 && in_dtype != DLTI_FP16) return DLTI_ERR_UNSUPPORTED;
   if (K2 % BK) return DLTI_ERR_BAD_ARG;
@@ -1107,7 +1115,7 @@ DLTI_API int dlti_gemm_2cta(const void* A, const void* B, void* C, const void* R
   p.nkb_main = (K + BK - 1) / BK;
   p.nkb_ext = (A2 && B2) ? K2 / BK : 0;
   p.C = C; p.R = R; p.ldc = ldc; p.ldr = ldr;
-  p.out_dtype = out_dtype; p.in_dtype = in_dtype; p.accumulate = accumulate;
+  p.out_dtype = out_dtype; p.in_dtype = in_dtype; p.accumulate = accumulate; p.relu2 = relu2;
   const int ob = out_dtype == DLTI_FP32 ? 4 : 2;
   p.vec_ok = ((reinterpret_cast<uintptr_t>(C) & 15) == 0) && ((ldc * ob) % 16 == 0) &&
              (!R || (((reinterpret_cast<uintptr_t>(R) & 15) == 0) && ((ldr * 2) % 16 == 0)));
@@ -1156,6 +1164,21 @@ DLTI_API int dlti_gemm_2cta(const void* A, const void* B, void* C, const void* R
   set_tail_split(p, grid, in_dtype, b_mn != 0);
   return b_mn ? launch2<true>(p, ta, tb, ta2, tb2, tbh, tb2h, grid, stream)
               : launch2<false>(p, ta, tb, ta2, tb2, tbh, tb2h, grid, stream);
+}
+
+DLTI_API int dlti_gemm_2cta(const void* A, const void* B, void* C, const void* R, int M, int N, int K,
+                            long long lda, long long ldb, long long ldc, long long ldr, int b_mn,
+                            const void* A2, const void* B2, int K2, long long lda2, long long ldb2,
+                            int in_dtype, int out_dtype, float alpha, int accumulate, int stream_k,
+                            cudaStream_t stream) {
+  return gemm_2cta_impl(A, B, C, R, M, N, K, lda, ldb, ldc, ldr, b_mn, A2, B2, K2, lda2, ldb2, in_dtype, out_dtype, alpha, accumulate,
+                        stream_k, 0, stream);
+}
+
+// h = relu(x W^T)^2: the up projection of a squared-relu feed-forward with the activation in the epilogue
+DLTI_API int dlti_gemm_relu2_2cta(const void* X, const void* W, void* Hout, int M, int N, int K, long long ldx, long long ldw,
+                                  long long ldh, int dtype, cudaStream_t stream) {
+  return gemm_2cta_impl(X, W, Hout, nullptr, M, N, K, ldx, ldw, ldh, 0, 0, nullptr, nullptr, 0, 0, 0, dtype, dtype, 1.f, 0, -1, 1, stream);
 }
 
 // h[M, ff] = silu(A · Wg^T) * (A · Wu^T) with W = [gate rows (ff) ; up rows (ff)] stored [2*ff, K]

@@ -178,6 +178,21 @@ def gemm_swiglu(x: torch.Tensor, w_gu: torch.Tensor, gather=None) -> torch.Tenso
     return h
 
 
+def gemm_relu2(x: torch.Tensor, w_up: torch.Tensor, ff: int) -> torch.Tensor | None:
+    """h = relu(x · W^T)^2 with the activation in the CTA-pair GEMM's epilogue (csrc/gemm2.cu), [M, ff] with a row pitch of
+    w_up's rows (ff rounded up to 8). None when the shape is not covered (fewer than 64 tiles)."""
+    M, K = x.shape
+    N = w_up.shape[0]
+    if not _TWO_CTA_DEFAULT or x.dtype == torch.float32 or x.stride(1) != 1 or ((M + 255) // 256) * ((N + 255) // 256) < 64:
+        return None
+    h = torch.empty((M, N), dtype=x.dtype, device=x.device)
+    f = _lib.fn("dlti_gemm_relu2_2cta", [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_longlong, C.c_longlong,
+                                         C.c_longlong, C.c_int, C.c_void_p])
+    _lib.check(f(_lib.ptr(x), _lib.ptr(w_up), _lib.ptr(h), M, N, K, x.stride(0), w_up.stride(0), h.stride(0), _lib.dtype_code(x.dtype),
+                 _lib.stream_ptr()), "dlti_gemm_relu2_2cta")
+    return h[:, :ff]
+
+
 def gemm_rope(x: torch.Tensor, w: torch.Tensor, pos: torch.Tensor, cos_t: torch.Tensor, sin_t: torch.Tensor,
               n_rot_heads: int, hd: int, a2: torch.Tensor | None = None, b2: torch.Tensor | None = None,
               gather=None) -> torch.Tensor:

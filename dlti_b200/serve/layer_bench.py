@@ -20,7 +20,7 @@ from ..ops import attention as A
 from ..ops import elementwise as E
 from ..ops import serving as S
 from ..ops import stack as K
-from ..ops.gemm import gemm, gemm_skinny, gemm_skinny_acc
+from ..ops.gemm import gemm, gemm_relu2, gemm_skinny, gemm_skinny_acc
 from .engine import LLMEngine, _pieces, chunk_pieces
 from .model_runner import TPContext
 from .tokenizer import ByteTokenizer
@@ -231,6 +231,9 @@ def kernels(width: int, peaks: dict, nseq: int, length: int, batch: int, ctx: in
         # activation
         ff, lf = cfg.layers[0].mlp.ff, ll.intermediate_size
         u = torch.zeros(n, ff, device=dev) if acc else rnd(n, ff)
+        if not acc:
+            a, b = rnd(n, d), rnd(ff, d)
+            k.run("sigosun", phase, "GEMM up + relu^2", lambda: gemm_relu2(a, b, ff), 2 * (n * d + ff * d + n * ff), 2.0 * n * ff * d)
         k.run("sigosun", phase, "relu^2", lambda: K.relu2(u, ff, bf, acc=acc), n * ff * ((8 if acc else 2) + 2))
         gu = torch.zeros(n, 2 * lf, device=dev) if acc else rnd(n, 2 * lf)
         if acc:

@@ -13,7 +13,7 @@ import torch
 from ..models.stack import AttentionMixer, LightningMixer, Mamba2Mixer, StackConfig, StackWeights, mixer_sections, round8
 from ..ops import _lib
 from ..ops import stack as K
-from ..ops.gemm import gemm_skinny_acc
+from ..ops.gemm import gemm_relu2, gemm_skinny_acc
 from .kv_cache import KVCache, KVSpec, StateCache, StateSpec
 
 
@@ -72,7 +72,9 @@ class StackRunner:
                 y = self._lightning(i, m, lw, xa, rows)
             xa = self._close(mm(y, lw["w_out"]), x, lw["norm1"])
             if l.mlp is not None:
-                h = K.relu2(mm(xa, lw["w_up"]), l.mlp.ff, self.dtype, acc=acc)
+                h = gemm_relu2(xa, lw["w_up"], l.mlp.ff) if x.is_cuda and not acc else None      # activation in the GEMM
+                if h is None:
+                    h = K.relu2(mm(xa, lw["w_up"]), l.mlp.ff, self.dtype, acc=acc)
                 xa = self._close(mm(h, lw["w_down"]), x, lw["norm2"])
             if self.trace is not None:
                 self.trace.append(x.clone())

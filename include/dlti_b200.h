@@ -366,6 +366,9 @@ int dlti_post_norm_add(const void* y, long long y_ld, float* x, const float* w, 
 /* out[i] = RMSnorm(x[idx[i]]) * w; idx NULL = all rows */
 int dlti_rms_rows(const float* x, const long long* idx, const float* w, void* out, long long out_ld, long long rows,
     int d, float eps, int one_plus, int dtype, dlti_stream_t stream);
+/* h = relu(x W^T)^2 in the epilogue of the CTA-pair GEMM (16-bit) */
+int dlti_gemm_relu2_2cta(const void* X, const void* W, void* Hout, int M, int N, int K, long long ldx, long long ldw,
+    long long ldh, int dtype, dlti_stream_t stream);
 /* h = relu(u)^2 over the first ff columns */
 int dlti_relu2(const void* u, long long u_ld, void* h, long long h_ld, long long rows, int ff, int acc, int dtype,
     dlti_stream_t stream);

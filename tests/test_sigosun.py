@@ -67,6 +67,20 @@ def test_squared_relu(device, dtype, ff):
     assert rel(K.relu2(acts(u, device, dtype), ff, dtype), torch.relu(u.double()).square()) < tol(dtype, 1e-6, 4e-3)
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("M,ff,K", [(2048, 2048, 264), (2100, 2051, 136), (16384, 200, 64)])
+def test_squared_relu_in_the_gemm_epilogue(M, ff, K):
+    from dlti_b200.ops.gemm import gemm, gemm_relu2
+    g = gen(M)
+    x, w = rnd(g, M, K).cuda(), torch.zeros(round8(ff), K, dtype=BF16)
+    w[:ff] = rnd(g, ff, K) * 0.1
+    h = gemm_relu2(x, w.cuda(), ff)
+    want = torch.relu(gemm(x, w.cuda()).float()[:, :ff]).square().to(BF16)
+    assert h.shape == (M, ff) and float((h.float() - want.float()).abs().max()) <= 0.02 * float(want.float().abs().max())
+    assert rel(h, torch.relu(x.double().cpu() @ w.double().t()[:, :ff]).square()) < 6e-3
+    assert gemm_relu2(x[:300], w.cuda(), ff) is None
+
+
 @pytest.mark.parametrize("device,dtype", MODES)
 @pytest.mark.parametrize("n,groups", [(48, 1), (48, 3), (60, 5), (96, 4), (2048, 1), (1040, 2)])
 def test_gated_norms(device, dtype, n, groups):
