@@ -953,8 +953,8 @@ DLTI_API int dlti_qk_norm_rope_cache(const void* proj, long long ld, int oq, int
     using B = __nv_bfloat16;
 #define QKV_CASE(LPH)                                                                                                            \
   if (dim == 8 * LPH) {                                                                                                          \
-    const int per = 4 * (32 / LPH) * (acc ? 1 : 4);                                                                              \
-    auto kern = acc ? qk_norm_rope_cache_vec_kernel<B, true, LPH, 1> : qk_norm_rope_cache_vec_kernel<B, false, LPH, 4>;            \
+    const int per = 4 * (32 / LPH) * (acc ? 1 : 2);                                                                              \
+    auto kern = acc ? qk_norm_rope_cache_vec_kernel<B, true, LPH, 1> : qk_norm_rope_cache_vec_kernel<B, false, LPH, 2>;            \
     DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, kern, dim3((unsigned)tokens, (jobs + per - 1) / per), dim3(128), 0, st, p, jobs, kvjobs)); \
   }
     QKV_CASE(8) QKV_CASE(16) QKV_CASE(32)
