@@ -59,6 +59,7 @@ struct AttnParams {
   // query row goes to row seq_out0[b] of O (and of the gates). Null: every row is a query, in place.
   const int *seq_q0, *seq_out0;
   const float* gate;     // optional [output rows, H] factors on the head outputs
+  const float* sink;     // optional [H]: one more term exp(sink) in the softmax denominator, without a value
   int vdim;              // value columns of a head that are written, head h at column h * vdim of O (0: 128)
 };
 
@@ -979,6 +980,7 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
       const bool write = qi < seqlen && qi >= q0;
       const long long orow_i = (SPLIT && p.seq_out0) ? p.seq_out0[b] + qi - q0 : row0 + qi;
       const int vdim = (SPLIT && p.vdim) ? p.vdim : HD;
+      if (SPLIT && p.sink) l += ex2_approx(p.sink[h] * LOG2E - m_ref);
       float inv = 1.f / l;
       if (SPLIT && p.gate && write) inv *= p.gate[orow_i * p.H + h];
       T* orow = reinterpret_cast<T*>(p.O) + orow_i * p.ldo + h * vdim;
@@ -1077,14 +1079,14 @@ DLTI_API int dlti_attn_fwd(const void* qkv, void* out, float* lse, const int* cu
 // Inference form with split softmax weights (see attn_fwd2_kernel), bf16: heads padded to 128 columns in qkv, vdim (a
 // multiple of 8) of them written; optional gate [output rows, H]; output row pitch ldo (a multiple of 8); optional
 // seq_q0 / seq_out0 (see AttnParams) for portions whose earlier keys and values lie in front of their rows.
-DLTI_API int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const int* cu_seqlens, const int* seq_q0,
+DLTI_API int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const float* sink, const int* cu_seqlens, const int* seq_q0,
                                  const int* seq_out0, int batch, int max_seqlen, long long T_total, int H, int KV, int vdim, float scale,
                                  cudaStream_t st) {
   if (H % KV || ldo % 8 || vdim % 8 || vdim < 8 || vdim > HD || (seq_q0 == nullptr) != (seq_out0 == nullptr) || (reinterpret_cast<uintptr_t>(out) & 15)) return DLTI_ERR_BAD_ARG;
   if (batch <= 0 || T_total <= 0) return 0;
   AttnParams p{};
   p.cu_seqlens = cu_seqlens; p.H = H; p.KV = KV; p.W = (H + 2 * KV) * HD;
-  p.O = out; p.ldo = ldo; p.T_total = T_total; p.scale = scale; p.dtype = DLTI_BF16; p.gate = gate;
+  p.O = out; p.ldo = ldo; p.T_total = T_total; p.scale = scale; p.dtype = DLTI_BF16; p.gate = gate; p.sink = sink;
   p.seq_q0 = seq_q0; p.seq_out0 = seq_out0; p.vdim = vdim;
   CUtensorMap tm;
   const int rc = make_map(&tm, qkv, T_total, p.W, 128);

@@ -24,12 +24,19 @@ struct PagedParams {
   const float* gate;                               // [rows, H] factors or null
   void* out; long long o_ld;                       // head h at column h * vdim
   long long rows;
+  const float* sink;                               // [H] or null: one more term exp(sink) in the softmax denominator, without a value
 };
 
+// softmax denominator of head h with its sink: l is a sum of 2^(score - m), m in log2 (natural: of e^(score - m))
+__device__ __forceinline__ float with_sink(const PagedParams& p, int h, float m, float l, bool natural = false) {
+  if (!p.sink) return l;
+  const float r = m == -INFINITY ? 0.f : m;
+  return l + (natural ? expf(p.sink[h] - r) : ex2(p.sink[h] * 1.4426950408889634f - r));
+}
 __device__ __forceinline__ int first_key(int pos, int chunk) { return chunk > 0 ? pos / chunk * chunk : 0; }
 
-constexpr int ROWS_MAXV = 16;                      // value dims per lane: heads of up to 512
-template <typename T>
+// ROWS_MAXV: value dims per lane
+template <typename T, int ROWS_MAXV>
 __global__ void __launch_bounds__(128) attn_rows_kernel(const PagedParams p) {
   extern __shared__ float sq_all[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -81,6 +88,7 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const PagedParams p) {
       }
     }
   }
+  l = with_sink(p, h, m, l, true);
   float f = l > 0.f ? 1.f / l : 0.f;
   if (p.gate) f *= p.gate[t * p.H + h];
   T* orow = reinterpret_cast<T*>(p.out) + t * p.o_ld + (long long)h * p.vdim;
@@ -94,7 +102,7 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const PagedParams p) {
 template <typename T>
 int launch_rows(const PagedParams& p, cudaStream_t st) {
   const size_t smem = (size_t)4 * p.dim * 4;
-  attn_rows_kernel<T><<<(unsigned)((p.rows * p.H + 3) / 4), 128, smem, st>>>(p);
+  (p.vdim <= 256 ? attn_rows_kernel<T, 8> : attn_rows_kernel<T, 32>)<<<(unsigned)((p.rows * p.H + 3) / 4), 128, smem, st>>>(p);
   dlti_count_launch();
   return (int)cudaGetLastError();
 }
@@ -322,6 +330,7 @@ __global__ void __launch_bounds__(256) attn_prefill_kernel(const PagedParams p) 
     l[y] += __shfl_xor_sync(0xffffffffu, l[y], 1);
     l[y] += __shfl_xor_sync(0xffffffffu, l[y], 2);
     if (pos[y] < 0) continue;
+    l[y] = with_sink(p, head[y], m[y], l[y]);
     float f = l[y] > 0.f ? 1.f / l[y] : 0.f;
     if (p.gate) f *= p.gate[row[y] * p.H + head[y]];
     bf16* orow = reinterpret_cast<bf16*>(p.out) + row[y] * p.o_ld + (long long)head[y] * p.vdim;
@@ -454,6 +463,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const PagedParams p, i
     }
     const int h = g * rep + h0 + r;
     if (splits == 1) {
+      gl = with_sink(p, h, gm, gl);
       float f = gl > 0.f ? 1.f / gl : 0.f;
       if (p.gate) f *= p.gate[(long long)b * p.H + h];
       reinterpret_cast<bf16*>(p.out)[(long long)b * p.o_ld + (long long)h * p.vdim + c] = __float2bfloat16(a * f);
@@ -480,6 +490,7 @@ __global__ void __launch_bounds__(128) attn_combine_kernel(const PagedParams p, 
     const float ms = part_ml[(base + s) * 2];
     gl += ms == -INFINITY ? 0.f : part_ml[(base + s) * 2 + 1] * ex2(ms - gm);
   }
+  gl = with_sink(p, h, gm, gl);
   float f = gl > 0.f ? 1.f / gl : 0.f;
   if (p.gate) f *= p.gate[(long long)b * p.H + h];
   for (int c = threadIdx.x; c < p.vdim; c += 128) {
@@ -554,13 +565,13 @@ int launch_decode(const PagedParams& p, int splits, float* ws, cudaStream_t st) 
 // rows of decode sequences (row s = sequence s < nd) and of prompts (sequence nd + i: rows nd + cu[i] ... nd + cu[i+1]).
 DLTI_API int dlti_attn_rows(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd, const int* tables,
                             int max_blocks, int bs, const int* ctx, const int* rseq, const int* pos, int H, int G, int dim, int vdim,
-                            int chunk, float scale, const float* gate, void* out, long long o_ld, long long rows, int dtype,
+                            int chunk, float scale, const float* gate, const float* sink, void* out, long long o_ld, long long rows, int dtype,
                             cudaStream_t st) {
   if (rows <= 0) return 0;
   if (H % G || dim < 1 || vdim < 1) return DLTI_ERR_BAD_ARG;
-  if (dim > 512 || vdim > 512) { dlti_set_error("attn_rows: heads of up to 512 dimensions"); return DLTI_ERR_TOO_LARGE; }
+  if (dim > 2048 || vdim > 1024) { dlti_set_error("attn_rows: queries of up to 2048 and values of up to 1024 dimensions"); return DLTI_ERR_TOO_LARGE; }
   PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, nullptr, rseq, pos, 0, H, G, dim, vdim, chunk, scale,
-                gate, out, o_ld, rows};
+                gate, out, o_ld, rows, sink};
   if (dtype == DLTI_BF16) return launch_rows<__nv_bfloat16>(p, st);
   if (dtype == DLTI_FP32) return launch_rows<float>(p, st);
   return DLTI_ERR_UNSUPPORTED;
@@ -576,25 +587,25 @@ static int check_mma(int H, int G, int dim, int vdim, int kd, int vd, int q_hd) 
 // the rows themselves must be in the pages already.
 DLTI_API int dlti_attn_paged_prefill(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
                                      const int* tables, int max_blocks, int bs, const int* ctx, const int* cu, int nd, int nseq,
-                                     int max_rows, int H, int G, int dim, int vdim, int chunk, float scale, const float* gate, void* out,
+                                     int max_rows, int H, int G, int dim, int vdim, int chunk, float scale, const float* gate, const float* sink, void* out,
                                      long long o_ld, cudaStream_t st) {
   if (nseq <= 0 || max_rows <= 0) return 0;
   if (int rc = check_mma(H, G, dim, vdim, kd, vd, q_hd)) return rc;
   if (q_ld % 2 || nseq > 65535) return DLTI_ERR_BAD_ARG;
   PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, cu, nullptr, nullptr, nd, H, G, dim, vdim, chunk, scale,
-                gate, out, o_ld, 0};
+                gate, out, o_ld, 0, sink};
   HEAD_DISPATCH(kd, vd, launch_prefill, p, nseq, max_rows, st);
 }
 
 // bf16. Row b = the newest token of sequence b, whose context is ctx[b] tokens. ws: batch * H * splits * (vdim + 2) floats.
 DLTI_API int dlti_attn_paged_decode(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
                                     const int* tables, int max_blocks, int bs, const int* ctx, int batch, int H, int G, int dim, int vdim,
-                                    int chunk, float scale, const float* gate, int splits, float* ws, void* out, long long o_ld,
+                                    int chunk, float scale, const float* gate, const float* sink, int splits, float* ws, void* out, long long o_ld,
                                     cudaStream_t st) {
   if (batch <= 0) return 0;
   if (int rc = check_mma(H, G, dim, vdim, kd, vd, q_hd)) return rc;
   if (q_ld % 2 || splits < 1 || batch > 65535) return DLTI_ERR_BAD_ARG;
   PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, nullptr, nullptr, nullptr, 0, H, G, dim, vdim, chunk, scale,
-                gate, out, o_ld, batch};
+                gate, out, o_ld, batch, sink};
   HEAD_DISPATCH(kd, vd, launch_decode, p, splits, ws, st);
 }

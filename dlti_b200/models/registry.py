@@ -13,7 +13,7 @@ from typing import Callable
 import torch
 
 from . import config as llama_config
-from . import sigosun
+from . import logozen, sigosun
 
 
 @dataclass(frozen=True)
@@ -56,6 +56,10 @@ FAMILIES: dict[str, Family] = {
     sigosun.ARCHITECTURE: Family(
         sigosun.ARCHITECTURE, sigosun.SigosunConfig, sigosun.PRESETS, sigosun.SigosunConfig.load, sigosun.load_weights,
         lambda cfg, device, dtype, seed=0: sigosun.from_state(cfg, sigosun.random_state(cfg, seed, device), device, dtype),
+        _stack_runner, (torch.bfloat16, torch.float32)),
+    logozen.ARCHITECTURE: Family(
+        logozen.ARCHITECTURE, logozen.LogozenConfig, logozen.PRESETS, logozen.LogozenConfig.load, logozen.load_weights,
+        lambda cfg, device, dtype, seed=0: logozen.from_state(cfg, logozen.random_state(cfg, seed, device), device, dtype),
         _stack_runner, (torch.bfloat16, torch.float32)),
 }
 

@@ -109,23 +109,10 @@ def named_tensors(w: StackWeights):
             yield p + "mlp.down", lw["w_down"][:d]
 
 
-def _copy(name: str, dst, src: torch.Tensor) -> None:
-    parts = dst if isinstance(dst, list) else [dst]
-    if sum(p.shape[0] for p in parts) != src.shape[0] or src.shape[1:] != parts[0].shape[1:]:
-        raise ValueError(f"tensor {name} has shape {tuple(src.shape)}, which does not fit the configuration")
-    o = 0
-    for p in parts:
-        p.copy_(src[o:o + p.shape[0]])
-        o += p.shape[0]
-
-
 def load_weights(cfg: SigosunConfig, directory: str | Path, device, dtype: torch.dtype) -> StackWeights:
     from .hf_io import CheckpointReader
-    rd = CheckpointReader(directory)
     w = StackWeights(cfg, device, dtype)
-    for name, dst in named_tensors(w):
-        _copy(name, dst, rd.get(name))
-    return w
+    return w.fill(named_tensors(w), CheckpointReader(directory).get)
 
 
 def random_state(cfg: SigosunConfig, seed: int = 0, device="cpu") -> dict[str, torch.Tensor]:
@@ -156,9 +143,7 @@ def random_state(cfg: SigosunConfig, seed: int = 0, device="cpu") -> dict[str, t
 
 def from_state(cfg: SigosunConfig, state: dict[str, torch.Tensor], device, dtype: torch.dtype) -> StackWeights:
     w = StackWeights(cfg, device, dtype)
-    for name, dst in named_tensors(w):
-        _copy(name, dst, state[name])
-    return w
+    return w.fill(named_tensors(w), state.__getitem__)
 
 
 def save_checkpoint(cfg: SigosunConfig, state: dict[str, torch.Tensor], directory: str | Path) -> None:

@@ -1,7 +1,8 @@
-"""Models described layer by layer: each layer names its token mixer (softmax attention, Mamba-2, lightning attention)
-and its feed-forward, with every size and constant a parameter. A design (models/sigosun.py) is a parser from its
-config.json to a `StackConfig` plus its tensor names; the weights container, the cache layout and the serving forward
-pass (serve/stack_runner.py) are shared by all of them.
+"""Models described layer by layer: each layer names its token mixer (softmax attention, latent attention, Mamba-2,
+lightning attention, mLSTM) and its feed-forward, with every size and constant a parameter; the model names how sublayers
+meet the residual. A design (models/sigosun.py, models/logozen.py) is a parser from its config.json to a `StackConfig` plus
+its tensor names; the weights container, the cache layout and the serving forward pass (serve/stack_runner.py) are shared
+by all of them.
 
 Weights are kept as merged input projections, one GEMM per mixer. Every section of a merged projection and the row
 pitch of every matrix is rounded up to 8 elements, so any head count or width meets the 16-byte rules of the TMA
@@ -16,6 +17,10 @@ import torch
 
 def round8(n: int) -> int:
     return (n + 7) // 8 * 8
+
+
+def round16(n: int) -> int:
+    return (n + 15) // 16 * 16
 
 
 # ---- layer descriptions ------------------------------------------------------------------------------------
@@ -67,14 +72,58 @@ class LightningMixer:
 
 
 @dataclass(frozen=True)
+class LatentAttentionMixer:
+    """Keys and values of all heads are linear in one cached latent per token; a rotated key part is shared by the heads."""
+    heads: int
+    dim: int                       # unrotated query / key size of a head
+    rot_dim: int                   # size of the part that carries the rotation
+    vdim: int
+    kv_rank: int                   # size of the latent
+    scale: float
+    rope: Rope | None = None       # on the rot_dim part
+    sink: bool = True              # a learned term per head in the softmax denominator
+    head_gate: bool = True
+
+    chunk = 0                      # every earlier position is seen
+
+    @property
+    def qk_dim(self) -> int:
+        return self.dim + self.rot_dim
+
+    @property
+    def rot_at(self) -> int:       # a cache row is [latent, zeros, rotated part, zeros], both parts padded to 16
+        return round16(self.kv_rank)
+
+    @property
+    def pitch(self) -> int:
+        return self.rot_at + round16(self.rot_dim)
+
+    @property
+    def head_pitch(self) -> int:
+        """Columns of a head when its keys and values are laid out one by one: 128 for the packed layout of the tcgen05
+        kernel, else rounded to 16 bytes."""
+        n = max(self.qk_dim, self.vdim)
+        return 128 if n <= 128 and self.vdim % 8 == 0 else round8(n)
+
+
+@dataclass(frozen=True)
+class MLstmMixer:
+    """Matrix memory with exponential gates, a running maximum and a normaliser."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+
+@dataclass(frozen=True)
 class DenseMlp:
     ff: int
-    act: str = "relu2"             # square of relu
+    act: str = "relu2"             # square of relu; "polynorm": sum of the normed first three powers
 
 
 @dataclass(frozen=True)
 class Layer:
-    mixer: AttentionMixer | Mamba2Mixer | LightningMixer
+    mixer: AttentionMixer | LatentAttentionMixer | Mamba2Mixer | LightningMixer | MLstmMixer
     mlp: DenseMlp | None = None
 
 
@@ -85,6 +134,11 @@ class StackConfig:
     norm_eps: float
     layers: list[Layer]
     norm_one_plus: bool = True     # layer and final norm weights are stored around zero: 1 + w
+    # 0: one residual, RMS norms on the sublayer outputs. n > 0: n residual streams with learned mixing around every
+    # sublayer (hyper-connections), a layer norm and a causal convolution of `canon` taps on its input
+    streams: int = 0
+    canon: int = 0
+    embed_scale: float = 1.0
     max_position_embeddings: int = 8192        # only a default for the server's max_model_len
     bos_token_id: int = 1
     eos_token_id: int = 2
@@ -107,8 +161,16 @@ class StackConfig:
             elif isinstance(m, Mamba2Mixer):
                 if m.heads % m.groups or m.inner % m.norm_groups:
                     raise ValueError(f"layer {i}: groups must divide the heads and norm_groups the inner size")
+            elif isinstance(m, LatentAttentionMixer):
+                if m.rope is not None and (m.rope.dims % 2 or m.rope.dims > m.rot_dim):
+                    raise ValueError(f"layer {i}: rotary dims {m.rope.dims} must be even and at most {m.rot_dim}")
+            elif isinstance(m, MLstmMixer):
+                if not m.gate_cap > 0:
+                    raise ValueError(f"layer {i}: gate_cap {m.gate_cap} must be positive")
             elif len(m.decay) != m.heads:
                 raise ValueError(f"layer {i}: {len(m.decay)} decays for {m.heads} heads")
+        if self.streams and self.canon < 1:
+            raise ValueError(f"canon taps {self.canon}: at least 1")
 
     @property
     def num_hidden_layers(self) -> int:
@@ -116,17 +178,23 @@ class StackConfig:
 
     @property
     def has_state(self) -> bool:
-        """Some layer carries recurrent state from token to token."""
-        return any(not isinstance(l.mixer, AttentionMixer) for l in self.layers)
+        """Some layer carries recurrent state (or earlier inputs of a convolution) from token to token."""
+        return self.canon > 1 or any(not isinstance(l.mixer, (AttentionMixer, LatentAttentionMixer)) for l in self.layers)
 
     @property
     def chunks(self) -> list[int]:
         """The distinct attention chunk sizes, in order of first use (0 = unlimited)."""
         out: list[int] = []
         for l in self.layers:
-            if isinstance(l.mixer, AttentionMixer) and l.mixer.chunk not in out:
+            if isinstance(l.mixer, (AttentionMixer, LatentAttentionMixer)) and l.mixer.chunk not in out:
                 out.append(l.mixer.chunk)
         return out
+
+    @property
+    def pack_prefix(self) -> int:
+        """Most cached rows per prompt row that are worth laying out in front of a portion. Latent attention makes their keys
+        and values anew by a GEMM, which beats reading the latents once per prompt row at any ratio short of this."""
+        return 64 if any(isinstance(l.mixer, LatentAttentionMixer) for l in self.layers) else 4
 
     def num_params(self) -> int:
         return sum(t.numel() for t in StackWeights(self, "meta", torch.bfloat16).tensors())
@@ -161,6 +229,10 @@ def mixer_sections(m) -> Sections:
         return Sections(**s)
     if isinstance(m, Mamba2Mixer):
         return Sections(z=m.inner, xbc=m.conv_channels, dt=m.heads)
+    if isinstance(m, LatentAttentionMixer):
+        return Sections(q=m.heads * m.qk_dim, dkv=m.kv_rank + m.rot_dim, **({"g": m.heads} if m.head_gate else {}))
+    if isinstance(m, MLstmMixer):                          # the log gates come last: their products stay fp32
+        return Sections(q=m.heads * m.dim, k=m.heads * m.dim, v=m.heads * m.vdim, g=m.heads * m.vdim, gates=2 * m.heads)
     return Sections(q=m.heads * m.dim, k=m.heads * m.dim, v=m.heads * m.vdim, g=m.heads * m.vdim)
 
 
@@ -202,12 +274,26 @@ class StackWeights:
                 w |= {"conv": torch.zeros(m.conv, round8(m.conv_channels), dtype=torch.float32, device=device),
                       "conv_b": vec(round8(m.conv_channels)), "dt_bias": vec(m.heads), "A_log": vec(m.heads),
                       "D": vec(m.heads), "norm": vec(m.inner)}
+            elif isinstance(m, LatentAttentionMixer):
+                w |= {"kv_norm": vec(m.kv_rank), "w_uk": mat(m.heads * m.dim, m.kv_rank), "w_uv": mat(m.heads * m.vdim, m.kv_rank)}
+                if m.sink:
+                    w["sink"] = vec(m.heads)
+            elif isinstance(m, MLstmMixer):
+                w |= {"gate_b": vec(2 * m.heads), "norm": vec(mixer_out(m))}
             else:
                 w |= {"decay": torch.tensor(m.decay, dtype=torch.float32).to(device),
                       "norm": vec(mixer_out(m))}
             if l.mlp is not None:
                 w |= {"w_up": mat(l.mlp.ff, d), "w_down": mat(d, l.mlp.ff), "norm2": vec(d)}
+                if l.mlp.act == "polynorm":
+                    w["act"] = vec(4)
+            if cfg.streams:
+                for q in (1, 2) if l.mlp is not None else (1,):
+                    w |= {f"hc{q}.in": vec(cfg.streams), f"hc{q}.out": vec(cfg.streams),
+                          f"hc{q}.mix": torch.zeros(cfg.streams, cfg.streams, dtype=torch.float32, device=device),
+                          f"canon{q}": torch.zeros(cfg.canon, round8(d), dtype=torch.float32, device=device)}      # tap-major
             self.layers.append(w)
+        self.derived: list[dict] = [{} for _ in cfg.layers]      # rearranged copies of weights, made by finish()
 
     def tensors(self):
         yield from (self.embed, self.lm_head, self.final_norm)
@@ -218,3 +304,30 @@ class StackWeights:
         """Rows of layer i's merged input projection that belong to `name`."""
         o, n = mixer_sections(self.cfg.layers[i].mixer).at[name]
         return self.layers[i]["w_in"][o:o + n]
+
+    def fill(self, named, get) -> "StackWeights":
+        """Copy the checkpoint tensor get(name) to every (name, destination) of `named`; a list of destinations takes its
+        rows one after the other."""
+        for name, dst in named:
+            src, parts = get(name), dst if isinstance(dst, list) else [dst]
+            if sum(p.shape[0] for p in parts) != src.shape[0] or src.shape[1:] != parts[0].shape[1:]:
+                raise ValueError(f"tensor {name} has shape {tuple(src.shape)}, which does not fit the configuration")
+            o = 0
+            for p in parts:
+                p.copy_(src[o:o + p.shape[0]])
+                o += p.shape[0]
+        return self.finish()
+
+    def finish(self) -> "StackWeights":
+        """Weights that the kernels want in another arrangement."""
+        for i, (l, w) in enumerate(zip(self.cfg.layers, self.layers)):
+            m = l.mixer
+            if isinstance(m, LatentAttentionMixer) and self.device.type == "cuda" and self.dtype != torch.float32:
+                # cache row -> [keys | values] of all heads; an identity block hands the rotated part to every head's key
+                H, hp = m.heads, m.head_pitch
+                e = torch.zeros(2, H, hp, m.pitch, dtype=self.dtype, device=self.device)
+                e[0, :, :m.dim, :m.kv_rank] = w["w_uk"][:H * m.dim].view(H, m.dim, m.kv_rank)
+                e[0, :, m.dim:m.qk_dim, m.rot_at:m.rot_at + m.rot_dim] = torch.eye(m.rot_dim, dtype=self.dtype, device=self.device)
+                e[1, :, :m.vdim, :m.kv_rank] = w["w_uv"][:H * m.vdim].view(H, m.vdim, m.kv_rank)
+                self.derived[i]["w_expand"] = e.view(2 * H * hp, m.pitch)
+        return self

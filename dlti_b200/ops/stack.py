@@ -1,5 +1,5 @@
-"""Ops of the layer-stack models (models/stack.py): kernels in csrc/stack.cu, recurrent.cu, attention_paged.cu and
-gemm_f32.cu; PyTorch restatements for CPU tensors, as in the other op modules.
+"""Ops of the layer-stack models (models/stack.py; more of them in streams.py and latent.py): kernels in csrc/stack.cu,
+recurrent.cu, attention_paged.cu and gemm_f32.cu; PyTorch restatements for CPU tensors, as in the other op modules.
 
 Activations are [rows, n] views whose row pitch is a multiple of 8 elements (`act`). The residual stream is fp32.
 Ops with `acc=True` consume the fp32 accumulator of gemm_skinny_acc and leave it zero."""
@@ -270,13 +270,13 @@ def paged_attention_ref(q, m, rows: Rows, kc, vc, gate):
     return out.reshape(T, -1).to(q.dtype)
 
 
-def attn_rows(q, m, rows: Rows, kc, vc, gate, out):
+def attn_rows(q, m, rows: Rows, kc, vc, gate, out, sink=None):
     """fp32-arithmetic attention of the rows of q, one warp per (row, head)."""
     hd = q.shape[1] // m.heads
-    f = _lib.fn("dlti_attn_rows", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _V, _I, _I, _I, _I, _I, _F, _V, _V, _L, _L, _I, _V])
+    f = _lib.fn("dlti_attn_rows", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _V, _I, _I, _I, _I, _I, _F, _V, _V, _V, _L, _L, _I, _V])
     _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], kc.shape[1],
-                 _p(rows.ctx), _p(rows.seq), _p(rows.pos), m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.scale, _p(gate), _p(out),
-                 out.stride(0), q.shape[0], _lib.dtype_code(q.dtype), _lib.stream_ptr()), "attn_rows")
+                 _p(rows.ctx), _p(rows.seq), _p(rows.pos), m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.scale, _p(gate), _p(sink),
+                 _p(out), out.stride(0), q.shape[0], _lib.dtype_code(q.dtype), _lib.stream_ptr()), "attn_rows")
     return out
 
 
@@ -293,7 +293,7 @@ def _workspace(device, floats: int) -> torch.Tensor:
     return ws
 
 
-def attn_paged_decode(q, m, rows: Rows, kc, vc, gate, out, splits: int | None = None):
+def attn_paged_decode(q, m, rows: Rows, kc, vc, gate, out, splits: int | None = None, sink=None):
     """Decode rows (bf16): row b of q against the visible keys of sequence b, split over CTAs."""
     B, hd, bs = q.shape[0], q.shape[1] // m.heads, kc.shape[1]
     if splits is None:
@@ -301,21 +301,21 @@ def attn_paged_decode(q, m, rows: Rows, kc, vc, gate, out, splits: int | None = 
         ctas = max(1, B) * m.kv_heads * -(-(m.heads // m.kv_heads) // 16)
         splits = max(1, min(32, 3 * 148 // ctas, -(-reach // 64)))     # one wave of three CTAs per SM
     ws = _workspace(q.device, B * m.heads * splits * (m.vdim + 2)) if splits > 1 else None
-    f = _lib.fn("dlti_attn_paged_decode", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _I, _I, _I, _I, _I, _I, _F, _V, _I, _V, _V, _L, _V])
+    f = _lib.fn("dlti_attn_paged_decode", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _I, _I, _I, _I, _I, _I, _F, _V, _V, _I, _V, _V, _L, _V])
     _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], bs,
-                 _p(rows.ctx), B, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.scale, _p(gate), splits, _p(ws), _p(out),
+                 _p(rows.ctx), B, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.scale, _p(gate), _p(sink), splits, _p(ws), _p(out),
                  out.stride(0), _lib.stream_ptr()), "attn_paged_decode")
     return out
 
 
-def attn_paged_prefill(q, m, rows: Rows, kc, vc, gate, out):
+def attn_paged_prefill(q, m, rows: Rows, kc, vc, gate, out, sink=None):
     """Prompt rows (bf16): q, gate and out cover all rows of the step."""
     hd = q.shape[1] // m.heads
     f = _lib.fn("dlti_attn_paged_prefill", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _F, _V, _V,
-                                            _L, _V])
+                                            _V, _L, _V])
     _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], kc.shape[1],
                  _p(rows.ctx), _p(rows.cu), rows.nd, rows.nseq - rows.nd, rows.max_seqlen, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk,
-                 m.scale, _p(gate), _p(out), out.stride(0), _lib.stream_ptr()), "attn_paged_prefill")
+                 m.scale, _p(gate), _p(sink), _p(out), out.stride(0), _lib.stream_ptr()), "attn_paged_prefill")
     return out
 
 
@@ -326,11 +326,15 @@ def packed_attention(qkv, m, rows: Rows, pieces: Pieces, kc, vc, gate):
     out = act(T, H * m.vdim, qkv.dtype, qkv.device)
     if nd:
         attn_paged_decode(qkv[:nd, :H * PACKED_HD], m, rows, kc, vc, gate, out)
-    q, o, g = qkv[nd:], out[nd:], None if gate is None else gate[nd:]
-    f = _lib.fn("dlti_attn_fwd_split", [_V, _V, _L, _V, _V, _V, _V, _I, _I, _L, _I, _I, _I, _F, _V])
-    _lib.check(f(_p(q), _p(o), o.stride(0), _p(g), _p(pieces.cu), _p(pieces.q0), _p(pieces.out0), pieces.cu.numel() - 1, pieces.longest,
-                 q.shape[0], H, m.kv_heads, m.vdim, m.scale, _lib.stream_ptr()), "attn_fwd_split")
+    attn_fwd_split(qkv[nd:], m, H, m.kv_heads, pieces, None if gate is None else gate[nd:], out[nd:])
     return out
+
+
+def attn_fwd_split(qkv, m, heads, kv_heads, pieces: Pieces, gate, out, sink=None):
+    """Causal attention of packed rows [q heads | k heads | v heads], each 128 columns, within every piece."""
+    f = _lib.fn("dlti_attn_fwd_split", [_V, _V, _L, _V, _V, _V, _V, _V, _I, _I, _L, _I, _I, _I, _F, _V])
+    _lib.check(f(_p(qkv), _p(out), out.stride(0), _p(gate), _p(sink), _p(pieces.cu), _p(pieces.q0), _p(pieces.out0), pieces.cu.numel() - 1,
+                 pieces.longest, qkv.shape[0], heads, kv_heads, m.vdim, m.scale, _lib.stream_ptr()), "attn_fwd_split")
 
 
 def paged_attention(q, m, rows: Rows, kc, vc, gate):
@@ -483,3 +487,59 @@ def _scan_chunked(q, k, v, decay, state, rows, seq0, nseq, heads, groups, N, P, 
                  0 if dt is None else dt.stride(0), _p(decay.dt_bias), _p(decay.A_log), _p(decay.D), _p(state), _p(rows.state),
                  _p(rows.ctx), _p(rows.cu), rows.nd, seq0, nseq, heads, N, P, _p(out), out.stride(0), *_conv_args(conv),
                  _lib.stream_ptr()), "linear_scan_chunked")
+
+
+def mlstm_scan_ref(q, k, v, gates, gate_b, cap, state, vec, rows: Rows, heads, N, P):
+    T, dtype = q.shape[0], v.dtype
+    qf, kf, vf = q.float().reshape(T, heads, N) * N ** -0.5, k.float().reshape(T, heads, N), v.float().reshape(T, heads, P)
+    g = cap * torch.tanh((gates[:, :2 * heads] + gate_b) / cap)
+    li, lf = g[:, :heads], torch.nn.functional.logsigmoid(g[:, heads:])
+    out = torch.zeros(T, heads, P)
+    sl = -(-P // 32)
+    for s in range(rows.nseq):
+        r0, n, start = rows.bounds(s)
+        slot = int(rows.state[s])
+        have = start > 0 and slot >= 0
+        S = state[slot].clone() if have else torch.zeros(heads, N, P)
+        w = vec[slot].view(heads, sl, N + 1)[:, 0].clone() if have else torch.zeros(heads, N + 1)
+        nv, m = w[:, :N], w[:, N]
+        for t in range(r0, r0 + n):
+            mn = torch.maximum(lf[t] + m, li[t])
+            a, b = 1 + torch.expm1(lf[t] + m - mn), torch.exp(li[t] - mn)
+            m = mn
+            S = a[:, None, None] * S + (b[:, None] * kf[t])[:, :, None] * vf[t][:, None, :]
+            nv = a[:, None] * nv + b[:, None] * kf[t]
+            den = torch.maximum((nv * qf[t]).sum(1).abs(), torch.exp(-m)) + 1e-6
+            out[t] = (qf[t][:, :, None] * S).sum(1) / den[:, None]
+        if slot >= 0:
+            state[slot] = S
+            vec[slot] = torch.cat([nv, m[:, None]], 1).repeat(1, sl)
+    return out.reshape(T, -1).to(dtype)
+
+
+def mlstm_vec(N: int, P: int) -> int:
+    """fp32 numbers per head that an mLSTM keeps beside its matrix: n and m, once per slice of 32 value columns."""
+    return -(-P // 32) * (N + 1)
+
+
+def mlstm_scan(q, k, v, gates, gate_b, cap, state, vec, rows: Rows, heads, N, P):
+    """mLSTM over the rows of every sequence: q, k [T, heads * N], v [T, heads * P] views; gates [T, >= 2 heads] raw fp32 log gates
+    (input, then forget) with bias gate_b; state [slots, heads, N, P] and vec [slots, heads, mlstm_vec] updated in place."""
+    if not _lib.use_native(q):
+        return mlstm_scan_ref(q, k, v, gates, gate_b, cap, state, vec, rows, heads, N, P)
+    out = act(q.shape[0], heads * P, v.dtype, q.device)
+    f = _lib.fn("dlti_mlstm_scan", [_V, _L, _V, _L, _V, _L, _V, _L, _V, _F, _F, _V, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _V, _L, _I, _I, _V])
+
+    def run(seq0, nseq, chunked):
+        _lib.check(f(_p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(gates), gates.stride(0), _p(gate_b), float(cap), N ** -0.5,
+                     _p(state), _p(vec), _p(rows.state), _p(rows.ctx), _p(rows.cu), rows.nd, seq0, nseq, heads, N, P, _p(out), out.stride(0),
+                     int(chunked), _lib.dtype_code(v.dtype), _lib.stream_ptr()), "mlstm_scan")
+
+    nd, nseq = rows.nd, rows.nseq
+    if nseq > nd and q.dtype == torch.bfloat16 and N % 8 == 0 and P % 8 == 0 and N <= 256 and rows.max_seqlen >= _CHUNKED_FROM:
+        if nd:
+            run(0, nd, False)
+        run(nd, nseq - nd, True)
+    else:
+        run(0, nseq, False)
+    return out

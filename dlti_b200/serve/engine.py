@@ -83,13 +83,13 @@ class StepLayout:
 
 
 PACK_FROM = 64               # longest piece of a step's prompts from which they are laid out for the varlen prefill kernel
-PACK_PREFIX = 4              # ... and the most cached rows in front of them, per prompt row
 
 
-def chunk_pieces(cu, starts, tables, bs: int, chunk: int):
+def chunk_pieces(cu, starts, tables, bs: int, chunk: int, pack_prefix: int = 4):
     """The prompt rows of a step cut where their positions reach a multiple of `chunk` (0: not at all), for
     ops.stack.Pieces. Returns (int32 array [cu | q0 | out0 | dst | prow | pslot] (only cu without cached rows), pieces,
-    longest piece, extended rows, cached rows), or None when the pieces are too short or the cached part too long."""
+    longest piece, extended rows, cached rows), or None when the pieces are too short or there are more than pack_prefix
+    cached rows per prompt row."""
     cue, q0, out0, dst, prow, pslot, longest, own = [0], [], [], [], [], [], 0, 0
     for i, a in enumerate(starts):
         n = cu[i + 1] - cu[i]
@@ -109,7 +109,7 @@ def chunk_pieces(cu, starts, tables, bs: int, chunk: int):
             longest, own = max(longest, e - lo), max(own, e - p)
             p = lo = e
     prefix = sum(map(len, prow))
-    if own < PACK_FROM or prefix > PACK_PREFIX * cu[-1]:
+    if own < PACK_FROM or prefix > pack_prefix * cu[-1]:
         return None
     arrays = [cue] + ([q0, out0, *dst, *prow, *pslot] if prefix else [])
     return np.concatenate([np.asarray(x, dtype=np.int32) for x in arrays]), len(q0), longest, cue[-1], prefix
@@ -281,7 +281,7 @@ class LLMEngine:
         segs, seg_at, nsg = [], {}, 0
         if full and npf:
             for c in self.cfg.chunks:
-                pc = chunk_pieces(cu, starts, tables[nd:], self.blocks.block_size, c)
+                pc = chunk_pieces(cu, starts, tables[nd:], self.blocks.block_size, c, self.cfg.pack_prefix)
                 if pc is not None:
                     seg_at[c] = (nsg, *pc[1:])
                     segs.append(pc[0])

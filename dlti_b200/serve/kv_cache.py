@@ -132,13 +132,18 @@ class KVSpec:
 
 @dataclass(frozen=True)
 class StateSpec:
-    """One layer's recurrent state of a sequence: `heads` fp32 matrices [rows, cols] and, for layers with a short
-    convolution, its last `conv_rows` inputs of `conv_channels` channels."""
-    heads: int
-    rows: int
-    cols: int
+    """One layer's recurrent state of a sequence: `heads` fp32 matrices [rows, cols] with `vec` further fp32 numbers each;
+    for layers with a short convolution, its last `conv_rows` inputs of `conv_channels` channels; for sublayers whose input is
+    convolved, the last `canon_rows` inputs of `canon_channels` channels of each of `canon_parts` sublayers."""
+    heads: int = 0
+    rows: int = 0
+    cols: int = 0
     conv_rows: int = 0
     conv_channels: int = 0
+    vec: int = 0
+    canon_parts: int = 0
+    canon_rows: int = 0
+    canon_channels: int = 0
 
 
 class SlotManager:
@@ -158,20 +163,27 @@ class SlotManager:
 
 
 class StateCache:
-    """Recurrent states of all slots: per layer `ssm` [slots, heads, rows, cols] fp32 and `conv`
-    [slots, conv_rows, channels] in the compute dtype (None where a layer has none)."""
+    """Recurrent states of all slots, per layer (None where a layer has none): `ssm` [slots, heads, rows, cols] and `vec`
+    [slots, heads, vec] fp32; in the compute dtype `conv` [slots, conv_rows, channels] and `canon` [parts, slots, canon_rows,
+    channels]."""
 
     def __init__(self, specs: list, num_slots: int, dtype: torch.dtype, device):
         self.num_slots = num_slots
-        self.ssm = [None if s is None else torch.zeros((num_slots, s.heads, s.rows, s.cols), dtype=torch.float32, device=device)
-                    for s in specs]
-        self.conv = [None if s is None or not s.conv_channels else
-                     torch.zeros((num_slots, s.conv_rows, s.conv_channels), dtype=dtype, device=device) for s in specs]
+
+        def each(have, shape, dt):
+            return [torch.zeros(shape(s), dtype=dt, device=device) if s is not None and have(s) else None for s in specs]
+
+        f32 = torch.float32
+        self.ssm = each(lambda s: s.heads, lambda s: (num_slots, s.heads, s.rows, s.cols), f32)
+        self.vec = each(lambda s: s.vec, lambda s: (num_slots, s.heads, s.vec), f32)
+        self.conv = each(lambda s: s.conv_channels, lambda s: (num_slots, s.conv_rows, s.conv_channels), dtype)
+        self.canon = each(lambda s: s.canon_parts, lambda s: (s.canon_parts, num_slots, s.canon_rows, s.canon_channels), dtype)
 
     @staticmethod
     def bytes_per_slot(specs: list, dtype: torch.dtype) -> int:
         es = torch.empty(0, dtype=dtype).element_size()
-        return sum(4 * s.heads * s.rows * s.cols + es * s.conv_rows * s.conv_channels for s in specs if s is not None)
+        return sum(4 * s.heads * (s.rows * s.cols + s.vec) + es * (s.conv_rows * s.conv_channels + s.canon_parts * s.canon_rows * s.canon_channels)
+                   for s in specs if s is not None)
 
 
 class KVCache:

@@ -1,23 +1,83 @@
 """Serving forward pass of the layer-stack models (models/stack.py): softmax attention over the paged cache and
 recurrent layers over per-sequence states, on the same engine, scheduler, block manager and sampler as the Llama family.
 
-A step's rows are [decode rows | prompt rows]; a prompt's rows may be any portion of it. Norms act on the sublayer
-outputs only, so every sublayer reads the residual itself: the fp32 stream and, for 16-bit compute, its rounded copy that
-the norm-and-add kernel writes next to it."""
+A step's rows are [decode rows | prompt rows]; a prompt's rows may be any portion of it. A model is a list of sublayers
+(mixers and feed-forwards); what lies between two of them — adding an output to the residual, norms, the next sublayer's
+input — is one object per kind of residual."""
 from __future__ import annotations
 
 import os
 
 import torch
 
-from ..models.stack import AttentionMixer, LightningMixer, Mamba2Mixer, StackConfig, StackWeights, mixer_sections, round8
+from ..models.stack import (AttentionMixer, LatentAttentionMixer, LightningMixer, Mamba2Mixer, MLstmMixer, StackConfig, StackWeights,
+                            mixer_sections, round8)
 from ..ops import _lib
+from ..ops import latent as LA
 from ..ops import stack as K
+from ..ops import streams as H
 from ..ops.gemm import gemm_relu2, gemm_skinny_acc
 from .kv_cache import KVCache, KVSpec, StateCache, StateSpec
 
 
 _FUSE_ACC = os.environ.get("DLTI_DECODE_FUSE_ACC", "1") == "1"    # A/B switch: consume the fp32 accumulators directly
+
+
+class OutputNorms:
+    """One residual; norms act on the sublayer outputs only, so every sublayer reads the residual itself: the fp32 stream and,
+    for 16-bit compute, its rounded copy that the norm-and-add kernel writes next to it. A sublayer is named (weights, 1 for
+    the mixer or 2 for the feed-forward, layer)."""
+
+    def __init__(self, run: "StackRunner", ids, rows: K.Rows, first, acc: bool):
+        self.run, self.acc = run, acc
+        self.x, self.h = K.embed_rows(ids, run.w.embed)
+
+    def step(self, y, done, then):
+        """The output y of the sublayer `done` goes to the residual; returns the input of the sublayer `then` (None: the last)."""
+        cfg = self.run.cfg
+        self.h = K.post_norm_add_(y, self.x, done[0][f"norm{done[1]}"], cfg.norm_eps, cfg.norm_one_plus, self.run.dtype, acc=self.acc)
+        return self.h
+
+    def residual(self):
+        return self.x.clone()
+
+    def final(self, idx):
+        cfg = self.run.cfg
+        return K.rms_rows(self.x, idx, self.run.w.final_norm, cfg.norm_eps, cfg.norm_one_plus, self.run.dtype)
+
+
+class HyperStreams:
+    """Several residual streams around pre-norm sublayers (ops/streams.py): one kernel between two sublayers renews the streams and
+    makes the next normed input; the convolution of the input is part of it when every sequence has one row."""
+
+    def __init__(self, run: "StackRunner", ids, rows: K.Rows, first, acc: bool):
+        self.run, self.rows, self.acc = run, rows, acc
+        self.single = rows.nd == ids.numel()
+        self.x = H.embed_streams(ids, run.w.embed, run.cfg.streams, run.cfg.embed_scale)
+        self.last = None
+        self.h = self._between(None, None, first)
+
+    def _between(self, y, done, then):
+        run = self.run
+        mix = w_out = w_in = norm = conv = None
+        if done is not None:
+            mix, w_out = done[0][f"hc{done[1]}.mix"], done[0][f"hc{done[1]}.out"]
+        if then is not None:
+            lw, q, i = then
+            w_in, norm = lw[f"hc{q}.in"], lw[f"norm{q}"]
+            conv = (lw[f"canon{q}"], run.states.canon[i][q - 1], self.rows)
+        h = H.hyper_(self.x, y, mix, w_out, w_in, norm, run.cfg.norm_eps, run.dtype, conv=conv if self.single else None,
+                     acc=self.acc and y is not None)
+        return h if self.single or then is None else H.canon(h, *conv)
+
+    def step(self, y, done, then):
+        return self._between(y, done, then)
+
+    def residual(self):
+        return self.x.sum(1)
+
+    def final(self, idx):
+        return H.hyper_(self.x, None, None, None, None, self.run.w.final_norm, self.run.cfg.norm_eps, self.run.dtype, idx=idx)
 
 
 class StackRunner:
@@ -29,13 +89,20 @@ class StackRunner:
         kv, st = [], []
         for l in cfg.layers:
             m = l.mixer
-            kv.append(KVSpec(m.kv_heads, round8(m.dim), round8(m.vdim), m.kv_from) if isinstance(m, AttentionMixer) else None)
-            if isinstance(m, Mamba2Mixer):
-                st.append(StateSpec(m.heads, m.state, m.vdim, m.conv - 1, m.conv_channels if m.conv > 1 else 0))
-            elif isinstance(m, LightningMixer):
-                st.append(StateSpec(m.heads, m.dim, m.vdim))
+            if isinstance(m, AttentionMixer):
+                kv.append(KVSpec(m.kv_heads, round8(m.dim), round8(m.vdim), m.kv_from))
             else:
-                st.append(None)
+                kv.append(KVSpec(1, m.pitch, 0) if isinstance(m, LatentAttentionMixer) else None)
+            state = {}
+            if isinstance(m, Mamba2Mixer):
+                state = dict(heads=m.heads, rows=m.state, cols=m.vdim, conv_rows=m.conv - 1, conv_channels=m.conv_channels if m.conv > 1 else 0)
+            elif isinstance(m, LightningMixer):
+                state = dict(heads=m.heads, rows=m.dim, cols=m.vdim)
+            elif isinstance(m, MLstmMixer):
+                state = dict(heads=m.heads, rows=m.dim, cols=m.vdim, vec=K.mlstm_vec(m.dim, m.vdim))
+            if cfg.streams:
+                state |= dict(canon_parts=1 if l.mlp is None else 2, canon_rows=cfg.canon - 1, canon_channels=cfg.hidden_size)
+            st.append(StateSpec(**state) if state else None)
         return kv, st
 
     def __init__(self, cfg: StackConfig, weights: StackWeights, kv: KVCache, states: StateCache | None, max_len: int):
@@ -43,12 +110,16 @@ class StackRunner:
         self.device, self.dtype = weights.device, weights.dtype
         self.sections = [mixer_sections(l.mixer) for l in cfg.layers]
         self.ropes = [K.rope_tables(max_len, l.mixer.rope.dims, l.mixer.rope.base, self.device)
-                      if isinstance(l.mixer, AttentionMixer) and l.mixer.rope is not None else None for l in cfg.layers]
+                      if getattr(l.mixer, "rope", None) is not None else None for l in cfg.layers]
         if self.device.type == "cuda" and "DLTI_PDL" not in os.environ:
             # serving weights are static: the decode GEMMs may fetch weight tiles while the previous kernel drains
             _lib.gpu_lib().dlti_set_pdl(2)
         self.pack_prompts = True     # False: all prompt attention reads the pages
-        self.trace = None            # set to a list: receives the residual stream after every layer (debugging)
+        self.trace = None            # set to a list: receives the residual after every layer (debugging)
+        self.mixers = {AttentionMixer: self._attention, LatentAttentionMixer: self._latent, Mamba2Mixer: self._mamba2,
+                       LightningMixer: self._lightning, MLstmMixer: self._mlstm}
+        # the sublayers in order: (layer weights, 1 mixer | 2 feed-forward, layer)
+        self.parts = [(lw, q, i) for i, (l, lw) in enumerate(zip(cfg.layers, weights.layers)) for q in ((1, 2) if l.mlp is not None else (1,))]
 
     @torch.no_grad()
     def forward(self, input_ids, positions, slots, *, num_decode: int = 0, block_tables=None, ctx_lens=None, cu_seqlens=None,
@@ -58,34 +129,31 @@ class StackRunner:
         cfg, w = self.cfg, self.w
         rows = K.Rows(positions, row_seq, slots, ctx_lens, cu_seqlens, block_tables, state_slots, int(num_decode), max_seqlen,
                       max_ctx)
-        x, xa = K.embed_rows(input_ids.view(-1), w.embed)
+        ids = input_ids.view(-1)
         # decode-sized steps stream the weights through the stream-K GEMM; the next op consumes its fp32 accumulator
-        self.acc = acc = _FUSE_ACC and x.is_cuda and self.dtype == torch.bfloat16 and x.shape[0] <= 256
-        mm = gemm_skinny_acc if acc else K.linear
-        for i, (l, lw) in enumerate(zip(cfg.layers, w.layers)):
-            m = l.mixer
-            if isinstance(m, AttentionMixer):
-                y = self._attention(i, m, lw, xa, rows, segs)
-            elif isinstance(m, Mamba2Mixer):
-                y = self._mamba2(i, m, lw, xa, rows)
+        self.acc = _FUSE_ACC and w.embed.is_cuda and self.dtype == torch.bfloat16 and ids.numel() <= 256
+        mm = gemm_skinny_acc if self.acc else K.linear
+        res = (HyperStreams if cfg.streams else OutputNorms)(self, ids, rows, self.parts[0], self.acc)
+        h = res.h
+        for part, then in zip(self.parts, self.parts[1:] + [None]):
+            lw, q, i = part
+            m = cfg.layers[i].mixer
+            if q == 1:
+                y = mm(self.mixers[type(m)](i, m, lw, h, rows, segs), lw["w_out"])
             else:
-                y = self._lightning(i, m, lw, xa, rows)
-            xa = self._close(mm(y, lw["w_out"]), x, lw["norm1"])
-            if l.mlp is not None:
-                h = gemm_relu2(xa, lw["w_up"], l.mlp.ff) if x.is_cuda and not acc else None      # activation in the GEMM
-                if h is None:
-                    h = K.relu2(mm(xa, lw["w_up"]), l.mlp.ff, self.dtype, acc=acc)
-                xa = self._close(mm(h, lw["w_down"]), x, lw["norm2"])
-            if self.trace is not None:
-                self.trace.append(x.clone())
+                y = mm(self._mlp(cfg.layers[i].mlp, lw, h, mm), lw["w_down"])
+            h = res.step(y, part, then)
+            if self.trace is not None and (then is None or then[2] != i):
+                self.trace.append(res.residual())
         if last_idx is not None and last_idx.numel() == 0:
             return torch.empty((0, cfg.vocab_size), dtype=torch.float32, device=self.device)
-        xn = K.rms_rows(x, last_idx, w.final_norm, cfg.norm_eps, cfg.norm_one_plus, self.dtype)
-        return K.linear_f32(xn, w.lm_head)[:, :cfg.vocab_size]
+        return K.linear_f32(res.final(last_idx), w.lm_head)[:, :cfg.vocab_size]
 
-    def _close(self, y, x, norm):
-        """End of a sublayer: x += norm(y); returns the next sublayer's input."""
-        return K.post_norm_add_(y, x, norm, self.cfg.norm_eps, self.cfg.norm_one_plus, self.dtype, acc=self.acc)
+    def _mlp(self, mlp, lw, h, mm):
+        if mlp.act == "polynorm":
+            return H.poly_norm(mm(h, lw["w_up"]), mlp.ff, lw["act"], self.cfg.norm_eps, self.dtype, acc=self.acc)
+        u = gemm_relu2(h, lw["w_up"], mlp.ff) if h.is_cuda and not self.acc else None      # activation in the GEMM
+        return K.relu2(mm(h, lw["w_up"]), mlp.ff, self.dtype, acc=self.acc) if u is None else u
 
     def _attention(self, i, m: AttentionMixer, lw, xa, rows: K.Rows, segs):
         # prompts with heads of up to 128: the varlen tcgen05 kernel on rows cut at the chunk edges; everything else
@@ -101,7 +169,7 @@ class StackRunner:
             return K.packed_attention(q, m, rows, packed, self.kv.k[i], self.kv.v[i], gate)
         return K.paged_attention(q, m, rows, self.kv.k[i], self.kv.v[i], gate)
 
-    def _mamba2(self, i, m: Mamba2Mixer, lw, xa, rows: K.Rows):
+    def _mamba2(self, i, m: Mamba2Mixer, lw, xa, rows: K.Rows, segs):
         s, st = self.sections[i], self.states
         inner, gn = m.inner, m.groups * m.state
         acc = self.acc and rows.nd == xa.shape[0]                 # the convolution of prompt rows reads its neighbours' inputs
@@ -113,10 +181,23 @@ class StackRunner:
                           m.state, m.vdim, conv_src=proj, conv_col=s["xbc"], conv_state=st.conv[i])
         return K.gated_norm(y, proj[:, s["z"]:s["z"] + inner], lw["norm"], self.cfg.norm_eps, m.norm_groups, gate_first=True)
 
-    def _lightning(self, i, m: LightningMixer, lw, xa, rows: K.Rows):
+    def _lightning(self, i, m: LightningMixer, lw, xa, rows: K.Rows, segs):
         s = self.sections[i]
         proj = K.linear(xa, lw["w_in"])
         qk, vv = m.heads * m.dim, m.heads * m.vdim
         y = K.linear_scan(proj[:, s["q"]:s["q"] + qk], proj[:, s["k"]:s["k"] + qk], proj[:, s["v"]:s["v"] + vv],
                           K.Decay(const=lw["decay"]), self.states.ssm[i], rows, m.heads, m.heads, m.dim, m.vdim, silu=True)
         return K.gated_norm(y, proj[:, s["g"]:s["g"] + vv], lw["norm"], self.cfg.norm_eps, 1, gate_first=False)
+
+    def _latent(self, i, m: LatentAttentionMixer, lw, xa, rows: K.Rows, segs):
+        proj = gemm_skinny_acc(xa, lw["w_in"]) if self.acc else K.linear(xa, lw["w_in"])
+        return LA.latent_attention(proj, self.sections[i], m, lw, self.w.derived[i].get("w_expand"), self.cfg.norm_eps, rows, self.ropes[i],
+                                   self.kv.k[i], self.dtype, (segs or {}).get(m.chunk) if self.pack_prompts else None, acc=self.acc)
+
+    def _mlstm(self, i, m: MLstmMixer, lw, xa, rows: K.Rows, segs):
+        s, st = self.sections[i], self.states
+        qk, vv = m.heads * m.dim, m.heads * m.vdim
+        proj, gates = H.linear_split(xa, lw["w_in"], s["gates"])
+        y = K.mlstm_scan(proj[:, s["q"]:s["q"] + qk], proj[:, s["k"]:s["k"] + qk], proj[:, s["v"]:s["v"] + vv], gates, lw["gate_b"], m.gate_cap,
+                         st.ssm[i], st.vec[i], rows, m.heads, m.dim, m.vdim)
+        return K.gated_norm(y, proj[:, s["g"]:s["g"] + vv], lw["norm"], self.cfg.norm_eps, m.heads, gate_first=False)

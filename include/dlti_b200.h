@@ -348,7 +348,7 @@ int dlti_sample(const void* logits, long long ld, int batch, int V, const float*
                 unsigned long long step, long long* out, float* out_logprob, int dtype,
                 dlti_stream_t stream);
 
-/* ---- Layer-stack models (models/stack.py): csrc/stack.cu, recurrent.cu, attention_paged.cu, gemm_f32.cu. Row pitches (*_ld) in
+/* ---- Layer-stack models (models/stack.py): csrc/stack.cu, streams.cu, recurrent.cu, attention_paged.cu, latent.cu, gemm_f32.cu. Row pitches (*_ld) in
  * elements. Sequences of a step: the first nd are single rows, sequence nd + i has rows nd + cu[i] ... nd + cu[i+1]; ctx[s] = tokens
  * of sequence s after the step, rseq[t] = sequence of row t, sslot[s] = its state slot (-1 = none). */
 /* C[M,N] = A[M,K] * B[N,K]^T in true fp32 (no TF32) */
@@ -404,24 +404,62 @@ int dlti_linear_scan_chunked(const void* q, long long q_ld, const void* k, long 
     conv_C, void* conv_state, dlti_stream_t stream);
 /* x = silu(x) in place */
 int dlti_silu_rows(void* x, long long ld, long long rows, int n, int dtype, dlti_stream_t stream);
-/* paged attention, one warp per (row, head), fp32 arithmetic; chunk > 0: a position sees its own chunk only */
+/* paged attention, one warp per (row, head), fp32 arithmetic; chunk > 0: a position sees its own chunk only. sink [H] (may be NULL, also
+ * below): one more term exp(sink) in a head's softmax denominator */
 int dlti_attn_rows(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd, const int*
     tables, int max_blocks, int bs, const int* ctx, const int* rseq, const int* pos, int H, int G, int dim, int vdim,
-    int chunk, float scale, const float* gate, void* out, long long o_ld, long long rows, int dtype, dlti_stream_t
-    stream);
+    int chunk, float scale, const float* gate, const float* sink, void* out, long long o_ld, long long rows, int dtype,
+    dlti_stream_t stream);
 /* paged attention of prompt portions (bf16, heads <= 256) */
 int dlti_attn_paged_prefill(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
     const int* tables, int max_blocks, int bs, const int* ctx, const int* cu, int nd, int nseq, int max_rows, int H,
-    int G, int dim, int vdim, int chunk, float scale, const float* gate, void* out, long long o_ld, dlti_stream_t
+    int G, int dim, int vdim, int chunk, float scale, const float* gate, const float* sink, void* out, long long o_ld, dlti_stream_t
     stream);
 /* paged attention of decode rows (bf16, grouped heads, split over CTAs); ws: batch * H * splits * (vdim + 2) floats */
 int dlti_attn_paged_decode(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
     const int* tables, int max_blocks, int bs, const int* ctx, int batch, int H, int G, int dim, int vdim, int chunk,
-    float scale, const float* gate, int splits, float* ws, void* out, long long o_ld, dlti_stream_t stream);
+    float scale, const float* gate, const float* sink, int splits, float* ws, void* out, long long o_ld, dlti_stream_t stream);
 /* varlen causal attention with the softmax weights as two bf16 terms; see attention.cu */
-int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const int* cu_seqlens, const int*
+int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const float* sink, const int* cu_seqlens, const int*
     seq_q0, const int* seq_out0, int batch, int max_seqlen, long long T_total, int H, int KV, int vdim, float scale,
     dlti_stream_t stream);
+
+/* mLSTM: the recurrence above with exponential gates, a running maximum and a normaliser; see recurrent.cu. gates [rows, >= 2 heads]
+ * raw fp32 (input, forget), vec [slots, heads, ceil(P / 32), N + 1] */
+int dlti_mlstm_scan(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long v_ld, const float* gates,
+    long long g_ld, const float* gate_b, float cap, float q_scale, float* state, float* vec, const int* sslot, const int* ctx, const
+    int* cu, int nd, int seq0, int nseq, int heads, int N, int P, void* out, long long o_ld, int chunked, int dtype, dlti_stream_t stream);
+/* streams.cu. Hyper-connections between two sublayers: x_t <- sum_s mix[s,t] x_s + out[t] y on x [rows, S, d] (y may be NULL), then
+ * h = layer_norm(sum_s in[s] x_s) * w (w may be NULL), then (cw, one token per sequence) plus its causal convolution */
+int dlti_hyper(float* x, int S, int d, const void* y, long long y_ld, const float* mix, const float* out, const float* in, const float*
+    w, float eps, const float* cw, int cw_ld, int taps, void* cstate, const int* sslot, const int* ctx, void* h, long long h_ld, const
+    long long* idx, long long rows, int acc, int dtype, dlti_stream_t stream);
+/* x[t, s] = table[ids[t]] * scale */
+int dlti_embed_streams(const long long* ids, const void* table, float* x, long long tokens, int S, int d, long long vocab, float scale,
+    int dtype, dlti_stream_t stream);
+/* out = h + causal convolution of h; state [slots, taps - 1, d] is read and renewed */
+int dlti_canon(const void* h, long long h_ld, int d, int taps, const float* w, int w_ld, void* state, const int* sslot, const int* ctx,
+    const int* cu, int nd, int seq0, int nseq, int max_rows, void* out, long long o_ld, int dtype, dlti_stream_t stream);
+/* out = a N(z) + b N(z^2) + c N(z^3) + e, N(y) = y / rms(y); coef = {a, b, c, e} */
+int dlti_poly_norm(const void* z, long long z_ld, const float* coef, void* out, long long o_ld, long long rows, int n, float eps, int
+    acc, int dtype, dlti_stream_t stream);
+/* accumulator columns [0, split) as dtype, the rest as fp32; the accumulator becomes zero */
+int dlti_split_rows(float* acc, void* out, long long o_ld, float* tail, long long t_ld, long long rows, int n, int split, int dtype,
+    dlti_stream_t stream);
+/* latent.cu: latent attention. A cache row is [c, zeros, k_rot, zeros], rot_at = round16(rank), pitch = rot_at + round16(rot) */
+int dlti_latent_prep(const void* proj, long long ld, int oq, int od, int og, int H, int dim, int rot, int rank, int rd, int interleaved,
+    const float* cos_t, const float* sin_t, const int* pos, const float* kvw, float eps, const long long* slots, void* cache, int
+    pitch, int rot_at, int nabs, void* qn, int qn_hd, void* ql, void* qp, long long qp_ld, int qp_hd, void* lat, const int* qdst, const int* dst,
+    float* gate, long long tokens, int acc, int dtype, dlti_stream_t stream);
+/* lat[rows[i]] = cache[slots[i]] */
+int dlti_latent_rows(void* lat, const void* cache, int pitch, const int* rows, const int* slots, long long n, dlti_stream_t stream);
+/* out[t, h] = a[t, h] B_h, B_h = K rows of b [H*K, N] (kn) or the transpose of N rows of b [H*N, K] */
+int dlti_head_gemm(const void* a, long long a_ld, int a_hd, const void* b, long long b_ld, void* out, long long o_ld, int o_hd, long long
+    rows, int H, int K, int N, int kn, int dtype, dlti_stream_t stream);
+/* absorbed latent attention (bf16): q [rows, H, pitch] against the cached rows, values = their first rank columns */
+int dlti_latent_decode(const void* q, const void* cache, int pitch, int rank, const int* tables, int max_blocks, int bs, const int* ctx,
+    const int* rseq, const int* pos, long long rows, int H, float scale, const float* sink, const float* gate, int heads_per_cta, int
+    splits, float* ws, void* out, int o_hd, dlti_stream_t stream);
 
 #ifdef DLTI_ATTN_TRACE
 /* Developer builds only (-DDLTI_ATTN_TRACE): clock64() timeline of CTA (0,0,0) of the last backward
