@@ -63,11 +63,11 @@ def attend(q, k, v, scale, sink):
     return out
 
 
-def latent_attention(h, p, m, eps):
-    T, H = h.shape[0], m["heads"]
-    q = (h @ p["q"].T).view(T, H, m["dim"] + m["rot_dim"])
+def latent_heads(q, down, gate, p, m, eps):
+    """Projected rows (queries, latent | shared key part, gate numbers) -> head outputs [T, H * vdim]."""
+    T, H = q.shape[0], m["heads"]
+    q = q.view(T, H, m["dim"] + m["rot_dim"])
     q_plain, q_rot = q[..., :m["dim"]], q[..., m["dim"]:]
-    down = h @ p["dkv"].T
     c = down[:, :m["kv_rank"]]
     c = c / root_mean_square(c, eps) * p["dkv.norm"]
     k_rot = rotate_pairs(down[:, m["kv_rank"]:], m["rot"]["base"], m["rot"]["dims"])
@@ -76,8 +76,11 @@ def latent_attention(h, p, m, eps):
     v = (c @ p["uv"].T).view(T, H, m["vdim"])
     k = torch.cat([k_plain, k_rot[:, None].expand(T, H, m["rot_dim"])], -1)
     o = attend(torch.cat([q_plain, q_rot], -1), k, v, m["scale"], p["sink"])
-    o = o * torch.sigmoid(h @ p["g"].T)[:, :, None]
-    return o.reshape(T, -1) @ p["o"].T
+    return (o * torch.sigmoid(gate)[:, :, None]).reshape(T, -1)
+
+
+def latent_attention(h, p, m, eps):
+    return latent_heads(h @ p["q"].T, h @ p["dkv"].T, h @ p["g"].T, p, m, eps) @ p["o"].T
 
 
 def log_sigmoid(z):

@@ -11,8 +11,8 @@ import torch
 
 from dlti_b200.models.stack import AttentionMixer, Rope, Sections, round8
 from dlti_b200.ops import _lib
-from tests.sigosun_util import (CONFIGS, K, R, SG, Replay, check, engine, mixed_schedule, model, mutated, oracle, random, random_portions,
-                                row_errors, rows_for, tokens)
+from tests.sigosun_util import (CONFIGS, K, R, SG, ZOO, Replay, check, engine, mixed_schedule, model, mutated, oracle, random,
+                                random_portions, row_errors, rows_for, tokens)
 
 F32, BF16 = torch.float32, torch.bfloat16
 GPU = pytest.mark.gpu
@@ -384,34 +384,15 @@ def test_residual_stream_after_every_layer():
 
 
 # ---- generation through the scheduler ----------------------------------------------------------------------
-def _greedy(name, prompt, n):
-    d, _, _, w = model(name)
-    seq = list(prompt)
-    for _ in range(n):
-        seq.append(int(R.forward(d, w, seq)[-1].argmax()))
-    return seq[len(prompt):]
-
-
-def _generate(name, device, **kw):
-    from dlti_b200.serve.params import SamplingParams
-    prompts = [tokens(name, n, 20 + n) for n in (5, 33, 1, 60, 18, 2)]
-    eng = engine(name, device, F32, max_num_seqs=3, **kw)
-    outs = eng.generate(prompts, SamplingParams(max_tokens=9, temperature=0.0, ignore_eos=True))
-    for p, o in zip(prompts, outs):
-        assert o["token_ids"] == _greedy(name, p, 9)
-    assert eng.blocks.num_free == eng.blocks.num_blocks and (eng.slots is None or len(eng.slots.free) == 3)
-    return eng
-
-
 @pytest.mark.parametrize("device", ["cpu", pytest.param("cuda", marks=GPU)])
 @pytest.mark.parametrize("kw", [dict(), dict(prefill_chunk=7), dict(mixed_batches=False), dict(async_scheduling=False)], ids=str)
 def test_greedy_generation(device, kw):
-    _generate("odd", device, **kw)
+    ZOO.check_generation("odd", device, **kw)
 
 
 @pytest.mark.parametrize("device", ["cpu", pytest.param("cuda", marks=GPU)])
 def test_greedy_generation_with_preemption(device):
-    eng = _generate("ones", device, num_blocks=6, max_len=128)
+    eng = ZOO.check_generation("ones", device, num_blocks=6, max_len=128)
     assert eng.sched.num_preemptions > 0
 
 
@@ -490,7 +471,7 @@ def test_prefix_caching_is_open_to_stateless_stacks():
     eng = engine("tall", "cpu", F32, enable_prefix_caching=True)
     p = tokens("tall", 50, 3)
     sp = SamplingParams(max_tokens=4, temperature=0.0, ignore_eos=True)
-    want = _greedy("tall", p, 4)
+    want = ZOO.greedy("tall", p, 4)
     assert eng.generate([p], sp)[0]["token_ids"] == want and eng.generate([p], sp)[0]["token_ids"] == want
     assert eng.blocks.hits >= 48
 
