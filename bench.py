@@ -55,10 +55,11 @@ def parse():
     ap.add_argument("--offload", action="store_true",
                     help="run the ds_config as shipped (ZeRO-Offload of optimizer state and parameters to pinned host "
                          "memory) instead of the HBM-resident default; a secondary measurement, not the headline (689 ms vs 631 ms per step on one B200)")
-    ap.add_argument("--workload", default="train", choices=["train", "sigosun"],
+    ap.add_argument("--workload", default="train", choices=["train", "sigosun", "logozen"],
                     help="train: the headline benchmark (default). sigosun: prefill and decode throughput of the Sigosun family "
-                         "beside Llama models of equal size, with every kernel's fraction of its roofline (1 GPU)")
-    ap.add_argument("--sizes", default="2048x4,4096x2", help="--workload sigosun: width x groups of four layers, comma-separated")
+                         "beside Llama models of equal size, with every kernel's fraction of its roofline (1 GPU). logozen: the Logozen "
+                         "family beside Sigosun models of equal size")
+    ap.add_argument("--sizes", default="2048x4,4096x2", help="--workload sigosun, logozen: width x groups of four Sigosun layers, comma-separated")
     return ap.parse_args()
 
 
@@ -126,13 +127,13 @@ def main() -> None:
     if a.impl == "reference":
         reference_arm(a)
         return
-    if a.workload == "sigosun":
+    if a.workload != "train":
         from dlti_b200.serve import layer_bench
         try:
             peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
         except OSError:
             peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
-        layer_bench.run_cli(a.steps, a.warmup, a.sizes, peaks, ClockSampler(0))
+        layer_bench.run_cli(a.steps, a.warmup, a.sizes, peaks, ClockSampler(0), a.workload)
         return
     if a.impl == "standin":
         sys.path.insert(0, os.path.join(ROOT, "baseline"))

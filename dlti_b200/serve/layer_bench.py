@@ -1,5 +1,6 @@
-"""Serving throughput of the Sigosun family beside Llama models of equal size, and the time of each kernel of the two
-against its roofline (`bench.py --workload sigosun`). Random weights; layer sizes of real models.
+"""Serving throughput of a layer-stack family beside the closest other family at equal size, and the time of each kernel of
+the two against its roofline: Sigosun beside Llama (`bench.py --workload sigosun`), Logozen beside Sigosun (`--workload
+logozen`). Random weights; layer sizes of real models.
 
 Steps go through LLMEngine.pack_step / _run_step (packing, host-to-device copy, forward, sampling; decode steps replay
 CUDA graphs), timed with CUDA events. Kernels are timed one call at a time with the L2 overwritten before each."""
@@ -13,13 +14,17 @@ import torch
 
 from ..models.config import LlamaConfig
 from ..models.registry import family_of
+from ..models.logozen import LogozenConfig
 from ..models.sigosun import SigosunConfig
-from ..models.stack import AttentionMixer, DenseMlp, Layer, LightningMixer, Mamba2Mixer, Rope, mixer_sections
+from ..models.stack import (AttentionMixer, DenseMlp, LatentAttentionMixer, Layer, LightningMixer, Mamba2Mixer, MLstmMixer, Rope,
+                            StackWeights, mixer_sections)
 from ..ops import _lib
 from ..ops import attention as A
 from ..ops import elementwise as E
+from ..ops import latent as LA
 from ..ops import serving as S
 from ..ops import stack as K
+from ..ops import streams as HS
 from ..ops.gemm import gemm, gemm_relu2, gemm_skinny, gemm_skinny_acc
 from .engine import LLMEngine, _pieces, chunk_pieces
 from .model_runner import TPContext
@@ -36,6 +41,20 @@ def _sigosun(width: int, blocks: int) -> SigosunConfig:
     for b in range(blocks):
         layers += [Layer(att, ff), Layer(replace(att, kv_from=4 * b), ff), Layer(mam, None), Layer(lig, None)]
     return SigosunConfig(hidden_size=width, vocab_size=32000, norm_eps=1e-6, layers=layers, name=f"sigosun-{width}x{4 * blocks}")
+
+
+def _logozen(width: int, params: int) -> LogozenConfig:
+    """Pairs of layers (mLSTM, latent attention), each with a feed-forward, that together hold about `params` parameters."""
+    heads = width // 128
+    att = LatentAttentionMixer(heads=heads, dim=64, rot_dim=64, vdim=128, kv_rank=512, scale=128 ** -0.5, rope=Rope(64, 1e6))
+    mem = MLstmMixer(heads=heads // 2, dim=128, vdim=256, gate_cap=15.0)
+    ff = DenseMlp(4 * width, act="polynorm")
+
+    def cfg(n):
+        return LogozenConfig(hidden_size=width, vocab_size=32000, norm_eps=1e-6, norm_one_plus=False, streams=4, canon=4, embed_scale=45.0,
+                             layers=[Layer(mem, ff), Layer(att, ff)] * n, name=f"logozen-{width}x{2 * n}")
+    one = cfg(2).num_params() - cfg(1).num_params()
+    return cfg(max(1, round(params / one)))
 
 
 def _llama(width: int, params: int) -> LlamaConfig:
@@ -104,11 +123,15 @@ def step_bytes(eng: LLMEngine, batch: int, ctx: int) -> int:
         return n + 2 * 2 * cfg.num_hidden_layers * batch * (ctx + 1) * w.KV * cfg.head_dim
     for i, l in enumerate(cfg.layers):
         m = l.mixer
-        if isinstance(m, AttentionMixer):
+        if eng.states is not None and eng.states.canon[i] is not None:
+            n += 2 * batch * size(eng.states.canon[i][:, 0])
+        if isinstance(m, LatentAttentionMixer):
+            n += 2 * batch * (ctx + 1) * m.pitch
+        elif isinstance(m, AttentionMixer):
             seen = ctx + 1 - (ctx // m.chunk * m.chunk if m.chunk else 0)
             n += 2 * batch * seen * m.kv_heads * (m.dim + m.vdim)
         else:
-            n += 2 * batch * 4 * eng.states.ssm[i][0].numel()
+            n += 2 * batch * 4 * (eng.states.ssm[i][0].numel() + (0 if eng.states.vec[i] is None else eng.states.vec[i][0].numel()))
     return n
 
 
@@ -288,17 +311,101 @@ def kernels(width: int, peaks: dict, nseq: int, length: int, batch: int, ctx: in
     return k.rows
 
 
-def main(steps: int, warmup: int, sizes: str, peaks: dict, sampler) -> dict:
+def logozen_kernels(width: int, peaks: dict, nseq: int, length: int, batch: int, ctx: int, iters: int) -> list[dict]:
+    """The kernels of Logozen in the same two steps; those of Sigosun come from kernels()."""
+    k = _Kernels(peaks, iters)
+    cfg = _logozen(width, 1)
+    mem, m, d, dev, bf = cfg.layers[0].mixer, cfg.layers[1].mixer, width, "cuda", torch.bfloat16
+    w = StackWeights(cfg, dev, bf).finish()
+    lw, w_expand = w.layers[1], w.derived[1]["w_expand"]
+    rnd = lambda *s: torch.randn(*s, device=dev, dtype=bf)
+    for t in (lw["w_uk"], lw["w_uv"], w_expand):
+        t.normal_(0, 0.04)
+    T, bs, heads, R = nseq * length, 16, m.heads, m.kv_rank
+    per = -(-max(length, ctx + 1) // bs)
+    n_all = max(nseq, batch)
+    tabs = torch.arange(n_all * per, dtype=torch.int32, device=dev).view(n_all, per)
+    cache = rnd(n_all * per, bs, 1, m.pitch)
+    tab_r = K.rope_tables(max(length, ctx + 1), m.rope.dims, m.rope.base, dev)
+    pslots = torch.cat([torch.arange(length) + i * per * bs for i in range(nseq)]).to(dev)
+    dslots = torch.tensor([i * per * bs + ctx for i in range(batch)], device=dev)
+    pr = _rows([(0, length)] * nseq, 0, tabs[:nseq].contiguous(), pslots, length)
+    dr = _rows([(ctx, 1)] * batch, batch, tabs[:batch].contiguous(), dslots, ctx + 1)
+    pieces = K.Pieces(torch.tensor([i * length for i in range(nseq + 1)], dtype=torch.int32, device=dev), length, T)
+    pairs = length * (length + 1) // 2
+    hp = m.head_pitch
+    buf, gate, out, lat = rnd(T, 3 * heads * hp), torch.rand(T, heads, device=dev), K.act(T, heads * m.vdim, bf, dev), rnd(T, m.pitch)
+    run = lambda phase, name, fn, nbytes, flops=0.0: k.run("logozen", phase, name, fn, nbytes, flops)
+    run("prefill", "attention (packed)", lambda: K.attn_fwd_split(buf, m, heads, heads, pieces, gate, out, sink=lw["sink"]),
+        T * heads * (2 * m.qk_dim + 2 * m.vdim) * 2, 2.0 * nseq * pairs * heads * (m.qk_dim + m.vdim))
+    useful = heads * (m.dim + m.vdim)
+    run("prefill", "GEMM latents -> keys, values", lambda: gemm(lat, w_expand, out=buf[:, heads * hp:]),
+        2 * (T * m.pitch + w_expand.numel() + 2 * T * heads * hp), 2.0 * T * useful * R)
+    qa, od = rnd(batch, heads * m.pitch), torch.empty(batch, heads * R, device=dev, dtype=bf)
+    gd = torch.rand(batch, heads, device=dev)
+    run("decode", "attention", lambda: LA.latent_decode(qa, m, dr, cache, gd, lw["sink"], od), batch * (ctx + 1) * m.pitch * 2,
+        2.0 * batch * (ctx + 1) * heads * (m.pitch + R))
+    qn, o = rnd(batch, heads * m.dim), torch.empty(batch, heads * m.vdim, device=dev, dtype=bf)
+    run("decode", "queries into the latent space", lambda: LA.head_gemm(qn, m.dim, lw["w_uk"], qa, m.pitch, heads, m.dim, R, True),
+        2 * (lw["w_uk"].numel() + qn.numel() + batch * heads * R))
+    run("decode", "latent outputs to values", lambda: LA.head_gemm(od, R, lw["w_uv"], o, m.vdim, heads, R, m.vdim, False),
+        2 * (lw["w_uv"].numel() + od.numel() + o.numel()))
+    sec, sm = mixer_sections(m), mixer_sections(mem)
+    S, ff = cfg.streams, cfg.layers[0].mlp.ff
+    inner, qk = mem.heads * mem.vdim, mem.heads * mem.dim
+    for phase, r, n, ns in (("prefill", pr, T, nseq), ("decode", dr, batch, batch)):
+        acc = phase == "decode"
+        es = 8 if acc else 2                                      # accumulators are read and zeroed
+        z = lambda c: torch.zeros(n, c, device=dev) if acc else rnd(n, c)
+        proj = z(sec.total)
+        run(phase, "latent norm + rope + cache", lambda: LA.latent_prep(proj, sec, m, lw["kv_norm"], 1e-6, r, tab_r, cache, bf, None if acc else pieces, acc),
+            n * (sec.total * es + heads * m.qk_dim * 2 + m.pitch * 2 * (1 if acc else 2) + 4 * heads))
+        x, y = torch.randn(n, S, d, device=dev), z(d)
+        c = w.layers[0]
+        state = torch.zeros(ns, cfg.canon - 1, d, device=dev, dtype=bf)
+        run(phase, "streams + norm (+ convolution)" if acc else "streams + norm", lambda: HS.hyper_(
+            x, y, c["hc1.mix"], c["hc1.out"], c["hc1.in"], c["norm1"], 1e-6, bf, conv=(c["canon1"], state, r) if acc else None, acc=acc),
+            n * d * (es + 8 * S + 2 + (4 * (cfg.canon - 1) if acc else 0)))
+        if not acc:
+            h = rnd(n, d)
+            run(phase, "input convolution", lambda: HS.canon(h, c["canon1"], state, r), n * d * 4)
+        u = z(ff)
+        run(phase, "PolyNorm", lambda: HS.poly_norm(u, ff, c["act"], 1e-6, bf, acc=acc), n * ff * (es + 2))
+        ssm = torch.zeros(ns, mem.heads, mem.dim, mem.vdim, device=dev)
+        vec = torch.zeros(ns, mem.heads, K.mlstm_vec(mem.dim, mem.vdim), device=dev)
+        p, g = rnd(n, sm["gates"]), torch.randn(n, 2 * mem.heads, device=dev)
+        bias = torch.full((2 * mem.heads,), 3.0, device=dev)
+        work = 2.0 * n * mem.heads * (32 * (mem.dim + mem.vdim) + 2 * mem.dim * mem.vdim) if not acc else 4.0 * n * mem.heads * mem.dim * mem.vdim
+        run(phase, "mLSTM scan", lambda: K.mlstm_scan(p[:, :qk], p[:, sm["k"]:sm["k"] + qk], p[:, sm["v"]:sm["v"] + inner], g, bias, 15.0, ssm, vec, r,
+                                                      mem.heads, mem.dim, mem.vdim),
+            n * (2 * qk + 2 * inner) * 2 + n * 8 * mem.heads + ns * 8 * (ssm[0].numel() + vec[0].numel()), work)
+        yb = rnd(n, inner)
+        run(phase, "unit heads + gate", lambda: K.gated_norm(yb, p[:, sm["g"]:sm["g"] + inner], c["norm"], 1e-6, mem.heads, False), n * inner * 6)
+        a = rnd(n, d)
+        split = lambda q, t: HS.linear_split(q, t, sm["gates"])
+        for name, wt, fn in (("GEMM latent attention in", w.layers[1]["w_in"], None), ("GEMM mLSTM in, gates fp32", w.layers[0]["w_in"], split),
+                             ("GEMM up", w.layers[0]["w_up"], None)):
+            N_, K_ = wt.shape
+            mm = fn or (gemm_skinny_acc if acc else gemm)
+            run(phase, name, lambda: mm(a, wt), 2 * (n * K_ + N_ * K_) + n * N_ * (4 if acc else 2), 2.0 * n * N_ * K_)
+            if acc and fn is None:
+                gemm_skinny(a, wt)                                # leaves the shared accumulator zero
+    return k.rows
+
+
+def main(steps: int, warmup: int, sizes: str, peaks: dict, sampler, workload: str = "sigosun") -> dict:
     iters, warmup = max(3, steps), max(3, warmup)
-    out = {"metric": "Sigosun serving tok/s beside Llama of equal size", "impl": "dlti_b200", "dtype": "bf16",
+    name, other = ("Logozen", "Sigosun") if workload == "logozen" else ("Sigosun", "Llama")
+    out = {"metric": f"{name} serving tok/s beside {other} of equal size", "impl": "dlti_b200", "dtype": "bf16",
            "data": "synthetic (random token ids; random-init weights)", "steps": iters, "warmup": warmup, "sizes": [], "kernels": {}}
     _lib.reset_launch_count()
     for spec in sizes.split(","):
         width, blocks = (int(x) for x in spec.split("x"))
         sig = _sigosun(width, blocks)
-        lla = _llama(width, sig.num_params() - 2 * sig.vocab_size * width)
+        params = sig.num_params() - 2 * sig.vocab_size * width
+        models = (_logozen(width, params), sig) if workload == "logozen" else (sig, _llama(width, params))
         row = {"width": width, "rows": []}
-        for cfg in (sig, lla):
+        for cfg in models:
             eng = _engine(cfg, 8704, 64)
             e = {"model": cfg.name, "layers": cfg.num_hidden_layers, "params_m": round(cfg.num_params() / 1e6)}
             for nseq, length in ((1, 8192), (4, 2048), (16, 512)):
@@ -312,7 +419,10 @@ def main(steps: int, warmup: int, sizes: str, peaks: dict, sampler) -> dict:
             del eng
             torch.cuda.empty_cache()
         out["sizes"].append(row)
-        out["kernels"][str(width)] = kernels(width, peaks, 4, 2048, 64, 1000, iters)
+        ks = kernels(width, peaks, 4, 2048, 64, 1000, iters)
+        if workload == "logozen":
+            ks = logozen_kernels(width, peaks, 4, 2048, 64, 1000, iters) + [r for r in ks if r["model"] == "sigosun"]
+        out["kernels"][str(width)] = ks
         torch.cuda.empty_cache()
     out["gpu_launches"] = _lib.launch_count()
     out["clocks"] = sampler.stop()
@@ -335,8 +445,8 @@ def print_tables(out: dict, emit=print) -> None:
             emit(f"{r['model']:8s} {r['phase']:8s} {r['kernel']:30s} {r['us']:9.2f} us, roof {r['roof_us']:8.2f} us = {r['frac_of_roof']:.3f} ({r['bound']})")
 
 
-def run_cli(steps: int, warmup: int, sizes: str, peaks: dict, sampler) -> None:
-    out = main(steps, warmup, sizes, peaks, sampler)
+def run_cli(steps: int, warmup: int, sizes: str, peaks: dict, sampler, workload: str) -> None:
+    out = main(steps, warmup, sizes, peaks, sampler, workload)
     import sys
     print_tables(out, lambda s: print(s, file=sys.stderr))
     print(json.dumps(out))
