@@ -338,10 +338,11 @@ __global__ void __launch_bounds__(128) head_gemm_any_kernel(const HeadGemmParams
   reinterpret_cast<T*>(p.out)[t * p.o_ld + (long long)h * p.o_hd + n] = Cvt<T>::from_f(acc);
 }
 
-// Absorbed attention, bf16. grid (splits, blocks of 16 HT heads, rows), 8 warps; row b belongs to sequence rseq[b] (null: b)
-// and sees its first min(pos[b] + 1, ctx) cached rows (pos null: all ctx). Per tile of 64 cached rows: warps 0-3 and 4-7 each
-// compute the scores of 16 keys over one half of the row's columns, all threads form the softmax weights (hi + lo bf16
-// terms), then a warp owns W16 groups of 16 latent columns of the output.
+// Absorbed attention, bf16. grid (splits, blocks of 16 HT heads, rows), 16 warps; row b belongs to sequence rseq[b] (null: b)
+// and sees its first min(pos[b] + 1, ctx) cached rows (pos null: all ctx). Per tile of 64 cached rows: a warp computes the
+// scores of 16 keys for 16 heads over one of 4 / HT parts of the row's columns, all threads form the softmax weights (hi + lo
+// bf16 terms), then a warp owns W16 groups of 16 latent columns of the output. The phases of a tile depend on one another, so
+// it takes many warps to hide their latencies.
 struct LatentParams {
   const void* q;                                           // [rows, H, pitch]
   const void* cache; int pitch, rank;
@@ -352,18 +353,19 @@ struct LatentParams {
   void* out;                                               // [rows, H, rot_at]
   int o_hd;
 };
+constexpr int LNT = 512, LNW = LNT / 32;
 constexpr int LKT = 64, LSP = LKT + 4, LPP = LKT + 8;      // keys a tile, score and weight row pitches
 template <int HT>
 struct LatentSmem {
-  static constexpr int ROWS = 16 * HT;
-  static constexpr int S = 0, P = S + 2 * ROWS * LSP * 4, A = P + 2 * ROWS * LPP * 2, SLOTS = A + 3 * ROWS * 4, Q = SLOTS + 2 * LKT * 4;
+  static constexpr int ROWS = 16 * HT, SIDES = 4 / HT;
+  static constexpr int S = 0, P = S + SIDES * ROWS * LSP * 4, A = P + 2 * ROWS * LPP * 2, SLOTS = A + 3 * ROWS * 4, Q = SLOTS + 2 * LKT * 4;
   static __host__ __device__ int bytes(int pitch) { return Q + (ROWS + 2 * LKT) * (pitch + 8) * 2; }
 };
 template <int HT, int W16>
-__global__ void __launch_bounds__(256) latent_decode_kernel(const LatentParams p, int splits, float* __restrict__ part_o,
+__global__ void __launch_bounds__(LNT) latent_decode_kernel(const LatentParams p, int splits, float* __restrict__ part_o,
                                                             float* __restrict__ part_ml) {
   using L = LatentSmem<HT>;
-  constexpr int ROWS = L::ROWS, TPR = 256 / ROWS, KPT = LKT / TPR;     // threads a row, keys a thread
+  constexpr int ROWS = L::ROWS, SIDES = L::SIDES, TPR = LNT / ROWS, KPT = LKT / TPR;     // threads a row, keys a thread
   extern __shared__ __align__(128) uint8_t smem[];
   float* sS = reinterpret_cast<float*>(smem + L::S);
   float* sA = reinterpret_cast<float*>(smem + L::A);       // alpha, then m, l
@@ -388,80 +390,76 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentParams p
     for (int i = 0; i < W16; ++i)
 #pragma unroll
       for (int x = 0; x < 8; ++x) o[t][i][x] = 0.f;
-  const int n16 = (p.rank + 15) >> 4, ksteps = p.pitch >> 4, khalf = (ksteps + 1) >> 1;
+  const int n16 = (p.rank + 15) >> 4, ksteps = p.pitch >> 4, kpart = (ksteps + SIDES - 1) / SIDES;
   if (jbeg < jend) {
-    auto tile_slots = [&](int it) {
-      if (threadIdx.x < LKT) {
-        const int j = min(jbeg + it * LKT + (int)threadIdx.x, jend - 1), blk = j / p.bs;
-        slots[(it & 1) * LKT + threadIdx.x] = tab[blk] * p.bs + j - blk * p.bs;
-      }
+    const int shift = (p.bs & (p.bs - 1)) ? -1 : 31 - __clz(p.bs);
+    // cache row of this thread's key of tile it: asked for two tiles ahead, so that the table's latency is not waited for
+    auto tile_slot = [&](int it) {
+      const int j = min(jbeg + it * LKT + (int)threadIdx.x, jend - 1), blk = shift < 0 ? j / p.bs : j >> shift;
+      return tab[blk] * p.bs + j - blk * p.bs;
     };
+    int next_slot = 0;
     auto load_tile = [&](int it) {
       const uint32_t dst = sK + (it & 1) * stage;
       const int j0 = jbeg + it * LKT;
-      for (int r = warp; r < LKT; r += 8) {
+      for (int r = warp; r < LKT; r += LNW) {
         const bf16* src = reinterpret_cast<const bf16*>(p.cache) + (long long)slots[(it & 1) * LKT + r] * p.pitch;
         for (int c = lane; c < pieces; c += 32) cp_async16(dst + r * kp + c * 16, src + c * 8, j0 + r < jend);
       }
       cp_async_commit();
     };
-    tile_slots(0);
+    if (threadIdx.x < LKT) {
+      slots[threadIdx.x] = tile_slot(0);
+      next_slot = tile_slot(1);
+    }
     __syncthreads();
     {
       const bf16* q = reinterpret_cast<const bf16*>(p.q) + (b * p.H + h0) * p.pitch;
-      for (int r = warp; r < ROWS; r += 8)
+      for (int r = warp; r < ROWS; r += LNW)
         for (int c = lane; c < pieces; c += 32) cp_async16(sQ + r * kp + c * 16, r < nh ? q + (long long)r * p.pitch + c * 8 : q, r < nh);
     }
     load_tile(0);
     const float sl2 = p.scale * LOG2E_F;
-    const int kb = (warp & 3) * 16, kside = warp >> 2;     // this warp's keys and columns in the score phase
+    // this warp's keys, heads and columns in the score phase
+    const int kb = (warp & 3) * 16, ht = (warp >> 2) % HT, kside = (warp >> 2) / HT;
     const int row = threadIdx.x / TPR, key0 = (threadIdx.x % TPR) * KPT;
     int it = 0;
     for (int j0 = jbeg; j0 < jend; j0 += LKT, ++it) {
       const bool more = j0 + LKT < jend;
-      if (more) tile_slots(it + 1);
+      if (threadIdx.x < LKT) slots[((it + 1) & 1) * LKT + threadIdx.x] = next_slot;
       cp_async_wait<0>();
       __syncthreads();                                     // tile it is there, everyone has finished with the other stage
       if (more) load_tile(it + 1);
+      if (threadIdx.x < LKT) next_slot = tile_slot(it + 2);
       const uint32_t kt = sK + (it & 1) * stage;
       {
-        float s[HT][2][4];
-#pragma unroll
-        for (int t = 0; t < HT; ++t)
-#pragma unroll
-          for (int x = 0; x < 4; ++x) s[t][0][x] = s[t][1][x] = 0.f;
-        const int k1 = kside ? ksteps : khalf;
+        float s[2][4] = {};
+        const int k1 = min(ksteps, (kside + 1) * kpart);
         const uint32_t ka = kt + (kb + (lane & 7) + ((lane >> 4) << 3)) * kp + ((lane >> 3) & 1) * 16;
-        const uint32_t qa = sQ + (lane & 15) * kp + (lane >> 4) * 16;
-#pragma unroll 4
-        for (int kk = kside ? khalf : 0; kk < k1; ++kk) {
-          uint32_t bb[4];
+        const uint32_t qa = sQ + (ht * 16 + (lane & 15)) * kp + (lane >> 4) * 16;
+#pragma unroll 3
+        for (int kk = kside * kpart; kk < k1; ++kk) {
+          uint32_t a[4], bb[4];
           ldsm4(bb, ka + kk * 32);
-#pragma unroll
-          for (int t = 0; t < HT; ++t) {
-            uint32_t a[4];
-            ldsm4(a, qa + t * 16 * kp + kk * 32);
-            mma_bf16(s[t][0], a, bb[0], bb[1]);
-            mma_bf16(s[t][1], a, bb[2], bb[3]);
-          }
+          ldsm4(a, qa + kk * 32);
+          mma_bf16(s[0], a, bb[0], bb[1]);
+          mma_bf16(s[1], a, bb[2], bb[3]);
         }
-        float* sp = sS + kside * ROWS * LSP;
+        float* sp = sS + (kside * ROWS + ht * 16 + (lane >> 2)) * LSP + kb + (lane & 3) * 2;
 #pragma unroll
-        for (int t = 0; t < HT; ++t)
+        for (int i = 0; i < 2; ++i)
 #pragma unroll
-          for (int i = 0; i < 2; ++i)
-#pragma unroll
-            for (int y = 0; y < 2; ++y)
-              *reinterpret_cast<float2*>(sp + (t * 16 + (lane >> 2) + 8 * y) * LSP + kb + i * 8 + (lane & 3) * 2) =
-                  make_float2(s[t][i][2 * y], s[t][i][2 * y + 1]);
+          for (int y = 0; y < 2; ++y) *reinterpret_cast<float2*>(sp + 8 * y * LSP + i * 8) = make_float2(s[i][2 * y], s[i][2 * y + 1]);
       }
       __syncthreads();
       {
         float v[KPT], mx = -INFINITY;
 #pragma unroll
         for (int i = 0; i < KPT; ++i) {
-          const float x = (sS[row * LSP + key0 + i] + sS[(ROWS + row) * LSP + key0 + i]) * sl2;
-          v[i] = j0 + key0 + i < jend ? x : -INFINITY;
+          float x = 0.f;
+#pragma unroll
+          for (int y = 0; y < SIDES; ++y) x += sS[(y * ROWS + row) * LSP + key0 + i];
+          v[i] = j0 + key0 + i < jend ? x * sl2 : -INFINITY;
           mx = fmaxf(mx, v[i]);
         }
 #pragma unroll
@@ -611,7 +609,7 @@ int launch_latent(const LatentParams& p, long long rows, int splits, float* ws, 
   if (smem > 227 * 1024) { dlti_set_error("latent_decode: cache rows too long for shared memory"); return DLTI_ERR_TOO_LARGE; }
   if (int rc = allow_smem(latent_decode_kernel<HT, W16>, smem, have)) return rc;
   float* ml = splits > 1 ? ws + rows * p.H * splits * p.o_hd : nullptr;
-  DLTI_CUDA_CHECK(dlti_launch_pdl(rows, latent_decode_kernel<HT, W16>, dim3(splits, (p.H + 16 * HT - 1) / (16 * HT), (unsigned)rows), dim3(256),
+  DLTI_CUDA_CHECK(dlti_launch_pdl(rows, latent_decode_kernel<HT, W16>, dim3(splits, (p.H + 16 * HT - 1) / (16 * HT), (unsigned)rows), dim3(LNT),
                                   (size_t)smem, st, p, splits, ws, ml));
   dlti_count_launch();
   if (splits > 1) {
@@ -704,7 +702,6 @@ DLTI_API int dlti_latent_decode(const void* q, const void* cache, int pitch, int
   if (rank > 512) { dlti_set_error("latent_decode: latents of up to 512 elements"); return DLTI_ERR_TOO_LARGE; }
   LatentParams p{q, cache, pitch, rank, tables, max_blocks, bs, ctx, rseq, pos, H, scale, sink, gate, out, o_hd};
   const bool two = heads_per_cta > 16;
-  if (rank <= 128) return two ? launch_latent<2, 1>(p, rows, splits, ws, st) : launch_latent<1, 1>(p, rows, splits, ws, st);
-  if (rank <= 256) return two ? launch_latent<2, 2>(p, rows, splits, ws, st) : launch_latent<1, 2>(p, rows, splits, ws, st);
-  return two ? launch_latent<2, 4>(p, rows, splits, ws, st) : launch_latent<1, 4>(p, rows, splits, ws, st);
+  if (rank <= 256) return two ? launch_latent<2, 1>(p, rows, splits, ws, st) : launch_latent<1, 1>(p, rows, splits, ws, st);
+  return two ? launch_latent<2, 2>(p, rows, splits, ws, st) : launch_latent<1, 2>(p, rows, splits, ws, st);
 }

@@ -277,6 +277,48 @@ __global__ void __launch_bounds__(512) gated_norm_vec_kernel(const T* __restrict
   }
 }
 
+// many small groups: a warp per group, eight groups a CTA
+template <typename T, bool GATE_FIRST, bool ACC, int VPT>
+__global__ void __launch_bounds__(256) gated_norm_warp_kernel(const T* __restrict__ y, long long y_ld, const void* __restrict__ gate,
+                                                              long long g_ld, const float* __restrict__ w, T* __restrict__ out,
+                                                              long long o_ld, int gs, int groups, long long total, float eps) {
+  griddep_wait();
+  griddep_launch();
+  const long long x = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (x >= total) return;
+  const long long t = x / groups;
+  const int c0 = (int)(x - t * groups) * gs, vec = gs >> 3, lane = threadIdx.x & 31;
+  const T* yr = y + t * y_ld;
+  const void* gr = reinterpret_cast<const uint8_t*>(gate) + t * g_ld * (ACC ? 4 : sizeof(T));
+  float v[VPT][8], g[VPT][8], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i)
+    if (lane + 32 * i < vec) {
+      take_n<T, false, 8>(yr, c0 + (lane + 32 * i) * 8, v[i]);
+      take_n<T, ACC, 8>(gr, c0 + (lane + 32 * i) * 8, g[i]);
+    }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i)
+    if (lane + 32 * i < vec)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float e = fast_sigmoid(g[i][j]);
+        if (GATE_FIRST) v[i][j] *= g[i][j] * e;
+        else g[i][j] = e;
+        ss += v[i][j] * v[i][j];
+      }
+  const float r = 1.f / sqrtf(warp_sum(ss) / (float)gs + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i)
+    if (lane + 32 * i < vec) {
+      float wv[8];
+      ld8(w + c0 + (lane + 32 * i) * 8, wv);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] *= r * wv[j] * (GATE_FIRST ? 1.f : g[i][j]);
+      put_n(out + t * o_ld + c0 + (lane + 32 * i) * 8, v[i]);
+    }
+}
+
 // Per-head norm + rotation of q and k, cache write of k and v, sigmoid of the head gates. One warp per (token, job):
 // jobs = H query heads, G key heads, G value heads, then one job for all head gates. A layer on another layer's keys
 // and values has no k / v jobs of its own; with a packed destination they copy the cached rows instead.
@@ -779,6 +821,17 @@ DLTI_API int dlti_gated_norm(const void* y, long long y_ld, const void* gate, lo
   if (dtype == DLTI_BF16 && gs % 8 == 0 && gs <= 8 * 512 * 4 && y_ld % 8 == 0 && g_ld % 8 == 0 && o_ld % 8 == 0 && groups <= 65535 &&
       ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
     using B = __nv_bfloat16;
+    if (groups > 1 && gs <= 512) {
+      auto kern = gate_first ? (acc ? (gs <= 256 ? gated_norm_warp_kernel<B, true, true, 1> : gated_norm_warp_kernel<B, true, true, 2>)
+                                    : (gs <= 256 ? gated_norm_warp_kernel<B, true, false, 1> : gated_norm_warp_kernel<B, true, false, 2>))
+                             : (acc ? (gs <= 256 ? gated_norm_warp_kernel<B, false, true, 1> : gated_norm_warp_kernel<B, false, true, 2>)
+                                    : (gs <= 256 ? gated_norm_warp_kernel<B, false, false, 1> : gated_norm_warp_kernel<B, false, false, 2>));
+      const long long total = rows * groups;
+      DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)((total + 7) / 8)), dim3(256), 0, st, (const B*)y, y_ld, gate, g_ld, w, (B*)out,
+                                      o_ld, gs, groups, total, eps));
+      dlti_count_launch();
+      return 0;
+    }
     const int vec = gs / 8, threads = vec <= 64 ? 64 : (vec <= 128 ? 128 : (vec <= 512 ? 256 : 512)), vpt = (vec + threads - 1) / threads;
 #define GNV(GF, AC) (vpt <= 1 ? gated_norm_vec_kernel<B, GF, AC, 1> : vpt <= 2 ? gated_norm_vec_kernel<B, GF, AC, 2> \
                      : gated_norm_vec_kernel<B, GF, AC, 4>)

@@ -67,7 +67,7 @@ def latent_decode(q, m: LatentAttentionMixer, rows: Rows, cache, gate, sink, out
     tile = 16 if m.heads <= 16 else 32
     if splits is None:
         reach = min(rows.max_ctx or 1 << 30, rows.tables.shape[1] * bs)
-        smem = tile * (68 * 8 + 72 * 4 + 12) + 512 + (tile + 128) * (m.pitch + 8) * 2
+        smem = 64 * 68 * 4 + tile * (72 * 4 + 12) + 512 + (tile + 128) * (m.pitch + 8) * 2
         room = 148 * max(1, min(2, 227 * 1024 // (smem + 1024)))
         splits = max(1, min(32, room // max(1, n * -(-m.heads // tile)), -(-reach // 64)))
     ws = _workspace(q.device, n * m.heads * splits * (o_hd + 2)) if splits > 1 else None
@@ -136,7 +136,7 @@ def expanded(buf, lat, m: LatentAttentionMixer, lw, w_expand, rows: Rows, cache,
         _lib.check(f(_p(lat), _p(cache), m.pitch, _p(pieces.prow), _p(pieces.pslot), pieces.prefix, _lib.stream_ptr()), "latent_rows")
     sink = lw.get("sink")
     if hp == PACKED_HD:
-        gemm(lat, w_expand, out=buf[:, H * hp:])
+        gemm(lat, w_expand, out=buf[:, H * hp:], two_cta=False)      # a short contraction: bound by the rows it writes
         attn_fwd_split(buf, m, H, H, pieces, gate, out, sink=sink)
         return out
     n = pieces.rows

@@ -339,7 +339,7 @@ def logozen_kernels(width: int, peaks: dict, nseq: int, length: int, batch: int,
     run("prefill", "attention (packed)", lambda: K.attn_fwd_split(buf, m, heads, heads, pieces, gate, out, sink=lw["sink"]),
         T * heads * (2 * m.qk_dim + 2 * m.vdim) * 2, 2.0 * nseq * pairs * heads * (m.qk_dim + m.vdim))
     useful = heads * (m.dim + m.vdim)
-    run("prefill", "GEMM latents -> keys, values", lambda: gemm(lat, w_expand, out=buf[:, heads * hp:]),
+    run("prefill", "GEMM latents -> keys, values", lambda: gemm(lat, w_expand, out=buf[:, heads * hp:], two_cta=False),
         2 * (T * m.pitch + w_expand.numel() + 2 * T * heads * hp), 2.0 * T * useful * R)
     qa, od = rnd(batch, heads * m.pitch), torch.empty(batch, heads * R, device=dev, dtype=bf)
     gd = torch.rand(batch, heads, device=dev)

@@ -409,7 +409,7 @@ def test_the_running_maximum_and_the_floor_matter():
 
 
 @pytest.mark.parametrize("device,dtype", MODES)
-@pytest.mark.parametrize("heads,vdim", [(3, 10), (4, 64), (1, 256), (5, 24)])
+@pytest.mark.parametrize("heads,vdim", [(3, 10), (4, 64), (1, 256), (5, 24), (2, 264), (2, 520)])
 def test_unit_heads_and_gate(device, dtype, heads, vdim):
     g, n = gen(vdim), heads * vdim
     y, z, w = rnd(g, 6, n), rnd(g, 6, n), rnd(g, n)
