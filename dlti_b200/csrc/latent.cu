@@ -9,8 +9,9 @@
 // Prompts take the expanded form instead: keys and values of all heads by one GEMM from the cached rows (an identity block
 // in its weight passes k_rot through), then ordinary causal attention (attention.cu, attention_paged.cu).
 //
-// A cache row is [c, zeros to a multiple of 16, k_rot, zeros to a multiple of 16]: rot_at = round16(rank) and
-// pitch = rot_at + round16(rot).
+// A cache row is [c, zeros to a multiple of 16, k_rot, zeros to a multiple of 16, 8 zeros]: rot_at = round16(rank) and
+// pitch = rot_at + round16(rot) + 8. The last 8 make the rows of a page lie in shared memory, copied in one piece, so that
+// ldmatrix reads eight of them without bank conflicts.
 #include "rows.cuh"
 #include "mma_sync.cuh"
 
@@ -338,11 +339,14 @@ __global__ void __launch_bounds__(128) head_gemm_any_kernel(const HeadGemmParams
   reinterpret_cast<T*>(p.out)[t * p.o_ld + (long long)h * p.o_hd + n] = Cvt<T>::from_f(acc);
 }
 
-// Absorbed attention, bf16. grid (splits, blocks of 16 HT heads, rows), 16 warps; row b belongs to sequence rseq[b] (null: b)
-// and sees its first min(pos[b] + 1, ctx) cached rows (pos null: all ctx). Per tile of 64 cached rows: a warp computes the
-// scores of 16 keys for 16 heads over one of 4 / HT parts of the row's columns, all threads form the softmax weights (hi + lo
-// bf16 terms), then a warp owns W16 groups of 16 latent columns of the output. The phases of a tile depend on one another, so
-// it takes many warps to hide their latencies.
+// Absorbed attention, bf16. grid (splits, blocks of 16 HT heads, rows); row b belongs to sequence rseq[b] (null: b) and sees its
+// first min(pos[b] + 1, ctx) cached rows (pos null: all ctx). Tiles of 32 cached rows go through three groups of warps that
+// work on different tiles at the same time:
+//   warp 16       copies the tile's rows from the pages, one bulk copy per page, `stages` tiles ahead
+//   warps 0-7     scores (a warp: 16 keys x 16 heads over one of 4 / HT parts of the row's columns), then the softmax weights
+//                 as hi + lo bf16 terms, two buffers
+//   warps 8-15    outputs: a warp owns W16 groups of 16 latent columns of all heads
+// Every wait is bounded: when one runs out the CTA gives up, and its outputs are NaN.
 struct LatentParams {
   const void* q;                                           // [rows, H, pitch]
   const void* cache; int pitch, rank;
@@ -353,137 +357,185 @@ struct LatentParams {
   void* out;                                               // [rows, H, rot_at]
   int o_hd;
 };
-constexpr int LNT = 512, LNW = LNT / 32;
-constexpr int LKT = 64, LSP = LKT + 4, LPP = LKT + 8;      // keys a tile, score and weight row pitches
+constexpr int LKT = 32, LSP = LKT + 4, LPP = LKT + 8;      // keys a tile, score and weight row pitches
+constexpr int LTHREADS = 17 * 32, LSTAGES = 6;             // most stages
+constexpr long long LWAIT = 4000000000LL;                  // ~2 s
 template <int HT>
 struct LatentSmem {
   static constexpr int ROWS = 16 * HT, SIDES = 4 / HT;
-  static constexpr int S = 0, P = S + SIDES * ROWS * LSP * 4, A = P + 2 * ROWS * LPP * 2, SLOTS = A + 3 * ROWS * 4, Q = SLOTS + 2 * LKT * 4;
-  static __host__ __device__ int bytes(int pitch) { return Q + (ROWS + 2 * LKT) * (pitch + 8) * 2; }
+  static constexpr int BARS = 0, ERR = BARS + (2 * LSTAGES + 4) * 8, S = ERR + 16;                // scores [2][SIDES][ROWS][LSP]
+  static constexpr int P = S + 2 * SIDES * ROWS * LSP * 4, A = P + 2 * 2 * ROWS * LPP * 2;        // weights [2][hi, lo][ROWS][LPP]
+  static constexpr int Q = A + 4 * ROWS * 4;                                                      // factors [2][ROWS], m, l
+  static __host__ __device__ int row(int pitch) { return pitch * 2; }
+  static __host__ __device__ int bytes(int pitch, int stages) { return Q + (ROWS + stages * LKT) * row(pitch); }
 };
 template <int HT, int W16>
-__global__ void __launch_bounds__(LNT) latent_decode_kernel(const LatentParams p, int splits, float* __restrict__ part_o,
-                                                            float* __restrict__ part_ml) {
+__global__ void __launch_bounds__(LTHREADS) latent_decode_kernel(const LatentParams p, int splits, int stages, float* __restrict__ part_o,
+                                                                float* __restrict__ part_ml) {
   using L = LatentSmem<HT>;
-  constexpr int ROWS = L::ROWS, SIDES = L::SIDES, TPR = LNT / ROWS, KPT = LKT / TPR;     // threads a row, keys a thread
+  constexpr int ROWS = L::ROWS, SIDES = L::SIDES, TPR = 256 / ROWS, KPT = LKT / TPR;       // softmax: threads a row, keys a thread
   extern __shared__ __align__(128) uint8_t smem[];
   float* sS = reinterpret_cast<float*>(smem + L::S);
-  float* sA = reinterpret_cast<float*>(smem + L::A);       // alpha, then m, l
-  int* slots = reinterpret_cast<int*>(smem + L::SLOTS);
+  float* sA = reinterpret_cast<float*>(smem + L::A);
+  volatile int* err = reinterpret_cast<volatile int*>(smem + L::ERR);
   const uint32_t sb = smem_u32(smem), sQ = sb + L::Q, sP = sb + L::P;
-  const int kp = (p.pitch + 8) * 2, stage = LKT * kp;      // bytes
+  const int kp = L::row(p.pitch), stage = LKT * kp;        // bytes
   const uint32_t sK = sQ + ROWS * kp;
+  const uint32_t full = sb + L::BARS, empty = full + 8 * LSTAGES, p_full = empty + 8 * LSTAGES, p_free = p_full + 16;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < stages; ++i) {
+      mbar_init(full + 8 * i, 1);
+      mbar_init(empty + 8 * i, 8);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(p_full + 8 * i, 8);
+      mbar_init(p_free + 8 * i, 8);
+    }
+    *err = 0;
+    mbar_fence_init();
+  }
   griddep_wait();
   griddep_launch();
-  const int split = blockIdx.x, h0 = blockIdx.y * ROWS, nh = min(ROWS, p.H - h0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  auto wait = [&](uint32_t bar, uint32_t parity) {
+    if (!mbar_try_wait(bar, parity)) {
+      const long long t0 = clock64();
+      while (!mbar_try_wait(bar, parity) && !*err)
+        if (clock64() - t0 > LWAIT) *err = 1;
+    }
+    __syncwarp();
+  };
+  const int split = blockIdx.x, h0 = blockIdx.y * ROWS, nh = min(ROWS, p.H - h0);
   const long long b = blockIdx.z;
   const int seq = p.rseq ? p.rseq[b] : (int)b;
   const int n = p.pos ? min(p.pos[b] + 1, p.ctx[seq]) : p.ctx[seq];
   const int tiles = (n + LKT - 1) / LKT, per = (tiles + splits - 1) / splits;
   const int jbeg = split * per * LKT, jend = min(n, jbeg + per * LKT);
-  const int* tab = p.tables + (long long)seq * p.max_blocks;
+  const int nt = jbeg < jend ? (jend - jbeg + LKT - 1) / LKT : 0;
+  const int n16 = (p.rank + 15) >> 4;
   const int pieces = p.pitch >> 3;
-  float o[HT][W16][8], m = -INFINITY, l = 0.f;             // m, l: of row threadIdx.x / TPR
+  if (nt > 0 && warp < 16) {
+    const bf16* q = reinterpret_cast<const bf16*>(p.q) + (b * p.H + h0) * p.pitch;
+    for (int r = warp; r < ROWS; r += 16)
+      for (int c = lane; c < pieces; c += 32) cp_async16(sQ + r * kp + c * 16, r < nh ? q + (long long)r * p.pitch + c * 8 : q, r < nh);
+    cp_async_commit();
+    cp_async_wait<0>();
+  }
+  __syncthreads();
+  float o[HT][W16][8];
 #pragma unroll
   for (int t = 0; t < HT; ++t)
 #pragma unroll
     for (int i = 0; i < W16; ++i)
 #pragma unroll
       for (int x = 0; x < 8; ++x) o[t][i][x] = 0.f;
-  const int n16 = (p.rank + 15) >> 4, ksteps = p.pitch >> 4, kpart = (ksteps + SIDES - 1) / SIDES;
-  if (jbeg < jend) {
+
+  if (warp == 16) {
+    // ---- copies: the lane of the first row of a page takes all its rows in the tile; rows past the end become zeros ----
+    const int* tab = p.tables + (long long)seq * p.max_blocks;
     const int shift = (p.bs & (p.bs - 1)) ? -1 : 31 - __clz(p.bs);
-    // cache row of this thread's key of tile it: asked for two tiles ahead, so that the table's latency is not waited for
-    auto tile_slot = [&](int it) {
-      const int j = min(jbeg + it * LKT + (int)threadIdx.x, jend - 1), blk = shift < 0 ? j / p.bs : j >> shift;
-      return tab[blk] * p.bs + j - blk * p.bs;
-    };
-    int next_slot = 0;
-    auto load_tile = [&](int it) {
-      const uint32_t dst = sK + (it & 1) * stage;
-      const int j0 = jbeg + it * LKT;
-      for (int r = warp; r < LKT; r += LNW) {
-        const bf16* src = reinterpret_cast<const bf16*>(p.cache) + (long long)slots[(it & 1) * LKT + r] * p.pitch;
-        for (int c = lane; c < pieces; c += 32) cp_async16(dst + r * kp + c * 16, src + c * 8, j0 + r < jend);
-      }
-      cp_async_commit();
-    };
-    if (threadIdx.x < LKT) {
-      slots[threadIdx.x] = tile_slot(0);
-      next_slot = tile_slot(1);
+    auto block_of = [&](int j) { return shift < 0 ? j / p.bs : j >> shift; };
+    auto entry = [&](int it) { return tab[block_of(min(jbeg + it * LKT + lane, n - 1))]; };
+    int page = nt > 0 ? entry(0) : 0;
+    for (int it = 0; it < nt; ++it) {
+      const int s = it % stages, j = jbeg + it * LKT + lane, rows = min(LKT, jend - (j - lane)), off = j - block_of(j) * p.bs;
+      const int next = entry(it + 1);                      // asked for one tile ahead
+      if (it >= stages) wait(empty + 8 * s, (it / stages - 1) & 1);
+      for (int i = lane; i < (LKT - rows) * pieces; i += 32)
+        *reinterpret_cast<uint4*>(smem + (sK - sb) + s * stage + rows * kp + i * 16) = make_uint4(0, 0, 0, 0);
+      __syncwarp();
+      if (lane == 0) mbar_expect_tx(full + 8 * s, rows * kp);
+      __syncwarp();
+      if (lane < rows && (lane == 0 || off == 0))
+        bulk_load_1d(sK + s * stage + lane * kp, reinterpret_cast<const bf16*>(p.cache) + ((long long)page * p.bs + off) * p.pitch,
+                     min(p.bs - off, rows - lane) * kp, full + 8 * s);
+      page = next;
     }
-    __syncthreads();
-    {
-      const bf16* q = reinterpret_cast<const bf16*>(p.q) + (b * p.H + h0) * p.pitch;
-      for (int r = warp; r < ROWS; r += LNW)
-        for (int c = lane; c < pieces; c += 32) cp_async16(sQ + r * kp + c * 16, r < nh ? q + (long long)r * p.pitch + c * 8 : q, r < nh);
-    }
-    load_tile(0);
-    const float sl2 = p.scale * LOG2E_F;
-    // this warp's keys, heads and columns in the score phase
-    const int kb = (warp & 3) * 16, ht = (warp >> 2) % HT, kside = (warp >> 2) / HT;
+  } else if (warp < 8) {
+    // ---- scores and weights ----
+    const int ksteps = (p.pitch - 8) >> 4, kpart = (ksteps + SIDES - 1) / SIDES;
+    const int kb = (warp & 1) * 16, ht = (warp >> 1) % HT, kside = (warp >> 1) / HT;
+    const int k0 = kside * kpart, k1 = min(ksteps, k0 + kpart);
     const int row = threadIdx.x / TPR, key0 = (threadIdx.x % TPR) * KPT;
-    int it = 0;
-    for (int j0 = jbeg; j0 < jend; j0 += LKT, ++it) {
-      const bool more = j0 + LKT < jend;
-      if (threadIdx.x < LKT) slots[((it + 1) & 1) * LKT + threadIdx.x] = next_slot;
-      cp_async_wait<0>();
-      __syncthreads();                                     // tile it is there, everyone has finished with the other stage
-      if (more) load_tile(it + 1);
-      if (threadIdx.x < LKT) next_slot = tile_slot(it + 2);
-      const uint32_t kt = sK + (it & 1) * stage;
-      {
-        float s[2][4] = {};
-        const int k1 = min(ksteps, (kside + 1) * kpart);
-        const uint32_t ka = kt + (kb + (lane & 7) + ((lane >> 4) << 3)) * kp + ((lane >> 3) & 1) * 16;
-        const uint32_t qa = sQ + (ht * 16 + (lane & 15)) * kp + (lane >> 4) * 16;
-#pragma unroll 3
-        for (int kk = kside * kpart; kk < k1; ++kk) {
+    const uint32_t qa = sQ + (ht * 16 + (lane & 15)) * kp + (lane >> 4) * 16;
+    const uint32_t ka = (kb + (lane & 7) + ((lane >> 4) << 3)) * kp + ((lane >> 3) & 1) * 16;
+    const float sl2 = p.scale * LOG2E_F;
+    float m = -INFINITY, l = 0.f;
+    for (int it = 0; it < nt; ++it) {
+      const int s = it % stages, j0 = jbeg + it * LKT, u = it & 1;
+      wait(full + 8 * s, (it / stages) & 1);
+      const uint32_t kt = sK + s * stage + ka;
+      float c[2][2][4] = {};                               // even and odd steps: two chains
+#pragma unroll 2
+      for (int kk = k0; kk + 1 < k1; kk += 2)
+#pragma unroll
+        for (int y = 0; y < 2; ++y) {
           uint32_t a[4], bb[4];
-          ldsm4(bb, ka + kk * 32);
-          ldsm4(a, qa + kk * 32);
-          mma_bf16(s[0], a, bb[0], bb[1]);
-          mma_bf16(s[1], a, bb[2], bb[3]);
+          ldsm4(bb, kt + (kk + y) * 32);
+          ldsm4(a, qa + (kk + y) * 32);
+          mma_bf16(c[y][0], a, bb[0], bb[1]);
+          mma_bf16(c[y][1], a, bb[2], bb[3]);
         }
-        float* sp = sS + (kside * ROWS + ht * 16 + (lane >> 2)) * LSP + kb + (lane & 3) * 2;
-#pragma unroll
-        for (int i = 0; i < 2; ++i)
-#pragma unroll
-          for (int y = 0; y < 2; ++y) *reinterpret_cast<float2*>(sp + 8 * y * LSP + i * 8) = make_float2(s[i][2 * y], s[i][2 * y + 1]);
+      if ((k1 - k0) & 1 && k1 > k0) {
+        uint32_t a[4], bb[4];
+        ldsm4(bb, kt + (k1 - 1) * 32);
+        ldsm4(a, qa + (k1 - 1) * 32);
+        mma_bf16(c[0][0], a, bb[0], bb[1]);
+        mma_bf16(c[0][1], a, bb[2], bb[3]);
       }
-      __syncthreads();
-      {
-        float v[KPT], mx = -INFINITY;
+      float* sp = sS + ((u * SIDES + kside) * ROWS + ht * 16 + (lane >> 2)) * LSP + kb + (lane & 3) * 2;
 #pragma unroll
-        for (int i = 0; i < KPT; ++i) {
-          float x = 0.f;
+      for (int i = 0; i < 2; ++i)
 #pragma unroll
-          for (int y = 0; y < SIDES; ++y) x += sS[(y * ROWS + row) * LSP + key0 + i];
-          v[i] = j0 + key0 + i < jend ? x * sl2 : -INFINITY;
-          mx = fmaxf(mx, v[i]);
-        }
+        for (int y = 0; y < 2; ++y)
+          *reinterpret_cast<float2*>(sp + 8 * y * LSP + i * 8) = make_float2(c[0][i][2 * y] + c[1][i][2 * y], c[0][i][2 * y + 1] + c[1][i][2 * y + 1]);
+      asm volatile("bar.sync 1, 256;" ::: "memory");       // scores of this tile are written; those of the last one have been read
+      float v[KPT], mx = -INFINITY;
 #pragma unroll
-        for (int d = TPR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
-        const float nm = fmaxf(m, mx);                     // finite: the tile has a visible key
-        const float alpha = ex2(m - nm);
-        m = nm;
-        l *= alpha;
-        if (threadIdx.x % TPR == 0) sA[row] = alpha;
-        bf16* pr = reinterpret_cast<bf16*>(smem + L::P) + row * LPP + key0;
+      for (int i = 0; i < KPT; ++i) {
+        float x = 0.f;
 #pragma unroll
-        for (int i = 0; i < KPT; i += 2) {
-          const float a = ex2(v[i] - nm), c = ex2(v[i + 1] - nm);
-          l += a + c;
-          uint32_t hi, lo;
-          split_pair(a, c, hi, lo);
-          *reinterpret_cast<uint32_t*>(pr + i) = hi;
-          *reinterpret_cast<uint32_t*>(pr + ROWS * LPP + i) = lo;
-        }
+        for (int y = 0; y < SIDES; ++y) x += sS[((u * SIDES + y) * ROWS + row) * LSP + key0 + i];
+        v[i] = j0 + key0 + i < jend ? x * sl2 : -INFINITY;
+        mx = fmaxf(mx, v[i]);
       }
-      __syncthreads();
+#pragma unroll
+      for (int d = TPR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+      const float nm = fmaxf(m, mx);                       // finite: the tile has a visible key
+      const float alpha = ex2(m - nm);
+      m = nm;
+      l *= alpha;
+      if (it >= 2) wait(p_free + 8 * u, ((it >> 1) - 1) & 1);
+      if (threadIdx.x % TPR == 0) sA[u * ROWS + row] = alpha;
+      bf16* pr = reinterpret_cast<bf16*>(smem + L::P) + (u * 2 * ROWS + row) * LPP + key0;
+#pragma unroll
+      for (int i = 0; i < KPT; i += 2) {
+        const float e0 = ex2(v[i] - nm), e1 = ex2(v[i + 1] - nm);
+        l += e0 + e1;
+        uint32_t hi, lo;
+        split_pair(e0, e1, hi, lo);
+        *reinterpret_cast<uint32_t*>(pr + i) = hi;
+        *reinterpret_cast<uint32_t*>(pr + ROWS * LPP + i) = lo;
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(p_full + 8 * u);
+    }
+#pragma unroll
+    for (int d = TPR / 2; d > 0; d >>= 1) l += __shfl_xor_sync(0xffffffffu, l, d);
+    if (threadIdx.x % TPR == 0) {
+      sA[2 * ROWS + row] = m;
+      sA[3 * ROWS + row] = l;
+    }
+  } else {
+    // ---- outputs ----
+    for (int it = 0; it < nt; ++it) {
+      const int s = it % stages, u = it & 1;
+      wait(full + 8 * s, (it / stages) & 1);
+      wait(p_full + 8 * u, (it >> 1) & 1);
+      const uint32_t vt = sK + s * stage + (lane & 15) * kp + (lane >> 4) * 16;
 #pragma unroll
       for (int t = 0; t < HT; ++t) {
-        const float a0 = sA[t * 16 + (lane >> 2)], a1 = sA[t * 16 + (lane >> 2) + 8];
+        const float a0 = sA[u * ROWS + t * 16 + (lane >> 2)], a1 = sA[u * ROWS + t * 16 + (lane >> 2) + 8];
 #pragma unroll
         for (int i = 0; i < W16; ++i)
 #pragma unroll
@@ -496,13 +548,13 @@ __global__ void __launch_bounds__(LNT) latent_decode_kernel(const LatentParams p
         for (int t = 0; t < HT; ++t)
 #pragma unroll
           for (int x = 0; x < 2; ++x)
-            ldsm4(w[t][x], sP + ((x * ROWS + t * 16 + (lane & 15)) * LPP + ks * 16 + (lane >> 4) * 8) * 2);
+            ldsm4(w[t][x], sP + (((u * 2 + x) * ROWS + t * 16 + (lane & 15)) * LPP + ks * 16 + (lane >> 4) * 8) * 2);
 #pragma unroll
         for (int i = 0; i < W16; ++i) {
-          const int c16 = warp * W16 + i;
+          const int c16 = (warp - 8) * W16 + i;
           if (c16 >= n16) break;                           // warp-uniform
           uint32_t bb[4];
-          ldsm4_t(bb, kt + (ks * 16 + (lane & 15)) * kp + (c16 * 16 + (lane >> 4) * 8) * 2);
+          ldsm4_t(bb, vt + ks * 16 * kp + c16 * 32);
 #pragma unroll
           for (int t = 0; t < HT; ++t)
 #pragma unroll
@@ -512,47 +564,46 @@ __global__ void __launch_bounds__(LNT) latent_decode_kernel(const LatentParams p
             }
         }
       }
+      __syncwarp();
+      if (lane == 0) {
+        mbar_arrive(p_free + 8 * u);
+        mbar_arrive(empty + 8 * s);
+      }
     }
-#pragma unroll
-    for (int d = TPR / 2; d > 0; d >>= 1) l += __shfl_xor_sync(0xffffffffu, l, d);
   }
-  // m, l to everyone. The row of 16-column group fragments: rows lane / 4 and lane / 4 + 8 of every m tile.
-  if (threadIdx.x % TPR == 0) {
-    const int r = threadIdx.x / TPR;
-    sA[ROWS + r] = m;
-    sA[2 * ROWS + r] = l;
-  }
-  __syncthreads();
+  __syncthreads();                                         // m and l are written
+  if (warp < 8 || warp == 16) return;
+  const float bad = *err ? __int_as_float(0x7fc00000) : 0.f;
 #pragma unroll
   for (int t = 0; t < HT; ++t)
 #pragma unroll
     for (int y = 0; y < 2; ++y) {
       const int r = t * 16 + (lane >> 2) + 8 * y, h = h0 + r;
       if (r >= nh) continue;
-      const float mr = sA[ROWS + r], lr = sA[2 * ROWS + r];
+      const float mr = sA[2 * ROWS + r], lr = sA[3 * ROWS + r] + bad;
       if (splits == 1) {
         const float d = p.sink ? lr + ex2(p.sink[h] * LOG2E_F - (mr == -INFINITY ? 0.f : mr)) : lr;
-        float f = d > 0.f ? 1.f / d : 0.f;
+        float f = d == 0.f ? 0.f : 1.f / d;
         if (p.gate) f *= p.gate[b * p.H + h];
         bf16* orow = reinterpret_cast<bf16*>(p.out) + (b * p.H + h) * p.o_hd;
 #pragma unroll
         for (int i = 0; i < W16; ++i) {
-          if (warp * W16 + i >= n16) break;
-          const int c = (warp * W16 + i) * 16 + (lane & 3) * 2;
+          const int c = ((warp - 8) * W16 + i) * 16 + (lane & 3) * 2;
+          if ((warp - 8) * W16 + i >= n16) break;
 #pragma unroll
           for (int x = 0; x < 2; ++x)
             *reinterpret_cast<__nv_bfloat162*>(orow + c + 8 * x) = __floats2bfloat162_rn(o[t][i][4 * x + 2 * y] * f, o[t][i][4 * x + 2 * y + 1] * f);
         }
       } else {
         const long long idx = (b * p.H + h) * splits + split;
-        if (warp == 0 && (lane & 3) == 0) {
+        if (warp == 8 && (lane & 3) == 0) {
           part_ml[idx * 2] = mr;
           part_ml[idx * 2 + 1] = lr;
         }
 #pragma unroll
         for (int i = 0; i < W16; ++i) {
-          if (warp * W16 + i >= n16) break;
-          const int c = (warp * W16 + i) * 16 + (lane & 3) * 2;
+          const int c = ((warp - 8) * W16 + i) * 16 + (lane & 3) * 2;
+          if ((warp - 8) * W16 + i >= n16) break;
 #pragma unroll
           for (int x = 0; x < 2; ++x)
             *reinterpret_cast<float2*>(part_o + idx * p.o_hd + c + 8 * x) = make_float2(o[t][i][4 * x + 2 * y], o[t][i][4 * x + 2 * y + 1]);
@@ -575,7 +626,7 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentParams 
     gl += ms == -INFINITY ? 0.f : part_ml[(base + s) * 2 + 1] * ex2(ms - gm);
   }
   if (p.sink) gl += ex2(p.sink[h] * LOG2E_F - (gm == -INFINITY ? 0.f : gm));
-  float f = gl > 0.f ? 1.f / gl : 0.f;
+  float f = gl == 0.f ? 0.f : 1.f / gl;
   if (p.gate) f *= p.gate[b * p.H + h];
   for (int c = threadIdx.x * 4; c < p.o_hd; c += 512) {
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -605,12 +656,14 @@ int allow_smem(K kernel, int bytes, int* have) {
 template <int HT, int W16>
 int launch_latent(const LatentParams& p, long long rows, int splits, float* ws, cudaStream_t st) {
   static int have[64] = {};
-  const int smem = LatentSmem<HT>::bytes(p.pitch);
+  int stages = LSTAGES;
+  while (stages > 2 && LatentSmem<HT>::bytes(p.pitch, stages) > 227 * 1024) --stages;
+  const int smem = LatentSmem<HT>::bytes(p.pitch, stages);
   if (smem > 227 * 1024) { dlti_set_error("latent_decode: cache rows too long for shared memory"); return DLTI_ERR_TOO_LARGE; }
   if (int rc = allow_smem(latent_decode_kernel<HT, W16>, smem, have)) return rc;
   float* ml = splits > 1 ? ws + rows * p.H * splits * p.o_hd : nullptr;
-  DLTI_CUDA_CHECK(dlti_launch_pdl(rows, latent_decode_kernel<HT, W16>, dim3(splits, (p.H + 16 * HT - 1) / (16 * HT), (unsigned)rows), dim3(LNT),
-                                  (size_t)smem, st, p, splits, ws, ml));
+  DLTI_CUDA_CHECK(dlti_launch_pdl(rows, latent_decode_kernel<HT, W16>, dim3(splits, (p.H + 16 * HT - 1) / (16 * HT), (unsigned)rows), dim3(LTHREADS),
+                                  (size_t)smem, st, p, splits, stages, ws, ml));
   dlti_count_launch();
   if (splits > 1) {
     DLTI_CUDA_CHECK(dlti_launch_pdl(rows, latent_combine_kernel, dim3(p.H, (unsigned)rows), dim3(128), 0, st, p, splits, (const float*)ws,
@@ -629,7 +682,7 @@ DLTI_API int dlti_latent_prep(const void* proj, long long ld, int oq, int od, in
                               void* cache, int pitch, int rot_at, int nabs, void* qn, int qn_hd, void* ql, void* qp, long long qp_ld, int qp_hd,
                               void* lat, const int* qdst, const int* dst, float* gate, long long tokens, int acc, int dtype, cudaStream_t st) {
   if (tokens <= 0) return 0;
-  if (H < 1 || dim < 1 || rot < 0 || rank < 1 || rd % 2 || rd > rot || rot_at < rank || pitch < rot_at + rot || (rd && (!cos_t || !sin_t)) ||
+  if (H < 1 || dim < 1 || rot < 0 || rank < 1 || rd % 2 || rd > rot || rot_at < rank || pitch < rot_at + rot || pitch % 8 || (rd && (!cos_t || !sin_t)) ||
       (nabs > 0 && (!qn || !ql)) || (nabs < tokens && (!qp || !lat)) || (og >= 0 && !gate)) return DLTI_ERR_BAD_ARG;
   if (acc && dtype != DLTI_BF16) return DLTI_ERR_UNSUPPORTED;
   PrepParams p{proj, ld, oq, od, og, H, dim, rot, rank, rd, interleaved, cos_t, sin_t, pos, kvw, eps, slots, cache, pitch, rot_at,
@@ -697,11 +750,12 @@ DLTI_API int dlti_latent_decode(const void* q, const void* cache, int pitch, int
                                 const int* rseq, const int* pos, long long rows, int H, float scale, const float* sink, const float* gate,
                                 int heads_per_cta, int splits, float* ws, void* out, int o_hd, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (H < 1 || rank < 1 || pitch % 16 || o_hd % 16 || o_hd < rank || rank > pitch || splits < 1 || rows > 65535 || (splits > 1 && !ws) ||
+  if (H < 1 || rank < 1 || pitch % 16 != 8 || o_hd % 16 || o_hd < rank || o_hd > pitch || splits < 1 || rows > 65535 || (splits > 1 && !ws) ||
       ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15)) return DLTI_ERR_BAD_ARG;
   if (rank > 512) { dlti_set_error("latent_decode: latents of up to 512 elements"); return DLTI_ERR_TOO_LARGE; }
   LatentParams p{q, cache, pitch, rank, tables, max_blocks, bs, ctx, rseq, pos, H, scale, sink, gate, out, o_hd};
   const bool two = heads_per_cta > 16;
-  if (rank <= 256) return two ? launch_latent<2, 1>(p, rows, splits, ws, st) : launch_latent<1, 1>(p, rows, splits, ws, st);
-  return two ? launch_latent<2, 2>(p, rows, splits, ws, st) : launch_latent<1, 2>(p, rows, splits, ws, st);
+  if (rank <= 128) return two ? launch_latent<2, 1>(p, rows, splits, ws, st) : launch_latent<1, 1>(p, rows, splits, ws, st);
+  if (rank <= 256) return two ? launch_latent<2, 2>(p, rows, splits, ws, st) : launch_latent<1, 2>(p, rows, splits, ws, st);
+  return two ? launch_latent<2, 4>(p, rows, splits, ws, st) : launch_latent<1, 4>(p, rows, splits, ws, st);
 }

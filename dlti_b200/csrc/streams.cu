@@ -331,8 +331,8 @@ __device__ __forceinline__ float3 block_sum3(float3 v, float* red) {
   __syncthreads();
   return make_float3(warp_sum(l < nw ? red[l] : 0.f), warp_sum(l < nw ? red[32 + l] : 0.f), warp_sum(l < nw ? red[64 + l] : 0.f));
 }
-template <typename T, bool ACC, int VPT>
-__global__ void __launch_bounds__(256) poly_norm_vec_kernel(const void* __restrict__ z, long long z_ld, const float* __restrict__ coef,
+template <typename T, bool ACC, int VPT, int NT>
+__global__ void __launch_bounds__(NT) poly_norm_vec_kernel(const void* __restrict__ z, long long z_ld, const float* __restrict__ coef,
                                                             T* __restrict__ out, long long o_ld, int n, float eps) {
   __shared__ float red[96];
   const float a = coef[0], b = coef[1], c = coef[2], e = coef[3];
@@ -469,9 +469,11 @@ DLTI_API int dlti_poly_norm(const void* z, long long z_ld, const float* coef, vo
   if (dtype == DLTI_BF16 && n % 8 == 0 && n <= 16384 && z_ld % 8 == 0 && o_ld % 8 == 0 &&
       ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
     using B = __nv_bfloat16;
-    const int vec = n / 8, vpt = vec <= 256 ? 1 : vec <= 512 ? 2 : vec <= 1024 ? 4 : 8, threads = ((vec + vpt - 1) / vpt + 31) / 32 * 32;
-#define PV(AC) (vpt == 1 ? poly_norm_vec_kernel<B, AC, 1> : vpt == 2 ? poly_norm_vec_kernel<B, AC, 2> \
-                : vpt == 4 ? poly_norm_vec_kernel<B, AC, 4> : poly_norm_vec_kernel<B, AC, 8>)
+    const int vec = n / 8, most = rows <= 256 ? 1024 : 256;          // few rows: all of a row's loads at once
+    const int vpt = vec <= most ? 1 : vec <= 2 * most ? 2 : vec <= 4 * most ? 4 : 8, threads = ((vec + vpt - 1) / vpt + 31) / 32 * 32;
+#define PV(AC) (most == 1024 ? (vpt == 1 ? poly_norm_vec_kernel<B, AC, 1, 1024> : poly_norm_vec_kernel<B, AC, 2, 1024>)   \
+                : vpt == 1 ? poly_norm_vec_kernel<B, AC, 1, 256> : vpt == 2 ? poly_norm_vec_kernel<B, AC, 2, 256>       \
+                : vpt == 4 ? poly_norm_vec_kernel<B, AC, 4, 256> : poly_norm_vec_kernel<B, AC, 8, 256>)
     auto kern = acc ? PV(true) : PV(false);
 #undef PV
     DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)rows), dim3(threads), 0, st, z, z_ld, coef, (B*)out, o_ld, n, eps));

@@ -91,12 +91,16 @@ class LatentAttentionMixer:
         return self.dim + self.rot_dim
 
     @property
-    def rot_at(self) -> int:       # a cache row is [latent, zeros, rotated part, zeros], both parts padded to 16
+    def rot_at(self) -> int:       # a cache row is [latent, zeros, rotated part, zeros], both parts padded to 16, ...
         return round16(self.kv_rank)
 
     @property
-    def pitch(self) -> int:
+    def cols(self) -> int:
         return self.rot_at + round16(self.rot_dim)
+
+    @property
+    def pitch(self) -> int:        # ... and 8 more: a page copied as it is into shared memory is read without bank conflicts
+        return self.cols + 8
 
     @property
     def head_pitch(self) -> int:
@@ -325,9 +329,9 @@ class StackWeights:
             if isinstance(m, LatentAttentionMixer) and self.device.type == "cuda" and self.dtype != torch.float32:
                 # cache row -> [keys | values] of all heads; an identity block hands the rotated part to every head's key
                 H, hp = m.heads, m.head_pitch
-                e = torch.zeros(2, H, hp, m.pitch, dtype=self.dtype, device=self.device)
+                e = torch.zeros(2, H, hp, m.cols, dtype=self.dtype, device=self.device)
                 e[0, :, :m.dim, :m.kv_rank] = w["w_uk"][:H * m.dim].view(H, m.dim, m.kv_rank)
                 e[0, :, m.dim:m.qk_dim, m.rot_at:m.rot_at + m.rot_dim] = torch.eye(m.rot_dim, dtype=self.dtype, device=self.device)
                 e[1, :, :m.vdim, :m.kv_rank] = w["w_uv"][:H * m.vdim].view(H, m.vdim, m.kv_rank)
-                self.derived[i]["w_expand"] = e.view(2 * H * hp, m.pitch)
+                self.derived[i]["w_expand"] = e.view(2 * H * hp, m.cols)
         return self

@@ -67,9 +67,8 @@ def latent_decode(q, m: LatentAttentionMixer, rows: Rows, cache, gate, sink, out
     tile = 16 if m.heads <= 16 else 32
     if splits is None:
         reach = min(rows.max_ctx or 1 << 30, rows.tables.shape[1] * bs)
-        smem = 64 * 68 * 4 + tile * (72 * 4 + 12) + 512 + (tile + 128) * (m.pitch + 8) * 2
-        room = 148 * max(1, min(2, 227 * 1024 // (smem + 1024)))
-        splits = max(1, min(32, room // max(1, n * -(-m.heads // tile)), -(-reach // 64)))
+        resident = 1 if m.pitch > 200 else 2                # CTAs of an SM (shared memory)
+        splits = max(1, min(32, 148 * resident // max(1, n * -(-m.heads // tile)), -(-reach // 64)))
     ws = _workspace(q.device, n * m.heads * splits * (o_hd + 2)) if splits > 1 else None
     f = _lib.fn("dlti_latent_decode", [_V, _V, _I, _I, _V, _I, _I, _V, _V, _V, _L, _I, _F, _V, _V, _I, _I, _V, _V, _I, _V])
     _lib.check(f(_p(q), _p(cache), m.pitch, m.kv_rank, _p(rows.tables), rows.tables.shape[1], bs, _p(rows.ctx),
@@ -134,7 +133,7 @@ def expanded(buf, lat, m: LatentAttentionMixer, lw, w_expand, rows: Rows, cache,
     if pieces.prefix:
         f = _lib.fn("dlti_latent_rows", [_V, _V, _I, _V, _V, _L, _V])
         _lib.check(f(_p(lat), _p(cache), m.pitch, _p(pieces.prow), _p(pieces.pslot), pieces.prefix, _lib.stream_ptr()), "latent_rows")
-    sink = lw.get("sink")
+    sink, lat = lw.get("sink"), lat[:, :m.cols]
     if hp == PACKED_HD:
         gemm(lat, w_expand, out=buf[:, H * hp:], two_cta=False)      # a short contraction: bound by the rows it writes
         attn_fwd_split(buf, m, H, H, pieces, gate, out, sink=sink)

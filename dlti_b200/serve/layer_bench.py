@@ -126,7 +126,7 @@ def step_bytes(eng: LLMEngine, batch: int, ctx: int) -> int:
         if eng.states is not None and eng.states.canon[i] is not None:
             n += 2 * batch * size(eng.states.canon[i][:, 0])
         if isinstance(m, LatentAttentionMixer):
-            n += 2 * batch * (ctx + 1) * m.pitch
+            n += 2 * batch * (ctx + 1) * m.cols
         elif isinstance(m, AttentionMixer):
             seen = ctx + 1 - (ctx // m.chunk * m.chunk if m.chunk else 0)
             n += 2 * batch * seen * m.kv_heads * (m.dim + m.vdim)
@@ -334,17 +334,17 @@ def logozen_kernels(width: int, peaks: dict, nseq: int, length: int, batch: int,
     pieces = K.Pieces(torch.tensor([i * length for i in range(nseq + 1)], dtype=torch.int32, device=dev), length, T)
     pairs = length * (length + 1) // 2
     hp = m.head_pitch
-    buf, gate, out, lat = rnd(T, 3 * heads * hp), torch.rand(T, heads, device=dev), K.act(T, heads * m.vdim, bf, dev), rnd(T, m.pitch)
+    buf, gate, out, lat = rnd(T, 3 * heads * hp), torch.rand(T, heads, device=dev), K.act(T, heads * m.vdim, bf, dev), rnd(T, m.pitch)[:, :m.cols]
     run = lambda phase, name, fn, nbytes, flops=0.0: k.run("logozen", phase, name, fn, nbytes, flops)
     run("prefill", "attention (packed)", lambda: K.attn_fwd_split(buf, m, heads, heads, pieces, gate, out, sink=lw["sink"]),
         T * heads * (2 * m.qk_dim + 2 * m.vdim) * 2, 2.0 * nseq * pairs * heads * (m.qk_dim + m.vdim))
     useful = heads * (m.dim + m.vdim)
     run("prefill", "GEMM latents -> keys, values", lambda: gemm(lat, w_expand, out=buf[:, heads * hp:], two_cta=False),
-        2 * (T * m.pitch + w_expand.numel() + 2 * T * heads * hp), 2.0 * T * useful * R)
+        2 * (T * m.cols + w_expand.numel() + 2 * T * heads * hp), 2.0 * T * useful * R)
     qa, od = rnd(batch, heads * m.pitch), torch.empty(batch, heads * R, device=dev, dtype=bf)
     gd = torch.rand(batch, heads, device=dev)
-    run("decode", "attention", lambda: LA.latent_decode(qa, m, dr, cache, gd, lw["sink"], od), batch * (ctx + 1) * m.pitch * 2,
-        2.0 * batch * (ctx + 1) * heads * (m.pitch + R))
+    run("decode", "attention", lambda: LA.latent_decode(qa, m, dr, cache, gd, lw["sink"], od), batch * (ctx + 1) * m.cols * 2,
+        2.0 * batch * (ctx + 1) * heads * (m.cols + R))
     qn, o = rnd(batch, heads * m.dim), torch.empty(batch, heads * m.vdim, device=dev, dtype=bf)
     run("decode", "queries into the latent space", lambda: LA.head_gemm(qn, m.dim, lw["w_uk"], qa, m.pitch, heads, m.dim, R, True),
         2 * (lw["w_uk"].numel() + qn.numel() + batch * heads * R))

@@ -446,7 +446,7 @@ int dlti_poly_norm(const void* z, long long z_ld, const float* coef, void* out, 
 /* accumulator columns [0, split) as dtype, the rest as fp32; the accumulator becomes zero */
 int dlti_split_rows(float* acc, void* out, long long o_ld, float* tail, long long t_ld, long long rows, int n, int split, int dtype,
     dlti_stream_t stream);
-/* latent.cu: latent attention. A cache row is [c, zeros, k_rot, zeros], rot_at = round16(rank), pitch = rot_at + round16(rot) */
+/* latent.cu: latent attention. A cache row is [c, zeros, k_rot, zeros], rot_at = round16(rank), pitch = rot_at + round16(rot) + 8 */
 int dlti_latent_prep(const void* proj, long long ld, int oq, int od, int og, int H, int dim, int rot, int rank, int rd, int interleaved,
     const float* cos_t, const float* sin_t, const int* pos, const float* kvw, float eps, const long long* slots, void* cache, int
     pitch, int rot_at, int nabs, void* qn, int qn_hd, void* ql, void* qp, long long qp_ld, int qp_hd, void* lat, const int* qdst, const int* dst,

@@ -631,7 +631,7 @@ def test_cache_holds_latents_and_states_only():
         att = isinstance(l.mixer, LatentAttentionMixer)
         assert (k is not None) == att and (ssm is None) == att and canon.shape[0] == (1 if l.mlp is None else 2)
         if att:
-            assert k.shape[2:] == (1, round16(l.mixer.kv_rank) + round16(l.mixer.rot_dim)) and v.numel() == 0
+            assert k.shape[2:] == (1, round16(l.mixer.kv_rank) + round16(l.mixer.rot_dim) + 8) and v.numel() == 0
 
 
 @pytest.mark.parametrize("device,dtype,t", WHOLE)
