@@ -319,7 +319,7 @@ def logozen_kernels(width: int, peaks: dict, nseq: int, length: int, batch: int,
     w = StackWeights(cfg, dev, bf).finish()
     lw, w_expand = w.layers[1], w.derived[1]["w_expand"]
     rnd = lambda *s: torch.randn(*s, device=dev, dtype=bf)
-    for t in (lw["w_uk"], lw["w_uv"], w_expand):
+    for t in (lw["w_uk"], lw["w_uv"], w_expand, *(l[n] for l in w.layers for n in ("w_in", "w_up"))):
         t.normal_(0, 0.04)
     T, bs, heads, R = nseq * length, 16, m.heads, m.kv_rank
     per = -(-max(length, ctx + 1) // bs)
