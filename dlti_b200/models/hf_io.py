@@ -54,9 +54,9 @@ class CheckpointReader:
     def get(self, name: str, rows: tuple[int, int] | None = None,
             cols: tuple[int, int] | None = None) -> torch.Tensor:
         """Whole tensor or a [rows, cols] slice (only those bytes are read)."""
-        sl = self._file(name).get_slice(name)
         if rows is None and cols is None:
-            return sl[:]
+            return self._file(name).get_tensor(name)
+        sl = self._file(name).get_slice(name)
         if len(sl.get_shape()) == 1:
             return sl[rows[0]:rows[1]]
         r = rows or (0, sl.get_shape()[0])

@@ -13,7 +13,7 @@ from typing import Callable
 import torch
 
 from . import config as llama_config
-from . import logozen, sigosun
+from . import latanex, logozen, sigosun
 
 
 @dataclass(frozen=True)
@@ -60,6 +60,10 @@ FAMILIES: dict[str, Family] = {
     logozen.ARCHITECTURE: Family(
         logozen.ARCHITECTURE, logozen.LogozenConfig, logozen.PRESETS, logozen.LogozenConfig.load, logozen.load_weights,
         lambda cfg, device, dtype, seed=0: logozen.from_state(cfg, logozen.random_state(cfg, seed, device), device, dtype),
+        _stack_runner, (torch.bfloat16, torch.float32)),
+    latanex.ARCHITECTURE: Family(
+        latanex.ARCHITECTURE, latanex.LatanexConfig, latanex.PRESETS, latanex.LatanexConfig.load, latanex.load_weights,
+        lambda cfg, device, dtype, seed=0: latanex.from_state(cfg, latanex.random_state(cfg, seed, device), device, dtype),
         _stack_runner, (torch.bfloat16, torch.float32)),
 }
 

@@ -1,7 +1,7 @@
 """Models described layer by layer: each layer names its token mixer (softmax attention, latent attention, Mamba-2,
-lightning attention, mLSTM) and its feed-forward, with every size and constant a parameter; the model names how sublayers
-meet the residual. A design (models/sigosun.py, models/logozen.py) is a parser from its config.json to a `StackConfig` plus
-its tensor names; the weights container, the cache layout and the serving forward pass (serve/stack_runner.py) are shared
+lightning attention, mLSTM, gated delta rule) and its feed-forward (dense or a mixture of experts), with every size and
+constant a parameter; the model names how sublayers meet the residual. A design (models/sigosun.py, models/logozen.py,
+models/latanex.py) is a parser from its config.json to a `StackConfig` plus its tensor names; the weights container, the cache layout and the serving forward pass (serve/stack_runner.py) are shared
 by all of them.
 
 Weights are kept as merged input projections, one GEMM per mixer. Every section of a merged projection and the row
@@ -43,6 +43,21 @@ class AttentionMixer:
     qk_norm: bool = True           # per-head RMS norm on q and k, before the rotation
     head_gate: bool = True         # each head's output times sigmoid of one projected number
     kv_from: int | None = None     # use the cached keys and values of this earlier layer
+    window: int = 0                # > 0: position i sees only itself and the window - 1 positions before it
+    softcap: float = 0.0           # > 0: scores become softcap * tanh(score / softcap)
+    sink: bool = False             # a learned term per head in the softmax denominator
+    bias: bool = False             # on the q, k and v projections
+    row_norm: bool = False         # RMS norm over all heads of q (and of k) at once
+    v_mix: bool = False            # values are mixed with those of the first such layer, by one learned share per layer
+
+    @property
+    def reach(self) -> tuple[int, int]:
+        return (self.chunk, self.window)
+
+    @property
+    def whole_rows(self) -> bool:
+        """Queries, keys and values are made from whole projection rows (ops.stack.qkv_rows), not head by head."""
+        return self.bias or self.row_norm or self.v_mix
 
 
 @dataclass(frozen=True)
@@ -84,7 +99,9 @@ class LatentAttentionMixer:
     sink: bool = True              # a learned term per head in the softmax denominator
     head_gate: bool = True
 
-    chunk = 0                      # every earlier position is seen
+    chunk = window = 0             # every earlier position is seen
+    reach = (0, 0)
+    softcap = 0.0
 
     @property
     def qk_dim(self) -> int:
@@ -120,15 +137,41 @@ class MLstmMixer:
 
 
 @dataclass(frozen=True)
+class DeltaMixer:
+    """Gated delta rule: a matrix per head that forgets by one factor and replaces, by a share, what it holds for a key. Short
+    convolutions on q, k and v, unit queries and keys shared by the heads of a group, a norm and a gate on the outputs."""
+    heads: int
+    kv_heads: int                  # query / key heads
+    dim: int
+    vdim: int
+    conv: int                      # taps of the causal convolutions
+
+
+@dataclass(frozen=True)
 class DenseMlp:
     ff: int
-    act: str = "relu2"             # square of relu; "polynorm": sum of the normed first three powers
+    act: str = "relu2"             # square of relu; "polynorm": sum of the normed first three powers; "swiglu": silu(gate) * up
+
+
+@dataclass(frozen=True)
+class MoeMlp:
+    """Mixture of clipped SwiGLU experts. The router's sigmoid scores pick `top` of them by score plus a correction, out of the
+    `keep` best of `groups` equal groups; the chosen scores, made to sum to `scale`, weigh the outputs."""
+    experts: int
+    top: int
+    ff: int
+    limit: float                   # gate <= limit, -limit <= up <= limit
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
+    shared_ff: int = 0             # > 0: one more expert of this size that runs for every token
+    shared_limit: float = 0.0
 
 
 @dataclass(frozen=True)
 class Layer:
-    mixer: AttentionMixer | LatentAttentionMixer | Mamba2Mixer | LightningMixer | MLstmMixer
-    mlp: DenseMlp | None = None
+    mixer: AttentionMixer | LatentAttentionMixer | Mamba2Mixer | LightningMixer | MLstmMixer | DeltaMixer
+    mlp: DenseMlp | MoeMlp | None = None
 
 
 @dataclass
@@ -142,7 +185,9 @@ class StackConfig:
     # sublayer (hyper-connections), a layer norm and a causal convolution of `canon` taps on its input
     streams: int = 0
     canon: int = 0
+    tanh_norms: bool = False       # one residual, a dynamic tanh norm before and after every sublayer instead
     embed_scale: float = 1.0
+    logit_scale: float = 1.0
     max_position_embeddings: int = 8192        # only a default for the server's max_model_len
     bos_token_id: int = 1
     eos_token_id: int = 2
@@ -162,6 +207,16 @@ class StackConfig:
                     if not isinstance(src, AttentionMixer) or src.kv_from is not None or \
                             (src.kv_heads, src.dim, src.vdim) != (m.kv_heads, m.dim, m.vdim):
                         raise ValueError(f"layer {i}: kv_from {m.kv_from} is not an earlier attention layer of the same shape")
+                if m.chunk and m.window:
+                    raise ValueError(f"layer {i}: attention is cut by a chunk or by a window, not by both")
+                if m.softcap < 0 or m.window < 0:
+                    raise ValueError(f"layer {i}: softcap {m.softcap} and window {m.window} must not be negative")
+                if m.whole_rows and (m.rope is not None or m.head_gate or m.kv_from is not None or m.qk_norm):
+                    raise ValueError(f"layer {i}: biases, row norms and value mixing do not combine with rotations, head gates, head "
+                                     "norms or shared keys")
+                src = self.v_mix_from(i)
+                if src is not None and (src.kv_heads, src.vdim) != (m.kv_heads, m.vdim):
+                    raise ValueError(f"layer {i}: values are mixed with those of a layer of another shape")
             elif isinstance(m, Mamba2Mixer):
                 if m.heads % m.groups or m.inner % m.norm_groups:
                     raise ValueError(f"layer {i}: groups must divide the heads and norm_groups the inner size")
@@ -171,8 +226,17 @@ class StackConfig:
             elif isinstance(m, MLstmMixer):
                 if not m.gate_cap > 0:
                     raise ValueError(f"layer {i}: gate_cap {m.gate_cap} must be positive")
+            elif isinstance(m, DeltaMixer):
+                if m.heads % m.kv_heads or m.conv < 1:
+                    raise ValueError(f"layer {i}: {m.heads} heads on {m.kv_heads} query/key heads, convolutions of {m.conv} taps")
             elif len(m.decay) != m.heads:
                 raise ValueError(f"layer {i}: {len(m.decay)} decays for {m.heads} heads")
+            e = l.mlp
+            if isinstance(e, MoeMlp):
+                if e.experts % e.groups or not 1 <= e.keep <= e.groups or not 1 <= e.top <= e.keep * (e.experts // e.groups):
+                    raise ValueError(f"layer {i}: {e.top} of {e.experts} experts from {e.keep} of {e.groups} groups")
+                if not self.tanh_norms:
+                    raise ValueError(f"layer {i}: mixtures of experts need the tanh norms, which add up their outputs")
         if self.streams and self.canon < 1:
             raise ValueError(f"canon taps {self.canon}: at least 1")
 
@@ -180,19 +244,20 @@ class StackConfig:
     def num_hidden_layers(self) -> int:
         return len(self.layers)
 
+    def v_mix_from(self, i: int) -> AttentionMixer | None:
+        """The layer whose values layer i mixes into its own (None: it mixes none, or is the first such layer itself)."""
+        mixing = [j for j, l in enumerate(self.layers[:i + 1]) if getattr(l.mixer, "v_mix", False)]
+        return self.layers[mixing[0]].mixer if len(mixing) > 1 and mixing[-1] == i else None
+
     @property
     def has_state(self) -> bool:
         """Some layer carries recurrent state (or earlier inputs of a convolution) from token to token."""
         return self.canon > 1 or any(not isinstance(l.mixer, (AttentionMixer, LatentAttentionMixer)) for l in self.layers)
 
     @property
-    def chunks(self) -> list[int]:
-        """The distinct attention chunk sizes, in order of first use (0 = unlimited)."""
-        out: list[int] = []
-        for l in self.layers:
-            if isinstance(l.mixer, (AttentionMixer, LatentAttentionMixer)) and l.mixer.chunk not in out:
-                out.append(l.mixer.chunk)
-        return out
+    def reaches(self) -> list[tuple[int, int]]:
+        """The distinct (chunk, window) limits of the attention layers, in order of first use (0 = unlimited)."""
+        return list(dict.fromkeys(l.mixer.reach for l in self.layers if isinstance(l.mixer, (AttentionMixer, LatentAttentionMixer))))
 
     @property
     def pack_prefix(self) -> int:
@@ -235,6 +300,8 @@ def mixer_sections(m) -> Sections:
         return Sections(z=m.inner, xbc=m.conv_channels, dt=m.heads)
     if isinstance(m, LatentAttentionMixer):
         return Sections(q=m.heads * m.qk_dim, dkv=m.kv_rank + m.rot_dim, **({"g": m.heads} if m.head_gate else {}))
+    if isinstance(m, DeltaMixer):                          # numbers that enter the decay and the step: products stay fp32
+        return Sections(q=m.kv_heads * m.dim, k=m.kv_heads * m.dim, v=m.heads * m.vdim, g=m.heads * m.vdim, gates=2 * m.heads)
     if isinstance(m, MLstmMixer):                          # the log gates come last: their products stay fp32
         return Sections(q=m.heads * m.dim, k=m.heads * m.dim, v=m.heads * m.vdim, g=m.heads * m.vdim, gates=2 * m.heads)
     return Sections(q=m.heads * m.dim, k=m.heads * m.dim, v=m.heads * m.vdim, g=m.heads * m.vdim)
@@ -242,6 +309,13 @@ def mixer_sections(m) -> Sections:
 
 def mixer_out(m) -> int:
     return m.heads * m.vdim
+
+
+def mlp_sections(e: DenseMlp | MoeMlp) -> Sections:
+    """Rows of a feed-forward's merged input projection (of an MoeMlp: its shared expert and, last, its router)."""
+    if isinstance(e, MoeMlp):
+        return Sections(**({"gate": e.shared_ff, "up": e.shared_ff} if e.shared_ff else {}), router=e.experts)
+    return Sections(gate=e.ff, up=e.ff) if e.act == "swiglu" else Sections(up=e.ff)
 
 
 class StackWeights:
@@ -263,6 +337,8 @@ class StackWeights:
         self.embed = torch.zeros(cfg.vocab_size, d, dtype=dtype, device=device)
         self.lm_head = mat(cfg.vocab_size, d)
         self.final_norm = vec(d)
+        if cfg.tanh_norms:
+            self.final_norm_b, self.final_norm_alpha = vec(d), vec(1)
         self.lora = None
         self.layers: list[dict] = []
         for l in cfg.layers:
@@ -273,6 +349,14 @@ class StackWeights:
                     w["q_norm"] = vec(m.dim)
                     if m.kv_from is None:
                         w["k_norm"] = vec(m.dim)
+                if m.row_norm:
+                    w |= {"q_norm": vec(m.heads * m.dim), "k_norm": vec(m.kv_heads * m.dim)}
+                if m.bias:
+                    w["b_in"] = vec(mixer_sections(m).total)
+                if m.sink:
+                    w["sink"] = vec(m.heads)
+                if m.v_mix:
+                    w["v_mix"] = vec(1)
             elif isinstance(m, Mamba2Mixer):
                 # convolution weights tap-major: one tap's channels are contiguous
                 w |= {"conv": torch.zeros(m.conv, round8(m.conv_channels), dtype=torch.float32, device=device),
@@ -284,13 +368,29 @@ class StackWeights:
                     w["sink"] = vec(m.heads)
             elif isinstance(m, MLstmMixer):
                 w |= {"gate_b": vec(2 * m.heads), "norm": vec(mixer_out(m))}
+            elif isinstance(m, DeltaMixer):
+                span = mixer_sections(m)["g"]              # the convolved sections, with the padding between them
+                w |= {"conv": torch.zeros(m.conv, span, dtype=torch.float32, device=device), "A_log": vec(m.heads), "dt_bias": vec(m.heads),
+                      "norm": vec(m.vdim)}
             else:
                 w |= {"decay": torch.tensor(m.decay, dtype=torch.float32).to(device),
                       "norm": vec(mixer_out(m))}
-            if l.mlp is not None:
-                w |= {"w_up": mat(l.mlp.ff, d), "w_down": mat(d, l.mlp.ff), "norm2": vec(d)}
-                if l.mlp.act == "polynorm":
+            e = l.mlp
+            if e is not None:
+                w |= {"w_up": mat(mlp_sections(e).total, d), "norm2": vec(d)}
+            if isinstance(e, MoeMlp):
+                def stack(rows, cols):
+                    return torch.zeros(e.experts, round8(rows), round8(cols), dtype=dtype, device=device)[:, :, :cols]
+                w |= {"correction": vec(e.experts), "e_up": stack(2 * round8(e.ff), d), "e_down": stack(d, e.ff)}
+                if e.shared_ff:
+                    w["w_down"] = mat(d, e.shared_ff)
+            elif e is not None:
+                w["w_down"] = mat(d, e.ff)
+                if e.act == "polynorm":
                     w["act"] = vec(4)
+            if cfg.tanh_norms:
+                w |= {k: t for q in ((1, 2) if e is not None else (1,)) for n in (f"norm{q}", f"norm{q}b")
+                      for k, t in ((n, vec(d)), (n + ".b", vec(d)), (n + ".alpha", vec(1)))}
             if cfg.streams:
                 for q in (1, 2) if l.mlp is not None else (1,):
                     w |= {f"hc{q}.in": vec(cfg.streams), f"hc{q}.out": vec(cfg.streams),
@@ -301,19 +401,27 @@ class StackWeights:
 
     def tensors(self):
         yield from (self.embed, self.lm_head, self.final_norm)
+        if self.cfg.tanh_norms:
+            yield from (self.final_norm_b, self.final_norm_alpha)
         for w in self.layers:
             yield from w.values()
 
-    def section(self, i: int, name: str) -> torch.Tensor:
-        """Rows of layer i's merged input projection that belong to `name`."""
+    def section(self, i: int, name: str, of: str = "w_in") -> torch.Tensor:
+        """Rows of layer i's merged input projection (of = "b_in": entries of its bias) that belong to `name`."""
         o, n = mixer_sections(self.cfg.layers[i].mixer).at[name]
-        return self.layers[i]["w_in"][o:o + n]
+        return self.layers[i][of][o:o + n]
+
+    def mlp_section(self, i: int, name: str) -> torch.Tensor:
+        """The same of its feed-forward's input projection."""
+        o, n = mlp_sections(self.cfg.layers[i].mlp).at[name]
+        return self.layers[i]["w_up"][o:o + n]
 
     def fill(self, named, get) -> "StackWeights":
         """Copy the checkpoint tensor get(name) to every (name, destination) of `named`; a list of destinations takes its
         rows one after the other."""
         for name, dst in named:
             src, parts = get(name), dst if isinstance(dst, list) else [dst]
+            src = src.reshape(1) if src.dim() == 0 else src              # single numbers
             if sum(p.shape[0] for p in parts) != src.shape[0] or src.shape[1:] != parts[0].shape[1:]:
                 raise ValueError(f"tensor {name} has shape {tuple(src.shape)}, which does not fit the configuration")
             o = 0
@@ -334,4 +442,7 @@ class StackWeights:
                 e[0, :, m.dim:m.qk_dim, m.rot_at:m.rot_at + m.rot_dim] = torch.eye(m.rot_dim, dtype=self.dtype, device=self.device)
                 e[1, :, :m.vdim, :m.kv_rank] = w["w_uv"][:H * m.vdim].view(H, m.vdim, m.kv_rank)
                 self.derived[i]["w_expand"] = e.view(2 * H * hp, m.cols)
+            elif isinstance(m, DeltaMixer):
+                self.derived[i]["norm"] = w["norm"].repeat(m.heads)
+                self.derived[i]["conv_b"] = torch.zeros(w["conv"].shape[1], dtype=torch.float32, device=self.device)
         return self

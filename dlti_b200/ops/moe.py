@@ -1,0 +1,143 @@
+"""Gated activations and mixtures of experts (csrc/moe.cu); PyTorch restatements for CPU tensors. Conventions as in ops/stack.py.
+
+A step's (token, choice) pairs are numbered token * top + choice. The router writes every expert's pairs as a list; the grouped
+GEMMs gather and scatter rows by these lists, so no permuted copy of the activations is made."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from ..models.stack import MoeMlp, mlp_sections, round8
+from . import _lib
+from .gemm import gemm_skinny_acc, gemm_swiglu
+from .stack import _F, _I, _L, _V, _p, act, linear
+
+LIMIT_OFF = 0.0              # limit of a plain SwiGLU: silu(g) * u without clipping
+
+
+@dataclass
+class ExpertSum:
+    """A feed-forward's output that is still to be added up: sum over k of weights[t, k] * rows[t * top + k], plus shared (None:
+    nothing). counts: the router's pair counters, which the consumer leaves zero."""
+    rows: torch.Tensor
+    weights: torch.Tensor
+    shared: torch.Tensor | None
+    counts: torch.Tensor | None = None
+
+    def value(self, d):
+        T, top = self.weights.shape
+        y = (self.rows[:, :d].float().view(T, top, d) * self.weights[:, :, None]).sum(1)
+        return y if self.shared is None else y + self.shared[:, :d].float()
+
+
+def _gated(g, u, limit):
+    if limit == LIMIT_OFF:
+        return torch.nn.functional.silu(g) * u
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return g * torch.sigmoid(1.702 * g) * (u + 1)
+
+
+def gated_act(p, og: int, ou: int, ff: int, limit: float, dtype, acc=False):
+    """Activation of the projection columns [og, og + ff) (gate) and [ou, ou + ff) (up): silu(g) u, or with a limit
+    g sigmoid(1.702 g) (u + 1) of the clipped values."""
+    if not _lib.use_native(p):
+        return _gated(p[:, og:og + ff].float(), p[:, ou:ou + ff].float(), limit).to(dtype)
+    h = act(p.shape[0], ff, dtype, p.device)
+    _route(p, None, 0, None, None, act_of=(og, ou, ff, limit, h), acc=acc)
+    return h
+
+
+def swiglu(h, w, ff: int, dtype, acc=False):
+    """silu(gate) * up of the merged projection w = [gate rows, up rows], each rounded up to 8."""
+    if h.is_cuda and not acc and dtype == torch.bfloat16 and ff % 128 == 0:
+        return gemm_swiglu(h, w)                       # activation in the GEMM for large steps
+    p = gemm_skinny_acc(h, w) if acc else linear(h, w)
+    return gated_act(p, 0, round8(ff), ff, LIMIT_OFF, dtype, acc=acc)
+
+
+_counters: dict = {}
+
+
+def _counts(device, n: int) -> torch.Tensor:
+    """Zero-on-entry pair counters: the op that adds the experts' outputs up leaves them zero again."""
+    key = (str(device), n)
+    if key not in _counters:
+        _counters[key] = torch.zeros(n, dtype=torch.int32, device=device)
+    return _counters[key]
+
+
+def _route(p, logits, col: int, correction, e: MoeMlp | None, act_of=None, acc=False, cap: int = 0):
+    """One launch: routing of the fp32 logits [T, >= col + experts] at column col, and / or the activation act_of = (gate column,
+    up column, ff, limit, destination) of the projection rows p. acc: both read the decode GEMM's accumulator and leave it zero."""
+    T = (p if p is not None else logits).shape[0]
+    dev = (p if p is not None else logits).device
+    wgt = lists = counts = None
+    if e is not None:
+        wgt = torch.empty((T, e.top), dtype=torch.float32, device=dev)
+        lists = torch.empty((e.experts, T), dtype=torch.int32, device=dev)
+        counts = _counts(dev, e.experts)
+    og, ou, ff, limit, h = act_of or (0, 0, 0, 0.0, None)
+    f = _lib.fn("dlti_moe_route", [_V, _L, _I, _V, _I, _I, _I, _I, _F, _V, _V, _V, _V, _L, _I, _I, _I, _F, _V, _L, _L, _I, _I, _V])
+    _lib.check(f(_p(logits), 0 if logits is None else logits.stride(0), col, _p(correction), e.experts if e else 0, e.top if e else 0,
+                 e.groups if e else 1, e.keep if e else 1, e.scale if e else 1.0, _p(wgt), _p(lists), _p(counts), _p(p) if h is not None else None,
+                 p.stride(0) if p is not None else 0, og, ou, ff, float(limit), _p(h), 0 if h is None else h.stride(0), T, int(acc),
+                 _lib.dtype_code(h.dtype) if h is not None else _lib.DT_BF16, _lib.stream_ptr()), "moe_route")
+    return wgt, lists, counts
+
+
+def route_ref(z, correction, e: MoeMlp):
+    """Router logits [T, experts] -> (chosen experts [T, top], weights [T, top])."""
+    s = torch.sigmoid(z)
+    c = s + correction
+    T, n = z.shape[0], e.experts // e.groups
+    if e.keep < e.groups:
+        best = c.view(T, e.groups, n).topk(min(2, n), -1).values.sum(-1).topk(e.keep, -1).indices
+        open_ = torch.zeros(T, e.groups, dtype=torch.bool).scatter_(1, best, True)
+        c = c.masked_fill(~open_.repeat_interleave(n, 1), float("-inf"))
+    idx = c.topk(e.top, -1).indices
+    w = s.gather(1, idx)
+    return idx, w / (w.sum(-1, keepdim=True) + 1e-20) * e.scale
+
+
+def grouped_gemm(x, w, lists, counts, out, *, rows: int, pairs_per_row: int, up: int = 0, limit: float = 0.0, max_rows: int = 0):
+    """out[pair, :rows] = x[pair // pairs_per_row] · w[e, :rows]^T for the pairs of every expert's list; w [E, rows, K]. up > 0: the
+    clipped activation of that product (gate) and the one with rows [up, up + rows) (up), in the kernel."""
+    E, K, T = w.shape[0], w.shape[2], lists.shape[1]
+    f = _lib.fn("dlti_moe_gemm", [_V, _L, _L, _I, _V, _L, _I, _I, _V, _V, _I, _I, _I, _I, _F, _V, _L, _I, _I, _V])
+    _lib.check(f(_p(x), x.stride(0), x.shape[0], pairs_per_row, _p(w), w.stride(1), w.stride(0) // w.stride(1), E, _p(lists), _p(counts), T,
+                 rows, up, K, float(limit), _p(out), out.stride(0), out.shape[0], _lib.dtype_code(x.dtype), _lib.stream_ptr()), "moe_gemm")
+    return out
+
+
+def moe(h, e: MoeMlp, lw, dtype, mm, acc=False) -> ExpertSum:
+    """Mixture of experts of the rows h; mm: the GEMM for the shared expert's output (its accumulator with acc)."""
+    T, d = h.shape
+    sec, ffr = mlp_sections(e), round8(e.ff)
+    og, ou = (sec["gate"], sec["up"]) if e.shared_ff else (0, 0)
+    if not _lib.use_native(h):
+        p = linear(h, lw["w_up"], out_dtype=torch.float32)
+        idx, wgt = route_ref(p[:, sec["router"]:sec["router"] + e.experts], lw["correction"], e)
+        rows = torch.zeros(T * e.top, d)
+        for j in range(e.experts):
+            pair = (idx.flatten() == j).nonzero()[:, 0]
+            if len(pair):
+                gu = h[pair // e.top].float() @ lw["e_up"][j].float().t()
+                a = _gated(gu[:, :e.ff], gu[:, ffr:ffr + e.ff], e.limit).to(dtype)
+                rows[pair] = a.float() @ lw["e_down"][j, :d].float().t()
+        shared = mm(gated_act(p, og, ou, e.shared_ff, e.shared_limit, dtype), lw["w_down"]) if e.shared_ff else None
+        return ExpertSum(rows.to(dtype), wgt, shared)
+    hs = act(T, e.shared_ff, dtype, h.device) if e.shared_ff else None
+    act_of = (og, ou, e.shared_ff, e.shared_limit, hs) if e.shared_ff else None
+    if acc:
+        p = gemm_skinny_acc(h, lw["w_up"])
+        wgt, lists, counts = _route(p, p, sec["router"], lw["correction"], e, act_of, acc=True)
+    else:
+        z = linear(h, lw["w_up"][sec["router"]:], out_dtype=torch.float32)
+        p = linear(h, lw["w_up"][:sec["router"]]) if e.shared_ff else None
+        wgt, lists, counts = _route(p, z, 0, lw["correction"], e, act_of)
+    a = act(T * e.top, e.ff, dtype, h.device)
+    grouped_gemm(h, lw["e_up"], lists, counts, a, rows=e.ff, pairs_per_row=e.top, up=ffr, limit=e.limit)
+    rows = act(T * e.top, d, dtype, h.device)
+    grouped_gemm(a, lw["e_down"], lists, counts, rows, rows=d, pairs_per_row=1)
+    return ExpertSum(rows, wgt, mm(hs, lw["w_down"]) if e.shared_ff else None, counts)

@@ -38,14 +38,17 @@ def linear(a: torch.Tensor, w: torch.Tensor, out_dtype=None) -> torch.Tensor:
     return gemm(a, w, out_dtype=out_dtype)
 
 
-def linear_f32(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-    """linear with an fp32 result (logits)."""
-    if not _lib.use_native(a) or a.dtype == torch.float32 or a.shape[0] > 256:
-        return linear(a, w, out_dtype=torch.float32)
+def linear_f32(a: torch.Tensor, w: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
+    """linear times scale with an fp32 result (logits)."""
+    if _lib.use_native(a) and a.dtype != torch.float32 and a.shape[0] > 256:
+        return gemm(a, w, out_dtype=torch.float32, alpha=scale)
+    if not _lib.use_native(a) or a.dtype == torch.float32:
+        y = linear(a, w, out_dtype=torch.float32)
+        return y if scale == 1.0 else y.mul_(scale)
     acc = gemm_skinny_acc(a, w)
     out = torch.empty_like(acc)
-    f = _lib.fn("dlti_take_rows", [_V, _V, _L, _I, _V])
-    _lib.check(f(_p(acc), _p(out), acc.shape[0], acc.shape[1], _lib.stream_ptr()), "take_rows")
+    f = _lib.fn("dlti_take_rows", [_V, _V, _F, _L, _I, _V])
+    _lib.check(f(_p(acc), _p(out), float(scale), acc.shape[0], acc.shape[1], _lib.stream_ptr()), "take_rows")
     return out
 
 
@@ -107,19 +110,19 @@ def relu2(u, ff, dtype, acc=False):
     return h
 
 
-def gated_norm(y, gate, w, eps, groups, gate_first, acc=False):
-    """gate_first: norm(y * silu(gate)) * w; else norm(y) * w * sigmoid(gate). The norm runs over `groups` equal parts of
-    the row. gate: [T, >= n] view (a section of a projection; of its accumulator with acc)."""
+def gated_norm(y, gate, w, eps, groups, gate_first, acc=False, silu=False):
+    """gate_first: norm(y * silu(gate)) * w; else norm(y) * w * sigmoid(gate), with silu: norm(y) * w * silu(gate). The norm runs
+    over `groups` equal parts of the row. gate: [T, >= n] view (a section of a projection; of its accumulator with acc)."""
     T, n = y.shape
     if not _lib.use_native(y):
         g = gate[:, :n].float()
         v = y.float() * torch.nn.functional.silu(g) if gate_first else y.float()
         v = _rms(v.reshape(T, groups, -1), eps).reshape(T, n) * w
-        return (v if gate_first else v * torch.sigmoid(g)).to(y.dtype)
+        return (v if gate_first else v * (torch.nn.functional.silu(g) if silu else torch.sigmoid(g))).to(y.dtype)
     out = act(T, n, y.dtype, y.device)
     f = _lib.fn("dlti_gated_norm", [_V, _L, _V, _L, _V, _V, _L, _L, _I, _I, _F, _I, _I, _I, _V])
     _lib.check(f(_p(y), y.stride(0), _p(gate), gate.stride(0), _p(w), _p(out), out.stride(0), T, n, groups, float(eps),
-                 int(gate_first), int(acc), _lib.dtype_code(y.dtype), _lib.stream_ptr()), "gated_norm")
+                 1 if gate_first else 2 if silu else 0, int(acc), _lib.dtype_code(y.dtype), _lib.stream_ptr()), "gated_norm")
     return out
 
 
@@ -170,9 +173,9 @@ class Rows:
 
 @dataclass
 class Pieces:
-    """The prompt rows of a step as independent causal sequences for one attention chunk size: a prompt is cut at every
-    chunk edge, and a portion that continues a chunk has the chunk's cached keys and values laid out in front of its own
-    rows. cu [n + 1]: boundaries in that extended layout; longest: its longest piece. With cached rows (prefix > 0): q0 [n]
+    """The prompt rows of a step as independent causal sequences for one kind of attention: a prompt is cut at every
+    chunk edge, and a portion that continues a chunk (or a window) has the cached keys and values that its rows can see laid
+    out in front of them. cu [n + 1]: boundaries in that extended layout; longest: its longest piece. With cached rows (prefix > 0): q0 [n]
     = cached rows of a piece, out0 [n] = prompt row of its first own row, dst [prompt rows] = extended row of each prompt
     row, prow / pslot [prefix] = extended row and cache slot of each cached token."""
     cu: torch.Tensor
@@ -242,13 +245,61 @@ def qk_norm_rope_cache(proj, sec, m, q_norm, k_norm, eps, rows: Rows, tabs, kc, 
                  _p(kp), _p(vp), _p(dst), rows.nd, _p(gate), T, H, G, m.dim, m.vdim, int(acc), _lib.dtype_code(dtype),
                  _lib.stream_ptr()), "qk_norm_rope_cache")
     if packed is not None and packed.prefix:
-        f = _lib.fn("dlti_prefix_rows", [_V, _L, _I, _V, _V, _V, _V, _I, _I, _I, _I, _L, _V])
-        _lib.check(f(_p(q[rows.nd:]), q.stride(0), hd, _p(packed.prow), _p(packed.pslot), _p(kc), _p(vc), kc.shape[3], vc.shape[3], H, G,
-                     packed.prefix, _lib.stream_ptr()), "prefix_rows")
+        prefix_rows(q[rows.nd:], m, packed, kc, vc)
     return q, gate
 
 
-def paged_attention_ref(q, m, rows: Rows, kc, vc, gate):
+def prefix_rows(buf, m, packed: Pieces, kc, vc):
+    """Cached keys and values in front of the portions of a step: packed prompt rows buf [rows, (H + 2 G) * 128]."""
+    f = _lib.fn("dlti_prefix_rows", [_V, _L, _I, _V, _V, _V, _V, _I, _I, _I, _I, _L, _V])
+    _lib.check(f(_p(buf), buf.stride(0), PACKED_HD, _p(packed.prow), _p(packed.pslot), _p(kc), _p(vc), kc.shape[3], vc.shape[3], m.heads,
+                 m.kv_heads, packed.prefix, _lib.stream_ptr()), "prefix_rows")
+
+
+def qkv_rows(proj, sec, m, lw, eps, rows: Rows, first, kc, vc, dtype, packed: Pieces | None = None, acc=False):
+    """Merged projection rows + bias -> queries and keys normed over the whole row (m.row_norm), values mixed with `first` [T, G *
+    vdim], the values of the first mixing layer (None: this layer mixes nothing in); keys and values go to the paged cache at
+    rows.slots. packed: as in qk_norm_rope_cache. Returns (queries or packed rows, values [T, G * vdim] before mixing, if they are
+    the first)."""
+    T, H, G = proj.shape[0], m.heads, m.kv_heads
+    _debug.check_range("qkv_rows", "slots", rows.slots, 0, kc.shape[0] * kc.shape[1], allow=-1)
+    b = lw.get("b_in")
+    qn, kn = (lw["q_norm"], lw["k_norm"]) if m.row_norm else (None, None)
+    keep = m.v_mix and first is None
+    if not _lib.use_native(proj):
+        p = proj.float() if b is None else proj.float() + b
+        q, k, v = (p[:, sec[s]:sec[s] + n] for s, n in (("q", H * m.dim), ("k", G * m.dim), ("v", G * m.vdim)))
+        if m.row_norm:
+            q, k = _rms(q, eps) * qn, _rms(k, eps) * kn
+        own = v.to(dtype)
+        if m.v_mix and not keep:
+            v = v + lw["v_mix"] * (first.float() - v)
+        ok = rows.slots >= 0
+        kc.view(-1, G, kc.shape[3])[rows.slots[ok], :, :m.dim] = k.reshape(T, G, m.dim).to(dtype)[ok]
+        vc.view(-1, G, vc.shape[3])[rows.slots[ok], :, :m.vdim] = v.reshape(T, G, m.vdim).to(dtype)[ok]
+        return q.to(dtype), own if keep else None
+    dev = proj.device
+    if packed is not None:
+        hd, n = PACKED_HD, rows.nd + packed.rows
+        q = (torch.empty if m.dim == m.vdim == hd else torch.zeros)((n, (H + 2 * G) * hd), dtype=dtype, device=dev)
+        kp, vp, dst = q[:, H * hd:], q[:, (H + G) * hd:], packed.dst
+    else:
+        hd, kp, vp, dst = round8(m.dim), None, None, None
+        q = torch.empty((T, H * hd), dtype=dtype, device=dev)
+    own = act(T, G * m.vdim, dtype, dev) if keep else None
+    mix = first if m.v_mix and not keep else None
+    f = _lib.fn("dlti_qkv_rows", [_V, _L, _I, _I, _I, _V, _V, _V, _F, _V, _L, _V, _V, _L, _V, _V, _V, _I, _I, _V, _L, _I, _V, _V, _V, _I, _L, _I,
+                                  _I, _I, _I, _I, _I, _V])
+    _lib.check(f(_p(proj), proj.stride(0), sec["q"], sec["k"], sec["v"], _p(b), _p(qn), _p(kn), float(eps), _p(mix), 0 if mix is None else
+                 mix.stride(0), _p(lw["v_mix"]) if mix is not None else None, _p(own), 0 if own is None else own.stride(0), _p(rows.slots), _p(kc),
+                 _p(vc), kc.shape[3], vc.shape[3], _p(q), q.stride(0), hd, _p(kp), _p(vp), _p(dst), rows.nd, T, H, G, m.dim, m.vdim, int(acc),
+                 _lib.dtype_code(dtype), _lib.stream_ptr()), "qkv_rows")
+    if packed is not None and packed.prefix:
+        prefix_rows(q[rows.nd:], m, packed, kc, vc)
+    return q, own
+
+
+def paged_attention_ref(q, m, rows: Rows, kc, vc, gate, sink=None):
     """Every row against the cached keys of its sequence that it may see."""
     T, H, G = q.shape[0], m.heads, m.kv_heads
     bs, hd = kc.shape[1], q.shape[1] // H
@@ -256,15 +307,20 @@ def paged_attention_ref(q, m, rows: Rows, kc, vc, gate):
     out = torch.zeros(T, H, m.vdim)
     for t in range(T):
         s, p = int(rows.seq[t]), int(rows.pos[t])
-        j = torch.arange(p // m.chunk * m.chunk if m.chunk else 0, min(p + 1, int(rows.ctx[s])))
+        lo = p // m.chunk * m.chunk if m.chunk else max(0, p - m.window + 1) if m.window else 0
+        j = torch.arange(lo, min(p + 1, int(rows.ctx[s])))
         if not len(j):
             continue
         sl = rows.tables[s, j // bs].long() * bs + j % bs
         k = kf[sl][..., :m.dim].repeat_interleave(H // G, 1)
         v = vf[sl][..., :m.vdim].repeat_interleave(H // G, 1)
         qq = q[t].float().view(H, hd)[:, :m.dim]
-        w = torch.softmax(torch.einsum("hd,jhd->hj", qq, k) * m.scale, -1)
-        out[t] = torch.einsum("hj,jhd->hd", w, v)
+        x = torch.einsum("hd,jhd->hj", qq, k) * m.scale
+        if m.softcap:
+            x = m.softcap * torch.tanh(x / m.softcap)
+        if sink is not None:
+            x = torch.cat([x, sink[:, None]], 1)
+        out[t] = torch.einsum("hj,jhd->hd", torch.softmax(x, -1)[:, :len(j)], v)
     if gate is not None:
         out *= gate[:, :, None]
     return out.reshape(T, -1).to(q.dtype)
@@ -273,10 +329,10 @@ def paged_attention_ref(q, m, rows: Rows, kc, vc, gate):
 def attn_rows(q, m, rows: Rows, kc, vc, gate, out, sink=None):
     """fp32-arithmetic attention of the rows of q, one warp per (row, head)."""
     hd = q.shape[1] // m.heads
-    f = _lib.fn("dlti_attn_rows", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _V, _I, _I, _I, _I, _I, _F, _V, _V, _V, _L, _L, _I, _V])
+    f = _lib.fn("dlti_attn_rows", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _V, _I, _I, _I, _I, _I, _I, _F, _F, _V, _V, _V, _L, _L, _I, _V])
     _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], kc.shape[1],
-                 _p(rows.ctx), _p(rows.seq), _p(rows.pos), m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.scale, _p(gate), _p(sink),
-                 _p(out), out.stride(0), q.shape[0], _lib.dtype_code(q.dtype), _lib.stream_ptr()), "attn_rows")
+                 _p(rows.ctx), _p(rows.seq), _p(rows.pos), m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.window, m.scale, m.softcap,
+                 _p(gate), _p(sink), _p(out), out.stride(0), q.shape[0], _lib.dtype_code(q.dtype), _lib.stream_ptr()), "attn_rows")
     return out
 
 
@@ -297,58 +353,59 @@ def attn_paged_decode(q, m, rows: Rows, kc, vc, gate, out, splits: int | None = 
     """Decode rows (bf16): row b of q against the visible keys of sequence b, split over CTAs."""
     B, hd, bs = q.shape[0], q.shape[1] // m.heads, kc.shape[1]
     if splits is None:
-        reach = min(rows.max_ctx or 1 << 30, m.chunk or 1 << 30, rows.tables.shape[1] * bs)
+        reach = min(rows.max_ctx or 1 << 30, m.chunk or m.window or 1 << 30, rows.tables.shape[1] * bs)
         ctas = max(1, B) * m.kv_heads * -(-(m.heads // m.kv_heads) // 16)
         splits = max(1, min(32, 3 * 148 // ctas, -(-reach // 64)))     # one wave of three CTAs per SM
     ws = _workspace(q.device, B * m.heads * splits * (m.vdim + 2)) if splits > 1 else None
-    f = _lib.fn("dlti_attn_paged_decode", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _I, _I, _I, _I, _I, _I, _F, _V, _V, _I, _V, _V, _L, _V])
+    f = _lib.fn("dlti_attn_paged_decode", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _I, _I, _I, _I, _I, _I, _I, _F, _F, _V, _V, _I, _V, _V, _L, _V])
     _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], bs,
-                 _p(rows.ctx), B, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.scale, _p(gate), _p(sink), splits, _p(ws), _p(out),
-                 out.stride(0), _lib.stream_ptr()), "attn_paged_decode")
+                 _p(rows.ctx), B, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.window, m.scale, m.softcap, _p(gate), _p(sink), splits, _p(ws),
+                 _p(out), out.stride(0), _lib.stream_ptr()), "attn_paged_decode")
     return out
 
 
 def attn_paged_prefill(q, m, rows: Rows, kc, vc, gate, out, sink=None):
     """Prompt rows (bf16): q, gate and out cover all rows of the step."""
     hd = q.shape[1] // m.heads
-    f = _lib.fn("dlti_attn_paged_prefill", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _F, _V, _V,
+    f = _lib.fn("dlti_attn_paged_prefill", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _V, _V,
                                             _V, _L, _V])
     _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], kc.shape[1],
                  _p(rows.ctx), _p(rows.cu), rows.nd, rows.nseq - rows.nd, rows.max_seqlen, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk,
-                 m.scale, _p(gate), _p(sink), _p(out), out.stride(0), _lib.stream_ptr()), "attn_paged_prefill")
+                 m.window, m.scale, m.softcap, _p(gate), _p(sink), _p(out), out.stride(0), _lib.stream_ptr()), "attn_paged_prefill")
     return out
 
 
-def packed_attention(qkv, m, rows: Rows, pieces: Pieces, kc, vc, gate):
-    """Attention of a step from the packed rows of qk_norm_rope_cache: decode rows through the pages, prompt rows through the
+def packed_attention(qkv, m, rows: Rows, pieces: Pieces, kc, vc, gate, sink=None):
+    """Attention of a step from the packed rows of qk_norm_rope_cache or qkv_rows: decode rows through the pages, prompt rows through the
     varlen tcgen05 kernel. Needs heads of up to 128 dimensions, values in multiples of 8."""
     T, H, nd = rows.pos.numel(), m.heads, rows.nd
     out = act(T, H * m.vdim, qkv.dtype, qkv.device)
     if nd:
-        attn_paged_decode(qkv[:nd, :H * PACKED_HD], m, rows, kc, vc, gate, out)
-    attn_fwd_split(qkv[nd:], m, H, m.kv_heads, pieces, None if gate is None else gate[nd:], out[nd:])
+        attn_paged_decode(qkv[:nd, :H * PACKED_HD], m, rows, kc, vc, gate, out, sink=sink)
+    attn_fwd_split(qkv[nd:], m, H, m.kv_heads, pieces, None if gate is None else gate[nd:], out[nd:], sink=sink)
     return out
 
 
 def attn_fwd_split(qkv, m, heads, kv_heads, pieces: Pieces, gate, out, sink=None):
     """Causal attention of packed rows [q heads | k heads | v heads], each 128 columns, within every piece."""
-    f = _lib.fn("dlti_attn_fwd_split", [_V, _V, _L, _V, _V, _V, _V, _V, _I, _I, _L, _I, _I, _I, _F, _V])
+    f = _lib.fn("dlti_attn_fwd_split", [_V, _V, _L, _V, _V, _V, _V, _V, _I, _I, _L, _I, _I, _I, _I, _F, _F, _V])
     _lib.check(f(_p(qkv), _p(out), out.stride(0), _p(gate), _p(sink), _p(pieces.cu), _p(pieces.q0), _p(pieces.out0), pieces.cu.numel() - 1,
-                 pieces.longest, qkv.shape[0], heads, kv_heads, m.vdim, m.scale, _lib.stream_ptr()), "attn_fwd_split")
+                 pieces.longest, qkv.shape[0], heads, kv_heads, m.vdim, m.window, m.scale, m.softcap, _lib.stream_ptr()),
+               "attn_fwd_split")
 
 
-def paged_attention(q, m, rows: Rows, kc, vc, gate):
+def paged_attention(q, m, rows: Rows, kc, vc, gate, sink=None):
     """Attention of every row of a step over the paged cache -> [T, heads * vdim], head outputs times `gate` [T, H]."""
     if not _lib.use_native(q):
-        return paged_attention_ref(q, m, rows, kc, vc, gate)
+        return paged_attention_ref(q, m, rows, kc, vc, gate, sink)
     _debug.check_paged("paged_attention", rows.tables, rows.ctx, kc.shape[0], kc.shape[1])
     out = act(q.shape[0], m.heads * m.vdim, q.dtype, q.device)
     if q.dtype == torch.float32 or max(kc.shape[3], vc.shape[3]) > 256:
-        return attn_rows(q, m, rows, kc, vc, gate, out)
+        return attn_rows(q, m, rows, kc, vc, gate, out, sink=sink)
     if rows.nd:
-        attn_paged_decode(q[:rows.nd], m, rows, kc, vc, gate, out)
+        attn_paged_decode(q[:rows.nd], m, rows, kc, vc, gate, out, sink=sink)
     if rows.nseq > rows.nd:
-        attn_paged_prefill(q, m, rows, kc, vc, gate, out)
+        attn_paged_prefill(q, m, rows, kc, vc, gate, out, sink=sink)
     return out
 
 

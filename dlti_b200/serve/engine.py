@@ -39,7 +39,7 @@ class StepLayout:
     a prefix copy carries everything but unused table rows.
 
     `full` (runners with per_sequence = True): ctx, tables and the recurrent-state slots sslot cover the prompts
-    too, rseq[T] names each row's sequence, and segs holds chunk_pieces of every attention chunk size (nsg entries)."""
+    too, rseq[T] names each row's sequence, and segs holds chunk_pieces of every kind of attention (nsg entries)."""
     _I64 = ("ids", "slots", "last", "seeds", "pslots", "pdst", "csrc")
     _I32 = ("pos", "src", "ctx", "cu", "ecu", "sslot", "rseq", "segs", "topk", "temp", "topp", "tables")
 
@@ -85,15 +85,15 @@ class StepLayout:
 PACK_FROM = 64               # longest piece of a step's prompts from which they are laid out for the varlen prefill kernel
 
 
-def chunk_pieces(cu, starts, tables, bs: int, chunk: int, pack_prefix: int = 4):
+def chunk_pieces(cu, starts, tables, bs: int, chunk: int, pack_prefix: int = 4, window: int = 0):
     """The prompt rows of a step cut where their positions reach a multiple of `chunk` (0: not at all), for
-    ops.stack.Pieces. Returns (int32 array [cu | q0 | out0 | dst | prow | pslot] (only cu without cached rows), pieces,
+    ops.stack.Pieces; with a window, a portion's cached rows are those that its first row sees. Returns (int32 array [cu | q0 | out0 | dst | prow | pslot] (only cu without cached rows), pieces,
     longest piece, extended rows, cached rows), or None when the pieces are too short or there are more than pack_prefix
     cached rows per prompt row."""
     cue, q0, out0, dst, prow, pslot, longest, own = [0], [], [], [], [], [], 0, 0
     for i, a in enumerate(starts):
         n = cu[i + 1] - cu[i]
-        lo = a // chunk * chunk if chunk else 0              # first position the first piece sees
+        lo = a // chunk * chunk if chunk else max(0, a - window + 1) if window else 0      # first position the first piece sees
         p, end = a, a + n
         while p < end:
             e = min(end, lo + chunk) if chunk else end
@@ -120,7 +120,7 @@ class PackedStep:
 
     def __init__(self, layout: StepLayout, slot, max_seqlen: int, max_ext: int = 0, segs: dict | None = None):
         self.layout, self.slot, self.max_seqlen, self.want_lp, self.max_ext = layout, slot, max_seqlen, False, max_ext
-        self.segs = segs or {}       # attention chunk size -> (offset in the segs section, then as chunk_pieces)
+        self.segs = segs or {}       # (attention chunk size, window) -> (offset in the segs section, then as chunk_pieces)
 
 
 def _pieces(s, n_rows: int, n: int, longest: int, rows: int, prefix: int):
@@ -280,10 +280,10 @@ class LLMEngine:
         full = self.per_sequence
         segs, seg_at, nsg = [], {}, 0
         if full and npf:
-            for c in self.cfg.chunks:
-                pc = chunk_pieces(cu, starts, tables[nd:], self.blocks.block_size, c, self.cfg.pack_prefix)
+            for reach in self.cfg.reaches:
+                pc = chunk_pieces(cu, starts, tables[nd:], self.blocks.block_size, reach[0], self.cfg.pack_prefix, reach[1])
                 if pc is not None:
-                    seg_at[c] = (nsg, *pc[1:])
+                    seg_at[reach] = (nsg, *pc[1:])
                     segs.append(pc[0])
                     nsg += len(pc[0])
         ns = npf if sampled_prompts is None else sampled_prompts

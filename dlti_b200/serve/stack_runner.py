@@ -10,10 +10,13 @@ import os
 
 import torch
 
-from ..models.stack import (AttentionMixer, LatentAttentionMixer, LightningMixer, Mamba2Mixer, MLstmMixer, StackConfig, StackWeights,
-                            mixer_sections, round8)
+from ..models.stack import (AttentionMixer, DeltaMixer, LatentAttentionMixer, LightningMixer, Mamba2Mixer, MLstmMixer, MoeMlp, StackConfig,
+                            StackWeights, mixer_sections, round8)
 from ..ops import _lib
+from ..ops import delta as D
+from ..ops import dyt as N
 from ..ops import latent as LA
+from ..ops import moe as M
 from ..ops import stack as K
 from ..ops import streams as H
 from ..ops.gemm import gemm_relu2, gemm_skinny_acc
@@ -80,6 +83,30 @@ class HyperStreams:
         return H.hyper_(self.x, None, None, None, None, self.run.w.final_norm, self.run.cfg.norm_eps, self.run.dtype, idx=idx)
 
 
+class TanhNorms:
+    """One fp32 residual, a dynamic tanh norm before and after every sublayer (ops/dyt.py): one elementwise kernel between two
+    sublayers, which also adds up the outputs of a mixture of experts."""
+
+    def __init__(self, run: "StackRunner", ids, rows: K.Rows, first, acc: bool):
+        self.run, self.acc = run, acc
+        self.x, self.h = N.embed_tanh(ids, run.w.embed, run.cfg.embed_scale, self._norm(first), run.dtype)
+
+    @staticmethod
+    def _norm(part, after=""):
+        lw, name = part[0], f"norm{part[1]}{after}"
+        return lw[name + ".alpha"], lw[name], lw[name + ".b"]
+
+    def step(self, y, done, then):
+        return N.tanh_between_(self.x, y, self._norm(done, "b"), None if then is None else self._norm(then), self.run.dtype, acc=self.acc)
+
+    def residual(self):
+        return self.x.clone()
+
+    def final(self, idx):
+        w = self.run.w
+        return N.tanh_rows(self.x, idx, (w.final_norm_alpha, w.final_norm, w.final_norm_b), self.run.dtype)
+
+
 class StackRunner:
     per_sequence = True
 
@@ -98,6 +125,8 @@ class StackRunner:
                 state = dict(heads=m.heads, rows=m.state, cols=m.vdim, conv_rows=m.conv - 1, conv_channels=m.conv_channels if m.conv > 1 else 0)
             elif isinstance(m, LightningMixer):
                 state = dict(heads=m.heads, rows=m.dim, cols=m.vdim)
+            elif isinstance(m, DeltaMixer):
+                state = dict(heads=m.heads, rows=m.dim, cols=m.vdim, conv_rows=m.conv - 1, conv_channels=mixer_sections(m)["g"] if m.conv > 1 else 0)
             elif isinstance(m, MLstmMixer):
                 state = dict(heads=m.heads, rows=m.dim, cols=m.vdim, vec=K.mlstm_vec(m.dim, m.vdim))
             if cfg.streams:
@@ -117,14 +146,14 @@ class StackRunner:
         self.pack_prompts = True     # False: all prompt attention reads the pages
         self.trace = None            # set to a list: receives the residual after every layer (debugging)
         self.mixers = {AttentionMixer: self._attention, LatentAttentionMixer: self._latent, Mamba2Mixer: self._mamba2,
-                       LightningMixer: self._lightning, MLstmMixer: self._mlstm}
+                       LightningMixer: self._lightning, MLstmMixer: self._mlstm, DeltaMixer: self._delta}
         # the sublayers in order: (layer weights, 1 mixer | 2 feed-forward, layer)
         self.parts = [(lw, q, i) for i, (l, lw) in enumerate(zip(cfg.layers, weights.layers)) for q in ((1, 2) if l.mlp is not None else (1,))]
 
     @torch.no_grad()
     def forward(self, input_ids, positions, slots, *, num_decode: int = 0, block_tables=None, ctx_lens=None, cu_seqlens=None,
                 max_seqlen: int = 0, last_idx=None, max_ctx: int = 0, state_slots=None, row_seq=None, segs=None) -> torch.Tensor:
-        """One pass over T token rows (see ops.stack.Rows for the arguments). segs: attention chunk size ->
+        """One pass over T token rows (see ops.stack.Rows for the arguments). segs: (attention chunk size, window) ->
         ops.stack.Pieces of the prompt rows (none: prompt attention reads the pages). Returns fp32 logits of the rows `last_idx`."""
         cfg, w = self.cfg, self.w
         rows = K.Rows(positions, row_seq, slots, ctx_lens, cu_seqlens, block_tables, state_slots, int(num_decode), max_seqlen,
@@ -133,27 +162,34 @@ class StackRunner:
         # decode-sized steps stream the weights through the stream-K GEMM; the next op consumes its fp32 accumulator
         self.acc = _FUSE_ACC and w.embed.is_cuda and self.dtype == torch.bfloat16 and ids.numel() <= 256
         mm = gemm_skinny_acc if self.acc else K.linear
-        res = (HyperStreams if cfg.streams else OutputNorms)(self, ids, rows, self.parts[0], self.acc)
+        res = (HyperStreams if cfg.streams else TanhNorms if cfg.tanh_norms else OutputNorms)(self, ids, rows, self.parts[0], self.acc)
         h = res.h
+        self.first_v = None          # values of the first layer that mixes values
         for part, then in zip(self.parts, self.parts[1:] + [None]):
             lw, q, i = part
             m = cfg.layers[i].mixer
             if q == 1:
                 y = mm(self.mixers[type(m)](i, m, lw, h, rows, segs), lw["w_out"])
             else:
-                y = mm(self._mlp(cfg.layers[i].mlp, lw, h, mm), lw["w_down"])
+                y = self._mlp(cfg.layers[i].mlp, lw, h, mm)
             h = res.step(y, part, then)
             if self.trace is not None and (then is None or then[2] != i):
                 self.trace.append(res.residual())
         if last_idx is not None and last_idx.numel() == 0:
             return torch.empty((0, cfg.vocab_size), dtype=torch.float32, device=self.device)
-        return K.linear_f32(res.final(last_idx), w.lm_head)[:, :cfg.vocab_size]
+        return K.linear_f32(res.final(last_idx), w.lm_head, cfg.logit_scale)[:, :cfg.vocab_size]
 
     def _mlp(self, mlp, lw, h, mm):
+        if isinstance(mlp, MoeMlp):
+            return M.moe(h, mlp, lw, self.dtype, mm, acc=self.acc)
         if mlp.act == "polynorm":
-            return H.poly_norm(mm(h, lw["w_up"]), mlp.ff, lw["act"], self.cfg.norm_eps, self.dtype, acc=self.acc)
-        u = gemm_relu2(h, lw["w_up"], mlp.ff) if h.is_cuda and not self.acc else None      # activation in the GEMM
-        return K.relu2(mm(h, lw["w_up"]), mlp.ff, self.dtype, acc=self.acc) if u is None else u
+            u = H.poly_norm(mm(h, lw["w_up"]), mlp.ff, lw["act"], self.cfg.norm_eps, self.dtype, acc=self.acc)
+        elif mlp.act == "swiglu":
+            u = M.swiglu(h, lw["w_up"], mlp.ff, self.dtype, acc=self.acc)
+        else:
+            u = gemm_relu2(h, lw["w_up"], mlp.ff) if h.is_cuda and not self.acc else None  # activation in the GEMM
+            u = K.relu2(mm(h, lw["w_up"]), mlp.ff, self.dtype, acc=self.acc) if u is None else u
+        return mm(u, lw["w_down"])
 
     def _attention(self, i, m: AttentionMixer, lw, xa, rows: K.Rows, segs):
         # prompts with heads of up to 128: the varlen tcgen05 kernel on rows cut at the chunk edges; everything else
@@ -161,13 +197,20 @@ class StackRunner:
         packed = None
         if (xa.is_cuda and self.dtype == torch.bfloat16 and 32 < max(m.dim, m.vdim) <= K.PACKED_HD and m.vdim % 8 == 0
                 and self.pack_prompts):
-            packed = (segs or {}).get(m.chunk)
+            packed = (segs or {}).get(m.reach)
         proj = gemm_skinny_acc(xa, lw["w_in"]) if self.acc else K.linear(xa, lw["w_in"])
-        q, gate = K.qk_norm_rope_cache(proj, self.sections[i], m, lw.get("q_norm"), lw.get("k_norm"), self.cfg.norm_eps, rows,
-                                       self.ropes[i], self.kv.k[i], self.kv.v[i], self.dtype, packed=packed, acc=self.acc)
+        sink = lw.get("sink")
+        if m.whole_rows:
+            q, own = K.qkv_rows(proj, self.sections[i], m, lw, self.cfg.norm_eps, rows, self.first_v, self.kv.k[i], self.kv.v[i], self.dtype,
+                                packed=packed, acc=self.acc)
+            self.first_v = own if own is not None else self.first_v
+            gate = None
+        else:
+            q, gate = K.qk_norm_rope_cache(proj, self.sections[i], m, lw.get("q_norm"), lw.get("k_norm"), self.cfg.norm_eps, rows,
+                                           self.ropes[i], self.kv.k[i], self.kv.v[i], self.dtype, packed=packed, acc=self.acc)
         if packed is not None:
-            return K.packed_attention(q, m, rows, packed, self.kv.k[i], self.kv.v[i], gate)
-        return K.paged_attention(q, m, rows, self.kv.k[i], self.kv.v[i], gate)
+            return K.packed_attention(q, m, rows, packed, self.kv.k[i], self.kv.v[i], gate, sink=sink)
+        return K.paged_attention(q, m, rows, self.kv.k[i], self.kv.v[i], gate, sink=sink)
 
     def _mamba2(self, i, m: Mamba2Mixer, lw, xa, rows: K.Rows, segs):
         s, st = self.sections[i], self.states
@@ -192,7 +235,7 @@ class StackRunner:
     def _latent(self, i, m: LatentAttentionMixer, lw, xa, rows: K.Rows, segs):
         proj = gemm_skinny_acc(xa, lw["w_in"]) if self.acc else K.linear(xa, lw["w_in"])
         return LA.latent_attention(proj, self.sections[i], m, lw, self.w.derived[i].get("w_expand"), self.cfg.norm_eps, rows, self.ropes[i],
-                                   self.kv.k[i], self.dtype, (segs or {}).get(m.chunk) if self.pack_prompts else None, acc=self.acc)
+                                   self.kv.k[i], self.dtype, (segs or {}).get(m.reach) if self.pack_prompts else None, acc=self.acc)
 
     def _mlstm(self, i, m: MLstmMixer, lw, xa, rows: K.Rows, segs):
         s, st = self.sections[i], self.states
@@ -201,3 +244,12 @@ class StackRunner:
         y = K.mlstm_scan(proj[:, s["q"]:s["q"] + qk], proj[:, s["k"]:s["k"] + qk], proj[:, s["v"]:s["v"] + vv], gates, lw["gate_b"], m.gate_cap,
                          st.ssm[i], st.vec[i], rows, m.heads, m.dim, m.vdim)
         return K.gated_norm(y, proj[:, s["g"]:s["g"] + vv], lw["norm"], self.cfg.norm_eps, m.heads, gate_first=False)
+
+    def _delta(self, i, m: DeltaMixer, lw, xa, rows: K.Rows, segs):
+        s, st, der = self.sections[i], self.states, self.w.derived[i]
+        qk, vv = m.kv_heads * m.dim, m.heads * m.vdim
+        proj, gates = H.linear_split(xa, lw["w_in"], s["gates"])
+        x, proj = K.short_conv(proj, 0, s["g"], lw["conv"], der["conv_b"], st.conv[i], rows, self.dtype)
+        y = D.delta_scan(x[:, :qk], x[:, s["k"]:s["k"] + qk], x[:, s["v"]:s["v"] + vv], gates, lw["A_log"], lw["dt_bias"], st.ssm[i], rows, m.heads,
+                         m.kv_heads, m.dim, m.vdim, conv_src=proj, conv_col=0, conv_state=st.conv[i])
+        return K.gated_norm(y, proj[:, s["g"]:s["g"] + vv], der["norm"], self.cfg.norm_eps, m.heads, gate_first=False, silu=True)
