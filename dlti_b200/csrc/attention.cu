@@ -61,6 +61,8 @@ struct AttnParams {
   const float* gate;     // optional [output rows, H] factors on the head outputs
   const float* sink;     // optional [H]: one more term exp(sink) in the softmax denominator, without a value
   int vdim;              // value columns of a head that are written, head h at column h * vdim of O (0: 128)
+  int window;            // > 0: a row sees itself and the window - 1 rows before it
+  float cap;             // CAP form: scores become cap tanh(score / cap)
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
@@ -757,8 +759,9 @@ __device__ __forceinline__ void mbar_wait_b(uint32_t bar, uint32_t parity) {
 
 // SPLIT: the softmax weights are written as two 16-bit terms (hi over columns 0-63 of the S buffer, what its rounding
 // left over columns 64-127) and both enter the PV product, so the weights keep fp32-like precision (16 mantissa bits)
-// for 1.5x the MMA work.
-template <typename T, bool SPLIT>
+// for 1.5x the MMA work. With a window a tile starts at the key block that its first row's window reaches into.
+// CAP: soft cap on the scores (see capped_log2 in mma_sync.cuh).
+template <typename T, bool SPLIT, bool CAP = false>
 __global__ void __launch_bounds__(F2_THREADS, 1)
 attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) {
   const int b = blockIdx.z, h = blockIdx.y;
@@ -774,6 +777,9 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
   const int nA = qbA + 1, nB = (qbB < nqb) ? qbB + 1 : 0;   // KV blocks each tile attends to
   const int nblk = nB > nA ? nB : nA;
   const bool hasB = nB > 0;
+  // first key block of each tile: that of the window of its first row
+  const int jA0 = SPLIT && p.window > 0 ? max(0, qbA * 128 - p.window + 1) >> 7 : 0;
+  const int jB0 = SPLIT && p.window > 0 ? max(0, qbB * 128 - p.window + 1) >> 7 : 0;
   const int kvh = h / (p.H / p.KV);
 
   extern __shared__ uint8_t smem_raw[];
@@ -819,14 +825,14 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
         tma_load_2d(sQ + 32768, &tm128, q_full, qcol, row0 + qbB * 128);
         tma_load_2d(sQ + 32768 + 16384, &tm128, q_full, qcol + 64, row0 + qbB * 128);
       }
-      for (int j = 0; j < nblk; ++j) {
-        const int s = j & 1;
-        const int r = row0 + j * 128;
-        if (j >= 2) mbar_wait_b(k_empty + 8 * s, ((j >> 1) - 1) & 1);
+      for (int i = 0; i < nblk - jA0; ++i) {
+        const int s = i & 1;
+        const int r = row0 + (jA0 + i) * 128;
+        if (i >= 2) mbar_wait_b(k_empty + 8 * s, ((i >> 1) - 1) & 1);
         mbar_expect_tx(k_full + 8 * s, 32768);
         tma_load_2d(sK + s * 32768, &tm128, k_full + 8 * s, kcol, r);
         tma_load_2d(sK + s * 32768 + 16384, &tm128, k_full + 8 * s, kcol + 64, r);
-        if (j >= 2) mbar_wait_b(v_empty + 8 * s, ((j >> 1) - 1) & 1);
+        if (i >= 2) mbar_wait_b(v_empty + 8 * s, ((i >> 1) - 1) & 1);
         mbar_expect_tx(v_full + 8 * s, 32768);
         tma_load_2d(sV + s * 32768, &tm128, v_full + 8 * s, vcol, r);
         tma_load_2d(sV + s * 32768 + 16384, &tm128, v_full + 8 * s, vcol + 64, r);
@@ -839,9 +845,11 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
       const uint32_t idesc_pv = umma_idesc_f16(p.dtype, 128, 128, false, true);
       const DescLoHi dQ0 = desc_split(sQ, 0, 1024), dK0 = desc_split(sK, 0, 1024);
       const DescLoHi dV0 = desc_split(sV, 128 * 128, 1024);     // MN-major view of a [128 keys x 128] tile
-      auto issue_s = [&](int X, int j) {
+      const int n = nblk - jA0, eA = nA - jA0, iB0 = jB0 - jA0, eB = nB - jA0;
+      // i: key block, counted from the first one that is loaded
+      auto issue_s = [&](int X, int i) {
         DescLoHi q = dQ0, k = dK0;
-        q.lo += X * 2048; k.lo += (j & 1) * 2048;                // 32 KB = 2048 descriptor units
+        q.lo += X * 2048; k.lo += (i & 1) * 2048;                // 32 KB = 2048 descriptor units
         const uint32_t tS = tmem + X * 128;
         if (!leader) return;
 #pragma unroll
@@ -849,11 +857,11 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
           umma_f16_ss(tS, q.at(koff_kmajor(128, kk)), k.at(koff_kmajor(128, kk)), idesc_s, kk > 0);
         umma_commit(s_full + 8 * X);
       };
-      auto issue_pv = [&](int X, int j) {
+      auto issue_pv = [&](int X, int i) {
         DescLoHi v = dV0;
-        v.lo += (j & 1) * 2048;
+        v.lo += (i & 1) * 2048;
         const uint32_t tO = tmem + 256 + X * 128, tP = tmem + X * 128;
-        const uint32_t acc_on = j > 0 ? 1u : 0u;
+        const uint32_t acc_on = i > (X ? iB0 : 0) ? 1u : 0u;
         if (!leader) return;
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk)
@@ -868,11 +876,11 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
       mbar_wait_b(k_full, 0);
       tc_fence_after();
       issue_s(0, 0);
-      if (hasB) issue_s(1, 0);
+      if (hasB && iB0 == 0) issue_s(1, 0);
       if (leader) umma_commit(k_empty);
-      for (int j = 0; j < nblk; ++j) {
+      for (int j = 0; j < n; ++j) {
         const int s = j & 1;
-        const bool actA = j < nA, actB = j < nB, nxtA = j + 1 < nA, nxtB = j + 1 < nB;
+        const bool actA = j < eA, actB = j >= iB0 && j < eB, nxtA = j + 1 < eA, nxtB = j + 1 >= iB0 && j + 1 < eB;
         mbar_wait_b(v_full + 8 * s, (j >> 1) & 1);
         if (nxtA || nxtB) mbar_wait_b(k_full + 8 * (s ^ 1), ((j + 1) >> 1) & 1);
         if (actA) {
@@ -886,7 +894,7 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
           if (!nxtB && leader) umma_commit(k_empty + 8 * (s ^ 1));
         }
         if (actB) {
-          mbar_wait_b(p_full + 8, j & 1);
+          mbar_wait_b(p_full + 8, (j - iB0) & 1);
           tc_fence_after();
           issue_pv(1, j);
           if (leader) umma_commit(v_empty + 8 * s);
@@ -900,24 +908,38 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
   } else {
     const int X = warp >> 2;                    // 0: tile A, 1: tile B
     const int nX = X ? nB : nA;
-    const int qbX = X ? qbB : qbA;
+    const int qbX = X ? qbB : qbA, jX0 = X ? jB0 : jA0;
     if (nX > 0) {
       const int quarter = warp & 3;
       const int r = quarter * 32 + lane;          // query row inside the tile
       const uint32_t tS = tmem + ((uint32_t)(quarter * 32) << 16) + X * 128;
       const uint32_t tO = tmem + ((uint32_t)(quarter * 32) << 16) + 256 + X * 128;
-      const float sl2 = p.scale * LOG2E;
+      const float sl2 = CAP ? 1.f : p.scale * LOG2E;
       float m_ref = -INFINITY, l = 0.f;
-      for (int j = 0; j < nX; ++j) {
+      for (int j = jX0; j < nX; ++j) {
         const bool diag = (j == qbX);
-        mbar_wait_b(s_full + 8 * X, j & 1);
+        const int it = j - jX0;
+        mbar_wait_b(s_full + 8 * X, it & 1);
         tc_fence_after();
         uint32_t v[128];
 #pragma unroll
         for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(tS + c * 32, *reinterpret_cast<uint32_t(*)[32]>(v + 32 * c));
         tmem_wait_ld();
+        if constexpr (CAP) {
+          const float c = p.cap * LOG2E, c2 = -2.f * c, f = 2.f * LOG2E * p.scale / p.cap;
+#pragma unroll
+          for (int i = 0; i < 128; ++i)
+            v[i] = __float_as_uint(fmaf(c2, __fdividef(1.f, 1.f + ex2_approx(__uint_as_float(v[i]) * f)), c));
+        }
         float mx = -INFINITY;
-        if (diag) {
+        if (SPLIT && p.window > 0 && (qbX - j) * 128 + 127 >= p.window) {     // some row's window starts in this block
+          const int lo = (qbX - j) * 128 + r - p.window + 1, hi = diag ? r : 127;
+#pragma unroll
+          for (int i = 0; i < 128; ++i) {
+            if (i < lo || i > hi) v[i] = __float_as_uint(-INFINITY);
+            mx = fmaxf(mx, __uint_as_float(v[i]));
+          }
+        } else if (diag) {
 #pragma unroll
           for (int i = 0; i < 128; ++i) {
             if (i > r) v[i] = __float_as_uint(-INFINITY);
@@ -928,8 +950,8 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
           for (int i = 0; i < 128; ++i) mx = fmaxf(mx, __uint_as_float(v[i]));
         }
         mx *= sl2;
-        if (j == 0) {
-          m_ref = mx;
+        if (it == 0) {
+          m_ref = fmaxf(mx, -1e30f);              // finite also where the window leaves a row nothing in its tile's first block
         } else {
           const float mnew = fmaxf(m_ref, mx);
           if (__any_sync(0xffffffffu, (mnew - m_ref) > 8.f)) {
@@ -937,7 +959,7 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
             const float alpha = ex2_approx(m_ref - mnew);
             m_ref = mnew;
             l *= alpha;
-            mbar_wait_b(pv_done + 8 * X, (j - 1) & 1);
+            mbar_wait_b(pv_done + 8 * X, (it - 1) & 1);
             tc_fence_after();
 #pragma unroll 1
             for (int c = 0; c < 8; ++c) {
@@ -974,7 +996,7 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
         __syncwarp();
         if (lane == 0) mbar_arrive(p_full + 8 * X);
       }
-      mbar_wait_b(pv_done + 8 * X, (nX - 1) & 1);
+      mbar_wait_b(pv_done + 8 * X, (nX - jX0 - 1) & 1);
       tc_fence_after();
       const int qi = qbX * 128 + r;
       const bool write = qi < seqlen && qi >= q0;
@@ -1077,17 +1099,17 @@ DLTI_API int dlti_attn_fwd(const void* qkv, void* out, float* lse, const int* cu
 
 // dqkv [T, (H+2KV)*128] receives dq | dk | dv. D_scratch: [H, T] fp32 workspace.
 // Inference form with split softmax weights (see attn_fwd2_kernel), bf16: heads padded to 128 columns in qkv, vdim (a
-// multiple of 8) of them written; optional gate [output rows, H]; output row pitch ldo (a multiple of 8); optional
+// multiple of 8) of them written; optional gate [output rows, H]; window / cap: see AttnParams (0: none); output row pitch ldo (a multiple of 8); optional
 // seq_q0 / seq_out0 (see AttnParams) for portions whose earlier keys and values lie in front of their rows.
 DLTI_API int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const float* sink, const int* cu_seqlens, const int* seq_q0,
-                                 const int* seq_out0, int batch, int max_seqlen, long long T_total, int H, int KV, int vdim, float scale,
-                                 cudaStream_t st) {
-  if (H % KV || ldo % 8 || vdim % 8 || vdim < 8 || vdim > HD || (seq_q0 == nullptr) != (seq_out0 == nullptr) || (reinterpret_cast<uintptr_t>(out) & 15)) return DLTI_ERR_BAD_ARG;
+                                 const int* seq_out0, int batch, int max_seqlen, long long T_total, int H, int KV, int vdim, int window,
+                                 float scale, float cap, cudaStream_t st) {
+  if (H % KV || window < 0 || cap < 0.f || ldo % 8 || vdim % 8 || vdim < 8 || vdim > HD || (seq_q0 == nullptr) != (seq_out0 == nullptr) || (reinterpret_cast<uintptr_t>(out) & 15)) return DLTI_ERR_BAD_ARG;
   if (batch <= 0 || T_total <= 0) return 0;
   AttnParams p{};
   p.cu_seqlens = cu_seqlens; p.H = H; p.KV = KV; p.W = (H + 2 * KV) * HD;
   p.O = out; p.ldo = ldo; p.T_total = T_total; p.scale = scale; p.dtype = DLTI_BF16; p.gate = gate; p.sink = sink;
-  p.seq_q0 = seq_q0; p.seq_out0 = seq_out0; p.vdim = vdim;
+  p.seq_q0 = seq_q0; p.seq_out0 = seq_out0; p.vdim = vdim; p.window = window; p.cap = cap;
   CUtensorMap tm;
   const int rc = make_map(&tm, qkv, T_total, p.W, 128);
   if (rc) return rc;
@@ -1096,9 +1118,10 @@ DLTI_API int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, cons
   DLTI_CUDA_CHECK(cudaGetDevice(&dev));
   if (!cfg[dev & 63]) {
     DLTI_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd2_kernel<__nv_bfloat16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, F2_SMEM));
+    DLTI_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd2_kernel<__nv_bfloat16, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, F2_SMEM));
     cfg[dev & 63] = true;
   }
-  attn_fwd2_kernel<__nv_bfloat16, true><<<dim3(((max_seqlen + 127) / 128 + 1) / 2, H, batch), F2_THREADS, F2_SMEM, st>>>(p, tm);
+  (cap > 0.f ? attn_fwd2_kernel<__nv_bfloat16, true, true> : attn_fwd2_kernel<__nv_bfloat16, true>)<<<dim3(((max_seqlen + 127) / 128 + 1) / 2, H, batch), F2_THREADS, F2_SMEM, st>>>(p, tm);
   dlti_count_launch();
   return (int)cudaGetLastError();
 }

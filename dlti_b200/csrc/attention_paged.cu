@@ -1,5 +1,6 @@
-// Attention over the paged cache for the layer-stack models: any head size, grouped key/value heads, causal or chunked
-// (position i sees keys of its own chunk of `chunk` positions only), optional per-head output gate.
+// Attention over the paged cache for the layer-stack models: any head size, grouped key/value heads, causal, chunked
+// (position i sees keys of its own chunk of `chunk` positions only) or windowed (itself and the window - 1 positions before
+// it), optional soft cap on the scores, per-head sink and per-head output gate.
 //
 //   attn_prefill_kernel  portions of prompts, bf16: a CTA owns 128 (token, head of a group) rows and streams key / value
 //                        tiles of 64 from the pages through shared memory into mma.sync
@@ -19,8 +20,8 @@ struct PagedParams {
   const void *kc, *vc; int kd, vd;                 // cache row pitches of a head
   const int* tables; int max_blocks; int bs;
   const int *ctx, *cu, *rseq, *pos; int nd;
-  int H, G, dim, vdim, chunk;
-  float scale;
+  int H, G, dim, vdim, chunk, window;
+  float scale, cap;                                // cap > 0: scores become cap tanh(score / cap)
   const float* gate;                               // [rows, H] factors or null
   void* out; long long o_ld;                       // head h at column h * vdim
   long long rows;
@@ -33,7 +34,13 @@ __device__ __forceinline__ float with_sink(const PagedParams& p, int h, float m,
   const float r = m == -INFINITY ? 0.f : m;
   return l + (natural ? expf(p.sink[h] - r) : ex2(p.sink[h] * 1.4426950408889634f - r));
 }
-__device__ __forceinline__ int first_key(int pos, int chunk) { return chunk > 0 ? pos / chunk * chunk : 0; }
+__device__ __forceinline__ int first_key(const PagedParams& p, int pos) {
+  return p.chunk > 0 ? pos / p.chunk * p.chunk : p.window > 0 ? max(0, pos - p.window + 1) : 0;
+}
+// a product q . k as the score in log2 units
+__device__ __forceinline__ float score_log2(const PagedParams& p, float s, float sl2) {
+  return p.cap > 0.f ? capped_log2(s, p.scale, p.cap) : s * sl2;
+}
 
 // ROWS_MAXV: value dims per lane
 template <typename T, int ROWS_MAXV>
@@ -54,7 +61,7 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const PagedParams p) {
   float m = -INFINITY, l = 0.f, o[ROWS_MAXV];
 #pragma unroll
   for (int i = 0; i < ROWS_MAXV; ++i) o[i] = 0.f;
-  for (int j0 = first_key(ps, p.chunk); j0 < nkeys; j0 += 32) {
+  for (int j0 = first_key(p, ps); j0 < nkeys; j0 += 32) {
     const int j = j0 + lane;
     float s = -INFINITY;
     long long slot = 0;
@@ -68,6 +75,7 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const PagedParams p) {
         a += b;
       }
       s = a * p.scale;
+      if (p.cap > 0.f) s = p.cap * tanhf(s / p.cap);
     }
     const float nm = fmaxf(m, warp_max(s));
     const float alpha = expf(m - nm);
@@ -232,7 +240,7 @@ __global__ void __launch_bounds__(256) attn_prefill_kernel(const PagedParams p) 
   const long long tile = (total + PF_ROWS - 1) / PF_ROWS - 1 - blockIdx.x;
   if (tile < 0) return;
   const long long r_first = tile * PF_ROWS, r_last = min(total, r_first + PF_ROWS) - 1;
-  const int jbeg = first_key(start + (int)(r_first / rep), p.chunk), jend = start + (int)(r_last / rep) + 1;
+  const int jbeg = first_key(p, start + (int)(r_first / rep)), jend = start + (int)(r_last / rep) + 1;
   const int* tab = p.tables + (long long)seq * p.max_blocks;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
@@ -247,13 +255,13 @@ __global__ void __launch_bounds__(256) attn_prefill_kernel(const PagedParams p) 
     head[x] = g * rep + (int)(r % rep);
     row[x] = row0 + i;
     pos[x] = ok ? start + i : -1;
-    jlo[x] = ok ? first_key(pos[x], p.chunk) : 0;
+    jlo[x] = ok ? first_key(p, pos[x]) : 0;
     qp[x] = ok ? reinterpret_cast<const bf16*>(p.q) + row[x] * p.q_ld + (long long)head[x] * p.q_hd : nullptr;
   }
   // key range of this warp's 16 rows
   const long long wr0 = r_first + warp * 16, wr1 = min(total, wr0 + 16) - 1;
   const bool warp_on = wr0 < total;
-  const int wlo = warp_on ? first_key(start + (int)(wr0 / rep), p.chunk) : 0, whi = warp_on ? start + (int)(wr1 / rep) : -1;
+  const int wlo = warp_on ? first_key(p, start + (int)(wr0 / rep)) : 0, whi = warp_on ? start + (int)(wr1 / rep) : -1;
 
   uint32_t qf[DK / 16][4];
   load_q<DK>(qf, qp[0], qp[1], p.dim);
@@ -296,7 +304,7 @@ __global__ void __launch_bounds__(256) attn_prefill_kernel(const PagedParams p) 
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         const int j = j0 + i * 8 + (lane & 3) * 2 + (x & 1), y = x >> 1;
-        s[i][x] = (j <= pos[y] && j >= jlo[y]) ? s[i][x] * sl2 : -INFINITY;
+        s[i][x] = (j <= pos[y] && j >= jlo[y]) ? score_log2(p, s[i][x], sl2) : -INFINITY;
         mx[y] = fmaxf(mx[y], s[i][x]);
       }
     float base[2];
@@ -361,7 +369,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const PagedParams p, i
   const int split = blockIdx.x, b = blockIdx.z, g = blockIdx.y / hblocks, h0 = (blockIdx.y % hblocks) * 16;
   const int nh = min(16, rep - h0);
   const int ctx = p.ctx[b];
-  const int kbeg = ctx > 0 ? first_key(ctx - 1, p.chunk) : 0;
+  const int kbeg = ctx > 0 ? first_key(p, ctx - 1) : 0;
   const int tiles = (ctx - kbeg + KT - 1) / KT, per = (tiles + splits - 1) / splits;
   const int jbeg = kbeg + split * per * KT, jend = min(ctx, jbeg + per * KT);
   const int* tab = p.tables + (long long)b * p.max_blocks;
@@ -405,7 +413,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const PagedParams p, i
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
           const int j = j0 + warp * 16 + i * 8 + (lane & 3) * 2 + (x & 1);
-          s[i][x] = j < jend ? s[i][x] * sl2 : -INFINITY;
+          s[i][x] = j < jend ? score_log2(p, s[i][x], sl2) : -INFINITY;
           mx[x >> 1] = fmaxf(mx[x >> 1], s[i][x]);
         }
 #pragma unroll
@@ -565,12 +573,12 @@ int launch_decode(const PagedParams& p, int splits, float* ws, cudaStream_t st) 
 // rows of decode sequences (row s = sequence s < nd) and of prompts (sequence nd + i: rows nd + cu[i] ... nd + cu[i+1]).
 DLTI_API int dlti_attn_rows(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd, const int* tables,
                             int max_blocks, int bs, const int* ctx, const int* rseq, const int* pos, int H, int G, int dim, int vdim,
-                            int chunk, float scale, const float* gate, const float* sink, void* out, long long o_ld, long long rows, int dtype,
+                            int chunk, int window, float scale, float cap, const float* gate, const float* sink, void* out, long long o_ld, long long rows, int dtype,
                             cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (H % G || dim < 1 || vdim < 1) return DLTI_ERR_BAD_ARG;
+  if (H % G || dim < 1 || vdim < 1 || (chunk > 0 && window > 0)) return DLTI_ERR_BAD_ARG;
   if (dim > 2048 || vdim > 1024) { dlti_set_error("attn_rows: queries of up to 2048 and values of up to 1024 dimensions"); return DLTI_ERR_TOO_LARGE; }
-  PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, nullptr, rseq, pos, 0, H, G, dim, vdim, chunk, scale,
+  PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, nullptr, rseq, pos, 0, H, G, dim, vdim, chunk, window, scale, cap,
                 gate, out, o_ld, rows, sink};
   if (dtype == DLTI_BF16) return launch_rows<__nv_bfloat16>(p, st);
   if (dtype == DLTI_FP32) return launch_rows<float>(p, st);
@@ -587,12 +595,12 @@ static int check_mma(int H, int G, int dim, int vdim, int kd, int vd, int q_hd) 
 // the rows themselves must be in the pages already.
 DLTI_API int dlti_attn_paged_prefill(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
                                      const int* tables, int max_blocks, int bs, const int* ctx, const int* cu, int nd, int nseq,
-                                     int max_rows, int H, int G, int dim, int vdim, int chunk, float scale, const float* gate, const float* sink, void* out,
+                                     int max_rows, int H, int G, int dim, int vdim, int chunk, int window, float scale, float cap, const float* gate, const float* sink, void* out,
                                      long long o_ld, cudaStream_t st) {
   if (nseq <= 0 || max_rows <= 0) return 0;
   if (int rc = check_mma(H, G, dim, vdim, kd, vd, q_hd)) return rc;
   if (q_ld % 2 || nseq > 65535) return DLTI_ERR_BAD_ARG;
-  PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, cu, nullptr, nullptr, nd, H, G, dim, vdim, chunk, scale,
+  PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, cu, nullptr, nullptr, nd, H, G, dim, vdim, chunk, window, scale, cap,
                 gate, out, o_ld, 0, sink};
   HEAD_DISPATCH(kd, vd, launch_prefill, p, nseq, max_rows, st);
 }
@@ -600,12 +608,12 @@ DLTI_API int dlti_attn_paged_prefill(const void* q, long long q_ld, int q_hd, co
 // bf16. Row b = the newest token of sequence b, whose context is ctx[b] tokens. ws: batch * H * splits * (vdim + 2) floats.
 DLTI_API int dlti_attn_paged_decode(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
                                     const int* tables, int max_blocks, int bs, const int* ctx, int batch, int H, int G, int dim, int vdim,
-                                    int chunk, float scale, const float* gate, const float* sink, int splits, float* ws, void* out, long long o_ld,
+                                    int chunk, int window, float scale, float cap, const float* gate, const float* sink, int splits, float* ws, void* out, long long o_ld,
                                     cudaStream_t st) {
   if (batch <= 0) return 0;
   if (int rc = check_mma(H, G, dim, vdim, kd, vd, q_hd)) return rc;
   if (q_ld % 2 || splits < 1 || batch > 65535) return DLTI_ERR_BAD_ARG;
-  PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, nullptr, nullptr, nullptr, 0, H, G, dim, vdim, chunk, scale,
+  PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, nullptr, nullptr, nullptr, 0, H, G, dim, vdim, chunk, window, scale, cap,
                 gate, out, o_ld, batch, sink};
   HEAD_DISPATCH(kd, vd, launch_decode, p, splits, ws, st);
 }

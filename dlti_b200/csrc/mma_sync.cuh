@@ -27,6 +27,11 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// log2(e) cap tanh(s scale / cap) as cap (1 - 2 / (1 + e^(2 x))): absolute error about 3e-7 cap
+__device__ __forceinline__ float capped_log2(float s, float scale, float cap) {
+  const float c = cap * 1.4426950408889634f;
+  return c - 2.f * c * __fdividef(1.f, 1.f + ex2(s * (2.f * 1.4426950408889634f * scale / cap)));
+}
 // two fp32 values as a bf16 pair and the bf16 pair of what the rounding left
 __device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
   const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);

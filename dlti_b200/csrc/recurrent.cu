@@ -8,7 +8,7 @@
 //             its own, keeps them for itself: vec [slots, heads, slices, N + 1] = n, then m.
 // States live in slots [slots, heads, N, P] and are carried from step to step; a sequence whose step starts at position
 // 0 starts from zero whatever its slot holds.
-#include "common.cuh"
+#include "recurrent.cuh"
 #include "mma_sync.cuh"
 
 namespace {
@@ -34,46 +34,10 @@ struct ScanParams {
   float* vec;
 };
 
-__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 // log gates of an mLSTM head: cap tanh(z / cap), for the forget gate the logarithm of its sigmoid
 __device__ __forceinline__ float log_in_gate(float z, float cap) { return cap * tanhf(z / cap); }
 __device__ __forceinline__ float log_forget_gate(float z, float cap) { return -softplus_f(-cap * tanhf(z / cap)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
-// exp(x) of a decay. Near 1 the rounding of exp itself repeats at every token and adds up over a long memory; 1 + expm1
-// rounds once.
-__device__ __forceinline__ float decay_of(float x) { return x > -0.5f ? 1.f + expm1f(x) : expf(x); }
-
-__device__ __forceinline__ void seq_rows(const ScanParams& p, int s, long long& row0, int& n, int& start) {
-  if (s < p.nd) {
-    row0 = s;
-    n = 1;
-  } else {
-    row0 = p.nd + p.cu[s - p.nd];
-    n = p.cu[s - p.nd + 1] - p.cu[s - p.nd];
-  }
-  start = p.ctx[s] - n;
-}
-
-// Shift the convolution inputs of one sequence: entry j becomes the input at position end - conv_rows + j. A thread
-// owns whole channels and walks j upwards, so reading an old entry (always at a higher index) is safe.
-template <typename T>
-__device__ __forceinline__ void conv_tail(const ScanParams& p, int s, int part, int parts) {
-  const int slot = p.sslot[s];
-  if (slot < 0) return;
-  long long row0;
-  int n, start;
-  seq_rows(p, s, row0, n, start);
-  const T* src = reinterpret_cast<const T*>(p.conv_src);
-  T* st = reinterpret_cast<T*>(p.conv_state) + (long long)slot * p.conv_rows * p.conv_C;
-  for (int c = part * blockDim.x + threadIdx.x; c < p.conv_C; c += parts * blockDim.x)
-    for (int j = 0; j < p.conv_rows; ++j) {
-      const int q = n - p.conv_rows + j;
-      T v = Cvt<T>::from_f(0.f);
-      if (q >= 0) v = src[(row0 + q) * p.conv_ld + p.conv_col + c];
-      else if (start > 0) v = st[(long long)(q + p.conv_rows) * p.conv_C + c];
-      st[(long long)j * p.conv_C + c] = v;
-    }
-}
 
 // Token-by-token form. CTA = (32 columns of P, head, sequence), 8 warps: lane = column, a warp owns the NR consecutive
 // rows [warp * NR, ...), so q and k are warp-uniform shared-memory reads. TT tokens are staged at a time; the warps'

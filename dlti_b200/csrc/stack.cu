@@ -23,12 +23,13 @@ __global__ void embed_rows_kernel(const long long* __restrict__ ids, const T* __
   }
 }
 
-// out = acc (fp32), acc = 0
-__global__ void take_rows_kernel(float* __restrict__ acc, float* __restrict__ out, long long vec) {
+// out = scale * acc (fp32), acc = 0
+__global__ void take_rows_kernel(float* __restrict__ acc, float* __restrict__ out, float scale, long long vec) {
   griddep_wait();
   griddep_launch();
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < vec; i += (long long)gridDim.x * blockDim.x) {
-    reinterpret_cast<float4*>(out)[i] = reinterpret_cast<float4*>(acc)[i];
+    const float4 v = reinterpret_cast<float4*>(acc)[i];
+    reinterpret_cast<float4*>(out)[i] = make_float4(scale * v.x, scale * v.y, scale * v.z, scale * v.w);
     reinterpret_cast<float4*>(acc)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
   }
 }
@@ -182,10 +183,12 @@ __global__ void relu2_vec_kernel(const void* __restrict__ u, long long u_ld, T* 
 }
 
 // Norm of a mixer output in `groups` equal parts with a multiplicative gate.
-//   GATE_FIRST:  out = norm(y * silu(g)) * w          (Mamba-2)
-//   otherwise:   out = norm(y) * w * sigmoid(g)       (lightning attention)
+//   GATE_SILU_FIRST:  out = norm(y * silu(g)) * w          (Mamba-2)
+//   GATE_SIGMOID:     out = norm(y) * w * sigmoid(g)       (lightning attention, mLSTM)
+//   GATE_SILU:        out = norm(y) * w * silu(g)          (delta rule)
 // One CTA per row, one warp per group in turn; a group is passed twice (second time from L1).
-template <typename T, bool GATE_FIRST, bool ACC>
+enum Gate : int { GATE_SIGMOID = 0, GATE_SILU_FIRST = 1, GATE_SILU = 2 };
+template <typename T, int GATE, bool ACC>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const T* __restrict__ y, long long y_ld, const void* __restrict__ gate,
                                                          long long g_ld, const float* __restrict__ w, T* __restrict__ out,
                                                          long long o_ld, int n, int groups, float eps) {
@@ -199,19 +202,19 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const T* __restrict__ y
   const int gs = n / groups;
   for (int c = threadIdx.x; c < n; c += blockDim.x) {
     const float g = take<T, ACC>(gr, c);
-    row_s[c] = GATE_FIRST ? Cvt<T>::to_f(yr[c]) * silu_f(g) : sigmoid_f(g);
+    row_s[c] = GATE == GATE_SILU_FIRST ? Cvt<T>::to_f(yr[c]) * silu_f(g) : GATE == GATE_SILU ? silu_f(g) : sigmoid_f(g);
   }
   __syncthreads();
   if (groups == 1) {
     float ss = 0.f;
     for (int c = threadIdx.x; c < n; c += blockDim.x) {
-      const float v = GATE_FIRST ? row_s[c] : Cvt<T>::to_f(yr[c]);
+      const float v = GATE == GATE_SILU_FIRST ? row_s[c] : Cvt<T>::to_f(yr[c]);
       ss += v * v;
     }
     ss = block_sum(ss, red);
     const float r = 1.f / sqrtf(ss / (float)n + eps);
     for (int c = threadIdx.x; c < n; c += blockDim.x) {
-      const float v = (GATE_FIRST ? row_s[c] : Cvt<T>::to_f(yr[c]) * row_s[c]) * r * w[c];
+      const float v = (GATE == GATE_SILU_FIRST ? row_s[c] : Cvt<T>::to_f(yr[c]) * row_s[c]) * r * w[c];
       out[t * o_ld + c] = Cvt<T>::from_f(v);
     }
     return;
@@ -219,19 +222,19 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const T* __restrict__ y
   for (int g = threadIdx.x >> 5; g < groups; g += blockDim.x >> 5) {
     float ss = 0.f;
     for (int c = g * gs + (threadIdx.x & 31); c < (g + 1) * gs; c += 32) {
-      const float v = GATE_FIRST ? row_s[c] : Cvt<T>::to_f(yr[c]);
+      const float v = GATE == GATE_SILU_FIRST ? row_s[c] : Cvt<T>::to_f(yr[c]);
       ss += v * v;
     }
     const float r = 1.f / sqrtf(warp_sum(ss) / (float)gs + eps);
     for (int c = g * gs + (threadIdx.x & 31); c < (g + 1) * gs; c += 32) {
-      const float v = (GATE_FIRST ? row_s[c] : Cvt<T>::to_f(yr[c]) * row_s[c]) * r * w[c];
+      const float v = (GATE == GATE_SILU_FIRST ? row_s[c] : Cvt<T>::to_f(yr[c]) * row_s[c]) * r * w[c];
       out[t * o_ld + c] = Cvt<T>::from_f(v);
     }
   }
 }
 
 // the same in 16-byte pieces for 16-bit T and groups of whole pieces: one CTA per (row, group), everything in registers
-template <typename T, bool GATE_FIRST, bool ACC, int VPT>
+template <typename T, int GATE, bool ACC, int VPT>
 __global__ void __launch_bounds__(512) gated_norm_vec_kernel(const T* __restrict__ y, long long y_ld, const void* __restrict__ gate,
                                                              long long g_ld, const float* __restrict__ w, T* __restrict__ out,
                                                              long long o_ld, int gs, float eps) {
@@ -258,8 +261,8 @@ __global__ void __launch_bounds__(512) gated_norm_vec_kernel(const T* __restrict
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const float e = fast_sigmoid(g[i][j]);
-        if (GATE_FIRST) v[i][j] *= g[i][j] * e;
-        else g[i][j] = e;
+        if (GATE == GATE_SILU_FIRST) v[i][j] *= g[i][j] * e;
+        else g[i][j] = GATE == GATE_SILU ? g[i][j] * e : e;
         ss += v[i][j] * v[i][j];
       }
   ss = block_sum(ss, red);
@@ -271,14 +274,14 @@ __global__ void __launch_bounds__(512) gated_norm_vec_kernel(const T* __restrict
       float wv[8];
       ld8(w + c0 + p * 8, wv);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) v[i][j] *= r * wv[j] * (GATE_FIRST ? 1.f : g[i][j]);
+      for (int j = 0; j < 8; ++j) v[i][j] *= r * wv[j] * (GATE == GATE_SILU_FIRST ? 1.f : g[i][j]);
       put_n(out + t * o_ld + c0 + p * 8, v[i]);
     }
   }
 }
 
 // many small groups: a warp per group, eight groups a CTA
-template <typename T, bool GATE_FIRST, bool ACC, int VPT>
+template <typename T, int GATE, bool ACC, int VPT>
 __global__ void __launch_bounds__(256) gated_norm_warp_kernel(const T* __restrict__ y, long long y_ld, const void* __restrict__ gate,
                                                               long long g_ld, const float* __restrict__ w, T* __restrict__ out,
                                                               long long o_ld, int gs, int groups, long long total, float eps) {
@@ -303,8 +306,8 @@ __global__ void __launch_bounds__(256) gated_norm_warp_kernel(const T* __restric
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const float e = fast_sigmoid(g[i][j]);
-        if (GATE_FIRST) v[i][j] *= g[i][j] * e;
-        else g[i][j] = e;
+        if (GATE == GATE_SILU_FIRST) v[i][j] *= g[i][j] * e;
+        else g[i][j] = GATE == GATE_SILU ? g[i][j] * e : e;
         ss += v[i][j] * v[i][j];
       }
   const float r = 1.f / sqrtf(warp_sum(ss) / (float)gs + eps);
@@ -314,7 +317,7 @@ __global__ void __launch_bounds__(256) gated_norm_warp_kernel(const T* __restric
       float wv[8];
       ld8(w + c0 + (lane + 32 * i) * 8, wv);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) v[i][j] *= r * wv[j] * (GATE_FIRST ? 1.f : g[i][j]);
+      for (int j = 0; j < 8; ++j) v[i][j] *= r * wv[j] * (GATE == GATE_SILU_FIRST ? 1.f : g[i][j]);
       put_n(out + t * o_ld + c0 + (lane + 32 * i) * 8, v[i]);
     }
 }
@@ -505,6 +508,95 @@ __global__ void __launch_bounds__(128) qk_norm_rope_cache_vec_kernel(const QkvPa
       void* pk = is_v ? p.vp : p.kp;
       if (pk) put_n(reinterpret_cast<T*>(pk) + to * p.q_ld + g * p.q_hd + e0, v[i]);
       if (own && slot >= 0) put_n(reinterpret_cast<T*>(is_v ? p.vc : p.kc) + (slot * p.G + g) * (is_v ? p.vd : p.kd) + e0, v[i]);
+    }
+  }
+}
+
+// Whole projection rows: bias, norm of q and of k over all their heads, values mixed with those of an earlier layer, cache
+// write of k and v. One CTA per token; the row waits in shared memory for its norms. W: elements per piece (8: 16-bit T, head
+// sizes and pitches multiples of 8).
+struct QkvRowParams {
+  const void* proj; long long ld; int oq, ok, ov;
+  const float *bias, *qn, *kn; float eps;                  // bias: laid out as the projection; any of them may be null
+  const void* first; long long f_ld; const float* share;   // values to mix in [tokens, G * vdim] and their share (null: none)
+  void* own; long long own_ld;                             // copy of the values before mixing (null: none)
+  const long long* slots; void *kc, *vc; int kd, vd;
+  void* q; long long q_ld; int q_hd;
+  void *kp, *vp; const int* dst; int nd;                   // packed keys / values, as in QkvParams
+  int H, G, dim, vdim;
+};
+template <typename T, bool ACC, int W>
+__device__ __forceinline__ void row_piece(const void* row, const float* bias, int c, float (&f)[W]) {
+  if constexpr (W == 1) f[0] = take<T, ACC>(row, c);
+  else take_n<T, ACC, W>(row, c, f);
+  if (bias) {
+#pragma unroll
+    for (int j = 0; j < W; ++j) f[j] += bias[c + j];
+  }
+}
+template <typename T, int W>
+__device__ __forceinline__ void put_piece(T* p, const float (&f)[W]) {
+  if constexpr (W == 1) *p = Cvt<T>::from_f(f[0]);
+  else put_n(p, f);
+}
+template <typename T, bool ACC, int W>
+__global__ void __launch_bounds__(256) qkv_rows_kernel(const QkvRowParams p) {
+  __shared__ float red[32];
+  extern __shared__ __align__(16) float row_q[];           // q, then k
+  griddep_wait();
+  griddep_launch();
+  const long long t = blockIdx.x;
+  const uint8_t* row = reinterpret_cast<const uint8_t*>(p.proj) + t * p.ld * (ACC ? 4 : sizeof(T));
+  const long long slot = p.slots[t];
+  const long long to = (p.dst && t >= p.nd) ? p.nd + (long long)p.dst[t - p.nd] : t;
+  const int nq = p.H * p.dim, nk = p.G * p.dim, nv = p.G * p.vdim;
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x * W; i < nq + nk; i += blockDim.x * W) {
+    float f[W];
+    row_piece<T, ACC, W>(row, p.bias, i < nq ? p.oq + i : p.ok + i - nq, f);
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < W; ++j) {
+      ss += f[j] * f[j];
+      row_q[i + j] = f[j];
+    }
+    if (i < nq) sq += ss;
+    else sk += ss;
+  }
+  const float share = p.first ? p.share[0] : 0.f;
+  for (int i = threadIdx.x * W; i < nv; i += blockDim.x * W) {
+    float f[W];
+    row_piece<T, ACC, W>(row, p.bias, p.ov + i, f);
+    if (p.own) put_piece<T, W>(reinterpret_cast<T*>(p.own) + t * p.own_ld + i, f);
+    if (p.first) {
+      float e[W];
+      row_piece<T, false, W>(reinterpret_cast<const T*>(p.first) + t * p.f_ld, nullptr, i, e);
+#pragma unroll
+      for (int j = 0; j < W; ++j) f[j] += share * (e[j] - f[j]);
+    }
+    const int g = i / p.vdim, c = i - g * p.vdim;
+    if (p.vp) put_piece<T, W>(reinterpret_cast<T*>(p.vp) + to * p.q_ld + (long long)g * p.q_hd + c, f);
+    if (slot >= 0) put_piece<T, W>(reinterpret_cast<T*>(p.vc) + (slot * p.G + g) * p.vd + c, f);
+  }
+  float rq = 1.f, rk = 1.f;
+  if (p.qn) {
+    rq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + p.eps);
+    rk = 1.f / sqrtf(block_sum(sk, red) / (float)nk + p.eps);
+  }
+  for (int i = threadIdx.x * W; i < nq + nk; i += blockDim.x * W) {      // a thread's own pieces: no barrier needed
+    const bool is_q = i < nq;
+    const int x = is_q ? i : i - nq, h = x / p.dim, c = x - h * p.dim;
+    float f[W];
+#pragma unroll
+    for (int j = 0; j < W; ++j) {
+      f[j] = row_q[i + j];
+      if (p.qn) f[j] *= (is_q ? rq : rk) * (is_q ? p.qn : p.kn)[x + j];
+    }
+    if (is_q) {
+      put_piece<T, W>(reinterpret_cast<T*>(p.q) + to * p.q_ld + (long long)h * p.q_hd + c, f);
+    } else {
+      if (p.kp) put_piece<T, W>(reinterpret_cast<T*>(p.kp) + to * p.q_ld + (long long)h * p.q_hd + c, f);
+      if (slot >= 0) put_piece<T, W>(reinterpret_cast<T*>(p.kc) + (slot * p.G + h) * p.kd + c, f);
     }
   }
 }
@@ -752,6 +844,43 @@ int post_norm_add_t(const void* y, long long y_ld, float* x, const float* w, voi
   return DLTI_ERR_TOO_LARGE;
 }
 
+template <int GATE>
+int gated_norm_mode(const void* y, long long y_ld, const void* gate, long long g_ld, const float* w, void* out, long long o_ld, long long rows,
+                    int n, int groups, float eps, int acc, int dtype, cudaStream_t st) {
+  const int gs = n / groups;
+  if (dtype == DLTI_BF16 && gs % 8 == 0 && gs <= 8 * 512 * 4 && y_ld % 8 == 0 && g_ld % 8 == 0 && o_ld % 8 == 0 && groups <= 65535 &&
+      ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+    using B = __nv_bfloat16;
+    if (groups > 1 && gs <= 512) {
+      auto kern = acc ? (gs <= 256 ? gated_norm_warp_kernel<B, GATE, true, 1> : gated_norm_warp_kernel<B, GATE, true, 2>)
+                      : (gs <= 256 ? gated_norm_warp_kernel<B, GATE, false, 1> : gated_norm_warp_kernel<B, GATE, false, 2>);
+      const long long total = rows * groups;
+      DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)((total + 7) / 8)), dim3(256), 0, st, (const B*)y, y_ld, gate, g_ld, w, (B*)out,
+                                      o_ld, gs, groups, total, eps));
+      dlti_count_launch();
+      return 0;
+    }
+    const int vec = gs / 8, threads = vec <= 64 ? 64 : (vec <= 128 ? 128 : (vec <= 512 ? 256 : 512)), vpt = (vec + threads - 1) / threads;
+#define GNV(AC) (vpt <= 1 ? gated_norm_vec_kernel<B, GATE, AC, 1> : vpt <= 2 ? gated_norm_vec_kernel<B, GATE, AC, 2> : gated_norm_vec_kernel<B, GATE, AC, 4>)
+    auto kern = acc ? GNV(true) : GNV(false);
+#undef GNV
+    DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)rows, groups), dim3(threads), 0, st, (const B*)y, y_ld, gate, g_ld, w, (B*)out,
+                                    o_ld, gs, eps));
+    dlti_count_launch();
+    return 0;
+  }
+  const size_t smem = (size_t)n * 4;
+  if (smem > 48 * 1024) { dlti_set_error("gated_norm: rows of up to 12288 elements"); return DLTI_ERR_TOO_LARGE; }
+#define GN_CASE(AC)                                                                                                            \
+  DISPATCH_T(dtype, DLTI_CUDA_CHECK(dlti_launch_pdl(rows, gated_norm_kernel<T, GATE, AC>, dim3((unsigned)rows), dim3(256), smem, st, \
+                                                    (const T*)y, y_ld, gate, g_ld, w, (T*)out, o_ld, n, groups, eps)))
+  if (acc) GN_CASE(true);
+  else GN_CASE(false);
+#undef GN_CASE
+  dlti_count_launch();
+  return 0;
+}
+
 }  // namespace
 
 DLTI_API int dlti_embed_rows(const long long* ids, const void* table, float* x, void* xa, long long xa_ld, long long tokens,
@@ -764,12 +893,12 @@ DLTI_API int dlti_embed_rows(const long long* ids, const void* table, float* x, 
   return 0;
 }
 
-// the decode GEMM's accumulator [rows, cols] as an fp32 result (cols a multiple of 4); zero on return
-DLTI_API int dlti_take_rows(float* acc, float* out, long long rows, int cols, cudaStream_t st) {
+// the decode GEMM's accumulator [rows, cols] times scale as an fp32 result (cols a multiple of 4); zero on return
+DLTI_API int dlti_take_rows(float* acc, float* out, float scale, long long rows, int cols, cudaStream_t st) {
   if (rows <= 0) return 0;
   if (cols % 4) return DLTI_ERR_BAD_ARG;
   const long long vec = rows * (cols / 4);
-  DLTI_CUDA_CHECK(dlti_launch_pdl(rows, take_rows_kernel, dim3(grid_for(vec, 256)), dim3(256), 0, st, acc, out, vec));
+  DLTI_CUDA_CHECK(dlti_launch_pdl(rows, take_rows_kernel, dim3(grid_for(vec, 256)), dim3(256), 0, st, acc, out, scale, vec));
   dlti_count_launch();
   return 0;
 }
@@ -813,47 +942,14 @@ DLTI_API int dlti_relu2(const void* u, long long u_ld, void* h, long long h_ld, 
   return 0;
 }
 
+// mode: see Gate
 DLTI_API int dlti_gated_norm(const void* y, long long y_ld, const void* gate, long long g_ld, const float* w, void* out, long long o_ld,
-                             long long rows, int n, int groups, float eps, int gate_first, int acc, int dtype, cudaStream_t st) {
+                             long long rows, int n, int groups, float eps, int mode, int acc, int dtype, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (groups < 1 || n % groups) return DLTI_ERR_BAD_ARG;
-  const int gs = n / groups;
-  if (dtype == DLTI_BF16 && gs % 8 == 0 && gs <= 8 * 512 * 4 && y_ld % 8 == 0 && g_ld % 8 == 0 && o_ld % 8 == 0 && groups <= 65535 &&
-      ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
-    using B = __nv_bfloat16;
-    if (groups > 1 && gs <= 512) {
-      auto kern = gate_first ? (acc ? (gs <= 256 ? gated_norm_warp_kernel<B, true, true, 1> : gated_norm_warp_kernel<B, true, true, 2>)
-                                    : (gs <= 256 ? gated_norm_warp_kernel<B, true, false, 1> : gated_norm_warp_kernel<B, true, false, 2>))
-                             : (acc ? (gs <= 256 ? gated_norm_warp_kernel<B, false, true, 1> : gated_norm_warp_kernel<B, false, true, 2>)
-                                    : (gs <= 256 ? gated_norm_warp_kernel<B, false, false, 1> : gated_norm_warp_kernel<B, false, false, 2>));
-      const long long total = rows * groups;
-      DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)((total + 7) / 8)), dim3(256), 0, st, (const B*)y, y_ld, gate, g_ld, w, (B*)out,
-                                      o_ld, gs, groups, total, eps));
-      dlti_count_launch();
-      return 0;
-    }
-    const int vec = gs / 8, threads = vec <= 64 ? 64 : (vec <= 128 ? 128 : (vec <= 512 ? 256 : 512)), vpt = (vec + threads - 1) / threads;
-#define GNV(GF, AC) (vpt <= 1 ? gated_norm_vec_kernel<B, GF, AC, 1> : vpt <= 2 ? gated_norm_vec_kernel<B, GF, AC, 2> \
-                     : gated_norm_vec_kernel<B, GF, AC, 4>)
-    auto kern = gate_first ? (acc ? GNV(true, true) : GNV(true, false)) : (acc ? GNV(false, true) : GNV(false, false));
-#undef GNV
-    DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)rows, groups), dim3(threads), 0, st, (const B*)y, y_ld, gate, g_ld, w, (B*)out,
-                                    o_ld, gs, eps));
-    dlti_count_launch();
-    return 0;
-  }
-  const size_t smem = (size_t)n * 4;
-  if (smem > 48 * 1024) { dlti_set_error("gated_norm: rows of up to 12288 elements"); return DLTI_ERR_TOO_LARGE; }
-#define GN_CASE(GF, AC)                                                                                                          \
-  DISPATCH_T(dtype, DLTI_CUDA_CHECK(dlti_launch_pdl(rows, gated_norm_kernel<T, GF, AC>, dim3((unsigned)rows), dim3(256), smem, st, \
-                                                    (const T*)y, y_ld, gate, g_ld, w, (T*)out, o_ld, n, groups, eps)))
-  if (gate_first && acc) GN_CASE(true, true);
-  else if (gate_first) GN_CASE(true, false);
-  else if (acc) GN_CASE(false, true);
-  else GN_CASE(false, false);
-#undef GN_CASE
-  dlti_count_launch();
-  return 0;
+  if (groups < 1 || n % groups || mode < 0 || mode > 2) return DLTI_ERR_BAD_ARG;
+  if (mode == GATE_SILU_FIRST) return gated_norm_mode<GATE_SILU_FIRST>(y, y_ld, gate, g_ld, w, out, o_ld, rows, n, groups, eps, acc, dtype, st);
+  if (mode == GATE_SILU) return gated_norm_mode<GATE_SILU>(y, y_ld, gate, g_ld, w, out, o_ld, rows, n, groups, eps, acc, dtype, st);
+  return gated_norm_mode<GATE_SIGMOID>(y, y_ld, gate, g_ld, w, out, o_ld, rows, n, groups, eps, acc, dtype, st);
 }
 
 DLTI_API int dlti_qk_norm_rope_cache(const void* proj, long long ld, int oq, int ok, int ov, int og, const float* qn, const float* kn,
@@ -889,6 +985,32 @@ DLTI_API int dlti_qk_norm_rope_cache(const void* proj, long long ld, int oq, int
   const int g = grid_for(tokens * jobs * 32, 256);
   if (acc) DISPATCH_T(dtype, DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, qk_norm_rope_cache_kernel<T, true>, dim3(g), dim3(256), 0, st, p)));
   else DISPATCH_T(dtype, DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, qk_norm_rope_cache_kernel<T, false>, dim3(g), dim3(256), 0, st, p)));
+  dlti_count_launch();
+  return 0;
+}
+
+// bias, qn / kn, first / share, own, kp / vp / dst may be null; see QkvRowParams
+DLTI_API int dlti_qkv_rows(const void* proj, long long ld, int oq, int ok, int ov, const float* bias, const float* qn, const float* kn, float eps,
+                           const void* first, long long f_ld, const float* share, void* own, long long own_ld, const long long* slots, void* kc,
+                           void* vc, int kd, int vd, void* q, long long q_ld, int q_hd, void* kp, void* vp, const int* dst, int nd,
+                           long long tokens, int H, int G, int dim, int vdim, int acc, int dtype, cudaStream_t st) {
+  if (tokens <= 0) return 0;
+  if (H % G || dim < 1 || vdim < 1 || (qn == nullptr) != (kn == nullptr) || (first && !share)) return DLTI_ERR_BAD_ARG;
+  QkvRowParams p{proj, ld, oq, ok, ov, bias, qn, kn, eps, first, f_ld, share, own, own_ld, slots, kc, vc, kd, vd, q, q_ld, q_hd, kp, vp, dst, nd,
+                 H, G, dim, vdim};
+  const size_t smem = (size_t)(H + G) * dim * 4;
+  if (smem > 96 * 1024) { dlti_set_error("qkv_rows: queries and keys of up to 24576 elements"); return DLTI_ERR_TOO_LARGE; }
+  const bool vec = dtype == DLTI_BF16 && ((dim | vdim | oq | ok | ov | kd | vd | q_hd) & 7) == 0 && ((ld | f_ld | own_ld | q_ld) & 7) == 0 &&
+                   ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(first) | reinterpret_cast<uintptr_t>(own) |
+                     reinterpret_cast<uintptr_t>(kc) | reinterpret_cast<uintptr_t>(vc) | reinterpret_cast<uintptr_t>(q) |
+                     reinterpret_cast<uintptr_t>(kp) | reinterpret_cast<uintptr_t>(vp)) & 15) == 0;
+  using B = __nv_bfloat16;
+  auto kern = vec ? (acc ? qkv_rows_kernel<B, true, 8> : qkv_rows_kernel<B, false, 8>)
+                  : dtype == DLTI_BF16 ? (acc ? qkv_rows_kernel<B, true, 1> : qkv_rows_kernel<B, false, 1>)
+                                       : (acc ? qkv_rows_kernel<float, true, 1> : qkv_rows_kernel<float, false, 1>);
+  if (dtype != DLTI_BF16 && dtype != DLTI_FP32) return DLTI_ERR_UNSUPPORTED;
+  if (smem > 48 * 1024) DLTI_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, kern, dim3((unsigned)tokens), dim3(256), smem, st, p));
   dlti_count_launch();
   return 0;
 }
