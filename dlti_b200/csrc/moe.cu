@@ -138,6 +138,7 @@ struct MoeGemmParams {
   int rows, wrows, up, K;                                  // output columns; weight rows of an expert; up > 0: row offset of the up part
   float limit;
   void* out; long long o_ld;
+  int x_rows, o_rows;                                      // list entries outside these are not followed (counters of an aborted step)
   int NT, MT, stages, accs;                                // columns of a tile (multiple of 32, at most 256), weight tiles of an expert
 };
 constexpr int MG_THREADS = 320, MG_W_BYTES = 32768, MG_MAX_STAGES = 8;
@@ -256,7 +257,7 @@ __global__ void __launch_bounds__(MG_THREADS, 1) moe_gemm_kernel(const MoeGemmPa
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int i = min((lane + 32 * y) * 4 + j, x.nn - 1);
-          r[y][j] = p.lists[(long long)x.e * p.cap + x.n0 + i] / p.div;
+          r[y][j] = min((unsigned)p.lists[(long long)x.e * p.cap + x.n0 + i] / p.div, (unsigned)p.x_rows - 1);
         }
       const int w0 = x.e * p.wrows + x.m * (p.up ? 128 : 256), w1 = w0 + (p.up ? p.up : 128);
       for (int kb = 0; kb < nkb; ++kb, ++it) {
@@ -337,6 +338,7 @@ __global__ void __launch_bounds__(MG_THREADS, 1) moe_gemm_kernel(const MoeGemmPa
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
           if (c + j >= x.nn) break;
+          if ((unsigned)dst[c + j] >= (unsigned)p.o_rows) continue;
           __nv_bfloat16* o = out + (long long)dst[c + j] * p.o_ld;
           const float fg = __uint_as_float(g[j]), fu = __uint_as_float(u[j]);
           if (p.up) {
@@ -386,7 +388,8 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restri
       }
       {
         const int i = threadIdx.x, tt = i / 16, k = i % 16;
-        sx[tt][k] = k0 + k < p.K ? X[(long long)(s_pair[tt] / p.div) * x_ld + k0 + k] : 0.f;
+        const unsigned src = min((unsigned)s_pair[tt] / p.div, (unsigned)p.x_rows - 1);
+        sx[tt][k] = k0 + k < p.K ? X[(long long)src * x_ld + k0 + k] : 0.f;
       }
       __syncthreads();
       for (int q = 0; q < parts; ++q) {
@@ -405,7 +408,7 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restri
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int i = tg * 4 + j;
-      if (n0 + i < cnt && r0 + r < p.rows)
+      if (n0 + i < cnt && r0 + r < p.rows && (unsigned)s_pair[i] < (unsigned)p.o_rows)
         reinterpret_cast<float*>(p.out)[(long long)s_pair[i] * p.o_ld + r0 + r] = p.up ? gated(acc[0][j], acc[1][j], p.limit) : acc[0][j];
     }
   }
@@ -450,8 +453,8 @@ DLTI_API int dlti_moe_gemm(const void* X, long long x_ld, long long x_rows, int 
                            const int* lists, const int* counts, int cap, int rows, int up, int K, float limit, void* out, long long o_ld,
                            int o_rows, int dtype, cudaStream_t st) {
   if (o_rows <= 0 || E <= 0) return 0;
-  if (rows < 1 || K < 1 || div < 1 || (up && up < rows) || (up ? up : 0) + rows > wrows) return DLTI_ERR_BAD_ARG;
-  MoeGemmParams p{lists, counts, E, cap, div, rows, wrows, up, K, limit, out, o_ld, 0, 0, 0, 0};
+  if (x_rows < 1 || x_rows > 0x7fffffffLL || rows < 1 || K < 1 || div < 1 || (up && up < rows) || (up ? up : 0) + rows > wrows) return DLTI_ERR_BAD_ARG;
+  MoeGemmParams p{lists, counts, E, cap, div, rows, wrows, up, K, limit, out, o_ld, (int)x_rows, o_rows, 0, 0, 0, 0};
   if (dtype == DLTI_FP32) {
     moe_gemm_f32_kernel<<<dim3((rows + 63) / 64, E), 256, 0, st>>>((const float*)X, x_ld, (const float*)Wt, w_ld, p);
     dlti_count_launch();

@@ -45,7 +45,8 @@ def tanh_between_(x, y, post, pre, dtype, acc=False):
         y = e.shared
     f = _lib.fn("dlti_tanh_between", [_V, _V, _L, _V, _L, _V, _I, _V, _I, _V, _V, _V, _V, _V, _V, _V, _L, _L, _I, _I, _I, _V])
     _lib.check(f(_p(x), _p(y), 0 if y is None else y.stride(0), _p(e.rows) if e else None, e.rows.stride(0) if e else 0,
-                 _p(e.weights) if e else None, e.weights.shape[1] if e else 0, _p(e.counts) if e else None, e.counts.numel() if e else 0,
+                 _p(e.weights) if e else None, e.weights.shape[1] if e else 0, _p(e.counts) if e else None,
+                 e.counts.numel() if e and e.counts is not None else 0,
                  *_three(post), *_three(pre), _p(h), 0 if h is None else h.stride(0), T, d, int(acc and y is not None),
                  _lib.dtype_code(dtype), _lib.stream_ptr()), "tanh_between")
     return h

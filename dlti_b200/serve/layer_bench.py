@@ -1,6 +1,7 @@
 """Serving throughput of a layer-stack family beside the closest other family at equal size, and the time of each kernel of
-the two against its roofline: Sigosun beside Llama (`bench.py --workload sigosun`), Logozen beside Sigosun (`--workload
-logozen`). Random weights; layer sizes of real models.
+the two against its roofline: Sigosun beside Llama (`bench.py --workload sigosun`), Logozen and Latanex beside Sigosun
+(`--workload logozen`, `--workload latanex`). Random weights; layer sizes of real models. A mixture of experts counts with
+the parameters that a token uses.
 
 Steps go through LLMEngine.pack_step / _run_step (packing, host-to-device copy, forward, sampling; decode steps replay
 CUDA graphs), timed with CUDA events. Kernels are timed one call at a time with the L2 overwritten before each."""
@@ -14,14 +15,18 @@ import torch
 
 from ..models.config import LlamaConfig
 from ..models.registry import family_of
+from ..models.latanex import LatanexConfig
 from ..models.logozen import LogozenConfig
 from ..models.sigosun import SigosunConfig
-from ..models.stack import (AttentionMixer, DenseMlp, LatentAttentionMixer, Layer, LightningMixer, Mamba2Mixer, MLstmMixer, Rope,
-                            StackWeights, mixer_sections)
+from ..models.stack import (AttentionMixer, DeltaMixer, DenseMlp, LatentAttentionMixer, Layer, LightningMixer, Mamba2Mixer, MLstmMixer, MoeMlp,
+                            Rope, StackWeights, mixer_sections, mlp_sections, round8)
 from ..ops import _lib
 from ..ops import attention as A
+from ..ops import delta as DR
+from ..ops import dyt as TN
 from ..ops import elementwise as E
 from ..ops import latent as LA
+from ..ops import moe as ME
 from ..ops import serving as S
 from ..ops import stack as K
 from ..ops import streams as HS
@@ -55,6 +60,33 @@ def _logozen(width: int, params: int) -> LogozenConfig:
                              layers=[Layer(mem, ff), Layer(att, ff)] * n, name=f"logozen-{width}x{2 * n}")
     one = cfg(2).num_params() - cfg(1).num_params()
     return cfg(max(1, round(params / one)))
+
+
+def _latanex(width: int, params: int) -> LatanexConfig:
+    """Pairs of layers (delta rule, windowed attention), each with a mixture of experts, of which a token uses about `params`
+    parameters."""
+    heads = width // 128
+    att = AttentionMixer(heads=heads, kv_heads=max(1, heads // 4), dim=128, vdim=128, scale=128 ** -0.5, qk_norm=False, head_gate=False,
+                         window=2048, softcap=30.0, sink=True, bias=True, row_norm=True, v_mix=True)
+    mem = DeltaMixer(heads=heads, kv_heads=heads, dim=128, vdim=128, conv=4)
+    moe = MoeMlp(experts=64, top=8, ff=width // 4, limit=7.0, groups=8, keep=4, scale=2.5, shared_ff=width // 2, shared_limit=7.0)
+
+    def cfg(n):
+        return LatanexConfig(hidden_size=width, vocab_size=32000, norm_eps=1e-6, norm_one_plus=False, tanh_norms=True, embed_scale=4.0,
+                             logit_scale=0.5, layers=[Layer(mem, moe), Layer(att, moe)] * n, name=f"latanex-{width}x{2 * n}")
+    one = active_params(cfg(2)) - active_params(cfg(1))
+    return cfg(max(1, round(params / one)))
+
+
+def active_params(cfg) -> int:
+    """Parameters that one token uses."""
+    idle = [(e.experts - e.top) * 3 * e.ff * cfg.hidden_size for l in getattr(cfg, "layers", []) if isinstance(e := l.mlp, MoeMlp)]
+    return cfg.num_params() - sum(idle)
+
+
+def experts_hit(e: MoeMlp, rows: int) -> float:
+    """Experts that `rows` tokens reach when all are equally likely."""
+    return e.experts * (1 - (1 - e.top / e.experts) ** rows)
 
 
 def _llama(width: int, params: int) -> LlamaConfig:
@@ -107,15 +139,17 @@ def prefill_ms(eng: LLMEngine, nseq: int, length: int, warmup: int, iters: int) 
 def decode_ms(eng: LLMEngine, batch: int, ctx: int, warmup: int, iters: int) -> float:
     bs = eng.blocks.block_size
     per = -(-(ctx + 1) // bs)
+    ids = torch.randint(3, eng.cfg.vocab_size, (batch,)).tolist()
     tabs = [list(range(i * per, (i + 1) * per)) for i in range(batch)]
     slots = [t[ctx // bs] * bs + ctx % bs for t in tabs]
-    step = lambda: eng.pack_step(batch, [5] * batch, [ctx] * batch, slots, [ctx + 1] * batch, tabs, [], 0, _greedy(batch),
+    step = lambda: eng.pack_step(batch, ids, [ctx] * batch, slots, [ctx + 1] * batch, tabs, [], 0, _greedy(batch),
                                  sslots=list(range(batch)))
     return _time(lambda: eng._run_step(step()), warmup, iters)
 
 
 def step_bytes(eng: LLMEngine, batch: int, ctx: int) -> int:
-    """What a decode step must move: every matrix once, the visible keys and values, recurrent states read and written."""
+    """What a decode step must move: every matrix that the rows reach once, the visible keys and values, recurrent states read and
+    written."""
     cfg, w = eng.cfg, eng.w
     size = lambda t: t.numel() * t.element_size()
     n = sum(size(t) for l in w.layers for t in l.values()) + size(w.lm_head)
@@ -123,12 +157,14 @@ def step_bytes(eng: LLMEngine, batch: int, ctx: int) -> int:
         return n + 2 * 2 * cfg.num_hidden_layers * batch * (ctx + 1) * w.KV * cfg.head_dim
     for i, l in enumerate(cfg.layers):
         m = l.mixer
+        if isinstance(l.mlp, MoeMlp):
+            n -= int((1 - experts_hit(l.mlp, batch) / l.mlp.experts) * (size(w.layers[i]["e_up"]) + size(w.layers[i]["e_down"])))
         if eng.states is not None and eng.states.canon[i] is not None:
             n += 2 * batch * size(eng.states.canon[i][:, 0])
         if isinstance(m, LatentAttentionMixer):
             n += 2 * batch * (ctx + 1) * m.cols
         elif isinstance(m, AttentionMixer):
-            seen = ctx + 1 - (ctx // m.chunk * m.chunk if m.chunk else 0)
+            seen = ctx + 1 - (ctx // m.chunk * m.chunk if m.chunk else max(0, ctx + 1 - m.window) if m.window else 0)
             n += 2 * batch * seen * m.kv_heads * (m.dim + m.vdim)
         else:
             n += 2 * batch * 4 * (eng.states.ssm[i][0].numel() + (0 if eng.states.vec[i] is None else eng.states.vec[i][0].numel()))
@@ -393,9 +429,97 @@ def logozen_kernels(width: int, peaks: dict, nseq: int, length: int, batch: int,
     return k.rows
 
 
+def latanex_kernels(width: int, peaks: dict, nseq: int, length: int, batch: int, ctx: int, iters: int) -> list[dict]:
+    """The kernels of Latanex in the same two steps; those of Sigosun come from kernels()."""
+    k = _Kernels(peaks, iters)
+    cfg = _latanex(width, 1)
+    mem, m, e, d, dev, bf = cfg.layers[0].mixer, cfg.layers[1].mixer, cfg.layers[1].mlp, width, "cuda", torch.bfloat16
+    w = StackWeights(cfg, dev, bf).finish()
+    lw, lm = w.layers[1], w.layers[0]
+    rnd = lambda *s: torch.randn(*s, device=dev, dtype=bf)
+    for t in [x[n] for x in w.layers for n in ("w_in", "w_up", "e_up", "e_down", "w_down")]:
+        t.normal_(0, d ** -0.5)
+    T, bs, H, G, hd = nseq * length, 16, m.heads, m.kv_heads, 128
+    per = -(-max(length, ctx + 1) // bs)
+    n_all = max(nseq, batch)
+    tabs = torch.arange(n_all * per, dtype=torch.int32, device=dev).view(n_all, per)
+    kc, vc = rnd(n_all * per, bs, G, hd), rnd(n_all * per, bs, G, hd)
+    pslots = torch.cat([torch.arange(length) + i * per * bs for i in range(nseq)]).to(dev)
+    dslots = torch.tensor([i * per * bs + ctx for i in range(batch)], device=dev)
+    pr = _rows([(0, length)] * nseq, 0, tabs[:nseq].contiguous(), pslots, length)
+    dr = _rows([(ctx, 1)] * batch, batch, tabs[:batch].contiguous(), dslots, ctx + 1)
+    pieces = K.Pieces(torch.tensor([i * length for i in range(nseq + 1)], dtype=torch.int32, device=dev), length, T)
+    run = lambda phase, name, fn, nbytes, flops=0.0: k.run("latanex", phase, name, fn, nbytes, flops)
+    pairs = length * (length + 1) // 2
+    sink, qkv, out = lw["sink"], rnd(T, (H + 2 * G) * hd), K.act(T, H * hd, bf, dev)
+    io, fl = T * (2 * H + 2 * G) * hd * 2, 4.0 * nseq * pairs * H * hd
+    run("prefill", "attention (packed)", lambda: K.packed_attention(qkv, m, pr, pieces, kc, vc, None, sink=sink), io, fl)
+    half = replace(m, window=length // 4)
+    run("prefill", "attention (packed, window of a quarter)", lambda: K.packed_attention(qkv, half, pr, pieces, kc, vc, None, sink=sink), io,
+        4.0 * nseq * (half.window * (half.window + 1) // 2 + (length - half.window) * half.window) * H * hd)
+    q = rnd(T, H * hd)
+    run("prefill", "attention (paged, heads > 128)", lambda: K.attn_paged_prefill(q, m, pr, kc, vc, None, out, sink=sink), io, fl)
+    qd, od = rnd(batch, H * hd), K.act(batch, H * hd, bf, dev)
+    run("decode", "attention", lambda: K.attn_paged_decode(qd, m, dr, kc, vc, None, od, sink=sink), batch * min(ctx + 1, m.window) * G * hd * 4)
+    sec, sm, su, ffr = mixer_sections(m), mixer_sections(mem), mlp_sections(e), round8(e.ff)
+    norms = [(torch.ones(1, device=dev), torch.ones(d, device=dev), torch.zeros(d, device=dev)) for _ in range(2)]
+    qk, vv = mem.kv_heads * mem.dim, mem.heads * mem.vdim
+    for phase, r, n, ns in (("prefill", pr, T, nseq), ("decode", dr, batch, batch)):
+        acc = phase == "decode"
+        es = 8 if acc else 2                                      # accumulators are read and zeroed
+        z = lambda c: torch.zeros(n, c, device=dev) if acc else rnd(n, c)
+        proj, first = z(sec.total), rnd(n, G * hd)
+        run(phase, "bias + row norm + values + cache", lambda: K.qkv_rows(proj, sec, m, lw, 1e-6, r, first, kc, vc, bf, None if acc else pieces, acc),
+            n * (sec.total * es + G * hd * 2 + (H + (0 if acc else 2 * G)) * hd * 2 + 2 * G * hd * 2))
+        x, y, rows_, wt = torch.randn(n, d, device=dev), z(d), rnd(n * e.top, d), torch.rand(n, e.top, device=dev)
+        run(phase, "tanh norms + residual", lambda: TN.tanh_between_(x, y, *norms, bf, acc=acc), n * d * (es + 8 + 2))
+        ex = ME.ExpertSum(rows_, wt, y)
+        run(phase, "sum of experts + tanh norms + residual", lambda: TN.tanh_between_(x, ex, *norms, bf, acc=acc), n * d * (es + 8 + 2 + 2 * e.top))
+        del rows_, ex
+        h, logits = rnd(n, d), torch.randn(n, round8(e.experts), device=dev)
+        counts = ME._counts(torch.device(dev, torch.cuda.current_device()), e.experts)
+
+        def route():
+            counts.zero_()
+            return ME._route(None, logits, 0, lw["correction"], e)
+        run(phase, "routing (and clearing its counters)", route, n * (e.experts * 4 + e.top * 8))
+        wgt, lists, cnt = route()
+        cnt = cnt.clone()
+        counts.zero_()                                            # as the next step wants them
+        hit = int((cnt > 0).sum())
+        a, rows_ = K.act(n * e.top, e.ff, bf, dev), K.act(n * e.top, d, bf, dev)
+        run(phase, "experts in + activation", lambda: ME.grouped_gemm(h, lw["e_up"], lists, cnt, a, rows=e.ff, pairs_per_row=e.top, up=ffr, limit=e.limit),
+            2 * (n * d + hit * 2 * e.ff * d + n * e.top * e.ff), 4.0 * n * e.top * e.ff * d)
+        run(phase, "experts out", lambda: ME.grouped_gemm(a, lw["e_down"], lists, cnt, rows_, rows=d, pairs_per_row=1),
+            2 * (n * e.top * (e.ff + d) + hit * e.ff * d), 2.0 * n * e.top * e.ff * d)
+        del a, rows_
+        p = z(su.total)
+        hs = K.act(n, e.shared_ff, bf, dev)
+        run(phase, "gated activation (shared expert)", lambda: ME._route(p, None, 0, None, None, (su["gate"], su["up"], e.shared_ff, 7.0, hs), acc=acc),
+            n * e.shared_ff * (2 * es + 2))
+        conv, ssm = torch.zeros(ns, mem.conv - 1, sm["g"], device=dev, dtype=bf), torch.zeros(ns, mem.heads, mem.dim, mem.vdim, device=dev)
+        pm, gates = rnd(n, sm["gates"]), torch.randn(n, 2 * mem.heads, device=dev)
+        run(phase, "short conv", lambda: K.short_conv(pm, 0, sm["g"], lm["conv"], w.derived[0]["conv_b"], conv, r, bf), n * sm["g"] * 4)
+        # useful work of the chunked form: products with the state (three), scores of keys and queries, the triangular system, its use
+        work = 2.0 * n * mem.heads * (3 * mem.dim * mem.vdim + 32 * 2 * mem.dim + 32 * 2 * mem.vdim) if not acc else 6.0 * n * mem.heads * mem.dim * mem.vdim
+        run(phase, "delta scan", lambda: DR.delta_scan(pm[:, :qk], pm[:, sm["k"]:sm["k"] + qk], pm[:, sm["v"]:sm["v"] + vv], gates, lm["A_log"], lm["dt_bias"],
+                                                       ssm, r, mem.heads, mem.kv_heads, mem.dim, mem.vdim, conv_src=pm, conv_col=0, conv_state=conv),
+            n * (2 * qk + 2 * vv) * 2 + n * 8 * mem.heads + ns * 8 * ssm[0].numel(), work)
+        yb = rnd(n, vv)
+        run(phase, "head norm + gate", lambda: K.gated_norm(yb, pm[:, sm["g"]:sm["g"] + vv], w.derived[0]["norm"], 1e-6, mem.heads, False, silu=True), n * vv * 6)
+        for name, wm, fn in (("GEMM attention in", lw["w_in"], None), ("GEMM delta in, gates fp32", lm["w_in"], lambda q, t: HS.linear_split(q, t, sm["gates"])),
+                             ("GEMM shared expert, router", lw["w_up"], None)):
+            N_, K_ = wm.shape
+            mm = fn or (gemm_skinny_acc if acc else gemm)
+            run(phase, name, lambda: mm(h, wm), 2 * (n * K_ + N_ * K_) + n * N_ * (4 if acc else 2), 2.0 * n * N_ * K_)
+            if acc and fn is None:
+                gemm_skinny(h, wm)                                # leaves the shared accumulator zero
+    return k.rows
+
+
 def main(steps: int, warmup: int, sizes: str, peaks: dict, sampler, workload: str = "sigosun") -> dict:
     iters, warmup = max(3, steps), max(3, warmup)
-    name, other = ("Logozen", "Sigosun") if workload == "logozen" else ("Sigosun", "Llama")
+    name, other = {"logozen": ("Logozen", "Sigosun"), "latanex": ("Latanex", "Sigosun")}.get(workload, ("Sigosun", "Llama"))
     out = {"metric": f"{name} serving tok/s beside {other} of equal size", "impl": "dlti_b200", "dtype": "bf16",
            "data": "synthetic (random token ids; random-init weights)", "steps": iters, "warmup": warmup, "sizes": [], "kernels": {}}
     _lib.reset_launch_count()
@@ -403,11 +527,12 @@ def main(steps: int, warmup: int, sizes: str, peaks: dict, sampler, workload: st
         width, blocks = (int(x) for x in spec.split("x"))
         sig = _sigosun(width, blocks)
         params = sig.num_params() - 2 * sig.vocab_size * width
-        models = (_logozen(width, params), sig) if workload == "logozen" else (sig, _llama(width, params))
+        models = {"logozen": lambda: (_logozen(width, params), sig), "latanex": lambda: (_latanex(width, params), sig),
+                  "sigosun": lambda: (sig, _llama(width, params))}[workload]()
         row = {"width": width, "rows": []}
         for cfg in models:
             eng = _engine(cfg, 8704, 64)
-            e = {"model": cfg.name, "layers": cfg.num_hidden_layers, "params_m": round(cfg.num_params() / 1e6)}
+            e = {"model": cfg.name, "layers": cfg.num_hidden_layers, "params_m": round(cfg.num_params() / 1e6), "active_params_m": round(active_params(cfg) / 1e6)}
             for nseq, length in ((1, 8192), (4, 2048), (16, 512)):
                 ms = prefill_ms(eng, nseq, length, warmup, iters)
                 e[f"prefill {nseq}x{length}"] = {"ms": round(ms, 3), "tok_s": round(nseq * length / ms * 1e3)}
@@ -420,8 +545,9 @@ def main(steps: int, warmup: int, sizes: str, peaks: dict, sampler, workload: st
             torch.cuda.empty_cache()
         out["sizes"].append(row)
         ks = kernels(width, peaks, 4, 2048, 64, 1000, iters)
-        if workload == "logozen":
-            ks = logozen_kernels(width, peaks, 4, 2048, 64, 1000, iters) + [r for r in ks if r["model"] == "sigosun"]
+        if workload != "sigosun":
+            own = logozen_kernels if workload == "logozen" else latanex_kernels
+            ks = own(width, peaks, 4, 2048, 64, 1000, iters) + [r for r in ks if r["model"] == "sigosun"]
         out["kernels"][str(width)] = ks
         torch.cuda.empty_cache()
     out["gpu_launches"] = _lib.launch_count()
@@ -434,7 +560,8 @@ def main(steps: int, warmup: int, sizes: str, peaks: dict, sampler, workload: st
 def print_tables(out: dict, emit=print) -> None:
     for s in out["sizes"]:
         a, b = s["rows"]
-        emit(f"# {a['model']} ({a['params_m']} M) | {b['model']} ({b['params_m']} M)")
+        size = lambda e: f"{e['model']} ({e['params_m']} M" + (")" if e["active_params_m"] == e["params_m"] else f", {e['active_params_m']} M a token)")
+        emit(f"# {size(a)} | {size(b)}")
         for key in a:
             if isinstance(a[key], dict):
                 emit(f"{key:20s} {a[key]['ms']:9.3f} ms {a[key]['tok_s']:9d} tok/s | {b[key]['ms']:9.3f} ms {b[key]['tok_s']:9d} tok/s | "
@@ -442,7 +569,7 @@ def print_tables(out: dict, emit=print) -> None:
     for w, rows in out["kernels"].items():
         emit(f"# kernels, width {w}")
         for r in rows:
-            emit(f"{r['model']:8s} {r['phase']:8s} {r['kernel']:30s} {r['us']:9.2f} us, roof {r['roof_us']:8.2f} us = {r['frac_of_roof']:.3f} ({r['bound']})")
+            emit(f"{r['model']:8s} {r['phase']:8s} {r['kernel']:40s} {r['us']:9.2f} us, roof {r['roof_us']:8.2f} us = {r['frac_of_roof']:.3f} ({r['bound']})")
 
 
 def run_cli(steps: int, warmup: int, sizes: str, peaks: dict, sampler, workload: str) -> None:
