@@ -14,11 +14,15 @@ namespace {
 
 struct Norm { const float *alpha, *w, *b; };
 
-// 16-bit results come from 1 - 2 / (1 + e^(2 z)), whose absolute error is about 1e-7
-template <typename T>
-__device__ __forceinline__ float tanh_t(float z) {
-  if constexpr (sizeof(T) == 4) return tanhf(z);
-  else return 1.f - __fdividef(2.f, 1.f + __expf(2.f * z));
+__device__ __forceinline__ float rcp_approx(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 template <typename T, int W>
 __device__ __forceinline__ void norm_piece(const Norm& n, float alpha, int c, const float (&x)[W], float (&out)[W]) {
@@ -30,8 +34,14 @@ __device__ __forceinline__ void norm_piece(const Norm& n, float alpha, int c, co
 #pragma unroll
     for (int j = 0; j < W; ++j) { w[j] = n.w[c + j]; b[j] = n.b[c + j]; }
   }
+  if constexpr (sizeof(T) == 4) {
 #pragma unroll
-  for (int j = 0; j < W; ++j) out[j] = fmaf(tanh_t<T>(alpha * x[j]), w[j], b[j]);
+    for (int j = 0; j < W; ++j) out[j] = fmaf(tanhf(alpha * x[j]), w[j], b[j]);
+  } else {                                                 // tanh z = 1 - 2 / (1 + e^(2 z)): absolute error about 1e-7
+    const float a = 2.f * 1.4426950408889634f * alpha;
+#pragma unroll
+    for (int j = 0; j < W; ++j) out[j] = fmaf(-2.f * w[j], rcp_approx(1.f + ex2_approx(a * x[j])), w[j] + b[j]);
+  }
 }
 template <typename T, bool ACC, int W>
 __device__ __forceinline__ void load_piece(const void* row, int c, float (&f)[W]) {
@@ -86,7 +96,7 @@ struct Between {
   void* h; long long h_ld;
   int d;
 };
-constexpr int TB_ROWS = 4;                                 // tokens per thread: the norm vectors are loaded once
+constexpr int TB_ROWS = 2;                                 // tokens per thread: the norm vectors are loaded once
 template <typename T, bool ACC, int W, int ROWS>
 __global__ void __launch_bounds__(128) tanh_between_kernel(const Between p, long long tokens) {
   const int c = (blockIdx.y * 128 + threadIdx.x) * W;

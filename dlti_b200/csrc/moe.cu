@@ -3,13 +3,15 @@
 //   moe_route        one warp per token: sigmoid scores, groups, the top experts and their weights; every (token, choice) pair
 //                    = token * top + choice is appended to its expert's list. Further blocks of the same launch apply a gated
 //                    activation to other columns of the same projection (the shared expert).
-//   moe_gemm         grouped GEMM over the lists, bf16: weights are the 128-row operand of tcgen05.mma and the pairs of a list its
-//                    columns (16 to 256 of them), so one kernel serves one decoded token and whole prompts. Source rows come by
-//                    TMA gather (four rows a copy), results go to row `pair` of the output. Two accumulators share a tile's
-//                    columns: the gate and the up rows, whose activation is the epilogue, or two neighbouring row tiles.
+//   moe_gemm         grouped GEMM over the lists, bf16, by CTA pairs: weights are the 256-row operand of tcgen05.mma and the
+//                    pairs of a list its columns (32 to 256 of them), so one kernel serves one decoded token and whole
+//                    prompts. The first GEMM of an expert gathers the pairs' source rows and leaves its results one list after
+//                    the other; the second reads them as they lie and scatters to row `pair`. Gate and up rows alternate in the
+//                    first one's weights, so that the activation is an exchange between neighbouring lanes of the epilogue.
 //   moe_gemm_f32     the same in fp32 FMAs
 //
 // Pair lists are filled with atomics, so their order differs from run to run; a pair's result does not depend on its place.
+#include "pair.cuh"
 #include "rows.cuh"
 
 namespace {
@@ -38,19 +40,35 @@ struct RouteParams {
 };
 constexpr int ROUTE_WARPS = 4;
 
-template <bool ACC>
-__device__ void route_token(const RouteParams& p, long long t, float* sc, float* sp, float* sg, int* sel) {
+__device__ __forceinline__ unsigned ordered(float v) {     // unsigned integers in the order of the floats
+  const unsigned u = __float_as_uint(v);
+  return u & 0x80000000u ? ~u : u | 0x80000000u;
+}
+// Expert choice of one token by one warp, R scores a lane. sc: choice scores, sg: group scores (shared memory); sel / share: the
+// chosen experts and their scores.
+template <bool ACC, int R>
+__device__ __forceinline__ void route_token(const RouteParams& p, long long t, float* sc, float* sg, int* sel, float* share) {
   const int lane = threadIdx.x & 31, n = p.E / p.groups;
   const float* zr = p.z + t * p.z_ld + p.col;
-  for (int e = lane; e < p.E; e += 32) {
-    float v = zr[e];
-    if (ACC) const_cast<float*>(zr)[e] = 0.f;
-    v = sigmoid_f(v);
-    sp[e] = v;
-    sc[e] = v + p.corr[e];
+  float s[R], c[R];
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int e = lane + 32 * i;
+    s[i] = 0.f;
+    c[i] = -INFINITY;
+    if (e < p.E) {
+      const float v = zr[e];
+      if (ACC) const_cast<float*>(zr)[e] = 0.f;
+      s[i] = sigmoid_f(v);
+      c[i] = s[i] + p.corr[e];
+    }
   }
-  __syncwarp();
   if (p.keep < p.groups) {
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+      if (lane + 32 * i < p.E) sc[lane + 32 * i] = c[i];
+    __syncwarp();
     for (int g = lane; g < p.groups; g += 32) {            // a group's score: its two largest choice scores
       float a = -INFINITY, b = -INFINITY;
       for (int e = g * n; e < (g + 1) * n; ++e) {
@@ -61,53 +79,82 @@ __device__ void route_token(const RouteParams& p, long long t, float* sc, float*
       sg[g] = n > 1 ? a + b : a;
     }
     __syncwarp();
-    for (int g = lane; g < p.groups; g += 32) {
-      int better = 0;
-      for (int o = 0; o < p.groups; ++o) better += sg[o] > sg[g] || (sg[o] == sg[g] && o < g);
-      if (better >= p.keep)
-        for (int e = g * n; e < (g + 1) * n; ++e) sc[e] = -INFINITY;
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const int e = lane + 32 * i;
+      if (e < p.E) {
+        const int g = e / n;
+        int better = 0;
+        for (int o = 0; o < p.groups; ++o) better += sg[o] > sg[g] || (sg[o] == sg[g] && o < g);
+        if (better >= p.keep) c[i] = -INFINITY;
+      }
     }
-    __syncwarp();
   }
   float sum = 0.f;
   for (int k = 0; k < p.top; ++k) {
-    float best = -INFINITY;
+    unsigned best = 0;
     int bi = p.E;
-    for (int e = lane; e < p.E; e += 32)
-      if (sc[e] > best) { best = sc[e]; bi = e; }
+    float bs = 0.f;
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float v = __shfl_xor_sync(0xffffffffu, best, o);
-      const int i = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (v > best || (v == best && i < bi)) { best = v; bi = i; }
+    for (int i = 0; i < R; ++i) {
+      const unsigned o = c[i] == -INFINITY ? 0u : ordered(c[i]);
+      if (o > best) { best = o; bi = lane + 32 * i; bs = s[i]; }
     }
-    if (bi >= p.E) bi = k;                                 // only where the scores are not numbers
+    const unsigned top = __reduce_max_sync(0xffffffffu, best);
+    int e = (int)__reduce_min_sync(0xffffffffu, best == top && bi < p.E ? (unsigned)bi : 0x7fffffffu);
+    if (e >= p.E) e = k;                                   // only where the scores are not numbers
+    bs = __shfl_sync(0xffffffffu, bi == e ? bs : 0.f, e & 31);
+    if ((e & 31) == lane)
+#pragma unroll
+      for (int i = 0; i < R; ++i)
+        if (e == lane + 32 * i) c[i] = -INFINITY;
     if (lane == 0) {
-      sel[k] = bi;
-      sc[bi] = -INFINITY;
+      sel[k] = e;
+      share[k] = bs;
     }
-    sum += sp[bi];
-    __syncwarp();
+    sum += bs;
   }
+  __syncwarp();
   const float f = p.scale / (sum + 1e-20f);
-  for (int k = lane; k < p.top; k += 32) {
-    const int e = sel[k];
-    p.wgt[t * p.top + k] = sp[e] * f;
-    const int r = atomicAdd(p.counts + e, 1);
-    if (r < p.T) p.lists[e * p.T + r] = (int)(t * p.top + k);
+  for (int k = lane; k < p.top; k += 32) p.wgt[t * p.top + k] = share[k] * f;
+}
+
+// A block routes `per` tokens a warp, counts its pairs in shared memory and takes its places in the lists with one atomic per expert.
+template <bool ACC, int R>
+__device__ __forceinline__ void route_block(const RouteParams& p, int per) {
+  extern __shared__ float route_s[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tokens = ROUTE_WARPS * per;
+  int* cnt = reinterpret_cast<int*>(route_s);              // [E] pairs of this block, then their first place
+  int* sel = cnt + p.E;                                    // [tokens][top]
+  int* rank = sel + tokens * p.top;                        // [tokens][top] (scores first)
+  float* sc = reinterpret_cast<float*>(rank + tokens * p.top) + warp * (p.E + p.groups);
+  for (int e = threadIdx.x; e < p.E; e += blockDim.x) cnt[e] = 0;
+  __syncthreads();
+  const long long t0 = (long long)blockIdx.x * tokens;
+  for (int i = 0; i < per; ++i) {
+    const int x = warp * per + i;
+    if (t0 + x >= p.T) break;
+    route_token<ACC, R>(p, t0 + x, sc, sc + p.E, sel + x * p.top, reinterpret_cast<float*>(rank + x * p.top));
+    __syncwarp();
+    for (int k = lane; k < p.top; k += 32) rank[x * p.top + k] = atomicAdd(cnt + sel[x * p.top + k], 1);
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < p.E; e += blockDim.x)
+    if (cnt[e]) cnt[e] = atomicAdd(p.counts + e, cnt[e]);
+  __syncthreads();
+  const int n = (int)min((long long)tokens, p.T - t0) * p.top;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const int e = sel[i], r = cnt[e] + rank[i];
+    if ((unsigned)r < (unsigned)p.T) p.lists[e * p.T + r] = (int)(t0 * p.top + i);
   }
 }
 
-template <typename T, bool ACC, int W>
-__global__ void __launch_bounds__(32 * ROUTE_WARPS) moe_route_kernel(const RouteParams p, int route_blocks) {
-  extern __shared__ float route_s[];
+template <typename T, bool ACC, int W, int R>
+__global__ void __launch_bounds__(32 * ROUTE_WARPS) moe_route_kernel(const RouteParams p, int route_blocks, int route_per) {
   griddep_wait();
   griddep_launch();
   if ((int)blockIdx.x < route_blocks) {
-    const int warp = threadIdx.x >> 5;
-    const long long t = (long long)blockIdx.x * ROUTE_WARPS + warp;
-    float* s = route_s + warp * (2 * p.E + p.groups + p.top);
-    if (t < p.T) route_token<ACC>(p, t, s, s + p.E, s + 2 * p.E, reinterpret_cast<int*>(s + 2 * p.E + p.groups));
+    route_block<ACC, R>(p, route_per);
     return;
   }
   const int per = p.ff / W;
@@ -135,19 +182,25 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) moe_route_kernel(const Route
 struct MoeGemmParams {
   const int *lists, *counts;
   int E, cap, div;                                         // experts; capacity of a list; pairs per source row
-  int rows, wrows, up, K;                                  // output columns; weight rows of an expert; up > 0: row offset of the up part
+  int rows, wrows, K;                                      // output columns; weight rows of an expert
   float limit;
   void* out; long long o_ld;
   int x_rows, o_rows;                                      // list entries outside these are not followed (counters of an aborted step)
-  int NT, MT, stages, accs;                                // columns of a tile (multiple of 32, at most 256), weight tiles of an expert
+  int NT, MT, stages;                                      // columns of a tile (multiple of 32, at most 256), weight tiles of an expert
 };
-constexpr int MG_THREADS = 320, MG_W_BYTES = 32768, MG_MAX_STAGES = 8;
+// UP: the source of list entry i is row lists[i] / div, its result (activation of rows 2 r and 2 r + 1) goes to row (start of the
+// list) + i. Otherwise the source is row (start of the list) + i and the result goes to row lists[i].
+constexpr int MG_GATHERS = 8, MG_THREADS = 320 + 32 * MG_GATHERS, MG_A_BYTES = 16384, MG_MAX_STAGES = 10, MG_SMEM = 226 * 1024;
+constexpr int MG_TAIL = 8 * (2 * MG_MAX_STAGES + 4) + 16;  // barriers, TMEM address
 constexpr long long MG_WAIT_LIMIT = 4000000000LL;
 
-__device__ __forceinline__ void tma_gather4(uint32_t dst, const CUtensorMap* m, uint32_t bar, int c, int r0, int r1, int r2, int r3) {
-  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile::gather4.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6, %7}], [%2];" ::"r"(dst),
-               "l"(reinterpret_cast<uint64_t>(m)), "r"(bar), "r"(c), "r"(r0), "r"(r1), "r"(r2), "r"(r3)
-               : "memory");
+// rows r0 .. r3 of a matrix (box of one row) one after the other; completion bytes on a barrier that may live in the peer CTA
+__device__ __forceinline__ void tma_gather4_2sm(uint32_t dst, const CUtensorMap* m, uint32_t bar_cluster, int c, int r0, int r1, int r2, int r3) {
+  asm volatile(
+      "cp.async.bulk.tensor.2d.shared::cluster.global.tile::gather4.mbarrier::complete_tx::bytes.cta_group::2 "
+      "[%0], [%1, {%3, %4, %5, %6, %7}], [%2];" ::"r"(dst),
+      "l"(reinterpret_cast<uint64_t>(m)), "r"(bar_cluster), "r"(c), "r"(r0), "r"(r1), "r"(r2), "r"(r3)
+      : "memory");
 }
 
 struct MoeTile { int e, m, n0, nn; };
@@ -160,79 +213,88 @@ __device__ __forceinline__ MoeTile moe_tile(const MoeGemmParams& p, const int* f
     else hi = mid - 1;
   }
   const int r = t - first[lo], c = cnt[lo];
-  const int nt = (c + p.NT - 1) / p.NT, per = ((c + nt - 1) / nt + 15) & ~15;
+  const int nt = (c + p.NT - 1) / p.NT, per = ((c + nt - 1) / nt + 31) & ~31;
   const int n0 = (r / p.MT) * per;
   return MoeTile{lo, r % p.MT, n0, min(c - n0, per)};
 }
 
-// warp 0: copies (lane 0 the weights, every lane its rows), warp 1: MMAs, warps 2-9: epilogue. Waits are bounded: a CTA that gives
-// up writes NaN.
-__global__ void __launch_bounds__(MG_THREADS, 1) moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw,
-                                                                 const __grid_constant__ CUtensorMap tx) {
+// A CTA of the pair stages 128 weight rows and half of the tile's columns; the leader issues the MMAs, and each CTA ends up with its
+// 128 rows of the accumulator (two of them, so that the epilogue overlaps the next tile). Warp 0: weights; warp 1: MMAs; warps 2-9:
+// epilogue; warps 10-17: the gathered columns, four rows a copy (a copy costs its issuing thread about 100 clk, so they share them),
+// or warp 10 where they lie together. Waits are bounded: a CTA that gives up writes NaN.
+template <bool UP>
+__global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(MG_THREADS, 1)
+moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, const __grid_constant__ CUtensorMap tx) {
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
-  const uint32_t stage_bytes = MG_W_BYTES + p.NT * 128;
-  const uint32_t bars = base + p.stages * stage_bytes;     // full[stages], empty[stages], acc_full[2], acc_empty[2], TMEM address
-  const uint32_t full = bars, empty = full + 8 * MG_MAX_STAGES, acc_full = empty + 8 * MG_MAX_STAGES, acc_empty = acc_full + 16, slot = acc_empty + 16;
+  const uint32_t stage_bytes = MG_A_BYTES + p.NT * 64;
+  const uint32_t full = base + p.stages * stage_bytes, empty = full + 8 * MG_MAX_STAGES, acc_full = empty + 8 * MG_MAX_STAGES,
+                 acc_empty = acc_full + 16, slot = acc_empty + 16;
   uint8_t* tail = smem_raw + (slot - smem_u32(smem_raw)) + 16;
   volatile uint32_t* slot_ptr = reinterpret_cast<volatile uint32_t*>(tail - 16);
   int* s_dst = reinterpret_cast<int*>(tail);               // [2][256]
-  int* s_first = s_dst + 512;                              // [E + 1]
-  int* s_cnt = s_first + p.E + 1;                          // [E]
-  __shared__ int s_scan[32], s_fail;
+  int* s_first = s_dst + 512;                              // [E]: tiles before an expert
+  int* s_row = s_first + p.E;                              // [E]: pairs before an expert
+  int* s_cnt = s_row + p.E;                                // [E]
+  __shared__ int2 s_scan[32];
+  __shared__ int s_fail;
   const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;
+  const uint32_t rank = __shfl_sync(0xffffffffu, cluster_ctarank(), 0);
+  const int cid = blockIdx.x >> 1, ncl = gridDim.x >> 1;
   if (threadIdx.x == 0) {
     tma_prefetch_desc(&tw);
     tma_prefetch_desc(&tx);
     s_fail = 0;
     for (int s = 0; s < p.stages; ++s) {
-      mbar_init(full + 8 * s, 1);
+      mbar_init(full + 8 * s, 1);                          // the leader's: bytes of both CTAs
       mbar_init(empty + 8 * s, 1);
     }
     for (int a = 0; a < 2; ++a) {
       mbar_init(acc_full + 8 * a, 1);
-      mbar_init(acc_empty + 8 * a, 8);
+      mbar_init(acc_empty + 8 * a, 16);                    // the leader's: eight warps of both CTAs
     }
     mbar_fence_init();
   }
-  if (warp == 1) {
-    tmem_alloc(slot, 512);
-    tmem_relinquish();
-  }
   griddep_wait();
   griddep_launch();
-  // tiles before every expert: a block-wide prefix sum, MG_THREADS experts at a time
-  int carry = 0;
+  cluster_sync_all();
+  if (warp == 1) {
+    tmem_alloc2(slot, 512);
+    tmem_relinquish2();
+  }
+  // tiles and pairs before every expert: a block-wide prefix sum, MG_THREADS experts at a time
+  int2 carry = make_int2(0, 0);
   for (int e0 = 0; e0 < p.E; e0 += MG_THREADS) {
     const int e = e0 + threadIdx.x;
-    const int c = e < p.E ? min(p.counts[e], p.cap) : 0;
+    const int c = e < p.E ? max(0, min(p.counts[e], p.cap)) : 0;
     const int v = (c + p.NT - 1) / p.NT * p.MT;
-    int x = v;
+    int x = v, y = c;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const int y = __shfl_up_sync(0xffffffffu, x, o);
-      if (lane >= o) x += y;
+      const int xo = __shfl_up_sync(0xffffffffu, x, o), yo = __shfl_up_sync(0xffffffffu, y, o);
+      if (lane >= o) { x += xo; y += yo; }
     }
-    if (lane == 31) s_scan[warp] = x;
+    if (lane == 31) s_scan[warp] = make_int2(x, y);
     __syncthreads();
-    int before = carry, all = 0;
+    int2 before = carry;
     for (int w = 0; w < MG_THREADS / 32; ++w) {
-      if (w < warp) before += s_scan[w];
-      all += s_scan[w];
+      if (w < warp) { before.x += s_scan[w].x; before.y += s_scan[w].y; }
+      carry.x += s_scan[w].x;
+      carry.y += s_scan[w].y;
     }
     if (e < p.E) {
       s_cnt[e] = c;
-      s_first[e] = before + x - v;
+      s_first[e] = before.x + x - v;
+      s_row[e] = before.y + y - c;
     }
-    carry += all;
     __syncthreads();
   }
-  const int total = carry;
+  const int total = carry.x;
   tc_fence_before();
-  __syncthreads();
+  cluster_sync_all();
   tc_fence_after();
   const uint32_t tmem = __shfl_sync(0xffffffffu, *slot_ptr, 0);
-  const int nkb = (p.K + 63) / 64, off1 = p.accs == 2 ? 128 : 256;
+  const int nkb = (p.K + 63) / 64;
   volatile int* fail = &s_fail;
   auto wait = [&](uint32_t bar, uint32_t parity) {
     if (mbar_try_wait(bar, parity)) return true;
@@ -244,115 +306,152 @@ __global__ void __launch_bounds__(MG_THREADS, 1) moe_gemm_kernel(const MoeGemmPa
       }
     return true;
   };
+  const uint32_t lead_full = mapa_rank(full, 0);
 
-  if (warp == 0) {
-    int it = 0;                                            // k blocks so far
-    for (int t = blockIdx.x; t < total; t += gridDim.x) {
-      const MoeTile x = moe_tile(p, s_first, s_cnt, t);
-      if (x.nn <= 0) continue;
-      const int groups = (x.nn + 3) >> 2;
-      int r[2][4];
-#pragma unroll
-      for (int y = 0; y < 2; ++y)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const int i = min((lane + 32 * y) * 4 + j, x.nn - 1);
-          r[y][j] = min((unsigned)p.lists[(long long)x.e * p.cap + x.n0 + i] / p.div, (unsigned)p.x_rows - 1);
+  if (warp == 0 || (!UP && warp == 10)) {
+    if (lane == 0) {
+      int s = 0, round = 0;
+      for (int t = cid; t < total && !*fail; t += ncl) {
+        const MoeTile x = moe_tile(p, s_first, s_cnt, t);
+        if (x.nn <= 0) continue;
+        const int w0 = x.e * p.wrows + x.m * 256 + (int)rank * 128;
+        const int nh = ((x.nn + 31) & ~31) >> 1, r0 = s_row[x.e] + x.n0 + (int)rank * nh;
+        const int groups = ((min(nh, x.nn) + 3) >> 2) + ((max(0, x.nn - nh) + 3) >> 2);
+        for (int kb = 0; kb < nkb; ++kb) {
+          if (round > 0 && !wait(empty + 8 * s, (round - 1) & 1)) break;
+          const uint32_t dst = base + s * stage_bytes, bar = lead_full + 8 * s;
+          if (warp == 0) {
+            if (rank == 0) mbar_expect_tx(full + 8 * s, 2 * MG_A_BYTES + (UP ? groups * 512 : p.NT * 128));
+            tma_load_2d_2sm(dst, &tw, bar, kb * 64, w0);
+          } else {
+            tma_load_2d_2sm(dst + MG_A_BYTES, &tx, bar, kb * 64, r0);
+          }
+          if (++s == p.stages) { s = 0; ++round; }
         }
-      const int w0 = x.e * p.wrows + x.m * (p.up ? 128 : 256), w1 = w0 + (p.up ? p.up : 128);
-      for (int kb = 0; kb < nkb; ++kb, ++it) {
-        const int s = it % p.stages;
-        if (it >= p.stages && !wait(empty + 8 * s, (it / p.stages - 1) & 1)) break;
-        const uint32_t dst = base + s * stage_bytes, bar = full + 8 * s;
-        if (lane == 0) {
-          mbar_expect_tx(bar, MG_W_BYTES + groups * 512);
-          tma_load_2d(dst, &tw, bar, kb * 64, w0);
-          tma_load_2d(dst + 16384, &tw, bar, kb * 64, w1);
-        }
-        __syncwarp();
-#pragma unroll
-        for (int y = 0; y < 2; ++y)
-          if (lane + 32 * y < groups)
-            tma_gather4(dst + MG_W_BYTES + (lane + 32 * y) * 512, &tx, bar, kb * 64, r[y][0], r[y][1], r[y][2], r[y][3]);
       }
-      if (*fail) break;
     }
   } else if (warp == 1) {
-    const bool leader = elect_one_sync();
-    int it = 0, tile = 0;
-    for (int t = blockIdx.x; t < total; t += gridDim.x) {
-      const MoeTile x = moe_tile(p, s_first, s_cnt, t);
-      if (x.nn <= 0) continue;
-      const int a = p.accs == 2 ? tile & 1 : 0, use = p.accs == 2 ? tile >> 1 : tile;
-      if (use > 0 && !wait(acc_empty + 8 * a, (use - 1) & 1)) break;
-      tc_fence_after();
-      const uint32_t idesc = umma_idesc_f16(DLTI_BF16, 128, (x.nn + 15) & ~15, false, false);
-      const uint32_t d0 = tmem + a * 256, d1 = d0 + off1;
-      for (int kb = 0; kb < nkb; ++kb, ++it) {
-        const int s = it % p.stages;
-        if (!wait(full + 8 * s, (it / p.stages) & 1)) break;
+    if (rank == 0) {
+      const bool leader = elect_one_sync();
+      int s = 0, round = 0, tile = 0;
+      for (int t = cid; t < total && !*fail; t += ncl) {
+        const MoeTile x = moe_tile(p, s_first, s_cnt, t);
+        if (x.nn <= 0) continue;
+        const int a = tile & 1, use = tile >> 1;
+        if (use > 0 && !wait(acc_empty + 8 * a, (use - 1) & 1)) break;
         tc_fence_after();
-        const uint32_t sm = base + s * stage_bytes;
-        const DescLoHi da = desc_split(sm, 0, 1024), dc = desc_split(sm + 16384, 0, 1024), db = desc_split(sm + MG_W_BYTES, 0, 1024);
-        if (leader) {
+        const uint32_t idesc = umma_idesc_f16(DLTI_BF16, 256, (x.nn + 31) & ~31, false, false), d = tmem + a * 256;
+        for (int kb = 0; kb < nkb; ++kb) {
+          if (!wait(full + 8 * s, round & 1)) break;
+          tc_fence_after();
+          const uint32_t sm = base + s * stage_bytes;
+          const DescLoHi da = desc_split(sm, 0, 1024), db = desc_split(sm + MG_A_BYTES, 0, 1024);
+          if (leader) {
 #pragma unroll
-          for (int kk = 0; kk < 4; ++kk) umma_f16_ss(d0, da.at(kk * 32), db.at(kk * 32), idesc, kb > 0 || kk > 0);
-#pragma unroll
-          for (int kk = 0; kk < 4; ++kk) umma_f16_ss(d1, dc.at(kk * 32), db.at(kk * 32), idesc, kb > 0 || kk > 0);
-          umma_commit(empty + 8 * s);
+            for (int kk = 0; kk < 4; ++kk) umma_f16_ss_2sm(d, da.at(kk * 32), db.at(kk * 32), idesc, kb > 0 || kk > 0);
+            umma_commit_2sm(empty + 8 * s);
+            if (kb == nkb - 1) umma_commit_2sm(acc_full + 8 * a);
+          }
+          __syncwarp();
+          if (++s == p.stages) { s = 0; ++round; }
         }
-        __syncwarp();
+        ++tile;
       }
-      if (*fail) break;
-      if (leader) umma_commit(acc_full + 8 * a);
-      __syncwarp();
-      ++tile;
     }
-  } else {
+  } else if (warp < 10) {
     const int quarter = warp & 3, half = (warp - 2) >> 2;
+    const uint32_t lead_empty = mapa_rank(acc_empty, 0);
     int tile = 0;
-    for (int t = blockIdx.x; t < total; t += gridDim.x) {
+    for (int t = cid; t < total; t += ncl) {
       const MoeTile x = moe_tile(p, s_first, s_cnt, t);
       if (x.nn <= 0) continue;
-      const int a = p.accs == 2 ? tile & 1 : 0, use = p.accs == 2 ? tile >> 1 : tile;
-      int* dst = s_dst + (tile & 1) * 256;
+      const int a = tile & 1, use = tile >> 1;
+      int* dst = s_dst + a * 256;
       const int i0 = threadIdx.x - 64;
-      if (i0 < x.nn) dst[i0] = p.lists[(long long)x.e * p.cap + x.n0 + i0];
+      if (i0 < x.nn) dst[i0] = UP ? s_row[x.e] + x.n0 + i0 : p.lists[(long long)x.e * p.cap + x.n0 + i0];
       asm volatile("bar.sync 1, 256;" ::: "memory");
       const bool ok = wait(acc_full + 8 * a, use & 1);
       tc_fence_after();
-      const uint32_t d0 = tmem + ((uint32_t)(quarter * 32) << 16) + a * 256;
-      const int row0 = x.m * (p.up ? 128 : 256) + quarter * 32 + lane;
-      __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + row0;
-      const bool ok0 = row0 < p.rows, ok1 = row0 + 128 < p.rows;
-      for (int c = half * 16; c < x.nn; c += 32) {
-        uint32_t g[16], u[16];
+      const uint32_t d = tmem + ((uint32_t)(quarter * 32) << 16) + a * 256;
+      const int row = x.m * 256 + (int)rank * 128 + quarter * 32 + lane;
+      // Each round of exchanges hands half of a lane's columns to the lane next to it (then two, then four away) for half of that
+      // one's rows: at the end lane l has column l % 8 of eight neighbouring rows, and stores them in one piece.
+      const int b0 = lane & 1, b1 = lane & 2, b2 = lane & 4, r0 = row & ~7;
+      auto swap_f = [&](bool odd, float a, float b, int d) { return __shfl_xor_sync(0xffffffffu, odd ? a : b, d); };
+      auto swap_u = [&](bool odd, uint32_t a, uint32_t b, int d) { return __shfl_xor_sync(0xffffffffu, odd ? a : b, d); };
+      using B = __nv_bfloat16;
+      for (int c = half * 32; c < x.nn; c += 64) {
+        uint32_t v[32];
         if (ok) {
-          tmem_ld_32x32b_x16(d0 + c, g);
-          tmem_ld_32x32b_x16(d0 + off1 + c, u);
+          tmem_ld_32x32b_x32(d + c, v);
           tmem_wait_ld();
         } else {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) g[j] = u[j] = 0x7fffffffu;
+          for (int j = 0; j < 32; ++j) v[j] = 0x7fffffffu;
         }
 #pragma unroll
-        for (int j = 0; j < 16; ++j) {
-          if (c + j >= x.nn) break;
-          if ((unsigned)dst[c + j] >= (unsigned)p.o_rows) continue;
-          __nv_bfloat16* o = out + (long long)dst[c + j] * p.o_ld;
-          const float fg = __uint_as_float(g[j]), fu = __uint_as_float(u[j]);
-          if (p.up) {
-            if (ok0) *o = __float2bfloat16(gated_fast(fg, fu, p.limit));
+        for (int j = 0; j < 32; j += 8) {
+          const int i = c + j + (lane & 7), to = dst[i & 255];      // stale past the tile's columns
+          B* out = reinterpret_cast<B*>(p.out) + (long long)to * p.o_ld;
+          const bool on = i < x.nn && (unsigned)to < (unsigned)p.o_rows;
+          if constexpr (UP) {                              // even lanes hold gates, odd lanes up values
+            float f[4];
+#pragma unroll
+            for (int y = 0; y < 4; ++y) {
+              const float v0 = __uint_as_float(v[j + 2 * y]), v1 = __uint_as_float(v[j + 2 * y + 1]), other = swap_f(b0, v0, v1, 1);
+              f[y] = gated_fast(b0 ? other : v0, b0 ? v1 : other, p.limit);
+            }
+            uint32_t u[2];
+#pragma unroll
+            for (int y = 0; y < 2; ++y) {
+              const float other = swap_f(b1, f[2 * y], f[2 * y + 1], 2);
+              u[y] = b1 ? Cvt<B>::pack2(other, f[2 * y + 1]) : Cvt<B>::pack2(f[2 * y], other);
+            }
+            const uint32_t other = swap_u(b2, u[0], u[1], 4);
+            if (on && r0 / 2 < p.rows) *reinterpret_cast<uint2*>(out + r0 / 2) = b2 ? make_uint2(other, u[1]) : make_uint2(u[0], other);
           } else {
-            if (ok0) *o = __float2bfloat16(fg);
-            if (ok1) o[128] = __float2bfloat16(fu);
+            uint32_t u[4];
+#pragma unroll
+            for (int y = 0; y < 4; ++y) {
+              const float v0 = __uint_as_float(v[j + 2 * y]), v1 = __uint_as_float(v[j + 2 * y + 1]), other = swap_f(b0, v0, v1, 1);
+              u[y] = b0 ? Cvt<B>::pack2(other, v1) : Cvt<B>::pack2(v0, other);
+            }
+            uint2 w[2];
+#pragma unroll
+            for (int y = 0; y < 2; ++y) {
+              const uint32_t other = swap_u(b1, u[2 * y], u[2 * y + 1], 2);
+              w[y] = b1 ? make_uint2(other, u[2 * y + 1]) : make_uint2(u[2 * y], other);
+            }
+            const uint32_t o0 = swap_u(b2, w[0].x, w[1].x, 4), o1 = swap_u(b2, w[0].y, w[1].y, 4);
+            if (on && r0 < p.rows) *reinterpret_cast<uint4*>(out + r0) = b2 ? make_uint4(o0, o1, w[1].x, w[1].y) : make_uint4(w[0].x, w[0].y, o0, o1);
           }
         }
       }
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(acc_empty + 8 * a);
+      if (lane == 0) mbar_arrive_peer(lead_empty + 8 * a);
       ++tile;
+    }
+  } else if (UP) {
+    // rows past the list keep what their shared memory held: their columns are dropped
+    const int g = (warp - 10) + lane * MG_GATHERS;          // a short list's copies are spread over the warps too
+    if (g < 32) {
+      int s = 0, round = 0;
+      for (int t = cid; t < total && !*fail; t += ncl) {
+        const MoeTile x = moe_tile(p, s_first, s_cnt, t);
+        if (x.nn <= 0) continue;
+        const int nh = ((x.nn + 31) & ~31) >> 1, first = (int)rank * nh, n = min(nh, x.nn - first);
+        const bool mine = 4 * g < n;
+        int src[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          src[i] = mine ? (int)min((unsigned)p.lists[(long long)x.e * p.cap + x.n0 + first + min(4 * g + i, n - 1)] / p.div, (unsigned)p.x_rows - 1) : 0;
+        for (int kb = 0; kb < nkb; ++kb) {
+          if (round > 0 && !wait(empty + 8 * s, (round - 1) & 1)) break;
+          if (mine) tma_gather4_2sm(base + s * stage_bytes + MG_A_BYTES + g * 512, &tx, lead_full + 8 * s, kb * 64, src[0], src[1], src[2], src[3]);
+          if (++s == p.stages) { s = 0; ++round; }
+        }
+      }
     }
   }
   if (*fail) {                                             // copies may still be in flight: leave their shared memory alone for a while
@@ -361,35 +460,47 @@ __global__ void __launch_bounds__(MG_THREADS, 1) moe_gemm_kernel(const MoeGemmPa
     }
   }
   tc_fence_before();
-  __syncthreads();
+  __syncwarp();
+  cluster_sync_all();                                      // the pair's tensor cores read both CTAs' shared memory until here
   if (warp == 1) {
     tc_fence_after();
-    tmem_dealloc(tmem, 512);
+    tmem_dealloc2(tmem, 512);
   }
 }
 
-// CTA = (64 weight rows, expert), 16 pairs at a time; thread = one row of 4 pairs
+// CTA = (64 outputs, expert), 16 pairs at a time; thread = one output of 4 pairs
+template <bool UP>
 __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restrict__ X, long long x_ld, const float* __restrict__ Wt, long long w_ld,
                                                            const MoeGemmParams p) {
   __shared__ float sw[2][16][65], sx[16][17];
-  __shared__ int s_pair[16];
-  const int e = blockIdx.y, r0 = blockIdx.x * 64, cnt = min(p.counts[e], p.cap);
+  __shared__ int s_src[16], s_to[16], s_start;
+  const int e = blockIdx.y, r0 = blockIdx.x * 64, cnt = max(0, min(p.counts[e], p.cap));
+  if (threadIdx.x < 32) {                                  // pairs before this expert
+    int before = 0;
+    for (int i = threadIdx.x; i < e; i += 32) before += max(0, min(p.counts[i], p.cap));
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) before += __shfl_xor_sync(0xffffffffu, before, o);
+    if (threadIdx.x == 0) s_start = before;
+  }
   const int r = threadIdx.x & 63, tg = threadIdx.x >> 6;
-  const int parts = p.up ? 2 : 1;
+  constexpr int parts = UP ? 2 : 1;
   for (int n0 = 0; n0 < cnt; n0 += 16) {
     __syncthreads();
-    if (threadIdx.x < 16) s_pair[threadIdx.x] = p.lists[(long long)e * p.cap + min(n0 + (int)threadIdx.x, cnt - 1)];
+    if (threadIdx.x < 16) {
+      const int i = min(n0 + (int)threadIdx.x, cnt - 1), pair = p.lists[(long long)e * p.cap + i];
+      s_src[threadIdx.x] = min(UP ? (unsigned)pair / p.div : (unsigned)(s_start + i), (unsigned)p.x_rows - 1);
+      s_to[threadIdx.x] = UP ? s_start + i : pair;
+    }
     __syncthreads();
     float acc[2][4] = {};
     for (int k0 = 0; k0 < p.K; k0 += 16) {
       for (int i = threadIdx.x; i < parts * 64 * 16; i += 256) {
         const int q = i / (64 * 16), rr = (i / 16) % 64, k = i % 16;
-        sw[q][k][rr] = (r0 + rr < p.rows && k0 + k < p.K) ? Wt[((long long)e * p.wrows + q * p.up + r0 + rr) * w_ld + k0 + k] : 0.f;
+        sw[q][k][rr] = (r0 + rr < p.rows && k0 + k < p.K) ? Wt[((long long)e * p.wrows + (UP ? 2 * (r0 + rr) + q : r0 + rr)) * w_ld + k0 + k] : 0.f;
       }
       {
         const int i = threadIdx.x, tt = i / 16, k = i % 16;
-        const unsigned src = min((unsigned)s_pair[tt] / p.div, (unsigned)p.x_rows - 1);
-        sx[tt][k] = k0 + k < p.K ? X[(long long)src * x_ld + k0 + k] : 0.f;
+        sx[tt][k] = k0 + k < p.K ? X[(long long)s_src[tt] * x_ld + k0 + k] : 0.f;
       }
       __syncthreads();
       for (int q = 0; q < parts; ++q) {
@@ -408,18 +519,22 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restri
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int i = tg * 4 + j;
-      if (n0 + i < cnt && r0 + r < p.rows && (unsigned)s_pair[i] < (unsigned)p.o_rows)
-        reinterpret_cast<float*>(p.out)[(long long)s_pair[i] * p.o_ld + r0 + r] = p.up ? gated(acc[0][j], acc[1][j], p.limit) : acc[0][j];
+      if (n0 + i < cnt && r0 + r < p.rows && (unsigned)s_to[i] < (unsigned)p.o_rows)
+        reinterpret_cast<float*>(p.out)[(long long)s_to[i] * p.o_ld + r0 + r] = UP ? gated(acc[0][j], acc[1][j], p.limit) : acc[0][j];
     }
   }
 }
 
 template <typename T, bool ACC, int W>
 int launch_route(const RouteParams& p, cudaStream_t st) {
-  const int rb = p.E ? (int)((p.T + ROUTE_WARPS - 1) / ROUTE_WARPS) : 0;
+  const int per = p.T >= 4096 ? 8 : p.T >= 1024 ? 2 : 1, tokens = ROUTE_WARPS * per;
+  const int rb = p.E ? (int)((p.T + tokens - 1) / tokens) : 0;
   const int ab = p.ff ? grid_for(p.T * (p.ff / W), 32 * ROUTE_WARPS) : 0;
-  const size_t smem = p.E ? (size_t)ROUTE_WARPS * (2 * p.E + p.groups + p.top) * 4 : 0;
-  DLTI_CUDA_CHECK(dlti_launch_pdl(p.T, moe_route_kernel<T, ACC, W>, dim3(rb + ab), dim3(32 * ROUTE_WARPS), smem, st, p, rb));
+  const size_t smem = p.E ? (size_t)(p.E + 2 * tokens * p.top + ROUTE_WARPS * (p.E + p.groups)) * 4 : 0;
+  if (smem > 48 * 1024) { dlti_set_error("moe_route: too many experts and choices"); return DLTI_ERR_TOO_LARGE; }
+  auto kern = p.E <= 32 ? moe_route_kernel<T, ACC, W, 1> : p.E <= 64 ? moe_route_kernel<T, ACC, W, 2> : p.E <= 128 ? moe_route_kernel<T, ACC, W, 4>
+              : p.E <= 256 ? moe_route_kernel<T, ACC, W, 8> : moe_route_kernel<T, ACC, W, 32>;
+  DLTI_CUDA_CHECK(dlti_launch_pdl(p.T, kern, dim3(rb + ab), dim3(32 * ROUTE_WARPS), smem, st, p, rb, per));
   dlti_count_launch();
   return 0;
 }
@@ -447,45 +562,48 @@ DLTI_API int dlti_moe_route(const float* z, long long z_ld, int col, const float
   return acc ? launch_route<float, true, 1>(r, st) : launch_route<float, false, 1>(r, st);
 }
 
-// out[pair, 0 .. rows) = X[pair / div] · W_e^T over the pairs lists[e, 0 .. counts[e]) of every expert; W_e = rows e * wrows ... of W.
-// up > 0: gate rows first, up rows `up` further on, out = clipped activation. X: x_rows rows, out: o_rows rows. cap: capacity of a list.
+// The pairs lists[e, 0 .. counts[e]) of every expert; W_e = rows e * wrows ... of W, cap = capacity of a list.
+// up: rows X[pair / div] times W_e, whose rows 2 r and 2 r + 1 are gate and up of output r; out = clipped activation, one list after the
+// other. Otherwise: rows of X in that order times W_e, result to out[pair]. X: x_rows rows, out: o_rows rows of `rows` columns.
 DLTI_API int dlti_moe_gemm(const void* X, long long x_ld, long long x_rows, int div, const void* Wt, long long w_ld, int wrows, int E,
                            const int* lists, const int* counts, int cap, int rows, int up, int K, float limit, void* out, long long o_ld,
                            int o_rows, int dtype, cudaStream_t st) {
   if (o_rows <= 0 || E <= 0) return 0;
-  if (x_rows < 1 || x_rows > 0x7fffffffLL || rows < 1 || K < 1 || div < 1 || (up && up < rows) || (up ? up : 0) + rows > wrows) return DLTI_ERR_BAD_ARG;
-  MoeGemmParams p{lists, counts, E, cap, div, rows, wrows, up, K, limit, out, o_ld, (int)x_rows, o_rows, 0, 0, 0, 0};
+  if (x_rows < 1 || x_rows > 0x7fffffffLL || rows < 1 || K < 1 || div < 1 || rows * (up ? 2 : 1) > wrows) return DLTI_ERR_BAD_ARG;
+  MoeGemmParams p{lists, counts, E, cap, div, rows, wrows, K, limit, out, o_ld, (int)x_rows, o_rows, 0, 0, 0};
   if (dtype == DLTI_FP32) {
-    moe_gemm_f32_kernel<<<dim3((rows + 63) / 64, E), 256, 0, st>>>((const float*)X, x_ld, (const float*)Wt, w_ld, p);
+    (up ? moe_gemm_f32_kernel<true> : moe_gemm_f32_kernel<false>)<<<dim3((rows + 63) / 64, E), 256, 0, st>>>((const float*)X, x_ld, (const float*)Wt,
+                                                                                                           w_ld, p);
     dlti_count_launch();
     return (int)cudaGetLastError();
   }
   if (dtype != DLTI_BF16) return DLTI_ERR_UNSUPPORTED;
   if (E > 1024) { dlti_set_error("moe_gemm: up to 1024 experts"); return DLTI_ERR_TOO_LARGE; }
+  if (o_ld % 8 || o_ld < rows || x_ld % 8 || ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(out)) & 15)) return DLTI_ERR_BAD_ARG;
   const long long avg = (o_rows + E - 1) / E;              // pairs of an expert, were they spread evenly
   p.NT = avg > 96 ? 256 : avg > 40 ? 128 : avg > 12 ? 64 : 32;
-  const int tile_rows = up ? 128 : 256;
-  p.MT = (rows + tile_rows - 1) / tile_rows;
-  p.accs = p.NT <= 128 ? 2 : 1;
-  const int stage = MG_W_BYTES + p.NT * 128, tail = 16 * MG_MAX_STAGES + 48 + 2048 + (2 * E + 1) * 4 + 16;
-  p.stages = (226 * 1024 - 1024 - tail) / stage;
+  p.MT = (rows * (up ? 2 : 1) + 255) / 256;
+  const int stage = MG_A_BYTES + p.NT * 64, tail = MG_TAIL + 2048 + 3 * E * 4;
+  p.stages = (MG_SMEM - 1024 - tail) / stage;
   if (p.stages > MG_MAX_STAGES) p.stages = MG_MAX_STAGES;
   const int smem = p.stages * stage + tail + 1024;
   CUtensorMap tw, tx;
   int rc;
   if ((rc = dlti_get_tmap(&tw, Wt, K, (uint64_t)E * wrows, w_ld, 64, 128))) return rc;
-  if ((rc = dlti_get_tmap(&tx, X, K, x_rows, x_ld, 64, 1))) return rc;
+  if ((rc = dlti_get_tmap(&tx, X, K, x_rows, x_ld, 64, up ? 1 : p.NT / 2))) return rc;
   static bool done[64] = {};
   int dev = 0;
   DLTI_CUDA_CHECK(cudaGetDevice(&dev));
   if (!done[dev & 63]) {
-    DLTI_CUDA_CHECK(cudaFuncSetAttribute(moe_gemm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024));
+    DLTI_CUDA_CHECK(cudaFuncSetAttribute(moe_gemm_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, MG_SMEM));
+    DLTI_CUDA_CHECK(cudaFuncSetAttribute(moe_gemm_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, MG_SMEM));
     done[dev & 63] = true;
   }
   // at most one tile per pair and weight tile
   const long long most = (long long)p.MT * (E < o_rows ? E + (o_rows - E) / p.NT + 1 : o_rows);
-  const int sms = dlti_num_sms();
-  DLTI_CUDA_CHECK(dlti_launch_pdl(cap, moe_gemm_kernel, dim3(most < sms ? (unsigned)most : sms), dim3(MG_THREADS), (size_t)smem, st, p, tw, tx));
+  const int clusters = dlti_num_sms() / 2;
+  DLTI_CUDA_CHECK(dlti_launch_pdl(cap, up ? moe_gemm_kernel<true> : moe_gemm_kernel<false>, dim3(2 * (most < clusters ? (unsigned)most : clusters)),
+                                  dim3(MG_THREADS), (size_t)smem, st, p, tw, tx));
   dlti_count_launch();
   return 0;
 }

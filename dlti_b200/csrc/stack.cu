@@ -280,29 +280,28 @@ __global__ void __launch_bounds__(512) gated_norm_vec_kernel(const T* __restrict
   }
 }
 
-// many small groups: a warp per group, eight groups a CTA
-template <typename T, int GATE, bool ACC, int VPT>
+// many small groups: LPG lanes per group (VPT > 1: a warp)
+template <typename T, int GATE, bool ACC, int VPT, int LPG>
 __global__ void __launch_bounds__(256) gated_norm_warp_kernel(const T* __restrict__ y, long long y_ld, const void* __restrict__ gate,
                                                               long long g_ld, const float* __restrict__ w, T* __restrict__ out,
                                                               long long o_ld, int gs, int groups, long long total, float eps) {
   griddep_wait();
   griddep_launch();
-  const long long x = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (x >= total) return;
+  const long long x0 = ((long long)blockIdx.x * 256 + threadIdx.x) / LPG, x = min(x0, total - 1);       // whole warps take part in the sums
   const long long t = x / groups;
-  const int c0 = (int)(x - t * groups) * gs, vec = gs >> 3, lane = threadIdx.x & 31;
+  const int c0 = (int)(x - t * groups) * gs, vec = x0 < total ? gs >> 3 : 0, lane = threadIdx.x % LPG;
   const T* yr = y + t * y_ld;
   const void* gr = reinterpret_cast<const uint8_t*>(gate) + t * g_ld * (ACC ? 4 : sizeof(T));
   float v[VPT][8], g[VPT][8], ss = 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i)
-    if (lane + 32 * i < vec) {
-      take_n<T, false, 8>(yr, c0 + (lane + 32 * i) * 8, v[i]);
-      take_n<T, ACC, 8>(gr, c0 + (lane + 32 * i) * 8, g[i]);
+    if (lane + LPG * i < vec) {
+      take_n<T, false, 8>(yr, c0 + (lane + LPG * i) * 8, v[i]);
+      take_n<T, ACC, 8>(gr, c0 + (lane + LPG * i) * 8, g[i]);
     }
 #pragma unroll
   for (int i = 0; i < VPT; ++i)
-    if (lane + 32 * i < vec)
+    if (lane + LPG * i < vec)
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const float e = fast_sigmoid(g[i][j]);
@@ -310,15 +309,18 @@ __global__ void __launch_bounds__(256) gated_norm_warp_kernel(const T* __restric
         else g[i][j] = GATE == GATE_SILU ? g[i][j] * e : e;
         ss += v[i][j] * v[i][j];
       }
-  const float r = 1.f / sqrtf(warp_sum(ss) / (float)gs + eps);
+#pragma unroll
+  for (int o = LPG / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float r = 1.f / sqrtf(ss / (float)gs + eps);
+  if (x0 >= total) return;
 #pragma unroll
   for (int i = 0; i < VPT; ++i)
-    if (lane + 32 * i < vec) {
+    if (lane + LPG * i < vec) {
       float wv[8];
-      ld8(w + c0 + (lane + 32 * i) * 8, wv);
+      ld8(w + c0 + (lane + LPG * i) * 8, wv);
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[i][j] *= r * wv[j] * (GATE == GATE_SILU_FIRST ? 1.f : g[i][j]);
-      put_n(out + t * o_ld + c0 + (lane + 32 * i) * 8, v[i]);
+      put_n(out + t * o_ld + c0 + (lane + LPG * i) * 8, v[i]);
     }
 }
 
@@ -601,6 +603,82 @@ __global__ void __launch_bounds__(256) qkv_rows_kernel(const QkvRowParams p) {
   }
 }
 
+// the same with the row in registers: 16-bit T, VPT pieces of 8 a thread, every load issued before the sums
+template <typename T, bool ACC, int VPT>
+__global__ void __launch_bounds__(128) qkv_rows_vec_kernel(const QkvRowParams p) {
+  __shared__ float2 red[4];
+  griddep_wait();
+  griddep_launch();
+  const long long t = blockIdx.x;
+  const uint8_t* row = reinterpret_cast<const uint8_t*>(p.proj) + t * p.ld * (ACC ? 4 : sizeof(T));
+  const long long slot = p.slots[t];
+  const long long to = (p.dst && t >= p.nd) ? p.nd + (long long)p.dst[t - p.nd] : t;
+  const int nq = p.H * p.dim, nk = p.G * p.dim, nv = p.G * p.vdim;
+  float f[VPT][8], sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int x = (threadIdx.x + i * 128) * 8;
+    if (x < nq + nk + nv) take_n<T, ACC, 8>(row, x < nq ? p.oq + x : x < nq + nk ? p.ok + x - nq : p.ov + x - nq - nk, f[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int x = (threadIdx.x + i * 128) * 8;
+    if (x >= nq + nk + nv) continue;
+    if (p.bias) {
+      float b[8];
+      ld8(p.bias + (x < nq ? p.oq + x : x < nq + nk ? p.ok + x - nq : p.ov + x - nq - nk), b);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[i][j] += b[j];
+    }
+    if (x < nq + nk) {
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss += f[i][j] * f[i][j];
+      if (x < nq) sq += ss;
+      else sk += ss;
+    }
+  }
+  float rq = 1.f, rk = 1.f;
+  if (p.qn) {
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(sq, sk);
+    __syncthreads();
+    const float2 a = red[0], b = red[1], c = red[2], d = red[3];
+    rq = rsqrtf((a.x + b.x + c.x + d.x) / (float)nq + p.eps);
+    rk = rsqrtf((a.y + b.y + c.y + d.y) / (float)nk + p.eps);
+  }
+  const float share = p.first ? p.share[0] : 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int x = (threadIdx.x + i * 128) * 8;
+    if (x >= nq + nk + nv) continue;
+    const bool is_q = x < nq, is_v = x >= nq + nk;
+    const int y = is_q ? x : is_v ? x - nq - nk : x - nq, hd = is_v ? p.vdim : p.dim, h = y / hd, c = y - h * hd;
+    if (is_v) {
+      if (p.own) put_n(reinterpret_cast<T*>(p.own) + t * p.own_ld + y, f[i]);
+      if (p.first) {
+        float e[8];
+        take_n<T, false, 8>(reinterpret_cast<const T*>(p.first) + t * p.f_ld, y, e);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[i][j] += share * (e[j] - f[i][j]);
+      }
+    } else if (p.qn) {
+      float w[8];
+      ld8((is_q ? p.qn : p.kn) + y, w);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[i][j] *= (is_q ? rq : rk) * w[j];
+    }
+    if (is_q) {
+      put_n(reinterpret_cast<T*>(p.q) + to * p.q_ld + (long long)h * p.q_hd + c, f[i]);
+    } else {
+      void* pk = is_v ? p.vp : p.kp;
+      if (pk) put_n(reinterpret_cast<T*>(pk) + to * p.q_ld + (long long)h * p.q_hd + c, f[i]);
+      if (slot >= 0) put_n(reinterpret_cast<T*>(is_v ? p.vc : p.kc) + (slot * p.G + h) * (is_v ? p.vd : p.kd) + c, f[i]);
+    }
+  }
+}
+
 // Causal convolution of `taps` per channel + silu over the rows of every sequence of a step. src = projection rows
 // (channel 0 at column `col`); inputs from before the step come from conv_state [slots, taps - 1, C] (zero at position
 // 0). ACC additionally leaves the rounded projection row in `raw` (columns raw0 .. raw0 + raw_n): the gate, the step
@@ -612,6 +690,7 @@ struct ConvParams {
   void* out; long long o_ld;
   void* raw; long long raw_ld; int raw_n;
   long long rows;
+  float* tail; long long tail_ld; int tail0;               // accumulator columns from tail0 on go here unrounded (null: nowhere)
 };
 template <typename T>
 __global__ void __launch_bounds__(256) short_conv_kernel(const ConvParams p) {
@@ -740,6 +819,11 @@ __global__ void __launch_bounds__(256) short_conv_acc_kernel(const ConvParams p)
     const long long t = i / pairs;
     const int col = 2 * (int)(i - t * pairs);
     const uint8_t* row = reinterpret_cast<const uint8_t*>(p.src) + t * p.ld * 4;
+    if (p.tail && col >= p.tail0) {
+      const float2 v = take2<float, true>(row, col);
+      *reinterpret_cast<float2*>(p.tail + t * p.tail_ld + col - p.tail0) = v;
+      continue;
+    }
     const float2 v = take2<T, true>(row, col);             // raw_n is a multiple of 8
     put2(reinterpret_cast<T*>(p.raw) + t * p.raw_ld, col, v.x, v.y);
     const int c = col - p.col;
@@ -770,6 +854,11 @@ __global__ void __launch_bounds__(128) short_conv_acc_vec_kernel(const ConvParam
   if (col >= p.raw_n) return;
   const long long t = blockIdx.x;
   float v[8];
+  if (p.tail && col >= p.tail0) {
+    take_n<float, true, 8>(reinterpret_cast<const uint8_t*>(p.src) + t * p.ld * 4, col, v);
+    st8(p.tail + t * p.tail_ld + col - p.tail0, v);
+    return;
+  }
   take_n<T, true, 8>(reinterpret_cast<const uint8_t*>(p.src) + t * p.ld * 4, col, v);
   put_n(reinterpret_cast<T*>(p.raw) + t * p.raw_ld + col, v);
   const int c = col - p.col;
@@ -852,10 +941,12 @@ int gated_norm_mode(const void* y, long long y_ld, const void* gate, long long g
       ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
     using B = __nv_bfloat16;
     if (groups > 1 && gs <= 512) {
-      auto kern = acc ? (gs <= 256 ? gated_norm_warp_kernel<B, GATE, true, 1> : gated_norm_warp_kernel<B, GATE, true, 2>)
-                      : (gs <= 256 ? gated_norm_warp_kernel<B, GATE, false, 1> : gated_norm_warp_kernel<B, GATE, false, 2>);
-      const long long total = rows * groups;
-      DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)((total + 7) / 8)), dim3(256), 0, st, (const B*)y, y_ld, gate, g_ld, w, (B*)out,
+#define GNW(AC) (gs <= 64 ? gated_norm_warp_kernel<B, GATE, AC, 1, 8> : gs <= 128 ? gated_norm_warp_kernel<B, GATE, AC, 1, 16> \
+                 : gs <= 256 ? gated_norm_warp_kernel<B, GATE, AC, 1, 32> : gated_norm_warp_kernel<B, GATE, AC, 2, 32>)
+      auto kern = acc ? GNW(true) : GNW(false);
+#undef GNW
+      const long long total = rows * groups, per = 256 / (gs <= 64 ? 8 : gs <= 128 ? 16 : 32);
+      DLTI_CUDA_CHECK(dlti_launch_pdl(rows, kern, dim3((unsigned)((total + per - 1) / per)), dim3(256), 0, st, (const B*)y, y_ld, gate, g_ld, w, (B*)out,
                                       o_ld, gs, groups, total, eps));
       dlti_count_launch();
       return 0;
@@ -1005,6 +1096,19 @@ DLTI_API int dlti_qkv_rows(const void* proj, long long ld, int oq, int ok, int o
                      reinterpret_cast<uintptr_t>(kc) | reinterpret_cast<uintptr_t>(vc) | reinterpret_cast<uintptr_t>(q) |
                      reinterpret_cast<uintptr_t>(kp) | reinterpret_cast<uintptr_t>(vp)) & 15) == 0;
   using B = __nv_bfloat16;
+  const int pieces = ((H + G) * dim + G * vdim) / 8;
+  if (vec && pieces <= 128 * 12 &&
+      ((reinterpret_cast<uintptr_t>(bias) | reinterpret_cast<uintptr_t>(qn) | reinterpret_cast<uintptr_t>(kn)) & 15) == 0) {
+#define QR_CASE(V)                                                                                                          \
+  if (pieces <= 128 * V) {                                                                                                  \
+    auto kern = acc ? qkv_rows_vec_kernel<B, true, V> : qkv_rows_vec_kernel<B, false, V>;                                    \
+    DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, kern, dim3((unsigned)tokens), dim3(128), 0, st, p));                             \
+    dlti_count_launch();                                                                                                    \
+    return 0;                                                                                                               \
+  }
+    QR_CASE(1) QR_CASE(2) QR_CASE(3) QR_CASE(4) QR_CASE(6) QR_CASE(8) QR_CASE(12)
+#undef QR_CASE
+  }
   auto kern = vec ? (acc ? qkv_rows_kernel<B, true, 8> : qkv_rows_kernel<B, false, 8>)
                   : dtype == DLTI_BF16 ? (acc ? qkv_rows_kernel<B, true, 1> : qkv_rows_kernel<B, false, 1>)
                                        : (acc ? qkv_rows_kernel<float, true, 1> : qkv_rows_kernel<float, false, 1>);
@@ -1028,11 +1132,11 @@ DLTI_API int dlti_prefix_rows(void* packed, long long ld, int hd, const int* row
 
 DLTI_API int dlti_short_conv(const void* src, long long ld, int col, int C, int taps, const float* w, const float* b, int w_ld,
                              const void* state, const int* sslot, const int* rseq, const int* ctx, const int* cu, int nd, void* out,
-                             long long o_ld, void* raw, long long raw_ld, int raw_n, long long rows, int acc, int dtype,
-                             cudaStream_t st) {
+                             long long o_ld, void* raw, long long raw_ld, int raw_n, float* tail, long long tail_ld, int tail0, long long rows,
+                             int acc, int dtype, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (taps < 1 || C < 1) return DLTI_ERR_BAD_ARG;
-  ConvParams p{src, ld, col, C, taps, w, b, w_ld, state, sslot, rseq, ctx, cu, nd, out, o_ld, raw, raw_ld, raw_n, rows};
+  if (taps < 1 || C < 1 || (tail && (!acc || tail0 % 8 || tail_ld % 4 || (reinterpret_cast<uintptr_t>(tail) & 15)))) return DLTI_ERR_BAD_ARG;
+  ConvParams p{src, ld, col, C, taps, w, b, w_ld, state, sslot, rseq, ctx, cu, nd, out, o_ld, raw, raw_ld, raw_n, rows, tail, tail_ld, tail0};
   if (acc) {
     if (nd != rows || !raw || raw_n % 2) return DLTI_ERR_BAD_ARG;
     if (dtype == DLTI_BF16 && C % 8 == 0 && ld % 8 == 0 && col % 8 == 0 && raw_n % 8 == 0 && raw_ld % 8 == 0 && o_ld % 8 == 0 && w_ld % 4 == 0 &&

@@ -10,7 +10,7 @@ from pathlib import Path
 
 import torch
 
-from .stack import AttentionMixer, DeltaMixer, DenseMlp, Layer, MoeMlp, StackConfig, StackWeights, mixer_sections, round8
+from .stack import AttentionMixer, DeltaMixer, DenseMlp, Layer, MoeMlp, StackConfig, StackWeights, mixer_sections
 
 ARCHITECTURE = "Latanex"
 
@@ -116,10 +116,9 @@ def named_tensors(w: StackWeights):
             for s in ("A_log", "dt_bias", "norm"):
                 yield p + "mix." + s, lw[s]
         if isinstance(e, MoeMlp):
-            ffr = round8(e.ff)
             for j in range(e.experts):
-                yield p + f"mlp.e{j}.gate", lw["e_up"][j, :e.ff]
-                yield p + f"mlp.e{j}.up", lw["e_up"][j, ffr:ffr + e.ff]
+                yield p + f"mlp.e{j}.gate", lw["e_up"][j, 0:2 * e.ff:2]
+                yield p + f"mlp.e{j}.up", lw["e_up"][j, 1:2 * e.ff:2]
                 yield p + f"mlp.e{j}.down", lw["e_down"][j, :d]
             yield p + "mlp.router", w.mlp_section(i, "router")
             yield p + "mlp.correction", lw["correction"]

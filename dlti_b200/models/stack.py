@@ -381,7 +381,8 @@ class StackWeights:
             if isinstance(e, MoeMlp):
                 def stack(rows, cols):
                     return torch.zeros(e.experts, round8(rows), round8(cols), dtype=dtype, device=device)[:, :, :cols]
-                w |= {"correction": vec(e.experts), "e_up": stack(2 * round8(e.ff), d), "e_down": stack(d, e.ff)}
+                # gate and up rows of an expert alternate
+                w |= {"correction": vec(e.experts), "e_up": stack(2 * e.ff, d), "e_down": stack(d, e.ff)}
                 if e.shared_ff:
                     w["w_down"] = mat(d, e.shared_ff)
             elif e is not None:

@@ -1,7 +1,7 @@
 """Gated activations and mixtures of experts (csrc/moe.cu); PyTorch restatements for CPU tensors. Conventions as in ops/stack.py.
 
-A step's (token, choice) pairs are numbered token * top + choice. The router writes every expert's pairs as a list; the grouped
-GEMMs gather and scatter rows by these lists, so no permuted copy of the activations is made."""
+A step's (token, choice) pairs are numbered token * top + choice. The router writes every expert's pairs as a list; the first
+grouped GEMM gathers its rows by these lists and the second scatters by them, so no permuted copy of the inputs is made."""
 from __future__ import annotations
 
 from dataclasses import dataclass
@@ -100,20 +100,21 @@ def route_ref(z, correction, e: MoeMlp):
     return idx, w / (w.sum(-1, keepdim=True) + 1e-20) * e.scale
 
 
-def grouped_gemm(x, w, lists, counts, out, *, rows: int, pairs_per_row: int, up: int = 0, limit: float = 0.0, max_rows: int = 0):
-    """out[pair, :rows] = x[pair // pairs_per_row] · w[e, :rows]^T for the pairs of every expert's list; w [E, rows, K]. up > 0: the
-    clipped activation of that product (gate) and the one with rows [up, up + rows) (up), in the kernel."""
+def grouped_gemm(x, w, lists, counts, out, *, rows: int, pairs_per_row: int, up: bool = False, limit: float = 0.0):
+    """Products of the pairs of every expert's list with its weights w [E, >= rows, K]. up: rows x[pair // pairs_per_row] times the
+    gate and up rows 2 r and 2 r + 1 of w; the clipped activations go to out one list after the other. Otherwise: rows of x in that
+    order; results go to out[pair]."""
     E, K, T = w.shape[0], w.shape[2], lists.shape[1]
     f = _lib.fn("dlti_moe_gemm", [_V, _L, _L, _I, _V, _L, _I, _I, _V, _V, _I, _I, _I, _I, _F, _V, _L, _I, _I, _V])
     _lib.check(f(_p(x), x.stride(0), x.shape[0], pairs_per_row, _p(w), w.stride(1), w.stride(0) // w.stride(1), E, _p(lists), _p(counts), T,
-                 rows, up, K, float(limit), _p(out), out.stride(0), out.shape[0], _lib.dtype_code(x.dtype), _lib.stream_ptr()), "moe_gemm")
+                 rows, int(up), K, float(limit), _p(out), out.stride(0), out.shape[0], _lib.dtype_code(x.dtype), _lib.stream_ptr()), "moe_gemm")
     return out
 
 
 def moe(h, e: MoeMlp, lw, dtype, mm, acc=False) -> ExpertSum:
     """Mixture of experts of the rows h; mm: the GEMM for the shared expert's output (its accumulator with acc)."""
     T, d = h.shape
-    sec, ffr = mlp_sections(e), round8(e.ff)
+    sec = mlp_sections(e)
     og, ou = (sec["gate"], sec["up"]) if e.shared_ff else (0, 0)
     if not _lib.use_native(h):
         p = linear(h, lw["w_up"], out_dtype=torch.float32)
@@ -123,7 +124,7 @@ def moe(h, e: MoeMlp, lw, dtype, mm, acc=False) -> ExpertSum:
             pair = (idx.flatten() == j).nonzero()[:, 0]
             if len(pair):
                 gu = h[pair // e.top].float() @ lw["e_up"][j].float().t()
-                a = _gated(gu[:, :e.ff], gu[:, ffr:ffr + e.ff], e.limit).to(dtype)
+                a = _gated(gu[:, 0:2 * e.ff:2], gu[:, 1:2 * e.ff:2], e.limit).to(dtype)
                 rows[pair] = a.float() @ lw["e_down"][j, :d].float().t()
         shared = mm(gated_act(p, og, ou, e.shared_ff, e.shared_limit, dtype), lw["w_down"]) if e.shared_ff else None
         return ExpertSum(rows.to(dtype), wgt, shared)
@@ -137,7 +138,7 @@ def moe(h, e: MoeMlp, lw, dtype, mm, acc=False) -> ExpertSum:
         p = linear(h, lw["w_up"][:sec["router"]]) if e.shared_ff else None
         wgt, lists, counts = _route(p, z, 0, lw["correction"], e, act_of)
     a = act(T * e.top, e.ff, dtype, h.device)
-    grouped_gemm(h, lw["e_up"], lists, counts, a, rows=e.ff, pairs_per_row=e.top, up=ffr, limit=e.limit)
+    grouped_gemm(h, lw["e_up"], lists, counts, a, rows=e.ff, pairs_per_row=e.top, up=True, limit=e.limit)
     rows = act(T * e.top, d, dtype, h.device)
     grouped_gemm(a, lw["e_down"], lists, counts, rows, rows=d, pairs_per_row=1)
     return ExpertSum(rows, wgt, mm(hs, lw["w_down"]) if e.shared_ff else None, counts)

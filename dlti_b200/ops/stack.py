@@ -410,10 +410,11 @@ def paged_attention(q, m, rows: Rows, kc, vc, gate, sink=None):
 
 
 # ---- recurrences -------------------------------------------------------------------------------------------
-def short_conv(proj, col, C_, w, b, state, rows: Rows, dtype, acc=False, width=0):
+def short_conv(proj, col, C_, w, b, state, rows: Rows, dtype, acc=False, width=0, split=0):
     """silu of the causal convolution of channels [col, col + C_) of the projection rows; w [taps, >= C_] tap-major,
     state [slots, taps - 1, C_] = inputs of earlier steps (read only; linear_scan's tail job renews it). Returns (out
-    [T, C_], proj): with acc (decode rows only) proj is the projection rounded to the compute dtype, else as given."""
+    [T, C_], proj): with acc (decode rows only) proj is the projection rounded to the compute dtype, else as given. split > 0 (with
+    acc): columns from split on as an fp32 result of their own, (out, proj [T, split], fp32 columns)."""
     T, taps = proj.shape[0], w.shape[0]
     if not _lib.use_native(proj):
         out = torch.zeros(T, C_)
@@ -426,12 +427,13 @@ def short_conv(proj, col, C_, w, b, state, rows: Rows, dtype, acc=False, width=0
             out[r0:r0 + n] = b[:C_] + sum(w[k, :C_] * x[k:k + n] for k in range(taps))
         return torch.nn.functional.silu(out).to(dtype), proj
     out = act(T, C_, dtype, proj.device)
-    raw = act(T, width, dtype, proj.device) if acc else None
-    f = _lib.fn("dlti_short_conv", [_V, _L, _I, _I, _I, _V, _V, _I, _V, _V, _V, _V, _V, _I, _V, _L, _V, _L, _I, _L, _I, _I, _V])
+    raw = act(T, split or width, dtype, proj.device) if acc else None
+    tail = torch.empty((T, width - split), dtype=torch.float32, device=proj.device) if split else None
+    f = _lib.fn("dlti_short_conv", [_V, _L, _I, _I, _I, _V, _V, _I, _V, _V, _V, _V, _V, _I, _V, _L, _V, _L, _I, _V, _L, _I, _L, _I, _I, _V])
     _lib.check(f(_p(proj), proj.stride(0), col, C_, taps, _p(w), _p(b), w.stride(0), _p(state), _p(rows.state), _p(rows.seq),
-                 _p(rows.ctx), _p(rows.cu), rows.nd, _p(out), out.stride(0), _p(raw), 0 if raw is None else raw.stride(0), width, T,
-                 int(acc), _lib.dtype_code(dtype), _lib.stream_ptr()), "short_conv")
-    return out, (raw if acc else proj)
+                 _p(rows.ctx), _p(rows.cu), rows.nd, _p(out), out.stride(0), _p(raw), 0 if raw is None else raw.stride(0), width, _p(tail),
+                 0 if tail is None else tail.stride(0), split, T, int(acc), _lib.dtype_code(dtype), _lib.stream_ptr()), "short_conv")
+    return (out, raw, tail) if split else (out, raw if acc else proj)
 
 
 @dataclass

@@ -461,7 +461,7 @@ def latanex_kernels(width: int, peaks: dict, nseq: int, length: int, batch: int,
     run("prefill", "attention (paged, heads > 128)", lambda: K.attn_paged_prefill(q, m, pr, kc, vc, None, out, sink=sink), io, fl)
     qd, od = rnd(batch, H * hd), K.act(batch, H * hd, bf, dev)
     run("decode", "attention", lambda: K.attn_paged_decode(qd, m, dr, kc, vc, None, od, sink=sink), batch * min(ctx + 1, m.window) * G * hd * 4)
-    sec, sm, su, ffr = mixer_sections(m), mixer_sections(mem), mlp_sections(e), round8(e.ff)
+    sec, sm, su = mixer_sections(m), mixer_sections(mem), mlp_sections(e)
     norms = [(torch.ones(1, device=dev), torch.ones(d, device=dev), torch.zeros(d, device=dev)) for _ in range(2)]
     qk, vv = mem.kv_heads * mem.dim, mem.heads * mem.vdim
     for phase, r, n, ns in (("prefill", pr, T, nseq), ("decode", dr, batch, batch)):
@@ -488,7 +488,7 @@ def latanex_kernels(width: int, peaks: dict, nseq: int, length: int, batch: int,
         counts.zero_()                                            # as the next step wants them
         hit = int((cnt > 0).sum())
         a, rows_ = K.act(n * e.top, e.ff, bf, dev), K.act(n * e.top, d, bf, dev)
-        run(phase, "experts in + activation", lambda: ME.grouped_gemm(h, lw["e_up"], lists, cnt, a, rows=e.ff, pairs_per_row=e.top, up=ffr, limit=e.limit),
+        run(phase, "experts in + activation", lambda: ME.grouped_gemm(h, lw["e_up"], lists, cnt, a, rows=e.ff, pairs_per_row=e.top, up=True, limit=e.limit),
             2 * (n * d + hit * 2 * e.ff * d + n * e.top * e.ff), 4.0 * n * e.top * e.ff * d)
         run(phase, "experts out", lambda: ME.grouped_gemm(a, lw["e_down"], lists, cnt, rows_, rows=d, pairs_per_row=1),
             2 * (n * e.top * (e.ff + d) + hit * e.ff * d), 2.0 * n * e.top * e.ff * d)
@@ -499,7 +499,12 @@ def latanex_kernels(width: int, peaks: dict, nseq: int, length: int, batch: int,
             n * e.shared_ff * (2 * es + 2))
         conv, ssm = torch.zeros(ns, mem.conv - 1, sm["g"], device=dev, dtype=bf), torch.zeros(ns, mem.heads, mem.dim, mem.vdim, device=dev)
         pm, gates = rnd(n, sm["gates"]), torch.randn(n, 2 * mem.heads, device=dev)
-        run(phase, "short conv", lambda: K.short_conv(pm, 0, sm["g"], lm["conv"], w.derived[0]["conv_b"], conv, r, bf), n * sm["g"] * 4)
+        cb, zp = w.derived[0]["conv_b"], torch.zeros(n, sm.total, device=dev) if acc else None
+        if acc:
+            run(phase, "short conv", lambda: K.short_conv(zp, 0, sm["g"], lm["conv"], cb, conv, r, bf, acc=True, width=sm.total, split=sm["gates"]),
+                n * (sm.total * 10 + sm["g"] * 2 + (mem.conv - 1) * sm["g"] * 2))
+        else:
+            run(phase, "short conv", lambda: K.short_conv(pm, 0, sm["g"], lm["conv"], cb, conv, r, bf), n * sm["g"] * 4)
         # useful work of the chunked form: products with the state (three), scores of keys and queries, the triangular system, its use
         work = 2.0 * n * mem.heads * (3 * mem.dim * mem.vdim + 32 * 2 * mem.dim + 32 * 2 * mem.vdim) if not acc else 6.0 * n * mem.heads * mem.dim * mem.vdim
         run(phase, "delta scan", lambda: DR.delta_scan(pm[:, :qk], pm[:, sm["k"]:sm["k"] + qk], pm[:, sm["v"]:sm["v"] + vv], gates, lm["A_log"], lm["dt_bias"],

@@ -248,8 +248,13 @@ class StackRunner:
     def _delta(self, i, m: DeltaMixer, lw, xa, rows: K.Rows, segs):
         s, st, der = self.sections[i], self.states, self.w.derived[i]
         qk, vv = m.kv_heads * m.dim, m.heads * m.vdim
-        proj, gates = H.linear_split(xa, lw["w_in"], s["gates"])
-        x, proj = K.short_conv(proj, 0, s["g"], lw["conv"], der["conv_b"], st.conv[i], rows, self.dtype)
+        if self.acc and rows.nd == xa.shape[0]:                   # the convolution of prompt rows reads its neighbours' inputs
+            proj = gemm_skinny_acc(xa, lw["w_in"])
+            x, proj, gates = K.short_conv(proj, 0, s["g"], lw["conv"], der["conv_b"], st.conv[i], rows, self.dtype, acc=True, width=proj.shape[1],
+                                          split=s["gates"])
+        else:
+            proj, gates = H.linear_split(xa, lw["w_in"], s["gates"])
+            x, proj = K.short_conv(proj, 0, s["g"], lw["conv"], der["conv_b"], st.conv[i], rows, self.dtype)
         y = D.delta_scan(x[:, :qk], x[:, s["k"]:s["k"] + qk], x[:, s["v"]:s["v"] + vv], gates, lw["A_log"], lw["dt_bias"], st.ssm[i], rows, m.heads,
                          m.kv_heads, m.dim, m.vdim, conv_src=proj, conv_col=0, conv_state=st.conv[i])
         return K.gated_norm(y, proj[:, s["g"]:s["g"] + vv], der["norm"], self.cfg.norm_eps, m.heads, gate_first=False, silu=True)

@@ -374,11 +374,11 @@ def test_mixture_of_experts(device, dtype, T, d, e):
         ff = e.shared_ff if j == "shared." else e.ff
         p |= {j + "gate": rnd(g, ff, d) * d ** -0.5, j + "up": rnd(g, ff, d) * d ** -0.5, j + "down": rnd(g, d, ff) * ff ** -0.5}
     new = lambda *s: torch.zeros(*s, dtype=dtype, device=device)
-    lw = {"w_up": new(sec.total, round8(d))[:, :d], "e_up": new(e.experts, 2 * ffr, round8(d))[..., :d], "e_down": new(e.experts, round8(d), ffr)[..., :e.ff],
+    lw = {"w_up": new(sec.total, round8(d))[:, :d], "e_up": new(e.experts, round8(2 * e.ff), round8(d))[..., :d], "e_down": new(e.experts, round8(d), ffr)[..., :e.ff],
           "correction": p["correction"].to(device), "w_down": new(round8(d), round8(e.shared_ff or 8))[:, :e.shared_ff or 8]}
     lw["w_up"][sec["router"]:sec["router"] + e.experts] = p["router"]
     for i in range(e.experts):
-        lw["e_up"][i, :e.ff], lw["e_up"][i, ffr:ffr + e.ff], lw["e_down"][i, :d] = (p[f"e{i}.{s}"] for s in ("gate", "up", "down"))
+        lw["e_up"][i, 0:2 * e.ff:2], lw["e_up"][i, 1:2 * e.ff:2], lw["e_down"][i, :d] = (p[f"e{i}.{s}"] for s in ("gate", "up", "down"))
     if e.shared_ff:
         lw["w_up"][sec["gate"]:sec["gate"] + e.shared_ff], lw["w_up"][sec["up"]:sec["up"] + e.shared_ff] = p["shared.gate"], p["shared.up"]
         lw["w_down"][:d] = p["shared.down"]
