@@ -191,7 +191,7 @@ struct MoeGemmParams {
 // UP: the source of list entry i is row lists[i] / div, its result (activation of rows 2 r and 2 r + 1) goes to row (start of the
 // list) + i. Otherwise the source is row (start of the list) + i and the result goes to row lists[i].
 constexpr int MG_GATHERS = 8, MG_THREADS = 320 + 32 * MG_GATHERS, MG_A_BYTES = 16384, MG_MAX_STAGES = 10, MG_SMEM = 226 * 1024;
-constexpr int MG_TAIL = 8 * (2 * MG_MAX_STAGES + 4) + 16;  // barriers, TMEM address
+constexpr int MG_TAIL = 8 * (3 * MG_MAX_STAGES + 4) + 16;  // barriers, TMEM address
 constexpr long long MG_WAIT_LIMIT = 4000000000LL;
 
 // rows r0 .. r3 of a matrix (box of one row) one after the other; completion bytes on a barrier that may live in the peer CTA
@@ -228,8 +228,8 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   const uint32_t stage_bytes = MG_A_BYTES + p.NT * 64;
-  const uint32_t full = base + p.stages * stage_bytes, empty = full + 8 * MG_MAX_STAGES, acc_full = empty + 8 * MG_MAX_STAGES,
-                 acc_empty = acc_full + 16, slot = acc_empty + 16;
+  const uint32_t full = base + p.stages * stage_bytes, empty = full + 8 * MG_MAX_STAGES, passed = empty + 8 * MG_MAX_STAGES,
+                 acc_full = passed + 8 * MG_MAX_STAGES, acc_empty = acc_full + 16, slot = acc_empty + 16;
   uint8_t* tail = smem_raw + (slot - smem_u32(smem_raw)) + 16;
   volatile uint32_t* slot_ptr = reinterpret_cast<volatile uint32_t*>(tail - 16);
   int* s_dst = reinterpret_cast<int*>(tail);               // [2][256]
@@ -248,6 +248,7 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
     for (int s = 0; s < p.stages; ++s) {
       mbar_init(full + 8 * s, 1);                          // the leader's: bytes of both CTAs
       mbar_init(empty + 8 * s, 1);
+      mbar_init(passed + 8 * s, MG_GATHERS);
     }
     for (int a = 0; a < 2; ++a) {
       mbar_init(acc_full + 8 * a, 1);
@@ -306,6 +307,8 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
       }
     return true;
   };
+  auto wait_warp = [&](uint32_t bar, uint32_t parity) { return __all_sync(0xffffffffu, wait(bar, parity)) != 0; };     // the warp stays together
+  auto failed = [&]() { return __any_sync(0xffffffffu, *fail) != 0; };
   const uint32_t lead_full = mapa_rank(full, 0);
 
   if (warp == 0 || (!UP && warp == 10)) {
@@ -318,7 +321,9 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
         const int nh = ((x.nn + 31) & ~31) >> 1, r0 = s_row[x.e] + x.n0 + (int)rank * nh;
         const int groups = ((min(nh, x.nn) + 3) >> 2) + ((max(0, x.nn - nh) + 3) >> 2);
         for (int kb = 0; kb < nkb; ++kb) {
-          if (round > 0 && !wait(empty + 8 * s, (round - 1) & 1)) break;
+          // Gathering, the weights of a k block follow the gathering warps: one without rows in this tile has nothing else that would
+          // keep it within a phase of the others.
+          if (UP ? !wait(passed + 8 * s, round & 1) : round > 0 && !wait(empty + 8 * s, (round - 1) & 1)) break;
           const uint32_t dst = base + s * stage_bytes, bar = lead_full + 8 * s;
           if (warp == 0) {
             if (rank == 0) mbar_expect_tx(full + 8 * s, 2 * MG_A_BYTES + (UP ? groups * 512 : p.NT * 128));
@@ -334,15 +339,15 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
     if (rank == 0) {
       const bool leader = elect_one_sync();
       int s = 0, round = 0, tile = 0;
-      for (int t = cid; t < total && !*fail; t += ncl) {
+      for (int t = cid; t < total && !failed(); t += ncl) {
         const MoeTile x = moe_tile(p, s_first, s_cnt, t);
         if (x.nn <= 0) continue;
         const int a = tile & 1, use = tile >> 1;
-        if (use > 0 && !wait(acc_empty + 8 * a, (use - 1) & 1)) break;
+        if (use > 0 && !wait_warp(acc_empty + 8 * a, (use - 1) & 1)) break;
         tc_fence_after();
         const uint32_t idesc = umma_idesc_f16(DLTI_BF16, 256, (x.nn + 31) & ~31, false, false), d = tmem + a * 256;
         for (int kb = 0; kb < nkb; ++kb) {
-          if (!wait(full + 8 * s, round & 1)) break;
+          if (!wait_warp(full + 8 * s, round & 1)) break;
           tc_fence_after();
           const uint32_t sm = base + s * stage_bytes;
           const DescLoHi da = desc_split(sm, 0, 1024), db = desc_split(sm + MG_A_BYTES, 0, 1024);
@@ -370,7 +375,7 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
       const int i0 = threadIdx.x - 64;
       if (i0 < x.nn) dst[i0] = UP ? s_row[x.e] + x.n0 + i0 : p.lists[(long long)x.e * p.cap + x.n0 + i0];
       asm volatile("bar.sync 1, 256;" ::: "memory");
-      const bool ok = wait(acc_full + 8 * a, use & 1);
+      const bool ok = wait_warp(acc_full + 8 * a, use & 1);
       tc_fence_after();
       const uint32_t d = tmem + ((uint32_t)(quarter * 32) << 16) + a * 256;
       const int row = x.m * 256 + (int)rank * 128 + quarter * 32 + lane;
@@ -435,22 +440,22 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
   } else if (UP) {
     // rows past the list keep what their shared memory held: their columns are dropped
     const int g = (warp - 10) + lane * MG_GATHERS;          // a short list's copies are spread over the warps too
-    if (g < 32) {
-      int s = 0, round = 0;
-      for (int t = cid; t < total && !*fail; t += ncl) {
-        const MoeTile x = moe_tile(p, s_first, s_cnt, t);
-        if (x.nn <= 0) continue;
-        const int nh = ((x.nn + 31) & ~31) >> 1, first = (int)rank * nh, n = min(nh, x.nn - first);
-        const bool mine = 4 * g < n;
-        int src[4];
+    int s = 0, round = 0;
+    for (int t = cid; t < total && !failed(); t += ncl) {
+      const MoeTile x = moe_tile(p, s_first, s_cnt, t);
+      if (x.nn <= 0) continue;
+      const int nh = ((x.nn + 31) & ~31) >> 1, first = (int)rank * nh, n = min(nh, x.nn - first);
+      const bool mine = g < 32 && 4 * g < n;
+      int src[4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
-          src[i] = mine ? (int)min((unsigned)p.lists[(long long)x.e * p.cap + x.n0 + first + min(4 * g + i, n - 1)] / p.div, (unsigned)p.x_rows - 1) : 0;
-        for (int kb = 0; kb < nkb; ++kb) {
-          if (round > 0 && !wait(empty + 8 * s, (round - 1) & 1)) break;
-          if (mine) tma_gather4_2sm(base + s * stage_bytes + MG_A_BYTES + g * 512, &tx, lead_full + 8 * s, kb * 64, src[0], src[1], src[2], src[3]);
-          if (++s == p.stages) { s = 0; ++round; }
-        }
+      for (int i = 0; i < 4; ++i)
+        src[i] = mine ? (int)min((unsigned)p.lists[(long long)x.e * p.cap + x.n0 + first + min(4 * g + i, n - 1)] / p.div, (unsigned)p.x_rows - 1) : 0;
+      for (int kb = 0; kb < nkb; ++kb) {
+        if (round > 0 && !wait_warp(empty + 8 * s, (round - 1) & 1)) break;
+        if (mine) tma_gather4_2sm(base + s * stage_bytes + MG_A_BYTES + g * 512, &tx, lead_full + 8 * s, kb * 64, src[0], src[1], src[2], src[3]);
+        __syncwarp();
+        if (lane == 0) mbar_arrive(passed + 8 * s);
+        if (++s == p.stages) { s = 0; ++round; }
       }
     }
   }
