@@ -24,6 +24,8 @@
 //
 // Replaces PyTorch SDPA (mem-efficient / math kernels on the reference's V100; FlashAttention-2
 // mma.sync code elsewhere) — SURVEY.md N5, O6, S5.
+#include <cstring>
+
 #include "common.cuh"
 
 #include <cstdlib>
@@ -43,6 +45,10 @@ constexpr int BWD_THREADS = 576;  // backward: producer, mma, 16 softmax warps (
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float LN2 = 0.6931471805599453f;
 
+struct SoftCap {
+  float a, c, f;         // scale / cap; cap in log2 units; factor of the exponent of e^(2 x)
+  uint64_t d[6];         // polynomial in (q . k)^2, each coefficient twice
+};
 struct AttnParams {
   const int* cu_seqlens;
   int H, KV;
@@ -62,13 +68,65 @@ struct AttnParams {
   const float* sink;     // optional [H]: one more term exp(sink) in the softmax denominator, without a value
   int vdim;              // value columns of a head that are written, head h at column h * vdim of O (0: 128)
   int window;            // > 0: a row sees itself and the window - 1 rows before it
-  float cap;             // CAP form: scores become cap tanh(score / cap)
+  SoftCap soft;          // CAP form: scores become cap tanh(score / cap)
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// two fp32 operations in one instruction
+__device__ __forceinline__ uint64_t f32x2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ float2 unpack_f32x2(uint64_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma_x2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul_x2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t add_x2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+// Products q . k as capped scores log2(e) cap tanh(s scale / cap). Where every |s scale / cap| is at most 0.75 an odd polynomial
+// (minimax fit of tanh there, absolute error 1e-8) takes the place of an exponential and a reciprocal each.
+__device__ __forceinline__ uint64_t cap_small(const SoftCap& k, uint64_t s) {
+  const uint64_t u = mul_x2(s, s);
+  uint64_t r = fma_x2(u, k.d[5], k.d[4]);
+#pragma unroll
+  for (int i = 3; i >= 0; --i) r = fma_x2(u, r, k.d[i]);
+  return mul_x2(s, r);
+}
+__device__ __forceinline__ float cap_any(const SoftCap& k, float s) { return fmaf(-2.f * k.c, __fdividef(1.f, 1.f + ex2_approx(s * k.f)), k.c); }
+SoftCap soft_cap(float scale, float cap) {
+  static const double poly[6] = {0.9999998324675243, -0.3333247087670237, 0.13320579466592894, -0.05314925351405913, 0.019237222771406357, -0.004493446792158483};
+  SoftCap k;
+  k.a = scale / cap;
+  k.c = cap * LOG2E;
+  k.f = 2.f * LOG2E * scale / cap;
+  double f = (double)scale * 1.4426950408889634, a2 = (double)scale / cap * scale / cap;
+  for (int i = 0; i < 6; ++i, f *= a2) {
+    const float x = (float)(f * poly[i]);
+    uint32_t b;
+    std::memcpy(&b, &x, 4);
+    k.d[i] = (uint64_t)b << 32 | b;
+  }
+  return k;
 }
 
 __device__ __forceinline__ uint32_t swz_off(int row, int chunk16) {
@@ -925,11 +983,27 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
 #pragma unroll
         for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(tS + c * 32, *reinterpret_cast<uint32_t(*)[32]>(v + 32 * c));
         tmem_wait_ld();
+        float top = -INFINITY;                    // CAP: the largest score of the block, seen or not
         if constexpr (CAP) {
-          const float c = p.cap * LOG2E, c2 = -2.f * c, f = 2.f * LOG2E * p.scale / p.cap;
+          float low = INFINITY;
 #pragma unroll
-          for (int i = 0; i < 128; ++i)
-            v[i] = __float_as_uint(fmaf(c2, __fdividef(1.f, 1.f + ex2_approx(__uint_as_float(v[i]) * f)), c));
+          for (int i = 0; i < 128; ++i) {
+            top = fmaxf(top, __uint_as_float(v[i]));
+            low = fminf(low, __uint_as_float(v[i]));
+          }
+          if (__all_sync(0xffffffffu, fmaxf(top, -low) * p.soft.a <= 0.75f)) {
+#pragma unroll
+            for (int i = 0; i < 128; i += 2) {
+              const float2 x = unpack_f32x2(cap_small(p.soft, f32x2(__uint_as_float(v[i]), __uint_as_float(v[i + 1]))));
+              v[i] = __float_as_uint(x.x);
+              v[i + 1] = __float_as_uint(x.y);
+            }
+            top = unpack_f32x2(cap_small(p.soft, f32x2(top, top))).x;
+          } else {
+#pragma unroll
+            for (int i = 0; i < 128; ++i) v[i] = __float_as_uint(cap_any(p.soft, __uint_as_float(v[i])));
+            top = cap_any(p.soft, top);
+          }
         }
         float mx = -INFINITY;
         if (SPLIT && p.window > 0 && (qbX - j) * 128 + 127 >= p.window) {     // some row's window starts in this block
@@ -945,6 +1019,8 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
             if (i > r) v[i] = __float_as_uint(-INFINITY);
             mx = fmaxf(mx, __uint_as_float(v[i]));
           }
+        } else if constexpr (CAP) {
+          mx = top;
         } else {
 #pragma unroll
           for (int i = 0; i < 128; ++i) mx = fmaxf(mx, __uint_as_float(v[i]));
@@ -1109,7 +1185,8 @@ DLTI_API int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, cons
   AttnParams p{};
   p.cu_seqlens = cu_seqlens; p.H = H; p.KV = KV; p.W = (H + 2 * KV) * HD;
   p.O = out; p.ldo = ldo; p.T_total = T_total; p.scale = scale; p.dtype = DLTI_BF16; p.gate = gate; p.sink = sink;
-  p.seq_q0 = seq_q0; p.seq_out0 = seq_out0; p.vdim = vdim; p.window = window; p.cap = cap;
+  p.seq_q0 = seq_q0; p.seq_out0 = seq_out0; p.vdim = vdim; p.window = window;
+  if (cap > 0.f) p.soft = soft_cap(scale, cap);
   CUtensorMap tm;
   const int rc = make_map(&tm, qkv, T_total, p.W, 128);
   if (rc) return rc;

@@ -532,7 +532,7 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restri
 
 template <typename T, bool ACC, int W>
 int launch_route(const RouteParams& p, cudaStream_t st) {
-  const int per = p.T >= 4096 ? 8 : p.T >= 1024 ? 2 : 1, tokens = ROUTE_WARPS * per;
+  const int per = p.T >= 4096 ? 2 : 1, tokens = ROUTE_WARPS * per;
   const int rb = p.E ? (int)((p.T + tokens - 1) / tokens) : 0;
   const int ab = p.ff ? grid_for(p.T * (p.ff / W), 32 * ROUTE_WARPS) : 0;
   const size_t smem = p.E ? (size_t)(p.E + 2 * tokens * p.top + ROUTE_WARPS * (p.E + p.groups)) * 4 : 0;

@@ -604,9 +604,9 @@ __global__ void __launch_bounds__(256) qkv_rows_kernel(const QkvRowParams p) {
 }
 
 // the same with the row in registers: 16-bit T, VPT pieces of 8 a thread, every load issued before the sums
-template <typename T, bool ACC, int VPT>
-__global__ void __launch_bounds__(128) qkv_rows_vec_kernel(const QkvRowParams p) {
-  __shared__ float2 red[4];
+template <typename T, bool ACC, int VPT, int THREADS>
+__global__ void __launch_bounds__(THREADS) qkv_rows_vec_kernel(const QkvRowParams p) {
+  __shared__ float2 red[THREADS / 32];
   griddep_wait();
   griddep_launch();
   const long long t = blockIdx.x;
@@ -617,12 +617,12 @@ __global__ void __launch_bounds__(128) qkv_rows_vec_kernel(const QkvRowParams p)
   float f[VPT][8], sq = 0.f, sk = 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
-    const int x = (threadIdx.x + i * 128) * 8;
+    const int x = (threadIdx.x + i * THREADS) * 8;
     if (x < nq + nk + nv) take_n<T, ACC, 8>(row, x < nq ? p.oq + x : x < nq + nk ? p.ok + x - nq : p.ov + x - nq - nk, f[i]);
   }
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
-    const int x = (threadIdx.x + i * 128) * 8;
+    const int x = (threadIdx.x + i * THREADS) * 8;
     if (x >= nq + nk + nv) continue;
     if (p.bias) {
       float b[8];
@@ -644,14 +644,19 @@ __global__ void __launch_bounds__(128) qkv_rows_vec_kernel(const QkvRowParams p)
     sk = warp_sum(sk);
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(sq, sk);
     __syncthreads();
-    const float2 a = red[0], b = red[1], c = red[2], d = red[3];
-    rq = rsqrtf((a.x + b.x + c.x + d.x) / (float)nq + p.eps);
-    rk = rsqrtf((a.y + b.y + c.y + d.y) / (float)nk + p.eps);
+    sq = sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < THREADS / 32; ++w) {
+      sq += red[w].x;
+      sk += red[w].y;
+    }
+    rq = rsqrtf(sq / (float)nq + p.eps);
+    rk = rsqrtf(sk / (float)nk + p.eps);
   }
   const float share = p.first ? p.share[0] : 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
-    const int x = (threadIdx.x + i * 128) * 8;
+    const int x = (threadIdx.x + i * THREADS) * 8;
     if (x >= nq + nk + nv) continue;
     const bool is_q = x < nq, is_v = x >= nq + nk;
     const int y = is_q ? x : is_v ? x - nq - nk : x - nq, hd = is_v ? p.vdim : p.dim, h = y / hd, c = y - h * hd;
@@ -1099,14 +1104,16 @@ DLTI_API int dlti_qkv_rows(const void* proj, long long ld, int oq, int ok, int o
   const int pieces = ((H + G) * dim + G * vdim) / 8;
   if (vec && pieces <= 128 * 12 &&
       ((reinterpret_cast<uintptr_t>(bias) | reinterpret_cast<uintptr_t>(qn) | reinterpret_cast<uintptr_t>(kn)) & 15) == 0) {
-#define QR_CASE(V)                                                                                                          \
-  if (pieces <= 128 * V) {                                                                                                  \
-    auto kern = acc ? qkv_rows_vec_kernel<B, true, V> : qkv_rows_vec_kernel<B, false, V>;                                    \
-    DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, kern, dim3((unsigned)tokens), dim3(128), 0, st, p));                             \
+    // a whole row's loads in flight: many threads in small steps, many rows in large ones
+#define QR_CASE(V, TH)                                                                                                      \
+  if (pieces <= TH * V) {                                                                                                   \
+    auto kern = acc ? qkv_rows_vec_kernel<B, true, V, TH> : qkv_rows_vec_kernel<B, false, V, TH>;                            \
+    DLTI_CUDA_CHECK(dlti_launch_pdl(tokens, kern, dim3((unsigned)tokens), dim3(TH), 0, st, p));                              \
     dlti_count_launch();                                                                                                    \
     return 0;                                                                                                               \
   }
-    QR_CASE(1) QR_CASE(2) QR_CASE(3) QR_CASE(4) QR_CASE(6) QR_CASE(8) QR_CASE(12)
+    if (tokens <= 512) { QR_CASE(1, 256) QR_CASE(1, 512) QR_CASE(2, 512) QR_CASE(3, 512) }
+    QR_CASE(1, 128) QR_CASE(2, 128) QR_CASE(3, 128) QR_CASE(4, 128) QR_CASE(6, 128) QR_CASE(8, 128) QR_CASE(12, 128)
 #undef QR_CASE
   }
   auto kern = vec ? (acc ? qkv_rows_kernel<B, true, 8> : qkv_rows_kernel<B, false, 8>)
