@@ -348,7 +348,8 @@ int dlti_sample(const void* logits, long long ld, int batch, int V, const float*
                 unsigned long long step, long long* out, float* out_logprob, int dtype,
                 dlti_stream_t stream);
 
-/* ---- Layer-stack models (models/stack.py): csrc/stack.cu, streams.cu, recurrent.cu, attention_paged.cu, latent.cu, gemm_f32.cu. Row pitches (*_ld) in
+/* ---- Layer-stack models (models/stack.py): csrc/stack.cu, streams.cu, recurrent.cu, attention_paged.cu, latent.cu, dyt.cu, moe.cu, delta.cu,
+ * gemm_f32.cu. Row pitches (*_ld) in
  * elements. Sequences of a step: the first nd are single rows, sequence nd + i has rows nd + cu[i] ... nd + cu[i+1]; ctx[s] = tokens
  * of sequence s after the step, rseq[t] = sequence of row t, sslot[s] = its state slot (-1 = none). */
 /* C[M,N] = A[M,K] * B[N,K]^T in true fp32 (no TF32) */
@@ -357,8 +358,8 @@ int dlti_gemm_f32(const float* A, const float* B, float* C, int M, int N, int K,
 /* x[t] = table[ids[t]] as fp32; xa (16-bit, may be NULL) = the same rows */
 int dlti_embed_rows(const long long* ids, const void* table, float* x, void* xa, long long xa_ld, long long tokens, int
     d, long long vocab, int dtype, dlti_stream_t stream);
-/* out = acc, acc = 0 (fp32 logits of the decode GEMM) */
-int dlti_take_rows(float* acc, float* out, long long rows, int cols, dlti_stream_t stream);
+/* out = scale * acc, acc = 0 (fp32 logits of the decode GEMM) */
+int dlti_take_rows(float* acc, float* out, float scale, long long rows, int cols, dlti_stream_t stream);
 /* x += RMSnorm(y) * w (1 + w with one_plus), fp32 residual x [rows,d]; xa (may be NULL) = x in dtype.
  * acc: y is the fp32 accumulator of dlti_gemm_skinny, zero on return (also below) */
 int dlti_post_norm_add(const void* y, long long y_ld, float* x, const float* w, void* xa, long long xa_ld, long long
@@ -372,9 +373,9 @@ int dlti_gemm_relu2_2cta(const void* X, const void* W, void* Hout, int M, int N,
 /* h = relu(u)^2 over the first ff columns */
 int dlti_relu2(const void* u, long long u_ld, void* h, long long h_ld, long long rows, int ff, int acc, int dtype,
     dlti_stream_t stream);
-/* norm over `groups` parts of a row: gate_first ? norm(y * silu(gate)) * w : norm(y) * w * sigmoid(gate) */
+/* norm over `groups` parts of a row. mode 0: norm(y) * w * sigmoid(gate), 1: norm(y * silu(gate)) * w, 2: norm(y) * w * silu(gate) */
 int dlti_gated_norm(const void* y, long long y_ld, const void* gate, long long g_ld, const float* w, void* out, long
-    long o_ld, long long rows, int n, int groups, float eps, int gate_first, int acc, int dtype, dlti_stream_t stream);
+    long o_ld, long long rows, int n, int groups, float eps, int mode, int acc, int dtype, dlti_stream_t stream);
 /* projection rows (sections at columns oq/ok/ov/og; ok, og < 0 = absent) -> normed and rotated q, k and v into the paged
  * cache at slots[t] (-1 = skip), sigmoid of the head gates. kp/vp: also packed k, v rows; dst: packed row of row t >= nd */
 int dlti_qk_norm_rope_cache(const void* proj, long long ld, int oq, int ok, int ov, int og, const float* qn, const
@@ -382,13 +383,21 @@ int dlti_qk_norm_rope_cache(const void* proj, long long ld, int oq, int ok, int 
     long* slots, void* kc, void* vc, int kd, int vd, void* q, long long q_ld, int q_hd, void* kp, void* vp, const int*
     dst, int nd, float* gate, long long tokens, int H, int G, int dim, int vdim, int acc, int dtype, dlti_stream_t
     stream);
-/* packed rows[i] <- zero queries, cached keys and values of slots[i] (portions that continue a chunk) */
+/* whole projection rows + bias -> q and k normed over all their heads, v mixed with `first` (share[0] of it); own = v before mixing. Null:
+ * bias, qn and kn, first and share, own; kp, vp, dst as above */
+int dlti_qkv_rows(const void* proj, long long ld, int oq, int ok, int ov, const float* bias, const float* qn, const float* kn, float eps,
+    const void* first, long long f_ld, const float* share, void* own, long long own_ld, const long long* slots, void* kc, void* vc, int kd,
+    int vd, void* q, long long q_ld, int q_hd, void* kp, void* vp, const int* dst, int nd, long long tokens, int H, int G, int dim, int vdim,
+    int acc, int dtype, dlti_stream_t stream);
+/* packed rows[i] <- zero queries, cached keys and values of slots[i] (portions that continue a chunk or a window) */
 int dlti_prefix_rows(void* packed, long long ld, int hd, const int* rows, const int* slots, const void* kc, const void*
     vc, int kd, int vd, int H, int G, long long n, dlti_stream_t stream);
-/* silu(causal convolution) of channels [col, col+C) of the rows of every sequence; inputs before the step come from state */
+/* silu(causal convolution) of channels [col, col+C) of the rows of every sequence; inputs before the step come from state. acc: raw = the
+ * accumulator's columns in dtype, from tail0 on (tail not null) in fp32 to tail */
 int dlti_short_conv(const void* src, long long ld, int col, int C, int taps, const float* w, const float* b, int w_ld,
     const void* state, const int* sslot, const int* rseq, const int* ctx, const int* cu, int nd, void* out, long long
-    o_ld, void* raw, long long raw_ld, int raw_n, long long rows, int acc, int dtype, dlti_stream_t stream);
+    o_ld, void* raw, long long raw_ld, int raw_n, float* tail, long long tail_ld, int tail0, long long rows, int acc, int dtype,
+    dlti_stream_t stream);
 /* S <- a S + k (s v)^T, o = S^T q + D v token by token over sequences [seq0, seq0+nseq); a constant (decay) or from raw step
  * sizes (dt, dt_bias, A_log); state [slots, heads, N, P] fp32; tail job: new convolution state from conv_src */
 int dlti_linear_scan(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long v_ld, int
@@ -404,25 +413,26 @@ int dlti_linear_scan_chunked(const void* q, long long q_ld, const void* k, long 
     conv_C, void* conv_state, dlti_stream_t stream);
 /* x = silu(x) in place */
 int dlti_silu_rows(void* x, long long ld, long long rows, int n, int dtype, dlti_stream_t stream);
-/* paged attention, one warp per (row, head), fp32 arithmetic; chunk > 0: a position sees its own chunk only. sink [H] (may be NULL, also
- * below): one more term exp(sink) in a head's softmax denominator */
+/* paged attention, one warp per (row, head), fp32 arithmetic; chunk > 0: a position sees its own chunk only; window > 0: itself and the
+ * window - 1 positions before it; cap > 0: scores become cap tanh(score / cap). sink [H] (may be NULL): one more term exp(sink) in a head's
+ * softmax denominator (all also below) */
 int dlti_attn_rows(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd, const int*
     tables, int max_blocks, int bs, const int* ctx, const int* rseq, const int* pos, int H, int G, int dim, int vdim,
-    int chunk, float scale, const float* gate, const float* sink, void* out, long long o_ld, long long rows, int dtype,
+    int chunk, int window, float scale, float cap, const float* gate, const float* sink, void* out, long long o_ld, long long rows, int dtype,
     dlti_stream_t stream);
 /* paged attention of prompt portions (bf16, heads <= 256) */
 int dlti_attn_paged_prefill(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
     const int* tables, int max_blocks, int bs, const int* ctx, const int* cu, int nd, int nseq, int max_rows, int H,
-    int G, int dim, int vdim, int chunk, float scale, const float* gate, const float* sink, void* out, long long o_ld, dlti_stream_t
+    int G, int dim, int vdim, int chunk, int window, float scale, float cap, const float* gate, const float* sink, void* out, long long o_ld, dlti_stream_t
     stream);
 /* paged attention of decode rows (bf16, grouped heads, split over CTAs); ws: batch * H * splits * (vdim + 2) floats */
 int dlti_attn_paged_decode(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
     const int* tables, int max_blocks, int bs, const int* ctx, int batch, int H, int G, int dim, int vdim, int chunk,
-    float scale, const float* gate, const float* sink, int splits, float* ws, void* out, long long o_ld, dlti_stream_t stream);
+    int window, float scale, float cap, const float* gate, const float* sink, int splits, float* ws, void* out, long long o_ld, dlti_stream_t stream);
 /* varlen causal attention with the softmax weights as two bf16 terms; see attention.cu */
 int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const float* sink, const int* cu_seqlens, const int*
-    seq_q0, const int* seq_out0, int batch, int max_seqlen, long long T_total, int H, int KV, int vdim, float scale,
-    dlti_stream_t stream);
+    seq_q0, const int* seq_out0, int batch, int max_seqlen, long long T_total, int H, int KV, int vdim, int window,
+    float scale, float cap, dlti_stream_t stream);
 
 /* mLSTM: the recurrence above with exponential gates, a running maximum and a normaliser; see recurrent.cu. gates [rows, >= 2 heads]
  * raw fp32 (input, forget), vec [slots, heads, ceil(P / 32), N + 1] */
@@ -460,6 +470,34 @@ int dlti_head_gemm(const void* a, long long a_ld, int a_hd, const void* b, long 
 int dlti_latent_decode(const void* q, const void* cache, int pitch, int rank, const int* tables, int max_blocks, int bs, const int* ctx,
     const int* rseq, const int* pos, long long rows, int H, float scale, const float* sink, const float* gate, int heads_per_cta, int
     splits, float* ws, void* out, int o_hd, dlti_stream_t stream);
+
+/* dyt.cu: dynamic tanh norms n(x) = tanh(alpha x) * w + b around sublayers. x = table[ids] * scale (fp32), h = n(x) */
+int dlti_tanh_embed(const long long* ids, const void* table, long long vocab, float scale, const float* alpha, const float* w, const float*
+    b, float* x, void* h, long long h_ld, long long tokens, int d, int dtype, dlti_stream_t stream);
+/* x += n1(y + sum_k weights[t, k] rows[t * top + k]), h = n2(x); y, rows (weights, counts), w2 (h) may be NULL; counts are cleared */
+int dlti_tanh_between(float* x, const void* y, long long y_ld, const void* rows, long long r_ld, const float* weights, int top, int* counts,
+    int ncounts, const float* alpha1, const float* w1, const float* b1, const float* alpha2, const float* w2, const float* b2, void* h,
+    long long h_ld, long long tokens, int d, int acc, int dtype, dlti_stream_t stream);
+/* h[i] = n(x[idx[i]]); idx NULL = all rows */
+int dlti_tanh_rows(const float* x, const long long* idx, const float* alpha, const float* w, const float* b, void* h, long long h_ld, long
+    long rows, int d, int dtype, dlti_stream_t stream);
+/* moe.cu: routing of the logits z (E > 0): sigmoid scores, groups, the top experts by score + corr, their scores made to sum to scale ->
+ * wgt [T, top] and, per expert, the list of its pairs token * top + choice (lists [E, T], counts [E] zero on entry); and / or (ff > 0)
+ * the gated activation of projection columns og (gate) and ou (up): silu(g) u, with a limit g sigmoid(1.702 g) (u + 1) of clipped values */
+int dlti_moe_route(const float* z, long long z_ld, int col, const float* corr, int E, int top, int groups, int keep, float scale, float* wgt,
+    int* lists, int* counts, const void* p, long long p_ld, int og, int ou, int ff, float limit, void* h, long long h_ld, long long T, int acc,
+    int dtype, dlti_stream_t stream);
+/* grouped GEMM over the lists. up: rows X[pair / div] times gate / up rows 2 r, 2 r + 1 of W_e, out = activation, one list after the other;
+ * else rows of X in that order times W_e, out[pair]. W_e = rows e * wrows ... of W */
+int dlti_moe_gemm(const void* X, long long x_ld, long long x_rows, int div, const void* W, long long w_ld, int wrows, int E, const int* lists,
+    const int* counts, int cap, int rows, int up, int K, float limit, void* out, long long o_ld, int o_rows, int dtype, dlti_stream_t stream);
+/* delta.cu: gated delta rule S <- g S, u = b (v - S^T k), S <- S + k u^T, o = S^T q over sequences [seq0, seq0+nseq); gates [rows, >= 2
+ * heads] raw fp32 (decay, step). ws NULL: token by token; else prompts in chunks of 64 tokens (bf16) with dlti_delta_workspace bytes */
+int dlti_delta_scan(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long v_ld, const float* gates, long
+    long g_ld, const float* A_log, const float* dt_bias, float* state, const int* sslot, const int* ctx, const int* cu, int nd, int seq0, int
+    nseq, int heads, int groups, int N, int P, void* out, long long o_ld, const void* conv_src, long long conv_ld, int conv_col, int
+    conv_rows, int conv_C, void* conv_state, void* ws, int longest, int dtype, dlti_stream_t stream);
+long long dlti_delta_workspace(long long rows, int nseq, int heads);
 
 #ifdef DLTI_ATTN_TRACE
 /* Developer builds only (-DDLTI_ATTN_TRACE): clock64() timeline of CTA (0,0,0) of the last backward

@@ -397,6 +397,35 @@ def test_mixture_of_experts(device, dtype, T, d, e):
         assert float((got - want)[clear].norm() / want[clear].norm()) < tol(dtype, 3e-6, 8e-3)
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("T,skew", [(1, 0), (16, 0), (64, 3), (300, 0), (300, 4), (2500, 1)])
+def test_expert_gemms_with_long_rows(T, skew):
+    """Dozens of k blocks, lists from none to thousands of rows: the stages of the kernels go round many times while some of their
+    warps have nothing to copy."""
+    g, E, top, d, ff = torch.Generator("cuda").manual_seed(T), 48, 4, 1544, 200
+    e = MoeMlp(E, top, ff, 2.0, 4, 3)
+    rnd_ = lambda *s: torch.randn(*s, device="cuda", generator=g).to(BF16)
+    h, wu, wd = rnd_(T, d), rnd_(E, 2 * ff, d) * d ** -0.5, rnd_(E, d, ff) * ff ** -0.5
+    z = torch.randn(T, E, device="cuda", generator=g) + skew * torch.randn(E, device="cuda", generator=g)
+    _, lists, counts = M._route(None, z, 0, torch.zeros(E, device="cuda"), e)
+    for _ in range(3):
+        a, out = K.act(T * top, ff, BF16, "cuda"), torch.full((T * top, d), 9.0, dtype=BF16, device="cuda")
+        M.grouped_gemm(h, wu, lists, counts, a, rows=ff, pairs_per_row=top, up=True, limit=2.0)
+        M.grouped_gemm(a, wd, lists, counts, out, rows=d, pairs_per_row=1)
+        o = 0
+        for j in range(E):
+            pair = lists[j, :int(counts[j])].long().cpu()
+            x = h[(pair // top).cuda()].double().cpu()
+            p = {"gate": wu[j, 0::2].double().cpu(), "up": wu[j, 1::2].double().cpu(), "down": torch.eye(ff, dtype=torch.double)}
+            if len(pair):
+                mid = a[o:o + len(pair)].cpu()
+                assert rel(mid, R.clipped_expert(x, p, "", 2.0)) < 6e-3
+                assert rel(out[pair.cuda()], mid.double() @ wd[j].double().cpu().t()) < 6e-3
+            o += len(pair)
+        assert o == T * top
+    counts.zero_()
+
+
 # ---- delta rule --------------------------------------------------------------------------------------------
 def _delta_case(device, dtype, heads, groups, N_, P, cuts, A_log, dt_bias, seed=0, t=None, change=None):
     g = gen(N_ + P + seed)
