@@ -276,22 +276,27 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaParams p) {
     }
   }
   __syncthreads();
-  float x[CQ];
-  if (threadIdx.x < CQ) {                                  // column j of the inverse by forward substitution
-    const int j = threadIdx.x;
+  // The inverse I takes the place of the keys and queries. Its 16 x 16 blocks on the diagonal by forward substitution, a column a
+  // thread; then one diagonal of blocks after the other: I_ij = -I_ii sum_(j <= k < i) A_ik I_kj, an element a thread.
+  float* I = reinterpret_cast<float*>(smem);
+  static_assert(2 * L::QK >= CQ * L::AP * 4, "");
+  if (threadIdx.x < CQ) {
+    const int b = threadIdx.x & ~15, j = threadIdx.x & 15;
+    float x[16];
 #pragma unroll
-    for (int t = 0; t < CQ; ++t) {
-      float a0 = t == j ? 1.f : 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
-      const float4* row = reinterpret_cast<const float4*>(A + t * L::AP);
+    for (int t = 0; t < 16; ++t) {
+      float a0 = t == j ? 1.f : 0.f, a1 = 0.f;
+      const float4* row = reinterpret_cast<const float4*>(A + (b + t) * L::AP + b);
 #pragma unroll
       for (int q = 0; q < (t + 3) / 4; ++q) {
         const float4 c = row[q];                           // entries at and after the diagonal are zero
         a0 = fmaf(-c.x, x[4 * q], a0);
         if (4 * q + 1 < t) a1 = fmaf(-c.y, x[4 * q + 1], a1);
-        if (4 * q + 2 < t) a2 = fmaf(-c.z, x[4 * q + 2], a2);
-        if (4 * q + 3 < t) a3 = fmaf(-c.w, x[4 * q + 3], a3);
+        if (4 * q + 2 < t) a0 = fmaf(-c.z, x[4 * q + 2], a0);
+        if (4 * q + 3 < t) a1 = fmaf(-c.w, x[4 * q + 3], a1);
       }
-      x[t] = (a0 + a1) + (a2 + a3);
+      x[t] = a0 + a1;
+      I[(b + t) * L::AP + b + j] = x[t];
     }
   } else if (threadIdx.x >= 128 && threadIdx.x < 128 + CQ) {
     const int t = threadIdx.x - 128;
@@ -304,15 +309,46 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaParams p) {
     if (t == 0) v[4 * CQ] = ex2(last);
   }
   __syncthreads();
-  if (threadIdx.x < CQ)
+  {
+    const int r = threadIdx.x >> 4, c = threadIdx.x & 15;
+    auto row_dot = [&](const float* row, const float* col) {       // 16 elements of a row and of a column
+      float a0 = 0.f, a1 = 0.f;
 #pragma unroll
-    for (int t = 0; t < CQ; ++t) A[t * L::AP + threadIdx.x] = x[t];
-  __syncthreads();
+      for (int m = 0; m < 16; m += 4) {
+        const float4 f = *reinterpret_cast<const float4*>(row + m);
+        a0 = fmaf(f.x, col[m * L::AP], a0);
+        a1 = fmaf(f.y, col[(m + 1) * L::AP], a1);
+        a0 = fmaf(f.z, col[(m + 2) * L::AP], a0);
+        a1 = fmaf(f.w, col[(m + 3) * L::AP], a1);
+      }
+      return a0 + a1;
+    };
+#pragma unroll
+    for (int dist = 1; dist < 4; ++dist) {
+      float y[3];
+#pragma unroll
+      for (int bj = 0; bj + dist < 4; ++bj) {
+        float sum = 0.f;
+#pragma unroll
+        for (int k = bj; k < bj + dist; ++k)
+          sum += row_dot(A + ((bj + dist) * 16 + r) * L::AP + k * 16, I + k * 16 * L::AP + bj * 16 + c);
+        I[((bj + dist) * 16 + r) * L::AP + bj * 16 + c] = sum;
+      }
+      __syncthreads();
+#pragma unroll
+      for (int bj = 0; bj + dist < 4; ++bj)
+        y[bj] = -row_dot(I + ((bj + dist) * 16 + r) * L::AP + (bj + dist) * 16, I + (bj + dist) * 16 * L::AP + bj * 16 + c);
+      __syncthreads();
+#pragma unroll
+      for (int bj = 0; bj + dist < 4; ++bj) I[((bj + dist) * 16 + r) * L::AP + bj * 16 + c] = y[bj];
+      __syncthreads();
+    }
+  }
   uint4* frag = reinterpret_cast<uint4*>(ws);
   for (int i = warp; i < 16; i += 8) {
     const int w = i >> 2, kb = i & 3;
     if (kb > w) continue;
-    const float* a = A + (w * 16 + (lane >> 2)) * L::AP + kb * 16 + (lane & 3) * 2;
+    const float* a = I + (w * 16 + (lane >> 2)) * L::AP + kb * 16 + (lane & 3) * 2;
     uint32_t hi[4], lo[4];
 #pragma unroll
     for (int z = 0; z < 4; ++z) {
