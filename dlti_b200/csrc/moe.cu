@@ -257,7 +257,6 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
     mbar_fence_init();
   }
   griddep_wait();
-  griddep_launch();
   cluster_sync_all();
   if (warp == 1) {
     tmem_alloc2(slot, 512);
@@ -294,6 +293,7 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
   tc_fence_before();
   cluster_sync_all();
   tc_fence_after();
+  griddep_launch();                                        // only now: the next kernel may want tensor memory too
   const uint32_t tmem = __shfl_sync(0xffffffffu, *slot_ptr, 0);
   const int nkb = (p.K + 63) / 64;
   volatile int* fail = &s_fail;
