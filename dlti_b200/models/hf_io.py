@@ -51,6 +51,9 @@ class CheckpointReader:
     def has(self, name: str) -> bool:
         return name in self.weight_map
 
+    def shape(self, name: str) -> list[int]:
+        return self._file(name).get_slice(name).get_shape()
+
     def get(self, name: str, rows: tuple[int, int] | None = None,
             cols: tuple[int, int] | None = None) -> torch.Tensor:
         """Whole tensor or a [rows, cols] slice (only those bytes are read)."""

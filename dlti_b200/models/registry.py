@@ -13,7 +13,7 @@ from typing import Callable
 import torch
 
 from . import config as llama_config
-from . import latanex, logozen, sigosun
+from . import latanex, logozen, ridazen, sigosun
 
 
 @dataclass(frozen=True)
@@ -64,6 +64,10 @@ FAMILIES: dict[str, Family] = {
     latanex.ARCHITECTURE: Family(
         latanex.ARCHITECTURE, latanex.LatanexConfig, latanex.PRESETS, latanex.LatanexConfig.load, latanex.load_weights,
         lambda cfg, device, dtype, seed=0: latanex.from_state(cfg, latanex.random_state(cfg, seed, device), device, dtype),
+        _stack_runner, (torch.bfloat16, torch.float32)),
+    ridazen.ARCHITECTURE: Family(
+        ridazen.ARCHITECTURE, ridazen.RidazenConfig, ridazen.PRESETS, ridazen.RidazenConfig.load, ridazen.load_weights,
+        lambda cfg, device, dtype, seed=0: ridazen.from_state(cfg, ridazen.random_state(cfg, seed, device), device, dtype),
         _stack_runner, (torch.bfloat16, torch.float32)),
 }
 

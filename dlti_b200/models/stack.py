@@ -1,8 +1,8 @@
 """Models described layer by layer: each layer names its token mixer (softmax attention, latent attention, Mamba-2,
 lightning attention, mLSTM, gated delta rule) and its feed-forward (dense or a mixture of experts), with every size and
-constant a parameter; the model names how sublayers meet the residual. A design (models/sigosun.py, models/logozen.py,
-models/latanex.py) is a parser from its config.json to a `StackConfig` plus its tensor names; the weights container, the cache layout and the serving forward pass (serve/stack_runner.py) are shared
-by all of them.
+constant a parameter. The model names how sublayers meet the residual and which layers run several times. A design (models/sigosun.py, models/logozen.py,
+models/latanex.py, models/ridazen.py) is a parser from its config.json to a `StackConfig` plus its tensor names; the weights container,
+the cache layout and the serving forward pass (serve/stack_runner.py) are shared by all of them.
 
 Weights are kept as merged input projections, one GEMM per mixer. Every section of a merged projection and the row
 pitch of every matrix is rounded up to 8 elements, so any head count or width meets the 16-byte rules of the TMA
@@ -10,7 +10,9 @@ GEMMs; padding rows are zero and padding columns are never read.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+import math
+from dataclasses import dataclass
+from functools import cached_property
 
 import torch
 
@@ -32,6 +34,35 @@ class Rope:
 
 
 @dataclass(frozen=True)
+class QueryTemp:
+    """Queries at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
+    coef: float
+    every: int
+
+
+@dataclass(frozen=True)
+class DistanceBias:
+    """A learned number per head and bucket of the distance n = query position - key position, added to the scores. The first
+    rows // 2 buckets are single distances, the others grow evenly in ln n up to `far`; everything beyond is in the last one."""
+    rows: int
+    far: int
+
+    def bucket(self, n: int) -> int:
+        half = self.rows // 2
+        if n < half:
+            return n
+        return min(self.rows - 1, half + math.floor(math.log(n / half) / math.log(self.far / half) * (self.rows - half)))
+
+    @cached_property
+    def buckets(self) -> list[int]:
+        """The buckets of the distances 0, 1, ... below the first one from which on all are in the last bucket."""
+        out = [self.bucket(n) for n in range(self.far + 1)]
+        while out and out[-1] == self.rows - 1:
+            out.pop()
+        return out
+
+
+@dataclass(frozen=True)
 class AttentionMixer:
     heads: int
     kv_heads: int
@@ -49,6 +80,10 @@ class AttentionMixer:
     bias: bool = False             # on the q, k and v projections
     row_norm: bool = False         # RMS norm over all heads of q (and of k) at once
     v_mix: bool = False            # values are mixed with those of the first such layer, by one learned share per layer
+    conv: int = 0                  # > 0: taps of a causal convolution on each channel of q, k and v, before the norms
+    q_temp: QueryTemp | None = None
+    bias_by: DistanceBias | None = None
+    out_gate: bool = False         # every output element times sigmoid of its own projected number
 
     @property
     def reach(self) -> tuple[int, int]:
@@ -58,6 +93,11 @@ class AttentionMixer:
     def whole_rows(self) -> bool:
         """Queries, keys and values are made from whole projection rows (ops.stack.qkv_rows), not head by head."""
         return self.bias or self.row_norm or self.v_mix
+
+    @property
+    def conv_heads(self) -> bool:
+        """Queries, keys and values are made head by head by the op that also convolves and scales (ops.stack.conv_qkv)."""
+        return self.conv > 0 or self.q_temp is not None or self.out_gate
 
 
 @dataclass(frozen=True)
@@ -155,23 +195,40 @@ class DenseMlp:
 
 @dataclass(frozen=True)
 class MoeMlp:
-    """Mixture of clipped SwiGLU experts. The router's sigmoid scores pick `top` of them by score plus a correction, out of the
-    `keep` best of `groups` equal groups; the chosen scores, made to sum to `scale`, weigh the outputs."""
+    """Mixture of experts. score "sigmoid": the router's sigmoid scores pick `top` experts by score plus a correction, out of the
+    `keep` best of `groups` equal groups; the chosen scores, made to sum to `scale`, weigh the outputs. "softmax": the largest
+    logits (the correction is their bias) are picked, and weighed by their softmax among the chosen, times scale."""
     experts: int
     top: int
     ff: int
-    limit: float                   # gate <= limit, -limit <= up <= limit
+    limit: float = 0.0             # act "swiglu": gate <= limit, -limit <= up <= limit
     groups: int = 1
     keep: int = 1
     scale: float = 1.0
     shared_ff: int = 0             # > 0: one more expert of this size that runs for every token
     shared_limit: float = 0.0
+    shared_gate: bool = False      # the shared expert's output times sigmoid of one projected number per token
+    act: str = "swiglu"            # clipped; "relu2": no gate, square of relu
+    score: str = "sigmoid"
+
+    @property
+    def gated(self) -> bool:
+        return self.act == "swiglu"
 
 
 @dataclass(frozen=True)
 class Layer:
     mixer: AttentionMixer | LatentAttentionMixer | Mamba2Mixer | LightningMixer | MLstmMixer | DeltaMixer
     mlp: DenseMlp | MoeMlp | None = None
+
+
+@dataclass(frozen=True)
+class Loop:
+    """Layers start ... stop - 1 run `times` times in a row with the same weights, each pass on a cache and states of its own.
+    Before each pass but the first the embedding is added to the residual."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass
@@ -186,8 +243,14 @@ class StackConfig:
     streams: int = 0
     canon: int = 0
     tanh_norms: bool = False       # one residual, a dynamic tanh norm before and after every sublayer instead
+    pre_norm: bool = False         # one residual, RMS norms on the sublayer inputs instead
+    residual_mult: float = 1.0     # pre_norm: on everything that is added to the residual
+    # pre_norm, > 0: after each layer, proj(gelu(gate x) * e) with the RMS norm on it, e = this many numbers of the token for the layer
+    token_side: int = 0
+    loop: Loop | None = None
     embed_scale: float = 1.0
     logit_scale: float = 1.0
+    logit_softcap: float = 0.0     # > 0: logits become softcap * tanh(logit / softcap)
     max_position_embeddings: int = 8192        # only a default for the server's max_model_len
     bos_token_id: int = 1
     eos_token_id: int = 2
@@ -214,6 +277,15 @@ class StackConfig:
                 if m.whole_rows and (m.rope is not None or m.head_gate or m.kv_from is not None or m.qk_norm):
                     raise ValueError(f"layer {i}: biases, row norms and value mixing do not combine with rotations, head gates, head "
                                      "norms or shared keys")
+                if m.conv_heads and (m.whole_rows or m.rope is not None or m.head_gate or m.kv_from is not None):
+                    raise ValueError(f"layer {i}: convolutions, query temperatures and output gates do not combine with whole-row "
+                                     "projections, rotations, head gates or shared keys")
+                if m.bias_by is not None and (m.softcap or m.sink):
+                    raise ValueError(f"layer {i}: distance biases do not combine with capped scores or sinks")
+                if m.bias_by is not None and not 1 <= m.bias_by.rows // 2 < m.bias_by.far:
+                    raise ValueError(f"layer {i}: {m.bias_by.rows} distance buckets up to {m.bias_by.far}")
+                if m.q_temp is not None and m.q_temp.every < 1 or m.conv < 0:
+                    raise ValueError(f"layer {i}: query temperature {m.q_temp}, convolutions of {m.conv} taps")
                 src = self.v_mix_from(i)
                 if src is not None and (src.kv_heads, src.vdim) != (m.kv_heads, m.vdim):
                     raise ValueError(f"layer {i}: values are mixed with those of a layer of another shape")
@@ -235,14 +307,40 @@ class StackConfig:
             if isinstance(e, MoeMlp):
                 if e.experts % e.groups or not 1 <= e.keep <= e.groups or not 1 <= e.top <= e.keep * (e.experts // e.groups):
                     raise ValueError(f"layer {i}: {e.top} of {e.experts} experts from {e.keep} of {e.groups} groups")
-                if not self.tanh_norms:
-                    raise ValueError(f"layer {i}: mixtures of experts need the tanh norms, which add up their outputs")
+                if not self.tanh_norms and not self.pre_norm:
+                    raise ValueError(f"layer {i}: mixtures of experts need the tanh norms or pre-norms, which add up their outputs")
+                if e.act not in ("swiglu", "relu2") or e.score not in ("sigmoid", "softmax") or e.shared_gate and not e.shared_ff:
+                    raise ValueError(f"layer {i}: experts {e.act}, scores {e.score}, gate on a shared expert of {e.shared_ff}")
+                if e.score == "softmax" and e.groups > 1:
+                    raise ValueError(f"layer {i}: groups of experts need sigmoid scores")
         if self.streams and self.canon < 1:
             raise ValueError(f"canon taps {self.canon}: at least 1")
+        if (self.token_side or self.residual_mult != 1.0 or self.loop) and not self.pre_norm:
+            raise ValueError("token inputs, residual factors and loops need the pre-norms")
+        if self.loop is not None:
+            a, b, n = self.loop.start, self.loop.stop, self.loop.times
+            if not 0 <= a < b <= len(self.layers) or n < 1:
+                raise ValueError(f"layers {a} ... {b - 1} of {len(self.layers)} cannot run {n} times")
+            if any(getattr(l.mixer, "kv_from", None) is not None or getattr(l.mixer, "v_mix", False) for l in self.layers):
+                raise ValueError("layers on another layer's keys or values do not run in a loop")
 
     @property
     def num_hidden_layers(self) -> int:
         return len(self.layers)
+
+    @property
+    def runs(self) -> list[int]:
+        """The layers in the order in which a token passes them; each run has a cache and states of its own."""
+        n = len(self.layers)
+        if self.loop is None:
+            return list(range(n))
+        a, b = self.loop.start, self.loop.stop
+        return [*range(a), *(list(range(a, b)) * self.loop.times), *range(b, n)]
+
+    @property
+    def restarts(self) -> set[int]:
+        """The runs before which the embedding is added once more."""
+        return set() if self.loop is None else {self.loop.start + t * (self.loop.stop - self.loop.start) for t in range(1, self.loop.times)}
 
     def v_mix_from(self, i: int) -> AttentionMixer | None:
         """The layer whose values layer i mixes into its own (None: it mixes none, or is the first such layer itself)."""
@@ -252,7 +350,8 @@ class StackConfig:
     @property
     def has_state(self) -> bool:
         """Some layer carries recurrent state (or earlier inputs of a convolution) from token to token."""
-        return self.canon > 1 or any(not isinstance(l.mixer, (AttentionMixer, LatentAttentionMixer)) for l in self.layers)
+        return self.canon > 1 or any(l.mixer.conv > 1 if isinstance(l.mixer, AttentionMixer) else not isinstance(l.mixer, LatentAttentionMixer)
+                                     for l in self.layers)
 
     @property
     def reaches(self) -> list[tuple[int, int]]:
@@ -293,8 +392,8 @@ def mixer_sections(m) -> Sections:
         s = {"q": m.heads * m.dim}
         if m.kv_from is None:
             s |= {"k": m.kv_heads * m.dim, "v": m.kv_heads * m.vdim}
-        if m.head_gate:
-            s["g"] = m.heads
+        if m.head_gate or m.out_gate:
+            s["g"] = m.heads * (m.vdim if m.out_gate else 1)
         return Sections(**s)
     if isinstance(m, Mamba2Mixer):
         return Sections(z=m.inner, xbc=m.conv_channels, dt=m.heads)
@@ -307,14 +406,21 @@ def mixer_sections(m) -> Sections:
     return Sections(q=m.heads * m.dim, k=m.heads * m.dim, v=m.heads * m.vdim, g=m.heads * m.vdim)
 
 
+def conv_span(m: AttentionMixer) -> int:
+    """Columns of the merged projection that the convolutions of an attention layer cover: q, k, v and the padding between them."""
+    return sum(round8(n) for n in (m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim))
+
+
 def mixer_out(m) -> int:
     return m.heads * m.vdim
 
 
 def mlp_sections(e: DenseMlp | MoeMlp) -> Sections:
-    """Rows of a feed-forward's merged input projection (of an MoeMlp: its shared expert and, last, its router)."""
+    """Rows of a feed-forward's merged input projection (of an MoeMlp: its shared expert and, last, what stays
+    fp32: its router and the shared expert's gate)."""
     if isinstance(e, MoeMlp):
-        return Sections(**({"gate": e.shared_ff, "up": e.shared_ff} if e.shared_ff else {}), router=e.experts)
+        shared = ({"gate": e.shared_ff} if e.gated else {}) | {"up": e.shared_ff}
+        return Sections(**(shared if e.shared_ff else {}), router=e.experts, **({"sg": 1} if e.shared_gate else {}))
     return Sections(gate=e.ff, up=e.ff) if e.act == "swiglu" else Sections(up=e.ff)
 
 
@@ -339,6 +445,7 @@ class StackWeights:
         self.final_norm = vec(d)
         if cfg.tanh_norms:
             self.final_norm_b, self.final_norm_alpha = vec(d), vec(1)
+        self.side_embed = torch.zeros(cfg.vocab_size, len(cfg.layers) * cfg.token_side, dtype=dtype, device=device) if cfg.token_side else None
         self.lora = None
         self.layers: list[dict] = []
         for l in cfg.layers:
@@ -357,6 +464,10 @@ class StackWeights:
                     w["sink"] = vec(m.heads)
                 if m.v_mix:
                     w["v_mix"] = vec(1)
+                if m.conv:                                 # tap-major, over the convolved sections with the padding between them
+                    w["conv"] = torch.zeros(m.conv, conv_span(m), dtype=torch.float32, device=device)
+                if m.bias_by is not None:
+                    w["rel"] = torch.zeros(m.bias_by.rows, m.heads, dtype=torch.float32, device=device)
             elif isinstance(m, Mamba2Mixer):
                 # convolution weights tap-major: one tap's channels are contiguous
                 w |= {"conv": torch.zeros(m.conv, round8(m.conv_channels), dtype=torch.float32, device=device),
@@ -382,7 +493,7 @@ class StackWeights:
                 def stack(rows, cols):
                     return torch.zeros(e.experts, round8(rows), round8(cols), dtype=dtype, device=device)[:, :, :cols]
                 # gate and up rows of an expert alternate
-                w |= {"correction": vec(e.experts), "e_up": stack(2 * e.ff, d), "e_down": stack(d, e.ff)}
+                w |= {"correction": vec(e.experts), "e_up": stack((2 if e.gated else 1) * e.ff, d), "e_down": stack(d, e.ff)}
                 if e.shared_ff:
                     w["w_down"] = mat(d, e.shared_ff)
             elif e is not None:
@@ -392,6 +503,8 @@ class StackWeights:
             if cfg.tanh_norms:
                 w |= {k: t for q in ((1, 2) if e is not None else (1,)) for n in (f"norm{q}", f"norm{q}b")
                       for k, t in ((n, vec(d)), (n + ".b", vec(d)), (n + ".alpha", vec(1)))}
+            if cfg.token_side:
+                w |= {"side_gate": mat(cfg.token_side, d), "side_proj": mat(d, cfg.token_side), "norm3": vec(d)}
             if cfg.streams:
                 for q in (1, 2) if l.mlp is not None else (1,):
                     w |= {f"hc{q}.in": vec(cfg.streams), f"hc{q}.out": vec(cfg.streams),
@@ -404,6 +517,8 @@ class StackWeights:
         yield from (self.embed, self.lm_head, self.final_norm)
         if self.cfg.tanh_norms:
             yield from (self.final_norm_b, self.final_norm_alpha)
+        if self.side_embed is not None:
+            yield self.side_embed
         for w in self.layers:
             yield from w.values()
 
@@ -435,7 +550,10 @@ class StackWeights:
         """Weights that the kernels want in another arrangement."""
         for i, (l, w) in enumerate(zip(self.cfg.layers, self.layers)):
             m = l.mixer
-            if isinstance(m, LatentAttentionMixer) and self.device.type == "cuda" and self.dtype != torch.float32:
+            if isinstance(m, AttentionMixer) and m.bias_by is not None:
+                # per head and distance, less that of the last bucket: softmax does not change, and keys beyond need nothing
+                self.derived[i]["bias"] = (w["rel"][m.bias_by.buckets] - w["rel"][-1]).t().contiguous()
+            elif isinstance(m, LatentAttentionMixer) and self.device.type == "cuda" and self.dtype != torch.float32:
                 # cache row -> [keys | values] of all heads; an identity block hands the rotated part to every head's key
                 H, hp = m.heads, m.head_pitch
                 e = torch.zeros(2, H, hp, m.cols, dtype=self.dtype, device=self.device)

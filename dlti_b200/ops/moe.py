@@ -10,8 +10,8 @@ import torch
 
 from ..models.stack import MoeMlp, mlp_sections, round8
 from . import _lib
-from .gemm import gemm_skinny_acc, gemm_swiglu
-from .stack import _F, _I, _L, _V, _p, act, linear
+from .gemm import gemm_relu2, gemm_skinny_acc, gemm_swiglu
+from .stack import _F, _I, _L, _V, _p, act, linear, relu2
 
 LIMIT_OFF = 0.0              # limit of a plain SwiGLU: silu(g) * u without clipping
 
@@ -19,16 +19,20 @@ LIMIT_OFF = 0.0              # limit of a plain SwiGLU: silu(g) * u without clip
 @dataclass
 class ExpertSum:
     """A feed-forward's output that is still to be added up: sum over k of weights[t, k] * rows[t * top + k], plus shared (None:
-    nothing). counts: the router's pair counters, which the consumer leaves zero."""
+    nothing) times share[t] (None: one). counts: the router's pair counters, which the consumer leaves zero."""
     rows: torch.Tensor
     weights: torch.Tensor
     shared: torch.Tensor | None
     counts: torch.Tensor | None = None
+    share: torch.Tensor | None = None
 
     def value(self, d):
         T, top = self.weights.shape
         y = (self.rows[:, :d].float().view(T, top, d) * self.weights[:, :, None]).sum(1)
-        return y if self.shared is None else y + self.shared[:, :d].float()
+        if self.shared is None:
+            return y
+        s = self.shared[:, :d].float()
+        return y + (s if self.share is None else s * self.share[:, None])
 
 
 def _gated(g, u, limit):
@@ -67,9 +71,13 @@ def _counts(device, n: int) -> torch.Tensor:
     return _counters[key]
 
 
-def _route(p, logits, col: int, correction, e: MoeMlp | None, act_of=None, acc=False, cap: int = 0):
-    """One launch: routing of the fp32 logits [T, >= col + experts] at column col, and / or the activation act_of = (gate column,
-    up column, ff, limit, destination) of the projection rows p. acc: both read the decode GEMM's accumulator and leave it zero."""
+_ACT = {"swiglu": 1, "relu2": 2}       # activations of the grouped GEMM (0: none)
+
+
+def _route(p, logits, col: int, correction, e: MoeMlp | None, act_of=None, acc=False, share=None):
+    """One launch: routing of the fp32 logits [T, >= col + experts] at column col, the sigmoid of one more column (share = (column,
+    destination [T])), and / or the activation act_of = (gate column (-1: square of relu of the other), up column, ff, limit,
+    destination) of the projection rows p. acc: both read the decode GEMM's accumulator and leave it zero."""
     T = (p if p is not None else logits).shape[0]
     dev = (p if p is not None else logits).device
     wgt = lists = counts = None
@@ -77,17 +85,22 @@ def _route(p, logits, col: int, correction, e: MoeMlp | None, act_of=None, acc=F
         wgt = torch.empty((T, e.top), dtype=torch.float32, device=dev)
         lists = torch.empty((e.experts, T), dtype=torch.int32, device=dev)
         counts = _counts(dev, e.experts)
+    sg, sigma = share or (-1, None)
     og, ou, ff, limit, h = act_of or (0, 0, 0, 0.0, None)
-    f = _lib.fn("dlti_moe_route", [_V, _L, _I, _V, _I, _I, _I, _I, _F, _V, _V, _V, _V, _L, _I, _I, _I, _F, _V, _L, _L, _I, _I, _V])
+    f = _lib.fn("dlti_moe_route", [_V, _L, _I, _V, _I, _I, _I, _I, _F, _I, _V, _V, _V, _I, _V, _V, _L, _I, _I, _I, _F, _V, _L, _L, _I, _I, _V])
     _lib.check(f(_p(logits), 0 if logits is None else logits.stride(0), col, _p(correction), e.experts if e else 0, e.top if e else 0,
-                 e.groups if e else 1, e.keep if e else 1, e.scale if e else 1.0, _p(wgt), _p(lists), _p(counts), _p(p) if h is not None else None,
-                 p.stride(0) if p is not None else 0, og, ou, ff, float(limit), _p(h), 0 if h is None else h.stride(0), T, int(acc),
-                 _lib.dtype_code(h.dtype) if h is not None else _lib.DT_BF16, _lib.stream_ptr()), "moe_route")
+                 e.groups if e else 1, e.keep if e else 1, e.scale if e else 1.0, int(e is not None and e.score == "softmax"), _p(wgt), _p(lists),
+                 _p(counts), sg, _p(sigma), _p(p) if h is not None else None, p.stride(0) if p is not None else 0, og, ou, ff, float(limit), _p(h),
+                 0 if h is None else h.stride(0), T, int(acc), _lib.dtype_code(h.dtype) if h is not None else _lib.DT_BF16, _lib.stream_ptr()),
+               "moe_route")
     return wgt, lists, counts
 
 
 def route_ref(z, correction, e: MoeMlp):
     """Router logits [T, experts] -> (chosen experts [T, top], weights [T, top])."""
+    if e.score == "softmax":
+        c, idx = (z + correction).topk(e.top, -1)
+        return idx, torch.softmax(c, -1) * e.scale
     s = torch.sigmoid(z)
     c = s + correction
     T, n = z.shape[0], e.experts // e.groups
@@ -100,14 +113,14 @@ def route_ref(z, correction, e: MoeMlp):
     return idx, w / (w.sum(-1, keepdim=True) + 1e-20) * e.scale
 
 
-def grouped_gemm(x, w, lists, counts, out, *, rows: int, pairs_per_row: int, up: bool = False, limit: float = 0.0):
-    """Products of the pairs of every expert's list with its weights w [E, >= rows, K]. up: rows x[pair // pairs_per_row] times the
-    gate and up rows 2 r and 2 r + 1 of w; the clipped activations go to out one list after the other. Otherwise: rows of x in that
-    order; results go to out[pair]."""
+def grouped_gemm(x, w, lists, counts, out, *, rows: int, pairs_per_row: int, up: bool = False, limit: float = 0.0, act: str = "swiglu"):
+    """Products of the pairs of every expert's list with its weights w [E, >= rows, K]. up: rows x[pair // pairs_per_row]; the
+    activations go to out one list after the other ("swiglu", clipped: rows 2 r and 2 r + 1 of w are gate and up of output r; "relu2":
+    row r is). Otherwise: rows of x in that order; results go to out[pair]."""
     E, K, T = w.shape[0], w.shape[2], lists.shape[1]
     f = _lib.fn("dlti_moe_gemm", [_V, _L, _L, _I, _V, _L, _I, _I, _V, _V, _I, _I, _I, _I, _F, _V, _L, _I, _I, _V])
     _lib.check(f(_p(x), x.stride(0), x.shape[0], pairs_per_row, _p(w), w.stride(1), w.stride(0) // w.stride(1), E, _p(lists), _p(counts), T,
-                 rows, int(up), K, float(limit), _p(out), out.stride(0), out.shape[0], _lib.dtype_code(x.dtype), _lib.stream_ptr()), "moe_gemm")
+                 rows, _ACT[act] if up else 0, K, float(limit), _p(out), out.stride(0), out.shape[0], _lib.dtype_code(x.dtype), _lib.stream_ptr()), "moe_gemm")
     return out
 
 
@@ -115,7 +128,8 @@ def moe(h, e: MoeMlp, lw, dtype, mm, acc=False) -> ExpertSum:
     """Mixture of experts of the rows h; mm: the GEMM for the shared expert's output (its accumulator with acc)."""
     T, d = h.shape
     sec = mlp_sections(e)
-    og, ou = (sec["gate"], sec["up"]) if e.shared_ff else (0, 0)
+    og, ou = (sec["gate"] if e.gated else -1, sec["up"]) if e.shared_ff else (0, 0)
+    sg = sec["sg"] if e.shared_gate else -1
     if not _lib.use_native(h):
         p = linear(h, lw["w_up"], out_dtype=torch.float32)
         idx, wgt = route_ref(p[:, sec["router"]:sec["router"] + e.experts], lw["correction"], e)
@@ -124,21 +138,33 @@ def moe(h, e: MoeMlp, lw, dtype, mm, acc=False) -> ExpertSum:
             pair = (idx.flatten() == j).nonzero()[:, 0]
             if len(pair):
                 gu = h[pair // e.top].float() @ lw["e_up"][j].float().t()
-                a = _gated(gu[:, 0:2 * e.ff:2], gu[:, 1:2 * e.ff:2], e.limit).to(dtype)
+                a = (_gated(gu[:, 0:2 * e.ff:2], gu[:, 1:2 * e.ff:2], e.limit) if e.gated else torch.relu(gu[:, :e.ff]).square()).to(dtype)
                 rows[pair] = a.float() @ lw["e_down"][j, :d].float().t()
-        shared = mm(gated_act(p, og, ou, e.shared_ff, e.shared_limit, dtype), lw["w_down"]) if e.shared_ff else None
-        return ExpertSum(rows.to(dtype), wgt, shared)
-    hs = act(T, e.shared_ff, dtype, h.device) if e.shared_ff else None
-    act_of = (og, ou, e.shared_ff, e.shared_limit, hs) if e.shared_ff else None
+        shared = None
+        if e.shared_ff:
+            shared = mm(gated_act(p, og, ou, e.shared_ff, e.shared_limit, dtype) if e.gated else relu2(p[:, ou:], e.shared_ff, dtype), lw["w_down"])
+        return ExpertSum(rows.to(dtype), wgt, shared, share=torch.sigmoid(p[:, sg]) if sg >= 0 else None)
+    hs, act_of, share = None, None, None
+    if e.shared_gate:
+        share = torch.empty(T, dtype=torch.float32, device=h.device)
     if acc:
         p = gemm_skinny_acc(h, lw["w_up"])
-        wgt, lists, counts = _route(p, p, sec["router"], lw["correction"], e, act_of, acc=True)
+        if e.shared_ff:
+            hs = act(T, e.shared_ff, dtype, h.device)
+            act_of = (og, ou, e.shared_ff, e.shared_limit, hs)
+        wgt, lists, counts = _route(p, p, sec["router"], lw["correction"], e, act_of, acc=True, share=(sg, share))
     else:
-        z = linear(h, lw["w_up"][sec["router"]:], out_dtype=torch.float32)
-        p = linear(h, lw["w_up"][:sec["router"]]) if e.shared_ff else None
-        wgt, lists, counts = _route(p, z, 0, lw["correction"], e, act_of)
+        r0 = sec["router"]
+        z = linear(h, lw["w_up"][r0:], out_dtype=torch.float32)
+        p = None
+        if e.shared_ff and not e.gated:
+            hs = gemm_relu2(h, lw["w_up"][:r0], e.shared_ff)               # activation in the GEMM for large steps
+        if e.shared_ff and hs is None:
+            p, hs = linear(h, lw["w_up"][:r0]), act(T, e.shared_ff, dtype, h.device)
+            act_of = (og, ou, e.shared_ff, e.shared_limit, hs)
+        wgt, lists, counts = _route(p, z, 0, lw["correction"], e, act_of, share=(sg - r0 if sg >= 0 else -1, share))
     a = act(T * e.top, e.ff, dtype, h.device)
-    grouped_gemm(h, lw["e_up"], lists, counts, a, rows=e.ff, pairs_per_row=e.top, up=True, limit=e.limit)
+    grouped_gemm(h, lw["e_up"], lists, counts, a, rows=e.ff, pairs_per_row=e.top, up=True, limit=e.limit, act=e.act)
     rows = act(T * e.top, d, dtype, h.device)
     grouped_gemm(a, lw["e_down"], lists, counts, rows, rows=d, pairs_per_row=1)
-    return ExpertSum(rows, wgt, mm(hs, lw["w_down"]) if e.shared_ff else None, counts)
+    return ExpertSum(rows, wgt, mm(hs, lw["w_down"]) if e.shared_ff else None, counts, share)

@@ -38,18 +38,28 @@ def linear(a: torch.Tensor, w: torch.Tensor, out_dtype=None) -> torch.Tensor:
     return gemm(a, w, out_dtype=out_dtype)
 
 
-def linear_f32(a: torch.Tensor, w: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
-    """linear times scale with an fp32 result (logits)."""
-    if _lib.use_native(a) and a.dtype != torch.float32 and a.shape[0] > 256:
-        return gemm(a, w, out_dtype=torch.float32, alpha=scale)
-    if not _lib.use_native(a) or a.dtype == torch.float32:
-        y = linear(a, w, out_dtype=torch.float32)
-        return y if scale == 1.0 else y.mul_(scale)
-    acc = gemm_skinny_acc(a, w)
-    out = torch.empty_like(acc)
-    f = _lib.fn("dlti_take_rows", [_V, _V, _F, _L, _I, _V])
-    _lib.check(f(_p(acc), _p(out), float(scale), acc.shape[0], acc.shape[1], _lib.stream_ptr()), "take_rows")
-    return out
+def linear_f32(a: torch.Tensor, w: torch.Tensor, scale: float = 1.0, cap: float = 0.0) -> torch.Tensor:
+    """linear times scale with an fp32 result (logits); cap > 0: cap * tanh(that / cap)."""
+    if not _lib.use_native(a):
+        y = linear(a, w, out_dtype=torch.float32) * scale
+        return cap * torch.tanh(y / cap) if cap else y
+    if a.dtype == torch.float32:
+        acc, alpha = linear(a, w), scale
+    elif a.shape[0] > 256:
+        acc, alpha = gemm(a, w, out_dtype=torch.float32, alpha=scale), 1.0
+    else:
+        acc = gemm_skinny_acc(a, w)
+        out = torch.empty_like(acc)
+        _take_rows(acc, out, scale, cap, True)
+        return out
+    if alpha != 1.0 or cap:
+        _take_rows(acc, acc, alpha, cap, False)
+    return acc
+
+
+def _take_rows(src, out, scale, cap, clear):
+    f = _lib.fn("dlti_take_rows", [_V, _V, _F, _F, _I, _L, _I, _V])
+    _lib.check(f(_p(src), _p(out), float(scale), float(cap), int(clear), src.shape[0], src.shape[1], _lib.stream_ptr()), "take_rows")
 
 
 # ---- rows --------------------------------------------------------------------------------------------------
@@ -249,6 +259,71 @@ def qk_norm_rope_cache(proj, sec, m, q_norm, k_norm, eps, rows: Rows, tabs, kc, 
     return q, gate
 
 
+_factors: dict = {}
+
+
+def temp_table(max_pos: int, temp, device):
+    """fp32 factors [max_pos] of the queries by position (models.stack.QueryTemp), from double precision."""
+    key = (max_pos, temp, str(device))
+    if key not in _factors:
+        p = torch.arange(max_pos, dtype=torch.int64)
+        _factors[key] = (1 + temp.coef * torch.log(((p + 1) // temp.every + 1).double())).float().to(device)
+    return _factors[key]
+
+
+def conv_qkv(proj, sec, m, lw, factors, eps, rows: Rows, state, kc, vc, dtype, packed: Pieces | None = None, acc=False):
+    """Merged projection rows -> convolved (m.conv; state [slots, taps - 1, columns before g] holds the inputs of earlier steps and is
+    renewed) queries and keys with per-head norms, queries times factors[position] (None: one), values; keys and values in the paged
+    cache at rows.slots. packed: as in qk_norm_rope_cache. acc (decode rows only): the projection is the decode GEMM's accumulator.
+    Returns (queries or packed rows, the projected output gates [T, H * vdim] before their sigmoid or None)."""
+    T, H, G, taps, dev = proj.shape[0], m.heads, m.kv_heads, m.conv, proj.device
+    _debug.check_range("conv_qkv", "slots", rows.slots, 0, kc.shape[0] * kc.shape[1], allow=-1)
+    qn, kn, w = lw.get("q_norm"), lw.get("k_norm"), lw.get("conv")
+    gate = proj[:, sec["g"]:sec["g"] + H * m.vdim] if m.out_gate else None
+    if not _lib.use_native(proj):
+        span = sec["v"] + round8(G * m.vdim)
+        x = proj[:, :span].float()
+        if taps:
+            y = torch.zeros(T, span)
+            for s in range(rows.nseq):
+                r0, n, start = rows.bounds(s)
+                slot = int(rows.state[s])
+                h = state[slot].float() if state is not None and start > 0 and slot >= 0 else torch.zeros(taps - 1, span)
+                u = torch.cat([h, x[r0:r0 + n]])
+                y[r0:r0 + n] = sum(w[k, :span] * u[k:k + n] for k in range(taps))
+                if slot >= 0 and state is not None:
+                    state[slot] = u[n:].to(dtype)
+            x = y
+        q, k, v = (x[:, sec[c]:sec[c] + n * d].reshape(T, n, d) for c, n, d in (("q", H, m.dim), ("k", G, m.dim), ("v", G, m.vdim)))
+        q, k = (t if g is None else _rms(t, eps) * g for t, g in ((q, qn), (k, kn)))
+        if factors is not None:
+            q = q * factors[rows.pos.long()][:, None, None]
+        ok = rows.slots >= 0
+        kc.view(-1, G, kc.shape[3])[rows.slots[ok], :, :m.dim] = k.to(dtype)[ok]
+        vc.view(-1, G, vc.shape[3])[rows.slots[ok], :, :m.vdim] = v.to(dtype)[ok]
+        return q.to(dtype).reshape(T, -1), gate
+    if acc and gate is not None:
+        gate = act(T, H * m.vdim, dtype, dev)
+    kp = vp = dst = None
+    if packed is not None:
+        hd, n = PACKED_HD, rows.nd + packed.rows
+        q = (torch.empty if m.dim == m.vdim == hd else torch.zeros)((n, (H + 2 * G) * hd), dtype=dtype, device=dev)
+        kp, vp, dst = q[:, H * hd:], q[:, (H + G) * hd:], packed.dst
+    else:
+        hd = round8(m.dim)
+        q = torch.empty((T, H * hd), dtype=dtype, device=dev)
+    f = _lib.fn("dlti_conv_qkv", [_V, _L, _I, _I, _I, _I, _V, _I, _I, _V, _I, _V, _V, _V, _V, _I, _I, _V, _V, _F, _V, _V, _V, _V, _V, _I, _I, _V,
+                                  _L, _I, _V, _V, _V, _V, _L, _L, _I, _I, _I, _I, _I, _I, _V])
+    _lib.check(f(_p(proj), proj.stride(0), sec["q"], sec["k"], sec["v"], sec["g"] if m.out_gate else -1, _p(w), taps, 0 if w is None else w.stride(0),
+                 _p(state), 0 if state is None else state.shape[2], _p(rows.state), _p(rows.seq), _p(rows.ctx), _p(rows.cu), rows.nd, rows.nseq,
+                 _p(qn), _p(kn), float(eps), _p(factors), _p(rows.pos), _p(rows.slots), _p(kc), _p(vc), kc.shape[3], vc.shape[3],
+                 _p(q), q.stride(0), hd, _p(kp), _p(vp), _p(dst), _p(gate) if acc else None, gate.stride(0) if acc and gate is not None else 0, T,
+                 H, G, m.dim, m.vdim, int(acc), _lib.dtype_code(dtype), _lib.stream_ptr()), "conv_qkv")
+    if packed is not None and packed.prefix:
+        prefix_rows(q[rows.nd:], m, packed, kc, vc)
+    return q, gate
+
+
 def prefix_rows(buf, m, packed: Pieces, kc, vc):
     """Cached keys and values in front of the portions of a step: packed prompt rows buf [rows, (H + 2 G) * 128]."""
     f = _lib.fn("dlti_prefix_rows", [_V, _L, _I, _V, _V, _V, _V, _I, _I, _I, _I, _L, _V])
@@ -299,7 +374,7 @@ def qkv_rows(proj, sec, m, lw, eps, rows: Rows, first, kc, vc, dtype, packed: Pi
     return q, own
 
 
-def paged_attention_ref(q, m, rows: Rows, kc, vc, gate, sink=None):
+def paged_attention_ref(q, m, rows: Rows, kc, vc, gate, sink=None, bias=None, out_gate=None):
     """Every row against the cached keys of its sequence that it may see."""
     T, H, G = q.shape[0], m.heads, m.kv_heads
     bs, hd = kc.shape[1], q.shape[1] // H
@@ -318,21 +393,34 @@ def paged_attention_ref(q, m, rows: Rows, kc, vc, gate, sink=None):
         x = torch.einsum("hd,jhd->hj", qq, k) * m.scale
         if m.softcap:
             x = m.softcap * torch.tanh(x / m.softcap)
+        if bias is not None:
+            far = p - j >= bias.shape[1]
+            x = x + bias[:, (p - j).clamp(max=bias.shape[1] - 1)].masked_fill(far, 0.0)
         if sink is not None:
             x = torch.cat([x, sink[:, None]], 1)
         out[t] = torch.einsum("hj,jhd->hd", torch.softmax(x, -1)[:, :len(j)], v)
     if gate is not None:
         out *= gate[:, :, None]
+    if out_gate is not None:
+        out *= torch.sigmoid(out_gate.float()).view(T, H, m.vdim)
     return out.reshape(T, -1).to(q.dtype)
 
 
-def attn_rows(q, m, rows: Rows, kc, vc, gate, out, sink=None):
+def _more(bias, out_gate):
+    """Score biases and output gates as the attention kernels take them."""
+    return (_p(bias), 0 if bias is None else bias.shape[1], _p(out_gate), 0 if out_gate is None else out_gate.stride(0))
+
+
+_MORE = [_V, _I, _V, _L]
+
+
+def attn_rows(q, m, rows: Rows, kc, vc, gate, out, sink=None, bias=None, out_gate=None):
     """fp32-arithmetic attention of the rows of q, one warp per (row, head)."""
     hd = q.shape[1] // m.heads
-    f = _lib.fn("dlti_attn_rows", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _V, _I, _I, _I, _I, _I, _I, _F, _F, _V, _V, _V, _L, _L, _I, _V])
+    f = _lib.fn("dlti_attn_rows", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _V, _I, _I, _I, _I, _I, _I, _F, _F, _V, _V, *_MORE, _V, _L, _L, _I, _V])
     _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], kc.shape[1],
                  _p(rows.ctx), _p(rows.seq), _p(rows.pos), m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.window, m.scale, m.softcap,
-                 _p(gate), _p(sink), _p(out), out.stride(0), q.shape[0], _lib.dtype_code(q.dtype), _lib.stream_ptr()), "attn_rows")
+                 _p(gate), _p(sink), *_more(bias, out_gate), _p(out), out.stride(0), q.shape[0], _lib.dtype_code(q.dtype), _lib.stream_ptr()), "attn_rows")
     return out
 
 
@@ -349,7 +437,7 @@ def _workspace(device, floats: int) -> torch.Tensor:
     return ws
 
 
-def attn_paged_decode(q, m, rows: Rows, kc, vc, gate, out, splits: int | None = None, sink=None):
+def attn_paged_decode(q, m, rows: Rows, kc, vc, gate, out, splits: int | None = None, sink=None, bias=None, out_gate=None):
     """Decode rows (bf16): row b of q against the visible keys of sequence b, split over CTAs."""
     B, hd, bs = q.shape[0], q.shape[1] // m.heads, kc.shape[1]
     if splits is None:
@@ -357,55 +445,63 @@ def attn_paged_decode(q, m, rows: Rows, kc, vc, gate, out, splits: int | None = 
         ctas = max(1, B) * m.kv_heads * -(-(m.heads // m.kv_heads) // 16)
         splits = max(1, min(32, 3 * 148 // ctas, -(-reach // 64)))     # one wave of three CTAs per SM
     ws = _workspace(q.device, B * m.heads * splits * (m.vdim + 2)) if splits > 1 else None
-    f = _lib.fn("dlti_attn_paged_decode", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _I, _I, _I, _I, _I, _I, _I, _F, _F, _V, _V, _I, _V, _V, _L, _V])
+    f = _lib.fn("dlti_attn_paged_decode", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _I, _I, _I, _I, _I, _I, _I, _F, _F, _V, _V, *_MORE, _I, _V, _V, _L, _V])
     _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], bs,
-                 _p(rows.ctx), B, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.window, m.scale, m.softcap, _p(gate), _p(sink), splits, _p(ws),
+                 _p(rows.ctx), B, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk, m.window, m.scale, m.softcap, _p(gate), _p(sink),
+                 *_more(bias, out_gate), splits, _p(ws),
                  _p(out), out.stride(0), _lib.stream_ptr()), "attn_paged_decode")
     return out
 
 
-def attn_paged_prefill(q, m, rows: Rows, kc, vc, gate, out, sink=None):
+def attn_paged_prefill(q, m, rows: Rows, kc, vc, gate, out, sink=None, bias=None, out_gate=None):
     """Prompt rows (bf16): q, gate and out cover all rows of the step."""
     hd = q.shape[1] // m.heads
     f = _lib.fn("dlti_attn_paged_prefill", [_V, _L, _I, _V, _V, _I, _I, _V, _I, _I, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _V, _V,
-                                            _V, _L, _V])
+                                            *_MORE, _V, _L, _V])
     _lib.check(f(_p(q), q.stride(0), hd, _p(kc), _p(vc), kc.shape[3], vc.shape[3], _p(rows.tables), rows.tables.shape[1], kc.shape[1],
                  _p(rows.ctx), _p(rows.cu), rows.nd, rows.nseq - rows.nd, rows.max_seqlen, m.heads, m.kv_heads, m.dim, m.vdim, m.chunk,
-                 m.window, m.scale, m.softcap, _p(gate), _p(sink), _p(out), out.stride(0), _lib.stream_ptr()), "attn_paged_prefill")
+                 m.window, m.scale, m.softcap, _p(gate), _p(sink), *_more(bias, out_gate), _p(out), out.stride(0), _lib.stream_ptr()),
+               "attn_paged_prefill")
     return out
 
 
-def packed_attention(qkv, m, rows: Rows, pieces: Pieces, kc, vc, gate, sink=None):
-    """Attention of a step from the packed rows of qk_norm_rope_cache or qkv_rows: decode rows through the pages, prompt rows through the
+def packed_attention(qkv, m, rows: Rows, pieces: Pieces, kc, vc, gate, sink=None, bias=None, out_gate=None):
+    """Attention of a step from the packed rows of qk_norm_rope_cache, qkv_rows or conv_qkv: decode rows through the pages, prompt rows through the
     varlen tcgen05 kernel. Needs heads of up to 128 dimensions, values in multiples of 8."""
     T, H, nd = rows.pos.numel(), m.heads, rows.nd
     out = act(T, H * m.vdim, qkv.dtype, qkv.device)
     if nd:
-        attn_paged_decode(qkv[:nd, :H * PACKED_HD], m, rows, kc, vc, gate, out, sink=sink)
-    attn_fwd_split(qkv[nd:], m, H, m.kv_heads, pieces, None if gate is None else gate[nd:], out[nd:], sink=sink)
+        attn_paged_decode(qkv[:nd, :H * PACKED_HD], m, rows, kc, vc, gate, out, sink=sink, bias=bias, out_gate=out_gate)
+    attn_fwd_split(qkv[nd:], m, H, m.kv_heads, pieces, None if gate is None else gate[nd:], out[nd:], sink=sink, bias=bias,
+                   out_gate=None if out_gate is None else out_gate[nd:])
     return out
 
 
-def attn_fwd_split(qkv, m, heads, kv_heads, pieces: Pieces, gate, out, sink=None):
+PACKED_BIAS = 4096           # distances with a bias of their own that the packed prompt kernel has room for
+
+
+def attn_fwd_split(qkv, m, heads, kv_heads, pieces: Pieces, gate, out, sink=None, bias=None, out_gate=None):
     """Causal attention of packed rows [q heads | k heads | v heads], each 128 columns, within every piece."""
-    f = _lib.fn("dlti_attn_fwd_split", [_V, _V, _L, _V, _V, _V, _V, _V, _I, _I, _L, _I, _I, _I, _I, _F, _F, _V])
+    f = _lib.fn("dlti_attn_fwd_split", [_V, _V, _L, _V, _V, _V, _V, _V, _I, _I, _L, _I, _I, _I, _I, _F, _F, *_MORE, _V])
     _lib.check(f(_p(qkv), _p(out), out.stride(0), _p(gate), _p(sink), _p(pieces.cu), _p(pieces.q0), _p(pieces.out0), pieces.cu.numel() - 1,
-                 pieces.longest, qkv.shape[0], heads, kv_heads, m.vdim, m.window, m.scale, m.softcap, _lib.stream_ptr()),
-               "attn_fwd_split")
+                 pieces.longest, qkv.shape[0], heads, kv_heads, m.vdim, m.window, m.scale, m.softcap, *_more(bias, out_gate),
+                 _lib.stream_ptr()), "attn_fwd_split")
 
 
-def paged_attention(q, m, rows: Rows, kc, vc, gate, sink=None):
-    """Attention of every row of a step over the paged cache -> [T, heads * vdim], head outputs times `gate` [T, H]."""
+def paged_attention(q, m, rows: Rows, kc, vc, gate, sink=None, bias=None, out_gate=None):
+    """Attention of every row of a step over the paged cache -> [T, heads * vdim], head outputs times `gate` [T, H]. bias [H, n]: added
+    to the scores at the distances below n; out_gate [T, heads * vdim]: outputs are multiplied by its sigmoid."""
+    more = dict(sink=sink, bias=bias, out_gate=out_gate)
     if not _lib.use_native(q):
-        return paged_attention_ref(q, m, rows, kc, vc, gate, sink)
+        return paged_attention_ref(q, m, rows, kc, vc, gate, **more)
     _debug.check_paged("paged_attention", rows.tables, rows.ctx, kc.shape[0], kc.shape[1])
     out = act(q.shape[0], m.heads * m.vdim, q.dtype, q.device)
     if q.dtype == torch.float32 or max(kc.shape[3], vc.shape[3]) > 256:
-        return attn_rows(q, m, rows, kc, vc, gate, out, sink=sink)
+        return attn_rows(q, m, rows, kc, vc, gate, out, **more)
     if rows.nd:
-        attn_paged_decode(q[:rows.nd], m, rows, kc, vc, gate, out, sink=sink)
+        attn_paged_decode(q[:rows.nd], m, rows, kc, vc, gate, out, **more)
     if rows.nseq > rows.nd:
-        attn_paged_prefill(q, m, rows, kc, vc, gate, out, sink=sink)
+        attn_paged_prefill(q, m, rows, kc, vc, gate, out, **more)
     return out
 
 

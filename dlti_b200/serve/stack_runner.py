@@ -11,12 +11,13 @@ import os
 import torch
 
 from ..models.stack import (AttentionMixer, DeltaMixer, LatentAttentionMixer, LightningMixer, Mamba2Mixer, MLstmMixer, MoeMlp, StackConfig,
-                            StackWeights, mixer_sections, round8)
+                            StackWeights, conv_span, mixer_sections, round8)
 from ..ops import _lib
 from ..ops import delta as D
 from ..ops import dyt as N
 from ..ops import latent as LA
 from ..ops import moe as M
+from ..ops import prenorm as P
 from ..ops import stack as K
 from ..ops import streams as H
 from ..ops.gemm import gemm_relu2, gemm_skinny_acc
@@ -107,14 +108,41 @@ class TanhNorms:
         return N.tanh_rows(self.x, idx, (w.final_norm_alpha, w.final_norm, w.final_norm_b), self.run.dtype)
 
 
+class PreNorms:
+    """One fp32 residual, RMS norms on the sublayer inputs (ops/prenorm.py): one kernel between two sublayers, which also adds up the
+    outputs of a mixture of experts, norms the output of a token input, and adds the embedding where a pass of a loop begins."""
+
+    def __init__(self, run: "StackRunner", ids, rows: K.Rows, first, acc: bool):
+        self.run, self.acc, self.again = run, acc, False
+        self.embed = (ids, run.w.embed, run.cfg.embed_scale)
+        self.x = torch.empty((ids.numel(), run.cfg.hidden_size), dtype=torch.float32, device=run.w.embed.device)
+        self.h = P.between_(self.x, None, first[0]["norm1"], run.cfg.norm_eps, run.dtype, embed=self.embed, fresh=True)
+
+    def step(self, y, done, then):
+        cfg = self.run.cfg
+        self.again = then is not None and then[1] == 1 and then[2] in cfg.restarts
+        side = then is not None and then[1] == 3                      # a token input reads the residual itself
+        return P.between_(self.x, y, None if then is None or side else then[0][f"norm{then[1]}"], cfg.norm_eps, self.run.dtype,
+                          mult=cfg.residual_mult, post=done[0]["norm3"] if done[1] == 3 else None, embed=self.embed if self.again else None,
+                          copy=side, acc=self.acc)
+
+    def residual(self):
+        ids, table, scale = self.embed
+        return self.x - table[ids].float() * scale if self.again else self.x.clone()
+
+    def final(self, idx):
+        cfg = self.run.cfg
+        return K.rms_rows(self.x, idx, self.run.w.final_norm, cfg.norm_eps, False, self.run.dtype)
+
+
 class StackRunner:
     per_sequence = True
 
     @staticmethod
     def cache_specs(cfg: StackConfig, weights: StackWeights):
-        """(key/value page specs, recurrent-state specs), one entry per layer. Head rows are padded to 16 bytes."""
+        """(key/value page specs, recurrent-state specs), one entry per run of a layer. Head rows are padded to 16 bytes."""
         kv, st = [], []
-        for l in cfg.layers:
+        for l in (cfg.layers[j] for j in cfg.runs):
             m = l.mixer
             if isinstance(m, AttentionMixer):
                 kv.append(KVSpec(m.kv_heads, round8(m.dim), round8(m.vdim), m.kv_from))
@@ -123,6 +151,8 @@ class StackRunner:
             state = {}
             if isinstance(m, Mamba2Mixer):
                 state = dict(heads=m.heads, rows=m.state, cols=m.vdim, conv_rows=m.conv - 1, conv_channels=m.conv_channels if m.conv > 1 else 0)
+            elif isinstance(m, AttentionMixer) and m.conv > 1:
+                state = dict(conv_rows=m.conv - 1, conv_channels=conv_span(m))
             elif isinstance(m, LightningMixer):
                 state = dict(heads=m.heads, rows=m.dim, cols=m.vdim)
             elif isinstance(m, DeltaMixer):
@@ -137,9 +167,14 @@ class StackRunner:
     def __init__(self, cfg: StackConfig, weights: StackWeights, kv: KVCache, states: StateCache | None, max_len: int):
         self.cfg, self.w, self.kv, self.states = cfg, weights, kv, states
         self.device, self.dtype = weights.device, weights.dtype
-        self.sections = [mixer_sections(l.mixer) for l in cfg.layers]
+        # one entry per run of a layer: caches and states belong to the run, weights to the layer
+        self.layers = [cfg.layers[j] for j in cfg.runs]
+        self.derived = [weights.derived[j] for j in cfg.runs]
+        self.sections = [mixer_sections(l.mixer) for l in self.layers]
         self.ropes = [K.rope_tables(max_len, l.mixer.rope.dims, l.mixer.rope.base, self.device)
-                      if getattr(l.mixer, "rope", None) is not None else None for l in cfg.layers]
+                      if getattr(l.mixer, "rope", None) is not None else None for l in self.layers]
+        self.temps = [K.temp_table(max_len, l.mixer.q_temp, self.device) if getattr(l.mixer, "q_temp", None) is not None else None
+                      for l in self.layers]
         if self.device.type == "cuda" and "DLTI_PDL" not in os.environ:
             # serving weights are static: the decode GEMMs may fetch weight tiles while the previous kernel drains
             _lib.gpu_lib().dlti_set_pdl(2)
@@ -147,8 +182,9 @@ class StackRunner:
         self.trace = None            # set to a list: receives the residual after every layer (debugging)
         self.mixers = {AttentionMixer: self._attention, LatentAttentionMixer: self._latent, Mamba2Mixer: self._mamba2,
                        LightningMixer: self._lightning, MLstmMixer: self._mlstm, DeltaMixer: self._delta}
-        # the sublayers in order: (layer weights, 1 mixer | 2 feed-forward, layer)
-        self.parts = [(lw, q, i) for i, (l, lw) in enumerate(zip(cfg.layers, weights.layers)) for q in ((1, 2) if l.mlp is not None else (1,))]
+        # the sublayers in order: (layer weights, 1 mixer | 2 feed-forward | 3 token input, run)
+        self.parts = [(weights.layers[j], q, i) for i, j in enumerate(cfg.runs)
+                      for q, have in ((1, True), (2, cfg.layers[j].mlp is not None), (3, cfg.token_side > 0)) if have]
 
     @torch.no_grad()
     def forward(self, input_ids, positions, slots, *, num_decode: int = 0, block_tables=None, ctx_lens=None, cu_seqlens=None,
@@ -162,22 +198,26 @@ class StackRunner:
         # decode-sized steps stream the weights through the stream-K GEMM; the next op consumes its fp32 accumulator
         self.acc = _FUSE_ACC and w.embed.is_cuda and self.dtype == torch.bfloat16 and ids.numel() <= 256
         mm = gemm_skinny_acc if self.acc else K.linear
-        res = (HyperStreams if cfg.streams else TanhNorms if cfg.tanh_norms else OutputNorms)(self, ids, rows, self.parts[0], self.acc)
+        kind = HyperStreams if cfg.streams else TanhNorms if cfg.tanh_norms else PreNorms if cfg.pre_norm else OutputNorms
+        res = kind(self, ids, rows, self.parts[0], self.acc)
         h = res.h
         self.first_v = None          # values of the first layer that mixes values
         for part, then in zip(self.parts, self.parts[1:] + [None]):
             lw, q, i = part
-            m = cfg.layers[i].mixer
+            m = self.layers[i].mixer
             if q == 1:
                 y = mm(self.mixers[type(m)](i, m, lw, h, rows, segs), lw["w_out"])
+            elif q == 2:
+                y = self._mlp(self.layers[i].mlp, lw, h, mm)
             else:
-                y = self._mlp(cfg.layers[i].mlp, lw, h, mm)
+                n = cfg.token_side
+                y = mm(P.token_gate(mm(h, lw["side_gate"]), ids, w.side_embed, cfg.runs[i] * n, n, self.dtype, acc=self.acc), lw["side_proj"])
             h = res.step(y, part, then)
             if self.trace is not None and (then is None or then[2] != i):
                 self.trace.append(res.residual())
         if last_idx is not None and last_idx.numel() == 0:
             return torch.empty((0, cfg.vocab_size), dtype=torch.float32, device=self.device)
-        return K.linear_f32(res.final(last_idx), w.lm_head, cfg.logit_scale)[:, :cfg.vocab_size]
+        return K.linear_f32(res.final(last_idx), w.lm_head, cfg.logit_scale, cfg.logit_softcap)[:, :cfg.vocab_size]
 
     def _mlp(self, mlp, lw, h, mm):
         if isinstance(mlp, MoeMlp):
@@ -198,19 +238,29 @@ class StackRunner:
         if (xa.is_cuda and self.dtype == torch.bfloat16 and 32 < max(m.dim, m.vdim) <= K.PACKED_HD and m.vdim % 8 == 0
                 and self.pack_prompts):
             packed = (segs or {}).get(m.reach)
-        proj = gemm_skinny_acc(xa, lw["w_in"]) if self.acc else K.linear(xa, lw["w_in"])
-        sink = lw.get("sink")
-        if m.whole_rows:
+        # the convolutions of prompt rows read their neighbours' inputs: conv_qkv takes the accumulators of decode steps only
+        acc = self.acc and (not m.conv_heads or rows.nd == xa.shape[0])
+        proj = gemm_skinny_acc(xa, lw["w_in"]) if acc else K.linear(xa, lw["w_in"])
+        sink, bias, out_gate = lw.get("sink"), self.derived[i].get("bias"), None
+        if bias is not None and bias.shape[1] > K.PACKED_BIAS:
+            packed = None
+        if m.conv_heads:
+            state = self.states.conv[i] if m.conv > 1 else None
+            q, out_gate = K.conv_qkv(proj, self.sections[i], m, lw, self.temps[i], self.cfg.norm_eps, rows, state, self.kv.k[i], self.kv.v[i],
+                                     self.dtype, packed=packed, acc=acc)
+            gate = None
+        elif m.whole_rows:
             q, own = K.qkv_rows(proj, self.sections[i], m, lw, self.cfg.norm_eps, rows, self.first_v, self.kv.k[i], self.kv.v[i], self.dtype,
-                                packed=packed, acc=self.acc)
+                                packed=packed, acc=acc)
             self.first_v = own if own is not None else self.first_v
             gate = None
         else:
             q, gate = K.qk_norm_rope_cache(proj, self.sections[i], m, lw.get("q_norm"), lw.get("k_norm"), self.cfg.norm_eps, rows,
-                                           self.ropes[i], self.kv.k[i], self.kv.v[i], self.dtype, packed=packed, acc=self.acc)
+                                           self.ropes[i], self.kv.k[i], self.kv.v[i], self.dtype, packed=packed, acc=acc)
+        more = dict(sink=sink, bias=bias, out_gate=out_gate)
         if packed is not None:
-            return K.packed_attention(q, m, rows, packed, self.kv.k[i], self.kv.v[i], gate, sink=sink)
-        return K.paged_attention(q, m, rows, self.kv.k[i], self.kv.v[i], gate, sink=sink)
+            return K.packed_attention(q, m, rows, packed, self.kv.k[i], self.kv.v[i], gate, **more)
+        return K.paged_attention(q, m, rows, self.kv.k[i], self.kv.v[i], gate, **more)
 
     def _mamba2(self, i, m: Mamba2Mixer, lw, xa, rows: K.Rows, segs):
         s, st = self.sections[i], self.states
@@ -234,7 +284,7 @@ class StackRunner:
 
     def _latent(self, i, m: LatentAttentionMixer, lw, xa, rows: K.Rows, segs):
         proj = gemm_skinny_acc(xa, lw["w_in"]) if self.acc else K.linear(xa, lw["w_in"])
-        return LA.latent_attention(proj, self.sections[i], m, lw, self.w.derived[i].get("w_expand"), self.cfg.norm_eps, rows, self.ropes[i],
+        return LA.latent_attention(proj, self.sections[i], m, lw, self.derived[i].get("w_expand"), self.cfg.norm_eps, rows, self.ropes[i],
                                    self.kv.k[i], self.dtype, (segs or {}).get(m.reach) if self.pack_prompts else None, acc=self.acc)
 
     def _mlstm(self, i, m: MLstmMixer, lw, xa, rows: K.Rows, segs):
@@ -246,7 +296,7 @@ class StackRunner:
         return K.gated_norm(y, proj[:, s["g"]:s["g"] + vv], lw["norm"], self.cfg.norm_eps, m.heads, gate_first=False)
 
     def _delta(self, i, m: DeltaMixer, lw, xa, rows: K.Rows, segs):
-        s, st, der = self.sections[i], self.states, self.w.derived[i]
+        s, st, der = self.sections[i], self.states, self.derived[i]
         qk, vv = m.kv_heads * m.dim, m.heads * m.vdim
         if self.acc and rows.nd == xa.shape[0]:                   # the convolution of prompt rows reads its neighbours' inputs
             proj = gemm_skinny_acc(xa, lw["w_in"])
