@@ -68,6 +68,10 @@ struct AttnParams {
   const float* sink;     // optional [H]: one more term exp(sink) in the softmax denominator, without a value
   int vdim;              // value columns of a head that are written, head h at column h * vdim of O (0: 128)
   int window;            // > 0: a row sees itself and the window - 1 rows before it
+  const float* bias;     // BIAS form: [H, span] added to the scores at the distances 0 ... span - 1
+  int span;
+  const void* ogate;     // optional [output rows, H * vdim], row pitch og_ld: outputs are multiplied by its sigmoid
+  long long og_ld;
   SoftCap soft;          // CAP form: scores become cap tanh(score / cap)
 };
 
@@ -818,8 +822,10 @@ __device__ __forceinline__ void mbar_wait_b(uint32_t bar, uint32_t parity) {
 // SPLIT: the softmax weights are written as two 16-bit terms (hi over columns 0-63 of the S buffer, what its rounding
 // left over columns 64-127) and both enter the PV product, so the weights keep fp32-like precision (16 mantissa bits)
 // for 1.5x the MMA work. With a window a tile starts at the key block that its first row's window reaches into.
-// CAP: soft cap on the scores (see capped_log2 in mma_sync.cuh).
-template <typename T, bool SPLIT, bool CAP = false>
+// CAP: soft cap on the scores (see capped_log2 in mma_sync.cuh). BIAS: the head's biases by distance lie in shared memory, in log2
+// units, between zeros for the distances that a block beside the biased ones covers; blocks farther away need none.
+constexpr int F2_BIAS_BEFORE = 127, F2_BIAS_PAD = 127 + 255;
+template <typename T, bool SPLIT, bool CAP = false, bool BIAS = false>
 __global__ void __launch_bounds__(F2_THREADS, 1)
 attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) {
   const int b = blockIdx.z, h = blockIdx.y;
@@ -867,6 +873,13 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
   if (warp == 9) {
     tmem_alloc(tmem_slot, 512);
     tmem_relinquish();
+  }
+  float* s_bias = reinterpret_cast<float*>(smem_raw + (bars + 256 - smem_u32(smem_raw)));
+  if constexpr (BIAS) {
+    for (int i = threadIdx.x; i < p.span + F2_BIAS_PAD; i += F2_THREADS) {
+      const int n = i - F2_BIAS_BEFORE;
+      s_bias[i] = n >= 0 && n < p.span ? p.bias[(long long)h * p.span + n] * LOG2E : 0.f;
+    }
   }
   tc_fence_before();
   __syncthreads();
@@ -1005,6 +1018,15 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
             top = cap_any(p.soft, top);
           }
         }
+        float f = sl2;                            // factor that takes what v holds to log2 units
+        if constexpr (BIAS) {
+          if ((qbX - j) * 128 - 127 < p.span) {
+            const float* tab = s_bias + (qbX - j) * 128 + r + F2_BIAS_BEFORE;
+#pragma unroll
+            for (int i = 0; i < 128; ++i) v[i] = __float_as_uint(fmaf(__uint_as_float(v[i]), sl2, tab[-i]));
+            f = 1.f;
+          }
+        }
         float mx = -INFINITY;
         if (SPLIT && p.window > 0 && (qbX - j) * 128 + 127 >= p.window) {     // some row's window starts in this block
           const int lo = (qbX - j) * 128 + r - p.window + 1, hi = diag ? r : 127;
@@ -1025,7 +1047,7 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
 #pragma unroll
           for (int i = 0; i < 128; ++i) mx = fmaxf(mx, __uint_as_float(v[i]));
         }
-        mx *= sl2;
+        mx *= f;
         if (it == 0) {
           m_ref = fmaxf(mx, -1e30f);              // finite also where the window leaves a row nothing in its tile's first block
         } else {
@@ -1055,8 +1077,8 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
           uint32_t pk[16], pl[16];
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
-            const float p0 = ex2_approx(fmaf(__uint_as_float(v[32 * c + 2 * i]), sl2, neg_m));
-            const float p1 = ex2_approx(fmaf(__uint_as_float(v[32 * c + 2 * i + 1]), sl2, neg_m));
+            const float p0 = ex2_approx(fmaf(__uint_as_float(v[32 * c + 2 * i]), f, neg_m));
+            const float p1 = ex2_approx(fmaf(__uint_as_float(v[32 * c + 2 * i + 1]), f, neg_m));
             l += p0 + p1;
             pk[i] = Cvt<T>::pack2(p0, p1);
             if constexpr (SPLIT) {
@@ -1093,6 +1115,16 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
             if (SPLIT && c * 32 + 8 * k >= vdim) break;
             int4 ov;
             uint32_t* ou = reinterpret_cast<uint32_t*>(&ov);
+            if (SPLIT && p.ogate) {
+              const int4 gv = *reinterpret_cast<const int4*>(reinterpret_cast<const T*>(p.ogate) + orow_i * p.og_ld + h * vdim + c * 32 + 8 * k);
+              const uint32_t gu[4] = {(uint32_t)gv.x, (uint32_t)gv.y, (uint32_t)gv.z, (uint32_t)gv.w};
+#pragma unroll
+              for (int q = 0; q < 4; ++q) {
+                const float2 z = Cvt<T>::unpack2(gu[q]);
+                o[8 * k + 2 * q] = __float_as_uint(__uint_as_float(o[8 * k + 2 * q]) * __fdividef(1.f, 1.f + __expf(-z.x)));
+                o[8 * k + 2 * q + 1] = __float_as_uint(__uint_as_float(o[8 * k + 2 * q + 1]) * __fdividef(1.f, 1.f + __expf(-z.y)));
+              }
+            }
 #pragma unroll
             for (int q = 0; q < 4; ++q)
               ou[q] = Cvt<T>::pack2(__uint_as_float(o[8 * k + 2 * q]) * inv, __uint_as_float(o[8 * k + 2 * q + 1]) * inv);
@@ -1111,6 +1143,7 @@ attn_fwd2_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tm128) 
   }
 }
 
+constexpr int F2_BIAS_MAX = 4096, F2_BIAS_SMEM = F2_SMEM + 4 * (F2_BIAS_MAX + F2_BIAS_PAD);
 constexpr int FWD_SMEM = 6 * 32768 + 256 + 1024;
 constexpr int BWD_SMEM_Q = 65536 + 2 * BWD_NYS_Q * 16384 + 1024 + 256 + 1024;
 constexpr int BWD_SMEM_KV = 65536 + 2 * BWD_NYS_KV * 16384 + BWD_STAT_BYTES + 256 + 1024;
@@ -1175,17 +1208,20 @@ DLTI_API int dlti_attn_fwd(const void* qkv, void* out, float* lse, const int* cu
 
 // dqkv [T, (H+2KV)*128] receives dq | dk | dv. D_scratch: [H, T] fp32 workspace.
 // Inference form with split softmax weights (see attn_fwd2_kernel), bf16: heads padded to 128 columns in qkv, vdim (a
-// multiple of 8) of them written; optional gate [output rows, H]; window / cap: see AttnParams (0: none); output row pitch ldo (a multiple of 8); optional
+// multiple of 8) of them written; optional gate [output rows, H], biases by distance (span of them a head) and gates per output element (ogate); window / cap: see AttnParams (0: none); output row pitch ldo (a multiple of 8); optional
 // seq_q0 / seq_out0 (see AttnParams) for portions whose earlier keys and values lie in front of their rows.
 DLTI_API int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const float* sink, const int* cu_seqlens, const int* seq_q0,
                                  const int* seq_out0, int batch, int max_seqlen, long long T_total, int H, int KV, int vdim, int window,
-                                 float scale, float cap, cudaStream_t st) {
+                                 float scale, float cap, const float* bias, int span, const void* ogate, long long og_ld, cudaStream_t st) {
+  if (bias && (cap > 0.f || span < 1 || span > F2_BIAS_MAX)) return DLTI_ERR_BAD_ARG;
+  if (ogate && (og_ld % 8 || (reinterpret_cast<uintptr_t>(ogate) & 15))) return DLTI_ERR_BAD_ARG;
   if (H % KV || window < 0 || cap < 0.f || ldo % 8 || vdim % 8 || vdim < 8 || vdim > HD || (seq_q0 == nullptr) != (seq_out0 == nullptr) || (reinterpret_cast<uintptr_t>(out) & 15)) return DLTI_ERR_BAD_ARG;
   if (batch <= 0 || T_total <= 0) return 0;
   AttnParams p{};
   p.cu_seqlens = cu_seqlens; p.H = H; p.KV = KV; p.W = (H + 2 * KV) * HD;
   p.O = out; p.ldo = ldo; p.T_total = T_total; p.scale = scale; p.dtype = DLTI_BF16; p.gate = gate; p.sink = sink;
   p.seq_q0 = seq_q0; p.seq_out0 = seq_out0; p.vdim = vdim; p.window = window;
+  p.bias = bias; p.span = span; p.ogate = ogate; p.og_ld = og_ld;
   if (cap > 0.f) p.soft = soft_cap(scale, cap);
   CUtensorMap tm;
   const int rc = make_map(&tm, qkv, T_total, p.W, 128);
@@ -1196,9 +1232,11 @@ DLTI_API int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, cons
   if (!cfg[dev & 63]) {
     DLTI_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd2_kernel<__nv_bfloat16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, F2_SMEM));
     DLTI_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd2_kernel<__nv_bfloat16, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, F2_SMEM));
+    DLTI_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd2_kernel<__nv_bfloat16, true, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, F2_BIAS_SMEM));
     cfg[dev & 63] = true;
   }
-  (cap > 0.f ? attn_fwd2_kernel<__nv_bfloat16, true, true> : attn_fwd2_kernel<__nv_bfloat16, true>)<<<dim3(((max_seqlen + 127) / 128 + 1) / 2, H, batch), F2_THREADS, F2_SMEM, st>>>(p, tm);
+  auto kern = bias ? attn_fwd2_kernel<__nv_bfloat16, true, false, true> : cap > 0.f ? attn_fwd2_kernel<__nv_bfloat16, true, true> : attn_fwd2_kernel<__nv_bfloat16, true>;
+  kern<<<dim3(((max_seqlen + 127) / 128 + 1) / 2, H, batch), F2_THREADS, F2_SMEM + (bias ? 4 * (span + F2_BIAS_PAD) : 0), st>>>(p, tm);
   dlti_count_launch();
   return (int)cudaGetLastError();
 }

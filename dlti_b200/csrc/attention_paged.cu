@@ -1,6 +1,6 @@
 // Attention over the paged cache for the layer-stack models: any head size, grouped key/value heads, causal, chunked
 // (position i sees keys of its own chunk of `chunk` positions only) or windowed (itself and the window - 1 positions before
-// it), optional soft cap on the scores, per-head sink and per-head output gate.
+// it), optional soft cap on the scores, bias by distance, per-head sink, gates on head outputs or on every output element.
 //
 //   attn_prefill_kernel  portions of prompts, bf16: a CTA owns 128 (token, head of a group) rows and streams key / value
 //                        tiles of 64 from the pages through shared memory into mma.sync
@@ -10,8 +10,8 @@
 //
 // Scores, softmax weights and sums are fp32. The weights enter the P*V product as two bf16 terms (hi + lo, 16 mantissa
 // bits), so the product is that of the fp32 weights with the bf16 values.
-#include "common.cuh"
 #include "mma_sync.cuh"
+#include "rows.cuh"
 
 namespace {
 
@@ -26,7 +26,16 @@ struct PagedParams {
   void* out; long long o_ld;                       // head h at column h * vdim
   long long rows;
   const float* sink;                               // [H] or null: one more term exp(sink) in the softmax denominator, without a value
+  const float* bias; int span;                     // [H, span] or null: added to the scores at the distances 0 ... span - 1
+  const void* ogate; long long og_ld;              // [rows, H * vdim] or null: outputs times sigmoid of it
 };
+// factor of output element c of head h
+template <typename T>
+__device__ __forceinline__ float gate_at(const PagedParams& p, long long row, int h, int c) {
+  if (!p.ogate) return 1.f;
+  const float z = Cvt<T>::to_f(reinterpret_cast<const T*>(p.ogate)[row * p.og_ld + (long long)h * p.vdim + c]);
+  return sizeof(T) == 4 ? sigmoid_f(z) : fast_sigmoid(z);
+}
 
 // softmax denominator of head h with its sink: l is a sum of 2^(score - m), m in log2 (natural: of e^(score - m))
 __device__ __forceinline__ float with_sink(const PagedParams& p, int h, float m, float l, bool natural = false) {
@@ -76,6 +85,7 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const PagedParams p) {
       }
       s = a * p.scale;
       if (p.cap > 0.f) s = p.cap * tanhf(s / p.cap);
+      if (p.bias && ps - j < p.span) s += p.bias[(long long)h * p.span + ps - j];
     }
     const float nm = fmaxf(m, warp_max(s));
     const float alpha = expf(m - nm);
@@ -103,7 +113,7 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const PagedParams p) {
 #pragma unroll
   for (int i = 0; i < ROWS_MAXV; ++i) {
     const int c = lane + 32 * i;
-    if (c < p.vdim) orow[c] = Cvt<T>::from_f(o[i] * f);
+    if (c < p.vdim) orow[c] = Cvt<T>::from_f(o[i] * f * gate_at<T>(p, t, h, c));
   }
 }
 
@@ -299,12 +309,14 @@ __global__ void __launch_bounds__(256) attn_prefill_kernel(const PagedParams p) 
 #pragma unroll
     for (int i = 0; i < KT / 16; ++i) scores16<DK>(s[2 * i], s[2 * i + 1], qf, kb, i * 16);
     float mx[2] = {-INFINITY, -INFINITY};
+    const bool near = p.bias && start + (int)(wr0 / rep) - (j0 + KT - 1) < p.span;
 #pragma unroll
     for (int i = 0; i < KT / 8; ++i)
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         const int j = j0 + i * 8 + (lane & 3) * 2 + (x & 1), y = x >> 1;
         s[i][x] = (j <= pos[y] && j >= jlo[y]) ? score_log2(p, s[i][x], sl2) : -INFINITY;
+        if (near && j <= pos[y] && pos[y] - j < p.span) s[i][x] += LOG2E_F * p.bias[(long long)head[y] * p.span + pos[y] - j];
         mx[y] = fmaxf(mx[y], s[i][x]);
       }
     float base[2];
@@ -345,6 +357,10 @@ __global__ void __launch_bounds__(256) attn_prefill_kernel(const PagedParams p) 
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i) {
       const int c = i * 8 + (lane & 3) * 2;
+      if (p.ogate) {
+        if (c < p.vdim) o[i][2 * y] *= gate_at<bf16>(p, row[y], head[y], c);
+        if (c + 1 < p.vdim) o[i][2 * y + 1] *= gate_at<bf16>(p, row[y], head[y], c + 1);
+      }
       if (c + 1 < p.vdim && (p.vdim & 1) == 0) {
         *reinterpret_cast<__nv_bfloat162*>(orow + c) = __floats2bfloat162_rn(o[i][2 * y] * f, o[i][2 * y + 1] * f);
       } else {
@@ -406,14 +422,16 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const PagedParams p, i
       if (j0 + warp * 16 >= jend) continue;
       const uint32_t kb = sbase + (it & 1) * L::BYTES, vb = kb + L::K_BYTES;
       float s[2][4] = {};
+      const bool near = p.bias && ctx - (j0 + KT) < p.span;
       scores16<DK>(s[0], s[1], qf, kb, warp * 16);
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
-          const int j = j0 + warp * 16 + i * 8 + (lane & 3) * 2 + (x & 1);
+          const int j = j0 + warp * 16 + i * 8 + (lane & 3) * 2 + (x & 1), hr = (lane >> 2) + 8 * (x >> 1);
           s[i][x] = j < jend ? score_log2(p, s[i][x], sl2) : -INFINITY;
+          if (near && j < jend && ctx - 1 - j < p.span && hr < nh) s[i][x] += LOG2E_F * p.bias[(long long)(g * rep + h0 + hr) * p.span + ctx - 1 - j];
           mx[x >> 1] = fmaxf(mx[x >> 1], s[i][x]);
         }
 #pragma unroll
@@ -474,7 +492,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const PagedParams p, i
       gl = with_sink(p, h, gm, gl);
       float f = gl > 0.f ? 1.f / gl : 0.f;
       if (p.gate) f *= p.gate[(long long)b * p.H + h];
-      reinterpret_cast<bf16*>(p.out)[(long long)b * p.o_ld + (long long)h * p.vdim + c] = __float2bfloat16(a * f);
+      reinterpret_cast<bf16*>(p.out)[(long long)b * p.o_ld + (long long)h * p.vdim + c] = __float2bfloat16(a * f * gate_at<bf16>(p, b, h, c));
     } else {
       const long long idx = ((long long)b * p.H + h) * splits + split;
       part_o[idx * p.vdim + c] = a;
@@ -507,7 +525,7 @@ __global__ void __launch_bounds__(128) attn_combine_kernel(const PagedParams p, 
       const float ms = part_ml[(base + s) * 2];
       if (ms != -INFINITY) a += part_o[(base + s) * p.vdim + c] * ex2(ms - gm);
     }
-    reinterpret_cast<bf16*>(p.out)[(long long)b * p.o_ld + (long long)h * p.vdim + c] = __float2bfloat16(a * f);
+    reinterpret_cast<bf16*>(p.out)[(long long)b * p.o_ld + (long long)h * p.vdim + c] = __float2bfloat16(a * f * gate_at<bf16>(p, b, h, c));
   }
 }
 
@@ -573,13 +591,14 @@ int launch_decode(const PagedParams& p, int splits, float* ws, cudaStream_t st) 
 // rows of decode sequences (row s = sequence s < nd) and of prompts (sequence nd + i: rows nd + cu[i] ... nd + cu[i+1]).
 DLTI_API int dlti_attn_rows(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd, const int* tables,
                             int max_blocks, int bs, const int* ctx, const int* rseq, const int* pos, int H, int G, int dim, int vdim,
-                            int chunk, int window, float scale, float cap, const float* gate, const float* sink, void* out, long long o_ld, long long rows, int dtype,
+                            int chunk, int window, float scale, float cap, const float* gate, const float* sink, const float* bias, int span,
+                            const void* ogate, long long og_ld, void* out, long long o_ld, long long rows, int dtype,
                             cudaStream_t st) {
   if (rows <= 0) return 0;
   if (H % G || dim < 1 || vdim < 1 || (chunk > 0 && window > 0)) return DLTI_ERR_BAD_ARG;
   if (dim > 2048 || vdim > 1024) { dlti_set_error("attn_rows: queries of up to 2048 and values of up to 1024 dimensions"); return DLTI_ERR_TOO_LARGE; }
   PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, nullptr, rseq, pos, 0, H, G, dim, vdim, chunk, window, scale, cap,
-                gate, out, o_ld, rows, sink};
+                gate, out, o_ld, rows, sink, bias, span, ogate, og_ld};
   if (dtype == DLTI_BF16) return launch_rows<__nv_bfloat16>(p, st);
   if (dtype == DLTI_FP32) return launch_rows<float>(p, st);
   return DLTI_ERR_UNSUPPORTED;
@@ -595,25 +614,26 @@ static int check_mma(int H, int G, int dim, int vdim, int kd, int vd, int q_hd) 
 // the rows themselves must be in the pages already.
 DLTI_API int dlti_attn_paged_prefill(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
                                      const int* tables, int max_blocks, int bs, const int* ctx, const int* cu, int nd, int nseq,
-                                     int max_rows, int H, int G, int dim, int vdim, int chunk, int window, float scale, float cap, const float* gate, const float* sink, void* out,
-                                     long long o_ld, cudaStream_t st) {
+                                     int max_rows, int H, int G, int dim, int vdim, int chunk, int window, float scale, float cap, const float* gate, const float* sink, const float* bias, int span,
+                                     const void* ogate, long long og_ld, void* out, long long o_ld, cudaStream_t st) {
   if (nseq <= 0 || max_rows <= 0) return 0;
   if (int rc = check_mma(H, G, dim, vdim, kd, vd, q_hd)) return rc;
   if (q_ld % 2 || nseq > 65535) return DLTI_ERR_BAD_ARG;
   PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, cu, nullptr, nullptr, nd, H, G, dim, vdim, chunk, window, scale, cap,
-                gate, out, o_ld, 0, sink};
+                gate, out, o_ld, 0, sink, bias, span, ogate, og_ld};
   HEAD_DISPATCH(kd, vd, launch_prefill, p, nseq, max_rows, st);
 }
 
 // bf16. Row b = the newest token of sequence b, whose context is ctx[b] tokens. ws: batch * H * splits * (vdim + 2) floats.
 DLTI_API int dlti_attn_paged_decode(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
                                     const int* tables, int max_blocks, int bs, const int* ctx, int batch, int H, int G, int dim, int vdim,
-                                    int chunk, int window, float scale, float cap, const float* gate, const float* sink, int splits, float* ws, void* out, long long o_ld,
+                                    int chunk, int window, float scale, float cap, const float* gate, const float* sink, const float* bias, int span,
+                                    const void* ogate, long long og_ld, int splits, float* ws, void* out, long long o_ld,
                                     cudaStream_t st) {
   if (batch <= 0) return 0;
   if (int rc = check_mma(H, G, dim, vdim, kd, vd, q_hd)) return rc;
   if (q_ld % 2 || splits < 1 || batch > 65535) return DLTI_ERR_BAD_ARG;
   PagedParams p{q, q_ld, q_hd, kc, vc, kd, vd, tables, max_blocks, bs, ctx, nullptr, nullptr, nullptr, 0, H, G, dim, vdim, chunk, window, scale, cap,
-                gate, out, o_ld, batch, sink};
+                gate, out, o_ld, batch, sink, bias, span, ogate, og_ld};
   HEAD_DISPATCH(kd, vd, launch_decode, p, splits, ws, st);
 }

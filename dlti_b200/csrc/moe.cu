@@ -1,7 +1,8 @@
 // Mixtures of experts and gated activations.
 //
-//   moe_route        one warp per token: sigmoid scores, groups, the top experts and their weights; every (token, choice) pair
-//                    = token * top + choice is appended to its expert's list. Further blocks of the same launch apply a gated
+//   moe_route        one warp per token: sigmoid scores, groups, the top experts and their weights (or the top logits and their
+//                    softmax); every (token, choice) pair
+//                    = token * top + choice is appended to its expert's list. Further blocks of the same launch apply an
 //                    activation to other columns of the same projection (the shared expert).
 //   moe_gemm         grouped GEMM over the lists, bf16, by CTA pairs: weights are the 256-row operand of tcgen05.mma and the
 //                    pairs of a list its columns (32 to 256 of them), so one kernel serves one decoded token and whole
@@ -33,8 +34,10 @@ struct RouteParams {
   const float* z; long long z_ld; int col;                 // router logits at column col of fp32 rows
   const float* corr;
   int E, top, groups, keep; float scale;
+  int softmax;                                             // logits + corr decide, weights = their softmax among the chosen
+  int sg; float* share;                                    // share[t] = sigmoid of column sg (sg < 0: none)
   float* wgt; int *lists, *counts;                         // [T, top]; [E, T]; [E]
-  const void* p; long long p_ld; int og, ou, ff; float limit;      // projection columns of the activation (ff 0: none)
+  const void* p; long long p_ld; int og, ou, ff; float limit;      // projection columns of the activation (ff 0: none; og < 0: square of relu)
   void* h; long long h_ld;
   long long T;
 };
@@ -59,9 +62,14 @@ __device__ __forceinline__ void route_token(const RouteParams& p, long long t, f
     if (e < p.E) {
       const float v = zr[e];
       if (ACC) const_cast<float*>(zr)[e] = 0.f;
-      s[i] = sigmoid_f(v);
-      c[i] = s[i] + p.corr[e];
+      s[i] = p.softmax ? v + p.corr[e] : sigmoid_f(v);
+      c[i] = p.softmax ? s[i] : s[i] + p.corr[e];
     }
+  }
+  if (p.sg >= 0 && lane == 0) {
+    float* zs = const_cast<float*>(p.z) + t * p.z_ld + p.sg;
+    p.share[t] = sigmoid_f(*zs);
+    if (ACC) *zs = 0.f;
   }
   if (p.keep < p.groups) {
     __syncwarp();
@@ -90,7 +98,7 @@ __device__ __forceinline__ void route_token(const RouteParams& p, long long t, f
       }
     }
   }
-  float sum = 0.f;
+  float sum = 0.f, largest = 0.f;
   for (int k = 0; k < p.top; ++k) {
     unsigned best = 0;
     int bi = p.E;
@@ -104,6 +112,10 @@ __device__ __forceinline__ void route_token(const RouteParams& p, long long t, f
     int e = (int)__reduce_min_sync(0xffffffffu, best == top && bi < p.E ? (unsigned)bi : 0x7fffffffu);
     if (e >= p.E) e = k;                                   // only where the scores are not numbers
     bs = __shfl_sync(0xffffffffu, bi == e ? bs : 0.f, e & 31);
+    if (p.softmax) {
+      if (k == 0) largest = bs;
+      bs = expf(bs - largest);
+    }
     if ((e & 31) == lane)
 #pragma unroll
       for (int i = 0; i < R; ++i)
@@ -164,7 +176,18 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) moe_route_kernel(const Route
     const int c = (int)(i - t * per) * W;
     const void* row = reinterpret_cast<const uint8_t*>(p.p) + t * p.p_ld * (ACC ? 4 : sizeof(T));
     T* o = reinterpret_cast<T*>(p.h) + t * p.h_ld + c;
-    if constexpr (W == 1) {
+    if (p.og < 0) {
+      float u[W];
+      if constexpr (W == 1) u[0] = take<T, ACC>(row, p.ou + c);
+      else take_n<T, ACC, W>(row, p.ou + c, u);
+#pragma unroll
+      for (int j = 0; j < W; ++j) {
+        u[j] = fmaxf(u[j], 0.f);
+        u[j] *= u[j];
+      }
+      if constexpr (W == 1) *o = Cvt<T>::from_f(u[0]);
+      else put_n(o, u);
+    } else if constexpr (W == 1) {
       const float g = take<T, ACC>(row, p.og + c), u = take<T, ACC>(row, p.ou + c);
       *o = Cvt<T>::from_f(gated(g, u, p.limit));
     } else {
@@ -188,8 +211,9 @@ struct MoeGemmParams {
   int x_rows, o_rows;                                      // list entries outside these are not followed (counters of an aborted step)
   int NT, MT, stages;                                      // columns of a tile (multiple of 32, at most 256), weight tiles of an expert
 };
-// UP: the source of list entry i is row lists[i] / div, its result (activation of rows 2 r and 2 r + 1) goes to row (start of the
-// list) + i. Otherwise the source is row (start of the list) + i and the result goes to row lists[i].
+// UP: the source of list entry i is row lists[i] / div, its result goes to row (start of the list) + i (MOE_SWIGLU: activation of
+// rows 2 r and 2 r + 1, MOE_RELU2: of row r). Otherwise the source is row (start of the list) + i and the result goes to row lists[i].
+enum MoeMode : int { MOE_DOWN = 0, MOE_SWIGLU = 1, MOE_RELU2 = 2 };
 constexpr int MG_GATHERS = 8, MG_THREADS = 320 + 32 * MG_GATHERS, MG_A_BYTES = 16384, MG_MAX_STAGES = 10, MG_SMEM = 226 * 1024;
 constexpr int MG_TAIL = 8 * (3 * MG_MAX_STAGES + 4) + 16;  // barriers, TMEM address
 constexpr long long MG_WAIT_LIMIT = 4000000000LL;
@@ -222,9 +246,10 @@ __device__ __forceinline__ MoeTile moe_tile(const MoeGemmParams& p, const int* f
 // 128 rows of the accumulator (two of them, so that the epilogue overlaps the next tile). Warp 0: weights; warp 1: MMAs; warps 2-9:
 // epilogue; warps 10-17: the gathered columns, four rows a copy (a copy costs its issuing thread about 100 clk, so they share them),
 // or warp 10 where they lie together. Waits are bounded: a CTA that gives up writes NaN.
-template <bool UP>
+template <int MODE>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(MG_THREADS, 1)
 moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, const __grid_constant__ CUtensorMap tx) {
+  constexpr bool UP = MODE != MOE_DOWN;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   const uint32_t stage_bytes = MG_A_BYTES + p.NT * 64;
@@ -399,7 +424,7 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
           const int i = c + j + (lane & 7), to = dst[i & 255];      // stale past the tile's columns
           B* out = reinterpret_cast<B*>(p.out) + (long long)to * p.o_ld;
           const bool on = i < x.nn && (unsigned)to < (unsigned)p.o_rows;
-          if constexpr (UP) {                              // even lanes hold gates, odd lanes up values
+          if constexpr (MODE == MOE_SWIGLU) {              // even lanes hold gates, odd lanes up values
             float f[4];
 #pragma unroll
             for (int y = 0; y < 4; ++y) {
@@ -418,7 +443,12 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
             uint32_t u[4];
 #pragma unroll
             for (int y = 0; y < 4; ++y) {
-              const float v0 = __uint_as_float(v[j + 2 * y]), v1 = __uint_as_float(v[j + 2 * y + 1]), other = swap_f(b0, v0, v1, 1);
+              float v0 = __uint_as_float(v[j + 2 * y]), v1 = __uint_as_float(v[j + 2 * y + 1]);
+              if constexpr (MODE == MOE_RELU2) {           // what is not a number stays so
+                v0 = v0 < 0.f ? 0.f : v0 * v0;
+                v1 = v1 < 0.f ? 0.f : v1 * v1;
+              }
+              const float other = swap_f(b0, v0, v1, 1);
               u[y] = b0 ? Cvt<B>::pack2(other, v1) : Cvt<B>::pack2(v0, other);
             }
             uint2 w[2];
@@ -474,9 +504,10 @@ moe_gemm_kernel(const MoeGemmParams p, const __grid_constant__ CUtensorMap tw, c
 }
 
 // CTA = (64 outputs, expert), 16 pairs at a time; thread = one output of 4 pairs
-template <bool UP>
+template <int MODE>
 __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restrict__ X, long long x_ld, const float* __restrict__ Wt, long long w_ld,
                                                            const MoeGemmParams p) {
+  constexpr bool UP = MODE != MOE_DOWN;
   __shared__ float sw[2][16][65], sx[16][17];
   __shared__ int s_src[16], s_to[16], s_start;
   const int e = blockIdx.y, r0 = blockIdx.x * 64, cnt = max(0, min(p.counts[e], p.cap));
@@ -488,7 +519,7 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restri
     if (threadIdx.x == 0) s_start = before;
   }
   const int r = threadIdx.x & 63, tg = threadIdx.x >> 6;
-  constexpr int parts = UP ? 2 : 1;
+  constexpr int parts = MODE == MOE_SWIGLU ? 2 : 1;
   for (int n0 = 0; n0 < cnt; n0 += 16) {
     __syncthreads();
     if (threadIdx.x < 16) {
@@ -501,7 +532,7 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restri
     for (int k0 = 0; k0 < p.K; k0 += 16) {
       for (int i = threadIdx.x; i < parts * 64 * 16; i += 256) {
         const int q = i / (64 * 16), rr = (i / 16) % 64, k = i % 16;
-        sw[q][k][rr] = (r0 + rr < p.rows && k0 + k < p.K) ? Wt[((long long)e * p.wrows + (UP ? 2 * (r0 + rr) + q : r0 + rr)) * w_ld + k0 + k] : 0.f;
+        sw[q][k][rr] = (r0 + rr < p.rows && k0 + k < p.K) ? Wt[((long long)e * p.wrows + (MODE == MOE_SWIGLU ? 2 * (r0 + rr) + q : r0 + rr)) * w_ld + k0 + k] : 0.f;
       }
       {
         const int i = threadIdx.x, tt = i / 16, k = i % 16;
@@ -524,8 +555,11 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restri
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int i = tg * 4 + j;
+      float v = acc[0][j];
+      if (MODE == MOE_SWIGLU) v = gated(v, acc[1][j], p.limit);
+      if (MODE == MOE_RELU2) v = v < 0.f ? 0.f : v * v;
       if (n0 + i < cnt && r0 + r < p.rows && (unsigned)s_to[i] < (unsigned)p.o_rows)
-        reinterpret_cast<float*>(p.out)[(long long)s_to[i] * p.o_ld + r0 + r] = UP ? gated(acc[0][j], acc[1][j], p.limit) : acc[0][j];
+        reinterpret_cast<float*>(p.out)[(long long)s_to[i] * p.o_ld + r0 + r] = v;
     }
   }
 }
@@ -548,18 +582,18 @@ int launch_route(const RouteParams& p, cudaStream_t st) {
 
 // experts 0: no routing; ff 0: no activation. acc: z and p are the decode GEMM's accumulator (zero on return in the columns read).
 DLTI_API int dlti_moe_route(const float* z, long long z_ld, int col, const float* corr, int E, int top, int groups, int keep, float scale,
-                            float* wgt, int* lists, int* counts, const void* p, long long p_ld, int og, int ou, int ff, float limit, void* h,
+                            int softmax, float* wgt, int* lists, int* counts, int sg, float* share, const void* p, long long p_ld, int og, int ou, int ff, float limit, void* h,
                             long long h_ld, long long T, int acc, int dtype, cudaStream_t st) {
   if (T <= 0) return 0;
   if (E && (!z || !corr || !wgt || !lists || !counts || groups < 1 || E % groups || keep < 1 || keep > groups || top < 1 || top > E / groups * keep))
     return DLTI_ERR_BAD_ARG;
   if (E > 1024 || T * (top > 1 ? top : 1) > 0x7fffffffLL) { dlti_set_error("moe_route: up to 1024 experts"); return DLTI_ERR_TOO_LARGE; }
-  if (ff && (!p || !h)) return DLTI_ERR_BAD_ARG;
+  if ((ff && (!p || !h)) || (softmax && groups > 1) || (sg >= 0 && (!E || !share))) return DLTI_ERR_BAD_ARG;
   if (!E && !ff) return 0;
-  const RouteParams r{z, z_ld, col, corr, E, top, groups, keep, scale, wgt, lists, counts, p, p_ld, og, ou, ff, limit, h, h_ld, T};
+  const RouteParams r{z, z_ld, col, corr, E, top, groups, keep, scale, softmax, sg, share, wgt, lists, counts, p, p_ld, og, ou, ff, limit, h, h_ld, T};
   using B = __nv_bfloat16;
   if (dtype == DLTI_BF16) {
-    const bool vec = ((ff | og | ou) & 7) == 0 && ((p_ld | h_ld) & 7) == 0 && ((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(h)) & 15) == 0;
+    const bool vec = ((ff | (og < 0 ? 0 : og) | ou) & 7) == 0 && ((p_ld | h_ld) & 7) == 0 && ((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(h)) & 15) == 0;
     if (vec) return acc ? launch_route<B, true, 8>(r, st) : launch_route<B, false, 8>(r, st);
     return acc ? launch_route<B, true, 1>(r, st) : launch_route<B, false, 1>(r, st);
   }
@@ -568,16 +602,16 @@ DLTI_API int dlti_moe_route(const float* z, long long z_ld, int col, const float
 }
 
 // The pairs lists[e, 0 .. counts[e]) of every expert; W_e = rows e * wrows ... of W, cap = capacity of a list.
-// up: rows X[pair / div] times W_e, whose rows 2 r and 2 r + 1 are gate and up of output r; out = clipped activation, one list after the
-// other. Otherwise: rows of X in that order times W_e, result to out[pair]. X: x_rows rows, out: o_rows rows of `rows` columns.
+// up: rows X[pair / div] times W_e; out = their activation, one list after the other (1: rows 2 r and 2 r + 1 are gate and up of output r,
+// clipped; 2: square of relu). Otherwise: rows of X in that order times W_e, result to out[pair]. X: x_rows rows, out: o_rows rows of `rows` columns.
 DLTI_API int dlti_moe_gemm(const void* X, long long x_ld, long long x_rows, int div, const void* Wt, long long w_ld, int wrows, int E,
                            const int* lists, const int* counts, int cap, int rows, int up, int K, float limit, void* out, long long o_ld,
                            int o_rows, int dtype, cudaStream_t st) {
   if (o_rows <= 0 || E <= 0) return 0;
-  if (x_rows < 1 || x_rows > 0x7fffffffLL || rows < 1 || K < 1 || div < 1 || rows * (up ? 2 : 1) > wrows) return DLTI_ERR_BAD_ARG;
+  if (x_rows < 1 || x_rows > 0x7fffffffLL || rows < 1 || K < 1 || div < 1 || up < 0 || up > 2 || rows * (up == MOE_SWIGLU ? 2 : 1) > wrows) return DLTI_ERR_BAD_ARG;
   MoeGemmParams p{lists, counts, E, cap, div, rows, wrows, K, limit, out, o_ld, (int)x_rows, o_rows, 0, 0, 0};
   if (dtype == DLTI_FP32) {
-    (up ? moe_gemm_f32_kernel<true> : moe_gemm_f32_kernel<false>)<<<dim3((rows + 63) / 64, E), 256, 0, st>>>((const float*)X, x_ld, (const float*)Wt,
+    (up == MOE_SWIGLU ? moe_gemm_f32_kernel<MOE_SWIGLU> : up ? moe_gemm_f32_kernel<MOE_RELU2> : moe_gemm_f32_kernel<MOE_DOWN>)<<<dim3((rows + 63) / 64, E), 256, 0, st>>>((const float*)X, x_ld, (const float*)Wt,
                                                                                                            w_ld, p);
     dlti_count_launch();
     return (int)cudaGetLastError();
@@ -587,7 +621,7 @@ DLTI_API int dlti_moe_gemm(const void* X, long long x_ld, long long x_rows, int 
   if (o_ld % 8 || o_ld < rows || x_ld % 8 || ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(out)) & 15)) return DLTI_ERR_BAD_ARG;
   const long long avg = (o_rows + E - 1) / E;              // pairs of an expert, were they spread evenly
   p.NT = avg > 96 ? 256 : avg > 40 ? 128 : avg > 12 ? 64 : 32;
-  p.MT = (rows * (up ? 2 : 1) + 255) / 256;
+  p.MT = (rows * (up == MOE_SWIGLU ? 2 : 1) + 255) / 256;
   const int stage = MG_A_BYTES + p.NT * 64, tail = MG_TAIL + 2048 + 3 * E * 4;
   p.stages = (MG_SMEM - 1024 - tail) / stage;
   if (p.stages > MG_MAX_STAGES) p.stages = MG_MAX_STAGES;
@@ -596,18 +630,18 @@ DLTI_API int dlti_moe_gemm(const void* X, long long x_ld, long long x_rows, int 
   int rc;
   if ((rc = dlti_get_tmap(&tw, Wt, K, (uint64_t)E * wrows, w_ld, 64, 128))) return rc;
   if ((rc = dlti_get_tmap(&tx, X, K, x_rows, x_ld, 64, up ? 1 : p.NT / 2))) return rc;
-  static bool done[64] = {};
+  auto kern = up == MOE_SWIGLU ? moe_gemm_kernel<MOE_SWIGLU> : up ? moe_gemm_kernel<MOE_RELU2> : moe_gemm_kernel<MOE_DOWN>;
+  static bool done[64][3] = {};
   int dev = 0;
   DLTI_CUDA_CHECK(cudaGetDevice(&dev));
-  if (!done[dev & 63]) {
-    DLTI_CUDA_CHECK(cudaFuncSetAttribute(moe_gemm_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, MG_SMEM));
-    DLTI_CUDA_CHECK(cudaFuncSetAttribute(moe_gemm_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, MG_SMEM));
-    done[dev & 63] = true;
+  if (!done[dev & 63][up]) {
+    DLTI_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, MG_SMEM));
+    done[dev & 63][up] = true;
   }
   // at most one tile per pair and weight tile
   const long long most = (long long)p.MT * (E < o_rows ? E + (o_rows - E) / p.NT + 1 : o_rows);
   const int clusters = dlti_num_sms() / 2;
-  DLTI_CUDA_CHECK(dlti_launch_pdl(cap, up ? moe_gemm_kernel<true> : moe_gemm_kernel<false>, dim3(2 * (most < clusters ? (unsigned)most : clusters)),
+  DLTI_CUDA_CHECK(dlti_launch_pdl(cap, kern, dim3(2 * (most < clusters ? (unsigned)most : clusters)),
                                   dim3(MG_THREADS), (size_t)smem, st, p, tw, tx));
   dlti_count_launch();
   return 0;

@@ -23,14 +23,16 @@ __global__ void embed_rows_kernel(const long long* __restrict__ ids, const T* __
   }
 }
 
-// out = scale * acc (fp32), acc = 0
-__global__ void take_rows_kernel(float* __restrict__ acc, float* __restrict__ out, float scale, long long vec) {
+// out = scale * acc (fp32), with cap > 0: cap * tanh(scale * acc / cap); clear: acc = 0 (otherwise out may be acc)
+__global__ void take_rows_kernel(float* acc, float* out, float scale, float cap, int clear, long long vec) {
   griddep_wait();
   griddep_launch();
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < vec; i += (long long)gridDim.x * blockDim.x) {
-    const float4 v = reinterpret_cast<float4*>(acc)[i];
-    reinterpret_cast<float4*>(out)[i] = make_float4(scale * v.x, scale * v.y, scale * v.z, scale * v.w);
-    reinterpret_cast<float4*>(acc)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 v = reinterpret_cast<float4*>(acc)[i];
+    if (clear) reinterpret_cast<float4*>(acc)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    v = make_float4(scale * v.x, scale * v.y, scale * v.z, scale * v.w);
+    if (cap > 0.f) v = make_float4(cap * tanhf(v.x / cap), cap * tanhf(v.y / cap), cap * tanhf(v.z / cap), cap * tanhf(v.w / cap));
+    reinterpret_cast<float4*>(out)[i] = v;
   }
 }
 
@@ -989,12 +991,13 @@ DLTI_API int dlti_embed_rows(const long long* ids, const void* table, float* x, 
   return 0;
 }
 
-// the decode GEMM's accumulator [rows, cols] times scale as an fp32 result (cols a multiple of 4); zero on return
-DLTI_API int dlti_take_rows(float* acc, float* out, float scale, long long rows, int cols, cudaStream_t st) {
+// [rows, cols] times scale as an fp32 result (cols a multiple of 4), softly capped with cap > 0. clear: acc is the decode GEMM's
+// accumulator, zero on return; otherwise out may be acc.
+DLTI_API int dlti_take_rows(float* acc, float* out, float scale, float cap, int clear, long long rows, int cols, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (cols % 4) return DLTI_ERR_BAD_ARG;
+  if (cols % 4 || cap < 0.f || (clear && acc == out)) return DLTI_ERR_BAD_ARG;
   const long long vec = rows * (cols / 4);
-  DLTI_CUDA_CHECK(dlti_launch_pdl(rows, take_rows_kernel, dim3(grid_for(vec, 256)), dim3(256), 0, st, acc, out, scale, vec));
+  DLTI_CUDA_CHECK(dlti_launch_pdl(rows, take_rows_kernel, dim3(grid_for(vec, 256)), dim3(256), 0, st, acc, out, scale, cap, clear, vec));
   dlti_count_launch();
   return 0;
 }

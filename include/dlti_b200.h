@@ -348,8 +348,8 @@ int dlti_sample(const void* logits, long long ld, int batch, int V, const float*
                 unsigned long long step, long long* out, float* out_logprob, int dtype,
                 dlti_stream_t stream);
 
-/* ---- Layer-stack models (models/stack.py): csrc/stack.cu, streams.cu, recurrent.cu, attention_paged.cu, latent.cu, dyt.cu, moe.cu, delta.cu,
- * gemm_f32.cu. Row pitches (*_ld) in
+/* ---- Layer-stack models (models/stack.py): csrc/stack.cu, streams.cu, recurrent.cu, attention_paged.cu, latent.cu, dyt.cu, prenorm.cu,
+ * conv_qkv.cu, moe.cu, delta.cu, gemm_f32.cu. Row pitches (*_ld) in
  * elements. Sequences of a step: the first nd are single rows, sequence nd + i has rows nd + cu[i] ... nd + cu[i+1]; ctx[s] = tokens
  * of sequence s after the step, rseq[t] = sequence of row t, sslot[s] = its state slot (-1 = none). */
 /* C[M,N] = A[M,K] * B[N,K]^T in true fp32 (no TF32) */
@@ -358,8 +358,8 @@ int dlti_gemm_f32(const float* A, const float* B, float* C, int M, int N, int K,
 /* x[t] = table[ids[t]] as fp32; xa (16-bit, may be NULL) = the same rows */
 int dlti_embed_rows(const long long* ids, const void* table, float* x, void* xa, long long xa_ld, long long tokens, int
     d, long long vocab, int dtype, dlti_stream_t stream);
-/* out = scale * acc, acc = 0 (fp32 logits of the decode GEMM) */
-int dlti_take_rows(float* acc, float* out, float scale, long long rows, int cols, dlti_stream_t stream);
+/* out = scale * acc, cap > 0: cap * tanh(scale * acc / cap) (fp32 logits); clear: acc = 0, else out may be acc */
+int dlti_take_rows(float* acc, float* out, float scale, float cap, int clear, long long rows, int cols, dlti_stream_t stream);
 /* x += RMSnorm(y) * w (1 + w with one_plus), fp32 residual x [rows,d]; xa (may be NULL) = x in dtype.
  * acc: y is the fp32 accumulator of dlti_gemm_skinny, zero on return (also below) */
 int dlti_post_norm_add(const void* y, long long y_ld, float* x, const float* w, void* xa, long long xa_ld, long long
@@ -415,24 +415,27 @@ int dlti_linear_scan_chunked(const void* q, long long q_ld, const void* k, long 
 int dlti_silu_rows(void* x, long long ld, long long rows, int n, int dtype, dlti_stream_t stream);
 /* paged attention, one warp per (row, head), fp32 arithmetic; chunk > 0: a position sees its own chunk only; window > 0: itself and the
  * window - 1 positions before it; cap > 0: scores become cap tanh(score / cap). sink [H] (may be NULL): one more term exp(sink) in a head's
- * softmax denominator (all also below) */
+ * softmax denominator; bias [H, span] (may be NULL): added to the scores at the distances below span; ogate [rows, H * vdim] (may be NULL):
+ * outputs are multiplied by its sigmoid (all also below) */
 int dlti_attn_rows(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd, const int*
     tables, int max_blocks, int bs, const int* ctx, const int* rseq, const int* pos, int H, int G, int dim, int vdim,
-    int chunk, int window, float scale, float cap, const float* gate, const float* sink, void* out, long long o_ld, long long rows, int dtype,
+    int chunk, int window, float scale, float cap, const float* gate, const float* sink, const float* bias, int span, const void* ogate,
+    long long og_ld, void* out, long long o_ld, long long rows, int dtype,
     dlti_stream_t stream);
 /* paged attention of prompt portions (bf16, heads <= 256) */
 int dlti_attn_paged_prefill(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
     const int* tables, int max_blocks, int bs, const int* ctx, const int* cu, int nd, int nseq, int max_rows, int H,
-    int G, int dim, int vdim, int chunk, int window, float scale, float cap, const float* gate, const float* sink, void* out, long long o_ld, dlti_stream_t
-    stream);
+    int G, int dim, int vdim, int chunk, int window, float scale, float cap, const float* gate, const float* sink, const float* bias, int span,
+    const void* ogate, long long og_ld, void* out, long long o_ld, dlti_stream_t stream);
 /* paged attention of decode rows (bf16, grouped heads, split over CTAs); ws: batch * H * splits * (vdim + 2) floats */
 int dlti_attn_paged_decode(const void* q, long long q_ld, int q_hd, const void* kc, const void* vc, int kd, int vd,
     const int* tables, int max_blocks, int bs, const int* ctx, int batch, int H, int G, int dim, int vdim, int chunk,
-    int window, float scale, float cap, const float* gate, const float* sink, int splits, float* ws, void* out, long long o_ld, dlti_stream_t stream);
+    int window, float scale, float cap, const float* gate, const float* sink, const float* bias, int span, const void* ogate, long long
+    og_ld, int splits, float* ws, void* out, long long o_ld, dlti_stream_t stream);
 /* varlen causal attention with the softmax weights as two bf16 terms; see attention.cu */
 int dlti_attn_fwd_split(const void* qkv, void* out, long long ldo, const float* gate, const float* sink, const int* cu_seqlens, const int*
     seq_q0, const int* seq_out0, int batch, int max_seqlen, long long T_total, int H, int KV, int vdim, int window,
-    float scale, float cap, dlti_stream_t stream);
+    float scale, float cap, const float* bias, int span, const void* ogate, long long og_ld, dlti_stream_t stream);
 
 /* mLSTM: the recurrence above with exponential gates, a running maximum and a normaliser; see recurrent.cu. gates [rows, >= 2 heads]
  * raw fp32 (input, forget), vec [slots, heads, ceil(P / 32), N + 1] */
@@ -481,14 +484,31 @@ int dlti_tanh_between(float* x, const void* y, long long y_ld, const void* rows,
 /* h[i] = n(x[idx[i]]); idx NULL = all rows */
 int dlti_tanh_rows(const float* x, const long long* idx, const float* alpha, const float* w, const float* b, void* h, long long h_ld, long
     long rows, int d, int dtype, dlti_stream_t stream);
-/* moe.cu: routing of the logits z (E > 0): sigmoid scores, groups, the top experts by score + corr, their scores made to sum to scale ->
+/* prenorm.cu: x (zero if fresh) += mult * (y * share[t] + sum_k weights[t, k] rows[t * top + k]), with post: mult * RMSnorm(that) * post; x +=
+ * scale * table[ids[t]]; h = RMSnorm(x) * pre (pre NULL: x). All but x may be NULL; counts are cleared */
+int dlti_prenorm_between(float* x, const void* y, long long y_ld, const void* rows, long long r_ld, const float* weights, int top, const float*
+    share, int* counts, int ncounts, float mult, const float* post, const long long* ids, const void* table, long long vocab, float scale, int
+    fresh, const float* pre, void* h, long long h_ld, long long tokens, int d, float eps, int acc, int dtype, dlti_stream_t stream);
+/* h[t, c] = gelu_tanh(u[t, c]) * table[ids[t], col + c], c < n */
+int dlti_token_gate(const void* u, long long u_ld, const long long* ids, const void* table, long long t_ld, long long vocab, int col, int n,
+    void* h, long long h_ld, long long tokens, int acc, int dtype, dlti_stream_t stream);
+/* conv_qkv.cu: projection rows -> causal convolution (w tap-major by column, NULL: none; state [slots, taps - 1, C] is read and renewed), per-head
+ * RMS norms of q and k, q times factors[pos[t]]; k and v into the paged cache at slots[t]; kp, vp, dst as in dlti_qk_norm_rope_cache. acc: also
+ * gate = columns from og on */
+int dlti_conv_qkv(const void* proj, long long ld, int oq, int ok, int ov, int og, const float* w, int taps, int w_ld, void* state, int C, const
+    int* sslot, const int* rseq, const int* ctx, const int* cu, int nd, int nseq, const float* qn, const float* kn, float eps, const float* factors,
+    const int* pos, const long long* slots, void* kc, void* vc, int kd, int vd, void* q, long long q_ld, int q_hd, void* kp, void* vp, const int*
+    dst, void* gate, long long g_ld, long long tokens, int H, int G, int dim, int vdim, int acc, int dtype, dlti_stream_t stream);
+/* moe.cu: routing of the logits z (E > 0): sigmoid scores, groups, the top experts by score + corr, their scores made to sum to scale
+ * (softmax: the top experts by logit + corr, scale times their softmax); share (sg >= 0) = sigmoid of column sg;
  * wgt [T, top] and, per expert, the list of its pairs token * top + choice (lists [E, T], counts [E] zero on entry); and / or (ff > 0)
- * the gated activation of projection columns og (gate) and ou (up): silu(g) u, with a limit g sigmoid(1.702 g) (u + 1) of clipped values */
-int dlti_moe_route(const float* z, long long z_ld, int col, const float* corr, int E, int top, int groups, int keep, float scale, float* wgt,
-    int* lists, int* counts, const void* p, long long p_ld, int og, int ou, int ff, float limit, void* h, long long h_ld, long long T, int acc,
+ * the gated activation of projection columns og (gate) and ou (up): silu(g) u, with a limit g sigmoid(1.702 g) (u + 1) of clipped values;
+ * og < 0: square of relu(u) */
+int dlti_moe_route(const float* z, long long z_ld, int col, const float* corr, int E, int top, int groups, int keep, float scale, int softmax,
+    float* wgt, int* lists, int* counts, int sg, float* share, const void* p, long long p_ld, int og, int ou, int ff, float limit, void* h, long long h_ld, long long T, int acc,
     int dtype, dlti_stream_t stream);
-/* grouped GEMM over the lists. up: rows X[pair / div] times gate / up rows 2 r, 2 r + 1 of W_e, out = activation, one list after the other;
- * else rows of X in that order times W_e, out[pair]. W_e = rows e * wrows ... of W */
+/* grouped GEMM over the lists. up: rows X[pair / div] times W_e, out = activation, one list after the other (1: of gate / up rows 2 r, 2 r + 1,
+ * 2: square of relu of row r); else rows of X in that order times W_e, out[pair]. W_e = rows e * wrows ... of W */
 int dlti_moe_gemm(const void* X, long long x_ld, long long x_rows, int div, const void* W, long long w_ld, int wrows, int E, const int* lists,
     const int* counts, int cap, int rows, int up, int K, float limit, void* out, long long o_ld, int o_rows, int dtype, dlti_stream_t stream);
 /* delta.cu: gated delta rule S <- g S, u = b (v - S^T k), S <- S + k u^T, o = S^T q over sequences [seq0, seq0+nseq); gates [rows, >= 2
