@@ -55,11 +55,11 @@ def parse():
     ap.add_argument("--offload", action="store_true",
                     help="run the ds_config as shipped (ZeRO-Offload of optimizer state and parameters to pinned host "
                          "memory) instead of the HBM-resident default; a secondary measurement, not the headline (689 ms vs 631 ms per step on one B200)")
-    ap.add_argument("--workload", default="train", choices=["train", "sigosun", "logozen", "latanex"],
+    ap.add_argument("--workload", default="train", choices=["train", "sigosun", "logozen", "latanex", "ridazen"],
                     help="train: the headline benchmark (default). sigosun: prefill and decode throughput of the Sigosun family "
                          "beside Llama models of equal size, with every kernel's fraction of its roofline (1 GPU). logozen "
-                         "and latanex: those families beside Sigosun models of equal size")
-    ap.add_argument("--sizes", default="2048x4,4096x2", help="--workload sigosun, logozen, latanex: width x groups of four Sigosun layers, comma-separated")
+                         "and latanex: those families beside Sigosun models of equal size. ridazen: beside Latanex models of equal size")
+    ap.add_argument("--sizes", default="2048x4,4096x2", help="--workload sigosun, logozen, latanex, ridazen: width x groups of four Sigosun layers, comma-separated")
     return ap.parse_args()
 
 

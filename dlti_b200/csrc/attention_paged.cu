@@ -236,7 +236,7 @@ __device__ __forceinline__ void weighted16(float (&o)[DV / 8][4], const float (&
 }
 
 constexpr int PF_ROWS = 128;                       // (token, head) rows of a prefill CTA
-template <int DK, int DV>
+template <int DK, int DV, bool EXTRA>              // EXTRA: biases by distance and / or gates on output elements
 __global__ void __launch_bounds__(256) attn_prefill_kernel(const PagedParams p) {
   using L = Tile<DK, DV>;
   extern __shared__ __align__(128) uint8_t smem[];
@@ -309,16 +309,30 @@ __global__ void __launch_bounds__(256) attn_prefill_kernel(const PagedParams p) 
 #pragma unroll
     for (int i = 0; i < KT / 16; ++i) scores16<DK>(s[2 * i], s[2 * i + 1], qf, kb, i * 16);
     float mx[2] = {-INFINITY, -INFINITY};
-    const bool near = p.bias && start + (int)(wr0 / rep) - (j0 + KT - 1) < p.span;
 #pragma unroll
     for (int i = 0; i < KT / 8; ++i)
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         const int j = j0 + i * 8 + (lane & 3) * 2 + (x & 1), y = x >> 1;
         s[i][x] = (j <= pos[y] && j >= jlo[y]) ? score_log2(p, s[i][x], sl2) : -INFINITY;
-        if (near && j <= pos[y] && pos[y] - j < p.span) s[i][x] += LOG2E_F * p.bias[(long long)head[y] * p.span + pos[y] - j];
-        mx[y] = fmaxf(mx[y], s[i][x]);
+        if (!EXTRA) mx[y] = fmaxf(mx[y], s[i][x]);
       }
+    if constexpr (EXTRA) {
+      if (p.bias && start + (int)(wr0 / rep) - (j0 + KT - 1) < p.span) {
+        const float* tab[2] = {p.bias + (long long)head[0] * p.span, p.bias + (long long)head[1] * p.span};
+#pragma unroll
+        for (int i = 0; i < KT / 8; ++i)
+#pragma unroll
+          for (int x = 0; x < 4; ++x) {
+            const int n = pos[x >> 1] - (j0 + i * 8 + (lane & 3) * 2 + (x & 1));
+            if ((unsigned)n < (unsigned)p.span) s[i][x] = fmaf(LOG2E_F, tab[x >> 1][n], s[i][x]);
+          }
+      }
+#pragma unroll
+      for (int i = 0; i < KT / 8; ++i)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) mx[x >> 1] = fmaxf(mx[x >> 1], s[i][x]);
+    }
     float base[2];
 #pragma unroll
     for (int y = 0; y < 2; ++y) {
@@ -357,7 +371,7 @@ __global__ void __launch_bounds__(256) attn_prefill_kernel(const PagedParams p) 
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i) {
       const int c = i * 8 + (lane & 3) * 2;
-      if (p.ogate) {
+      if (EXTRA && p.ogate) {
         if (c < p.vdim) o[i][2 * y] *= gate_at<bf16>(p, row[y], head[y], c);
         if (c + 1 < p.vdim) o[i][2 * y + 1] *= gate_at<bf16>(p, row[y], head[y], c + 1);
       }
@@ -542,11 +556,13 @@ int allow_smem(K kernel, int bytes, bool* done) {
 
 template <int DK, int DV>
 int launch_prefill(const PagedParams& p, int nseq, int max_rows, cudaStream_t st) {
-  static bool done[64] = {};
+  static bool done[2][64] = {};
   const int smem = 2 * Tile<DK, DV>::BYTES;
-  if (int rc = allow_smem(attn_prefill_kernel<DK, DV>, smem, done)) return rc;
+  const bool extra = p.bias || p.ogate;
+  auto kern = extra ? attn_prefill_kernel<DK, DV, true> : attn_prefill_kernel<DK, DV, false>;
+  if (int rc = allow_smem(kern, smem, done[extra])) return rc;
   const long long tiles = ((long long)max_rows * (p.H / p.G) + PF_ROWS - 1) / PF_ROWS;
-  attn_prefill_kernel<DK, DV><<<dim3((unsigned)tiles, p.G, nseq), 256, smem, st>>>(p);
+  kern<<<dim3((unsigned)tiles, p.G, nseq), 256, smem, st>>>(p);
   dlti_count_launch();
   return (int)cudaGetLastError();
 }

@@ -190,7 +190,7 @@ int between(const Between& p, long long tokens, cudaStream_t st) {
   }
   if constexpr (sizeof(T) == 2) {
     if (((p.d | p.y_ld | p.r_ld | p.h_ld) & 7) == 0 && aligned16({p.x, p.y, p.rows, p.post, p.table, p.pre, p.h})) {
-      PB_CASE(8, 1, 128) PB_CASE(8, 1, 256) PB_CASE(8, 2, 256) PB_CASE(8, 4, 256)
+      PB_CASE(8, 1, 128) PB_CASE(8, 1, 256) PB_CASE(8, 1, 512) PB_CASE(8, 2, 512)
     }
   }
   PB_CASE(1, 1, 256) PB_CASE(1, 4, 256) PB_CASE(1, 16, 256) PB_CASE(1, 32, 512)

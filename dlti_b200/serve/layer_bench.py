@@ -1,7 +1,7 @@
 """Serving throughput of a layer-stack family beside the closest other family at equal size, and the time of each kernel of
 the two against its roofline: Sigosun beside Llama (`bench.py --workload sigosun`), Logozen and Latanex beside Sigosun
-(`--workload logozen`, `--workload latanex`). Random weights; layer sizes of real models. A mixture of experts counts with
-the parameters that a token uses.
+(`--workload logozen`, `--workload latanex`), Ridazen beside Latanex (`--workload ridazen`). Random weights; layer sizes of real models. A mixture of experts counts with
+the parameters that a token uses, a layer that runs several times with those of every run.
 
 Steps go through LLMEngine.pack_step / _run_step (packing, host-to-device copy, forward, sampling; decode steps replay
 CUDA graphs), timed with CUDA events. Kernels are timed one call at a time with the L2 overwritten before each."""
@@ -17,9 +17,10 @@ from ..models.config import LlamaConfig
 from ..models.registry import family_of
 from ..models.latanex import LatanexConfig
 from ..models.logozen import LogozenConfig
+from ..models.ridazen import RidazenConfig
 from ..models.sigosun import SigosunConfig
-from ..models.stack import (AttentionMixer, DeltaMixer, DenseMlp, LatentAttentionMixer, Layer, LightningMixer, Mamba2Mixer, MLstmMixer, MoeMlp,
-                            Rope, StackWeights, mixer_sections, mlp_sections, round8)
+from ..models.stack import (AttentionMixer, DeltaMixer, DenseMlp, DistanceBias, LatentAttentionMixer, Layer, LightningMixer, Loop, Mamba2Mixer,
+                            MLstmMixer, MoeMlp, QueryTemp, Rope, StackWeights, mixer_sections, mlp_sections, round8)
 from ..ops import _lib
 from ..ops import attention as A
 from ..ops import delta as DR
@@ -27,6 +28,7 @@ from ..ops import dyt as TN
 from ..ops import elementwise as E
 from ..ops import latent as LA
 from ..ops import moe as ME
+from ..ops import prenorm as PN
 from ..ops import serving as S
 from ..ops import stack as K
 from ..ops import streams as HS
@@ -78,10 +80,31 @@ def _latanex(width: int, params: int) -> LatanexConfig:
     return cfg(max(1, round(params / one)))
 
 
+def _ridazen(width: int, params: int) -> RidazenConfig:
+    """Attention layers with mixtures of experts, the second and third of them run twice; a token uses about `params` parameters."""
+    heads = width // 128
+    att = AttentionMixer(heads=heads, kv_heads=max(1, heads // 4), dim=128, vdim=128, scale=128 ** -0.5, head_gate=False, conv=4,
+                         q_temp=QueryTemp(0.1, 1024), bias_by=DistanceBias(32, 128), out_gate=True)
+    moe = MoeMlp(experts=64, top=8, ff=width // 4, act="relu2", score="softmax", shared_ff=width // 2, shared_gate=True)
+
+    def cfg(n):
+        return RidazenConfig(hidden_size=width, vocab_size=32000, norm_eps=1e-6, norm_one_plus=False, pre_norm=True, residual_mult=0.7, token_side=128,
+                             loop=Loop(1, 3, 2), logit_scale=0.5, logit_softcap=30.0, layers=[Layer(att, moe)] * n, name=f"ridazen-{width}x{n}")
+    one = active_params(cfg(5)) - active_params(cfg(4))
+    return cfg(max(4, 4 + round((params - active_params(cfg(4)) + 2 * 32000 * width) / one)))
+
+
 def active_params(cfg) -> int:
-    """Parameters that one token uses."""
-    idle = [(e.experts - e.top) * 3 * e.ff * cfg.hidden_size for l in getattr(cfg, "layers", []) if isinstance(e := l.mlp, MoeMlp)]
-    return cfg.num_params() - sum(idle)
+    """Parameters that one token uses, those of a layer once per run."""
+    layers = getattr(cfg, "layers", [])
+    idle = [(e.experts - e.top) * (3 if e.gated else 2) * e.ff * cfg.hidden_size if isinstance(e := l.mlp, MoeMlp) else 0 for l in layers]
+    n = cfg.num_params() - sum(idle)
+    if layers and (cfg.loop is not None or cfg.token_side):
+        w = StackWeights(cfg, "meta", torch.bfloat16)
+        n -= 0 if w.side_embed is None else w.side_embed.numel() - w.side_embed.shape[1]
+        own = [sum(t.numel() for t in lw.values()) - x for lw, x in zip(w.layers, idle)]
+        n += sum(own[j] for j in cfg.runs) - sum(own)
+    return n
 
 
 def experts_hit(e: MoeMlp, rows: int) -> float:
@@ -152,13 +175,15 @@ def step_bytes(eng: LLMEngine, batch: int, ctx: int) -> int:
     written."""
     cfg, w = eng.cfg, eng.w
     size = lambda t: t.numel() * t.element_size()
-    n = sum(size(t) for l in w.layers for t in l.values()) + size(w.lm_head)
+    runs = cfg.runs if eng.per_sequence else range(len(w.layers))
+    n = sum(size(t) for j in runs for t in w.layers[j].values()) + size(w.lm_head)
     if not eng.per_sequence:
         return n + 2 * 2 * cfg.num_hidden_layers * batch * (ctx + 1) * w.KV * cfg.head_dim
-    for i, l in enumerate(cfg.layers):
+    for i, j in enumerate(runs):
+        l = cfg.layers[j]
         m = l.mixer
         if isinstance(l.mlp, MoeMlp):
-            n -= int((1 - experts_hit(l.mlp, batch) / l.mlp.experts) * (size(w.layers[i]["e_up"]) + size(w.layers[i]["e_down"])))
+            n -= int((1 - experts_hit(l.mlp, batch) / l.mlp.experts) * (size(w.layers[j]["e_up"]) + size(w.layers[j]["e_down"])))
         if eng.states is not None and eng.states.canon[i] is not None:
             n += 2 * batch * size(eng.states.canon[i][:, 0])
         if isinstance(m, LatentAttentionMixer):
@@ -166,6 +191,8 @@ def step_bytes(eng: LLMEngine, batch: int, ctx: int) -> int:
         elif isinstance(m, AttentionMixer):
             seen = ctx + 1 - (ctx // m.chunk * m.chunk if m.chunk else max(0, ctx + 1 - m.window) if m.window else 0)
             n += 2 * batch * seen * m.kv_heads * (m.dim + m.vdim)
+            if m.conv > 1:
+                n += 2 * 2 * batch * eng.states.conv[i][0].numel()
         else:
             n += 2 * batch * 4 * (eng.states.ssm[i][0].numel() + (0 if eng.states.vec[i] is None else eng.states.vec[i][0].numel()))
     return n
@@ -522,9 +549,100 @@ def latanex_kernels(width: int, peaks: dict, nseq: int, length: int, batch: int,
     return k.rows
 
 
+def ridazen_kernels(width: int, peaks: dict, nseq: int, length: int, batch: int, ctx: int, iters: int) -> list[dict]:
+    """The kernels of Ridazen in the same two steps; those of Latanex come from latanex_kernels()."""
+    k = _Kernels(peaks, iters)
+    cfg = _ridazen(width, 1)
+    m, e, d, dev, bf, side = cfg.layers[0].mixer, cfg.layers[0].mlp, width, "cuda", torch.bfloat16, cfg.token_side
+    w = StackWeights(replace(cfg, layers=cfg.layers[:1], loop=None), dev, bf)
+    lw = w.layers[0]
+    lw["rel"].normal_()
+    bias = w.finish().derived[0]["bias"]
+    rnd = lambda *s: torch.randn(*s, device=dev, dtype=bf)
+    for n in ("w_in", "w_up", "e_up", "e_down", "w_down", "side_gate", "side_proj"):
+        lw[n].normal_(0, d ** -0.5)
+    T, bs, H, G, hd = nseq * length, 16, m.heads, m.kv_heads, 128
+    per = -(-max(length, ctx + 1) // bs)
+    n_all = max(nseq, batch)
+    tabs = torch.arange(n_all * per, dtype=torch.int32, device=dev).view(n_all, per)
+    kc, vc = rnd(n_all * per, bs, G, hd), rnd(n_all * per, bs, G, hd)
+    pslots = torch.cat([torch.arange(length) + i * per * bs for i in range(nseq)]).to(dev)
+    dslots = torch.tensor([i * per * bs + ctx for i in range(batch)], device=dev)
+    pr = _rows([(0, length)] * nseq, 0, tabs[:nseq].contiguous(), pslots, length)
+    dr = _rows([(ctx, 1)] * batch, batch, tabs[:batch].contiguous(), dslots, ctx + 1)
+    pieces = K.Pieces(torch.tensor([i * length for i in range(nseq + 1)], dtype=torch.int32, device=dev), length, T)
+    run = lambda phase, name, fn, nbytes, flops=0.0: k.run("ridazen", phase, name, fn, nbytes, flops)
+    pairs = length * (length + 1) // 2
+    sec, su = mixer_sections(m), mlp_sections(e)
+    qkv, out, proj = rnd(T, (H + 2 * G) * hd), K.act(T, H * hd, bf, dev), rnd(T, sec.total)
+    more = dict(bias=bias, out_gate=proj[:, sec["g"]:sec["g"] + H * hd])
+    io, fl = T * (3 * H + 2 * G) * hd * 2, 4.0 * nseq * pairs * H * hd
+    run("prefill", "attention (packed)", lambda: K.packed_attention(qkv, m, pr, pieces, kc, vc, None, **more), io, fl)
+    q = rnd(T, H * hd)
+    run("prefill", "attention (paged, heads > 128)", lambda: K.attn_paged_prefill(q, m, pr, kc, vc, None, out, **more), io, fl)
+    qd, od, gd = rnd(batch, H * hd), K.act(batch, H * hd, bf, dev), rnd(batch, H * hd)
+    run("decode", "attention", lambda: K.attn_paged_decode(qd, m, dr, kc, vc, None, od, bias=bias, out_gate=gd), batch * (ctx + 1) * G * hd * 4)
+    del qkv, out, q, proj
+    factors = K.temp_table(max(length, ctx + 1), m.q_temp, dev)
+    pre, post = torch.ones(d, device=dev), torch.ones(d, device=dev)
+    for phase, r, n, ns in (("prefill", pr, T, nseq), ("decode", dr, batch, batch)):
+        acc = phase == "decode"
+        es = 8 if acc else 2                                      # accumulators are read and zeroed
+        z = lambda c: torch.zeros(n, c, device=dev) if acc else rnd(n, c)
+        proj, state = z(sec.total), torch.zeros(ns, m.conv - 1, sec["g"], device=dev, dtype=bf)
+        cols = sec.total if acc else sec["g"]                     # prompts leave the gates to the attention kernel
+        run(phase, "conv + head norms + cache", lambda: K.conv_qkv(proj, sec, m, lw, factors, 1e-6, r, state, kc, vc, bf, None if acc else pieces, acc),
+            n * (cols * es + (H + (H if acc else 2 * G)) * hd * 2 + 2 * G * hd * 2) + ns * state[0].numel() * 4)
+        x, y, rows_, wt = torch.randn(n, d, device=dev), z(d), rnd(n * e.top, d), torch.rand(n, e.top, device=dev)
+        run(phase, "residual + norm", lambda: PN.between_(x, y, pre, 1e-6, bf, mult=0.7, acc=acc), n * d * (es + 8 + 2))
+        run(phase, "norm + residual + norm", lambda: PN.between_(x, y, pre, 1e-6, bf, mult=0.7, post=post, acc=acc), n * d * (es + 8 + 2))
+        ex = ME.ExpertSum(rows_, wt, y, share=wt[:, 0].contiguous())
+        run(phase, "sum of experts + residual", lambda: PN.between_(x, ex, None, 1e-6, bf, mult=0.7, copy=True, acc=acc),
+            n * d * (es + 8 + 2 + 2 * e.top))
+        del rows_, ex
+        h, logits = rnd(n, d), torch.randn(n, round8(e.experts) + 8, device=dev)
+        counts, share = ME._counts(torch.device(dev, torch.cuda.current_device()), e.experts), torch.empty(n, device=dev)
+
+        def route():
+            counts.zero_()
+            return ME._route(None, logits, 0, lw["correction"], e, share=(round8(e.experts), share))
+        run(phase, "routing (and clearing its counters)", route, n * (e.experts * 4 + e.top * 8))
+        wgt, lists, cnt = route()
+        cnt = cnt.clone()
+        counts.zero_()                                            # as the next step wants them
+        hit = int((cnt > 0).sum())
+        a, rows_ = K.act(n * e.top, e.ff, bf, dev), K.act(n * e.top, d, bf, dev)
+        run(phase, "experts in + activation", lambda: ME.grouped_gemm(h, lw["e_up"], lists, cnt, a, rows=e.ff, pairs_per_row=e.top, up=True, act=e.act),
+            2 * (n * d + hit * e.ff * d + n * e.top * e.ff), 2.0 * n * e.top * e.ff * d)
+        run(phase, "experts out", lambda: ME.grouped_gemm(a, lw["e_down"], lists, cnt, rows_, rows=d, pairs_per_row=1),
+            2 * (n * e.top * (e.ff + d) + hit * e.ff * d), 2.0 * n * e.top * e.ff * d)
+        del a, rows_
+        ids, emb = torch.randint(0, 1000, (n,), device=dev), rnd(1000, side)
+        u, hs = z(round8(side)), rnd(n, side)
+        run(phase, "token input gate", lambda: PN.token_gate(u, ids, emb, 0, side, bf, acc=acc), n * side * (es + 4))
+        if acc:
+            p, hu = z(su.total), K.act(n, e.shared_ff, bf, dev)
+            run(phase, "relu^2 (shared expert)", lambda: ME._route(p, None, 0, None, None, (-1, su["up"], e.shared_ff, 0.0, hu), acc=True),
+                n * e.shared_ff * (es + 2))
+        else:
+            run(phase, "GEMM shared expert in + relu^2", lambda: gemm_relu2(h, lw["w_up"][:su["router"]], e.shared_ff),
+                2 * (n * d + su["router"] * d + n * e.shared_ff), 2.0 * n * su["router"] * d)
+            run(phase, "GEMM router", lambda: K.linear(h, lw["w_up"][su["router"]:], out_dtype=torch.float32),
+                2 * (n * d + (su.total - su["router"]) * d) + 4 * n * (su.total - su["router"]), 2.0 * n * (su.total - su["router"]) * d)
+        for name, a, wm in (("GEMM attention in", h, lw["w_in"]), ("GEMM token input in", h, lw["side_gate"]), ("GEMM token input out", hs, lw["side_proj"]),
+                            *((("GEMM shared expert, router", h, lw["w_up"]),) if acc else ())):
+            N_, K_ = wm.shape
+            mm = gemm_skinny_acc if acc else gemm
+            run(phase, name, lambda: mm(a, wm), 2 * (n * K_ + N_ * K_) + n * N_ * (4 if acc else 2), 2.0 * n * N_ * K_)
+            if acc:
+                gemm_skinny(a, wm)                                # leaves the shared accumulator zero
+    return k.rows
+
+
 def main(steps: int, warmup: int, sizes: str, peaks: dict, sampler, workload: str = "sigosun") -> dict:
     iters, warmup = max(3, steps), max(3, warmup)
-    name, other = {"logozen": ("Logozen", "Sigosun"), "latanex": ("Latanex", "Sigosun")}.get(workload, ("Sigosun", "Llama"))
+    name, other = {"logozen": ("Logozen", "Sigosun"), "latanex": ("Latanex", "Sigosun"),
+                   "ridazen": ("Ridazen", "Latanex")}.get(workload, ("Sigosun", "Llama"))
     out = {"metric": f"{name} serving tok/s beside {other} of equal size", "impl": "dlti_b200", "dtype": "bf16",
            "data": "synthetic (random token ids; random-init weights)", "steps": iters, "warmup": warmup, "sizes": [], "kernels": {}}
     _lib.reset_launch_count()
@@ -533,6 +651,7 @@ def main(steps: int, warmup: int, sizes: str, peaks: dict, sampler, workload: st
         sig = _sigosun(width, blocks)
         params = sig.num_params() - 2 * sig.vocab_size * width
         models = {"logozen": lambda: (_logozen(width, params), sig), "latanex": lambda: (_latanex(width, params), sig),
+                  "ridazen": lambda: (_ridazen(width, params), _latanex(width, params)),
                   "sigosun": lambda: (sig, _llama(width, params))}[workload]()
         row = {"width": width, "rows": []}
         for cfg in models:
@@ -549,10 +668,11 @@ def main(steps: int, warmup: int, sizes: str, peaks: dict, sampler, workload: st
             del eng
             torch.cuda.empty_cache()
         out["sizes"].append(row)
-        ks = kernels(width, peaks, 4, 2048, 64, 1000, iters)
-        if workload != "sigosun":
-            own = logozen_kernels if workload == "logozen" else latanex_kernels
-            ks = own(width, peaks, 4, 2048, 64, 1000, iters) + [r for r in ks if r["model"] == "sigosun"]
+        own = {"sigosun": kernels, "logozen": logozen_kernels, "latanex": latanex_kernels, "ridazen": ridazen_kernels}
+        beside = {"sigosun": [], "ridazen": ["latanex"]}.get(workload, ["sigosun"])
+        ks = own[workload](width, peaks, 4, 2048, 64, 1000, iters)
+        for b in beside:
+            ks += [r for r in own[b](width, peaks, 4, 2048, 64, 1000, iters) if r["model"] == b]
         out["kernels"][str(width)] = ks
         torch.cuda.empty_cache()
     out["gpu_launches"] = _lib.launch_count()

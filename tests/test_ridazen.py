@@ -249,7 +249,7 @@ def _packs(device, dtype, dim, vdim):
 
 
 SHAPES = [(6, 3, 14, 10), (8, 2, 64, 64), (4, 4, 128, 128), (3, 3, 40, 72), (2, 1, 256, 256), (20, 1, 33, 8), (2, 1, 264, 40), (4, 1, 64, 128)]
-KINDS = [(3, (0.4, 17), (12, 70)), (4, (0.2, 50), (32, 128)), (1, (0.25, 1), (2, 2)), (2, None, (64, 40)), (0, (0.3, 64), None), (6, None, (16, 300)),
+KINDS = [(3, (0.4, 17), (12, 70)), (4, (0.2, 50), (32, 128)), (1, (0.1, 1), (2, 2)), (2, None, (64, 40)), (0, (0.3, 64), None), (6, None, (16, 300)),
          (0, None, None)]
 
 
@@ -262,7 +262,8 @@ def test_attention_over_portions(device, dtype, shape, taps, temp, bias):
         c = AttentionCase(device, dtype, shape, taps, temp, bias, [170, 75, 20, 33])
         for parts in ({0: 64, 1: 2, 2: 16}, {0: 1, 1: 15, 3: 31}, {2: 1, 0: 65, 1: 1}, {3: 2, 0: 1, 1: 1, 2: 1}, {0: 2, 1: 55}, {0: 1, 1: 1, 2: 1}, {0: 36}):
             c.step(parts, packed)
-        c.check(tol(dtype, 1e-5, 1.5e-2))
+        # one tap alone makes heavy-tailed heads: sharper scores
+        c.check(tol(dtype, 1e-5, 2.5e-2 if taps == 1 else 1.5e-2))
 
 
 @pytest.mark.gpu
