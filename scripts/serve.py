@@ -77,7 +77,7 @@ def make_engine(a, info, cfg, w, tp, tok):
 
 def add_args(ap):
     ap.add_argument("--model", type=str, default=None, help="checkpoint directory (Hugging Face Llama, or another family of models/registry.py) or preset name")
-    ap.add_argument("--model_config", type=str, default=None, help="preset: tiny | llama2-7b | llama2-70b | sigosun-1b | logozen-1b | latanex-3b | ...")
+    ap.add_argument("--model_config", type=str, default=None, help="preset: tiny | llama2-7b | llama2-70b | sigosun-1b | logozen-1b | latanex-3b | ridazen-3b | ...")
     ap.add_argument("--adapter", type=str, default=None, help="PEFT LoRA adapter directory served on top of the base")
     ap.add_argument("--merge_adapter", action="store_true",
                     help="fold the adapter into the base weights at load time (W' = W + alpha/r B A) instead of "
